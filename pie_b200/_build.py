@@ -19,11 +19,15 @@ import sys
 import sysconfig
 from concurrent.futures import ThreadPoolExecutor
 from pathlib import Path
+from typing import Optional, Sequence
 
 ROOT = Path(__file__).resolve().parent
 CSRC = ROOT / "csrc"
 OUT = ROOT / "_C"
 KERNEL_LIB = OUT / "libpie_kernels.so"
+
+# sources whose kernels a latent-attention model launches
+LATENT_SOURCES = ("attention_tc", "elementwise", "gemm2_tcgen05", "gemm_tcgen05", "latent", "sampling")
 
 NVCC_FLAGS = [
     "-gencode", "arch=compute_100a,code=sm_100a", "-lineinfo", "-O3", "-std=c++17",
@@ -53,12 +57,13 @@ def _run(cmd, log_name: str) -> None:
         raise RuntimeError(f"build step failed: {' '.join(map(str, cmd))}\n{proc.stdout}\n{proc.stderr}")
 
 
-def build_kernels(verbose: bool = False, ptxas_info: bool = False) -> Path:
-    """Compile csrc/kernels/*.cu for sm_100a and link libpie_kernels.so."""
+def build_kernels(verbose: bool = False, ptxas_info: bool = False, only: Optional[Sequence[str]] = None,
+                  target: Path = KERNEL_LIB) -> Path:
+    """Compile csrc/kernels/*.cu (or just the sources named in `only`) for sm_100a and link `target`."""
     OUT.mkdir(exist_ok=True)
     kdir = CSRC / "kernels"
     headers = list(kdir.glob("*.cuh")) + list(kdir.glob("*.h"))
-    sources = sorted(kdir.glob("*.cu"))
+    sources = sorted(kdir.glob("*.cu")) if only is None else [kdir / f"{stem}.cu" for stem in only]
     objs = []
     jobs = []
     for src in sources:
@@ -74,12 +79,23 @@ def build_kernels(verbose: bool = False, ptxas_info: bool = False) -> Path:
             print(f"[pie_b200] compiling {len(jobs)} CUDA source(s) for sm_100a", file=sys.stderr)
         with ThreadPoolExecutor(max_workers=min(8, len(jobs))) as ex:
             list(ex.map(lambda j: _run(*j), jobs))
-    if jobs or _newer(objs, KERNEL_LIB):
+    if jobs or _newer(objs, target):
         # link beside the target and rename: a reader (or a snapshot of the tree) never sees a half-written library
-        tmp = KERNEL_LIB.with_suffix(".so.tmp")
+        tmp = target.with_suffix(".so.tmp")
         _run([_nvcc(), "-shared", "-o", str(tmp), *map(str, objs), "-Xcompiler", "-fPIC"], "link_kernels")
-        os.replace(tmp, KERNEL_LIB)
-    return KERNEL_LIB
+        os.replace(tmp, target)
+    return target
+
+
+def kernels_for(cfg) -> Path:
+    """A kernel library that can run models of configuration `cfg`, compiling what is missing. The whole library is
+    taken when it is up to date; otherwise a family with a source list of its own gets a library of just those."""
+    kdir = CSRC / "kernels"
+    if not _newer([*kdir.glob("*.cu"), *kdir.glob("*.cuh")], KERNEL_LIB):
+        return KERNEL_LIB
+    if cfg.latent is not None:
+        return build_kernels(only=LATENT_SOURCES, target=OUT / "libpie_kernels_latent.so")
+    return build_kernels()
 
 
 def host_module_path() -> Path:

@@ -139,7 +139,8 @@ class TorchDriver:
                  page_size: int = 16, max_requests: int = 512, max_tokens: int = 8192, seed: int = 0,
                  par: Optional[ParallelContext] = None, gemm_backend: str = "tcgen05", use_graphs: bool = True,
                  swap_pages: int = 0, gpu_mem_utilization: float = 0.9, max_kv_tokens_per_request: int = 0,
-                 memory_profile: str = "", kv_dtype: str = "auto", rs_slots: int = 0, vision=None, audio=None):
+                 memory_profile: str = "", kv_dtype: str = "auto", rs_slots: int = 0, vision=None, audio=None,
+                 compute_dtype: str = "auto"):
         self.cfg = cfg
         self.device = torch.device(device)
         if self.device.type == "cuda" and self.device.index is None:
@@ -148,7 +149,15 @@ class TorchDriver:
         self._bound = threading.local()
         self.adapters: dict = {}
         self._lora_bindings = None
+        # the kernels compute in bf16 with 32-bit accumulation; compute_dtype "float32" runs a latent-attention model in
+        # true 32-bit throughout (weights, activations, cache), for verification
         self.dtype = torch_dtype(cfg.dtype) if not self.cuda else torch.bfloat16
+        if compute_dtype != "auto":
+            if self.cuda and compute_dtype == "float32" and cfg.latent is None:
+                raise NotImplementedError(f"32-bit kernels for model type {cfg.model_type}")
+            self.dtype = torch_dtype(compute_dtype)
+        if cfg.latent is not None and kv_dtype == "fp8_e4m3":
+            raise NotImplementedError("fp8 pages for latent rows")
         self.par = par or ParallelContext()
         if self.cuda:
             torch.cuda.set_device(self.device)
@@ -170,14 +179,15 @@ class TorchDriver:
                     t = torch.tensor([num_pages], dtype=torch.int64, device=self.device)
                     dist.all_reduce(t, op=dist.ReduceOp.MIN)
                     num_pages = int(t.item())
-        self.kv = KVCache(cfg.num_hidden_layers, num_pages, hkv, page_size, cfg.head_dim, self.dtype,
-                          self.device, swap_pages, kv_dtype=kv_dtype)
+        self.kv = KVCache(len(cfg.latent_cache_layers) if cfg.latent is not None else cfg.num_hidden_layers, num_pages, hkv,
+                          page_size, cfg.head_dim, self.dtype, self.device, swap_pages, kv_dtype=kv_dtype,
+                          latent=cfg.latent is not None)
         self.model.kv_scale = self.kv.scale
-        # Gated DeltaNet layers keep their state in slots of a recurrent-state cache, one per resident context
+        # Gated DeltaNet, Mamba-2 and token-shifted layers keep their state in slots of a recurrent-state cache, one per resident context
         self.rs = None
         if cfg.recurrent_layers:
             if self.par.tp_size > 1:
-                raise NotImplementedError("recurrent (Gated DeltaNet / Mamba-2) layers under tensor parallelism")
+                raise NotImplementedError("recurrent-state layers under tensor parallelism")
             from .recurrent import RecurrentStateCache
             self.rs = RecurrentStateCache(cfg, rs_slots or max(2 * max_requests, 16), self.device)
         # media: a vision encoder (models.vision.VisionEncoder) and the clips it has encoded, by the runtime's slot
@@ -200,7 +210,8 @@ class TorchDriver:
         import os as _os
         self._prefix_cache: dict = {}
         self.cascade = (self.cuda and _os.environ.get("PIE_CASCADE", "1") != "0" and self.window_left < 0
-                        and self.cfg.layer_types is None and self.kv.scale is None and not self.softcap)
+                        and self.cfg.layer_types is None and self.kv.scale is None and not self.softcap
+                        and self.cfg.latent is None)
         rows = max(max_requests, 1024)
         self.max_rows = rows
         self.slab = _Slab({
@@ -265,6 +276,8 @@ class TorchDriver:
     # ------------------------------------------------------------------ adapters
     def create_adapter(self, adapter_id: int, rank: int, alpha: float, seed: int = 0) -> None:
         from .lora import LoraAdapter
+        if self.cfg.latent is not None:
+            raise NotImplementedError("LoRA adapters on latent attention")
         if self.par.tp_size > 1:
             raise NotImplementedError("LoRA adapters are served by single-GPU replicas")
         self.adapters[adapter_id] = LoraAdapter(self.cfg, rank, alpha, self.device, self.dtype, self.model.hq,
@@ -410,7 +423,7 @@ class TorchDriver:
             page_indices=s.d("page_indices"), kv_page_indptr=s.d("kv_page_indptr"), item_req=s.d("item_req"),
             item_start=s.d("item_start"), item_end=s.d("item_end"), req_item_indptr=s.d("req_item_indptr"),
             num_items=s.d("num_items"), scratch=self.scratch, max_items=self.max_items, num_reqs=rb,
-            num_ctas=self.num_ctas, page_size=self.page_size, window_left=self.window_left)
+            num_ctas=self.num_ctas, page_size=self.page_size, window_left=self.window_left, kv_lens=s.d("kv_lens"))
         if cascade:
             plan.item_slot, plan.item_tile, plan.tile_members = s.d("item_slot"), s.d("item_tile"), s.d("tile_members")
         return ForwardInputs(tokens=s.d("tokens", rb), positions=s.d("positions", rb), slots=s.d("slots", rb),
@@ -424,11 +437,11 @@ class TorchDriver:
         if rb not in cache:
             from .recurrent import RecurrentInputs
             s, dev = self.slab, self.device
-            scratch = torch.empty(rb, self.rs.conv_channels, dtype=torch.float32, device=dev) if self.cuda else None
             cache[rb] = RecurrentInputs(
                 torch.arange(rb + 1, dtype=torch.int32, device=dev), torch.arange(rb, dtype=torch.int32, device=dev),
                 s.d("rs_slots", rb), s.d("rs_reset", rb), list(range(rb + 1)), [-1] * rb, [0] * rb,
-                self.rs.conv_state, self.rs.rec_state, self.rs.layer_index, scratch)
+                self.rs.conv_state, self.rs.rec_state, self.rs.layer_index, shift_state=self.rs.shift_state,
+                **self.rs.device_scratch(rb, rb))
         return cache[rb]
 
     def _fill_rs_decode(self, req: ForwardRequest, r: int, rb: int) -> None:
@@ -602,9 +615,8 @@ class TorchDriver:
         rows = rows.astype(np.int32)
         self.stats["logit_rows"] = self.stats.get("logit_rows", 0) + len(rows)
         if self.cuda:
-            group = self.model.hq // self.model.hkv
-            tile_rows = ops.prefill_tile_rows(self.model.hq, self.model.hkv, self.model.cfg.head_dim, self.page_size,
-                                              softcap=self.softcap)
+            group = self.model.prefill_group
+            tile_rows = self.model.prefill_tile_rows(self.page_size)
             tile_req, tile_q = ops.plan_prefill_tiles(np.asarray(req.qo_indptr), group, tile_rows, kv_lens)
             nt = len(tile_req)
             s.h("tile_req")[:nt], s.h("tile_qstart")[:nt] = tile_req, tile_q
@@ -760,6 +772,12 @@ class TorchDriver:
                 s.d("min_p", k).view(torch.float32), s.d("seeds", k, torch.int64), mask_bits, mask_row)
         if self.model.sharded_logits:
             return self.par.comm.sample_sharded(lg, *args, out=out)
+        if lg.dtype != torch.bfloat16:
+            # 32-bit logits: the sampler reads bf16, an unmasked greedy row takes the exact arg-max
+            drawn = ops.sample(lg.to(torch.bfloat16), *args)
+            greedy = args[0] <= 0 if mask_row is None else (args[0] <= 0) & (mask_row < 0)
+            out[:k].copy_(torch.where(greedy, lg.argmax(-1).to(torch.int32), drawn))
+            return out
         return ops.sample(lg, *args, out=out)
 
     def _logit_mask_rows(self, req, token_slots):
@@ -997,6 +1015,8 @@ class TorchDriver:
             s.h("slots")[r:rb] = -1
             s.h("kv_page_indptr")[r + 1:rb + 1] = req.kv_page_indptr[-1]
         cascade = self._plan_decode(kv_lens, np.asarray(req.kv_page_indptr), np.asarray(req.kv_page_indices), r, rb)
+        if self.rs is not None:
+            self._fill_rs_decode(req, r, rb)
         o, n = s.offsets["tile_qstart"]
         end = o + n
         po, _ = s.offsets["page_indices"]

@@ -19,12 +19,15 @@ from .schema import CopyDir, CopyRequest
 
 class KVCache:
     def __init__(self, layers: int, num_pages: int, kv_heads: int, page_size: int, head_dim: int,
-                 dtype, device, swap_pages: int = 0, kv_dtype: str = "auto"):
+                 dtype, device, swap_pages: int = 0, kv_dtype: str = "auto", latent: bool = False):
         """kv_dtype "auto": pages in the activation dtype. "fp8_e4m3": one byte per element plus one
         fp32 scale per (token, KV head) row in `scale` [layers, pages + 1, 2, kv_heads, page_size]
         (written by the RoPE + KV-write kernel, read by decode attention; prefill attention works on
         pages expanded to bf16 for the batch). Counterpart of the reference's per-token-head fp8 format
-        (driver/cuda/src/kv_cache_format.hpp, kernels/kv_paged.cu:188-325)."""
+        (driver/cuda/src/kv_cache_format.hpp, kernels/kv_paged.cu:188-325).
+
+        `latent`: pages of latent attention, one row of `head_dim` elements per token (latent, then the rotated key part
+        that all heads share) in ``[layers, pages + 1, page_size, row]``; `layers` counts the layers that write rows."""
         if page_size % 16:
             raise ValueError("kv page size must be a multiple of 16")
         if kv_dtype not in ("auto", "bf16", "fp8_e4m3"):
@@ -39,20 +42,20 @@ class KVCache:
         self.layers, self.num_pages, self.kv_heads = layers, num_pages, kv_heads
         self.page_size, self.head_dim, self.dtype = page_size, head_dim, dtype
         self.device = torch.device(device)
+        self.page_shape = (page_size, head_dim) if latent else (2, kv_heads, page_size, head_dim)
         # zero-filled: unwritten slots are multiplied by p == 0 in attention and must be finite
-        self.data = torch.zeros(layers, num_pages + 1, 2, kv_heads, page_size, head_dim, dtype=dtype,
-                                device=self.device)
+        self.data = torch.zeros(layers, num_pages + 1, *self.page_shape, dtype=dtype, device=self.device)
         self.pad_page = num_pages
         self.swap_pages = swap_pages
         self.host = None
         if swap_pages > 0:
-            self.host = torch.zeros(layers, swap_pages, 2, kv_heads, page_size, head_dim, dtype=dtype,
+            self.host = torch.zeros(layers, swap_pages, *self.page_shape, dtype=dtype,
                                     pin_memory=self.device.type == "cuda")
         self._copy_stream = torch.cuda.Stream(self.device) if self.device.type == "cuda" else None
 
     @property
     def page_bytes_all_layers(self) -> int:
-        return self.layers * 2 * self.kv_heads * self.page_size * self.head_dim * self.data.element_size()
+        return self.data[:, 0].numel() * self.data.element_size()
 
     @staticmethod
     def bytes_per_page(layers, kv_heads, page_size, head_dim, elem_size=2) -> int:

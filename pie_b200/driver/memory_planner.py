@@ -44,6 +44,8 @@ class MemoryPlan:
 
 
 def kv_bytes_per_page(cfg: ModelConfig, page_size: int, tp: int = 1, kv_dtype_bytes: int = 2) -> int:
+    if cfg.latent is not None:
+        return cfg.kv_elems_per_token * page_size * kv_dtype_bytes
     hkv = max(1, cfg.num_key_value_heads // tp)
     return cfg.num_hidden_layers * 2 * hkv * page_size * cfg.head_dim * kv_dtype_bytes
 
@@ -54,6 +56,11 @@ def arena_bytes(cfg: ModelConfig, max_tokens: int, max_requests: int, tp: int = 
     inter = (cfg.moe_intermediate_size * cfg.num_experts_per_tok if cfg.is_moe else cfg.intermediate_size) // tp
     qkv = (cfg.num_attention_heads + 2 * cfg.num_key_value_heads) * cfg.head_dim // tp
     per_token = 2 * (3 * h + qkv + cfg.num_attention_heads * cfg.head_dim // tp + 3 * inter)
+    if cfg.latent is not None:
+        # fp32 residual stream (two copies), projections, per-head latent queries and outputs, feed-forward; in prefill
+        # also the keys and values of every head
+        heads = max(s.heads * (s.qk_dim + s.vdim + 2 * s.row) for s in cfg.latent)
+        per_token = 2 * (8 * h + heads + 3 * inter) + 2 * max(s.heads for s in cfg.latent) * 3 * 128
     logits = max_requests * cfg.vocab_size * (2 + 4)       # bf16 logits + fp32 rows for probes
     return max_tokens * per_token + logits
 

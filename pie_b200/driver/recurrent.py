@@ -1,6 +1,6 @@
-"""Recurrent-state cache of the Gated DeltaNet and Mamba-2 layers: per (recurrent layer, slot) the tail of the
-short convolution's inputs and the fp32 state (delta-rule state [heads, dk, dv], or state-space state
-[heads, head_dim, state]). A slot belongs to one resident context; the runtime's
+"""Recurrent-state cache of the Gated DeltaNet and Mamba-2 layers and of token-shifted blocks: per (recurrent layer,
+slot) the tail of the short convolution's inputs and the fp32 state (delta-rule state [heads, dk, dv], or state-space
+state [heads, head_dim, state]), or the previous token's normalised input (token shift, [width] fp32). A slot belongs to one resident context; the runtime's
 slot pool (`runtime/rs_cache.py`) hands slots out, tells the driver when a slot must start from zero
 (`rs_reset`) and asks for a slot copy when a context forks.
 
@@ -27,10 +27,13 @@ class RecurrentInputs:
     qo_host: List[int]
     slots_host: List[int]
     reset_host: List[int]
-    conv_state: torch.Tensor       # [L, S, C, K - 1] fp32
-    rec_state: torch.Tensor        # [L, S, Hv, dk, dv] fp32
+    conv_state: Optional[torch.Tensor]       # [L, S, C, K - 1] fp32
+    rec_state: Optional[torch.Tensor]        # [L, S, Hv, dk, dv] fp32
     layer_index: Dict[int, int]    # model layer -> index into the first dimension of the caches
     scratch: Optional[torch.Tensor] = None   # [N, C] fp32 convolution output (device path)
+    shift_state: Optional[torch.Tensor] = None   # [L, S, W] fp32 previous token's input (token shift)
+    shift_stage: Optional[torch.Tensor] = None   # [R, W] fp32: a portion's last input until its readers are done
+    staged: Optional[int] = None   # requests the stage is committed for (0: none of this fire's portions uses it)
 
 
 class RecurrentStateCache:
@@ -40,6 +43,13 @@ class RecurrentStateCache:
         if cfg.linear_layers and cfg.mamba_layers:
             raise NotImplementedError("Gated DeltaNet and Mamba-2 layers in one model")
         self.layer_index = {li: i for i, li in enumerate(lin)}
+        self.conv_state = self.rec_state = self.shift_state = None
+        self.conv_channels = 0
+        if cfg.token_shift:
+            if cfg.mamba_layers or cfg.linear_layers:
+                raise NotImplementedError("token shift beside Gated DeltaNet or Mamba-2 layers")
+            self.shift_state = torch.zeros(len(lin), num_slots, cfg.hidden_size, dtype=torch.float32, device=self.device)
+            return
         if cfg.mamba_layers:       # [heads, head_dim, state] per slot, convolution over x | B | C
             c, k = cfg.mamba_conv_channels, 4
             hv, dk, dv = cfg.mamba_num_heads, cfg.mamba_head_dim, cfg.ssm_state_size
@@ -51,8 +61,20 @@ class RecurrentStateCache:
         self.rec_state = torch.zeros(len(lin), num_slots, hv, dk, dv, dtype=torch.float32, device=self.device)
 
     @property
+    def buffers(self) -> List[torch.Tensor]:
+        return [b for b in (self.conv_state, self.rec_state, self.shift_state) if b is not None]
+
+    @property
     def bytes_per_slot(self) -> int:
-        return (self.conv_state[:, 0].numel() + self.rec_state[:, 0].numel()) * 4
+        return sum(b[:, 0].numel() for b in self.buffers) * 4
+
+    def device_scratch(self, n: int, r: int) -> dict:
+        """Device scratch of a fire of n tokens in r requests."""
+        if self.device.type != "cuda":
+            return {}
+        if self.shift_state is not None:
+            return {"shift_stage": torch.empty(max(r, 1), self.cfg.hidden_size, dtype=torch.float32, device=self.device)}
+        return {"scratch": torch.empty(max(n, 1), self.conv_channels, dtype=torch.float32, device=self.device)}
 
     def inputs(self, qo_indptr, rs_slots, rs_reset) -> RecurrentInputs:
         qo = np.ascontiguousarray(qo_indptr, dtype=np.int32)
@@ -68,20 +90,18 @@ class RecurrentStateCache:
         tok_req = np.repeat(np.arange(r, dtype=np.int32), np.diff(qo))
         dev = self.device
         t = lambda a: torch.from_numpy(a).to(dev)
-        n = int(qo[-1])
-        scratch = (torch.empty(max(n, 1), self.conv_channels, dtype=torch.float32, device=dev)
-                   if dev.type == "cuda" else None)
         return RecurrentInputs(t(qo), t(tok_req), t(slots), t(reset), qo.tolist(), slots.tolist(), reset.tolist(),
-                               self.conv_state, self.rec_state, self.layer_index, scratch)
+                               self.conv_state, self.rec_state, self.layer_index, shift_state=self.shift_state,
+                               **self.device_scratch(int(qo[-1]), r))
 
     def copy_slot(self, src: int, dst: int) -> None:
         """dst <- src in every layer (a forked context continues from its parent's state)."""
         if src == dst:
             return
         if self.device.type != "cuda":
-            self.conv_state[:, dst].copy_(self.conv_state[:, src])
-            self.rec_state[:, dst].copy_(self.rec_state[:, src])
+            for buf in self.buffers:
+                buf[:, dst].copy_(buf[:, src])
             return
         from .. import ops
-        for buf in (self.conv_state, self.rec_state):
+        for buf in self.buffers:
             ops.gdn_copy_slot(buf, src, dst)

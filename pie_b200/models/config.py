@@ -14,7 +14,7 @@ LLAMA_LIKE = {"llama", "qwen2", "qwen3", "mistral", "phi3"}   # pre-norm decoder
 # `model_type` strings of checkpoints this build loads (the architecture registry of the loader)
 SUPPORTED_MODEL_TYPES = ("llama", "mistral", "qwen2", "qwen3", "phi3", "qwen3_moe", "mixtral", "olmo2", "olmo3", "gpt_oss",
                          "qwen3_5", "qwen3_next", "mamba2_hybrid", "gemma2", "gemma3_text", "gemma3", "qwen2_moe", "qwen2_vl",
-                         "qwen2_audio")
+                         "qwen2_audio", "puzutar")
 MAMBA_TYPES = {"mamba2_hybrid"}         # Mamba-2 (state-space) mixers in llama-like blocks, between full-attention layers
 GDN_TYPES = {"qwen3_5", "qwen3_next"}   # hybrids: Gated DeltaNet (linear attention) layers between full-attention layers
 POST_NORM = {"olmo2", "olmo3"}       # same block with the norms after attention / MLP and q, k norms over all heads
@@ -22,6 +22,58 @@ MOE_TYPES = {"qwen3_moe", "mixtral", "gpt_oss", "qwen2_moe"}
 # Gemma-2 / Gemma-3: norms before AND after attention and MLP, gains stored as (w - 1), GeGLU, scaled embeddings,
 # alternating local / global layers (Gemma-3: a RoPE base of their own for the local ones; Gemma-2: soft-capped logits)
 GEMMA_TYPES = {"gemma2", "gemma3_text", "gemma3"}
+# configs that name the design under "architecture" instead of "model_type"
+ARCHITECTURES = {"Puzutar": "puzutar"}
+
+
+def config_model_type(cfg: dict) -> str:
+    """The registry name a `config.json` dictionary asks for ("" when it names none)."""
+    return cfg.get("model_type") or ARCHITECTURES.get(cfg.get("architecture", ""), "")
+
+
+@dataclass
+class LatentSpec:
+    """Sizes of one latent-attention mixer: per head `dim` unrotated and `rot_dim` rotated query / key dimensions
+    (the first `rot_dims` of the latter rotate) and `vdim` value dimensions; keys and values are projections of a
+    latent of `kv_rank` numbers per token, which is cached together with one rotated key part shared by all heads.
+    A query sees itself and the `window` - 1 tokens before it. `kv_from`: the layer whose cache this one reads."""
+    heads: int
+    dim: int
+    rot_dim: int
+    vdim: int
+    kv_rank: int
+    window: int
+    scale: float
+    rope_base: float
+    rot_dims: int
+    kv_from: Optional[int] = None
+
+    @property
+    def qk_dim(self) -> int:
+        return self.dim + self.rot_dim
+
+    @property
+    def rank_pad(self) -> int:
+        """Columns of the latent inside a cache row: a multiple of 16 (one tensor-core k step)."""
+        return _pad(self.kv_rank, 16)
+
+    @property
+    def row(self) -> int:
+        """Columns of a cache row: latent, then the rotated key part, each padded with zeros."""
+        return self.rank_pad + _pad(self.rot_dim, 16)
+
+    @property
+    def q_rows(self) -> int:
+        return self.heads * self.qk_dim
+
+    @property
+    def proj_rows(self) -> int:
+        """Rows of the fused query (+ latent and shared key, unless the layer borrows another's cache) projection."""
+        return self.q_rows + (self.kv_rank + self.rot_dim if self.kv_from is None else 0)
+
+
+def _pad(n: int, m: int = 8) -> int:
+    return -(-n // m) * m
 
 
 @dataclass
@@ -75,6 +127,12 @@ class ModelConfig:
     ssm_state_size: int = 0
     mamba_n_groups: int = 1
     mamba_norm_grouped: bool = False   # gated RMSNorm per B / C group (Nemotron-H) instead of over the whole inner width (Mamba-2)
+    # parallel blocks over a 32-bit residual stream: x += mixer(shifted norm(x)) + ff(norm(x)), then the token input
+    latent: Optional[list] = None      # LatentSpec per layer
+    ff_sizes: Optional[list] = None    # per layer width of the xIELU feed-forward (0: the layer has none)
+    norm_groups: int = 1               # RMSNorm over this many equal parts of the width, each with its own mean square
+    token_shift: bool = False          # the mixer reads h + (previous token's h - h) * shift: state of a sequence
+    token_side_dim: int = 0            # width of the per-layer token input (0: none)
     # quantisation of the linear weights: None | "fp8_block" (128x128 weight scales)
     quantization: Optional[str] = None
     dtype: str = "bfloat16"
@@ -102,7 +160,30 @@ class ModelConfig:
     @property
     def recurrent_layers(self) -> list:
         """Layers whose state lives in the recurrent-state cache (Gated DeltaNet or Mamba-2)."""
-        return [li for li in range(self.num_hidden_layers) if self.is_linear_layer(li) or self.is_mamba_layer(li)]
+        return [li for li in range(self.num_hidden_layers)
+                if self.token_shift or self.is_linear_layer(li) or self.is_mamba_layer(li)]
+
+    @property
+    def latent_cache_layers(self) -> list:
+        """Layers that write latent rows; the others read the rows of one of these."""
+        return [li for li, s in enumerate(self.latent) if s.kv_from is None]
+
+    @property
+    def latent_cache_index(self) -> dict:
+        """Layer -> index into the first dimension of the latent cache."""
+        own = {li: i for i, li in enumerate(self.latent_cache_layers)}
+        return {li: own[li if s.kv_from is None else s.kv_from] for li, s in enumerate(self.latent)}
+
+    @property
+    def kv_elems_per_token(self) -> int:
+        """Cache elements one token takes over all layers (unsharded)."""
+        if self.latent is not None:
+            return len(self.latent_cache_layers) * self.latent_row
+        return self.num_hidden_layers * 2 * self.num_key_value_heads * self.head_dim
+
+    @property
+    def latent_row(self) -> int:
+        return max(s.row for s in self.latent)
 
     @property
     def mamba_inner(self) -> int:
@@ -130,6 +211,8 @@ class ModelConfig:
 
     def layer_window_left(self, li: int) -> int:
         """Keys left of the query that layer `li` sees (-1: all). HF `sliding_window` counts the query itself."""
+        if self.latent is not None:
+            return self.latent[li].window - 1
         if not self.sliding_window or self.sliding_window <= 0:
             return -1
         if self.layer_types is not None and self.layer_types[li] != "sliding_attention":
@@ -155,7 +238,9 @@ class ModelConfig:
 
     @staticmethod
     def from_hf(cfg: dict, name: str = "") -> "ModelConfig":
-        mt = cfg.get("model_type", "llama")
+        mt = config_model_type(cfg) or "llama"
+        if mt == "puzutar":
+            return _puzutar_config(cfg, name)
         if mt == "gemma3" and "text_config" in cfg:       # multimodal wrapper: the language model's own section
             cfg = dict(cfg["text_config"], model_type="gemma3_text")
             mt = "gemma3_text"
@@ -245,6 +330,67 @@ class ModelConfig:
         p = Path(path)
         with open(p / "config.json") as f:
             return ModelConfig.from_hf(json.load(f), name=p.name)
+
+
+def _puzutar_config(cfg: dict, name: str) -> ModelConfig:
+    specs, ffs = [], []
+    for i, layer in enumerate(cfg["layers"]):
+        if layer["type"] != "latent_attention":
+            raise ValueError(f"layer {i}: unknown mixer {layer['type']!r}")
+        m, mlp = layer["mixer"], layer.get("mlp")
+        if mlp is not None and mlp["kind"] != "dense":
+            raise ValueError(f"layer {i}: unknown feed-forward {mlp['kind']!r}")
+        rot = m["rot"]
+        src = m.get("kv_from")
+        s = LatentSpec(heads=m["heads"], dim=m["dim"], rot_dim=m["rot_dim"], vdim=m["vdim"], kv_rank=m["kv_rank"],
+                       window=m["mask"]["size"], scale=float(m["scale"]), rope_base=float(rot["base"]),
+                       rot_dims=rot["dims"], kv_from=src)
+        if s.rot_dims % 2 or s.rot_dims > s.rot_dim or s.window < 1:
+            raise ValueError(f"layer {i}: rotation over {s.rot_dims} of {s.rot_dim} dimensions, window {s.window}")
+        if src is not None:
+            j = specs[src] if 0 <= src < i else None
+            if j is None or j.kv_from is not None or (j.kv_rank, j.rot_dim) != (s.kv_rank, s.rot_dim):
+                raise ValueError(f"layer {i}: kv_from {src} is not an earlier layer with a latent of the same sizes")
+        specs.append(s)
+        ffs.append(int(mlp["ff"]) if mlp else 0)
+    if cfg["width"] % cfg["norm"]["groups"]:
+        raise ValueError(f"width {cfg['width']} does not split into {cfg['norm']['groups']} norm groups")
+    side = cfg.get("token_side") or {}
+    return ModelConfig(
+        model_type="puzutar", hidden_size=cfg["width"], intermediate_size=max(ffs), num_hidden_layers=len(specs),
+        num_attention_heads=max(s.heads for s in specs), num_key_value_heads=1, head_dim=max(s.row for s in specs),
+        vocab_size=cfg["vocab"], max_position_embeddings=cfg.get("max_position_embeddings", 131072),
+        rms_norm_eps=cfg["norm"]["eps"], tie_word_embeddings=True, hidden_act="xielu", latent=specs, ff_sizes=ffs,
+        norm_groups=cfg["norm"]["groups"], token_shift=True, token_side_dim=side.get("dim", 0), dtype="bfloat16", name=name)
+
+
+def _puzutar_dict(cfg: ModelConfig) -> dict:
+    """The `config.json` dictionary `_puzutar_config` reads `cfg` from."""
+    layers = []
+    for s, ff in zip(cfg.latent, cfg.ff_sizes):
+        m = {"heads": s.heads, "dim": s.dim, "rot_dim": s.rot_dim, "vdim": s.vdim, "kv_rank": s.kv_rank, "scale": s.scale,
+             "mask": {"size": s.window}, "rot": {"base": s.rope_base, "dims": s.rot_dims}}
+        if s.kv_from is not None:
+            m["kv_from"] = s.kv_from
+        layers.append({"type": "latent_attention", "mixer": m, "mlp": {"kind": "dense", "ff": ff} if ff else None})
+    return {"architecture": "Puzutar", "width": cfg.hidden_size, "vocab": cfg.vocab_size, "layers": layers,
+            "norm": {"eps": cfg.rms_norm_eps, "groups": cfg.norm_groups}, "token_side": {"dim": cfg.token_side_dim}}
+
+
+def puzutar_shape(layers: int = 32, width: int = 4096, heads: int = 32, dim: int = 96, rot_dim: int = 32, vdim: int = 128,
+                  kv_rank: int = 256, window: int = 1024, ff: int = 14336, vocab: int = 32000, groups: int = 4,
+                  side: int = 64, share: int = 2) -> dict:
+    """config.json dictionary of a uniform model: of every `share` layers in a row the first keeps latents, the
+    others read them."""
+    spec = []
+    for i in range(layers):
+        m = dict(heads=heads, dim=dim, rot_dim=rot_dim, vdim=vdim, kv_rank=kv_rank, scale=(dim + rot_dim) ** -0.5,
+                 mask={"size": window}, rot={"base": 500000.0, "dims": rot_dim})
+        if i % share:
+            m["kv_from"] = i - i % share
+        spec.append({"type": "latent_attention", "mixer": m, "mlp": {"kind": "dense", "ff": ff}})
+    return {"architecture": "Puzutar", "width": width, "vocab": vocab, "layers": spec, "norm": {"eps": 1e-6, "groups": groups},
+            "token_side": {"dim": side}}
 
 
 def _is_fp8_weight_config(q: dict) -> bool:
@@ -361,10 +507,25 @@ PRESETS = {
                            dtype="float32"),
 }
 
+# presets of designs whose layers are described one by one: the arguments of `puzutar_shape`
+LAYERED_PRESETS = {
+    "puzutar-8b": dict(),
+    "tiny-puzutar": dict(layers=3, width=256, heads=2, dim=48, rot_dim=16, vdim=40, kv_rank=64, window=40, ff=384, vocab=32000,
+                         groups=2, side=16),
+}
+
 
 def preset(name: str, **overrides) -> ModelConfig:
+    if name in LAYERED_PRESETS:
+        shape = dict(LAYERED_PRESETS[name])
+        if "num_hidden_layers" in overrides:
+            shape["layers"] = overrides.pop("num_hidden_layers")
+        cfg = _puzutar_config(puzutar_shape(**shape), name)
+        for k, v in overrides.items():
+            setattr(cfg, k, v)
+        return cfg
     if name not in PRESETS:
-        raise KeyError(f"unknown model preset {name!r}; known: {sorted(PRESETS)}")
+        raise KeyError(f"unknown model preset {name!r}; known: {sorted(list(PRESETS) + list(LAYERED_PRESETS))}")
     kw = dict(PRESETS[name])
     kw.update(overrides)
     return ModelConfig(name=name, **kw)

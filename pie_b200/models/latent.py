@@ -1,0 +1,95 @@
+"""Parallel blocks with latent attention over a 32-bit residual stream (Puzutar).
+
+One layer: h = grouped RMSNorm(x), hs = h shifted towards the previous token's h; x += mixer(hs) + ff(h); then the
+per-layer token input, x += RMSNorm(W_proj (gelu(W_gate x) * e)). The norm of a layer also finishes the token input of
+the layer before (`LatentStream` carries what is pending), and the products that end both sublayers run as one GEMM over
+their inputs side by side.
+
+Latent attention runs in its absorbed form: with W_uk folded into the query and W_uv applied to the result, keys and
+values of every head are the cached rows themselves, so that a step reads one row per token whatever the head count.
+"""
+from __future__ import annotations
+
+import torch
+
+from ..ops import latent as lops
+from .config import ModelConfig, _pad
+
+
+class LatentStream:
+    """The residual stream between layers: x [N, padded width] fp32, and a token input not yet added to it."""
+
+    def __init__(self, x):
+        self.x, self.y, self.y_norm = x, None, None
+
+    def finish(self, cfg: ModelConfig):
+        """The stream with everything pending added."""
+        if self.y is not None:
+            self.x, _, _ = lops.stream_norm(self.x, cfg.hidden_size, cfg.rms_norm_eps, self.y, self.y_norm)
+            self.y = self.y_norm = None
+        return self.x
+
+
+def rope_table(base: float, dims: int, device) -> torch.Tensor:
+    inv = float(base) ** (-2.0 * torch.arange(dims // 2, dtype=torch.float64) / dims)
+    return inv.float().to(device)
+
+
+def prepare_latent(m) -> None:
+    """Derived tensors of every layer: the per-head factors in the layout the absorbed products read, rotation tables."""
+    cfg, tables = m.cfg, {}
+    m.vocab_local = cfg.vocab_size
+    m.cache_index = cfg.latent_cache_index
+    if m.w["lm_head"].shape == m.w["embed"].shape:
+        m.w["lm_head"] = m.w["embed"]                   # tied and unpadded: one copy
+    for s, lw in zip(cfg.latent, m.w["layers"]):
+        key = (s.rope_base, s.rot_dims)
+        if key not in tables:
+            tables[key] = rope_table(*key, m.device)
+        lw["rope"] = tables[key]
+        # query into the latent: [H, rank, dim]; latent into the value: [H, vdim, rank_pad] (a cached row is padded)
+        lw["w_uk_t"] = lw["w_uk"].view(s.heads, s.dim, s.kv_rank).transpose(1, 2).contiguous()
+        uv = lw["w_uv"].view(s.heads, s.vdim, s.kv_rank)
+        lw["w_uv_p"] = torch.nn.functional.pad(uv, (0, s.rank_pad - s.kv_rank)).contiguous()
+
+
+def latent_mixer(m, hs, lw: dict, li: int, fi, cache, out) -> None:
+    """Latent attention of layer `li` on hs [N, width]; the heads' values go to out [N, heads * vdim] (W_o follows)."""
+    s, n = m.cfg.latent[li], hs.shape[0]
+    page = cache.shape[2]
+    layer_cache = cache[m.cache_index[li]]
+    qkv = m._gemm(hs, lw["w_latent_in"])
+    q = lops.latent_rows(qkv, fi.positions, fi.slots, lw["rope"], lw.get("latent_norm"), layer_cache if s.kv_from is None else None,
+                         s, m.cfg.rms_norm_eps, s.row, s.rank_pad, copy_nope=False)
+    nope = qkv[:, :s.q_rows].view(n, s.heads, s.qk_dim)[..., :s.dim] if qkv.shape[1] == s.q_rows else \
+        qkv.as_strided((n, s.heads, s.dim), (qkv.stride(0), s.qk_dim, 1))
+    lops.per_head(nope, lw["w_uk_t"], q[..., :s.kv_rank])
+    o = lops.latent_attention(q, layer_cache, fi.attn, fi.rs, fi.slots, s, page, s.window - 1)
+    lops.per_head(o, lw["w_uv_p"], out.as_strided((n, s.heads, s.vdim), (out.stride(0), s.vdim, 1)))
+
+
+def parallel_latent_block(m, st: LatentStream, lw: dict, li: int, fi, cache) -> None:
+    cfg = m.cfg
+    s, ff, W, eps = cfg.latent[li], cfg.ff_sizes[li], cfg.hidden_size, cfg.rms_norm_eps
+    x, h, hs = lops.stream_norm(st.x, W, eps, st.y, st.y_norm, lw["ln1"], cfg.norm_groups, lw.get("shift"), fi.rs, li)
+    n, hv = x.shape[0], s.heads * s.vdim
+    cols = lw["w_block_out"].shape[1]
+    both = torch.empty(n, cols, dtype=h.dtype, device=h.device)       # attention heads | feed-forward activations
+    if _pad(hv) > hv:
+        both[:, hv:_pad(hv)] = 0
+    latent_mixer(m, hs if hs is not None else h, lw, li, fi, cache, both[:, :hv])
+    if ff:
+        act = both[:, _pad(hv):]
+        act.copy_(m._gemm(h, lw["w_up"]))
+        lops.bias_xielu(act, lw["b_up"], lw["act"])
+    side = cfg.token_side_dim
+    st.x, xc = lops.stream_add(x, m._gemm(both, lw["w_block_out"]), lw.get("b_down"), copy=side > 0)
+    st.y = st.y_norm = None
+    if side:
+        g = lops.side_gate(m._gemm(xc, lw["side_gate"]), m.w["side_embed"], fi.tokens, li * side, side)
+        st.y, st.y_norm = m._gemm(g, lw["side_proj"]), lw["side_norm"]
+
+
+def final_rows(m, rows):
+    """The model's norm on the rows that need logits."""
+    return lops.stream_norm(rows, m.cfg.hidden_size, m.cfg.rms_norm_eps, norm_w=m.w["final_norm"], groups=m.cfg.norm_groups)[1]

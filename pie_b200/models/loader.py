@@ -13,6 +13,7 @@ against a safetensors reader, producing this rank's weight dict. Ops:
   Cast(dtype) / DequantFp8Block() dtype change / 128x128 block-scaled fp8 -> bf16
   Transpose(a, b)                 swap two dimensions (GPT-OSS stores experts as [E, in, out])
   Mxfp4(blocks, scales)           e2m1 nibbles with one e8m0 scale per 32 -> values [.., rows, cols]
+  Pad(multiple)                   zeros appended until every dimension is a multiple (tile and TMA alignment)
   Attach(path)                    store under a runtime name
 
 The program is serialisable (`program_to_json`), so a per-rank plan can be compiled once and
@@ -30,7 +31,7 @@ from typing import Callable, Dict, List, Optional, Sequence, Tuple
 
 import torch
 
-from .config import ModelConfig
+from .config import ModelConfig, _pad, _puzutar_dict
 from .weights import kv_head_range, torch_dtype
 
 
@@ -58,6 +59,7 @@ def ExpandRows(x, factor, like): return Op("expand_rows", {"factor": factor, "li
 def Transpose(x, a, b): return Op("transpose", {"a": a, "b": b}, [x])
 def AddScalar(x, value): return Op("add_scalar", {"value": value}, [x])
 def RowScales(scale, like): return Op("row_scales", {"like": like}, [scale])
+def Pad(x, multiple=8): return Op("pad", {"multiple": multiple}, [x])
 def Mxfp4(blocks, scales): return Op("mxfp4", {}, [blocks, scales])
 
 _E2M1 = (0.0, 0.5, 1.0, 1.5, 2.0, 3.0, 4.0, 6.0, -0.0, -0.5, -1.0, -1.5, -2.0, -3.0, -4.0, -6.0)
@@ -136,6 +138,8 @@ def compile_program(cfg: ModelConfig, names: Sequence[str], tp_size: int = 1, tp
                     ep: bool = False, dtype: str = "bfloat16") -> Program:
     """Layout plan for a Llama/Qwen-family checkpoint (HF names) on rank (tp_rank of tp_size)."""
     names = set(names)
+    if cfg.latent is not None:
+        return _compile_latent(cfg, names, tp_size, dtype)
     T, r, d = tp_size, tp_rank, cfg.head_dim
     kv0, kvn = kv_head_range(cfg, r, T)
     # the language model's tensors may sit under a prefix ("model.", or a multimodal wrapper's "model.language_model.")
@@ -299,6 +303,70 @@ def compile_program(cfg: ModelConfig, names: Sequence[str], tp_size: int = 1, tp
                                 "vocab_start": r * (cfg.vocab_size // T) if T > 1 else 0})
 
 
+def _compile_latent(cfg: ModelConfig, names: set, tp_size: int, dtype: str) -> Program:
+    """Layout plan of a model with latent-attention mixers in parallel blocks (Puzutar names). Fused per layer: the query
+    projection with the latent's (`w_latent_in`), and the two products that end a parallel block, attention output and
+    feed-forward, side by side along K (`w_block_out`), since both add to the same residual. Every dimension a GEMM
+    sees is padded with zeros to a multiple of 8."""
+    if tp_size > 1:
+        raise NotImplementedError("latent attention under tensor parallelism")
+    W, S = cfg.hidden_size, cfg.token_side_dim
+    att: Dict[str, Op] = {}
+
+    def r(n, *shape):
+        if n not in names:
+            raise KeyError(f"checkpoint has no tensor {n}")
+        return Op("read", {"name": n, "shape": list(shape)})
+
+    att["embed"] = r("embed", cfg.vocab_size, W)
+    att["lm_head"] = Pad(r("embed", cfg.vocab_size, W))
+    att["final_norm"] = r("final.norm", W)
+    if S:
+        att["side_embed"] = r("side.embed", cfg.vocab_size, cfg.num_hidden_layers * S)
+    for li, (s, ff) in enumerate(zip(cfg.latent, cfg.ff_sizes)):
+        L, P = f"l{li}.", f"layers.{li}."
+        att[P + "ln1"] = r(L + "norm1", W)
+        if cfg.token_shift:
+            att[P + "shift"] = r(L + "shift", W)
+        q = r(L + "mix.q", s.q_rows, W)
+        if s.kv_from is None:
+            q = Concat([q, r(L + "mix.dkv", s.kv_rank + s.rot_dim, W)], 0)
+            att[P + "latent_norm"] = r(L + "mix.dkv.norm", s.kv_rank)
+        att[P + "w_latent_in"] = Pad(q)
+        att[P + "w_uk"] = r(L + "mix.uk", s.heads * s.dim, s.kv_rank)
+        att[P + "w_uv"] = r(L + "mix.uv", s.heads * s.vdim, s.kv_rank)
+        outs = [Pad(r(L + "mix.o", W, s.heads * s.vdim))]
+        if ff:
+            att[P + "w_up"], att[P + "b_up"] = Pad(r(L + "mlp.up", ff, W)), Pad(r(L + "mlp.up.b", ff))
+            att[P + "act"], att[P + "b_down"] = r(L + "mlp.act", 2), Pad(r(L + "mlp.down.b", W))
+            outs.append(Pad(r(L + "mlp.down", W, ff)))
+        att[P + "w_block_out"] = Concat(outs, 1) if ff else outs[0]
+        if S:
+            att[P + "side_gate"], att[P + "side_proj"] = Pad(r(L + "side.gate", S, W)), Pad(r(L + "side.proj", W, S))
+            att[P + "side_norm"] = r(L + "side.norm", W)
+    return Program(att, dtype, {"tp_size": 1, "tp_rank": 0, "ep": False, "layers": cfg.num_hidden_layers, "vocab_start": 0})
+
+
+class TensorDictReader:
+    """The reader interface over a dictionary of checkpoint tensors (random initialisation, tests)."""
+
+    def __init__(self, tensors: Dict[str, torch.Tensor]):
+        self.tensors = tensors
+
+    def names(self) -> List[str]:
+        return list(self.tensors)
+
+    def get(self, name) -> torch.Tensor:
+        return self.tensors[name]
+
+    def get_slice(self, name):
+        class _Slice:
+            def __init__(self, t): self.t = t
+            def get_shape(self): return list(self.t.shape)
+            def __getitem__(self, i): return self.t[i]
+        return _Slice(self.tensors[name])
+
+
 class SafetensorsReader:
     """Index over the *.safetensors shards of a checkpoint directory (lazy, sliceable reads)."""
 
@@ -356,6 +424,10 @@ def _eval(op: Op, reader, dtype) -> torch.Tensor:
             a, b = a.view(torch.uint8), b.view(torch.uint8)
         y = torch.stack([a, b], dim=1).reshape(a.shape[0] * 2, *a.shape[1:])
         return y.view(torch.float8_e4m3fn) if f8 else y
+    if k == "pad":
+        m, x = op.args["multiple"], xs[0]
+        extra = [(-n) % m for n in x.shape]
+        return torch.nn.functional.pad(x, [v for e in reversed(extra) for v in (0, e)]) if any(extra) else x
     if k == "stack":
         return torch.stack(xs, dim=0)
     if k == "zeros_like":
@@ -391,7 +463,10 @@ def infer_shape(op: Op, reader) -> Tuple[int, ...]:
     """Shape of an expression from the checkpoint's header alone (no tensor bytes are read)."""
     k = op.kind
     if k == "read":
-        return tuple(reader.get_slice(op.args["name"]).get_shape())
+        shape = tuple(reader.get_slice(op.args["name"]).get_shape())
+        if "shape" in op.args and shape != tuple(op.args["shape"]):
+            raise LoaderTypeError(f"{op.args['name']} is {shape}, the architecture needs {tuple(op.args['shape'])}")
+        return shape
     xs = [infer_shape(i, reader) for i in op.inputs]
     x = xs[0] if xs else ()
     if k == "shard":
@@ -420,6 +495,8 @@ def infer_shape(op: Op, reader) -> Tuple[int, ...]:
         return (len(xs),) + x
     if k in ("zeros_like", "float", "add_scalar"):
         return x
+    if k == "pad":
+        return tuple(_pad(n, op.args["multiple"]) for n in x)
     if k == "squeeze":
         d = op.args["dim"]
         if x[d] != 1:
@@ -479,7 +556,7 @@ def typecheck_program(prog: Program, cfg: ModelConfig, reader) -> Dict[str, Tupl
     architecture needs on this rank; all mismatches are reported together, before any tensor is read.
     Returns the inferred shapes. Counterpart of the weight loader's type checker in the reference
     (driver/weight_loader/src/typecheck.rs)."""
-    want = expected_shapes(cfg, prog.meta.get("tp_size", 1), prog.meta.get("ep", False))
+    want = {} if cfg.latent is not None else expected_shapes(cfg, prog.meta.get("tp_size", 1), prog.meta.get("ep", False))
     shapes, errors = {}, []
     for path, op in prog.attach.items():
         try:
@@ -652,11 +729,38 @@ def load_checkpoint(path, device="cpu", tp_size: int = 1, tp_rank: int = 0, ep: 
     return cfg, _cached_load(p, prog, reader, device)
 
 
+def _latent_tensors(cfg: ModelConfig, weights: dict) -> Dict[str, torch.Tensor]:
+    """Checkpoint tensors of a latent-attention model from its runtime layout (the inverse of `_compile_latent`)."""
+    W, S = cfg.hidden_size, cfg.token_side_dim
+    t = {"embed": weights["embed"], "final.norm": weights["final_norm"]}
+    if S:
+        t["side.embed"] = weights["side_embed"]
+    for li, (lw, s, ff) in enumerate(zip(weights["layers"], cfg.latent, cfg.ff_sizes)):
+        L, hv = f"l{li}.", s.heads * s.vdim
+        t[L + "norm1"] = lw["ln1"]
+        if cfg.token_shift:
+            t[L + "shift"] = lw["shift"]
+        t[L + "mix.q"], t[L + "mix.uk"], t[L + "mix.uv"] = lw["w_latent_in"][:s.q_rows, :W], lw["w_uk"], lw["w_uv"]
+        if s.kv_from is None:
+            t[L + "mix.dkv"], t[L + "mix.dkv.norm"] = lw["w_latent_in"][s.q_rows:s.proj_rows, :W], lw["latent_norm"]
+        t[L + "mix.o"] = lw["w_block_out"][:W, :hv]
+        if ff:
+            t[L + "mlp.up"], t[L + "mlp.up.b"], t[L + "mlp.act"] = lw["w_up"][:ff, :W], lw["b_up"][:ff], lw["act"]
+            t[L + "mlp.down"], t[L + "mlp.down.b"] = lw["w_block_out"][:W, _pad(hv):_pad(hv) + ff], lw["b_down"][:W]
+        if S:
+            t[L + "side.gate"], t[L + "side.proj"], t[L + "side.norm"] = lw["side_gate"][:S, :W], lw["side_proj"][:W, :S], lw["side_norm"]
+    return t
+
+
 def export_hf_checkpoint(cfg: ModelConfig, weights: dict, path) -> None:
     """Write unsharded runtime weights back out under Hugging Face names (tests, tooling)."""
     from safetensors.torch import save_file
     p = Path(path)
     p.mkdir(parents=True, exist_ok=True)
+    if cfg.latent is not None:
+        save_file({k: v.contiguous().cpu() for k, v in _latent_tensors(cfg, weights).items()}, str(p / "model.safetensors"))
+        (p / "config.json").write_text(json.dumps(_puzutar_dict(cfg)))
+        return
     d, hq, hkv = cfg.head_dim, cfg.num_attention_heads, cfg.num_key_value_heads
     ungain = (lambda g: g.float() - 1.0) if cfg.norm_plus_one else (lambda g: g)      # Gemma stores (gain - 1)
     t: Dict[str, torch.Tensor] = {"model.embed_tokens.weight": weights["embed"], "model.norm.weight": ungain(weights["final_norm"])}

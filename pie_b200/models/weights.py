@@ -11,6 +11,7 @@ Runtime layout per layer (this rank's shard under tensor parallelism):
   OLMo-2 (post-norm): no ln1; ln2 follows attention, ln3 follows the MLP; q_norm [hq*d], k_norm [hkv*d]
   Gemma-2/3 (sandwich norms): ln1 / ln2 before attention / MLP, ln_pa / ln_pf on their outputs before the
   residual add; gains hold the full multiplier (the loader adds the checkpoint's implicit 1)
+  Puzutar (latent attention in parallel blocks): see `loader._compile_latent`
 MoE layers replace w_gate_up / w_down by router [E, H], experts_gate_up [E_local, 2*Im, H]
 (interleaved) and experts_down [E_local, H, Im].
 
@@ -89,6 +90,8 @@ def random_weights(cfg: ModelConfig, device="cpu", dtype=None, seed: int = 0, tp
     """
     dtype = dtype or torch_dtype(cfg.dtype)
     gen = _Gen(seed, device, dtype, std)
+    if cfg.latent is not None:
+        return _random_latent(cfg, gen, tp_size)
     H, d = cfg.hidden_size, cfg.head_dim
     hq, hkv = cfg.num_attention_heads, cfg.num_key_value_heads
     T, r = tp_size, tp_rank
@@ -209,6 +212,33 @@ def random_weights(cfg: ModelConfig, device="cpu", dtype=None, seed: int = 0, tp
     w["lm_head"] = head
     w["lm_head_vocab_start"] = r * (cfg.vocab_size // T) if T > 1 else 0
     return w
+
+
+def _random_latent(cfg: ModelConfig, gen: _Gen, tp_size: int) -> dict:
+    """Random checkpoint tensors of a latent-attention model, brought into the runtime layout by the loader."""
+    from .loader import TensorDictReader, compile_program, execute_program
+    W, S = cfg.hidden_size, cfg.token_side_dim
+    gain = lambda n: 1 + gen.normal(n, std=0.1)
+    t = {"embed": gen.normal(cfg.vocab_size, W), "final.norm": gain(W)}
+    if S:
+        t["side.embed"] = gen.normal(cfg.vocab_size, cfg.num_hidden_layers * S, std=0.5)
+    for li, (s, ff) in enumerate(zip(cfg.latent, cfg.ff_sizes)):
+        L = f"l{li}."
+        t[L + "norm1"], t[L + "shift"] = gain(W), 0.5 + gen.normal(W, std=0.2)
+        t[L + "mix.q"] = gen.normal(s.q_rows, W)
+        if s.kv_from is None:
+            t[L + "mix.dkv"], t[L + "mix.dkv.norm"] = gen.normal(s.kv_rank + s.rot_dim, W), gain(s.kv_rank)
+        t[L + "mix.uk"] = gen.normal(s.heads * s.dim, s.kv_rank, std=s.kv_rank ** -0.5)
+        t[L + "mix.uv"] = gen.normal(s.heads * s.vdim, s.kv_rank, std=s.kv_rank ** -0.5)
+        t[L + "mix.o"] = gen.normal(W, s.heads * s.vdim)
+        if ff:
+            t[L + "mlp.up"], t[L + "mlp.up.b"], t[L + "mlp.act"] = gen.normal(ff, W), gen.normal(ff, std=0.1), gen.normal(2, std=0.5)
+            t[L + "mlp.down"], t[L + "mlp.down.b"] = gen.normal(W, ff), gen.normal(W, std=0.1)
+        if S:
+            t[L + "side.gate"], t[L + "side.proj"] = gen.normal(S, W, std=W ** -0.5), gen.normal(W, S)
+            t[L + "side.norm"] = gen.normal(W, std=0.1)
+    prog = compile_program(cfg, list(t), tp_size, 0, False, str(gen.dtype).replace("torch.", ""))
+    return execute_program(prog, TensorDictReader(t), gen.device)
 
 
 def weights_nbytes(w) -> int:

@@ -781,6 +781,7 @@ class DecodePlan:
     item_slot: Optional[torch.Tensor] = None
     item_tile: Optional[torch.Tensor] = None
     tile_members: Optional[torch.Tensor] = None
+    kv_lens: Optional[torch.Tensor] = None
 
 
 def decode_scratch_floats(max_items: int, hq: int, head_dim: int) -> int:
@@ -964,7 +965,7 @@ def sample(logits, temperature, top_k, top_p, min_p, seeds, mask_bits=None, mask
 
 def row_stats(logits):
     """[rows, 3] fp32: max, log-sum-exp and entropy of the unscaled next-token distribution."""
-    if not logits.is_cuda:
+    if not logits.is_cuda or logits.dtype != torch.bfloat16:
         return reference.row_stats(logits)
     rows, vocab = logits.shape
     out = torch.empty(rows, 3, dtype=torch.float32, device=logits.device)

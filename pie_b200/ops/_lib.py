@@ -61,6 +61,13 @@ _SIGNATURES = {
     "pie_gdn_mixer": [p, i32, p, p, p, p, p, p, p, p, p, p, p, p, i32, i32, i32, i32, i32, i32, i32, f32, p],
     "pie_gdn_copy_slot": [p, i64, i64, i32, i32, i32, p],
     "pie_mamba2_mixer": [p, i32, p, p, p, p, p, p, p, p, p, p, p, p, p, i32, i32, i32, i32, i32, i32, p],
+    "pie_stream_embed": [p, p, p, i32, i32, i32, i32, i32, p],
+    "pie_stream_norm": [p, i32, i32, p],
+    "pie_latent_rows": [p, i32, p],
+    "pie_latent_attn_warp": [p, i32, p],
+    "pie_bias_xielu": [p, i32, p, p, i32, i32, i32, p],
+    "pie_stream_add": [p, p, p, p, p, i32, i32, i32, p],
+    "pie_side_gate": [p, i32, p, i32, p, p, i32, i32, i32, i32, i32, i32, p],
     "pie_gemm_set_workspace": [i32, p, i64, p, i32],
     "pie_gemm_set_pairs": [i32],
     "pie_gemm_set_swap": [i32],
@@ -82,6 +89,14 @@ class KernelLibraryError(RuntimeError):
 
 def lib_path() -> Path:
     return _LIB_PATH
+
+
+def use_library(path) -> None:
+    """Load the kernels from `path` (a library built for one model family) instead of the whole library."""
+    global _LIB_PATH
+    if _LIB is not None and Path(path) != _LIB_PATH:
+        raise KernelLibraryError("a kernel library is already loaded")
+    _LIB_PATH = Path(path)
 
 
 def load(required: bool = True):

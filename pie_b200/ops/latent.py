@@ -1,0 +1,140 @@
+"""Ops of blocks over a 32-bit residual stream with token shift, latent attention and per-layer token input. CUDA tensors
+go to `csrc/kernels/latent*.cu` (bf16 when serving, float32 on the 32-bit path), CPU tensors to :mod:`.latent_reference`.
+"""
+from __future__ import annotations
+
+import ctypes as C
+from typing import Optional
+
+import torch
+
+from . import _lib, latent_reference as ref
+from ._lib import check, fn, ptr, stream_ptr
+
+p, i32, f32 = C.c_void_p, C.c_int, C.c_float
+
+
+def _struct(name: str, *fields):
+    return type(name, (C.Structure,), {"_fields_": [(n, t) for names, t in fields for n in names.split()]})
+
+
+# mirrors of the argument structs in csrc/kernels/latent.cu
+StreamNormArgs = _struct("StreamNormArgs", ("x y y_norm x_out norm_w shift h hs tok_req qo_indptr slots reset state stage", p),
+                         ("n width ldx ldy ldh groups rows_per_block", i32), ("eps", f32))
+LatentRowsArgs = _struct("LatentRowsArgs", ("qkv positions slots inv_freq norm_w q_out cache", p),
+                         ("n ld heads dim rot_dim rot_dims rank rank_pad cache_row copy_nope q_width q_rot q_zero", i32), ("eps", f32))
+LatentAttnArgs = _struct("LatentAttnArgs", ("q cache page_indices kv_page_indptr qo_indptr kv_lens tok_req slots mask_bits "
+                                            "mask_word_indptr out", p),
+                         ("n heads row rank_pad cache_row page_size window_left", i32), ("scale", f32))
+
+
+def _f32(t) -> int:
+    return 1 if t.dtype == torch.float32 else 0
+
+
+def stream_embed(tokens, table, ld: int):
+    """Rows of `table` as a 32-bit stream [N, ld] (zeros beyond the table's width)."""
+    if not table.is_cuda:
+        return ref.stream_embed(tokens, table, ld)
+    n, w = tokens.numel(), table.shape[1]
+    x = torch.empty(n, ld, dtype=torch.float32, device=table.device)
+    check(fn("pie_stream_embed")(ptr(tokens), ptr(table), ptr(x), n, w, ld, table.shape[0], _f32(table), stream_ptr()), "stream_embed")
+    return x
+
+
+def stream_norm(x, width: int, eps: float, y=None, y_norm=None, norm_w=None, groups: int = 1, shift=None, rs=None, layer: int = 0,
+                dtype=None):
+    """Per token: x += y / rms(y) * y_norm (if y); h = RMSNorm(x) in `groups` parts * norm_w; hs = h + (h of the token
+    before - h) * shift. The token before the first one of a portion comes from the sequence's state in `rs`
+    (a `driver.recurrent.RecurrentInputs`), which advances. Returns (x, h, hs); what was not asked for is None."""
+    dtype = dtype or (norm_w if norm_w is not None else y).dtype
+    if not x.is_cuda:
+        return ref.stream_norm(x, width, eps, y, y_norm, norm_w, groups, shift, rs, layer, dtype)
+    n, ld = x.shape
+    new = lambda dt: torch.empty(n, ld, dtype=dt, device=x.device)
+    x_out = new(torch.float32) if y is not None else None
+    h = new(dtype) if norm_w is not None else None
+    hs = new(dtype) if shift is not None else None
+    a = StreamNormArgs(x=ptr(x), y=ptr(y), y_norm=ptr(y_norm), x_out=ptr(x_out), norm_w=ptr(norm_w), shift=ptr(shift), h=ptr(h),
+                       hs=ptr(hs), n=n, width=width, ldx=ld, ldy=y.stride(0) if y is not None else 0, ldh=ld, groups=groups,
+                       rows_per_block=max(1, min(8, n // 592)), eps=eps)
+    commit = 0
+    if shift is not None:
+        state = rs.shift_state[layer]
+        a.tok_req, a.qo_indptr, a.slots, a.reset = ptr(rs.tok_req), ptr(rs.qo_indptr), ptr(rs.slots), ptr(rs.reset)
+        a.state, a.stage = ptr(state), ptr(rs.shift_stage)
+        if rs.staged is None:               # portions of two tokens or more leave their last h in the stage
+            rs.staged = len(rs.slots_host) if any(b - a > 1 for a, b in zip(rs.qo_host, rs.qo_host[1:])) else 0
+        commit = rs.staged
+    check(fn("pie_stream_norm")(C.byref(a), 1 if dtype == torch.float32 else 0, commit, stream_ptr()), "stream_norm")
+    return (x if x_out is None else x_out), h, hs
+
+
+def latent_rows(qkv, positions, slots, inv_freq, norm_w, cache, spec, eps: float, q_width: int, q_rot: int, copy_nope: bool):
+    """Rotate the queries of the fused projection into rows [N, heads, q_width] (rotated part at column q_rot; with
+    `copy_nope` the unrotated part in front of it, else the columns before rank_pad are left for `per_head`), and write
+    the new tokens' cache rows: normalised latent, rotated shared key part. `cache` None: a layer that borrows rows."""
+    n = qkv.shape[0]
+    q = torch.empty(n, spec.heads, q_width, dtype=qkv.dtype, device=qkv.device)
+    if not qkv.is_cuda:
+        return ref.latent_rows(qkv, positions, slots, inv_freq, norm_w, cache, spec, eps, q, q_rot, copy_nope)
+    a = LatentRowsArgs(qkv=ptr(qkv), positions=ptr(positions), slots=ptr(slots), inv_freq=ptr(inv_freq), norm_w=ptr(norm_w),
+                       q_out=ptr(q), cache=ptr(cache), n=n, ld=qkv.stride(0), heads=spec.heads, dim=spec.dim, rot_dim=spec.rot_dim,
+                       rot_dims=spec.rot_dims, rank=spec.kv_rank, rank_pad=spec.rank_pad,
+                       cache_row=cache.shape[-1] if cache is not None else 0, copy_nope=1 if copy_nope else 0, q_width=q_width,
+                       q_rot=q_rot, q_zero=q_rot if copy_nope else spec.kv_rank, eps=eps)
+    check(fn("pie_latent_rows")(C.byref(a), _f32(qkv), stream_ptr()), "latent_rows")
+    return q
+
+
+def per_head(x, w, out):
+    """out[:, h, :] = x[:, h, :] @ w[h].T for x [N, H, K] and w [H, M, K]; x and out may be strided views."""
+    if not x.is_cuda or x.dtype == torch.float32:
+        out.copy_(torch.bmm(x.transpose(0, 1), w.transpose(1, 2)).transpose(0, 1))
+        return out
+    out.copy_(torch.bmm(x.transpose(0, 1), w.transpose(1, 2)).transpose(0, 1))
+    return out
+
+
+def latent_attention(q, cache, plan, rs, slots, spec, page_size: int, window_left: int):
+    """Softmax over the visible cache rows of q [N, heads, row] . row * scale; returns the weighted latents
+    [N, heads, rank_pad]. The absorbed form: keys and values of every head are the rows themselves."""
+    if not q.is_cuda:
+        return ref.latent_attention(q, cache, plan, spec, window_left)
+    n = q.shape[0]
+    out = torch.empty(n, spec.heads, spec.rank_pad, dtype=q.dtype, device=q.device)
+    a = LatentAttnArgs(q=ptr(q), cache=ptr(cache), page_indices=ptr(plan.page_indices), kv_page_indptr=ptr(plan.kv_page_indptr),
+                       qo_indptr=ptr(rs.qo_indptr), kv_lens=ptr(plan.kv_lens), tok_req=ptr(rs.tok_req), slots=ptr(slots),
+                       mask_bits=ptr(getattr(plan, "mask_bits", None)), mask_word_indptr=ptr(getattr(plan, "mask_word_indptr", None)),
+                       out=ptr(out), n=n, heads=spec.heads, row=q.shape[2], rank_pad=spec.rank_pad, cache_row=cache.shape[-1],
+                       page_size=page_size, window_left=window_left, scale=spec.scale)
+    check(fn("pie_latent_attn_warp")(C.byref(a), _f32(q), stream_ptr()), "latent_attn_warp")
+    return out
+
+
+def bias_xielu(y, bias, act):
+    """y = xIELU(y + bias) in place; y may be a column range of a wider buffer."""
+    if not y.is_cuda:
+        return ref.bias_xielu(y, bias, act)
+    check(fn("pie_bias_xielu")(ptr(y), y.stride(0), ptr(bias), ptr(act), y.shape[0], y.shape[1], _f32(y), stream_ptr()), "bias_xielu")
+    return y
+
+
+def stream_add(x, d, bias=None, copy: bool = False):
+    """(x + d + bias, the same in d's type or None): a sublayer's output joins the 32-bit stream."""
+    if not x.is_cuda:
+        return ref.stream_add(x, d, bias, copy)
+    out = torch.empty_like(x)
+    cp = torch.empty_like(d) if copy and d.dtype != torch.float32 else None
+    check(fn("pie_stream_add")(ptr(x), ptr(d), ptr(bias), ptr(out), ptr(cp), x.shape[0], x.shape[1], _f32(d), stream_ptr()), "stream_add")
+    return out, (out if d.dtype == torch.float32 else cp)
+
+
+def side_gate(z, table, tokens, col0: int, dim: int):
+    """gelu_tanh(z) * table[tokens, col0:col0 + dim], zeros in the padding columns of z."""
+    if not z.is_cuda:
+        return ref.side_gate(z, table, tokens, col0, dim)
+    g = torch.empty(z.shape[0], z.shape[1], dtype=z.dtype, device=z.device)
+    check(fn("pie_side_gate")(ptr(z), z.stride(0), ptr(table), table.stride(0), ptr(tokens), ptr(g), g.stride(0), dim, col0,
+                              table.shape[0], z.shape[0], _f32(z), stream_ptr()), "side_gate")
+    return g

@@ -171,7 +171,7 @@ def _human(n: int) -> str:
 def cmd_model(args) -> int:
     """`pie model list | download <org/name> [--revision R] [--all] | remove <org/name> [--yes]`
     (server/src/cli/model_cmd.rs:20-254)."""
-    from ..models.config import PRESETS
+    from ..models.config import LAYERED_PRESETS, PRESETS, preset
     from . import hf
     if args.action == "download":
         if not args.repo:
@@ -195,6 +195,10 @@ def cmd_model(args) -> int:
     for name, kw in PRESETS.items():
         print(f"  {name:18s} {kw['model_type']:10s} layers={kw['num_hidden_layers']:3d} hidden={kw['hidden_size']:5d} "
               f"heads={kw['num_attention_heads']}/{kw['num_key_value_heads']} vocab={kw['vocab_size']}")
+    for name in LAYERED_PRESETS:
+        c = preset(name)
+        print(f"  {name:18s} {c.model_type:10s} layers={c.num_hidden_layers:3d} hidden={c.hidden_size:5d} "
+              f"heads={c.num_attention_heads} latent={c.latent[0].kv_rank} vocab={c.vocab_size}")
     return 0
 
 

@@ -75,7 +75,7 @@ def _dir_size(p: Path) -> int:
 
 def list_cached(cache: Optional[Path] = None) -> List[Tuple[str, bool, str, int]]:
     """[(repo id, supported, architecture or reason, bytes)] for every `models--*` directory of the cache."""
-    from ..models.config import SUPPORTED_MODEL_TYPES
+    from ..models.config import SUPPORTED_MODEL_TYPES, config_model_type
     root = cache or hf_cache_root()
     out = []
     if not root.is_dir():
@@ -88,7 +88,7 @@ def list_cached(cache: Optional[Path] = None) -> List[Tuple[str, bool, str, int]
         ok, why = False, "no config"
         if snap is not None and (snap / "config.json").is_file():
             try:
-                mt = json.loads((snap / "config.json").read_text()).get("model_type", "")
+                mt = config_model_type(json.loads((snap / "config.json").read_text()))
                 ok, why = (True, mt) if mt in SUPPORTED_MODEL_TYPES else (False, f"unsupported type: {mt}")
             except (OSError, ValueError):
                 pass
