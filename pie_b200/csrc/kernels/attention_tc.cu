@@ -89,7 +89,10 @@ __device__ __forceinline__ float fast_tanh(float x) {
 // and cap_post = cap / sm_scale, so that the unchanged scale by sm_scale * log2(e) gives cap * tanh(s * sm_scale / cap).
 // G = query heads per KV head; NT = MMA tiles of 128 rows per CTA (they share the K/V stages);
 // D = head dimension (64 or 128).
-template <int G, int NT, int D, bool CAP = false>
+// TOK: keys and values lie token by token, [tokens][hkv][2][D] (tma_kv then has the dimensions D, hkv * 2, tokens), and a
+// "page" is 16 consecutive tokens: the layout a projection of latents writes. Its value heads may be narrower than D.
+// out_ld / out_cols: elements per token of `out` and per head (columns past out_cols are not stored; a multiple of 8).
+template <int G, int NT, int D, bool CAP = false, bool TOK = false>
 __global__ void __launch_bounds__(AtCfg<NT, D>::THREADS, 1)
 paged_prefill_attn_tc_kernel(const __grid_constant__ CUtensorMap tma_q, const __grid_constant__ CUtensorMap tma_kv,
                              const int* __restrict__ page_indices, const int* __restrict__ kv_page_indptr,
@@ -98,7 +101,7 @@ paged_prefill_attn_tc_kernel(const __grid_constant__ CUtensorMap tma_q, const __
                              const uint32_t* __restrict__ mask_bits, const long* __restrict__ mask_word_indptr,
                              bf16* __restrict__ out, float* __restrict__ lse_out, const float* __restrict__ sinks_log2,
                              int hq, int hkv, int pad_page, float scale_log2, int window_left, int* status,
-                             float cap_pre, float cap_post) {
+                             float cap_pre, float cap_post, int out_ld, int out_cols) {
     constexpr int TQ = AT_ROWS / G;          // query tokens per MMA tile
     constexpr int HALVES = D / 64;
     constexpr uint32_t AT_Q_BYTES = AtCfg<NT, D>::Q_BYTES, AT_KV_TILE = AtCfg<NT, D>::KV_TILE;
@@ -149,6 +152,11 @@ paged_prefill_attn_tc_kernel(const __grid_constant__ CUtensorMap tma_q, const __
         kv_hi = max(kv_hi, hi);
     }
     const int npages = (kv_hi + 15) >> 4;
+    // a sliding window hides every block before the one its first query's first key lies in: blocks are counted from there
+    const int jb = window_left >= 0 ? max(0, kv_len - qo_len + qstart - window_left) / AT_BK : 0;
+#pragma unroll
+    for (int t = 0; t < NT; ++t) nkb_t[t] = max(0, nkb_t[t] - jb);
+    nkb = max(0, nkb - jb);
 
     if (threadIdx.x == 0) {
         mbar_init(q_full(), 1);
@@ -198,7 +206,7 @@ paged_prefill_attn_tc_kernel(const __grid_constant__ CUtensorMap tma_q, const __
                 int pg_id[4];
 #pragma unroll
                 for (int pg = 0; pg < 4; ++pg) {
-                    const int pi = j * 4 + pg;
+                    const int pi = (jb + j) * 4 + pg;
                     pg_id[pg] = pi < npages ? pages[pi] : pad_page;
                 }
                 if (!mbar_wait(k_empty(s), par, status, PIE_ERR_WAIT_TMA)) { ok = false; break; }
@@ -207,8 +215,13 @@ paged_prefill_attn_tc_kernel(const __grid_constant__ CUtensorMap tma_q, const __
                 for (int pg = 0; pg < 4; ++pg) {
                     const int krow = ((pg_id[pg] * 2) * hkv + h) * 16;
 #pragma unroll
-                    for (int half = 0; half < HALVES; ++half)
-                        tma_load_2d(k_s + s * AT_KV_TILE + half * AT_KV_HALF + pg * 2048, &tma_kv, k_full(s), half * 64, krow);
+                    for (int half = 0; half < HALVES; ++half) {
+                        const uint32_t dst = k_s + s * AT_KV_TILE + half * AT_KV_HALF + pg * 2048;
+                        if constexpr (TOK)
+                            tma_load_3d(dst, &tma_kv, k_full(s), half * 64, 2 * h, pg_id[pg] * 16);
+                        else
+                            tma_load_2d(dst, &tma_kv, k_full(s), half * 64, krow);
+                    }
                 }
                 if (!mbar_wait(v_empty(s), par, status, PIE_ERR_WAIT_TMA)) { ok = false; break; }
                 mbar_arrive_expect_tx(v_full(s), AT_KV_TILE);
@@ -216,8 +229,13 @@ paged_prefill_attn_tc_kernel(const __grid_constant__ CUtensorMap tma_q, const __
                 for (int pg = 0; pg < 4; ++pg) {
                     const int vrow = ((pg_id[pg] * 2 + 1) * hkv + h) * 16;
 #pragma unroll
-                    for (int half = 0; half < HALVES; ++half)
-                        tma_load_2d(v_s + s * AT_KV_TILE + half * AT_KV_HALF + pg * 2048, &tma_kv, v_full(s), half * 64, vrow);
+                    for (int half = 0; half < HALVES; ++half) {
+                        const uint32_t dst = v_s + s * AT_KV_TILE + half * AT_KV_HALF + pg * 2048;
+                        if constexpr (TOK)
+                            tma_load_3d(dst, &tma_kv, v_full(s), half * 64, 2 * h + 1, pg_id[pg] * 16);
+                        else
+                            tma_load_2d(dst, &tma_kv, v_full(s), half * 64, vrow);
+                    }
                 }
             }
             // no copy may be in flight when the CTA exits
@@ -311,7 +329,7 @@ paged_prefill_attn_tc_kernel(const __grid_constant__ CUtensorMap tma_q, const __
                 for (int i = 0; i < 32; ++i)
                     sv[c * 32 + i] = CAP ? cap_post * fast_tanh(__uint_as_float(v[i]) * cap_pre) : __uint_as_float(v[i]);
             }
-            const int kb0 = j * AT_BK;
+            const int kb0 = (jb + j) * AT_BK;
             const bool inner = !custom && kb0 + AT_BK <= lim && kb0 >= lo;
             if (!__all_sync(0xffffffffu, inner)) {
                 // 64-bit allow mask of this row for the block
@@ -396,7 +414,7 @@ paged_prefill_attn_tc_kernel(const __grid_constant__ CUtensorMap tma_q, const __
             // attention sink: a per-head logit in the softmax denominator without a value row
             if (sinks_log2 && l > 0.f) l += exp2f(sinks_log2[head] - m_ref * scale_log2);
             const float inv = l > 0.f ? 1.f / l : 0.f;
-            bf16* dst = out + ((size_t)(q_base + (valid ? qtok : 0)) * hq + head) * D;
+            bf16* dst = out + (size_t)(q_base + (valid ? qtok : 0)) * out_ld + (size_t)head * out_cols;
 #pragma unroll
             for (int c = 0; c < D / 32; ++c) {
                 uint32_t v[32];
@@ -405,6 +423,7 @@ paged_prefill_attn_tc_kernel(const __grid_constant__ CUtensorMap tma_q, const __
                 if (valid) {
 #pragma unroll
                     for (int i8 = 0; i8 < 4; ++i8) {
+                        if (TOK && c * 32 + i8 * 8 >= out_cols) break;
                         float tv[8];
 #pragma unroll
                         for (int i = 0; i < 8; ++i) tv[i] = __uint_as_float(v[i8 * 8 + i]) * inv;
@@ -505,7 +524,7 @@ PIE_API int pie_paged_prefill_attn_tc_softcap(const void* q, const void* kv_laye
         kern<<<grid, Cfg::THREADS, Cfg::SMEM, st>>>(                                                                  \
             tq, tkv, page_indices, kv_page_indptr, qo_indptr, kv_lens, tile_req, tile_qstart, mask_bits,              \
             mask_word_indptr, (bf16*)out, lse_out, sinks_log2, hq, hkv, total_pages - 1, scale_log2, window_left,     \
-            status, cap_pre, cap_post);                                                                               \
+            status, cap_pre, cap_post, hq * D_, D_);                                                                  \
         return (int)cudaGetLastError();                                                                               \
     }
 #define GO2(G_, NT_)           \
@@ -540,3 +559,47 @@ PIE_API int pie_paged_prefill_attn_tc(const void* q, const void* kv_layer, const
                                              status, 0.f, st);
 }
 
+
+// Prefill attention over keys and values that were projected from latents for this pass: kv [total_tokens][heads][2][D],
+// "page" p of page_indices = tokens 16 p .. 16 p + 15 (page ids from total_tokens / 16 on read zeros). q [n_tokens][heads][D]
+// with zeros past the query's width; out row of a token at out_ld elements, vdim (a multiple of 8) per head. Tiles of 256.
+PIE_API int pie_projected_prefill_attn_tc(const void* q, const void* kv, const int* page_indices, const int* kv_page_indptr,
+                                          const int* qo_indptr, const int* kv_lens, const int* tile_req, const int* tile_qstart,
+                                          int num_tiles, const uint32_t* mask_bits, const long* mask_word_indptr, void* out,
+                                          int n_tokens, int heads, int head_dim, int total_tokens, int vdim, int out_ld,
+                                          float sm_scale, int window_left, int* status, cudaStream_t st) {
+    if (num_tiles <= 0) return 0;
+    const int D_ = head_dim;
+    if ((D_ != 64 && D_ != 128) || vdim > D_ || vdim % 8 || out_ld % 8 || total_tokens % 16 || !status) return (int)cudaErrorInvalidValue;
+    EncodeTiledFnA enc = at_encoder();
+    if (!enc) return (int)cudaErrorNotSupported;
+    CUtensorMap tq, tkv;
+    cuuint32_t estr[3] = {1, 1, 1};
+    cuuint64_t qd[3] = {(cuuint64_t)D_, (cuuint64_t)heads, (cuuint64_t)n_tokens};
+    cuuint64_t qs[2] = {(cuuint64_t)D_ * 2, (cuuint64_t)heads * D_ * 2};
+    cuuint32_t qb[3] = {64, 1, (cuuint32_t)AT_ROWS};
+    cuuint64_t kd[3] = {(cuuint64_t)D_, (cuuint64_t)heads * 2, (cuuint64_t)total_tokens};
+    cuuint64_t ks[2] = {(cuuint64_t)D_ * 2, (cuuint64_t)heads * 2 * D_ * 2};
+    cuuint32_t kb[3] = {64, 1, 16};
+    if (enc(&tq, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 3, const_cast<void*>(q), qd, qs, qb, estr, CU_TENSOR_MAP_INTERLEAVE_NONE,
+            CU_TENSOR_MAP_SWIZZLE_128B, CU_TENSOR_MAP_L2_PROMOTION_L2_256B, CU_TENSOR_MAP_FLOAT_OOB_FILL_NONE) != CUDA_SUCCESS ||
+        enc(&tkv, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 3, const_cast<void*>(kv), kd, ks, kb, estr, CU_TENSOR_MAP_INTERLEAVE_NONE,
+            CU_TENSOR_MAP_SWIZZLE_128B, CU_TENSOR_MAP_L2_PROMOTION_L2_256B, CU_TENSOR_MAP_FLOAT_OOB_FILL_NONE) != CUDA_SUCCESS)
+        return (int)cudaErrorInvalidValue;
+    const float scale_log2 = sm_scale * 1.4426950408889634f;
+    const dim3 grid(num_tiles, heads);
+#define GO(D__)                                                                                                       \
+    {                                                                                                                 \
+        auto kern = paged_prefill_attn_tc_kernel<1, 2, D__, false, true>;                                             \
+        using Cfg = AtCfg<2, D__>;                                                                                    \
+        cudaError_t e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)Cfg::SMEM);      \
+        if (e != cudaSuccess) return (int)e;                                                                          \
+        kern<<<grid, Cfg::THREADS, Cfg::SMEM, st>>>(tq, tkv, page_indices, kv_page_indptr, qo_indptr, kv_lens, tile_req,  \
+                                                    tile_qstart, mask_bits, mask_word_indptr, (bf16*)out, nullptr,    \
+                                                    nullptr, heads, heads, total_tokens / 16, scale_log2, window_left, status,  \
+                                                    0.f, 0.f, out_ld, vdim);                                          \
+        return (int)cudaGetLastError();                                                                               \
+    }
+    if (D_ == 128) GO(128) else GO(64)
+#undef GO
+}

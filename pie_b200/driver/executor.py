@@ -636,7 +636,9 @@ class TorchDriver:
                 mask_indptr = torch.tensor(indptr, dtype=torch.int64, device=self.device)
             plan = ops.PrefillPlan(s.d("page_indices"), s.d("kv_page_indptr"), s.d("qo_indptr"), s.d("kv_lens"),
                                    s.d("tile_req"), s.d("tile_qstart"), nt, self.page_size, mask_bits, mask_indptr,
-                                   window_left=self.window_left, tile_rows=tile_rows)
+                                   window_left=self.window_left, tile_rows=tile_rows,
+                                   host=ops.AttnBatch(np.asarray(req.qo_indptr), np.asarray(req.kv_page_indptr),
+                                                      np.asarray(req.kv_page_indices), kv_lens))
             fi = ForwardInputs(s.d("tokens", n), s.d("positions", n), s.d("slots", n), plan,
                                logit_rows=s.d("logit_rows", len(rows)), is_decode=False,
                                attn_num_pages=len(req.kv_page_indices))

@@ -378,18 +378,18 @@ def _puzutar_dict(cfg: ModelConfig) -> dict:
 
 
 def puzutar_shape(layers: int = 32, width: int = 4096, heads: int = 32, dim: int = 96, rot_dim: int = 32, vdim: int = 128,
-                  kv_rank: int = 256, window: int = 1024, ff: int = 14336, vocab: int = 32000, groups: int = 4,
+                  kv_rank: int = 256, window: int = 1024, ff: int = 21504, vocab: int = 128256, groups: int = 8,
                   side: int = 64, share: int = 2) -> dict:
     """config.json dictionary of a uniform model: of every `share` layers in a row the first keeps latents, the
     others read them."""
     spec = []
     for i in range(layers):
         m = dict(heads=heads, dim=dim, rot_dim=rot_dim, vdim=vdim, kv_rank=kv_rank, scale=(dim + rot_dim) ** -0.5,
-                 mask={"size": window}, rot={"base": 500000.0, "dims": rot_dim})
+                 mask={"size": window}, rot={"base": 10000.0, "dims": rot_dim})
         if i % share:
             m["kv_from"] = i - i % share
         spec.append({"type": "latent_attention", "mixer": m, "mlp": {"kind": "dense", "ff": ff}})
-    return {"architecture": "Puzutar", "width": width, "vocab": vocab, "layers": spec, "norm": {"eps": 1e-6, "groups": groups},
+    return {"architecture": "Puzutar", "width": width, "vocab": vocab, "layers": spec, "norm": {"eps": 1e-5, "groups": groups},
             "token_side": {"dim": side}}
 
 
@@ -435,6 +435,10 @@ PRESETS = {
     "llama-3.1-8b": dict(model_type="llama", hidden_size=4096, intermediate_size=14336,
                          num_hidden_layers=32, num_attention_heads=32, num_key_value_heads=8,
                          head_dim=128, vocab_size=128256, rope_theta=500000.0, rms_norm_eps=1e-5),
+    # the 8B shape with a sliding window: what `puzutar-8b` is measured beside
+    "llama-8b-window": dict(model_type="mistral", hidden_size=4096, intermediate_size=14336, num_hidden_layers=32,
+                            num_attention_heads=32, num_key_value_heads=8, head_dim=128, vocab_size=128256,
+                            rope_theta=500000.0, rms_norm_eps=1e-5, sliding_window=1024),
     "qwen3-32b": dict(model_type="qwen3", hidden_size=5120, intermediate_size=25600,
                       num_hidden_layers=64, num_attention_heads=64, num_key_value_heads=8, head_dim=128,
                       vocab_size=151936, rope_theta=1000000.0, rms_norm_eps=1e-6, qk_norm=True),

@@ -5,8 +5,9 @@ per-layer token input, x += RMSNorm(W_proj (gelu(W_gate x) * e)). The norm of a 
 the layer before (`LatentStream` carries what is pending), and the products that end both sublayers run as one GEMM over
 their inputs side by side.
 
-Latent attention runs in its absorbed form: with W_uk folded into the query and W_uv applied to the result, keys and
+Latent attention decodes in its absorbed form: with W_uk folded into the query and W_uv applied to the result, keys and
 values of every head are the cached rows themselves, so that a step reads one row per token whatever the head count.
+Prefill has many queries per key: it projects keys and values out of the visible latents and runs on the tcgen05 kernel.
 """
 from __future__ import annotations
 
@@ -51,6 +52,14 @@ def prepare_latent(m) -> None:
         lw["w_uk_t"] = lw["w_uk"].view(s.heads, s.dim, s.kv_rank).transpose(1, 2).contiguous()
         uv = lw["w_uv"].view(s.heads, s.vdim, s.kv_rank)
         lw["w_uv_p"] = torch.nn.functional.pad(uv, (0, s.rank_pad - s.kv_rank)).contiguous()
+        d = lops.projected_width(s)
+        if m.device.type == "cuda" and m.dtype == torch.bfloat16 and d:
+            # cache row -> (key | value) of every head, D columns each; the rotated key part is copied by a unit block
+            w = torch.zeros(s.heads, 2, d, s.row, dtype=m.dtype, device=m.device)
+            w[:, 0, :s.dim, :s.kv_rank] = lw["w_uk"].view(s.heads, s.dim, s.kv_rank)
+            w[:, 0, s.dim:s.qk_dim, s.rank_pad:s.rank_pad + s.rot_dim] = torch.eye(s.rot_dim, dtype=m.dtype, device=m.device)
+            w[:, 1, :s.vdim, :s.kv_rank] = uv
+            lw["w_kv_row"] = w.view(-1, s.row)
 
 
 def latent_mixer(m, hs, lw: dict, li: int, fi, cache, out) -> None:
@@ -59,6 +68,12 @@ def latent_mixer(m, hs, lw: dict, li: int, fi, cache, out) -> None:
     page = cache.shape[2]
     layer_cache = cache[m.cache_index[li]]
     qkv = m._gemm(hs, lw["w_latent_in"])
+    if "w_kv_row" in lw and not fi.is_decode and fi.attn.mask_bits is None and page % 16 == 0:
+        q = lops.latent_rows(qkv, fi.positions, fi.slots, lw["rope"], lw.get("latent_norm"),
+                             layer_cache if s.kv_from is None else None, s, m.cfg.rms_norm_eps, lops.projected_width(s), s.dim,
+                             copy_nope=True)
+        lops.projected_prefill_attention(q, layer_cache, fi.attn, lw["w_kv_row"], s, page, s.window - 1, out)
+        return
     q = lops.latent_rows(qkv, fi.positions, fi.slots, lw["rope"], lw.get("latent_norm"), layer_cache if s.kv_from is None else None,
                          s, m.cfg.rms_norm_eps, s.row, s.rank_pad, copy_nope=False)
     nope = qkv[:, :s.q_rows].view(n, s.heads, s.qk_dim)[..., :s.dim] if qkv.shape[1] == s.q_rows else \

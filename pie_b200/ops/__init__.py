@@ -859,6 +859,8 @@ class PrefillPlan:
     mask_word_indptr: Optional[torch.Tensor] = None
     window_left: int = -1
     tile_rows: int = 64           # 128 / 256: tiles planned for the tcgen05 kernel
+    host: Optional[AttnBatch] = None        # the same batch on the host, and what a model's layers derive from it
+    derived: dict = field(default_factory=dict)
 
 
 def paged_prefill_attention(q, kv_layer, plan: PrefillPlan, sm_scale: float, out=None, lse_out=None,

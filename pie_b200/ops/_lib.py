@@ -65,6 +65,10 @@ _SIGNATURES = {
     "pie_stream_norm": [p, i32, i32, p],
     "pie_latent_rows": [p, i32, p],
     "pie_latent_attn_warp": [p, i32, p],
+    "pie_latent_attn_mma_tiles": [i32, i32, i32],
+    "pie_latent_attn_mma": [p, i32, p],
+    "pie_per_head": [p, p],
+    "pie_projected_prefill_attn_tc": [p, p, p, p, p, p, p, p, i32, p, p, p, i32, i32, i32, i32, i32, i32, f32, i32, p, p],
     "pie_bias_xielu": [p, i32, p, p, i32, i32, i32, p],
     "pie_stream_add": [p, p, p, p, p, i32, i32, i32, p],
     "pie_side_gate": [p, i32, p, i32, p, p, i32, i32, i32, i32, i32, i32, p],

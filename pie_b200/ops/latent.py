@@ -4,21 +4,22 @@ go to `csrc/kernels/latent*.cu` (bf16 when serving, float32 on the 32-bit path),
 from __future__ import annotations
 
 import ctypes as C
-from typing import Optional
 
+import numpy as np
 import torch
 
-from . import _lib, latent_reference as ref
+from .. import ops
+from . import latent_reference as ref
 from ._lib import check, fn, ptr, stream_ptr
 
-p, i32, f32 = C.c_void_p, C.c_int, C.c_float
+p, i32, i64, f32 = C.c_void_p, C.c_int, C.c_long, C.c_float
 
 
 def _struct(name: str, *fields):
     return type(name, (C.Structure,), {"_fields_": [(n, t) for names, t in fields for n in names.split()]})
 
 
-# mirrors of the argument structs in csrc/kernels/latent.cu
+# mirrors of the argument structs in csrc/kernels/latent.cu and latent_attn.cu
 StreamNormArgs = _struct("StreamNormArgs", ("x y y_norm x_out norm_w shift h hs tok_req qo_indptr slots reset state stage", p),
                          ("n width ldx ldy ldh groups rows_per_block", i32), ("eps", f32))
 LatentRowsArgs = _struct("LatentRowsArgs", ("qkv positions slots inv_freq norm_w q_out cache", p),
@@ -26,6 +27,11 @@ LatentRowsArgs = _struct("LatentRowsArgs", ("qkv positions slots inv_freq norm_w
 LatentAttnArgs = _struct("LatentAttnArgs", ("q cache page_indices kv_page_indptr qo_indptr kv_lens tok_req slots mask_bits "
                                             "mask_word_indptr out", p),
                          ("n heads row rank_pad cache_row page_size window_left", i32), ("scale", f32))
+
+LatentMmaArgs = _struct("LatentMmaArgs", ("q cache page_indices kv_page_indptr item_req item_start item_end req_item_indptr "
+                                          "num_items qo_indptr kv_lens mask_bits mask_word_indptr out scratch", p),
+                        ("items max_items heads row rank_pad cache_row page_size window_left stages reqs", i32), ("scale_log2", f32))
+PerHeadArgs = _struct("PerHeadArgs", ("x w out", p), ("x_tok x_head out_tok out_head", i64), ("n heads m k", i32))
 
 
 def _f32(t) -> int:
@@ -92,23 +98,94 @@ def per_head(x, w, out):
     if not x.is_cuda or x.dtype == torch.float32:
         out.copy_(torch.bmm(x.transpose(0, 1), w.transpose(1, 2)).transpose(0, 1))
         return out
-    out.copy_(torch.bmm(x.transpose(0, 1), w.transpose(1, 2)).transpose(0, 1))
+    n, heads, k = x.shape
+    a = PerHeadArgs(x=ptr(x), w=ptr(w), out=ptr(out), x_tok=x.stride(0), x_head=x.stride(1), out_tok=out.stride(0),
+                    out_head=out.stride(1), n=n, heads=heads, m=w.shape[1], k=k)
+    check(fn("pie_per_head")(C.byref(a), stream_ptr()), "per_head")
     return out
 
 
 def latent_attention(q, cache, plan, rs, slots, spec, page_size: int, window_left: int):
     """Softmax over the visible cache rows of q [N, heads, row] . row * scale; returns the weighted latents
-    [N, heads, rank_pad]. The absorbed form: keys and values of every head are the rows themselves."""
+    [N, heads, rank_pad]. The absorbed form: keys and values of every head are the rows themselves. Decode splits a
+    request's keys over the plan's work items."""
     if not q.is_cuda:
         return ref.latent_attention(q, cache, plan, spec, window_left)
     n = q.shape[0]
     out = torch.empty(n, spec.heads, spec.rank_pad, dtype=q.dtype, device=q.device)
-    a = LatentAttnArgs(q=ptr(q), cache=ptr(cache), page_indices=ptr(plan.page_indices), kv_page_indptr=ptr(plan.kv_page_indptr),
-                       qo_indptr=ptr(rs.qo_indptr), kv_lens=ptr(plan.kv_lens), tok_req=ptr(rs.tok_req), slots=ptr(slots),
-                       mask_bits=ptr(getattr(plan, "mask_bits", None)), mask_word_indptr=ptr(getattr(plan, "mask_word_indptr", None)),
-                       out=ptr(out), n=n, heads=spec.heads, row=q.shape[2], rank_pad=spec.rank_pad, cache_row=cache.shape[-1],
-                       page_size=page_size, window_left=window_left, scale=spec.scale)
-    check(fn("pie_latent_attn_warp")(C.byref(a), _f32(q), stream_ptr()), "latent_attn_warp")
+    decode = isinstance(plan, ops.DecodePlan)
+    tiles = fn("pie_latent_attn_mma_tiles")(spec.heads, spec.row, spec.rank_pad) if q.dtype == torch.bfloat16 else 0
+    if not tiles:           # 32-bit, or a latent wider than the tensor-core kernel takes
+        a = LatentAttnArgs(q=ptr(q), cache=ptr(cache), page_indices=ptr(plan.page_indices), kv_page_indptr=ptr(plan.kv_page_indptr),
+                           qo_indptr=ptr(rs.qo_indptr), kv_lens=ptr(plan.kv_lens), tok_req=ptr(rs.tok_req), slots=ptr(slots),
+                           mask_bits=ptr(getattr(plan, "mask_bits", None)),
+                           mask_word_indptr=ptr(getattr(plan, "mask_word_indptr", None)), out=ptr(out), n=n, heads=spec.heads,
+                           row=q.shape[2], rank_pad=spec.rank_pad, cache_row=cache.shape[-1], page_size=page_size,
+                           window_left=window_left, scale=spec.scale)
+        check(fn("pie_latent_attn_warp")(C.byref(a), _f32(q), stream_ptr()), "latent_attn_warp")
+        return out
+    a = LatentMmaArgs(q=ptr(q), cache=ptr(cache), page_indices=ptr(plan.page_indices), kv_page_indptr=ptr(plan.kv_page_indptr),
+                      qo_indptr=ptr(rs.qo_indptr), kv_lens=ptr(plan.kv_lens), out=ptr(out), heads=spec.heads, row=spec.row,
+                      rank_pad=spec.rank_pad, cache_row=cache.shape[-1], page_size=page_size, window_left=window_left,
+                      reqs=len(rs.slots_host), scale_log2=spec.scale * 1.4426950408889634)
+    ctas = ops.num_sms(q.device) * 2
+    if decode:
+        a.item_req, a.item_start, a.item_end = ptr(plan.item_req), ptr(plan.item_start), ptr(plan.item_end)
+        a.req_item_indptr, a.num_items, a.scratch = ptr(plan.req_item_indptr), ptr(plan.num_items), ptr(plan.scratch)
+        a.max_items = plan.max_items
+    else:
+        key, rows = ("absorbed", spec.heads), 16 * tiles
+        if key not in plan.derived:
+            tr, tqs = ops.plan_prefill_tiles(plan.host.qo_indptr, 1, max(1, rows // min(spec.heads, rows)), plan.host.kv_lens)
+            plan.derived[key] = torch.from_numpy(np.stack([tr, tqs]).astype(np.int32)).to(q.device)
+        t = plan.derived[key]
+        a.item_req, a.item_start, a.items, a.max_items = ptr(t[0]), ptr(t[1]), t.shape[1], t.shape[1]
+        a.mask_bits, a.mask_word_indptr = ptr(plan.mask_bits), ptr(plan.mask_word_indptr)
+        ctas = t.shape[1]
+    check(fn("pie_latent_attn_mma")(C.byref(a), ctas, stream_ptr()), "latent_attn_mma")
+    return out
+
+
+def projected_width(spec) -> int:
+    """Head width of the prefill kernel that takes this mixer's keys and values projected out of the latents; 0: none."""
+    need = max(spec.qk_dim, spec.vdim)
+    return 0 if need > 128 or spec.vdim % 8 else (64 if need <= 64 else 128)
+
+
+def _projected_context(plan, window_left: int, page_size: int, device):
+    """Rows of the cache that a prefill's tokens can see, in 16-token pieces: (cache pieces to gather, page table of the
+    gathered copy, its page indptr, key counts), as one int32 device tensor sliced up. Keys before a request's window
+    are left out, so every count is relative to the first piece kept."""
+    h = plan.host
+    qlens, kv = np.diff(h.qo_indptr), np.asarray(h.kv_lens, dtype=np.int64)
+    lo = np.maximum(0, kv - qlens - window_left) // 16
+    hi = -(-kv // 16)
+    per = page_size // 16
+    pieces = [np.asarray(h.page_indices[h.kv_page_indptr[r] + np.arange(lo[r], hi[r]) // per], np.int64) * per + np.arange(lo[r], hi[r]) % per
+              for r in range(len(kv))]
+    flat = np.concatenate(pieces)
+    indptr = np.concatenate([[0], np.cumsum(hi - lo)])
+    buf = torch.from_numpy(np.concatenate([flat, np.arange(len(flat)), indptr, kv - lo * 16]).astype(np.int32)).to(device)
+    return buf.split([len(flat), len(flat), len(indptr), len(kv)])
+
+
+def projected_prefill_attention(q, cache, plan, w_kv, spec, page_size: int, window_left: int, out):
+    """Prefill attention on keys and values projected from the visible latents for this pass: one GEMM (the shared rotated
+    key part passes through it on a unit block) gives [tokens, heads, 2, D], which the tcgen05 kernel reads in place.
+    q [N, heads, D] = (unrotated | rotated | zeros); out [N, heads * vdim], may be a column range."""
+    key = ("projected", window_left)
+    if key not in plan.derived:
+        if plan.mask_bits is not None:
+            raise ValueError("custom masks index keys of the whole context")
+        plan.derived[key] = _projected_context(plan, window_left, page_size, q.device)
+    src, table, indptr, kv_lens = plan.derived[key]
+    row, d = cache.shape[-1], q.shape[2]
+    rows = ops.gather_rows(cache.view(-1, 16 * row), src).view(-1, row)
+    kv = ops.gemm(rows[:, :spec.row], w_kv)
+    check(fn("pie_projected_prefill_attn_tc")(
+        ptr(q), ptr(kv), ptr(table), ptr(indptr), ptr(plan.qo_indptr), ptr(kv_lens), ptr(plan.tile_req), ptr(plan.tile_qstart),
+        plan.num_tiles, None, None, ptr(out), q.shape[0], spec.heads, d, rows.shape[0], spec.vdim, out.stride(0), spec.scale,
+        window_left, ptr(ops.kernel_status(q.device)), stream_ptr()), "projected_prefill_attn_tc")
     return out
 
 
