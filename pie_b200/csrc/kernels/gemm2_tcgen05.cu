@@ -32,7 +32,7 @@ template <int BN, int EPI>
 __global__ void __cluster_dims__(2, 1, 1) __launch_bounds__(GEMM_THREADS, 1)
 gemm2_bf16_kernel(const __grid_constant__ CUtensorMap tma_a, const __grid_constant__ CUtensorMap tma_b,
                   bf16* __restrict__ C, const bf16* __restrict__ R, int M, int N, int K, int ldc, int ldr,
-                  int* status, const __grid_constant__ TpArgs tp, const StreamKArgs sk) {
+                  int* status, const __grid_constant__ TpArgs tp, const StreamKArgs sk, const __grid_constant__ EpiArgs ex) {
     using Cfg = Gemm2Cfg<BN>;
     constexpr int STAGES = Cfg::STAGES;
     constexpr int PAIR_M = 2 * GEMM_BM;
@@ -181,6 +181,7 @@ gemm2_bf16_kernel(const __grid_constant__ CUtensorMap tma_a, const __grid_consta
         SegmentWalk walk(sk.enabled != 0, num_tiles, num_kb, pid, npairs);
         Segment seg;
         const long long total_units = (long long)num_tiles * num_kb;
+        const XieluCoef act(EPI == EPI_XIELU ? ex.act : nullptr);
         const uint32_t leader_tempty0 = map_to_cta(tempty_bar(0), 0);
         const uint32_t leader_tempty1 = map_to_cta(tempty_bar(1), 0);
         for (; walk.next(seg); ++tcount) {
@@ -255,7 +256,7 @@ gemm2_bf16_kernel(const __grid_constant__ CUtensorMap tma_a, const __grid_consta
                         }
                     }
                     epilogue_store_64<EPI>(v0, v1, stage, m_blk * PAIR_M + (int)crank * GEMM_BM + q * 32,
-                                           n_blk * BN + c * 64, M, N, C, ldc, R, ldr, tp, N);
+                                           n_blk * BN + c * 64, M, N, C, ldc, R, ldr, tp, N, ex, &act);
                 }
             }
             tc_fence_before();
@@ -313,14 +314,14 @@ extern "C" __attribute__((visibility("default"))) int pie_gemm_set_pair_threshol
 template <int BN, int EPI>
 static int launch_gemm2(const CUtensorMap& ta, const CUtensorMap& tb, void* C, const void* R, int M, int N,
                         int K, int ldc, int ldr, int* status, int pairs, int streamk, float* ws, int* cnt,
-                        cudaStream_t st, const TpArgs& tp) {
+                        cudaStream_t st, const TpArgs& tp, const EpiArgs& ex) {
     using Cfg = Gemm2Cfg<BN>;
     auto kern = gemm2_bf16_kernel<BN, EPI>;
     cudaError_t e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)Cfg::SMEM_BYTES);
     if (e != cudaSuccess) return (int)e;
     StreamKArgs sk{ws, cnt, streamk, g_pair_dbg};
     kern<<<2 * pairs, GEMM_THREADS, Cfg::SMEM_BYTES, st>>>(ta, tb, (bf16*)C, (const bf16*)R, M, N, K, ldc, ldr,
-                                                           status, tp, sk);
+                                                           status, tp, sk, ex);
     return (int)cudaGetLastError();
 }
 
@@ -328,7 +329,7 @@ static int launch_gemm2(const CUtensorMap& ta, const CUtensorMap& tb, void* C, c
 // when the shape is better served by the single-CTA kernel.
 int pie_gemm2_dispatch(const void* A, const void* W, void* C, const void* R, int M, int N, int K, int lda,
                        int ldw, int ldc, int ldr, int epilogue, int* status, int num_sms, cudaStream_t st,
-                       const TpArgs* tp_in, float* ws, long ws_floats, int* cnt, int cnt_ints, int* handled) {
+                       const TpArgs* tp_in, float* ws, long ws_floats, int* cnt, int cnt_ints, int* handled, const EpiArgs& ex) {
     *handled = 0;
     // small problems are launch/fix-up bound: the single-CTA kernel's narrower tiles fill the machine
     // better. Measured cross-over on B200 (M = 256 / 512 decode shapes): pairs win from 2e10 MACs,
@@ -358,10 +359,12 @@ int pie_gemm2_dispatch(const void* A, const void* W, void* C, const void* R, int
     *handled = 1;
 #define GO(BN_)                                                                                                     \
     switch (epilogue) {                                                                                             \
-        case EPI_STORE: return launch_gemm2<BN_, EPI_STORE>(ta, tb, C, R, M, N, K, ldc, ldr, status, pairs, streamk, ws, cnt, st, tp);       \
-        case EPI_RESIDUAL: return launch_gemm2<BN_, EPI_RESIDUAL>(ta, tb, C, R, M, N, K, ldc, ldr, status, pairs, streamk, ws, cnt, st, tp); \
-        case EPI_SWIGLU: return launch_gemm2<BN_, EPI_SWIGLU>(ta, tb, C, R, M, N, K, ldc, ldr, status, pairs, streamk, ws, cnt, st, tp);     \
-        case EPI_RS: return launch_gemm2<BN_, EPI_RS>(ta, tb, C, R, M, N, K, ldc, ldr, status, pairs, streamk, ws, cnt, st, tp);             \
+        case EPI_STORE: return launch_gemm2<BN_, EPI_STORE>(ta, tb, C, R, M, N, K, ldc, ldr, status, pairs, streamk, ws, cnt, st, tp, ex);       \
+        case EPI_RESIDUAL: return launch_gemm2<BN_, EPI_RESIDUAL>(ta, tb, C, R, M, N, K, ldc, ldr, status, pairs, streamk, ws, cnt, st, tp, ex); \
+        case EPI_SWIGLU: return launch_gemm2<BN_, EPI_SWIGLU>(ta, tb, C, R, M, N, K, ldc, ldr, status, pairs, streamk, ws, cnt, st, tp, ex);     \
+        case EPI_XIELU: return launch_gemm2<BN_, EPI_XIELU>(ta, tb, C, R, M, N, K, ldc, ldr, status, pairs, streamk, ws, cnt, st, tp, ex); \
+        case EPI_STREAM: return launch_gemm2<BN_, EPI_STREAM>(ta, tb, C, R, M, N, K, ldc, ldr, status, pairs, streamk, ws, cnt, st, tp, ex); \
+        case EPI_RS: return launch_gemm2<BN_, EPI_RS>(ta, tb, C, R, M, N, K, ldc, ldr, status, pairs, streamk, ws, cnt, st, tp, ex);             \
         default: *handled = 0; return (int)cudaErrorInvalidValue;                                                   \
     }
     if (bn == 256) { GO(256) } else if (bn == 128) { GO(128) } else { GO(64) }

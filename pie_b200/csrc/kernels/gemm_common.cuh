@@ -14,11 +14,36 @@ enum GemmEpilogue : int {
     EPI_RESIDUAL = 1,  // C = acc + R
     EPI_SWIGLU = 2,    // C[:, j] = silu(acc[:, 2j]) * acc[:, 2j+1]   (C is [M, N/2])
     EPI_RS = 3,        // reduce-scatter: rows go to their owner rank's receive buffer (peer stores)
+    EPI_XIELU = 4,     // C = xIELU(acc + bias), see EpiArgs
+    EPI_STREAM = 5,    // out32 = res32 + acc + bias: a 32-bit residual stream; C = the same in bf16
     // Swapped operands (small batches): the kernel computes C^T = W * A^T, so its rows are output
     // features and its columns tokens; these epilogues write the tile back transposed.
-    EPI_STORE_T = 4,
-    EPI_RESIDUAL_T = 5,
-    EPI_SWIGLU_T = 6,
+    EPI_STORE_T = 6,
+    EPI_RESIDUAL_T = 7,
+    EPI_SWIGLU_T = 8,
+    EPI_XIELU_T = 9,
+    EPI_STREAM_T = 10,
+};
+
+// Operands of the epilogues with a bias. xIELU(z) = a z^2 + z / 2 for z > 0, b (e^z - 1 - z) + z / 2 below, with
+// a = softplus(act[0]) and b = 1/2 + softplus(act[1]).
+struct EpiArgs {
+    const bf16* bias = nullptr;    // [N], or null
+    const bf16* act = nullptr;     // the activation's two learned numbers
+    const float* res32 = nullptr;  // [M, ld32]; may be out32 itself
+    float* out32 = nullptr;
+    int ld32 = 0;
+};
+
+struct XieluCoef {
+    float a, b;
+    __device__ explicit XieluCoef(const bf16* act) {
+        auto sp = [](float z) { return log1pf(__expf(-fabsf(z))) + fmaxf(z, 0.f); };
+        a = act ? sp(__bfloat162float(act[0])) : 0.f;
+        b = act ? 0.5f + sp(__bfloat162float(act[1])) : 0.f;
+    }
+    // the result is rounded to bf16: e^z - 1 - z loses digits near zero only, where z / 2 outweighs it
+    __device__ float operator()(float z) const { return (z > 0.f ? a * z * z : b * (__expf(z) - 1.f - z)) + 0.5f * z; }
 };
 
 constexpr int TP_MAX_RANKS = 8;
@@ -180,7 +205,8 @@ template <int EPI>
 __device__ __forceinline__ void epilogue_store_64(const uint32_t (&v0)[32], const uint32_t (&v1)[32],
                                                   uint8_t* stage, int row0, int col0, int M, int N,
                                                   bf16* __restrict__ C, int ldc, const bf16* __restrict__ R,
-                                                  int ldr, const TpArgs& tp, int n_end) {
+                                                  int ldr, const TpArgs& tp, int n_end, const EpiArgs& ex = EpiArgs(),
+                                                  const XieluCoef* act = nullptr) {
     const int lane = threadIdx.x & 31;
     auto slot = [&](int r, int c) { return reinterpret_cast<bf16x8*>(stage + r * 128 + ((c ^ (r & 7)) << 4)); };
     if (EPI == EPI_SWIGLU) {
@@ -206,6 +232,47 @@ __device__ __forceinline__ void epilogue_store_64(const uint32_t (&v0)[32], cons
         __syncwarp();
         return;
     }
+    float f[64];                       // the 64 values of this thread's row (EPI_XIELU, EPI_STREAM)
+    if constexpr (EPI == EPI_XIELU || EPI == EPI_STREAM) {
+#pragma unroll
+        for (int c = 0; c < 8; ++c) {
+            float b[8] = {0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f};
+            if (ex.bias && col0 + c * 8 < n_end) unpack8(*reinterpret_cast<const bf16x8*>(ex.bias + col0 + c * 8), b);
+#pragma unroll
+            for (int e = 0; e < 8; ++e) {
+                f[8 * c + e] = __uint_as_float(c < 4 ? v0[8 * c + e] : v1[8 * (c - 4) + e]) + b[e];
+                if (EPI == EPI_XIELU) f[8 * c + e] = (*act)(f[8 * c + e]);
+            }
+        }
+    }
+    if constexpr (EPI == EPI_STREAM) {
+        // 32 columns (128 bytes of a 32-bit row) at a time through the staging tile, in and out
+        auto slot4 = [&](int r, int c) { return reinterpret_cast<float4*>(stage + r * 128 + ((c ^ (r & 7)) << 4)); };
+#pragma unroll
+        for (int half = 0; half < 2; ++half) {
+#pragma unroll
+            for (int i = 0; i < 8; ++i) {
+                const int r = i * 4 + (lane >> 3), c = lane & 7, row = row0 + r, col = col0 + half * 32 + c * 4;
+                if (row < M && col < n_end) *slot4(r, c) = *reinterpret_cast<const float4*>(ex.res32 + (size_t)row * ex.ld32 + col);
+            }
+            __syncwarp();
+#pragma unroll
+            for (int c = 0; c < 8; ++c) {
+                const float4 x = *slot4(lane, c);
+                float* y = f + half * 32 + c * 4;
+                y[0] += x.x; y[1] += x.y; y[2] += x.z; y[3] += x.w;
+                *slot4(lane, c) = make_float4(y[0], y[1], y[2], y[3]);
+            }
+            __syncwarp();
+#pragma unroll
+            for (int i = 0; i < 8; ++i) {
+                const int r = i * 4 + (lane >> 3), c = lane & 7, row = row0 + r, col = col0 + half * 32 + c * 4;
+                if (row < M && col < n_end) *reinterpret_cast<float4*>(ex.out32 + (size_t)row * ex.ld32 + col) = *slot4(r, c);
+            }
+            __syncwarp();
+        }
+        if (!C) return;
+    }
     if (EPI == EPI_RESIDUAL) {
         // bring the residual tile in with coalesced loads, add in fp32 on the owning thread
 #pragma unroll
@@ -224,7 +291,8 @@ __device__ __forceinline__ void epilogue_store_64(const uint32_t (&v0)[32], cons
     for (int c = 0; c < 8; ++c) {
         float o[8];
 #pragma unroll
-        for (int e = 0; e < 8; ++e) o[e] = __uint_as_float(c < 4 ? v0[8 * c + e] : v1[8 * (c - 4) + e]);
+        for (int e = 0; e < 8; ++e)
+            o[e] = (EPI == EPI_XIELU || EPI == EPI_STREAM) ? f[8 * c + e] : __uint_as_float(c < 4 ? v0[8 * c + e] : v1[8 * (c - 4) + e]);
         if (EPI == EPI_RESIDUAL) {
             float rr[8];
             unpack8(*slot(lane, c), rr);
@@ -262,7 +330,7 @@ template <int EPI>
 __device__ __forceinline__ void epilogue_store_64_t(const uint32_t (&v0)[32], const uint32_t (&v1)[32],
                                                     uint8_t* stage, int feat0, int tok0, int F, int tok_end,
                                                     bf16* __restrict__ C, int ldc, const bf16* __restrict__ R,
-                                                    int ldr) {
+                                                    int ldr, const EpiArgs& ex = EpiArgs(), const XieluCoef* act = nullptr) {
     const int lane = threadIdx.x & 31;
     bf16* st = reinterpret_cast<bf16*>(stage);
     const int feat = feat0 + lane;
@@ -286,9 +354,34 @@ __device__ __forceinline__ void epilogue_store_64_t(const uint32_t (&v0)[32], co
         __syncwarp();
         return;
     }
+    float bias = 0.f;
+    if constexpr (EPI == EPI_XIELU_T || EPI == EPI_STREAM_T) bias = ex.bias && feat < F ? __bfloat162float(ex.bias[feat]) : 0.f;
+    if constexpr (EPI == EPI_STREAM_T) {
+        // the warp's 32 features of a token are 128 bytes of its stream row; all loads of a batch leave before its stores,
+        // which may be to the same addresses
+#pragma unroll
+        for (int b = 0; b < 4; ++b) {
+            float x[16];
+#pragma unroll
+            for (int i = 0; i < 16; ++i) {
+                const int tok = tok0 + b * 16 + i;
+                x[i] = tok < tok_end && feat < F ? ex.res32[(size_t)tok * ex.ld32 + feat] : 0.f;
+            }
+#pragma unroll
+            for (int i = 0; i < 16; ++i) {
+                const int t = b * 16 + i, tok = tok0 + t;
+                x[i] += __uint_as_float(t < 32 ? v0[t] : v1[t - 32]) + bias;
+                if (tok < tok_end && feat < F) ex.out32[(size_t)tok * ex.ld32 + feat] = x[i];
+                st[t * 32 + lane] = __float2bfloat16(x[i]);
+            }
+        }
+        if (!C) return;
+    }
 #pragma unroll
     for (int t = 0; t < 64; ++t) {
+        if constexpr (EPI == EPI_STREAM_T) break;
         float o = __uint_as_float(t < 32 ? v0[t] : v1[t - 32]);
+        if constexpr (EPI == EPI_XIELU_T) o = (*act)(o + bias);
         if (EPI == EPI_RESIDUAL_T) {
             const int tok = tok0 + t;
             if (tok < tok_end && feat < F) o += __bfloat162float(R[(size_t)tok * ldr + feat]);

@@ -53,7 +53,7 @@ __global__ void __launch_bounds__(GEMM_THREADS, OCC)
 gemm_bf16_kernel(const __grid_constant__ CUtensorMap tma_a, const __grid_constant__ CUtensorMap tma_b,
                  bf16* __restrict__ C, const bf16* __restrict__ R, int M, int N, int K, int ldc,
                  int ldr, int* status, const __grid_constant__ TpArgs tp, const StreamKArgs sk,
-                 const int* __restrict__ tile_expert, int bn) {
+                 const int* __restrict__ tile_expert, int bn, const __grid_constant__ EpiArgs ex) {
     using Cfg = GemmCfg<BN, OCC>;
     constexpr int STAGES = Cfg::STAGES;
     constexpr bool SWAPPED = EPI >= EPI_STORE_T;   // tma_a walks the weights, tma_b the activation
@@ -241,6 +241,7 @@ gemm_bf16_kernel(const __grid_constant__ CUtensorMap tma_a, const __grid_constan
         SegmentWalk walk(sk.enabled != 0, num_tiles, num_kb, blockIdx.x, gridDim.x);
         Segment seg;
         const long long total_units = (long long)num_tiles * num_kb;
+        const XieluCoef act((EPI == EPI_XIELU || EPI == EPI_XIELU_T) ? ex.act : nullptr);
         for (; walk.next(seg); ++tcount) {
             const int m_blk = seg.tile % tiles_m, n_blk = seg.tile / tiles_m;
             if (GROUPED && tile_expert[m_blk] < 0) { --tcount; continue; }
@@ -318,10 +319,10 @@ gemm_bf16_kernel(const __grid_constant__ CUtensorMap tma_a, const __grid_constan
                     }
                     if constexpr (EPI >= EPI_STORE_T)
                         epilogue_store_64_t<EPI>(v0, v1, stage, m_blk * GEMM_BM + q * 32, n_blk * bn + c * 64, M,
-                                                 min(N, (n_blk + 1) * bn), C, ldc, R, ldr);
+                                                 min(N, (n_blk + 1) * bn), C, ldc, R, ldr, ex, &act);
                     else
                         epilogue_store_64<EPI>(v0, v1, stage, m_blk * GEMM_BM + q * 32, n_blk * bn + c * 64, M, N, C,
-                                               ldc, R, ldr, tp, min(N, (n_blk + 1) * bn));
+                                               ldc, R, ldr, tp, min(N, (n_blk + 1) * bn), ex, &act);
                 }
             }
             tc_fence_before();
@@ -448,7 +449,8 @@ PIE_API int pie_gemm_set_swap(int max_m) { g_gemm_swap_max_m = max_m; return 0; 
 
 int pie_gemm2_dispatch(const void* A, const void* W, void* C, const void* R, int M, int N, int K, int lda,
                        int ldw, int ldc, int ldr, int epilogue, int* status, int num_sms, cudaStream_t st,
-                       const TpArgs* tp_in, float* ws, long ws_floats, int* cnt, int cnt_ints, int* handled);
+                       const TpArgs* tp_in, float* ws, long ws_floats, int* cnt, int cnt_ints, int* handled,
+                       const EpiArgs& ex = EpiArgs());
 
 struct GemmPlan {
     int bn;        // tile width of the launch (multiple of 16)
@@ -544,7 +546,7 @@ PIE_API int pie_gemm_plan(int M, int N, int K, int num_sms, int with_workspace, 
 template <int BN, int EPI>
 static int launch_gemm(const CUtensorMap& ta, const CUtensorMap& tb, void* C, const void* R, int M,
                        int N, int K, int ldc, int ldr, int* status, const GemmPlan& plan,
-                       const GemmWorkspace& w, cudaStream_t st, const TpArgs& tp = TpArgs{}) {
+                       const GemmWorkspace& w, cudaStream_t st, const TpArgs& tp = TpArgs{}, const EpiArgs& ex = EpiArgs()) {
     using Cfg = GemmCfg<BN>;
     auto kern = gemm_bf16_kernel<BN, EPI>;
     cudaError_t e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize,
@@ -552,7 +554,7 @@ static int launch_gemm(const CUtensorMap& ta, const CUtensorMap& tb, void* C, co
     if (e != cudaSuccess) return (int)e;
     StreamKArgs sk{w.ws, w.cnt, plan.streamk, g_gemm_dbg, g_gemm_trace};
     e = launch_pdl(kern, dim3(plan.grid), dim3(GEMM_THREADS), Cfg::SMEM_BYTES, st, ta, tb, (bf16*)C, (const bf16*)R,
-                   M, N, K, ldc, ldr, status, tp, sk, (const int*)nullptr, plan.bn);
+                   M, N, K, ldc, ldr, status, tp, sk, (const int*)nullptr, plan.bn, ex);
     return (int)(e != cudaSuccess ? e : cudaGetLastError());
 }
 
@@ -566,9 +568,8 @@ static int current_workspace(GemmWorkspace* out) {
 
 // C[M,N] (or [M,N/2] for the SwiGLU epilogue) = A[M,K] * W[N,K]^T.
 // `status` is a device int that stays 0 unless a bounded wait ran out.
-PIE_API int pie_gemm_bf16(const void* A, const void* W, void* C, const void* R, int M, int N, int K,
-                          int lda, int ldw, int ldc, int ldr, int epilogue, int force_bn,
-                          int* status, int num_sms, cudaStream_t st) {
+static int gemm_bf16(const void* A, const void* W, void* C, const void* R, int M, int N, int K, int lda, int ldw, int ldc, int ldr,
+                     int epilogue, int force_bn, int* status, int num_sms, cudaStream_t st, const EpiArgs& ex) {
     if (M <= 0 || N <= 0) return 0;
     if (K <= 0 || K % 8 || N % 8 || ldc % 8 || (epilogue == EPI_RESIDUAL && ldr % 8))
         return (int)cudaErrorInvalidValue;
@@ -578,7 +579,7 @@ PIE_API int pie_gemm_bf16(const void* A, const void* W, void* C, const void* R, 
     if (g_gemm_pairs && force_bn == 0) {
         int handled = 0;
         const int rc = pie_gemm2_dispatch(A, W, C, R, M, N, K, lda, ldw, ldc, ldr, epilogue, status, num_sms, st,
-                                          nullptr, w.ws, w.ws_floats, w.cnt, w.cnt_ints, &handled);
+                                          nullptr, w.ws, w.ws_floats, w.cnt, w.cnt_ints, &handled, ex);
         if (handled || rc) return rc;
     }
     if (force_bn == 0 && M <= (g_gemm_swap_max_m >= 1000 ? 128 : g_gemm_swap_max_m) && M <= 128 && N >= 128 && K >= 512) {
@@ -602,6 +603,8 @@ PIE_API int pie_gemm_bf16(const void* A, const void* W, void* C, const void* R, 
         case EPI_STORE: return launch_gemm<BN_, EPI_STORE_T>(ta, tb, C, R, N, M, K, ldc, ldr, status, plan, w, st); \
         case EPI_RESIDUAL: return launch_gemm<BN_, EPI_RESIDUAL_T>(ta, tb, C, R, N, M, K, ldc, ldr, status, plan, w, st); \
         case EPI_SWIGLU: return launch_gemm<BN_, EPI_SWIGLU_T>(ta, tb, C, R, N, M, K, ldc, ldr, status, plan, w, st); \
+        case EPI_XIELU: return launch_gemm<BN_, EPI_XIELU_T>(ta, tb, C, R, N, M, K, ldc, ldr, status, plan, w, st, TpArgs{}, ex); \
+        case EPI_STREAM: return launch_gemm<BN_, EPI_STREAM_T>(ta, tb, C, R, N, M, K, ldc, ldr, status, plan, w, st, TpArgs{}, ex); \
         default: return (int)cudaErrorInvalidValue;                                               \
     }
         if (bt == 64) { GO_T(64) } else { GO_T(128) }
@@ -621,6 +624,8 @@ direct:
         case EPI_STORE: return launch_gemm<BN_, EPI_STORE>(ta, tb, C, R, M, N, K, ldc, ldr, status, plan, w, st); \
         case EPI_RESIDUAL: return launch_gemm<BN_, EPI_RESIDUAL>(ta, tb, C, R, M, N, K, ldc, ldr, status, plan, w, st); \
         case EPI_SWIGLU: return launch_gemm<BN_, EPI_SWIGLU>(ta, tb, C, R, M, N, K, ldc, ldr, status, plan, w, st); \
+        case EPI_XIELU: return launch_gemm<BN_, EPI_XIELU>(ta, tb, C, R, M, N, K, ldc, ldr, status, plan, w, st, TpArgs{}, ex); \
+        case EPI_STREAM: return launch_gemm<BN_, EPI_STREAM>(ta, tb, C, R, M, N, K, ldc, ldr, status, plan, w, st, TpArgs{}, ex); \
         default: return (int)cudaErrorInvalidValue;                                               \
     }
     if (bn == 256) { GO(256) }
@@ -628,6 +633,35 @@ direct:
     else if (bn == 64) { GO(64) }
 #undef GO
     return (int)cudaErrorInvalidValue;
+}
+
+PIE_API int pie_gemm_bf16(const void* A, const void* W, void* C, const void* R, int M, int N, int K,
+                          int lda, int ldw, int ldc, int ldr, int epilogue, int force_bn,
+                          int* status, int num_sms, cudaStream_t st) {
+    if (epilogue < EPI_STORE || epilogue > EPI_SWIGLU) return (int)cudaErrorInvalidValue;
+    return gemm_bf16(A, W, C, R, M, N, K, lda, ldw, ldc, ldr, epilogue, force_bn, status, num_sms, st, EpiArgs());
+}
+
+// C = xIELU(A * W^T + bias): `act` holds the activation's two learned numbers.
+PIE_API int pie_gemm_bf16_xielu(const void* A, const void* W, void* C, const void* bias, const void* act, int M, int N, int K,
+                                int lda, int ldw, int ldc, int* status, int num_sms, cudaStream_t st) {
+    if (!act) return (int)cudaErrorInvalidValue;
+    EpiArgs ex;
+    ex.bias = (const bf16*)bias;
+    ex.act = (const bf16*)act;
+    return gemm_bf16(A, W, C, nullptr, M, N, K, lda, ldw, ldc, 0, EPI_XIELU, 0, status, num_sms, st, ex);
+}
+
+// x_out = x + A * W^T + bias over a 32-bit stream [M, ldx] (x_out may be x); C, if given, receives x_out in bf16.
+PIE_API int pie_gemm_bf16_stream(const void* A, const void* W, const void* bias, const float* x, float* x_out, int ldx, void* C,
+                                 int M, int N, int K, int lda, int ldw, int ldc, int* status, int num_sms, cudaStream_t st) {
+    if (!x || !x_out || ldx % 4) return (int)cudaErrorInvalidValue;
+    EpiArgs ex;
+    ex.bias = (const bf16*)bias;
+    ex.res32 = x;
+    ex.out32 = x_out;
+    ex.ld32 = ldx;
+    return gemm_bf16(A, W, C, nullptr, M, N, K, lda, ldw, ldc, 0, EPI_STREAM, 0, status, num_sms, st, ex);
 }
 
 // Tensor-parallel GEMM: `tp_blob` points at a host copy of TpArgs (see pie_tp_args_size).
@@ -714,7 +748,7 @@ PIE_API int pie_grouped_gemm_bf16(const void* A, const void* W, void* C, const i
                                              (int)GemmCfg<BN_>::SMEM_BYTES);                              \
         if (e != cudaSuccess) return (int)e;                                                              \
         e = launch_pdl(kern, dim3(grid), dim3(GEMM_THREADS), GemmCfg<BN_>::SMEM_BYTES, st, ta, tb, (bf16*)C, \
-                       (const bf16*)nullptr, M, N, K, ldc, 0, status, tp, sk, tile_expert, bn);               \
+                       (const bf16*)nullptr, M, N, K, ldc, 0, status, tp, sk, tile_expert, bn, EpiArgs());    \
         return (int)(e != cudaSuccess ? e : cudaGetLastError());                                          \
     }
     if (epilogue == EPI_STORE) {

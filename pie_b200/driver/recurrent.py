@@ -1,6 +1,7 @@
 """Recurrent-state cache of the Gated DeltaNet and Mamba-2 layers and of token-shifted blocks: per (recurrent layer,
 slot) the tail of the short convolution's inputs and the fp32 state (delta-rule state [heads, dk, dv], or state-space
-state [heads, head_dim, state]), or the previous token's normalised input (token shift, [width] fp32). A slot belongs to one resident context; the runtime's
+state [heads, head_dim, state]), or the previous token's normalised input (token shift, [width] fp32).
+A slot belongs to one resident context; the runtime's
 slot pool (`runtime/rs_cache.py`) hands slots out, tells the driver when a slot must start from zero
 (`rs_reset`) and asks for a slot copy when a context forks.
 

@@ -93,12 +93,18 @@ def parallel_latent_block(m, st: LatentStream, lw: dict, li: int, fi, cache) -> 
     if _pad(hv) > hv:
         both[:, hv:_pad(hv)] = 0
     latent_mixer(m, hs if hs is not None else h, lw, li, fi, cache, both[:, :hv])
-    if ff:
+    side = cfg.token_side_dim
+    fused = m.gemm_backend == "tcgen05" and h.dtype == torch.bfloat16
+    if ff and fused:
+        lops.gemm_xielu(h, lw["w_up"], lw["b_up"], lw["act"], both[:, _pad(hv):])
+    elif ff:
         act = both[:, _pad(hv):]
         act.copy_(m._gemm(h, lw["w_up"]))
         lops.bias_xielu(act, lw["b_up"], lw["act"])
-    side = cfg.token_side_dim
-    st.x, xc = lops.stream_add(x, m._gemm(both, lw["w_block_out"]), lw.get("b_down"), copy=side > 0)
+    if fused:
+        st.x, xc = lops.gemm_stream(both, lw["w_block_out"], lw.get("b_down"), x, copy=side > 0)
+    else:
+        st.x, xc = lops.stream_add(x, m._gemm(both, lw["w_block_out"]), lw.get("b_down"), copy=side > 0)
     st.y = st.y_norm = None
     if side:
         g = lops.side_gate(m._gemm(xc, lw["side_gate"]), m.w["side_embed"], fi.tokens, li * side, side)

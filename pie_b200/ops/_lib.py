@@ -65,6 +65,8 @@ _SIGNATURES = {
     "pie_stream_norm": [p, i32, i32, p],
     "pie_latent_rows": [p, i32, p],
     "pie_latent_attn_warp": [p, i32, p],
+    "pie_gemm_bf16_xielu": [p, p, p, p, p, i32, i32, i32, i32, i32, i32, p, i32, p],
+    "pie_gemm_bf16_stream": [p, p, p, p, p, i32, p, i32, i32, i32, i32, i32, i32, p, i32, p],
     "pie_latent_attn_mma_tiles": [i32, i32, i32],
     "pie_latent_attn_mma": [p, i32, p],
     "pie_per_head": [p, p],

@@ -207,6 +207,26 @@ def stream_add(x, d, bias=None, copy: bool = False):
     return out, (out if d.dtype == torch.float32 else cp)
 
 
+def gemm_xielu(x, w, bias, act, out):
+    """out = xIELU(x @ w.T + bias), bf16; bias and activation in the GEMM's epilogue. `out` may be a column range."""
+    m, k = x.shape
+    ops.ensure_gemm_workspace(x.device)
+    check(fn("pie_gemm_bf16_xielu")(ptr(x), ptr(w), ptr(out), ptr(bias), ptr(act), m, w.shape[0], k, x.stride(0), w.stride(0),
+                                    out.stride(0), ptr(ops.kernel_status(x.device)), ops.num_sms(x.device), stream_ptr()), "gemm_xielu")
+    return out
+
+
+def gemm_stream(a, w, bias, x, copy: bool = False):
+    """x += a @ w.T + bias in place for a 32-bit stream x, in the GEMM's epilogue; returns (x, x in bf16 if `copy`)."""
+    m, k = a.shape
+    cp = torch.empty(m, w.shape[0], dtype=a.dtype, device=a.device) if copy else None
+    ops.ensure_gemm_workspace(a.device)
+    check(fn("pie_gemm_bf16_stream")(ptr(a), ptr(w), ptr(bias), ptr(x), ptr(x), x.stride(0), ptr(cp), m, w.shape[0], k, a.stride(0),
+                                     w.stride(0), w.shape[0], ptr(ops.kernel_status(a.device)), ops.num_sms(a.device), stream_ptr()),
+          "gemm_stream")
+    return x, cp
+
+
 def side_gate(z, table, tokens, col0: int, dim: int):
     """gelu_tanh(z) * table[tokens, col0:col0 + dim], zeros in the padding columns of z."""
     if not z.is_cuda:
