@@ -42,8 +42,12 @@ struct XieluCoef {
         a = act ? sp(__bfloat162float(act[0])) : 0.f;
         b = act ? 0.5f + sp(__bfloat162float(act[1])) : 0.f;
     }
-    // the result is rounded to bf16: e^z - 1 - z loses digits near zero only, where z / 2 outweighs it
-    __device__ float operator()(float z) const { return (z > 0.f ? a * z * z : b * (__expf(z) - 1.f - z)) + 0.5f * z; }
+    // Both sides at once, each zero on the other's half. The result is rounded to bf16: e^z - 1 - z loses digits near
+    // zero only, where z / 2 outweighs it.
+    __device__ __forceinline__ float operator()(float z) const {
+        const float n = fminf(z, 0.f), p = fmaxf(z, 0.f);
+        return fmaf(b, (__expf(n) - 1.f) - n, fmaf(a * p, p, 0.5f * z));
+    }
 };
 
 constexpr int TP_MAX_RANKS = 8;

@@ -265,8 +265,14 @@ __global__ void __launch_bounds__(256) latent_rows_kernel(const LatentRowsArgs a
     if (is_q) {
         const T* src = row + (size_t)u * (a.dim + a.rot_dim);
         T* dst = static_cast<T*>(a.q_out) + ((size_t)t * a.heads + u) * a.q_width;
-        if (a.copy_nope)
-            for (int i = lane; i < a.dim; i += 32) dst[i] = src[i];
+        if (a.copy_nope) {
+            constexpr int E = 16 / sizeof(T);
+            const bool vec = ((uintptr_t)src & 15) == 0 && ((uintptr_t)dst & 15) == 0 && a.dim % E == 0;
+            if (vec)
+                for (int i = lane; i < a.dim / E; i += 32) reinterpret_cast<uint4*>(dst)[i] = reinterpret_cast<const uint4*>(src)[i];
+            else
+                for (int i = lane; i < a.dim; i += 32) dst[i] = src[i];
+        }
         for (int i = a.q_zero + lane; i < a.q_rot; i += 32) dst[i] = from_f<T>(0.f);
         rot_src = src + a.dim;
         rot_dst = dst + a.q_rot;
@@ -398,16 +404,22 @@ __global__ void stream_add_kernel(const float* __restrict__ x, const T* __restri
 }
 
 // g = gelu_tanh(z) * e, e = columns [col0, col0 + dim) of the token's row in the side table; zeros in the padding columns.
-template <typename T>
-__global__ void side_gate_kernel(const T* __restrict__ z, int ldz, const T* __restrict__ table, int ldt, const int* __restrict__ tokens,
-                                 T* __restrict__ g, int ldg, int dim, int col0, int vocab, long total) {
+// z arrives as `splits` arrays of Z, z_split elements apart, that add up to it (one array: the product itself).
+template <typename T, typename Z>
+__global__ void side_gate_kernel(const Z* __restrict__ z, int ldz, long z_split, int splits, const T* __restrict__ table, int ldt,
+                                 const int* __restrict__ tokens, T* __restrict__ g, int ldg, int dim, int col0, int vocab, long total) {
+    pdl_trigger();
+    pdl_wait();
     for (long i = blockIdx.x * (long)blockDim.x + threadIdx.x; i < total; i += (long)gridDim.x * blockDim.x) {
         const long t = i / ldg;
         const int c = (int)(i - t * ldg), id = tokens[t];
         float v = 0.f;
         if (c < dim && id >= 0 && id < vocab) {
-            const float x = to_f(z[t * ldz + c]);
-            v = 0.5f * x * (1.f + tanhf(0.7978845608028654f * (x + 0.044715f * x * x * x))) * to_f(table[(size_t)id * ldt + col0 + c]);
+            const float e = to_f(table[(size_t)id * ldt + col0 + c]);
+            float x = 0.f;
+#pragma unroll 4
+            for (int s = 0; s < splits; ++s) x += to_f(z[s * z_split + t * ldz + c]);
+            v = 0.5f * x * (1.f + tanhf(0.7978845608028654f * (x + 0.044715f * x * x * x))) * e;
         }
         g[i] = from_f<T>(v);
     }
@@ -503,15 +515,17 @@ PIE_API int pie_stream_add(const float* x, const void* d, const void* bias, floa
     return (int)cudaGetLastError();
 }
 
-PIE_API int pie_side_gate(const void* z, int ldz, const void* table, int ldt, const int* tokens, void* g, int ldg, int dim, int col0,
-                          int vocab, int rows, int f32, cudaStream_t st) {
+// z_f32: the partial products are 32-bit (else they have the type of the others, which f32 gives)
+PIE_API int pie_side_gate(const void* z, int ldz, long z_split, int splits, int z_f32, const void* table, int ldt, const int* tokens,
+                          void* g, int ldg, int dim, int col0, int vocab, int rows, int f32, cudaStream_t st) {
     const long total = (long)rows * ldg;
     if (total <= 0) return 0;
-    if (f32)
-        side_gate_kernel<float><<<grid_for(total), 256, 0, st>>>((const float*)z, ldz, (const float*)table, ldt, tokens, (float*)g, ldg, dim,
-                                                                 col0, vocab, total);
-    else
-        side_gate_kernel<bf16><<<grid_for(total), 256, 0, st>>>((const bf16*)z, ldz, (const bf16*)table, ldt, tokens, (bf16*)g, ldg, dim,
-                                                                col0, vocab, total);
-    return (int)cudaGetLastError();
+    if (splits < 1) return (int)cudaErrorInvalidValue;
+#define GO(T_, Z_)                                                                                                                 \
+    return (int)launch_pdl(side_gate_kernel<T_, Z_>, dim3(grid_for(total)), dim3(256), 0, st, (const Z_*)z, ldz, z_split, splits,   \
+                           (const T_*)table, ldt, tokens, (T_*)g, ldg, dim, col0, vocab, total)
+    if (f32) GO(float, float);
+    if (z_f32) GO(bf16, float);
+    GO(bf16, bf16);
+#undef GO
 }

@@ -5,7 +5,7 @@
 // of a prefill - and packs (token, head) into 16 * MT rows. Per 64 keys: S = Q K^T with the rows split over MT warps and
 // the keys over the other warps, softmax over shared memory with several threads per row, O += P V with the latent's
 // columns split over the eight warps. The cache rows arrive by cp.async in a ring of stages.
-// Also here: the merge of split spans, and the small per-head products around the attention.
+// Also here: the merge of split spans, and the small products around the attention.
 #include "common.cuh"
 
 namespace pie {
@@ -53,6 +53,7 @@ struct LatentMmaArgs {
     void* out;                     // [n, heads, rank_pad]
     float* scratch;                // decode: [max_items, heads, rank_pad] partial outputs, then [max_items, heads] log2 sums
     int items, max_items, heads, row, rank_pad, cache_row, page_size, window_left, stages, reqs;
+    int page_shift;                // log2(page_size)
     float scale_log2;
 };
 
@@ -104,20 +105,27 @@ __global__ void __launch_bounds__(256, (MT * NTW <= 8) ? 2 : 1) latent_attn_mma_
             k_lo = max(k_lo, a.item_start[item]);
             k_hi = min(k_hi, a.item_end[item]);
         }
-        k_lo = k_lo / LA_BK * LA_BK;
         const int tiles = k_hi > k_lo ? (k_hi - k_lo + LA_BK - 1) / LA_BK : 0;
         const int* pages = a.page_indices + a.kv_page_indptr[r];
 
+        // a warp brings eight rows: a lane each finds the row's address, then the lanes walk the rows' 16-byte chunks
         auto load_tile = [&](int t) {
             if (t < tiles) {
-                const uint32_t dst = la_smem(ring + (t % a.stages) * stage_elems);
-                for (int i = tid; i < LA_BK * chunks; i += 256) {
-                    const int kr = i / chunks, c = i - kr * chunks, key = k_lo + t * LA_BK + kr;
-                    const bool ok = key < k_hi;
-                    const int kk = ok ? key : k_lo;
-                    const bf16* src = static_cast<const bf16*>(a.cache) +
-                                      ((size_t)pages[kk / a.page_size] * a.page_size + kk % a.page_size) * a.cache_row + c * 8;
-                    la_cp16(dst + (kr * ldk + c * 8) * 2, src, ok);
+                const int key = k_lo + t * LA_BK + warp * 8 + (lane & 7);
+                const int kk = min(key, k_hi - 1);
+                const unsigned long long src = reinterpret_cast<unsigned long long>(
+                    static_cast<const bf16*>(a.cache) +
+                    ((((size_t)pages[kk >> a.page_shift]) << a.page_shift) + (kk & (a.page_size - 1))) * a.cache_row);
+                const uint32_t dst = la_smem(ring + (t % a.stages) * stage_elems + warp * 8 * ldk);
+                int kr = 0, c = lane;
+                while (c >= chunks) { c -= chunks; ++kr; }
+                for (int i = 0; i < 8 * chunks; i += 32) {
+                    // whole warps run the shuffles; a chunk past the eighth row is not copied
+                    const unsigned long long base = __shfl_sync(0xffffffffu, src, kr & 7);
+                    const bool ok = __shfl_sync(0xffffffffu, key, kr & 7) < k_hi;
+                    if (kr < 8) la_cp16(dst + (kr * ldk + c * 8) * 2, reinterpret_cast<const bf16*>(base) + c * 8, ok);
+                    c += 32;
+                    while (c >= chunks) { c -= chunks; ++kr; }
                 }
             }
             la_commit();
@@ -151,31 +159,43 @@ __global__ void __launch_bounds__(256, (MT * NTW <= 8) ? 2 : 1) latent_attn_mma_
             load_tile(t + a.stages - 1);
             const bf16* k_s = ring + (t % a.stages) * stage_elems;
             // ---- S: rows [16 wm, +16), keys [wn * 8 MT, +8 MT)
-            float s[MT][4];
+            float s[MT][4], s2[MT][4];                            // two chains: even and odd k steps
 #pragma unroll
-            for (int n = 0; n < MT; ++n) s[n][0] = s[n][1] = s[n][2] = s[n][3] = 0.f;
+            for (int n = 0; n < MT; ++n)
+#pragma unroll
+                for (int e = 0; e < 4; ++e) s[n][e] = s2[n][e] = 0.f;
             const uint32_t qa = la_smem(q_s + (wm * 16 + (lane & 15)) * ldk + (lane >> 4) * 8);
             const int key0 = wn * 8 * MT;
             const uint32_t kb = MT == 1 ? la_smem(k_s + (key0 + (lane & 7)) * ldk + ((lane >> 3) & 1) * 8)
                                         : la_smem(k_s + (key0 + (lane & 7) + ((lane >> 4) << 3)) * ldk + ((lane >> 3) & 1) * 8);
-#pragma unroll 4
-            for (int k = 0; k < (a.row >> 4); ++k) {
+            auto score_step = [&](int k, float (&acc)[MT][4]) {
                 uint32_t fa[4];
                 la_ldm4(fa, qa + k * 32);
                 if constexpr (MT == 1) {
                     uint32_t b0, b1;
                     la_ldm2(b0, b1, kb + k * 32);
-                    la_mma(s[0], fa, b0, b1);
+                    la_mma(acc[0], fa, b0, b1);
                 } else {
 #pragma unroll
                     for (int n = 0; n < MT; n += 2) {
                         uint32_t fb[4];
                         la_ldm4(fb, kb + n * 8 * ldk * 2 + k * 32);
-                        la_mma(s[n], fa, fb[0], fb[1]);
-                        la_mma(s[n + 1], fa, fb[2], fb[3]);
+                        la_mma(acc[n], fa, fb[0], fb[1]);
+                        la_mma(acc[n + 1], fa, fb[2], fb[3]);
                     }
                 }
+            };
+            const int ksteps = a.row >> 4;
+#pragma unroll 3
+            for (int k = 0; k + 1 < ksteps; k += 2) {
+                score_step(k, s);
+                score_step(k + 1, s2);
             }
+            if (ksteps & 1) score_step(ksteps - 1, s);
+#pragma unroll
+            for (int n = 0; n < MT; ++n)
+#pragma unroll
+                for (int e = 0; e < 4; ++e) s[n][e] += s2[n][e];
 #pragma unroll
             for (int n = 0; n < MT; ++n) {
                 float* d = s_s + (wm * 16 + (lane >> 2)) * LDS + key0 + n * 8 + (lane & 3) * 2;
@@ -315,54 +335,81 @@ __global__ void __launch_bounds__(256) latent_merge_kernel(const float* __restri
     }
 }
 
-// ------------------------------------------------------- per-head products
-struct PerHeadArgs {
+// ----------------------------------------------- small products around them
+// out[t, h, :] = W_h x[t, h, :]: per-head factors, or a product split along K (a "head" then is a K range of length k, and
+// out collects 32-bit partial sums).
+struct SmallProductArgs {
     const void* x;                 // x[t, h, k] at t * x_tok + h * x_head + k
-    const void* w;                 // [heads, m, k] contiguous
+    const void* w;                 // w[h, m, k] at h * w_head + m * w_row + k
     void* out;                     // out[t, h, m] at t * out_tok + h * out_head + m
-    long x_tok, x_head, out_tok, out_head;
-    int n, heads, m, k;
+    long x_tok, x_head, w_head, w_row, out_tok, out_head;
+    int n, heads, m, k, k_total;   // k_total > 0: the last head's range ends there
+    int out_f32;
 };
 
 constexpr int PH_T = 64, PH_K = 64, PH_LD = PH_K + 8;
 
-// out[t, h, :] = W_h x[t, h, :]. One CTA per (64 tokens, 64 outputs, head); four warps of 16 tokens. `vec`: every row
-// starts on a 16-byte boundary and k is a multiple of 8, else the tiles are filled element by element.
+// One CTA per (64 tokens, 64 outputs, head); four warps of 16 tokens, K in double-buffered chunks of 64. VEC: every row
+// starts on a 16-byte boundary and the K ranges are multiples of 8, else the tiles are filled element by element.
 template <bool VEC>
-__global__ void __launch_bounds__(128) per_head_kernel(const PerHeadArgs a) {
-    __shared__ __align__(16) bf16 x_s[PH_T * PH_LD];
-    __shared__ __align__(16) bf16 w_s[PH_T * PH_LD];
+__global__ void __launch_bounds__(128) small_product_kernel(const SmallProductArgs a) {
+    __shared__ __align__(16) bf16 x_s[2][PH_T * PH_LD];
+    __shared__ __align__(16) bf16 w_s[2][PH_T * PH_LD];
     const int t0 = blockIdx.x * PH_T, m0 = blockIdx.y * PH_T, h = blockIdx.z;
     const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
-    pdl_trigger();
-    pdl_wait();
+    const int kn = a.k_total > 0 ? min(a.k, a.k_total - h * a.k) : a.k;
     const bf16* x = static_cast<const bf16*>(a.x) + (size_t)h * a.x_head;
-    const bf16* w = static_cast<const bf16*>(a.w) + (size_t)h * a.m * a.k;
-    float acc[8][4];
-#pragma unroll
-    for (int n = 0; n < 8; ++n) acc[n][0] = acc[n][1] = acc[n][2] = acc[n][3] = 0.f;
-    for (int k0 = 0; k0 < a.k; k0 += PH_K) {
-        if (k0) __syncthreads();
+    const bf16* w = static_cast<const bf16*>(a.w) + (size_t)h * a.w_head;
+    auto load_w = [&](int k0, int b) {
         if constexpr (VEC) {
             for (int i = tid; i < PH_T * (PH_K / 8); i += 128) {
                 const int r = i >> 3, c = (i & 7) * 8;
-                const bool kok = k0 + c < a.k, xok = kok && t0 + r < a.n, wok = kok && m0 + r < a.m;
-                la_cp16(la_smem(x_s + r * PH_LD + c), x + (size_t)(xok ? t0 + r : 0) * a.x_tok + (xok ? k0 + c : 0), xok);
-                la_cp16(la_smem(w_s + r * PH_LD + c), w + (size_t)(wok ? m0 + r : 0) * a.k + (wok ? k0 + c : 0), wok);
+                const bool ok = k0 + c < kn && m0 + r < a.m;
+                la_cp16(la_smem(w_s[b] + r * PH_LD + c), w + (size_t)(ok ? m0 + r : 0) * a.w_row + (ok ? k0 + c : 0), ok);
             }
-            la_commit();
-            la_wait<0>();
         } else {
             for (int i = tid; i < PH_T * PH_K; i += 128) {
                 const int r = i / PH_K, c = i - r * PH_K;
-                const bool kok = k0 + c < a.k;
-                x_s[r * PH_LD + c] = kok && t0 + r < a.n ? x[(size_t)(t0 + r) * a.x_tok + k0 + c] : __float2bfloat16(0.f);
-                w_s[r * PH_LD + c] = kok && m0 + r < a.m ? w[(size_t)(m0 + r) * a.k + k0 + c] : __float2bfloat16(0.f);
+                w_s[b][r * PH_LD + c] = k0 + c < kn && m0 + r < a.m ? w[(size_t)(m0 + r) * a.w_row + k0 + c] : __float2bfloat16(0.f);
             }
         }
+    };
+    auto load_x = [&](int k0, int b) {
+        if constexpr (VEC) {
+            for (int i = tid; i < PH_T * (PH_K / 8); i += 128) {
+                const int r = i >> 3, c = (i & 7) * 8;
+                const bool ok = k0 + c < kn && t0 + r < a.n;
+                la_cp16(la_smem(x_s[b] + r * PH_LD + c), x + (size_t)(ok ? t0 + r : 0) * a.x_tok + (ok ? k0 + c : 0), ok);
+            }
+        } else {
+            for (int i = tid; i < PH_T * PH_K; i += 128) {
+                const int r = i / PH_K, c = i - r * PH_K;
+                x_s[b][r * PH_LD + c] = k0 + c < kn && t0 + r < a.n ? x[(size_t)(t0 + r) * a.x_tok + k0 + c] : __float2bfloat16(0.f);
+            }
+        }
+    };
+    float acc[8][4];
+#pragma unroll
+    for (int n = 0; n < 8; ++n) acc[n][0] = acc[n][1] = acc[n][2] = acc[n][3] = 0.f;
+    pdl_trigger();
+    load_w(0, 0);                  // weights depend on nothing
+    pdl_wait();
+    load_x(0, 0);
+    la_commit();
+    const int chunks = (kn + PH_K - 1) / PH_K;
+    for (int j = 0; j < chunks; ++j) {
+        const int b = j & 1;
+        if (j + 1 < chunks) {
+            load_w((j + 1) * PH_K, b ^ 1);
+            load_x((j + 1) * PH_K, b ^ 1);
+            la_commit();
+            la_wait<1>();
+        } else {
+            la_wait<0>();
+        }
         __syncthreads();
-        const uint32_t xa = la_smem(x_s + (warp * 16 + (lane & 15)) * PH_LD + (lane >> 4) * 8);
-        const uint32_t wb = la_smem(w_s + ((lane & 7) + ((lane >> 4) << 3)) * PH_LD + ((lane >> 3) & 1) * 8);
+        const uint32_t xa = la_smem(x_s[b] + (warp * 16 + (lane & 15)) * PH_LD + (lane >> 4) * 8);
+        const uint32_t wb = la_smem(w_s[b] + ((lane & 7) + ((lane >> 4) << 3)) * PH_LD + ((lane >> 3) & 1) * 8);
 #pragma unroll
         for (int k = 0; k < PH_K / 16; ++k) {
             uint32_t fa[4];
@@ -375,14 +422,26 @@ __global__ void __launch_bounds__(128) per_head_kernel(const PerHeadArgs a) {
                 la_mma(acc[n + 1], fa, fb[2], fb[3]);
             }
         }
+        __syncthreads();
     }
+    const bool pair = ((a.out_tok | a.out_head | a.m) & 1) == 0 && ((uintptr_t)a.out & 7) == 0;
 #pragma unroll
     for (int n = 0; n < 8; ++n)
 #pragma unroll
-        for (int e = 0; e < 4; ++e) {
-            const int t = t0 + warp * 16 + (lane >> 2) + (e >> 1) * 8, m = m0 + n * 8 + (lane & 3) * 2 + (e & 1);
-            if (t < a.n && m < a.m)
-                static_cast<bf16*>(a.out)[(size_t)t * a.out_tok + (size_t)h * a.out_head + m] = __float2bfloat16(acc[n][e]);
+        for (int half = 0; half < 2; ++half) {
+            const int t = t0 + warp * 16 + (lane >> 2) + half * 8, m = m0 + n * 8 + (lane & 3) * 2;
+            if (t >= a.n || m >= a.m) continue;
+            const size_t at = (size_t)t * a.out_tok + (size_t)h * a.out_head + m;
+            const float p = acc[n][half * 2], q = acc[n][half * 2 + 1];
+            if (a.out_f32) {
+                float* d = static_cast<float*>(a.out) + at;
+                if (pair) *reinterpret_cast<float2*>(d) = make_float2(p, q);
+                else { d[0] = p; if (m + 1 < a.m) d[1] = q; }
+            } else {
+                bf16* d = static_cast<bf16*>(a.out) + at;
+                if (pair) *reinterpret_cast<bf162*>(d) = __floats2bfloat162_rn(p, q);
+                else { d[0] = __float2bfloat16(p); if (m + 1 < a.m) d[1] = __float2bfloat16(q); }
+            }
         }
 }
 
@@ -402,7 +461,7 @@ PIE_API int pie_latent_attn_mma_tiles(int heads, int row, int rank_pad) {
 PIE_API int pie_latent_attn_mma(const LatentMmaArgs* args, int num_ctas, cudaStream_t st) {
     LatentMmaArgs a = *args;
     const int mt = pie_latent_attn_mma_tiles(a.heads, a.row, a.rank_pad);
-    if (!mt || a.rank_pad > a.row || a.row > a.cache_row || a.cache_row % 8 || num_ctas <= 0) return (int)cudaErrorInvalidValue;
+    if (!mt || a.rank_pad > a.row || a.page_size != 1 << a.page_shift || a.row > a.cache_row || a.cache_row % 8 || num_ctas <= 0) return (int)cudaErrorInvalidValue;
     if (a.item_end && (!a.scratch || !a.req_item_indptr || !a.num_items)) return (int)cudaErrorInvalidValue;
     if (!a.num_items && a.items <= 0) return 0;
     const int fixed = la_fixed_bytes(mt, a.row), stage = la_stage_bytes(a.row);
@@ -435,12 +494,14 @@ PIE_API int pie_latent_attn_mma(const LatentMmaArgs* args, int num_ctas, cudaStr
     return (int)cudaGetLastError();
 }
 
-PIE_API int pie_per_head(const PerHeadArgs* args, cudaStream_t st) {
-    const PerHeadArgs& a = *args;
-    if (a.n <= 0) return 0;
-    const bool vec = a.k % 8 == 0 && a.x_tok % 8 == 0 && a.x_head % 8 == 0 && ((uintptr_t)a.x & 15) == 0 && ((uintptr_t)a.w & 15) == 0;
+PIE_API int pie_small_product(const SmallProductArgs* args, cudaStream_t st) {
+    const SmallProductArgs& a = *args;
+    if (a.n <= 0 || a.m <= 0 || a.heads <= 0) return 0;
+    if (a.k <= 0 || (a.k_total > 0 && (long)(a.heads - 1) * a.k >= a.k_total)) return (int)cudaErrorInvalidValue;
+    const bool vec = a.k % 8 == 0 && a.k_total % 8 == 0 && a.w_row % 8 == 0 && a.w_head % 8 == 0 && ((uintptr_t)a.w & 15) == 0 &&
+                     a.x_tok % 8 == 0 && a.x_head % 8 == 0 && ((uintptr_t)a.x & 15) == 0;
     const dim3 grid((a.n + PH_T - 1) / PH_T, (a.m + PH_T - 1) / PH_T, a.heads);
-    const cudaError_t e = vec ? launch_pdl(per_head_kernel<true>, grid, dim3(128), 0, st, a)
-                              : launch_pdl(per_head_kernel<false>, grid, dim3(128), 0, st, a);
+    const cudaError_t e = vec ? launch_pdl(small_product_kernel<true>, grid, dim3(128), 0, st, a)
+                              : launch_pdl(small_product_kernel<false>, grid, dim3(128), 0, st, a);
     return (int)(e != cudaSuccess ? e : cudaGetLastError());
 }

@@ -482,7 +482,7 @@ class TorchDriver:
         else:
             plan = None
             item_req, st, en, indptr = ops.plan_decode_items(kv_lens, self.model.hkv, self.num_ctas, self.max_items,
-                                                             window_left=self.window_left)
+                                                             window_left=self.window_left, even=self.cfg.latent is not None)
             ni = len(item_req)
             s.h("item_req")[:ni], s.h("item_start")[:ni], s.h("item_end")[:ni] = item_req, st, en
         s.h("req_item_indptr")[:r + 1] = indptr

@@ -107,8 +107,14 @@ def parallel_latent_block(m, st: LatentStream, lw: dict, li: int, fi, cache) -> 
         st.x, xc = lops.stream_add(x, m._gemm(both, lw["w_block_out"]), lw.get("b_down"), copy=side > 0)
     st.y = st.y_norm = None
     if side:
-        g = lops.side_gate(m._gemm(xc, lw["side_gate"]), m.w["side_embed"], fi.tokens, li * side, side)
-        st.y, st.y_norm = m._gemm(g, lw["side_proj"]), lw["side_norm"]
+        z = lops.split_product(xc, lw["side_gate"]) if fused else m._gemm(xc, lw["side_gate"])
+        g = lops.side_gate(z, m.w["side_embed"], fi.tokens, li * side, side)
+        if fused and n <= 256:                          # short K, few rows: latency bound
+            st.y = torch.empty(n, lw["side_proj"].shape[0], dtype=g.dtype, device=g.device)
+            lops.per_head(g[:, None], lw["side_proj"][None], st.y[:, None])
+        else:
+            st.y = m._gemm(g, lw["side_proj"])
+        st.y_norm = lw["side_norm"]
 
 
 def final_rows(m, rows):

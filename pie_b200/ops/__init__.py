@@ -572,21 +572,28 @@ _DECODE_UNITS_PER_CTA = int(os.environ.get("PIE_DECODE_UNITS", "4"))
 
 
 def plan_decode_items(kv_lens: np.ndarray, hkv: int, target_ctas: int, max_items: int = 0,
-                      min_chunk: int = 256, window_left: int = -1):
+                      min_chunk: int = 256, window_left: int = -1, even: bool = False):
     """Split each request's KV range into chunks so that items*hkv fills the machine. With a
     sliding window only the last window_left + 1 keys are covered, from the 16-token boundary
     at or below the first visible key (the kernel masks the keys below it).
 
+    `even`: as many items as CTAs instead of several per CTA, equal parts of a request.
     Returns (item_req, item_start, item_end, req_item_indptr) as int32 arrays.
     """
     full_lens = np.asarray(kv_lens, dtype=np.int64)
     lo = np.zeros_like(full_lens)
     if window_left >= 0:
-        lo = np.maximum(0, full_lens - 1 - window_left) // 16 * 16
+        lo = np.maximum(0, full_lens - 1 - window_left) // (1 if even else 16) * (1 if even else 16)
     kv_lens = full_lens - lo
     total = int(kv_lens.sum())
     chunk = max(min_chunk, -(-total * hkv // max(1, target_ctas * _DECODE_UNITS_PER_CTA)))
     chunk = -(-chunk // 16) * 16
+    if even:
+        # one CTA per item, for kernels that pay per item: as many items as fit one wave of CTAs (whole requests if they
+        # alone fill it), a request's keys in equal parts
+        chunk = max(64, -(-total // max(1, target_ctas)))
+        while int(np.maximum(1, -(-kv_lens // chunk)).sum()) > max(target_ctas, len(kv_lens)):
+            chunk += -(-chunk // 8)
     while True:
         n_items = np.maximum(1, -(-kv_lens // chunk))
         if max_items <= 0 or int(n_items.sum()) <= max_items:
@@ -597,6 +604,8 @@ def plan_decode_items(kv_lens: np.ndarray, hkv: int, target_ctas: int, max_items
     tot = int(indptr[-1])
     item_req = np.repeat(np.arange(len(kv_lens), dtype=np.int32), n_items)
     within = np.arange(tot, dtype=np.int64) - np.repeat(indptr[:-1].astype(np.int64), n_items)
+    if even:
+        chunk = -(-kv_lens // n_items)[item_req]
     start = within * chunk
     end = np.minimum(start + chunk, kv_lens[item_req])
     start, end = start + lo[item_req], end + lo[item_req]

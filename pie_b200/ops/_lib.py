@@ -69,11 +69,11 @@ _SIGNATURES = {
     "pie_gemm_bf16_stream": [p, p, p, p, p, i32, p, i32, i32, i32, i32, i32, i32, p, i32, p],
     "pie_latent_attn_mma_tiles": [i32, i32, i32],
     "pie_latent_attn_mma": [p, i32, p],
-    "pie_per_head": [p, p],
+    "pie_small_product": [p, p],
     "pie_projected_prefill_attn_tc": [p, p, p, p, p, p, p, p, i32, p, p, p, i32, i32, i32, i32, i32, i32, f32, i32, p, p],
     "pie_bias_xielu": [p, i32, p, p, i32, i32, i32, p],
     "pie_stream_add": [p, p, p, p, p, i32, i32, i32, p],
-    "pie_side_gate": [p, i32, p, i32, p, p, i32, i32, i32, i32, i32, i32, p],
+    "pie_side_gate": [p, i32, i64, i32, i32, p, i32, p, p, i32, i32, i32, i32, i32, i32, p],
     "pie_gemm_set_workspace": [i32, p, i64, p, i32],
     "pie_gemm_set_pairs": [i32],
     "pie_gemm_set_swap": [i32],

@@ -30,8 +30,10 @@ LatentAttnArgs = _struct("LatentAttnArgs", ("q cache page_indices kv_page_indptr
 
 LatentMmaArgs = _struct("LatentMmaArgs", ("q cache page_indices kv_page_indptr item_req item_start item_end req_item_indptr "
                                           "num_items qo_indptr kv_lens mask_bits mask_word_indptr out scratch", p),
-                        ("items max_items heads row rank_pad cache_row page_size window_left stages reqs", i32), ("scale_log2", f32))
-PerHeadArgs = _struct("PerHeadArgs", ("x w out", p), ("x_tok x_head out_tok out_head", i64), ("n heads m k", i32))
+                        ("items max_items heads row rank_pad cache_row page_size window_left stages reqs page_shift", i32),
+                        ("scale_log2", f32))
+SmallProductArgs = _struct("SmallProductArgs", ("x w out", p), ("x_tok x_head w_head w_row out_tok out_head", i64),
+                           ("n heads m k k_total out_f32", i32))
 
 
 def _f32(t) -> int:
@@ -99,9 +101,9 @@ def per_head(x, w, out):
         out.copy_(torch.bmm(x.transpose(0, 1), w.transpose(1, 2)).transpose(0, 1))
         return out
     n, heads, k = x.shape
-    a = PerHeadArgs(x=ptr(x), w=ptr(w), out=ptr(out), x_tok=x.stride(0), x_head=x.stride(1), out_tok=out.stride(0),
-                    out_head=out.stride(1), n=n, heads=heads, m=w.shape[1], k=k)
-    check(fn("pie_per_head")(C.byref(a), stream_ptr()), "per_head")
+    a = SmallProductArgs(x=ptr(x), w=ptr(w), out=ptr(out), x_tok=x.stride(0), x_head=x.stride(1), w_head=w.stride(0), w_row=w.stride(1),
+                         out_tok=out.stride(0), out_head=out.stride(1), n=n, heads=heads, m=w.shape[1], k=k)
+    check(fn("pie_small_product")(C.byref(a), stream_ptr()), "per_head")
     return out
 
 
@@ -114,8 +116,9 @@ def latent_attention(q, cache, plan, rs, slots, spec, page_size: int, window_lef
     n = q.shape[0]
     out = torch.empty(n, spec.heads, spec.rank_pad, dtype=q.dtype, device=q.device)
     decode = isinstance(plan, ops.DecodePlan)
-    tiles = fn("pie_latent_attn_mma_tiles")(spec.heads, spec.row, spec.rank_pad) if q.dtype == torch.bfloat16 else 0
-    if not tiles:           # 32-bit, or a latent wider than the tensor-core kernel takes
+    tiles = fn("pie_latent_attn_mma_tiles")(spec.heads, spec.row, spec.rank_pad) \
+        if q.dtype == torch.bfloat16 and page_size & (page_size - 1) == 0 else 0
+    if not tiles:           # 32-bit, or a shape that the tensor-core kernel does not take
         a = LatentAttnArgs(q=ptr(q), cache=ptr(cache), page_indices=ptr(plan.page_indices), kv_page_indptr=ptr(plan.kv_page_indptr),
                            qo_indptr=ptr(rs.qo_indptr), kv_lens=ptr(plan.kv_lens), tok_req=ptr(rs.tok_req), slots=ptr(slots),
                            mask_bits=ptr(getattr(plan, "mask_bits", None)),
@@ -127,7 +130,7 @@ def latent_attention(q, cache, plan, rs, slots, spec, page_size: int, window_lef
     a = LatentMmaArgs(q=ptr(q), cache=ptr(cache), page_indices=ptr(plan.page_indices), kv_page_indptr=ptr(plan.kv_page_indptr),
                       qo_indptr=ptr(rs.qo_indptr), kv_lens=ptr(plan.kv_lens), out=ptr(out), heads=spec.heads, row=spec.row,
                       rank_pad=spec.rank_pad, cache_row=cache.shape[-1], page_size=page_size, window_left=window_left,
-                      reqs=len(rs.slots_host), scale_log2=spec.scale * 1.4426950408889634)
+                      reqs=len(rs.slots_host), page_shift=page_size.bit_length() - 1, scale_log2=spec.scale * 1.4426950408889634)
     ctas = ops.num_sms(q.device) * 2
     if decode:
         a.item_req, a.item_start, a.item_end = ptr(plan.item_req), ptr(plan.item_start), ptr(plan.item_end)
@@ -228,10 +231,29 @@ def gemm_stream(a, w, bias, x, copy: bool = False):
 
 
 def side_gate(z, table, tokens, col0: int, dim: int):
-    """gelu_tanh(z) * table[tokens, col0:col0 + dim], zeros in the padding columns of z."""
+    """gelu_tanh(z) * table[tokens, col0:col0 + dim], zeros in the padding columns of z. z [N, cols], or 32-bit partial
+    products [splits, N, cols] that add up to it."""
     if not z.is_cuda:
         return ref.side_gate(z, table, tokens, col0, dim)
-    g = torch.empty(z.shape[0], z.shape[1], dtype=z.dtype, device=z.device)
-    check(fn("pie_side_gate")(ptr(z), z.stride(0), ptr(table), table.stride(0), ptr(tokens), ptr(g), g.stride(0), dim, col0,
-                              table.shape[0], z.shape[0], _f32(z), stream_ptr()), "side_gate")
+    splits = z.shape[0] if z.dim() == 3 else 1
+    n, cols = z.shape[-2:]
+    g = torch.empty(n, cols, dtype=table.dtype, device=z.device)
+    check(fn("pie_side_gate")(ptr(z), z.stride(-2), z.stride(0), splits, _f32(z), ptr(table), table.stride(0), ptr(tokens), ptr(g), cols,
+                              dim, col0, table.shape[0], n, _f32(table), stream_ptr()), "side_gate")
     return g
+
+
+def split_product(x, w):
+    """x @ w.T for a narrow w [M, K], bf16 in, as 32-bit partial products [splits, N, M] over ranges of K (the reader adds
+    them up): enough CTAs for a product with few output tiles and a long K."""
+    n, k = x.shape
+    m = w.shape[0]
+    tiles = -(-n // 64) * -(-m // 64)
+    splits = max(1, min(16, k // 256, 4 * ops.num_sms(x.device) // tiles))
+    per = -(-(-(-k // splits)) // 64) * 64
+    splits = -(-k // per)
+    z = torch.empty(splits, n, m, dtype=torch.float32, device=x.device)
+    a = SmallProductArgs(x=ptr(x), w=ptr(w), out=ptr(z), x_tok=x.stride(0), x_head=per, w_head=per, w_row=w.stride(0), out_tok=m,
+                         out_head=n * m, n=n, heads=splits, m=m, k=per, k_total=k, out_f32=1)
+    check(fn("pie_small_product")(C.byref(a), stream_ptr()), "split_product")
+    return z
