@@ -28,9 +28,15 @@ __device__ __forceinline__ void la_ldm4t(uint32_t (&r)[4], uint32_t a) {
                  : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(a));
 }
 __device__ __forceinline__ void la_mma(float (&d)[4], const uint32_t (&a)[4], uint32_t b0, uint32_t b1) {
-    asm volatile("mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0,%1,%2,%3}, {%4,%5,%6,%7}, {%8,%9}, {%0,%1,%2,%3};\n"
+    asm("mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0,%1,%2,%3}, {%4,%5,%6,%7}, {%8,%9}, {%0,%1,%2,%3};\n"
                  : "+f"(d[0]), "+f"(d[1]), "+f"(d[2]), "+f"(d[3])
                  : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b0), "r"(b1));
+}
+
+__device__ __forceinline__ float la_exp2(float x) {
+    float y;
+    asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
+    return y;
 }
 
 constexpr int LA_BK = 64;          // keys per tile
@@ -82,7 +88,7 @@ __global__ void __launch_bounds__(256, (MT * NTW <= 8) ? 2 : 1) latent_attn_mma_
     int* lim_s = lo_s + ROWS;
     bf16* ring = reinterpret_cast<bf16*>(la_raw + la_fixed_bytes(MT, a.row));
     const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
-    const int chunks = a.row >> 3, stage_elems = LA_BK * ldk;
+    const int chunks = a.row >> 3, stage_elems = LA_BK * ldk, lrow = warp * 8 + (lane >> 2);
     const bool prefill = a.item_end == nullptr;
     const int hg = min(a.heads, ROWS), h0 = blockIdx.y * hg, hn = min(hg, a.heads - h0);
     const int tq = prefill ? ROWS / hg : 1;
@@ -108,35 +114,28 @@ __global__ void __launch_bounds__(256, (MT * NTW <= 8) ? 2 : 1) latent_attn_mma_
         const int tiles = k_hi > k_lo ? (k_hi - k_lo + LA_BK - 1) / LA_BK : 0;
         const int* pages = a.page_indices + a.kv_page_indptr[r];
 
-        // a warp brings eight rows: a lane each finds the row's address, then the lanes walk the rows' 16-byte chunks
+        // a warp brings eight rows, four lanes to a row; the page of a thread's next row is looked up one tile ahead
+        auto page_of = [&](int t) { return t < tiles ? pages[min(k_lo + t * LA_BK + lrow, k_hi - 1) >> a.page_shift] : 0; };
+        int next_page = page_of(0);
         auto load_tile = [&](int t) {
             if (t < tiles) {
-                const int key = k_lo + t * LA_BK + warp * 8 + (lane & 7);
-                const int kk = min(key, k_hi - 1);
-                const unsigned long long src = reinterpret_cast<unsigned long long>(
-                    static_cast<const bf16*>(a.cache) +
-                    ((((size_t)pages[kk >> a.page_shift]) << a.page_shift) + (kk & (a.page_size - 1))) * a.cache_row);
-                const uint32_t dst = la_smem(ring + (t % a.stages) * stage_elems + warp * 8 * ldk);
-                int kr = 0, c = lane;
-                while (c >= chunks) { c -= chunks; ++kr; }
-                for (int i = 0; i < 8 * chunks; i += 32) {
-                    // whole warps run the shuffles; a chunk past the eighth row is not copied
-                    const unsigned long long base = __shfl_sync(0xffffffffu, src, kr & 7);
-                    const bool ok = __shfl_sync(0xffffffffu, key, kr & 7) < k_hi;
-                    if (kr < 8) la_cp16(dst + (kr * ldk + c * 8) * 2, reinterpret_cast<const bf16*>(base) + c * 8, ok);
-                    c += 32;
-                    while (c >= chunks) { c -= chunks; ++kr; }
-                }
+                const int key = k_lo + t * LA_BK + lrow, kk = min(key, k_hi - 1);
+                const bf16* src = static_cast<const bf16*>(a.cache) +
+                                  (((size_t)next_page << a.page_shift) + (kk & (a.page_size - 1))) * a.cache_row;
+                const uint32_t dst = la_smem(ring + (t % a.stages) * stage_elems + lrow * ldk);
+                const bool ok = key < k_hi;
+                next_page = page_of(t + 1);
+#pragma unroll 3
+                for (int c = lane & 3; c < chunks; c += 4) la_cp16(dst + c * 16, src + c * 8, ok);
             }
             la_commit();
         };
         __syncthreads();                                          // the previous item is done with shared memory
-        for (int i = tid; i < ROWS * chunks; i += 256) {
-            const int row = i / chunks, c = i - row * chunks;
+        for (int row = lrow; row < ROWS; row += 64) {
             const bool ok = row < used;
             const int tok = ok ? row / hn : 0, h = ok ? row - tok * hn : 0;
-            const bf16* src = static_cast<const bf16*>(a.q) + ((size_t)(q_base + qs + tok) * a.heads + h0 + h) * a.row + c * 8;
-            la_cp16(la_smem(q_s + row * ldk + c * 8), src, ok);
+            const bf16* src = static_cast<const bf16*>(a.q) + ((size_t)(q_base + qs + tok) * a.heads + h0 + h) * a.row;
+            for (int c = lane & 3; c < chunks; c += 4) la_cp16(la_smem(q_s + row * ldk) + c * 16, src + c * 8, ok);
         }
         if (tid < ROWS) {
             const int pos = past + qs + tid / hn;
@@ -168,30 +167,39 @@ __global__ void __launch_bounds__(256, (MT * NTW <= 8) ? 2 : 1) latent_attn_mma_
             const int key0 = wn * 8 * MT;
             const uint32_t kb = MT == 1 ? la_smem(k_s + (key0 + (lane & 7)) * ldk + ((lane >> 3) & 1) * 8)
                                         : la_smem(k_s + (key0 + (lane & 7) + ((lane >> 4) << 3)) * ldk + ((lane >> 3) & 1) * 8);
-            auto score_step = [&](int k, float (&acc)[MT][4]) {
-                uint32_t fa[4];
-                la_ldm4(fa, qa + k * 32);
-                if constexpr (MT == 1) {
-                    uint32_t b0, b1;
-                    la_ldm2(b0, b1, kb + k * 32);
-                    la_mma(acc[0], fa, b0, b1);
-                } else {
+            // KB k steps at a time: their fragments are all on the way before the first product needs one
+            constexpr int KB = MT == 4 ? 2 : 3;
+            const int ksteps = a.row >> 4;
+            for (int k0 = 0; k0 < ksteps; k0 += KB) {
+                uint32_t fa[KB][4], fb[KB][MT == 1 ? 1 : MT / 2][4];
 #pragma unroll
-                    for (int n = 0; n < MT; n += 2) {
-                        uint32_t fb[4];
-                        la_ldm4(fb, kb + n * 8 * ldk * 2 + k * 32);
-                        la_mma(acc[n], fa, fb[0], fb[1]);
-                        la_mma(acc[n + 1], fa, fb[2], fb[3]);
+                for (int i = 0; i < KB; ++i) {
+                    if (k0 + i < ksteps) {
+                        la_ldm4(fa[i], qa + (k0 + i) * 32);
+                        if constexpr (MT == 1) {
+                            la_ldm2(fb[i][0][0], fb[i][0][1], kb + (k0 + i) * 32);
+                        } else {
+#pragma unroll
+                            for (int n = 0; n < MT / 2; ++n) la_ldm4(fb[i][n], kb + n * 16 * ldk * 2 + (k0 + i) * 32);
+                        }
                     }
                 }
-            };
-            const int ksteps = a.row >> 4;
-#pragma unroll 3
-            for (int k = 0; k + 1 < ksteps; k += 2) {
-                score_step(k, s);
-                score_step(k + 1, s2);
+#pragma unroll
+                for (int i = 0; i < KB; ++i) {
+                    if (k0 + i < ksteps) {
+                        float(&acc)[MT][4] = (i & 1) ? s2 : s;
+                        if constexpr (MT == 1) {
+                            la_mma(acc[0], fa[i], fb[i][0][0], fb[i][0][1]);
+                        } else {
+#pragma unroll
+                            for (int n = 0; n < MT / 2; ++n) {
+                                la_mma(acc[2 * n], fa[i], fb[i][n][0], fb[i][n][1]);
+                                la_mma(acc[2 * n + 1], fa[i], fb[i][n][2], fb[i][n][3]);
+                            }
+                        }
+                    }
+                }
             }
-            if (ksteps & 1) score_step(ksteps - 1, s);
 #pragma unroll
             for (int n = 0; n < MT; ++n)
 #pragma unroll
@@ -199,36 +207,44 @@ __global__ void __launch_bounds__(256, (MT * NTW <= 8) ? 2 : 1) latent_attn_mma_
 #pragma unroll
             for (int n = 0; n < MT; ++n) {
                 float* d = s_s + (wm * 16 + (lane >> 2)) * LDS + key0 + n * 8 + (lane & 3) * 2;
-                d[0] = s[n][0];
-                d[1] = s[n][1];
-                d[8 * LDS] = s[n][2];
-                d[8 * LDS + 1] = s[n][3];
+                *reinterpret_cast<float2*>(d) = make_float2(s[n][0], s[n][1]);
+                *reinterpret_cast<float2*>(d + 8 * LDS) = make_float2(s[n][2], s[n][3]);
             }
             __syncthreads();
             // ---- softmax: TPR threads per row
             {
+                // a thread has VPT / 2 pairs of neighbouring keys, 2 TPR apart; scores stay unscaled, the maximum too
                 const int row = tid / TPR, sub = tid % TPR, kbase = k_lo + t * LA_BK;
                 const int lo = lo_s[row] - kbase, lim = lim_s[row] - kbase;
                 const uint32_t* rb = bits ? bits + (size_t)(qs + min(row / hn, tn - 1)) * words : nullptr;
                 float v[VPT], mx = -INFINITY;
 #pragma unroll
-                for (int i = 0; i < VPT; ++i) {
-                    const int c = sub + i * TPR;
-                    bool see = c >= lo && c < lim;
-                    if (rb && see) see = rb[(kbase + c) >> 5] >> ((kbase + c) & 31) & 1u;
-                    v[i] = see ? s_s[row * LDS + c] * a.scale_log2 : -INFINITY;
-                    mx = fmaxf(mx, v[i]);
+                for (int i = 0; i < VPT; i += 2) {
+                    const float2 x = *reinterpret_cast<const float2*>(s_s + row * LDS + sub * 2 + i * TPR);
+                    v[i] = x.x;
+                    v[i + 1] = x.y;
+                }
+                if (!__all_sync(0xffffffffu, lo <= 0 && lim >= LA_BK && !rb)) {
+#pragma unroll
+                    for (int i = 0; i < VPT; ++i) {
+                        const int c = sub * 2 + (i & 1) + (i & ~1) * TPR;
+                        bool see = c >= lo && c < lim;
+                        if (rb && see) see = rb[(kbase + c) >> 5] >> ((kbase + c) & 31) & 1u;
+                        if (!see) v[i] = -INFINITY;
+                    }
                 }
 #pragma unroll
+                for (int i = 0; i < VPT; ++i) mx = fmaxf(mx, v[i]);
+#pragma unroll
                 for (int d = TPR / 2; d > 0; d >>= 1) mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, d));
-                const float mn = fmaxf(row_m, mx), base = mn == -INFINITY ? 0.f : mn;
-                const float al = exp2f(row_m - base);             // 0 while nothing was seen
+                const float mn = fmaxf(row_m, mx), base = mn == -INFINITY ? 0.f : mn * a.scale_log2;
+                const float al = la_exp2(fmaf(row_m, a.scale_log2, -base));      // 0 while nothing was seen
                 float sum = 0.f;
 #pragma unroll
-                for (int i = 0; i < VPT; ++i) {
-                    const float p = exp2f(v[i] - base);
-                    sum += p;
-                    p_s[row * LDP + sub + i * TPR] = __float2bfloat16(p);
+                for (int i = 0; i < VPT; i += 2) {
+                    const float p0 = la_exp2(fmaf(v[i], a.scale_log2, -base)), p1 = la_exp2(fmaf(v[i + 1], a.scale_log2, -base));
+                    sum += p0 + p1;
+                    *reinterpret_cast<bf162*>(p_s + row * LDP + sub * 2 + i * TPR) = __floats2bfloat162_rn(p0, p1);
                 }
 #pragma unroll
                 for (int d = TPR / 2; d > 0; d >>= 1) sum += __shfl_xor_sync(0xffffffffu, sum, d);
@@ -241,6 +257,7 @@ __global__ void __launch_bounds__(256, (MT * NTW <= 8) ? 2 : 1) latent_attn_mma_
 #pragma unroll
             for (int m = 0; m < MT; ++m) {
                 const float a0 = alpha_s[m * 16 + (lane >> 2)], a1 = alpha_s[m * 16 + 8 + (lane >> 2)];
+                if (__all_sync(0xffffffffu, a0 == 1.f && a1 == 1.f)) continue;      // no row's maximum moved
 #pragma unroll
                 for (int n = 0; n < NTW; ++n) {
                     o[m][n][0] *= a0;
@@ -275,7 +292,7 @@ __global__ void __launch_bounds__(256, (MT * NTW <= 8) ? 2 : 1) latent_attn_mma_
         }
         la_wait<0>();
         if (tid % TPR == 0) {
-            m_s[tid / TPR] = row_m;
+            m_s[tid / TPR] = row_m * a.scale_log2;
             l_s[tid / TPR] = row_l;
         }
         __syncthreads();
@@ -461,7 +478,9 @@ PIE_API int pie_latent_attn_mma_tiles(int heads, int row, int rank_pad) {
 PIE_API int pie_latent_attn_mma(const LatentMmaArgs* args, int num_ctas, cudaStream_t st) {
     LatentMmaArgs a = *args;
     const int mt = pie_latent_attn_mma_tiles(a.heads, a.row, a.rank_pad);
-    if (!mt || a.rank_pad > a.row || a.page_size != 1 << a.page_shift || a.row > a.cache_row || a.cache_row % 8 || num_ctas <= 0) return (int)cudaErrorInvalidValue;
+    if (!mt || a.rank_pad > a.row || a.page_size != 1 << a.page_shift || a.row > a.cache_row || a.cache_row % 8 ||
+        num_ctas <= 0)
+        return (int)cudaErrorInvalidValue;
     if (a.item_end && (!a.scratch || !a.req_item_indptr || !a.num_items)) return (int)cudaErrorInvalidValue;
     if (!a.num_items && a.items <= 0) return 0;
     const int fixed = la_fixed_bytes(mt, a.row), stage = la_stage_bytes(a.row);
