@@ -450,7 +450,7 @@ PIE_API int pie_stream_norm(const StreamNormArgs* args, int f32, int commit_requ
     const int part = a.width / a.groups;
     const bool vec = part % 4 == 0 && a.ldx % 4 == 0 && a.ldy % 4 == 0 && a.ldh % 4 == 0;
     const int per = (a.width / (vec ? 4 : 1) + 255) / 256;
-    if (per > 16) return (int)cudaErrorInvalidValue;
+    if (per > (vec ? 16 : 32)) return (int)cudaErrorInvalidValue;
     const dim3 grid((a.n + a.rows_per_block - 1) / a.rows_per_block);
     const size_t smem = ((vec ? a.width / 4 : a.width) + a.groups) * sizeof(float);
 #define GO(T_, M_, V_)                                                                       \
@@ -460,7 +460,7 @@ PIE_API int pie_stream_norm(const StreamNormArgs* args, int f32, int commit_requ
     }
 #define GO_M(T_, V_)                                                                         \
     if (per <= 1) GO(T_, 1, V_) else if (per <= 2) GO(T_, 2, V_) else if (per <= 4) GO(T_, 4, V_) \
-    else if (per <= 8) GO(T_, 8, V_) else GO(T_, 16, V_)
+    else if (per <= 8) GO(T_, 8, V_) else if (per <= 16) GO(T_, 16, V_) else GO(T_, 32, 1)
     if (f32) { if (vec) { GO_M(float, 4) } else { GO_M(float, 1) } }
     else { if (vec) { GO_M(bf16, 4) } else { GO_M(bf16, 1) } }
 #undef GO_M

@@ -967,6 +967,10 @@ def sample(logits, temperature, top_k, top_p, min_p, seeds, mask_bits=None, mask
     rows, vocab = logits.shape
     if out is None:
         out = torch.empty(rows, dtype=torch.int32, device=logits.device)
+    if vocab % 8 or logits.stride(0) % 8 or logits.data_ptr() % 16:       # the kernel reads 16-byte vectors: fill up with -inf
+        full = torch.full((rows, -(-vocab // 8) * 8), float("-inf"), dtype=logits.dtype, device=logits.device)
+        full[:, :vocab] = logits
+        logits, vocab = full, full.shape[1]
     mask_words = mask_bits.shape[1] if mask_bits is not None else 0
     check(fn("pie_sample")(ptr(logits), logits.stride(0), rows, vocab, ptr(temperature), ptr(top_k),
                            ptr(top_p), ptr(min_p), ptr(seeds), ptr(mask_bits), ptr(mask_row),
@@ -976,7 +980,7 @@ def sample(logits, temperature, top_k, top_p, min_p, seeds, mask_bits=None, mask
 
 def row_stats(logits):
     """[rows, 3] fp32: max, log-sum-exp and entropy of the unscaled next-token distribution."""
-    if not logits.is_cuda or logits.dtype != torch.bfloat16:
+    if not logits.is_cuda or logits.dtype != torch.bfloat16 or logits.shape[1] % 8 or logits.stride(0) % 8:
         return reference.row_stats(logits)
     rows, vocab = logits.shape
     out = torch.empty(rows, 3, dtype=torch.float32, device=logits.device)

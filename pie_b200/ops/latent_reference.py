@@ -29,8 +29,9 @@ def stream_norm(x, width, eps, y, y_norm, norm_w, groups, shift, rs, layer, dtyp
                 if b == a:
                     continue
                 slot = rs.slots_host[r]
-                prev[a] = 0 if rs.reset_host[r] else state[slot]
-                state[slot] = hf[b - 1]
+                prev[a] = 0 if rs.reset_host[r] or slot < 0 else state[slot]
+                if slot >= 0:
+                    state[slot] = hf[b - 1]
             hs = torch.zeros(x.shape, dtype=dtype)
             hs[:, :width] = (hf + (prev - hf) * shift.float()).to(dtype)
     return x, h, hs
