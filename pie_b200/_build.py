@@ -28,7 +28,7 @@ KERNEL_LIB = OUT / "libpie_kernels.so"
 
 # sources whose kernels a latent-attention model launches
 LATENT_SOURCES = ("attention_tc", "elementwise", "gemm2_tcgen05", "gemm_tcgen05", "latent",
-                  "latent_attn", "sampling")
+                  "latent_attn", "latent_attn_tc", "sampling")
 
 NVCC_FLAGS = [
     "-gencode", "arch=compute_100a,code=sm_100a", "-lineinfo", "-O3", "-std=c++17",

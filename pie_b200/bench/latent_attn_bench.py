@@ -42,11 +42,17 @@ def _decode_plan(kv, hkv, window, max_items, scratch, dev, even):
     r = len(kv)
     t = lambda a: torch.from_numpy(np.ascontiguousarray(a, np.int32)).to(dev)
     per = -(-int(kv.max()) // 16)
-    ctas = ops.num_sms(dev) * 2
-    ir, st, en, ip = ops.plan_decode_items(kv, hkv, ctas, max_items, window_left=window - 1, even=even)
-    return ops.DecodePlan(page_indices=t(np.random.default_rng(0).permutation(r * per)), kv_page_indptr=t(np.arange(r + 1) * per), item_req=t(ir),
+    ctas, ci = ops.num_sms(dev) * (1 if even else 2), None
+    if even:
+        ir, st, en, ip, ci = ops.plan_even_items(kv, ctas, max_items, window - 1)
+        ci = t(ci)
+    else:
+        ir, st, en, ip = ops.plan_decode_items(kv, hkv, ctas, max_items, window_left=window - 1)
+    ids = np.random.default_rng(0).permutation(r * per)
+    return ops.DecodePlan(page_indices=t(ids), kv_page_indptr=t(np.arange(r + 1) * per), item_req=t(ir),
                           item_start=t(st), item_end=t(en), req_item_indptr=t(ip), num_items=t([len(ir)]), scratch=scratch,
-                          max_items=max_items, num_reqs=r, num_ctas=ctas, page_size=16, window_left=window - 1, kv_lens=t(kv)), r * per
+                          max_items=max_items, num_reqs=r, num_ctas=ctas, page_size=16, window_left=window - 1, kv_lens=t(kv),
+                          cta_items=ci), r * per
 
 
 def main(argv=None):

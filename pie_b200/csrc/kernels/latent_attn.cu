@@ -6,7 +6,7 @@
 // the keys over the other warps, softmax over shared memory with several threads per row, O += P V with the latent's
 // columns split over the eight warps. The cache rows arrive by cp.async in a ring of stages.
 // Also here: the merge of split spans, and the small products around the attention.
-#include "common.cuh"
+#include "latent_args.cuh"
 
 namespace pie {
 
@@ -42,27 +42,6 @@ __device__ __forceinline__ float la_exp2(float x) {
 constexpr int LA_BK = 64;          // keys per tile
 constexpr int LA_MAX_STAGES = 4;
 
-struct LatentMmaArgs {
-    const void* q;                 // [n, heads, row]
-    const void* cache;             // [pages, page_size, cache_row]
-    const int* page_indices;
-    const int* kv_page_indptr;
-    const int* item_req;           // request of an item
-    const int* item_start;         // decode: first key; prefill: first query token (within the request)
-    const int* item_end;           // decode: one past the last key; null: prefill
-    const int* req_item_indptr;    // decode: items of a request
-    const int* num_items;          // device count, or null (items)
-    const int* qo_indptr;
-    const int* kv_lens;
-    const uint32_t* mask_bits;     // prefill: custom mask words, or null
-    const long* mask_word_indptr;
-    void* out;                     // [n, heads, rank_pad]
-    float* scratch;                // decode: [max_items, heads, rank_pad] partial outputs, then [max_items, heads] log2 sums
-    int items, max_items, heads, row, rank_pad, cache_row, page_size, window_left, stages, reqs;
-    int page_shift;                // log2(page_size)
-    float scale_log2;
-};
-
 // Bytes of the parts of shared memory in front of the ring, and of one stage.
 __host__ __device__ constexpr int la_rows(int mt) { return 16 * mt; }
 __host__ __device__ inline int la_ldk(int row) { return row + 8; }          // odd multiple of 16 bytes mod 128: no bank conflicts
@@ -94,9 +73,9 @@ __global__ void __launch_bounds__(256, (MT * NTW <= 8) ? 2 : 1) latent_attn_mma_
     const int tq = prefill ? ROWS / hg : 1;
     pdl_trigger();
     pdl_wait();
-    const int n_items = a.num_items ? min(*a.num_items, a.max_items) : a.items;
+    const int item1 = prefill ? a.items : min(a.cta_items[blockIdx.x + 1], a.max_items), step = prefill ? gridDim.x : 1;
 
-    for (int item = blockIdx.x; item < n_items; item += gridDim.x) {
+    for (int item = prefill ? blockIdx.x : a.cta_items[blockIdx.x]; item < item1; item += step) {
         const int r = a.item_req[item];
         if (r < 0 || r >= a.reqs) continue;
         const int q_base = a.qo_indptr[r], qlen = a.qo_indptr[r + 1] - q_base;
@@ -475,14 +454,21 @@ PIE_API int pie_latent_attn_mma_tiles(int heads, int row, int rank_pad) {
     return la_fixed_bytes(mt, row) + 2 * la_stage_bytes(row) <= 227 * 1024 ? mt : 0;
 }
 
+// The merge of a decode launch's split requests (also for the tcgen05 kernel).
+int pie_latent_merge(const LatentMmaArgs& a, cudaStream_t st) {
+    const cudaError_t e = launch_pdl(latent_merge_kernel, dim3((a.reqs * a.heads + 7) / 8), dim3(256), 0, st, (const float*)a.scratch,
+                                     a.req_item_indptr, (bf16*)a.out, a.heads, a.rank_pad, a.max_items, a.reqs);
+    return (int)(e != cudaSuccess ? e : cudaGetLastError());
+}
+
 PIE_API int pie_latent_attn_mma(const LatentMmaArgs* args, int num_ctas, cudaStream_t st) {
     LatentMmaArgs a = *args;
     const int mt = pie_latent_attn_mma_tiles(a.heads, a.row, a.rank_pad);
     if (!mt || a.rank_pad > a.row || a.page_size != 1 << a.page_shift || a.row > a.cache_row || a.cache_row % 8 ||
         num_ctas <= 0)
         return (int)cudaErrorInvalidValue;
-    if (a.item_end && (!a.scratch || !a.req_item_indptr || !a.num_items)) return (int)cudaErrorInvalidValue;
-    if (!a.num_items && a.items <= 0) return 0;
+    if (a.item_end && (!a.scratch || !a.req_item_indptr || !a.cta_items)) return (int)cudaErrorInvalidValue;
+    if (!a.item_end && a.items <= 0) return 0;
     const int fixed = la_fixed_bytes(mt, a.row), stage = la_stage_bytes(a.row);
     const int ntw = a.rank_pad <= 128 ? 2 : (a.rank_pad <= 256 ? 4 : 8);
     // two CTAs per SM where the registers allow it: half of the shared memory each
@@ -505,11 +491,7 @@ PIE_API int pie_latent_attn_mma(const LatentMmaArgs* args, int num_ctas, cudaStr
     else if (mt == 2) { if (ntw == 2) GO(2, 2) else if (ntw == 4) GO(2, 4) else GO(2, 8) }
     else { if (ntw == 2) GO(4, 2) else if (ntw == 4) GO(4, 4) else return (int)cudaErrorInvalidValue; }
 #undef GO
-    if (a.item_end) {
-        const cudaError_t e = launch_pdl(latent_merge_kernel, dim3((a.reqs * a.heads + 7) / 8), dim3(256), 0, st,
-                                         (const float*)a.scratch, a.req_item_indptr, (bf16*)a.out, a.heads, a.rank_pad, a.max_items, a.reqs);
-        if (e != cudaSuccess) return (int)e;
-    }
+    if (a.item_end) return pie_latent_merge(a, st);
     return (int)cudaGetLastError();
 }
 

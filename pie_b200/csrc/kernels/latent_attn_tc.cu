@@ -1,0 +1,375 @@
+// Latent decode attention on the 5th-generation tensor cores, with keys on the rows of the accumulators.
+//
+// The few query rows of a decode step (one token, up to 32 heads) would leave most of a 128-row MMA empty, so both
+// products are turned around: S^T = K Q^T has 128 keys as rows and the heads as columns, O^T += V^T P^T has 128 latent
+// columns as rows. The tile of cache rows in shared memory serves as K (K-major) and as V^T (MN-major) as it stands, and
+// every byte of it is read twice by the tensor cores and by nobody else.
+//   warp 0      TMA producer: the item's query rows; per tile the 128 keys' pages, as boxes of 16 rows x 64 columns with the
+//               128-byte swizzle, into a ring of two stages (all lanes look pages up and issue)
+//   warp 1      tcgen05.mma issuer: S^T of a tile into TMEM, and O^T of the tile before into its own TMEM columns once
+//               the softmax warps have handed over P
+//   warps 2-5   softmax, one key per thread: a column of S^T is a head, so its maximum is a warp reduction per head and an
+//               exchange between the four warps; exponentials against a reference maximum that follows the true one lazily
+//               (O^T is rescaled in TMEM only when a head's maximum outgrows it by 2^8); P as bf16 into a swizzled tile
+//               [heads][keys]. At the end of an item the sums are reduced and O^T leaves, normalised, for `out` (a request
+//               that was not split) or the split-KV scratch.
+// A CTA runs a contiguous range of work items: the keys of all requests are cut evenly over the CTAs.
+// Every wait is bounded; on a time-out the kernel records a status word and leaves.
+#include "latent_args.cuh"
+#include "tcgen05.cuh"
+
+namespace pie {
+using namespace sm100;
+
+constexpr int LT_HEADS = 32;                 // heads per CTA (columns of S^T and O^T)
+constexpr int LT_KEYS = 128;                 // keys per tile (rows of S^T)
+constexpr int LT_STAGES = 2;
+constexpr int LT_THREADS = 192;
+constexpr uint32_t LT_BLOCK = LT_KEYS * 128;           // 64 columns of a tile: 128 rows of 128 bytes
+constexpr uint32_t LT_QBLOCK = LT_HEADS * 128;
+constexpr uint32_t LT_P_BYTES = LT_HEADS * LT_KEYS * 2;
+constexpr float LT_RESCALE_LOG2 = 8.f;
+
+__host__ __device__ inline int lt_mtiles(int rank_pad) { return (rank_pad + 127) / 128; }
+__host__ __device__ inline int lt_blocks(int row, int rank_pad) {        // 64-column blocks: all of the row, and whole V^T tiles
+    const int k = (row + 63) / 64, v = 2 * lt_mtiles(rank_pad);
+    return k > v ? k : v;
+}
+__host__ __device__ inline uint32_t lt_smem(int row, int rank_pad) {
+    const uint32_t nb = lt_blocks(row, rank_pad);
+    return LT_STAGES * nb * LT_BLOCK + nb * LT_QBLOCK + LT_P_BYTES + 1024 /*align*/ + 256 /*barriers*/ + 8 * LT_HEADS * 4;
+}
+
+// MN-major SW128 operand: 64 elements of the contiguous dimension per 128-byte row, 8-row groups of the other dimension
+// 1024 bytes apart, the next 64 elements `lbo` bytes further.
+__device__ __forceinline__ uint64_t lt_desc_mn(uint32_t saddr, uint32_t lbo) {
+    uint64_t d = 0;
+    d |= (uint64_t)((saddr & 0x3FFFFu) >> 4);
+    d |= (uint64_t)(lbo >> 4) << 16;
+    d |= (uint64_t)(1024 >> 4) << 32;
+    d |= (uint64_t)1 << 46;
+    d |= (uint64_t)2 << 61;
+    return d;
+}
+__device__ __forceinline__ float lt_exp2(float x) {
+    float y;
+    asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
+    return y;
+}
+__device__ __forceinline__ float lt_warp_max(float x) {
+    float y;
+    asm volatile("redux.sync.max.f32 %0, %1, 0xffffffff;" : "=f"(y) : "f"(x));
+    return y;
+}
+__device__ __forceinline__ void lt_softmax_sync() { asm volatile("bar.sync 1, 128;" ::: "memory"); }
+
+// What every role derives from an item of the work list.
+struct LtItem {
+    int tok, k0, lo, hi, tiles;    // query token; first key loaded (a multiple of 16); visible keys [lo, hi); tiles of keys
+    const int* pages;
+    bool whole;                    // the request's only item: normalised output instead of a partial one
+};
+__device__ __forceinline__ LtItem lt_item(const LatentMmaArgs& a, int item) {
+    LtItem t;
+    const int r = a.item_req[item];
+    if (r < 0 || r >= a.reqs) {
+        t.tiles = 0;
+        t.whole = true;
+        return t;
+    }
+    const int kv_len = a.kv_lens[r];
+    t.tok = a.qo_indptr[r];
+    t.pages = a.page_indices + a.kv_page_indptr[r];
+    t.lo = max(max(0, kv_len - 1 - a.window_left), a.item_start[item]);
+    t.hi = min(kv_len, a.item_end[item]);
+    t.k0 = t.lo & ~15;
+    t.tiles = t.hi > t.lo ? (t.hi - t.k0 + LT_KEYS - 1) / LT_KEYS : 0;
+    t.whole = a.req_item_indptr[r + 1] - a.req_item_indptr[r] == 1;
+    return t;
+}
+
+// MT: 128-column tiles of the latent (rows of O^T).
+template <int MT>
+__global__ void __launch_bounds__(LT_THREADS, 1)
+latent_attn_tc_kernel(const __grid_constant__ CUtensorMap tma_q, const __grid_constant__ CUtensorMap tma_c, const LatentMmaArgs a,
+                      int* status) {
+    constexpr uint32_t TMEM_COLS = MT <= 1 ? 64 : 128;         // S^T, then MT x O^T, 32 columns each
+    extern __shared__ uint8_t lt_raw[];
+    const uint32_t raw = smem_addr(lt_raw), base = (raw + 1023u) & ~1023u;
+    uint8_t* base_ptr = lt_raw + (base - raw);
+    const int nb = lt_blocks(a.row, a.rank_pad);
+    const uint32_t stage_bytes = nb * LT_BLOCK;
+    const uint32_t k_s = base, q_s = k_s + LT_STAGES * stage_bytes, p_s = q_s + nb * LT_QBLOCK, bar0 = p_s + LT_P_BYTES;
+    auto k_full = [&](int s) { return bar0 + 8u * s; };
+    auto k_empty = [&](int s) { return bar0 + 16u + 8u * s; };
+    const uint32_t q_full = bar0 + 32, q_empty = bar0 + 40, s_full = bar0 + 48, p_full = bar0 + 56, o_final = bar0 + 64, o_free = bar0 + 72;
+    volatile uint32_t* tmem_slot = reinterpret_cast<volatile uint32_t*>(base_ptr + (bar0 - base) + 80);
+    float* mx_s = reinterpret_cast<float*>(base_ptr + (bar0 - base) + 256);      // [4 warps][heads]
+    float* l_s = mx_s + 4 * LT_HEADS;
+
+    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+    const int h0 = blockIdx.y * LT_HEADS, hn = min(LT_HEADS, a.heads - h0);
+    if (threadIdx.x == 0) {
+        for (int s = 0; s < LT_STAGES; ++s) {
+            mbar_init(k_full(s), 1);
+            mbar_init(k_empty(s), 1);
+        }
+        mbar_init(q_full, 1);
+        mbar_init(q_empty, 1);
+        mbar_init(s_full, 1);
+        mbar_init(p_full, 4);
+        mbar_init(o_final, 1);
+        mbar_init(o_free, 4);
+        fence_barrier_init();
+        fence_proxy_async();
+    }
+    if (warp == 1) {
+        tmem_alloc(smem_addr(const_cast<uint32_t*>(tmem_slot)), TMEM_COLS);
+        tmem_relinquish();
+    }
+    tc_fence_before();
+    __syncthreads();
+    tc_fence_after();
+    const uint32_t tmem_s = *tmem_slot, tmem_o = tmem_s + LT_HEADS;
+    pdl_trigger();
+    pdl_wait();
+    const int item0 = a.cta_items[blockIdx.x], item1 = min(a.cta_items[blockIdx.x + 1], a.max_items);
+
+    if (warp == 0) {
+        // ------------------------------------------------------ TMA producer
+        uint32_t g = 0, ni = 0;
+        bool ok = true;
+        for (int item = item0; item < item1 && ok; ++item) {
+            const LtItem t = lt_item(a, item);
+            if (t.tiles == 0) continue;
+            bool w = true;
+            if (lane == 0) {
+                w = mbar_wait(q_empty, (ni & 1u) ^ 1u, status, PIE_ERR_WAIT_TMA);
+                if (w) mbar_arrive_expect_tx(q_full, nb * LT_QBLOCK);
+            }
+            ok = __shfl_sync(0xffffffffu, (int)w, 0) != 0;
+            if (!ok) break;
+            ++ni;
+            for (int b = lane; b < nb; b += 32) tma_load_2d(q_s + b * LT_QBLOCK, &tma_q, q_full, b * 64, t.tok * a.heads + h0);
+            for (int j = 0; j < t.tiles && ok; ++j, ++g) {
+                const int s = g % LT_STAGES;
+                // a lane's boxes are all of one 16-key piece; a piece past the end reads zeros (rows outside the tensor)
+                const int key = t.k0 + j * LT_KEYS + (lane & 7) * 16;
+                const int row = key < t.hi ? (t.pages[key >> a.page_shift] << a.page_shift) + (key & (a.page_size - 1)) : a.cache_rows;
+                if (lane == 0) {
+                    w = mbar_wait(k_empty(s), ((g / LT_STAGES) & 1u) ^ 1u, status, PIE_ERR_WAIT_TMA);
+                    if (w) mbar_arrive_expect_tx(k_full(s), stage_bytes);
+                }
+                ok = __shfl_sync(0xffffffffu, (int)w, 0) != 0;
+                if (!ok) break;
+                for (int i = lane; i < 8 * nb; i += 32)
+                    tma_load_2d(k_s + s * stage_bytes + (i >> 3) * LT_BLOCK + (i & 7) * 2048, &tma_c, k_full(s), (i >> 3) * 64, row);
+            }
+        }
+        // no copy of this CTA may still be in flight when it exits
+        if (lane == 0) {
+            const uint32_t first = g > (uint32_t)LT_STAGES ? g - LT_STAGES : 0u;
+            for (uint32_t j = first; j < g; ++j)
+                mbar_wait(k_full(j % LT_STAGES), (j / LT_STAGES) & 1u, status, PIE_ERR_WAIT_TMA, 200000000ll);
+            if (ni > 0) mbar_wait(q_full, (ni - 1) & 1u, status, PIE_ERR_WAIT_TMA, 200000000ll);
+        }
+    } else if (warp == 1) {
+        // -------------------------------------------------------- MMA issuer
+        if (lane == 0) {
+            constexpr uint32_t idesc_s = make_idesc_bf16(LT_KEYS, LT_HEADS);
+            constexpr uint32_t idesc_o = make_idesc_bf16(128, LT_HEADS) | (1u << 15);      // A is MN-major
+            uint32_t g = 0, ni = 0;
+            bool ok = true;
+            for (int item = item0; item < item1 && ok; ++item) {
+                const LtItem t = lt_item(a, item);
+                if (t.tiles == 0) continue;
+                if (!mbar_wait(q_full, ni & 1u, status, PIE_ERR_WAIT_TMA)) { ok = false; break; }
+                for (int j = 0; j < t.tiles; ++j, ++g) {
+                    const int s = g % LT_STAGES;
+                    const uint32_t tile = k_s + s * stage_bytes;
+                    if (!mbar_wait(k_full(s), (g / LT_STAGES) & 1u, status, PIE_ERR_WAIT_TMA)) { ok = false; break; }
+                    tc_fence_after();
+                    for (int k = 0; k < (a.row >> 4); ++k)
+                        umma_bf16(tmem_s, make_smem_desc_sw128(tile + (k >> 2) * LT_BLOCK) + 2u * (k & 3),
+                                  make_smem_desc_sw128(q_s + (k >> 2) * LT_QBLOCK) + 2u * (k & 3), idesc_s, k != 0);
+                    // all products issued so far are complete when this arrives, the O^T of the tile before included
+                    umma_commit(s_full);
+                    if (j == t.tiles - 1) umma_commit(q_empty);
+                    if (!mbar_wait(p_full, g & 1u, status, PIE_ERR_WAIT_EPILOGUE)) { ok = false; break; }
+                    if (j == 0 && !mbar_wait(o_free, (ni & 1u) ^ 1u, status, PIE_ERR_WAIT_EPILOGUE)) { ok = false; break; }
+                    tc_fence_after();
+#pragma unroll
+                    for (int m = 0; m < MT; ++m)
+#pragma unroll
+                        for (int k = 0; k < LT_KEYS / 16; ++k)
+                            umma_bf16(tmem_o + m * LT_HEADS, lt_desc_mn(tile + 2 * m * LT_BLOCK + k * 2048, LT_BLOCK),
+                                      make_smem_desc_sw128(p_s + (k >> 2) * (LT_HEADS * 128)) + 2u * (k & 3), idesc_o, (j | k) != 0);
+                    umma_commit(k_empty(s));
+                    if (j == t.tiles - 1) umma_commit(o_final);
+                }
+                ++ni;
+            }
+        }
+    } else {
+        // ---------------------------------------- softmax: thread = key of the tile, lane = head in the exchanges
+        const int q4 = warp & 3;                         // the TMEM lane quarter this warp may access
+        const uint32_t quarter = (uint32_t)(q4 * 32) << 16;
+        const float thr = LT_RESCALE_LOG2 / a.scale_log2;
+        uint8_t* p_row = base_ptr + (p_s - base) + (q4 >> 1) * (LT_HEADS * 128);
+        const int kin = (q4 & 1) * 32 + lane;            // key within the 64-key half of P
+        float* lse = a.scratch + (size_t)a.max_items * a.heads * a.rank_pad;
+        uint32_t g = 0, ni = 0;
+        bool ok = true;
+        for (int item = item0; item < item1 && ok; ++item) {
+            const LtItem t = lt_item(a, item);
+            if (t.tiles == 0) {
+                if (!t.whole) {                          // a span that a narrower layer sees nothing of: no weight in the merge
+                    if (q4 == 0 && lane < hn) lse[(size_t)item * a.heads + h0 + lane] = -INFINITY;
+                    for (int i = threadIdx.x - 64; i < hn * a.rank_pad; i += 128)
+                        a.scratch[((size_t)item * a.heads + h0) * a.rank_pad + i] = 0.f;
+                }
+                continue;
+            }
+            float m_ref = -INFINITY, neg[LT_HEADS], l[LT_HEADS];
+#pragma unroll
+            for (int h = 0; h < LT_HEADS; ++h) neg[h] = l[h] = 0.f;
+            for (int j = 0; j < t.tiles; ++j, ++g) {
+                const bool got = mbar_wait(s_full, g & 1u, status, PIE_ERR_WAIT_MMA);
+                if (!__all_sync(0xffffffffu, got)) { ok = false; break; }
+                tc_fence_after();
+                uint32_t v[32];
+                tmem_ld_32x32(tmem_s + quarter, v);
+                tmem_ld_wait();
+                const int key = t.k0 + j * LT_KEYS + q4 * 32 + lane;
+                const bool see = key >= t.lo && key < t.hi;
+                float mine = -INFINITY;
+#pragma unroll
+                for (int h = 0; h < LT_HEADS; ++h) {
+                    if (!see) v[h] = __float_as_uint(-INFINITY);
+                    const float m = lt_warp_max(__uint_as_float(v[h]));
+                    if (lane == h) mine = m;
+                }
+                mx_s[q4 * LT_HEADS + lane] = mine;
+                lt_softmax_sync();
+                const float tmax = fmaxf(fmaxf(mx_s[lane], mx_s[LT_HEADS + lane]), fmaxf(mx_s[2 * LT_HEADS + lane], mx_s[3 * LT_HEADS + lane]));
+                if (__any_sync(0xffffffffu, tmax > m_ref + thr)) {
+                    const float m_new = fmaxf(m_ref, tmax);
+                    const float alpha = m_new == -INFINITY ? 1.f : lt_exp2((m_ref - m_new) * a.scale_log2);
+                    const float nl = m_new == -INFINITY ? 0.f : -m_new * a.scale_log2;
+                    m_ref = m_new;
+#pragma unroll
+                    for (int h = 0; h < LT_HEADS; ++h) {
+                        neg[h] = __shfl_sync(0xffffffffu, nl, h);
+                        l[h] *= __shfl_sync(0xffffffffu, alpha, h);
+                    }
+                    if (j > 0) {
+#pragma unroll
+                        for (int m = 0; m < MT; ++m) {
+                            uint32_t o[32];
+                            tmem_ld_32x32(tmem_o + quarter + m * LT_HEADS, o);
+                            tmem_ld_wait();
+#pragma unroll
+                            for (int h = 0; h < LT_HEADS; ++h)
+                                o[h] = __float_as_uint(__uint_as_float(o[h]) * __shfl_sync(0xffffffffu, alpha, h));
+                            tmem_st_32x32(tmem_o + quarter + m * LT_HEADS, o);
+                        }
+                        tmem_st_wait();
+                    }
+                }
+#pragma unroll
+                for (int h = 0; h < LT_HEADS; ++h) {
+                    const float p = lt_exp2(fmaf(__uint_as_float(v[h]), a.scale_log2, neg[h]));
+                    l[h] += p;
+                    *reinterpret_cast<bf16*>(p_row + h * 128 + (((kin >> 3) ^ (h & 7)) << 4) + (kin & 7) * 2) = __float2bfloat16(p);
+                }
+                fence_proxy_async();
+                tc_fence_before();
+                __syncwarp();
+                if (lane == 0) mbar_arrive(p_full);
+            }
+            if (!ok) break;
+            const bool done = mbar_wait(o_final, ni & 1u, status, PIE_ERR_WAIT_MMA);
+            if (!__all_sync(0xffffffffu, done)) { ok = false; break; }
+            ++ni;
+            tc_fence_after();
+            float mine = 0.f;
+#pragma unroll
+            for (int h = 0; h < LT_HEADS; ++h) {
+                const float sum = warp_sum(l[h]);
+                if (lane == h) mine = sum;
+            }
+            l_s[q4 * LT_HEADS + lane] = mine;
+            lt_softmax_sync();
+            const float lt = l_s[lane] + l_s[LT_HEADS + lane] + l_s[2 * LT_HEADS + lane] + l_s[3 * LT_HEADS + lane];
+            const float inv = lt > 0.f ? 1.f / lt : 0.f;
+            if (!t.whole && q4 == 0 && lane < hn)
+                lse[(size_t)item * a.heads + h0 + lane] = lt > 0.f ? m_ref * a.scale_log2 + log2f(lt) : -INFINITY;
+#pragma unroll
+            for (int m = 0; m < MT; ++m) {
+                uint32_t o[32];
+                tmem_ld_32x32(tmem_o + quarter + m * LT_HEADS, o);
+                tmem_ld_wait();
+                const int col = m * 128 + q4 * 32 + lane;
+#pragma unroll
+                for (int h = 0; h < LT_HEADS; ++h) {
+                    const float y = __uint_as_float(o[h]) * __shfl_sync(0xffffffffu, inv, h);
+                    if (h >= hn || col >= a.rank_pad) continue;
+                    if (t.whole)
+                        static_cast<bf16*>(a.out)[((size_t)t.tok * a.heads + h0 + h) * a.rank_pad + col] = __float2bfloat16(y);
+                    else
+                        a.scratch[((size_t)item * a.heads + h0 + h) * a.rank_pad + col] = y;
+                }
+            }
+            tc_fence_before();
+            __syncwarp();
+            if (lane == 0) mbar_arrive(o_free);
+        }
+    }
+    tc_fence_before();
+    __syncthreads();
+    if (warp == 1) {
+        __syncwarp();
+        tc_fence_after();
+        tmem_dealloc(tmem_s, TMEM_COLS);
+    }
+}
+
+}  // namespace pie
+
+using namespace pie;
+
+extern "C" int pie_make_tma_2d_bf16(CUtensorMap* map, const void* ptr, long rows, long cols, long ld, int box_rows);
+int pie_latent_merge(const LatentMmaArgs& a, cudaStream_t st);
+
+PIE_API int pie_latent_attn_tc_supported(int row, int rank_pad, int page_size) {
+    return row > 0 && row % 16 == 0 && rank_pad % 16 == 0 && rank_pad <= row && rank_pad <= 384 && page_size >= 16 &&
+           (page_size & (page_size - 1)) == 0 && lt_smem(row, rank_pad) <= 227 * 1024 ? 1 : 0;
+}
+
+// Decode only: one query token per request, work items cut over `num_ctas` CTAs (cta_items).
+PIE_API int pie_latent_attn_tc(const LatentMmaArgs* args, int num_ctas, int* status, cudaStream_t st) {
+    const LatentMmaArgs& a = *args;
+    if (!pie_latent_attn_tc_supported(a.row, a.rank_pad, a.page_size) || a.page_size != 1 << a.page_shift || a.row > a.cache_row ||
+        a.cache_row % 16 || !a.item_end || !a.scratch || !a.req_item_indptr || !a.cta_items || a.reqs <= 0 || num_ctas <= 0 || !status)
+        return (int)cudaErrorInvalidValue;
+    CUtensorMap tq, tc;
+    if (pie_make_tma_2d_bf16(&tq, a.q, (long)a.reqs * a.heads, a.row, a.row, LT_HEADS) != 0 ||
+        pie_make_tma_2d_bf16(&tc, a.cache, a.cache_rows, a.cache_row, a.cache_row, 16) != 0)
+        return (int)cudaErrorInvalidValue;
+    const uint32_t smem = lt_smem(a.row, a.rank_pad);
+    const dim3 grid(num_ctas, (a.heads + LT_HEADS - 1) / LT_HEADS);
+#define GO(M_)                                                                                                                       \
+    {                                                                                                                                \
+        cudaError_t e = cudaFuncSetAttribute(latent_attn_tc_kernel<M_>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);     \
+        if (e != cudaSuccess) return (int)e;                                                                                         \
+        e = launch_pdl(latent_attn_tc_kernel<M_>, grid, dim3(LT_THREADS), (size_t)smem, st, tq, tc, a, status);                      \
+        if (e != cudaSuccess) return (int)e;                                                                                         \
+    }
+    switch (lt_mtiles(a.rank_pad)) {
+        case 1: GO(1) break;
+        case 2: GO(2) break;
+        default: GO(3) break;
+    }
+#undef GO
+    return pie_latent_merge(a, st);
+}

@@ -206,6 +206,12 @@ class TorchDriver:
         # the widest window any layer needs (-1: some layer sees everything); layers that differ mask per call
         self.window_left = self.cfg.plan_window_left
         self.max_items = max_requests + self.num_ctas * 8
+        # CTAs a latent decode plan is cut for: one per SM where every layer runs on the tcgen05 kernel, else two
+        self.latent_ctas = 0
+        if cfg.latent is not None and self.cuda:
+            from ..ops import latent as lops
+            tc = self.dtype == torch.bfloat16 and all(lops.decode_on_tcgen05(s, page_size) for s in cfg.latent)
+            self.latent_ctas = ops.num_sms(self.device) * (1 if tc else 2)
         # shared-prefix decode plans: forks of one context read their common pages once per step
         import os as _os
         self._prefix_cache: dict = {}
@@ -424,6 +430,8 @@ class TorchDriver:
             item_start=s.d("item_start"), item_end=s.d("item_end"), req_item_indptr=s.d("req_item_indptr"),
             num_items=s.d("num_items"), scratch=self.scratch, max_items=self.max_items, num_reqs=rb,
             num_ctas=self.num_ctas, page_size=self.page_size, window_left=self.window_left, kv_lens=s.d("kv_lens"))
+        if self.cfg.latent is not None:
+            plan.num_ctas, plan.cta_items = self.latent_ctas, s.d("item_slot", self.latent_ctas + 1)
         if cascade:
             plan.item_slot, plan.item_tile, plan.tile_members = s.d("item_slot"), s.d("item_tile"), s.d("tile_members")
         return ForwardInputs(tokens=s.d("tokens", rb), positions=s.d("positions", rb), slots=s.d("slots", rb),
@@ -481,8 +489,12 @@ class TorchDriver:
             self.stats["cascade_tokens_saved"] = self.stats.get("cascade_tokens_saved", 0) + plan.shared_tokens
         else:
             plan = None
-            item_req, st, en, indptr = ops.plan_decode_items(kv_lens, self.model.hkv, self.num_ctas, self.max_items,
-                                                             window_left=self.window_left, even=self.cfg.latent is not None)
+            if self.cfg.latent is not None:
+                item_req, st, en, indptr, cta_items = ops.plan_even_items(kv_lens, self.latent_ctas, self.max_items, self.window_left)
+                s.h("item_slot")[:len(cta_items)] = cta_items
+            else:
+                item_req, st, en, indptr = ops.plan_decode_items(kv_lens, self.model.hkv, self.num_ctas, self.max_items,
+                                                                 window_left=self.window_left)
             ni = len(item_req)
             s.h("item_req")[:ni], s.h("item_start")[:ni], s.h("item_end")[:ni] = item_req, st, en
         s.h("req_item_indptr")[:r + 1] = indptr
@@ -536,6 +548,7 @@ class TorchDriver:
             s.h("kv_page_indptr")[:rb + 1] = 0
             s.h("req_item_indptr")[:rb + 1] = 0
             s.h("num_items")[0] = 0
+            s.h("item_slot")[:] = 0            # no CTA has an item (latent decode plans)
             s.upload("tile_qstart")
             self.graphs[key] = self._capture(rb, cascade)
             n += 1

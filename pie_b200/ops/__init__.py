@@ -572,28 +572,21 @@ _DECODE_UNITS_PER_CTA = int(os.environ.get("PIE_DECODE_UNITS", "4"))
 
 
 def plan_decode_items(kv_lens: np.ndarray, hkv: int, target_ctas: int, max_items: int = 0,
-                      min_chunk: int = 256, window_left: int = -1, even: bool = False):
+                      min_chunk: int = 256, window_left: int = -1):
     """Split each request's KV range into chunks so that items*hkv fills the machine. With a
     sliding window only the last window_left + 1 keys are covered, from the 16-token boundary
     at or below the first visible key (the kernel masks the keys below it).
 
-    `even`: as many items as CTAs instead of several per CTA, equal parts of a request.
     Returns (item_req, item_start, item_end, req_item_indptr) as int32 arrays.
     """
     full_lens = np.asarray(kv_lens, dtype=np.int64)
     lo = np.zeros_like(full_lens)
     if window_left >= 0:
-        lo = np.maximum(0, full_lens - 1 - window_left) // (1 if even else 16) * (1 if even else 16)
+        lo = np.maximum(0, full_lens - 1 - window_left) // 16 * 16
     kv_lens = full_lens - lo
     total = int(kv_lens.sum())
     chunk = max(min_chunk, -(-total * hkv // max(1, target_ctas * _DECODE_UNITS_PER_CTA)))
     chunk = -(-chunk // 16) * 16
-    if even:
-        # one CTA per item, for kernels that pay per item: as many items as fit one wave of CTAs (whole requests if they
-        # alone fill it), a request's keys in equal parts
-        chunk = max(64, -(-total // max(1, target_ctas)))
-        while int(np.maximum(1, -(-kv_lens // chunk)).sum()) > max(target_ctas, len(kv_lens)):
-            chunk += -(-chunk // 8)
     while True:
         n_items = np.maximum(1, -(-kv_lens // chunk))
         if max_items <= 0 or int(n_items.sum()) <= max_items:
@@ -604,12 +597,39 @@ def plan_decode_items(kv_lens: np.ndarray, hkv: int, target_ctas: int, max_items
     tot = int(indptr[-1])
     item_req = np.repeat(np.arange(len(kv_lens), dtype=np.int32), n_items)
     within = np.arange(tot, dtype=np.int64) - np.repeat(indptr[:-1].astype(np.int64), n_items)
-    if even:
-        chunk = -(-kv_lens // n_items)[item_req]
     start = within * chunk
     end = np.minimum(start + chunk, kv_lens[item_req])
     start, end = start + lo[item_req], end + lo[item_req]
     return item_req, start.astype(np.int32), end.astype(np.int32), indptr
+
+
+def plan_even_items(kv_lens: np.ndarray, ctas: int, max_items: int = 0, window_left: int = -1, min_keys: int = 128):
+    """The keys of all requests (a sliding window's worth each) laid end to end and cut evenly over `ctas` CTAs, on 16-key
+    boundaries: for kernels whose CTAs pay per work item. A CTA gets no less than `min_keys`, the rest then stay idle.
+
+    Returns (item_req, item_start, item_end, req_item_indptr, cta_items) as int32 arrays; CTA c runs the items
+    cta_items[c] .. cta_items[c + 1] - 1."""
+    kv = np.asarray(kv_lens, dtype=np.int64)
+    lo = np.maximum(0, kv - 1 - window_left) // 16 * 16 if window_left >= 0 else np.zeros_like(kv)
+    span = -(-np.maximum(kv - lo, 1) // 16)                         # in units of 16 keys
+    ends = np.cumsum(span)
+    starts = ends - span
+    total = int(ends[-1]) if len(kv) else 0
+    n = max(1, min(ctas, total * 16 // min_keys))
+    if max_items > 0:
+        n = min(n, max(1, max_items - len(kv)))
+    cuts = total * np.arange(n + 1, dtype=np.int64) // n
+    at = np.unique(np.concatenate([starts, cuts]))
+    at = at[at < total]
+    req = np.searchsorted(ends, at, side="right")
+    stop = np.minimum(np.append(at[1:], total), ends[req])
+    start = lo[req] + (at - starts[req]) * 16
+    end = np.minimum(lo[req] + (stop - starts[req]) * 16, kv[req])
+    indptr = np.searchsorted(req, np.arange(len(kv) + 1))
+    cta_items = np.full(ctas + 1, len(at), dtype=np.int64)
+    cta_items[:n] = np.searchsorted(at, cuts[:-1])
+    i32 = lambda a: a.astype(np.int32)
+    return i32(req), i32(start), i32(end), i32(indptr), i32(cta_items)
 
 
 @dataclass
@@ -791,6 +811,7 @@ class DecodePlan:
     item_tile: Optional[torch.Tensor] = None
     tile_members: Optional[torch.Tensor] = None
     kv_lens: Optional[torch.Tensor] = None
+    cta_items: Optional[torch.Tensor] = None    # plans of `plan_even_items`: the items of every CTA (num_ctas + 1 offsets)
 
 
 def decode_scratch_floats(max_items: int, hq: int, head_dim: int) -> int:

@@ -69,6 +69,8 @@ _SIGNATURES = {
     "pie_gemm_bf16_stream": [p, p, p, p, p, i32, p, i32, i32, i32, i32, i32, i32, p, i32, p],
     "pie_latent_attn_mma_tiles": [i32, i32, i32],
     "pie_latent_attn_mma": [p, i32, p],
+    "pie_latent_attn_tc_supported": [i32, i32, i32],
+    "pie_latent_attn_tc": [p, i32, p, p],
     "pie_small_product": [p, p],
     "pie_projected_prefill_attn_tc": [p, p, p, p, p, p, p, p, i32, p, p, p, i32, i32, i32, i32, i32, i32, f32, i32, p, p],
     "pie_bias_xielu": [p, i32, p, p, i32, i32, i32, p],

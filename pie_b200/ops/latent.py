@@ -4,6 +4,7 @@ go to `csrc/kernels/latent*.cu` (bf16 when serving, float32 on the 32-bit path),
 from __future__ import annotations
 
 import ctypes as C
+import os
 
 import numpy as np
 import torch
@@ -29,8 +30,8 @@ LatentAttnArgs = _struct("LatentAttnArgs", ("q cache page_indices kv_page_indptr
                          ("n heads row rank_pad cache_row page_size window_left", i32), ("scale", f32))
 
 LatentMmaArgs = _struct("LatentMmaArgs", ("q cache page_indices kv_page_indptr item_req item_start item_end req_item_indptr "
-                                          "num_items qo_indptr kv_lens mask_bits mask_word_indptr out scratch", p),
-                        ("items max_items heads row rank_pad cache_row page_size window_left stages reqs page_shift", i32),
+                                          "cta_items qo_indptr kv_lens mask_bits mask_word_indptr out scratch", p),
+                        ("items max_items heads row rank_pad cache_row page_size window_left stages reqs page_shift cache_rows", i32),
                         ("scale_log2", f32))
 SmallProductArgs = _struct("SmallProductArgs", ("x w out", p), ("x_tok x_head w_head w_row out_tok out_head", i64),
                            ("n heads m k k_total out_f32", i32))
@@ -107,6 +108,12 @@ def per_head(x, w, out):
     return out
 
 
+def decode_on_tcgen05(spec, page_size: int) -> bool:
+    """Whether bf16 decode of this mixer runs on the tcgen05 kernel (PIE_LATENT_TC=0: never; then mma.sync)."""
+    return os.environ.get("PIE_LATENT_TC", "1") != "0" and \
+        bool(fn("pie_latent_attn_tc_supported")(spec.row, spec.rank_pad, page_size))
+
+
 def latent_attention(q, cache, plan, rs, slots, spec, page_size: int, window_left: int):
     """Softmax over the visible cache rows of q [N, heads, row] . row * scale; returns the weighted latents
     [N, heads, rank_pad]. The absorbed form: keys and values of every head are the rows themselves. Decode splits a
@@ -130,12 +137,15 @@ def latent_attention(q, cache, plan, rs, slots, spec, page_size: int, window_lef
     a = LatentMmaArgs(q=ptr(q), cache=ptr(cache), page_indices=ptr(plan.page_indices), kv_page_indptr=ptr(plan.kv_page_indptr),
                       qo_indptr=ptr(rs.qo_indptr), kv_lens=ptr(plan.kv_lens), out=ptr(out), heads=spec.heads, row=spec.row,
                       rank_pad=spec.rank_pad, cache_row=cache.shape[-1], page_size=page_size, window_left=window_left,
-                      reqs=len(rs.slots_host), page_shift=page_size.bit_length() - 1, scale_log2=spec.scale * 1.4426950408889634)
-    ctas = ops.num_sms(q.device) * 2
+                      reqs=len(rs.slots_host), page_shift=page_size.bit_length() - 1,
+                      cache_rows=cache.shape[0] * cache.shape[1], scale_log2=spec.scale * 1.4426950408889634)
     if decode:
         a.item_req, a.item_start, a.item_end = ptr(plan.item_req), ptr(plan.item_start), ptr(plan.item_end)
-        a.req_item_indptr, a.num_items, a.scratch = ptr(plan.req_item_indptr), ptr(plan.num_items), ptr(plan.scratch)
-        a.max_items = plan.max_items
+        a.req_item_indptr, a.cta_items, a.scratch = ptr(plan.req_item_indptr), ptr(plan.cta_items), ptr(plan.scratch)
+        a.max_items, ctas = plan.max_items, plan.num_ctas
+        if decode_on_tcgen05(spec, page_size):
+            check(fn("pie_latent_attn_tc")(C.byref(a), ctas, ptr(ops.kernel_status(q.device)), stream_ptr()), "latent_attn_tc")
+            return out
     else:
         key, rows = ("absorbed", spec.heads), 16 * tiles
         if key not in plan.derived:

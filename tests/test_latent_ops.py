@@ -140,17 +140,17 @@ def paged(c, kr, s, page, dt, dev, seed=0):
     return cache.to(dev, dt), ids.tolist()
 
 
-def plans(qlen, kv, ids, page, window, dev, s, even=True):
+def plans(qlen, kv, ids, page, window, dev, s):
     t = lambda a: torch.from_numpy(np.ascontiguousarray(a, np.int32)).to(dev)
     qo, ptr_ = np.array([0, qlen]), np.array([0, len(ids)])
     host = ops.AttnBatch(qo, ptr_, np.asarray(ids), np.array([kv]), None, window - 1)
     if dev == "cpu":
         return host
     if qlen == 1:
-        ir, st, en, ip = ops.plan_decode_items(np.array([kv]), 1, 9, 64, window_left=window - 1, even=even)
+        ir, st, en, ip, ci = ops.plan_even_items(np.array([kv]), 3, 64, window - 1, min_keys=32)
         scratch = torch.empty(ops.decode_scratch_floats(64, s.heads, s.row), device=dev)
-        return ops.DecodePlan(t(ids), t(ptr_), t(ir), t(st), t(en), t(ip), t([len(ir)]), scratch, 64, 1, 9, page, window - 1,
-                              kv_lens=t([kv]))
+        return ops.DecodePlan(t(ids), t(ptr_), t(ir), t(st), t(en), t(ip), t([len(ir)]), scratch, 64, 1, 3, page, window - 1,
+                              kv_lens=t([kv]), cta_items=t(ci))
     tr, tq = ops.plan_prefill_tiles(qo, 1, 256, [kv])
     return ops.PrefillPlan(t(ids), t(ptr_), t(qo), t([kv]), t(tr), t(tq), len(tr), page, window_left=window - 1, tile_rows=256, host=host)
 
