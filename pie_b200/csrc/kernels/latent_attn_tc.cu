@@ -6,13 +6,13 @@
 // every byte of it is read twice by the tensor cores and by nobody else.
 //   warp 0      TMA producer: the item's query rows; per tile the 128 keys' pages, as boxes of 16 rows x 64 columns with the
 //               128-byte swizzle, into a ring of two stages (all lanes look pages up and issue)
-//   warp 1      tcgen05.mma issuer: S^T of a tile into TMEM, and O^T of the tile before into its own TMEM columns once
-//               the softmax warps have handed over P
-//   warps 2-5   softmax, one key per thread: a column of S^T is a head, so its maximum is a warp reduction per head and an
-//               exchange between the four warps; exponentials against a reference maximum that follows the true one lazily
-//               (O^T is rescaled in TMEM only when a head's maximum outgrows it by 2^8); P as bf16 into a swizzled tile
-//               [heads][keys]. At the end of an item the sums are reduced and O^T leaves, normalised, for `out` (a request
-//               that was not split) or the split-KV scratch.
+//   warp 1      tcgen05.mma issuer: S^T of a tile into one of two TMEM buffers, a tile ahead where the keys have arrived, and
+//               O^T into its own TMEM columns once the softmax warps have handed over P
+//   warps 2-9   softmax, two groups of four warps with 16 heads each, one key per thread: a column of S^T is a head, so its
+//               maximum is a warp reduction per head and an exchange between the group's four warps; exponentials
+//               against a reference maximum that follows the true one lazily (O^T is rescaled in TMEM only when a head's
+//               maximum outgrows it by 2^8); P as bf16 into a swizzled tile [heads][keys]. At the end of an item the sums are
+//               reduced and O^T leaves, normalised, for `out` (a request that was not split) or the split-KV scratch.
 // A CTA runs a contiguous range of work items: the keys of all requests are cut evenly over the CTAs.
 // Every wait is bounded; on a time-out the kernel records a status word and leaves.
 #include "latent_args.cuh"
@@ -24,7 +24,8 @@ using namespace sm100;
 constexpr int LT_HEADS = 32;                 // heads per CTA (columns of S^T and O^T)
 constexpr int LT_KEYS = 128;                 // keys per tile (rows of S^T)
 constexpr int LT_STAGES = 2;
-constexpr int LT_THREADS = 192;
+constexpr int LT_HALF = LT_HEADS / 2;        // heads per softmax group
+constexpr int LT_THREADS = 64 + 256;
 constexpr uint32_t LT_BLOCK = LT_KEYS * 128;           // 64 columns of a tile: 128 rows of 128 bytes
 constexpr uint32_t LT_QBLOCK = LT_HEADS * 128;
 constexpr uint32_t LT_P_BYTES = LT_HEADS * LT_KEYS * 2;
@@ -37,7 +38,7 @@ __host__ __device__ inline int lt_blocks(int row, int rank_pad) {        // 64-c
 }
 __host__ __device__ inline uint32_t lt_smem(int row, int rank_pad) {
     const uint32_t nb = lt_blocks(row, rank_pad);
-    return LT_STAGES * nb * LT_BLOCK + nb * LT_QBLOCK + LT_P_BYTES + 1024 /*align*/ + 256 /*barriers*/ + 8 * LT_HEADS * 4;
+    return LT_STAGES * nb * LT_BLOCK + nb * LT_QBLOCK + 2 * LT_P_BYTES + 1024 /*align*/ + 256 /*barriers*/ + 12 * LT_HEADS * 4 /*exchanges*/;
 }
 
 // MN-major SW128 operand: 64 elements of the contiguous dimension per 128-byte row, 8-row groups of the other dimension
@@ -61,7 +62,23 @@ __device__ __forceinline__ float lt_warp_max(float x) {
     asm volatile("redux.sync.max.f32 %0, %1, 0xffffffff;" : "=f"(y) : "f"(x));
     return y;
 }
-__device__ __forceinline__ void lt_softmax_sync() { asm volatile("bar.sync 1, 128;" ::: "memory"); }
+__device__ __forceinline__ void lt_group_sync(int group) { asm volatile("bar.sync %0, 128;" ::"r"(group + 1) : "memory"); }
+// 32 lanes x 16 columns of 32-bit accumulators
+__device__ __forceinline__ void lt_tmem_ld(uint32_t taddr, uint32_t (&v)[16]) {
+    asm volatile(
+        "tcgen05.ld.sync.aligned.32x32b.x16.b32 {%0,%1,%2,%3,%4,%5,%6,%7,%8,%9,%10,%11,%12,%13,%14,%15}, [%16];\n"
+        : "=r"(v[0]), "=r"(v[1]), "=r"(v[2]), "=r"(v[3]), "=r"(v[4]), "=r"(v[5]), "=r"(v[6]), "=r"(v[7]), "=r"(v[8]), "=r"(v[9]),
+          "=r"(v[10]), "=r"(v[11]), "=r"(v[12]), "=r"(v[13]), "=r"(v[14]), "=r"(v[15])
+        : "r"(taddr)
+        : "memory");
+}
+__device__ __forceinline__ void lt_tmem_st(uint32_t taddr, const uint32_t (&v)[16]) {
+    asm volatile(
+        "tcgen05.st.sync.aligned.32x32b.x16.b32 [%0], {%1,%2,%3,%4,%5,%6,%7,%8,%9,%10,%11,%12,%13,%14,%15,%16};\n" ::"r"(taddr),
+        "r"(v[0]), "r"(v[1]), "r"(v[2]), "r"(v[3]), "r"(v[4]), "r"(v[5]), "r"(v[6]), "r"(v[7]), "r"(v[8]), "r"(v[9]), "r"(v[10]),
+        "r"(v[11]), "r"(v[12]), "r"(v[13]), "r"(v[14]), "r"(v[15])
+        : "memory");
+}
 
 // What every role derives from an item of the work list.
 struct LtItem {
@@ -93,19 +110,22 @@ template <int MT>
 __global__ void __launch_bounds__(LT_THREADS, 1)
 latent_attn_tc_kernel(const __grid_constant__ CUtensorMap tma_q, const __grid_constant__ CUtensorMap tma_c, const LatentMmaArgs a,
                       int* status) {
-    constexpr uint32_t TMEM_COLS = MT <= 1 ? 64 : 128;         // S^T, then MT x O^T, 32 columns each
+    constexpr uint32_t TMEM_COLS = MT <= 2 ? 128 : 256;        // two S^T, then MT x O^T, 32 columns each
     extern __shared__ uint8_t lt_raw[];
     const uint32_t raw = smem_addr(lt_raw), base = (raw + 1023u) & ~1023u;
     uint8_t* base_ptr = lt_raw + (base - raw);
     const int nb = lt_blocks(a.row, a.rank_pad);
     const uint32_t stage_bytes = nb * LT_BLOCK;
-    const uint32_t k_s = base, q_s = k_s + LT_STAGES * stage_bytes, p_s = q_s + nb * LT_QBLOCK, bar0 = p_s + LT_P_BYTES;
+    const uint32_t k_s = base, q_s = k_s + LT_STAGES * stage_bytes, p_s = q_s + nb * LT_QBLOCK, bar0 = p_s + 2 * LT_P_BYTES;
     auto k_full = [&](int s) { return bar0 + 8u * s; };
     auto k_empty = [&](int s) { return bar0 + 16u + 8u * s; };
-    const uint32_t q_full = bar0 + 32, q_empty = bar0 + 40, s_full = bar0 + 48, p_full = bar0 + 56, o_final = bar0 + 64, o_free = bar0 + 72;
-    volatile uint32_t* tmem_slot = reinterpret_cast<volatile uint32_t*>(base_ptr + (bar0 - base) + 80);
-    float* mx_s = reinterpret_cast<float*>(base_ptr + (bar0 - base) + 256);      // [4 warps][heads]
-    float* l_s = mx_s + 4 * LT_HEADS;
+    const uint32_t q_full = bar0 + 32, q_empty = bar0 + 40, o_final = bar0 + 48, o_free = bar0 + 56, pv_done = bar0 + 64;
+    // one per buffer: two tiles may be under way, and a parity wait tells apart neighbouring phases only
+    auto s_full = [&](uint32_t n) { return bar0 + 72u + 8u * (n & 1u); };
+    auto p_full = [&](uint32_t n) { return bar0 + 88u + 8u * (n & 1u); };
+    volatile uint32_t* tmem_slot = reinterpret_cast<volatile uint32_t*>(base_ptr + (bar0 - base) + 104);
+    float* mx_s = reinterpret_cast<float*>(base_ptr + (bar0 - base) + 256);      // [2 tiles][2 groups][4 warps][heads]
+    float* l_s = mx_s + 8 * LT_HEADS;                                           // [2 groups][4 warps][heads]
 
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     const int h0 = blockIdx.y * LT_HEADS, hn = min(LT_HEADS, a.heads - h0);
@@ -116,10 +136,13 @@ latent_attn_tc_kernel(const __grid_constant__ CUtensorMap tma_q, const __grid_co
         }
         mbar_init(q_full, 1);
         mbar_init(q_empty, 1);
-        mbar_init(s_full, 1);
-        mbar_init(p_full, 4);
+        for (int b = 0; b < 2; ++b) {
+            mbar_init(s_full(b), 1);
+            mbar_init(p_full(b), 8);
+        }
         mbar_init(o_final, 1);
-        mbar_init(o_free, 4);
+        mbar_init(o_free, 8);
+        mbar_init(pv_done, 1);
         fence_barrier_init();
         fence_proxy_async();
     }
@@ -130,7 +153,7 @@ latent_attn_tc_kernel(const __grid_constant__ CUtensorMap tma_q, const __grid_co
     tc_fence_before();
     __syncthreads();
     tc_fence_after();
-    const uint32_t tmem_s = *tmem_slot, tmem_o = tmem_s + LT_HEADS;
+    const uint32_t tmem_s = *tmem_slot, tmem_o = tmem_s + 2 * LT_HEADS;
     pdl_trigger();
     pdl_wait();
     const int item0 = a.cta_items[blockIdx.x], item1 = min(a.cta_items[blockIdx.x + 1], a.max_items);
@@ -184,39 +207,60 @@ latent_attn_tc_kernel(const __grid_constant__ CUtensorMap tma_q, const __grid_co
                 const LtItem t = lt_item(a, item);
                 if (t.tiles == 0) continue;
                 if (!mbar_wait(q_full, ni & 1u, status, PIE_ERR_WAIT_TMA)) { ok = false; break; }
+                // S^T of tile n (counted over all items) into TMEM buffer n & 1
+                auto issue_s = [&](uint32_t n, bool last) {
+                    const uint32_t tile = k_s + (n % LT_STAGES) * stage_bytes;
+                    tc_fence_after();
+                    for (int k = 0; k < (a.row >> 4); ++k)
+                        umma_bf16(tmem_s + (n & 1u) * LT_HEADS, make_smem_desc_sw128(tile + (k >> 2) * LT_BLOCK) + 2u * (k & 3),
+                                  make_smem_desc_sw128(q_s + (k >> 2) * LT_QBLOCK) + 2u * (k & 3), idesc_s, k != 0);
+                    // arrives when all products issued so far are complete, O^T of the tile before the last included
+                    umma_commit(s_full(n));
+                    if (last) umma_commit(q_empty);
+                };
+                auto keys_ready = [&](uint32_t n) {
+                    return mbar_wait(k_full(n % LT_STAGES), (n / LT_STAGES) & 1u, status, PIE_ERR_WAIT_TMA);
+                };
+                if (!keys_ready(g)) { ok = false; break; }
+                issue_s(g, t.tiles == 1);
                 for (int j = 0; j < t.tiles; ++j, ++g) {
                     const int s = g % LT_STAGES;
                     const uint32_t tile = k_s + s * stage_bytes;
-                    if (!mbar_wait(k_full(s), (g / LT_STAGES) & 1u, status, PIE_ERR_WAIT_TMA)) { ok = false; break; }
-                    tc_fence_after();
-                    for (int k = 0; k < (a.row >> 4); ++k)
-                        umma_bf16(tmem_s, make_smem_desc_sw128(tile + (k >> 2) * LT_BLOCK) + 2u * (k & 3),
-                                  make_smem_desc_sw128(q_s + (k >> 2) * LT_QBLOCK) + 2u * (k & 3), idesc_s, k != 0);
-                    // all products issued so far are complete when this arrives, the O^T of the tile before included
-                    umma_commit(s_full);
-                    if (j == t.tiles - 1) umma_commit(q_empty);
-                    if (!mbar_wait(p_full, g & 1u, status, PIE_ERR_WAIT_EPILOGUE)) { ok = false; break; }
+                    const bool more = j + 1 < t.tiles;
+                    // the next tile's scores go first where its keys are there: the softmax then finds them finished
+                    const bool ahead = more && mbar_try_wait(k_full((g + 1) % LT_STAGES), ((g + 1) / LT_STAGES) & 1u);
+                    if (ahead) issue_s(g + 1, j + 2 == t.tiles);
+                    if (!mbar_wait(p_full(g), (g >> 1) & 1u, status, PIE_ERR_WAIT_EPILOGUE)) { ok = false; break; }
                     if (j == 0 && !mbar_wait(o_free, (ni & 1u) ^ 1u, status, PIE_ERR_WAIT_EPILOGUE)) { ok = false; break; }
                     tc_fence_after();
+                    const uint32_t p_tile = p_s + (g & 1u) * LT_P_BYTES;
 #pragma unroll
                     for (int m = 0; m < MT; ++m)
 #pragma unroll
                         for (int k = 0; k < LT_KEYS / 16; ++k)
                             umma_bf16(tmem_o + m * LT_HEADS, lt_desc_mn(tile + 2 * m * LT_BLOCK + k * 2048, LT_BLOCK),
-                                      make_smem_desc_sw128(p_s + (k >> 2) * (LT_HEADS * 128)) + 2u * (k & 3), idesc_o, (j | k) != 0);
+                                      make_smem_desc_sw128(p_tile + (k >> 2) * (LT_HEADS * 128)) + 2u * (k & 3), idesc_o, (j | k) != 0);
                     umma_commit(k_empty(s));
-                    if (j == t.tiles - 1) umma_commit(o_final);
+                    umma_commit(pv_done);
+                    if (!more) umma_commit(o_final);
+                    if (more && !ahead) {
+                        if (!keys_ready(g + 1)) { ok = false; break; }
+                        issue_s(g + 1, j + 2 == t.tiles);
+                    }
                 }
                 ++ni;
             }
         }
     } else {
-        // ---------------------------------------- softmax: thread = key of the tile, lane = head in the exchanges
-        const int q4 = warp & 3;                         // the TMEM lane quarter this warp may access
+        // ------------------- softmax: thread = key of the tile, lane = head of the group in the exchanges
+        const int q4 = warp & 3, group = (warp - 2) >> 2, hb = group * LT_HALF;      // q4: the TMEM lane quarter of this warp
         const uint32_t quarter = (uint32_t)(q4 * 32) << 16;
         const float thr = LT_RESCALE_LOG2 / a.scale_log2;
-        uint8_t* p_row = base_ptr + (p_s - base) + (q4 >> 1) * (LT_HEADS * 128);
         const int kin = (q4 & 1) * 32 + lane;            // key within the 64-key half of P
+        uint8_t* p_row = base_ptr + (p_s - base) + (q4 >> 1) * (LT_HEADS * 128) + hb * 128 + (kin & 7) * 2;
+        float* lx = l_s + group * 4 * LT_HALF;
+        const int hl = lane & (LT_HALF - 1), head = h0 + hb + hl;       // of this lane in the exchanges
+        const bool owner = q4 == 0 && lane < LT_HALF && hb + hl < hn;
         float* lse = a.scratch + (size_t)a.max_items * a.heads * a.rank_pad;
         uint32_t g = 0, ni = 0;
         bool ok = true;
@@ -224,68 +268,73 @@ latent_attn_tc_kernel(const __grid_constant__ CUtensorMap tma_q, const __grid_co
             const LtItem t = lt_item(a, item);
             if (t.tiles == 0) {
                 if (!t.whole) {                          // a span that a narrower layer sees nothing of: no weight in the merge
-                    if (q4 == 0 && lane < hn) lse[(size_t)item * a.heads + h0 + lane] = -INFINITY;
-                    for (int i = threadIdx.x - 64; i < hn * a.rank_pad; i += 128)
+                    if (owner) lse[(size_t)item * a.heads + head] = -INFINITY;
+                    for (int i = threadIdx.x - 64; i < hn * a.rank_pad; i += 256)
                         a.scratch[((size_t)item * a.heads + h0) * a.rank_pad + i] = 0.f;
                 }
                 continue;
             }
-            float m_ref = -INFINITY, neg[LT_HEADS], l[LT_HEADS];
+            float m_ref = -INFINITY, neg[LT_HALF], l[LT_HALF];
 #pragma unroll
-            for (int h = 0; h < LT_HEADS; ++h) neg[h] = l[h] = 0.f;
+            for (int h = 0; h < LT_HALF; ++h) neg[h] = l[h] = 0.f;
             for (int j = 0; j < t.tiles; ++j, ++g) {
-                const bool got = mbar_wait(s_full, g & 1u, status, PIE_ERR_WAIT_MMA);
+                const bool got = mbar_wait(s_full(g), (g >> 1) & 1u, status, PIE_ERR_WAIT_MMA);
                 if (!__all_sync(0xffffffffu, got)) { ok = false; break; }
                 tc_fence_after();
-                uint32_t v[32];
-                tmem_ld_32x32(tmem_s + quarter, v);
+                uint32_t v[LT_HALF];
+                lt_tmem_ld(tmem_s + quarter + (g & 1u) * LT_HEADS + hb, v);
                 tmem_ld_wait();
                 const int key = t.k0 + j * LT_KEYS + q4 * 32 + lane;
                 const bool see = key >= t.lo && key < t.hi;
                 float mine = -INFINITY;
 #pragma unroll
-                for (int h = 0; h < LT_HEADS; ++h) {
+                for (int h = 0; h < LT_HALF; ++h) {
                     if (!see) v[h] = __float_as_uint(-INFINITY);
                     const float m = lt_warp_max(__uint_as_float(v[h]));
-                    if (lane == h) mine = m;
+                    if (hl == h) mine = m;
                 }
-                mx_s[q4 * LT_HEADS + lane] = mine;
-                lt_softmax_sync();
-                const float tmax = fmaxf(fmaxf(mx_s[lane], mx_s[LT_HEADS + lane]), fmaxf(mx_s[2 * LT_HEADS + lane], mx_s[3 * LT_HEADS + lane]));
+                float* mx = mx_s + ((g & 1u) * 2 + group) * 4 * LT_HALF;      // a warp may be a tile ahead of a reader
+                if (lane < LT_HALF) mx[q4 * LT_HALF + hl] = mine;
+                lt_group_sync(group);
+                const float tmax = fmaxf(fmaxf(mx[hl], mx[LT_HALF + hl]), fmaxf(mx[2 * LT_HALF + hl], mx[3 * LT_HALF + hl]));
                 if (__any_sync(0xffffffffu, tmax > m_ref + thr)) {
                     const float m_new = fmaxf(m_ref, tmax);
                     const float alpha = m_new == -INFINITY ? 1.f : lt_exp2((m_ref - m_new) * a.scale_log2);
                     const float nl = m_new == -INFINITY ? 0.f : -m_new * a.scale_log2;
                     m_ref = m_new;
 #pragma unroll
-                    for (int h = 0; h < LT_HEADS; ++h) {
+                    for (int h = 0; h < LT_HALF; ++h) {
                         neg[h] = __shfl_sync(0xffffffffu, nl, h);
                         l[h] *= __shfl_sync(0xffffffffu, alpha, h);
                     }
                     if (j > 0) {
+                        const bool settled = mbar_wait(pv_done, (g - 1) & 1u, status, PIE_ERR_WAIT_MMA);
+                        if (!__all_sync(0xffffffffu, settled)) { ok = false; break; }
+                        tc_fence_after();
 #pragma unroll
                         for (int m = 0; m < MT; ++m) {
-                            uint32_t o[32];
-                            tmem_ld_32x32(tmem_o + quarter + m * LT_HEADS, o);
+                            uint32_t o[LT_HALF];
+                            lt_tmem_ld(tmem_o + quarter + m * LT_HEADS + hb, o);
                             tmem_ld_wait();
 #pragma unroll
-                            for (int h = 0; h < LT_HEADS; ++h)
+                            for (int h = 0; h < LT_HALF; ++h)
                                 o[h] = __float_as_uint(__uint_as_float(o[h]) * __shfl_sync(0xffffffffu, alpha, h));
-                            tmem_st_32x32(tmem_o + quarter + m * LT_HEADS, o);
+                            lt_tmem_st(tmem_o + quarter + m * LT_HEADS + hb, o);
                         }
                         tmem_st_wait();
                     }
                 }
+                uint8_t* prow = p_row + (g & 1u) * LT_P_BYTES;
 #pragma unroll
-                for (int h = 0; h < LT_HEADS; ++h) {
+                for (int h = 0; h < LT_HALF; ++h) {
                     const float p = lt_exp2(fmaf(__uint_as_float(v[h]), a.scale_log2, neg[h]));
                     l[h] += p;
-                    *reinterpret_cast<bf16*>(p_row + h * 128 + (((kin >> 3) ^ (h & 7)) << 4) + (kin & 7) * 2) = __float2bfloat16(p);
+                    *reinterpret_cast<bf16*>(prow + h * 128 + (((kin >> 3) ^ (h & 7)) << 4)) = __float2bfloat16(p);
                 }
                 fence_proxy_async();
                 tc_fence_before();
                 __syncwarp();
-                if (lane == 0) mbar_arrive(p_full);
+                if (lane == 0) mbar_arrive(p_full(g));
             }
             if (!ok) break;
             const bool done = mbar_wait(o_final, ni & 1u, status, PIE_ERR_WAIT_MMA);
@@ -294,30 +343,29 @@ latent_attn_tc_kernel(const __grid_constant__ CUtensorMap tma_q, const __grid_co
             tc_fence_after();
             float mine = 0.f;
 #pragma unroll
-            for (int h = 0; h < LT_HEADS; ++h) {
+            for (int h = 0; h < LT_HALF; ++h) {
                 const float sum = warp_sum(l[h]);
-                if (lane == h) mine = sum;
+                if (hl == h) mine = sum;
             }
-            l_s[q4 * LT_HEADS + lane] = mine;
-            lt_softmax_sync();
-            const float lt = l_s[lane] + l_s[LT_HEADS + lane] + l_s[2 * LT_HEADS + lane] + l_s[3 * LT_HEADS + lane];
+            if (lane < LT_HALF) lx[q4 * LT_HALF + hl] = mine;
+            lt_group_sync(group);
+            const float lt = lx[hl] + lx[LT_HALF + hl] + lx[2 * LT_HALF + hl] + lx[3 * LT_HALF + hl];
             const float inv = lt > 0.f ? 1.f / lt : 0.f;
-            if (!t.whole && q4 == 0 && lane < hn)
-                lse[(size_t)item * a.heads + h0 + lane] = lt > 0.f ? m_ref * a.scale_log2 + log2f(lt) : -INFINITY;
+            if (!t.whole && owner) lse[(size_t)item * a.heads + head] = lt > 0.f ? m_ref * a.scale_log2 + log2f(lt) : -INFINITY;
 #pragma unroll
             for (int m = 0; m < MT; ++m) {
-                uint32_t o[32];
-                tmem_ld_32x32(tmem_o + quarter + m * LT_HEADS, o);
+                uint32_t o[LT_HALF];
+                lt_tmem_ld(tmem_o + quarter + m * LT_HEADS + hb, o);
                 tmem_ld_wait();
                 const int col = m * 128 + q4 * 32 + lane;
 #pragma unroll
-                for (int h = 0; h < LT_HEADS; ++h) {
+                for (int h = 0; h < LT_HALF; ++h) {
                     const float y = __uint_as_float(o[h]) * __shfl_sync(0xffffffffu, inv, h);
-                    if (h >= hn || col >= a.rank_pad) continue;
+                    if (hb + h >= hn || col >= a.rank_pad) continue;
                     if (t.whole)
-                        static_cast<bf16*>(a.out)[((size_t)t.tok * a.heads + h0 + h) * a.rank_pad + col] = __float2bfloat16(y);
+                        static_cast<bf16*>(a.out)[((size_t)t.tok * a.heads + h0 + hb + h) * a.rank_pad + col] = __float2bfloat16(y);
                     else
-                        a.scratch[((size_t)item * a.heads + h0 + h) * a.rank_pad + col] = y;
+                        a.scratch[((size_t)item * a.heads + h0 + hb + h) * a.rank_pad + col] = y;
                 }
             }
             tc_fence_before();
