@@ -38,7 +38,7 @@ __host__ __device__ inline int lt_blocks(int row, int rank_pad) {        // 64-c
 }
 __host__ __device__ inline uint32_t lt_smem(int row, int rank_pad) {
     const uint32_t nb = lt_blocks(row, rank_pad);
-    return LT_STAGES * nb * LT_BLOCK + nb * LT_QBLOCK + 2 * LT_P_BYTES + 1024 /*align*/ + 256 /*barriers*/ + 12 * LT_HEADS * 4 /*exchanges*/;
+    return LT_STAGES * nb * LT_BLOCK + nb * LT_QBLOCK + 2 * LT_P_BYTES + 1024 /*align*/ + 256 /*barriers*/ + 8 * LT_HEADS * 4 /*exchanges*/ + 128 + 8;
 }
 
 // MN-major SW128 operand: 64 elements of the contiguous dimension per 128-byte row, 8-row groups of the other dimension
@@ -63,6 +63,19 @@ __device__ __forceinline__ float lt_warp_max(float x) {
     return y;
 }
 __device__ __forceinline__ void lt_group_sync(int group) { asm volatile("bar.sync %0, 128;" ::"r"(group + 1) : "memory"); }
+// Barrier of a group that also tells whether any of its threads passed `flag`.
+__device__ __forceinline__ bool lt_group_any(int group, bool flag) {
+    uint32_t r;
+    asm volatile(
+        "{\n"
+        ".reg .pred p, q;\n"
+        "setp.ne.b32 q, %1, 0;\n"
+        "bar.red.or.pred p, %2, 128, q;\n"
+        "selp.u32 %0, 1, 0, p;\n"
+        "}\n"
+        : "=r"(r) : "r"((uint32_t)flag), "r"(group + 1) : "memory");
+    return r != 0;
+}
 // 32 lanes x 16 columns of 32-bit accumulators
 __device__ __forceinline__ void lt_tmem_ld(uint32_t taddr, uint32_t (&v)[16]) {
     asm volatile(
@@ -80,23 +93,24 @@ __device__ __forceinline__ void lt_tmem_st(uint32_t taddr, const uint32_t (&v)[1
         : "memory");
 }
 
-// What every role derives from an item of the work list.
+// What every role derives from an item of the work list. A warp looks 32 items up at once, one per lane.
 struct LtItem {
     int tok, k0, lo, hi, tiles;    // query token; first key loaded (a multiple of 16); visible keys [lo, hi); tiles of keys
-    const int* pages;
-    bool whole;                    // the request's only item: normalised output instead of a partial one
-};
-__device__ __forceinline__ LtItem lt_item(const LatentMmaArgs& a, int item) {
-    LtItem t;
-    const int r = a.item_req[item];
-    if (r < 0 || r >= a.reqs) {
-        t.tiles = 0;
-        t.whole = true;
-        return t;
+    int pages;                     // offset of the request's page table
+    int whole;                     // the request's only item: normalised output instead of a partial one
+    __device__ __forceinline__ LtItem of_lane(int src) const {
+        const unsigned all = 0xffffffffu;
+        return LtItem{__shfl_sync(all, tok, src),   __shfl_sync(all, k0, src),    __shfl_sync(all, lo, src),   __shfl_sync(all, hi, src),
+                      __shfl_sync(all, tiles, src), __shfl_sync(all, pages, src), __shfl_sync(all, whole, src)};
     }
+};
+__device__ __forceinline__ LtItem lt_item(const LatentMmaArgs& a, int item, int item1) {
+    LtItem t{0, 0, 0, 0, 0, 0, 1};
+    const int r = item < item1 ? a.item_req[item] : -1;
+    if (r < 0 || r >= a.reqs) return t;
     const int kv_len = a.kv_lens[r];
     t.tok = a.qo_indptr[r];
-    t.pages = a.page_indices + a.kv_page_indptr[r];
+    t.pages = a.kv_page_indptr[r];
     t.lo = max(max(0, kv_len - 1 - a.window_left), a.item_start[item]);
     t.hi = min(kv_len, a.item_end[item]);
     t.k0 = t.lo & ~15;
@@ -124,8 +138,10 @@ latent_attn_tc_kernel(const __grid_constant__ CUtensorMap tma_q, const __grid_co
     auto s_full = [&](uint32_t n) { return bar0 + 72u + 8u * (n & 1u); };
     auto p_full = [&](uint32_t n) { return bar0 + 88u + 8u * (n & 1u); };
     volatile uint32_t* tmem_slot = reinterpret_cast<volatile uint32_t*>(base_ptr + (bar0 - base) + 104);
-    float* mx_s = reinterpret_cast<float*>(base_ptr + (bar0 - base) + 256);      // [2 tiles][2 groups][4 warps][heads]
-    float* l_s = mx_s + 8 * LT_HEADS;                                           // [2 groups][4 warps][heads]
+    float* mx_s = reinterpret_cast<float*>(base_ptr + (bar0 - base) + 256);      // [2 groups][4 warps][heads]
+    float* l_s = mx_s + 4 * LT_HEADS;                                           // [2 groups][4 warps][heads]
+    int* tiles_s = reinterpret_cast<int*>(l_s + 4 * LT_HEADS);                  // tiles of the MMA warp's next 32 items
+    volatile int* failed = tiles_s + 32;                                        // [2 groups] a warp of the group gave up on a wait
 
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     const int h0 = blockIdx.y * LT_HEADS, hn = min(LT_HEADS, a.heads - h0);
@@ -143,6 +159,7 @@ latent_attn_tc_kernel(const __grid_constant__ CUtensorMap tma_q, const __grid_co
         mbar_init(o_final, 1);
         mbar_init(o_free, 8);
         mbar_init(pv_done, 1);
+        failed[0] = failed[1] = 0;
         fence_barrier_init();
         fence_proxy_async();
     }
@@ -162,8 +179,10 @@ latent_attn_tc_kernel(const __grid_constant__ CUtensorMap tma_q, const __grid_co
         // ------------------------------------------------------ TMA producer
         uint32_t g = 0, ni = 0;
         bool ok = true;
+        LtItem mine{};
         for (int item = item0; item < item1 && ok; ++item) {
-            const LtItem t = lt_item(a, item);
+            if (((item - item0) & 31) == 0) mine = lt_item(a, item + lane, item1);
+            const LtItem t = mine.of_lane((item - item0) & 31);
             if (t.tiles == 0) continue;
             bool w = true;
             if (lane == 0) {
@@ -178,7 +197,7 @@ latent_attn_tc_kernel(const __grid_constant__ CUtensorMap tma_q, const __grid_co
                 const int s = g % LT_STAGES;
                 // a lane's boxes are all of one 16-key piece; a piece past the end reads zeros (rows outside the tensor)
                 const int key = t.k0 + j * LT_KEYS + (lane & 7) * 16;
-                const int row = key < t.hi ? (t.pages[key >> a.page_shift] << a.page_shift) + (key & (a.page_size - 1)) : a.cache_rows;
+                const int row = key < t.hi ? (a.page_indices[t.pages + (key >> a.page_shift)] << a.page_shift) + (key & (a.page_size - 1)) : a.cache_rows;
                 if (lane == 0) {
                     w = mbar_wait(k_empty(s), ((g / LT_STAGES) & 1u) ^ 1u, status, PIE_ERR_WAIT_TMA);
                     if (w) mbar_arrive_expect_tx(k_full(s), stage_bytes);
@@ -198,14 +217,18 @@ latent_attn_tc_kernel(const __grid_constant__ CUtensorMap tma_q, const __grid_co
         }
     } else if (warp == 1) {
         // -------------------------------------------------------- MMA issuer
-        if (lane == 0) {
-            constexpr uint32_t idesc_s = make_idesc_bf16(LT_KEYS, LT_HEADS);
-            constexpr uint32_t idesc_o = make_idesc_bf16(128, LT_HEADS) | (1u << 15);      // A is MN-major
-            uint32_t g = 0, ni = 0;
-            bool ok = true;
-            for (int item = item0; item < item1 && ok; ++item) {
-                const LtItem t = lt_item(a, item);
-                if (t.tiles == 0) continue;
+        constexpr uint32_t idesc_s = make_idesc_bf16(LT_KEYS, LT_HEADS);
+        constexpr uint32_t idesc_o = make_idesc_bf16(128, LT_HEADS) | (1u << 15);      // A is MN-major
+        uint32_t g = 0, ni = 0;
+        bool ok = true;
+        for (int chunk = item0; chunk < item1; chunk += 32) {
+            __syncwarp();
+            tiles_s[lane] = lt_item(a, chunk + lane, item1).tiles;
+            __syncwarp();
+            if (lane != 0) continue;
+            for (int i = 0; i < min(32, item1 - chunk) && ok; ++i) {
+                const int tiles = tiles_s[i];
+                if (tiles == 0) continue;
                 if (!mbar_wait(q_full, ni & 1u, status, PIE_ERR_WAIT_TMA)) { ok = false; break; }
                 // S^T of tile n (counted over all items) into TMEM buffer n & 1
                 auto issue_s = [&](uint32_t n, bool last) {
@@ -222,14 +245,14 @@ latent_attn_tc_kernel(const __grid_constant__ CUtensorMap tma_q, const __grid_co
                     return mbar_wait(k_full(n % LT_STAGES), (n / LT_STAGES) & 1u, status, PIE_ERR_WAIT_TMA);
                 };
                 if (!keys_ready(g)) { ok = false; break; }
-                issue_s(g, t.tiles == 1);
-                for (int j = 0; j < t.tiles; ++j, ++g) {
+                issue_s(g, tiles == 1);
+                for (int j = 0; j < tiles; ++j, ++g) {
                     const int s = g % LT_STAGES;
                     const uint32_t tile = k_s + s * stage_bytes;
-                    const bool more = j + 1 < t.tiles;
+                    const bool more = j + 1 < tiles;
                     // the next tile's scores go first where its keys are there: the softmax then finds them finished
                     const bool ahead = more && mbar_try_wait(k_full((g + 1) % LT_STAGES), ((g + 1) / LT_STAGES) & 1u);
-                    if (ahead) issue_s(g + 1, j + 2 == t.tiles);
+                    if (ahead) issue_s(g + 1, j + 2 == tiles);
                     if (!mbar_wait(p_full(g), (g >> 1) & 1u, status, PIE_ERR_WAIT_EPILOGUE)) { ok = false; break; }
                     if (j == 0 && !mbar_wait(o_free, (ni & 1u) ^ 1u, status, PIE_ERR_WAIT_EPILOGUE)) { ok = false; break; }
                     tc_fence_after();
@@ -245,7 +268,7 @@ latent_attn_tc_kernel(const __grid_constant__ CUtensorMap tma_q, const __grid_co
                     if (!more) umma_commit(o_final);
                     if (more && !ahead) {
                         if (!keys_ready(g + 1)) { ok = false; break; }
-                        issue_s(g + 1, j + 2 == t.tiles);
+                        issue_s(g + 1, j + 2 == tiles);
                     }
                 }
                 ++ni;
@@ -255,7 +278,6 @@ latent_attn_tc_kernel(const __grid_constant__ CUtensorMap tma_q, const __grid_co
         // ------------------- softmax: thread = key of the tile, lane = head of the group in the exchanges
         const int q4 = warp & 3, group = (warp - 2) >> 2, hb = group * LT_HALF;      // q4: the TMEM lane quarter of this warp
         const uint32_t quarter = (uint32_t)(q4 * 32) << 16;
-        const float thr = LT_RESCALE_LOG2 / a.scale_log2;
         const int kin = (q4 & 1) * 32 + lane;            // key within the 64-key half of P
         uint8_t* p_row = base_ptr + (p_s - base) + (q4 >> 1) * (LT_HEADS * 128) + hb * 128 + (kin & 7) * 2;
         float* lx = l_s + group * 4 * LT_HALF;
@@ -264,8 +286,10 @@ latent_attn_tc_kernel(const __grid_constant__ CUtensorMap tma_q, const __grid_co
         float* lse = a.scratch + (size_t)a.max_items * a.heads * a.rank_pad;
         uint32_t g = 0, ni = 0;
         bool ok = true;
+        LtItem own{};
         for (int item = item0; item < item1 && ok; ++item) {
-            const LtItem t = lt_item(a, item);
+            if (((item - item0) & 31) == 0) own = lt_item(a, item + lane, item1);
+            const LtItem t = own.of_lane((item - item0) & 31);
             if (t.tiles == 0) {
                 if (!t.whole) {                          // a span that a narrower layer sees nothing of: no weight in the merge
                     if (owner) lse[(size_t)item * a.heads + head] = -INFINITY;
@@ -278,26 +302,35 @@ latent_attn_tc_kernel(const __grid_constant__ CUtensorMap tma_q, const __grid_co
 #pragma unroll
             for (int h = 0; h < LT_HALF; ++h) neg[h] = l[h] = 0.f;
             for (int j = 0; j < t.tiles; ++j, ++g) {
-                const bool got = mbar_wait(s_full(g), (g >> 1) & 1u, status, PIE_ERR_WAIT_MMA);
-                if (!__all_sync(0xffffffffu, got)) { ok = false; break; }
+                // a wait that ran out is told to the group at its next barrier, which every warp reaches: all leave together
+                if (!mbar_wait(s_full(g), (g >> 1) & 1u, status, PIE_ERR_WAIT_MMA)) failed[group] = 1;
+                __syncwarp();
                 tc_fence_after();
                 uint32_t v[LT_HALF];
                 lt_tmem_ld(tmem_s + quarter + (g & 1u) * LT_HEADS + hb, v);
                 tmem_ld_wait();
                 const int key = t.k0 + j * LT_KEYS + q4 * 32 + lane;
                 const bool see = key >= t.lo && key < t.hi;
-                float mine = -INFINITY;
+                float e[LT_HALF], top = -INFINITY;        // exponents against the reference
 #pragma unroll
                 for (int h = 0; h < LT_HALF; ++h) {
-                    if (!see) v[h] = __float_as_uint(-INFINITY);
-                    const float m = lt_warp_max(__uint_as_float(v[h]));
-                    if (hl == h) mine = m;
+                    e[h] = see ? fmaf(__uint_as_float(v[h]), a.scale_log2, neg[h]) : -INFINITY;
+                    top = fmaxf(top, e[h]);
                 }
-                float* mx = mx_s + ((g & 1u) * 2 + group) * 4 * LT_HALF;      // a warp may be a tile ahead of a reader
-                if (lane < LT_HALF) mx[q4 * LT_HALF + hl] = mine;
-                lt_group_sync(group);
-                const float tmax = fmaxf(fmaxf(mx[hl], mx[LT_HALF + hl]), fmaxf(mx[2 * LT_HALF + hl], mx[3 * LT_HALF + hl]));
-                if (__any_sync(0xffffffffu, tmax > m_ref + thr)) {
+                // while no head's score outgrows its reference by 2^8 (the first tile sets it), nobody needs a maximum
+                const bool outgrown = lt_group_any(group, j == 0 || top > LT_RESCALE_LOG2);
+                if (failed[group]) { ok = false; break; }
+                if (outgrown) {
+                    float mine = -INFINITY;
+#pragma unroll
+                    for (int h = 0; h < LT_HALF; ++h) {
+                        const float m = lt_warp_max(see ? __uint_as_float(v[h]) : -INFINITY);
+                        if (hl == h) mine = m;
+                    }
+                    float* mx = mx_s + group * 4 * LT_HALF;
+                    if (lane < LT_HALF) mx[q4 * LT_HALF + hl] = mine;
+                    lt_group_sync(group);
+                    const float tmax = fmaxf(fmaxf(mx[hl], mx[LT_HALF + hl]), fmaxf(mx[2 * LT_HALF + hl], mx[3 * LT_HALF + hl]));
                     const float m_new = fmaxf(m_ref, tmax);
                     const float alpha = m_new == -INFINITY ? 1.f : lt_exp2((m_ref - m_new) * a.scale_log2);
                     const float nl = m_new == -INFINITY ? 0.f : -m_new * a.scale_log2;
@@ -306,10 +339,11 @@ latent_attn_tc_kernel(const __grid_constant__ CUtensorMap tma_q, const __grid_co
                     for (int h = 0; h < LT_HALF; ++h) {
                         neg[h] = __shfl_sync(0xffffffffu, nl, h);
                         l[h] *= __shfl_sync(0xffffffffu, alpha, h);
+                        e[h] = see ? fmaf(__uint_as_float(v[h]), a.scale_log2, neg[h]) : -INFINITY;
                     }
                     if (j > 0) {
-                        const bool settled = mbar_wait(pv_done, (g - 1) & 1u, status, PIE_ERR_WAIT_MMA);
-                        if (!__all_sync(0xffffffffu, settled)) { ok = false; break; }
+                        if (!mbar_wait(pv_done, (g - 1) & 1u, status, PIE_ERR_WAIT_MMA)) failed[group] = 1;
+                        __syncwarp();
                         tc_fence_after();
 #pragma unroll
                         for (int m = 0; m < MT; ++m) {
@@ -327,7 +361,7 @@ latent_attn_tc_kernel(const __grid_constant__ CUtensorMap tma_q, const __grid_co
                 uint8_t* prow = p_row + (g & 1u) * LT_P_BYTES;
 #pragma unroll
                 for (int h = 0; h < LT_HALF; ++h) {
-                    const float p = lt_exp2(fmaf(__uint_as_float(v[h]), a.scale_log2, neg[h]));
+                    const float p = lt_exp2(e[h]);
                     l[h] += p;
                     *reinterpret_cast<bf16*>(prow + h * 128 + (((kin >> 3) ^ (h & 7)) << 4)) = __float2bfloat16(p);
                 }
@@ -337,8 +371,8 @@ latent_attn_tc_kernel(const __grid_constant__ CUtensorMap tma_q, const __grid_co
                 if (lane == 0) mbar_arrive(p_full(g));
             }
             if (!ok) break;
-            const bool done = mbar_wait(o_final, ni & 1u, status, PIE_ERR_WAIT_MMA);
-            if (!__all_sync(0xffffffffu, done)) { ok = false; break; }
+            if (!mbar_wait(o_final, ni & 1u, status, PIE_ERR_WAIT_MMA)) failed[group] = 1;
+            __syncwarp();
             ++ni;
             tc_fence_after();
             float mine = 0.f;
@@ -349,6 +383,7 @@ latent_attn_tc_kernel(const __grid_constant__ CUtensorMap tma_q, const __grid_co
             }
             if (lane < LT_HALF) lx[q4 * LT_HALF + hl] = mine;
             lt_group_sync(group);
+            if (failed[group]) break;
             const float lt = lx[hl] + lx[LT_HALF + hl] + lx[2 * LT_HALF + hl] + lx[3 * LT_HALF + hl];
             const float inv = lt > 0.f ? 1.f / lt : 0.f;
             if (!t.whole && owner) lse[(size_t)item * a.heads + head] = lt > 0.f ? m_ref * a.scale_log2 + log2f(lt) : -INFINITY;
