@@ -102,8 +102,10 @@ def main(argv=None):
         q = torch.randn(n_req * n, 32, 128, **bf)
         w_kv = torch.randn(32 * 2 * 128, s.row, **bf) * 0.06
         out = torch.empty(n_req * n, 32 * 128, **bf)
-        sec = _time(lambda: lops.projected_prefill_attention(q, cache, plan, w_kv, s, 16, w - 1, out), flush)
         kvb = n_req * n * 32 * 256 * 2
+        sec = _time(lambda: ops.gemm(cache[:-1].view(-1, s.row), w_kv), flush)
+        report(f"  of it the projection, {n_req} x {n}", sec, n_req * n * s.row * 2 + kvb, 2.0 * n_req * n * 32 * 256 * s.row)
+        sec = _time(lambda: lops.projected_prefill_attention(q, cache, plan, w_kv, s, 16, w - 1, out), flush)
         report(f"latent prefill with its projection, {n_req} x {n}", sec, n_req * n * (32 * 256 * 2 + s.row * 2) + 2 * kvb,
                pairs * 32 * 4.0 * 128 + 2.0 * n_req * n * 32 * 256 * s.row)
         tr, tq = ops.plan_prefill_tiles(qo, 4, 256, kv)

@@ -197,7 +197,8 @@ latent_attn_tc_kernel(const __grid_constant__ CUtensorMap tma_q, const __grid_co
                 const int s = g % LT_STAGES;
                 // a lane's boxes are all of one 16-key piece; a piece past the end reads zeros (rows outside the tensor)
                 const int key = t.k0 + j * LT_KEYS + (lane & 7) * 16;
-                const int row = key < t.hi ? (a.page_indices[t.pages + (key >> a.page_shift)] << a.page_shift) + (key & (a.page_size - 1)) : a.cache_rows;
+                const int row = key < t.hi ? (a.page_indices[t.pages + (key >> a.page_shift)] << a.page_shift) + (key & (a.page_size - 1))
+                                           : a.cache_rows;
                 if (lane == 0) {
                     w = mbar_wait(k_empty(s), ((g / LT_STAGES) & 1u) ^ 1u, status, PIE_ERR_WAIT_TMA);
                     if (w) mbar_arrive_expect_tx(k_full(s), stage_bytes);
@@ -377,10 +378,11 @@ latent_attn_tc_kernel(const __grid_constant__ CUtensorMap tma_q, const __grid_co
             tc_fence_after();
             float mine = 0.f;
 #pragma unroll
-            for (int h = 0; h < LT_HALF; ++h) {
-                const float sum = warp_sum(l[h]);
-                if (hl == h) mine = sum;
-            }
+            for (int d = 16; d > 0; d >>= 1)              // sixteen independent chains at a time
+#pragma unroll
+                for (int h = 0; h < LT_HALF; ++h) l[h] += __shfl_xor_sync(0xffffffffu, l[h], d);
+#pragma unroll
+            for (int h = 0; h < LT_HALF; ++h) mine = hl == h ? l[h] : mine;
             if (lane < LT_HALF) lx[q4 * LT_HALF + hl] = mine;
             lt_group_sync(group);
             if (failed[group]) break;
@@ -388,21 +390,28 @@ latent_attn_tc_kernel(const __grid_constant__ CUtensorMap tma_q, const __grid_co
             const float inv = lt > 0.f ? 1.f / lt : 0.f;
             if (!t.whole && owner) lse[(size_t)item * a.heads + head] = lt > 0.f ? m_ref * a.scale_log2 + log2f(lt) : -INFINITY;
 #pragma unroll
+            for (int h = 0; h < LT_HALF; ++h) l[h] = __shfl_sync(0xffffffffu, inv, h);
+            const int heads_here = min(LT_HALF, hn - hb);
+#pragma unroll
             for (int m = 0; m < MT; ++m) {
                 uint32_t o[LT_HALF];
                 lt_tmem_ld(tmem_o + quarter + m * LT_HEADS + hb, o);
                 tmem_ld_wait();
                 const int col = m * 128 + q4 * 32 + lane;
+                if (col >= a.rank_pad) continue;
+                if (t.whole) {
+                    bf16* dst = static_cast<bf16*>(a.out) + ((size_t)t.tok * a.heads + h0 + hb) * a.rank_pad + col;
 #pragma unroll
-                for (int h = 0; h < LT_HALF; ++h) {
-                    const float y = __uint_as_float(o[h]) * __shfl_sync(0xffffffffu, inv, h);
-                    if (hb + h >= hn || col >= a.rank_pad) continue;
-                    if (t.whole)
-                        static_cast<bf16*>(a.out)[((size_t)t.tok * a.heads + h0 + hb + h) * a.rank_pad + col] = __float2bfloat16(y);
-                    else
-                        a.scratch[((size_t)item * a.heads + h0 + hb + h) * a.rank_pad + col] = y;
+                    for (int h = 0; h < LT_HALF; ++h)
+                        if (h < heads_here) dst[h * a.rank_pad] = __float2bfloat16(__uint_as_float(o[h]) * l[h]);
+                } else {
+                    float* dst = a.scratch + ((size_t)item * a.heads + h0 + hb) * a.rank_pad + col;
+#pragma unroll
+                    for (int h = 0; h < LT_HALF; ++h)
+                        if (h < heads_here) dst[h * a.rank_pad] = __uint_as_float(o[h]) * l[h];
                 }
             }
+            __syncwarp();
             tc_fence_before();
             __syncwarp();
             if (lane == 0) mbar_arrive(o_free);
@@ -437,7 +446,7 @@ PIE_API int pie_latent_attn_tc(const LatentMmaArgs* args, int num_ctas, int* sta
         return (int)cudaErrorInvalidValue;
     CUtensorMap tq, tc;
     if (pie_make_tma_2d_bf16(&tq, a.q, (long)a.reqs * a.heads, a.row, a.row, LT_HEADS) != 0 ||
-        pie_make_tma_2d_bf16(&tc, a.cache, a.cache_rows, a.cache_row, a.cache_row, 16) != 0)
+        pie_make_tma_2d_bf16(&tc, a.cache, a.cache_rows, a.row, a.cache_row, 16) != 0)
         return (int)cudaErrorInvalidValue;
     const uint32_t smem = lt_smem(a.row, a.rank_pad);
     const dim3 grid(num_ctas, (a.heads + LT_HEADS - 1) / LT_HEADS);
