@@ -2,7 +2,7 @@
 
     bin/trace_run --model DIR --dtype bfloat16|float32 --out DIR --max-tokens N < steps.jsonl
 
-A step is one JSON line ``{"step": 0, "entries": [{"id": "a", "tokens": [5, 17], "want": [1]}], "end": ["b"]}``: the next
+A step is one JSON line ``{"step": 4, "entries": [{"id": "q7", "tokens": [812, 9], "want": [1]}], "end": ["q3"]}``: the next
 tokens of each request and the places among them whose logits are wanted; requests in `end` are finished after the
 step and give back what they hold. The logits of a step go to ``DIR/<step>.f32`` (little-endian 32-bit floats,
 [wanted, vocab]), and ``done <step>`` is printed. Nothing is sampled.
