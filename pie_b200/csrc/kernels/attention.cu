@@ -610,31 +610,7 @@ using namespace pie;
         if (!ok_) return (int)cudaErrorInvalidValue;                   \
     } while (0)
 
-// Status word of the current device for the bounds reports of the decode kernel (see
-// pie_set_status_word); null when the embedder registered none: the kernel then only clamps.
-namespace {
-constexpr int kStatusDevices = 64;
-int* g_status_word[kStatusDevices] = {};
-int* status_word() {
-    int dev = -1;
-    if (cudaGetDevice(&dev) != cudaSuccess || dev < 0 || dev >= kStatusDevices) return nullptr;
-    return g_status_word[dev];
-}
-}  // namespace
-
-// Register a device int32 (on the current device) that kernels without a status argument set to a
-// PieKernelStatus code when they drop work; pass null to unregister.
-PIE_API int pie_set_status_word(int* word) {
-    int dev = -1;
-    cudaError_t e = cudaGetDevice(&dev);
-    if (e != cudaSuccess) return (int)e;
-    if (dev < 0 || dev >= kStatusDevices) return (int)cudaErrorInvalidValue;
-    g_status_word[dev] = word;
-    return 0;
-}
-
-// The status word registered for the current device (null if none): for kernels of other files.
-PIE_API int* pie_status_word_current() { return status_word(); }
+extern "C" int* pie_status_word_current();      // elementwise.cu
 
 // Merge pass of split-KV decode on its own (used by the fp8-KV decode kernel of attention_kv8.cu).
 PIE_API int pie_decode_merge(const float* o_part, const float* lse_part, const int* req_item_indptr, void* out,
@@ -686,7 +662,7 @@ static int launch_decode(const void* q, const void* kv_layer, const int* page_in
             launch_pdl(kern, dim3(num_ctas), dim3(DEC_WARPS * 32), SM, st,
                 (const bf16*)q, (const bf16*)kv_layer, page_indices, kv_page_indptr, item_req,
                 item_start, item_end, req_item_indptr, num_items_ptr, (bf16*)out, o_part, lse_part, hq,
-                hkv, page_size, scale_log2, window_left, sinks_log2, max_items, num_reqs, status_word(),
+                hkv, page_size, scale_log2, window_left, sinks_log2, max_items, num_reqs, pie_status_word_current(),
                 (const int*)nullptr, (const int*)nullptr, (const int*)nullptr, cap_log2);
         } else if (cascade) {
             auto kern = paged_decode_attn_kernel<D, G, true>;
@@ -694,7 +670,7 @@ static int launch_decode(const void* q, const void* kv_layer, const int* page_in
             launch_pdl(kern, dim3(num_ctas), dim3(DEC_WARPS * 32), SM, st,
                 (const bf16*)q, (const bf16*)kv_layer, page_indices, kv_page_indptr, item_req,
                 item_start, item_end, req_item_indptr, num_items_ptr, (bf16*)out, o_part, lse_part, hq,
-                hkv, page_size, scale_log2, window_left, sinks_log2, max_items, num_reqs, status_word(),
+                hkv, page_size, scale_log2, window_left, sinks_log2, max_items, num_reqs, pie_status_word_current(),
                 item_slot, item_tile, tile_members, 0.f);
         } else {
             auto kern = paged_decode_attn_kernel<D, G, false>;
@@ -702,7 +678,7 @@ static int launch_decode(const void* q, const void* kv_layer, const int* page_in
             launch_pdl(kern, dim3(num_ctas), dim3(DEC_WARPS * 32), SM, st,
                 (const bf16*)q, (const bf16*)kv_layer, page_indices, kv_page_indptr, item_req,
                 item_start, item_end, req_item_indptr, num_items_ptr, (bf16*)out, o_part, lse_part, hq,
-                hkv, page_size, scale_log2, window_left, sinks_log2, max_items, num_reqs, status_word(),
+                hkv, page_size, scale_log2, window_left, sinks_log2, max_items, num_reqs, pie_status_word_current(),
                 (const int*)nullptr, (const int*)nullptr, (const int*)nullptr, 0.f);
         }
     });

@@ -342,6 +342,32 @@ __global__ void brle_expand_ragged_kernel(const uint32_t* __restrict__ run_ends,
 
 using namespace pie;
 
+// Status word of the current device for kernels without a status argument (see
+// pie_set_status_word); null when the embedder registered none: a kernel then reports nothing.
+namespace {
+constexpr int kStatusDevices = 64;
+int* g_status_word[kStatusDevices] = {};
+int* status_word() {
+    int dev = -1;
+    if (cudaGetDevice(&dev) != cudaSuccess || dev < 0 || dev >= kStatusDevices) return nullptr;
+    return g_status_word[dev];
+}
+}  // namespace
+
+// Register a device int32 (on the current device) that kernels without a status argument set to a
+// PieKernelStatus code when they drop work; pass null to unregister.
+PIE_API int pie_set_status_word(int* word) {
+    int dev = -1;
+    cudaError_t e = cudaGetDevice(&dev);
+    if (e != cudaSuccess) return (int)e;
+    if (dev < 0 || dev >= kStatusDevices) return (int)cudaErrorInvalidValue;
+    g_status_word[dev] = word;
+    return 0;
+}
+
+// The status word registered for the current device (null if none): for kernels of other files.
+PIE_API int* pie_status_word_current() { return status_word(); }
+
 PIE_API int pie_embed_gather(const int* tokens, const void* table, void* out, int n_tokens,
                              int hidden, int vocab_start, int vocab_count, cudaStream_t st) {
     if (n_tokens <= 0) return 0;
