@@ -124,7 +124,8 @@ template <int MT>
 __global__ void __launch_bounds__(LT_THREADS, 1)
 latent_attn_tc_kernel(const __grid_constant__ CUtensorMap tma_q, const __grid_constant__ CUtensorMap tma_c, const LatentMmaArgs a,
                       int* status) {
-    constexpr uint32_t TMEM_COLS = MT <= 2 ? 128 : 256;        // two S^T, then MT x O^T, 32 columns each
+    constexpr uint32_t TMEM_COLS = 128;                        // two S^T, then MT x O^T, 32 columns each
+    static_assert(MT <= 2, "TMEM columns");
     extern __shared__ uint8_t lt_raw[];
     const uint32_t raw = smem_addr(lt_raw), base = (raw + 1023u) & ~1023u;
     uint8_t* base_ptr = lt_raw + (base - raw);
@@ -434,7 +435,7 @@ extern "C" int pie_make_tma_2d_bf16(CUtensorMap* map, const void* ptr, long rows
 int pie_latent_merge(const LatentMmaArgs& a, cudaStream_t st);
 
 PIE_API int pie_latent_attn_tc_supported(int row, int rank_pad, int page_size) {
-    return row > 0 && row % 16 == 0 && rank_pad % 16 == 0 && rank_pad <= row && rank_pad <= 384 && page_size >= 16 &&
+    return row > 0 && row % 16 == 0 && rank_pad % 16 == 0 && rank_pad <= row && rank_pad <= 256 && page_size >= 16 &&
            (page_size & (page_size - 1)) == 0 && lt_smem(row, rank_pad) <= 227 * 1024 ? 1 : 0;
 }
 
@@ -457,11 +458,7 @@ PIE_API int pie_latent_attn_tc(const LatentMmaArgs* args, int num_ctas, int* sta
         e = launch_pdl(latent_attn_tc_kernel<M_>, grid, dim3(LT_THREADS), (size_t)smem, st, tq, tc, a, status);                      \
         if (e != cudaSuccess) return (int)e;                                                                                         \
     }
-    switch (lt_mtiles(a.rank_pad)) {
-        case 1: GO(1) break;
-        case 2: GO(2) break;
-        default: GO(3) break;
-    }
+    if (lt_mtiles(a.rank_pad) == 1) GO(1) else GO(2)
 #undef GO
     return pie_latent_merge(a, st);
 }

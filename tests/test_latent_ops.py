@@ -198,6 +198,46 @@ def test_latent_attention_sees_its_window_and_no_more(path, kw):
 
 
 @gpu
+@pytest.mark.parametrize("dtype", [F32, BF16])
+@pytest.mark.parametrize("heads,rank", [(20, 48), (40, 256), (3, 320), (33, 130)])
+def test_decode_batch_cut_over_ctas_under_layers_of_unequal_windows(heads, rank, dtype):
+    """One plan for the widest layer, cut so that requests are split and CTAs have several items; a layer with a narrower
+    window sees nothing of some items. Padding requests at the end have no items."""
+    kvs, page = [1, 40, 300, 700, 129, 16, 17, 128], 16
+    plan_window, r = 600, len(kvs)
+    s0 = spec_of(heads=heads, kv_rank=rank, scale=0.3)
+    cs = [rnd(k, rank, seed=10 + i, dtype=dtype, std=0.5) for i, k in enumerate(kvs)]
+    krs = [rnd(k, s0.rot_dim, seed=30 + i, dtype=dtype) for i, k in enumerate(kvs)]
+    caches, ids, ptr_, base = [], [], [0], 0
+    for c, kr in zip(cs, krs):
+        cache, pid = paged(c, kr, s0, page, dtype, "cpu", seed=len(ids))
+        caches.append(cache[:-1])
+        ids += [x + base for x in pid]
+        base += len(cache) - 1
+        ptr_.append(len(ids))
+    cache = torch.cat(caches + [torch.zeros(1, page, s0.row)]).to("cuda", dtype)
+    q = torch.zeros(r + 2, heads, s0.row)
+    q[..., :rank] = rnd(r + 2, heads, rank, seed=1, dtype=dtype)
+    q[..., s0.rank_pad:s0.rank_pad + s0.rot_dim] = rnd(r + 2, heads, s0.rot_dim, seed=2, dtype=dtype)
+    t = lambda a: torch.from_numpy(np.ascontiguousarray(a, np.int32)).cuda()
+    for ctas in (1, 3, 11):
+        ir, st, en, ip, ci = ops.plan_even_items(np.array(kvs), ctas, 64, plan_window - 1, min_keys=32)
+        pad = lambda a: np.concatenate([a, [a[-1]] * 2])
+        plan = ops.DecodePlan(t(ids), t(pad(np.array(ptr_))), t(ir), t(st), t(en), t(pad(ip)), t([len(ir)]),
+                              torch.full((ops.decode_scratch_floats(64, heads, s0.row),), float("nan"), device="cuda"), 64, r + 2, ctas,
+                              page, plan_window - 1, kv_lens=t(kvs + [0, 0]), cta_items=t(ci))
+        rs = recurrent(list(range(r + 3)), list(range(r)) + [-1, -1], [0] * (r + 2), torch.zeros(1, r, 8, device="cuda"), "cuda")
+        slots = t([0] * r + [-1, -1])
+        for window in (600, 100, 7, 1):
+            s = spec_of(heads=heads, kv_rank=rank, scale=0.3, window=window)
+            got = lops.latent_attention(q.to("cuda", dtype), cache, plan, rs, slots, s, page, window - 1)
+            for i, k in enumerate(kvs):
+                ref = attention_oracle(q[i:i + 1, :, :rank], q[i:i + 1, :, s.rank_pad:s.rank_pad + s.rot_dim], cs[i], krs[i], s, k - 1)
+                close(got[i:i + 1, :, :rank], ref, dtype, f32=2e-4, bf16=2e-2)
+    ops.check_kernel_status()
+
+
+@gpu
 @pytest.mark.parametrize("dims", [(24, 12, 16), (96, 32, 128), (50, 14, 64), (16, 16, 8), (100, 20, 40)])
 def test_projected_prefill(dims):
     """Prefill on projected keys and values: unequal requests, cached pasts, windows that start inside a page."""
