@@ -30,6 +30,10 @@ KERNEL_LIB = OUT / "libpie_kernels.so"
 LATENT_SOURCES = ("attention_tc", "elementwise", "gemm2_tcgen05", "gemm_tcgen05", "latent",
                   "latent_attn", "latent_attn_tc", "sampling")
 
+# sources whose kernels sandwich-normed blocks with linear attention launch
+SANDWICH_SOURCES = ("attention_bias", "elementwise", "gdn", "gemm2_tcgen05", "gemm_tcgen05", "latent", "latent_attn", "linear_attn", "moe",
+                    "sampling")
+
 NVCC_FLAGS = [
     "-gencode", "arch=compute_100a,code=sm_100a", "-lineinfo", "-O3", "-std=c++17",
     "--expt-relaxed-constexpr", "-Xcompiler", "-fPIC", "-Xcompiler", "-fvisibility=hidden",
@@ -96,6 +100,8 @@ def kernels_for(cfg) -> Path:
         return KERNEL_LIB
     if cfg.latent is not None:
         return build_kernels(only=LATENT_SOURCES, target=OUT / "libpie_kernels_latent.so")
+    if cfg.blocks is not None:
+        return build_kernels(only=SANDWICH_SOURCES, target=OUT / "libpie_kernels_sandwich.so")
     return build_kernels()
 
 

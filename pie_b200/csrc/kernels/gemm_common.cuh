@@ -23,6 +23,7 @@ enum GemmEpilogue : int {
     EPI_SWIGLU_T = 8,
     EPI_XIELU_T = 9,
     EPI_STREAM_T = 10,
+    EPI_CLAMP_GLU = 11,  // as EPI_SWIGLU with g = min(gate, limit), u = clamp(up, +-limit): g * sigmoid(1.702 g) * (u + 1)
 };
 
 // Operands of the epilogues with a bias. xIELU(z) = a z^2 + z / 2 for z > 0, b (e^z - 1 - z) + z / 2 below, with
@@ -33,7 +34,18 @@ struct EpiArgs {
     const float* res32 = nullptr;  // [M, ld32]; may be out32 itself
     float* out32 = nullptr;
     int ld32 = 0;
+    float limit = 0.f;             // EPI_CLAMP_GLU
 };
+
+template <int EPI>
+__device__ __forceinline__ float glu_value(float g, float u, float limit) {
+    if (EPI == EPI_CLAMP_GLU) {
+        g = fminf(g, limit);
+        u = fminf(fmaxf(u, -limit), limit);
+        return g / (1.f + __expf(-1.702f * g)) * (u + 1.f);
+    }
+    return g / (1.f + __expf(-g)) * u;
+}
 
 struct XieluCoef {
     float a, b;
@@ -151,7 +163,7 @@ __device__ __forceinline__ int streamk_cta_of(long long unit, long long total, i
 template <int EPI>
 __device__ __forceinline__ void epilogue_store_chunk(const uint32_t (&v)[32], int row, int col0, int M, int N,
                                                      bf16* __restrict__ C, int ldc, const bf16* __restrict__ R,
-                                                     int ldr, const TpArgs& tp) {
+                                                     int ldr, const TpArgs& tp, float limit = 0.f) {
     if (row >= M || col0 >= N) return;
     if (EPI == EPI_RS) {
         const int owner = row / tp.rows_per_rank;
@@ -165,14 +177,14 @@ __device__ __forceinline__ void epilogue_store_chunk(const uint32_t (&v)[32], in
             for (int e = 0; e < 8; ++e) o[e] = __uint_as_float(v[8 * j + e]);
             *reinterpret_cast<bf16x8*>(dst + 8 * j) = pack8(o);
         }
-    } else if (EPI == EPI_SWIGLU) {
+    } else if (EPI == EPI_SWIGLU || EPI == EPI_CLAMP_GLU) {
         bf16* dst = C + (size_t)row * ldc + (col0 >> 1);
         float o[16];
 #pragma unroll
         for (int j = 0; j < 16; ++j) {
             const float g = __uint_as_float(v[2 * j]);
             const float u = __uint_as_float(v[2 * j + 1]);
-            o[j] = g / (1.f + __expf(-g)) * u;
+            o[j] = glu_value<EPI>(g, u, limit);
         }
 #pragma unroll
         for (int j = 0; j < 2; ++j)
@@ -213,15 +225,15 @@ __device__ __forceinline__ void epilogue_store_64(const uint32_t (&v0)[32], cons
                                                   const XieluCoef* act = nullptr) {
     const int lane = threadIdx.x & 31;
     auto slot = [&](int r, int c) { return reinterpret_cast<bf16x8*>(stage + r * 128 + ((c ^ (r & 7)) << 4)); };
-    if (EPI == EPI_SWIGLU) {
+    if (EPI == EPI_SWIGLU || EPI == EPI_CLAMP_GLU) {
         // 64 accumulator columns -> 32 outputs (64 B) per row
         float o[32];
 #pragma unroll
         for (int j = 0; j < 16; ++j) {
             const float g0 = __uint_as_float(v0[2 * j]), u0 = __uint_as_float(v0[2 * j + 1]);
             const float g1 = __uint_as_float(v1[2 * j]), u1 = __uint_as_float(v1[2 * j + 1]);
-            o[j] = g0 / (1.f + __expf(-g0)) * u0;
-            o[16 + j] = g1 / (1.f + __expf(-g1)) * u1;
+            o[j] = glu_value<EPI>(g0, u0, ex.limit);
+            o[16 + j] = glu_value<EPI>(g1, u1, ex.limit);
         }
 #pragma unroll
         for (int c = 0; c < 4; ++c) *slot(lane, c) = pack8(o + 8 * c);

@@ -726,12 +726,11 @@ PIE_API int pie_gemm_bf16_tp(const void* A, const void* W, void* C, int M, int N
 // 128-row tiles; W is [E, N, K] contiguous; tile_expert [max_mtiles] (device) gives each tile's
 // expert or -1. C [max_mtiles*128, N] (or N/2 with the SwiGLU epilogue). Graph-safe: the launch
 // shape depends only on max_mtiles.
-PIE_API int pie_grouped_gemm_bf16(const void* A, const void* W, void* C, const int* tile_expert, int max_mtiles,
-                                  int num_experts, int N, int K, int lda, int ldc, int epilogue, int* status,
-                                  int num_sms, cudaStream_t st) {
+static int grouped_gemm(const void* A, const void* W, void* C, const int* tile_expert, int max_mtiles, int num_experts, int N, int K,
+                        int lda, int ldc, int epilogue, int* status, int num_sms, cudaStream_t st, const EpiArgs& ex) {
     if (max_mtiles <= 0 || N <= 0 || num_experts <= 0) return 0;
     if (K <= 0 || K % 8 || N % 8 || ldc % 8) return (int)cudaErrorInvalidValue;
-    if (epilogue == EPI_SWIGLU && N % 32) return (int)cudaErrorInvalidValue;
+    if ((epilogue == EPI_SWIGLU || epilogue == EPI_CLAMP_GLU) && N % 32) return (int)cudaErrorInvalidValue;
     const int M = max_mtiles * GEMM_BM;
     const int bn = N >= 128 ? 128 : 64;
     CUtensorMap ta, tb;
@@ -748,14 +747,32 @@ PIE_API int pie_grouped_gemm_bf16(const void* A, const void* W, void* C, const i
                                              (int)GemmCfg<BN_>::SMEM_BYTES);                              \
         if (e != cudaSuccess) return (int)e;                                                              \
         e = launch_pdl(kern, dim3(grid), dim3(GEMM_THREADS), GemmCfg<BN_>::SMEM_BYTES, st, ta, tb, (bf16*)C, \
-                       (const bf16*)nullptr, M, N, K, ldc, 0, status, tp, sk, tile_expert, bn, EpiArgs());    \
+                       (const bf16*)nullptr, M, N, K, ldc, 0, status, tp, sk, tile_expert, bn, ex);    \
         return (int)(e != cudaSuccess ? e : cudaGetLastError());                                          \
     }
     if (epilogue == EPI_STORE) {
         if (bn == 128) GO(128, EPI_STORE) else GO(64, EPI_STORE)
     } else if (epilogue == EPI_SWIGLU) {
         if (bn == 128) GO(128, EPI_SWIGLU) else GO(64, EPI_SWIGLU)
+    } else if (epilogue == EPI_CLAMP_GLU) {
+        if (bn == 128) GO(128, EPI_CLAMP_GLU) else GO(64, EPI_CLAMP_GLU)
     }
 #undef GO
     return (int)cudaErrorInvalidValue;
+}
+
+PIE_API int pie_grouped_gemm_bf16(const void* A, const void* W, void* C, const int* tile_expert, int max_mtiles,
+                                  int num_experts, int N, int K, int lda, int ldc, int epilogue, int* status,
+                                  int num_sms, cudaStream_t st) {
+    if (epilogue != EPI_STORE && epilogue != EPI_SWIGLU) return (int)cudaErrorInvalidValue;
+    return grouped_gemm(A, W, C, tile_expert, max_mtiles, num_experts, N, K, lda, ldc, epilogue, status, num_sms, st, EpiArgs());
+}
+
+// The clamped GLU of experts without biases in the epilogue: C [max_mtiles*128, N/2], see EPI_CLAMP_GLU.
+PIE_API int pie_grouped_gemm_clamp_glu(const void* A, const void* W, void* C, const int* tile_expert, int max_mtiles,
+                                       int num_experts, int N, int K, int lda, int ldc, float limit, int* status,
+                                       int num_sms, cudaStream_t st) {
+    EpiArgs ex;
+    ex.limit = limit;
+    return grouped_gemm(A, W, C, tile_expert, max_mtiles, num_experts, N, K, lda, ldc, EPI_CLAMP_GLU, status, num_sms, st, ex);
 }

@@ -5,54 +5,20 @@
 // T is the activation type: bf16 when serving, float for the 32-bit path. The residual stream, norms, shift state,
 // angles, scores and softmax weights are 32-bit in both. Leading dimensions (ld*) are in elements; columns between a
 // row's width and its padded width are written as zeros, since the GEMMs read them.
-#include "common.cuh"
+#include "typed.cuh"
 
 namespace pie {
 
-template <typename T> __device__ __forceinline__ float to_f(T v);
-template <> __device__ __forceinline__ float to_f<float>(float v) { return v; }
-template <> __device__ __forceinline__ float to_f<bf16>(bf16 v) { return __bfloat162float(v); }
-template <typename T> __device__ __forceinline__ T from_f(float v);
-template <> __device__ __forceinline__ float from_f<float>(float v) { return v; }
-template <> __device__ __forceinline__ bf16 from_f<bf16>(float v) { return __float2bfloat16(v); }
-
-// VEC consecutive elements as floats (VEC 4: one 8- or 16-byte access)
-template <int VEC, typename T>
-__device__ __forceinline__ void load_vec(const T* p, float (&f)[VEC]) {
-    if constexpr (VEC == 1) {
-        f[0] = to_f(*p);
-    } else if constexpr (sizeof(T) == 4) {
-        const float4 v = *reinterpret_cast<const float4*>(p);
-        f[0] = v.x; f[1] = v.y; f[2] = v.z; f[3] = v.w;
-    } else {
-        const uint2 v = *reinterpret_cast<const uint2*>(p);
-        const float2 a = __bfloat1622float2(*reinterpret_cast<const bf162*>(&v.x));
-        const float2 b = __bfloat1622float2(*reinterpret_cast<const bf162*>(&v.y));
-        f[0] = a.x; f[1] = a.y; f[2] = b.x; f[3] = b.y;
-    }
-}
-template <int VEC, typename T>
-__device__ __forceinline__ void store_vec(T* p, const float (&f)[VEC]) {
-    if constexpr (VEC == 1) {
-        *p = from_f<T>(f[0]);
-    } else if constexpr (sizeof(T) == 4) {
-        *reinterpret_cast<float4*>(p) = make_float4(f[0], f[1], f[2], f[3]);
-    } else {
-        const bf162 a = __floats2bfloat162_rn(f[0], f[1]), b = __floats2bfloat162_rn(f[2], f[3]);
-        *reinterpret_cast<uint2*>(p) = make_uint2(*reinterpret_cast<const uint32_t*>(&a), *reinterpret_cast<const uint32_t*>(&b));
-    }
-}
-
 // ---------------------------------------------------------------- embedding
-// x[t, :] = table[tokens[t], :] in 32-bit (zeros for an id outside the table and in the padding columns).
+// x[t, :] = table[tokens[t], :] * scale in 32-bit (zeros for an id outside the table and in the padding columns).
 template <typename T>
 __global__ void stream_embed_kernel(const int* __restrict__ tokens, const T* __restrict__ table, float* __restrict__ x,
-                                    int width, int ldx, int vocab) {
+                                    int width, int ldx, int vocab, float scale) {
     const int t = blockIdx.x, id = tokens[t];
     const bool ok = id >= 0 && id < vocab;
     const T* src = table + (size_t)(ok ? id : 0) * width;
     float* dst = x + (size_t)t * ldx;
-    for (int i = threadIdx.x; i < ldx; i += blockDim.x) dst[i] = ok && i < width ? to_f(src[i]) : 0.f;
+    for (int i = threadIdx.x; i < ldx; i += blockDim.x) dst[i] = ok && i < width ? to_f(src[i]) * scale : 0.f;
 }
 
 // ------------------------------------------- stream norm (+ token shift)
@@ -79,7 +45,8 @@ struct StreamNormArgs {
 // token of a block it comes from the state (start of a portion) or is computed again from the stream. A single-token
 // portion updates its state in place (no other block reads it); a longer one leaves its last h in `stage`, because the
 // block with its first token may still be reading the state (shift_commit_kernel moves it).
-template <typename T, int MAXV, int VEC>
+// GT is the type of the gains (norm_w, y_norm).
+template <typename T, int MAXV, int VEC, typename GT = T>
 __global__ void __launch_bounds__(256) stream_norm_kernel(const StreamNormArgs a) {
     extern __shared__ float sq[];                 // one sum of squares per vector, then one factor per group
     __shared__ float red[32];
@@ -88,8 +55,8 @@ __global__ void __launch_bounds__(256) stream_norm_kernel(const StreamNormArgs a
     const int nvec = a.width / VEC, part = a.width / a.groups, part_vec = part / VEC;
     float* factor = sq + nvec;
     const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
-    const T* y_norm = static_cast<const T*>(a.y_norm);
-    const T* norm_w = static_cast<const T*>(a.norm_w);
+    const GT* y_norm = static_cast<const GT*>(a.y_norm);
+    const GT* norm_w = static_cast<const GT*>(a.norm_w);
     const T* shift = static_cast<const T*>(a.shift);
 
     auto load_stream = [&](int t, float (&v)[MAXV][VEC]) {
@@ -434,14 +401,16 @@ static int grid_for(long total) {
 
 using namespace pie;
 
-PIE_API int pie_stream_embed(const int* tokens, const void* table, float* x, int n, int width, int ldx, int vocab, int f32, cudaStream_t st) {
+PIE_API int pie_stream_embed(const int* tokens, const void* table, float* x, int n, int width, int ldx, int vocab, float scale, int f32,
+                             cudaStream_t st) {
     if (n <= 0) return 0;
-    if (f32) stream_embed_kernel<float><<<n, 256, 0, st>>>(tokens, (const float*)table, x, width, ldx, vocab);
-    else stream_embed_kernel<bf16><<<n, 256, 0, st>>>(tokens, (const bf16*)table, x, width, ldx, vocab);
+    if (f32) stream_embed_kernel<float><<<n, 256, 0, st>>>(tokens, (const float*)table, x, width, ldx, vocab, scale);
+    else stream_embed_kernel<bf16><<<n, 256, 0, st>>>(tokens, (const bf16*)table, x, width, ldx, vocab, scale);
     return (int)cudaGetLastError();
 }
 
-PIE_API int pie_stream_norm(const StreamNormArgs* args, int f32, int commit_requests, cudaStream_t st) {
+// gain_f32: norm_w and y_norm are 32-bit also where the activations are not
+PIE_API int pie_stream_norm(const StreamNormArgs* args, int f32, int gain_f32, int commit_requests, cudaStream_t st) {
     const StreamNormArgs& a = *args;
     if (a.n <= 0) return 0;
     if (a.groups <= 0 || a.width % a.groups || a.rows_per_block <= 0 || a.x_out == a.x || (a.y && !a.x_out) ||
@@ -453,16 +422,17 @@ PIE_API int pie_stream_norm(const StreamNormArgs* args, int f32, int commit_requ
     if (per > (vec ? 16 : 32)) return (int)cudaErrorInvalidValue;
     const dim3 grid((a.n + a.rows_per_block - 1) / a.rows_per_block);
     const size_t smem = ((vec ? a.width / 4 : a.width) + a.groups) * sizeof(float);
-#define GO(T_, M_, V_)                                                                       \
+#define GO(T_, M_, V_, G_)                                                                   \
     {                                                                                        \
-        cudaError_t e = launch_pdl(stream_norm_kernel<T_, M_, V_>, grid, dim3(256), smem, st, a); \
+        cudaError_t e = launch_pdl(stream_norm_kernel<T_, M_, V_, G_>, grid, dim3(256), smem, st, a); \
         if (e != cudaSuccess) return (int)e;                                                 \
     }
-#define GO_M(T_, V_)                                                                         \
-    if (per <= 1) GO(T_, 1, V_) else if (per <= 2) GO(T_, 2, V_) else if (per <= 4) GO(T_, 4, V_) \
-    else if (per <= 8) GO(T_, 8, V_) else if (per <= 16) GO(T_, 16, V_) else GO(T_, 32, 1)
-    if (f32) { if (vec) { GO_M(float, 4) } else { GO_M(float, 1) } }
-    else { if (vec) { GO_M(bf16, 4) } else { GO_M(bf16, 1) } }
+#define GO_M(T_, V_, G_)                                                                     \
+    if (per <= 1) GO(T_, 1, V_, G_) else if (per <= 2) GO(T_, 2, V_, G_) else if (per <= 4) GO(T_, 4, V_, G_) \
+    else if (per <= 8) GO(T_, 8, V_, G_) else if (per <= 16) GO(T_, 16, V_, G_) else GO(T_, 32, 1, G_)
+    if (f32) { if (vec) { GO_M(float, 4, float) } else { GO_M(float, 1, float) } }
+    else if (gain_f32) { if (vec) { GO_M(bf16, 4, float) } else { GO_M(bf16, 1, float) } }
+    else { if (vec) { GO_M(bf16, 4, bf16) } else { GO_M(bf16, 1, bf16) } }
 #undef GO_M
 #undef GO
     if (a.shift && commit_requests > 0)

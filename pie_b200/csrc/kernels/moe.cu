@@ -25,10 +25,13 @@ constexpr int MOE_TILE = 128;
 // One warp per token. logits [N, E] (bf16 or fp32), E <= 512.
 // ids receives the expert index relative to e_lo, or -1 for an expert outside [e_lo, e_lo+e_cnt)
 // (expert parallelism: those routes belong to another rank and take no slot here).
-template <typename T>
+// SCORED: experts are chosen by probability + `correction` and weighted by the probability alone (never renormalised); the
+// logits are `splits` fp32 arrays, split_stride apart, that add up to them.
+template <typename T, bool SCORED = false>
 __global__ void moe_route_kernel(const T* __restrict__ logits, int ld, int n, int E, int k, int renorm,
                                  int e_lo, int e_cnt, int* __restrict__ ids, float* __restrict__ w,
-                                 int* __restrict__ pos, int* __restrict__ counts) {
+                                 int* __restrict__ pos, int* __restrict__ counts, const float* __restrict__ correction = nullptr,
+                                 int splits = 1, long split_stride = 0) {
     const int warp = (blockIdx.x * blockDim.x + threadIdx.x) >> 5, lane = threadIdx.x & 31;
     if (warp >= n) return;
     const T* row = logits + (size_t)warp * ld;
@@ -38,21 +41,32 @@ __global__ void moe_route_kernel(const T* __restrict__ logits, int ld, int n, in
     for (int i = 0; i < MOE_MAX_E / 32; ++i) {
         const int e = i * 32 + lane;
         v[i] = e < E ? (float)row[e] : -INFINITY;
+        if (SCORED && e < E)
+            for (int j = 1; j < splits; ++j) v[i] += (float)row[j * split_stride + e];
         mx = fmaxf(mx, v[i]);
     }
     mx = warp_max(mx);
     float sum = 0.f;
 #pragma unroll
     for (int i = 0; i < MOE_MAX_E / 32; ++i) {
-        v[i] = (i * 32 + lane) < E ? __expf(v[i] - mx) : -1.f;   // -1 = excluded
+        v[i] = (i * 32 + lane) < E ? (SCORED ? expf(v[i] - mx) : __expf(v[i] - mx)) : -1.f;   // -1 = excluded
         if (v[i] > 0.f) sum += v[i];
     }
     sum = warp_sum(sum);
+    float prob[SCORED ? MOE_MAX_E / 32 : 1];
+    if (SCORED) {
+#pragma unroll
+        for (int i = 0; i < MOE_MAX_E / 32; ++i) {
+            const int e = i * 32 + lane;
+            prob[i] = v[i];
+            v[i] = e < E ? v[i] / sum + correction[e] : -INFINITY;
+        }
+    }
     float picked_sum = 0.f;
     float my_w = 0.f;
     int my_id = 0;
     for (int j = 0; j < k; ++j) {
-        float best = -2.f;
+        float best = SCORED ? -INFINITY : -2.f;
         int bi = 0x7fffffff;
 #pragma unroll
         for (int i = 0; i < MOE_MAX_E / 32; ++i) {
@@ -65,12 +79,20 @@ __global__ void moe_route_kernel(const T* __restrict__ logits, int ld, int n, in
             const int oi = __shfl_xor_sync(0xffffffffu, bi, o);
             if (ob > best || (ob == best && oi < bi)) { best = ob; bi = oi; }
         }
-        if ((bi & 31) == lane) v[bi >> 5] = -1.f;
+        if (SCORED) {
+            float p = 0.f;
+#pragma unroll
+            for (int i = 0; i < MOE_MAX_E / 32; ++i)
+                if (i * 32 + lane == bi) { p = prob[i]; v[i] = -INFINITY; }
+            best = __shfl_sync(0xffffffffu, p, bi & 31);
+        } else if ((bi & 31) == lane) {
+            v[bi >> 5] = -1.f;
+        }
         picked_sum += best;
         if (lane == j) { my_w = best; my_id = bi; }
     }
     if (lane < k) {
-        const float denom = renorm ? picked_sum : sum;
+        const float denom = renorm && !SCORED ? picked_sum : sum;
         const int local = my_id - e_lo;
         const bool mine = local >= 0 && local < e_cnt;
         ids[(size_t)warp * k + lane] = mine ? local : -1;
@@ -127,13 +149,14 @@ __global__ void moe_permute_kernel(const bf16* __restrict__ x, int ldx, const in
     for (int c = threadIdx.x; c < H / 8; c += blockDim.x) dst[c] = src[c];
 }
 
-// One block per token. RS: the (partial) row goes to the receive buffer of the rank that owns
+// One block per token. `self`: a route without a slot is an expert that returns its input, row t of `self`. RS: the (partial) row goes to the receive buffer of the rank that owns
 // token t (reduce-scatter by peer stores, same protocol as the GEMM's EPI_RS epilogue); the last
 // block to finish raises this rank's flag on every owner.
 template <bool RS>
 __global__ void moe_combine_kernel(const bf16* __restrict__ y, const int* __restrict__ slot_of,
                                    const float* __restrict__ w, const bf16* __restrict__ residual, int ldr, int H,
-                                   int k, bf16* __restrict__ out, int ldo, const __grid_constant__ TpArgs tp) {
+                                   int k, bf16* __restrict__ out, int ldo, const __grid_constant__ TpArgs tp,
+                                   const bf16* __restrict__ self = nullptr, int lds = 0) {
     const int t = blockIdx.x;
     bf16* dst_row;
     if (RS) {
@@ -150,10 +173,10 @@ __global__ void moe_combine_kernel(const bf16* __restrict__ y, const int* __rest
             for (int i = 0; i < 8; ++i) acc[i] = 0.f;
         for (int j = 0; j < k; ++j) {
             const int slot = slot_of[(size_t)t * k + j];
-            if (slot < 0) continue;
+            if (slot < 0 && !self) continue;
             const float wj = w[(size_t)t * k + j];
             float v[8];
-            unpack8(*reinterpret_cast<const bf16x8*>(y + (size_t)slot * H + c * 8), v);
+            unpack8(*reinterpret_cast<const bf16x8*>(slot < 0 ? self + (size_t)t * lds + c * 8 : y + (size_t)slot * H + c * 8), v);
 #pragma unroll
             for (int i = 0; i < 8; ++i) acc[i] += wj * v[i];
         }
@@ -183,6 +206,17 @@ PIE_API int pie_moe_route(const void* logits, int logits_fp32, int ld, int n, in
     return (int)cudaGetLastError();
 }
 
+// Routing by score + correction over E outputs of which the first e_cnt take slots (the others are identity experts).
+PIE_API int pie_moe_route_scored(const float* logits, int splits, long split_stride, int ld, int n, int E, int k, int e_cnt,
+                                 const float* correction, int* ids, float* w, int* pos, int* counts, cudaStream_t st) {
+    if (n <= 0) return 0;
+    if (E > MOE_MAX_E || k > 32 || k > E || k <= 0 || splits < 1 || !correction || e_cnt > E) return (int)cudaErrorInvalidValue;
+    const int threads = 128, blocks = (n * 32 + threads - 1) / threads;
+    moe_route_kernel<float, true><<<blocks, threads, 0, st>>>(logits, ld, n, E, k, 0, 0, e_cnt, ids, w, pos, counts, correction, splits,
+                                                              split_stride);
+    return (int)cudaGetLastError();
+}
+
 PIE_API int pie_moe_align(int* counts, int E, int max_mtiles, int* seg_start, int* tile_expert, int* counts_out,
                           cudaStream_t st) {
     if (E > MOE_MAX_E || E <= 0) return (int)cudaErrorInvalidValue;
@@ -204,6 +238,16 @@ PIE_API int pie_moe_combine(const void* y, const int* slot_of, const float* w, c
     if (H % 8 || ldo % 8 || (residual && ldr % 8)) return (int)cudaErrorInvalidValue;
     moe_combine_kernel<false><<<n, 128, 0, st>>>((const bf16*)y, slot_of, w, (const bf16*)residual, ldr, H, k,
                                                  (bf16*)out, ldo, TpArgs{});
+    return (int)cudaGetLastError();
+}
+
+// out[t] = sum over routes of w * y[slot], or of w * x[t] where the route has no slot.
+PIE_API int pie_moe_combine_identity(const void* y, const int* slot_of, const float* w, const void* x, int ldx, int n, int H, int k,
+                                     void* out, int ldo, cudaStream_t st) {
+    if (n <= 0) return 0;
+    if (H % 8 || ldo % 8 || ldx % 8 || !x) return (int)cudaErrorInvalidValue;
+    moe_combine_kernel<false><<<n, 128, 0, st>>>((const bf16*)y, slot_of, w, nullptr, 0, H, k, (bf16*)out, ldo, TpArgs{}, (const bf16*)x,
+                                                 ldx);
     return (int)cudaGetLastError();
 }
 

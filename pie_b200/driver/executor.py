@@ -149,15 +149,17 @@ class TorchDriver:
         self._bound = threading.local()
         self.adapters: dict = {}
         self._lora_bindings = None
-        # the kernels compute in bf16 with 32-bit accumulation; compute_dtype "float32" runs a latent-attention model in
+        # the kernels compute in bf16 with 32-bit accumulation; compute_dtype "float32" runs a model with a 32-bit stream in
         # true 32-bit throughout (weights, activations, cache), for verification
         self.dtype = torch_dtype(cfg.dtype) if not self.cuda else torch.bfloat16
         if compute_dtype != "auto":
-            if self.cuda and compute_dtype == "float32" and cfg.latent is None:
+            if self.cuda and compute_dtype == "float32" and not cfg.stream32:
                 raise NotImplementedError(f"32-bit kernels for model type {cfg.model_type}")
             self.dtype = torch_dtype(compute_dtype)
-        if cfg.latent is not None and kv_dtype == "fp8_e4m3":
-            raise NotImplementedError("fp8 pages for latent rows")
+        if cfg.stream32 and kv_dtype == "fp8_e4m3":
+            raise NotImplementedError(f"fp8 pages for model type {cfg.model_type}")
+        if cfg.blocks is not None and par is not None and par.tp_size > 1:
+            raise NotImplementedError("layers described one by one under tensor parallelism")
         self.par = par or ParallelContext()
         if self.cuda:
             torch.cuda.set_device(self.device)
@@ -171,7 +173,7 @@ class TorchDriver:
         self.memory_plan = None
         if num_pages <= 0:
             num_pages, max_requests, max_tokens = self._plan_memory(gpu_mem_utilization, memory_profile, max_requests,
-                                                                    max_tokens)
+                                                                    max_tokens, rs_slots)
             if self.par.tp_size > 1:
                 # page ids are global to the replica: every rank must hold the same number of pages
                 import torch.distributed as dist
@@ -181,7 +183,7 @@ class TorchDriver:
                     num_pages = int(t.item())
         self.kv = KVCache(len(cfg.latent_cache_layers) if cfg.latent is not None else cfg.num_hidden_layers, num_pages, hkv,
                           page_size, cfg.head_dim, self.dtype, self.device, swap_pages, kv_dtype=kv_dtype,
-                          latent=cfg.latent is not None)
+                          latent=cfg.latent is not None, layer_shapes=cfg.kv_layers if cfg.blocks is not None else None)
         self.model.kv_scale = self.kv.scale
         # Gated DeltaNet, Mamba-2 and token-shifted layers keep their state in slots of a recurrent-state cache, one per resident context
         self.rs = None
@@ -189,7 +191,7 @@ class TorchDriver:
             if self.par.tp_size > 1:
                 raise NotImplementedError("recurrent-state layers under tensor parallelism")
             from .recurrent import RecurrentStateCache
-            self.rs = RecurrentStateCache(cfg, rs_slots or max(2 * max_requests, 16), self.device)
+            self.rs = RecurrentStateCache(cfg, rs_slots or self._default_rs_slots(max_requests), self.device)
         # media: a vision encoder (models.vision.VisionEncoder) and the clips it has encoded, by the runtime's slot
         self.vision, self.audio = vision, audio
         self.media: Dict[int, torch.Tensor] = {}
@@ -217,7 +219,7 @@ class TorchDriver:
         self._prefix_cache: dict = {}
         self.cascade = (self.cuda and _os.environ.get("PIE_CASCADE", "1") != "0" and self.window_left < 0
                         and self.cfg.layer_types is None and self.kv.scale is None and not self.softcap
-                        and self.cfg.latent is None)
+                        and not self.cfg.stream32)
         rows = max(max_requests, 1024)
         self.max_rows = rows
         self.slab = _Slab({
@@ -254,7 +256,11 @@ class TorchDriver:
         self.stats = {"fires": 0, "graph_replays": 0, "eager": 0, "kernel_launches": 0}
 
     # ------------------------------------------------------------------ planning
-    def _plan_memory(self, util: float, profile: str, max_requests: int, max_tokens: int):
+    def _default_rs_slots(self, max_requests: int) -> int:
+        """One state slot per request of a full batch where a slot is large, else room for as many idle contexts again."""
+        return max(max_requests if self.cfg.blocks is not None else 2 * max_requests, 16)
+
+    def _plan_memory(self, util: float, profile: str, max_requests: int, max_tokens: int, rs_slots: int = 0):
         """KV pages (and, with a named profile, the forward limits) from what the device has left once
         the weights are resident: `driver.memory_planner` splits `util` of the device between the
         activation arena of the largest pass and the page pool. Without a profile the caller's limits
@@ -265,6 +271,9 @@ class TorchDriver:
         free, total = torch.cuda.mem_get_info(self.device)
         usable = int(total * util) - (total - free)          # what `util` of the device leaves beside the weights
         tp = self.par.tp_size
+        if self.cfg.blocks is not None:
+            # linear-attention states are large (a slot holds every layer's [heads, dim, vdim] in 32-bit)
+            usable -= 4 * sum(b.recurrent.state_elems for b in self.cfg.blocks) * (rs_slots or self._default_rs_slots(max_requests))
         if profile:
             plan = mp.plan(self.cfg, usable, 1.0, profile, self.page_size, tp)
             max_requests, max_tokens = plan.max_requests, plan.max_tokens
@@ -282,8 +291,8 @@ class TorchDriver:
     # ------------------------------------------------------------------ adapters
     def create_adapter(self, adapter_id: int, rank: int, alpha: float, seed: int = 0) -> None:
         from .lora import LoraAdapter
-        if self.cfg.latent is not None:
-            raise NotImplementedError("LoRA adapters on latent attention")
+        if self.cfg.stream32:
+            raise NotImplementedError(f"LoRA adapters on model type {self.cfg.model_type}")
         if self.par.tp_size > 1:
             raise NotImplementedError("LoRA adapters are served by single-GPU replicas")
         self.adapters[adapter_id] = LoraAdapter(self.cfg, rank, alpha, self.device, self.dtype, self.model.hq,
@@ -449,7 +458,7 @@ class TorchDriver:
                 torch.arange(rb + 1, dtype=torch.int32, device=dev), torch.arange(rb, dtype=torch.int32, device=dev),
                 s.d("rs_slots", rb), s.d("rs_reset", rb), list(range(rb + 1)), [-1] * rb, [0] * rb,
                 self.rs.conv_state, self.rs.rec_state, self.rs.layer_index, shift_state=self.rs.shift_state,
-                **self.rs.device_scratch(rb, rb))
+                linear_state=self.rs.linear_state, linear_at=self.rs.linear_at, **self.rs.device_scratch(rb, rb))
         return cache[rb]
 
     def _fill_rs_decode(self, req: ForwardRequest, r: int, rb: int) -> None:

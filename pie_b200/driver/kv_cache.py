@@ -17,9 +17,20 @@ from .. import ops
 from .schema import CopyDir, CopyRequest
 
 
+class LayerPages:
+    """Pages of layers with unequal shapes: one tensor [pages + 1, 2, kv heads, page, D] per layer that has a cache."""
+
+    def __init__(self, layers):
+        self.layers = layers
+
+    def __getitem__(self, i: int):
+        return self.layers[i]
+
+
 class KVCache:
     def __init__(self, layers: int, num_pages: int, kv_heads: int, page_size: int, head_dim: int,
-                 dtype, device, swap_pages: int = 0, kv_dtype: str = "auto", latent: bool = False):
+                 dtype, device, swap_pages: int = 0, kv_dtype: str = "auto", latent: bool = False,
+                 layer_shapes=None):
         """kv_dtype "auto": pages in the activation dtype. "fp8_e4m3": one byte per element plus one
         fp32 scale per (token, KV head) row in `scale` [layers, pages + 1, 2, kv_heads, page_size]
         (written by the RoPE + KV-write kernel, read by decode attention; prefill attention works on
@@ -27,7 +38,10 @@ class KVCache:
         (driver/cuda/src/kv_cache_format.hpp, kernels/kv_paged.cu:188-325).
 
         `latent`: pages of latent attention, one row of `head_dim` elements per token (latent, then the rotated key part
-        that all heads share) in ``[layers, pages + 1, page_size, row]``; `layers` counts the layers that write rows."""
+        that all heads share) in ``[layers, pages + 1, page_size, row]``; `layers` counts the layers that write rows.
+
+        `layer_shapes`: (kv heads, head_dim) of every layer that has a cache, where a model's layers differ (`data` is then a
+        `LayerPages`; it may be empty)."""
         if page_size % 16:
             raise ValueError("kv page size must be a multiple of 16")
         if kv_dtype not in ("auto", "bf16", "fp8_e4m3"):
@@ -42,20 +56,23 @@ class KVCache:
         self.layers, self.num_pages, self.kv_heads = layers, num_pages, kv_heads
         self.page_size, self.head_dim, self.dtype = page_size, head_dim, dtype
         self.device = torch.device(device)
-        self.page_shape = (page_size, head_dim) if latent else (2, kv_heads, page_size, head_dim)
+        if layer_shapes is not None:
+            shapes = [(1, (2, h, page_size, d)) for h, d in layer_shapes]
+        else:
+            shapes = [(layers, (page_size, head_dim) if latent else (2, kv_heads, page_size, head_dim))]
         # zero-filled: unwritten slots are multiplied by p == 0 in attention and must be finite
-        self.data = torch.zeros(layers, num_pages + 1, *self.page_shape, dtype=dtype, device=self.device)
+        self.parts = [torch.zeros(n, num_pages + 1, *shape, dtype=dtype, device=self.device) for n, shape in shapes]
+        self.data = self.parts[0] if layer_shapes is None else LayerPages([t[0] for t in self.parts])
         self.pad_page = num_pages
         self.swap_pages = swap_pages
         self.host = None
         if swap_pages > 0:
-            self.host = torch.zeros(layers, swap_pages, *self.page_shape, dtype=dtype,
-                                    pin_memory=self.device.type == "cuda")
+            self.host = [torch.zeros(n, swap_pages, *shape, dtype=dtype, pin_memory=self.device.type == "cuda") for n, shape in shapes]
         self._copy_stream = torch.cuda.Stream(self.device) if self.device.type == "cuda" else None
 
     @property
     def page_bytes_all_layers(self) -> int:
-        return self.data[:, 0].numel() * self.data.element_size()
+        return sum(t[:, 0].numel() * t.element_size() for t in self.parts)
 
     @staticmethod
     def bytes_per_page(layers, kv_heads, page_size, head_dim, elem_size=2) -> int:
@@ -71,7 +88,8 @@ class KVCache:
         if req.direction == CopyDir.D2D:
             s = torch.from_numpy(src).to(self.device)
             d = torch.from_numpy(dst).to(self.device)
-            ops.copy_pages(self.data, s, d)
+            for t in self.parts:
+                ops.copy_pages(t, s, d)
             if self.scale is not None:
                 ops.copy_pages(self.scale, s, d)
             return
@@ -80,23 +98,26 @@ class KVCache:
         if self.host is None:
             raise RuntimeError("no swap pool configured")
         if req.direction == CopyDir.H2H:
-            self.host[:, torch.from_numpy(dst).long()] = self.host[:, torch.from_numpy(src).long()]
+            for h in self.host:
+                h[:, torch.from_numpy(dst).long()] = h[:, torch.from_numpy(src).long()]
             return
         if self._copy_stream is None:
-            for s, d in zip(src.tolist(), dst.tolist()):
-                if req.direction == CopyDir.D2H:
-                    self.host[:, d] = self.data[:, s]
-                else:
-                    self.data[:, d] = self.host[:, s]
+            for t, h in zip(self.parts, self.host):
+                for s, d in zip(src.tolist(), dst.tolist()):
+                    if req.direction == CopyDir.D2H:
+                        h[:, d] = t[:, s]
+                    else:
+                        t[:, d] = h[:, s]
             return
         cur = torch.cuda.current_stream(self.device)
         self._copy_stream.wait_stream(cur)
         with torch.cuda.stream(self._copy_stream):
-            for s, d in zip(src.tolist(), dst.tolist()):
-                if req.direction == CopyDir.D2H:
-                    self.host[:, d].copy_(self.data[:, s], non_blocking=True)
-                else:
-                    self.data[:, d].copy_(self.host[:, s], non_blocking=True)
+            for t, h in zip(self.parts, self.host):
+                for s, d in zip(src.tolist(), dst.tolist()):
+                    if req.direction == CopyDir.D2H:
+                        h[:, d].copy_(t[:, s], non_blocking=True)
+                    else:
+                        t[:, d].copy_(h[:, s], non_blocking=True)
         if req.direction == CopyDir.H2D:
             cur.wait_stream(self._copy_stream)
         else:

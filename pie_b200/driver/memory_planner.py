@@ -44,7 +44,7 @@ class MemoryPlan:
 
 
 def kv_bytes_per_page(cfg: ModelConfig, page_size: int, tp: int = 1, kv_dtype_bytes: int = 2) -> int:
-    if cfg.latent is not None:
+    if cfg.stream32:
         return cfg.kv_elems_per_token * page_size * kv_dtype_bytes
     hkv = max(1, cfg.num_key_value_heads // tp)
     return cfg.num_hidden_layers * 2 * hkv * page_size * cfg.head_dim * kv_dtype_bytes
@@ -61,8 +61,22 @@ def arena_bytes(cfg: ModelConfig, max_tokens: int, max_requests: int, tp: int = 
         # also the keys and values of every head
         heads = max(s.heads * (s.qk_dim + s.vdim + 2 * s.row) for s in cfg.latent)
         per_token = 2 * (8 * h + heads + 3 * inter) + 2 * max(s.heads for s in cfg.latent) * 3 * 128
+    if cfg.blocks is not None:
+        per_token = 2 * 8 * h + max(_block_bytes(b) for b in cfg.blocks)
     logits = max_requests * cfg.vocab_size * (2 + 4)       # bf16 logits + fp32 rows for probes
     return max_tokens * per_token + logits
+
+
+def _block_bytes(b) -> int:
+    """Activation bytes per token of one sandwich-normed block: projections, 32-bit mixer outputs, the states between the
+    64-token pieces of a prompt, feed-forward (an expert's segment may be padded by 128 rows: the experts' weights dwarf it)."""
+    r, a, f = b.recurrent, b.attention, b.ff
+    bytes_ = 2 * (2 * r.qk + 2 * r.values) + 4 * (r.qk + 2 * r.values) + 4 * r.state_elems // 64
+    if a is not None:
+        bytes_ += 2 * (a.heads * (a.dim + 2 * a.vdim) + a.kv_heads * (a.dim + a.vdim) + 2 * a.kv_heads * a.group_pad * a.head_dim)
+    if f is not None:
+        bytes_ += 2 * 3 * f.ff * getattr(f, "top", 1)
+    return bytes_
 
 
 def plan(cfg: ModelConfig, free_bytes: int, gpu_mem_utilization: float = 0.9, profile: str = "auto",

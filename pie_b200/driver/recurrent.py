@@ -1,6 +1,7 @@
 """Recurrent-state cache of the Gated DeltaNet and Mamba-2 layers and of token-shifted blocks: per (recurrent layer,
 slot) the tail of the short convolution's inputs and the fp32 state (delta-rule state [heads, dk, dv], or state-space
-state [heads, head_dim, state]), or the previous token's normalised input (token shift, [width] fp32).
+state [heads, head_dim, state]), or the previous token's normalised input (token shift, [width] fp32). Linear-attention
+mixers of layers described one by one (any head sizes) keep [heads, dim, vdim] fp32 each, all layers of a slot in one row.
 A slot belongs to one resident context; the runtime's
 slot pool (`runtime/rs_cache.py`) hands slots out, tells the driver when a slot must start from zero
 (`rs_reset`) and asks for a slot copy when a context forks.
@@ -34,6 +35,9 @@ class RecurrentInputs:
     scratch: Optional[torch.Tensor] = None   # [N, C] fp32 convolution output (device path)
     shift_state: Optional[torch.Tensor] = None   # [L, S, W] fp32 previous token's input (token shift)
     shift_stage: Optional[torch.Tensor] = None   # [R, W] fp32: a portion's last input until its readers are done
+    linear_state: Optional[torch.Tensor] = None  # [S, elements] fp32: the states of all linear-attention layers of a slot
+    linear_at: Optional[Dict[int, int]] = None   # model layer -> its first element in a row of `linear_state`
+    pieces: Optional[tuple] = None # the portions cut for the chunked form (`ops.linear.chunk_pieces`)
     staged: Optional[int] = None   # requests the stage is committed for (0: none of this fire's portions uses it)
 
 
@@ -44,8 +48,16 @@ class RecurrentStateCache:
         if cfg.linear_layers and cfg.mamba_layers:
             raise NotImplementedError("Gated DeltaNet and Mamba-2 layers in one model")
         self.layer_index = {li: i for i, li in enumerate(lin)}
-        self.conv_state = self.rec_state = self.shift_state = None
+        self.conv_state = self.rec_state = self.shift_state = self.linear_state = None
+        self.linear_at: Optional[Dict[int, int]] = None
         self.conv_channels = 0
+        if cfg.blocks is not None:
+            self.linear_at, at = {}, 0
+            for li, b in enumerate(cfg.blocks):
+                self.linear_at[li] = at
+                at += -(-b.recurrent.state_elems // 4) * 4
+            self.linear_state = torch.zeros(num_slots, at, dtype=torch.float32, device=self.device)
+            return
         if cfg.token_shift:
             if cfg.mamba_layers or cfg.linear_layers:
                 raise NotImplementedError("token shift beside Gated DeltaNet or Mamba-2 layers")
@@ -63,7 +75,8 @@ class RecurrentStateCache:
 
     @property
     def buffers(self) -> List[torch.Tensor]:
-        return [b for b in (self.conv_state, self.rec_state, self.shift_state) if b is not None]
+        linear = self.linear_state[None] if self.linear_state is not None else None
+        return [b for b in (self.conv_state, self.rec_state, self.shift_state, linear) if b is not None]
 
     @property
     def bytes_per_slot(self) -> int:
@@ -71,7 +84,7 @@ class RecurrentStateCache:
 
     def device_scratch(self, n: int, r: int) -> dict:
         """Device scratch of a fire of n tokens in r requests."""
-        if self.device.type != "cuda":
+        if self.device.type != "cuda" or self.linear_state is not None:
             return {}
         if self.shift_state is not None:
             return {"shift_stage": torch.empty(max(r, 1), self.cfg.hidden_size, dtype=torch.float32, device=self.device)}
@@ -93,7 +106,7 @@ class RecurrentStateCache:
         t = lambda a: torch.from_numpy(a).to(dev)
         return RecurrentInputs(t(qo), t(tok_req), t(slots), t(reset), qo.tolist(), slots.tolist(), reset.tolist(),
                                self.conv_state, self.rec_state, self.layer_index, shift_state=self.shift_state,
-                               **self.device_scratch(int(qo[-1]), r))
+                               linear_state=self.linear_state, linear_at=self.linear_at, **self.device_scratch(int(qo[-1]), r))
 
     def copy_slot(self, src: int, dst: int) -> None:
         """dst <- src in every layer (a forked context continues from its parent's state)."""

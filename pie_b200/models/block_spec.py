@@ -1,0 +1,222 @@
+"""Descriptions of layers that a configuration lists one by one (sandwich-normed blocks over a 32-bit residual stream):
+each block names its mixer and its feed-forward, with sizes and constants of its own. The Retodra reader and writer of
+`config.json` are at the end.
+"""
+from __future__ import annotations
+
+import math
+from dataclasses import dataclass
+from typing import List, Optional, Union
+
+
+@dataclass
+class GatedLinearSpec:
+    """Gated linear attention: a state [dim, vdim] per head whose rows decay by sigmoid(z)^(1 / tau), z a projection of
+    rank `rank` (None: the checkpoint tells)."""
+    heads: int
+    dim: int
+    vdim: int
+    tau: float
+    rank: Optional[int] = None
+
+    @property
+    def qk(self) -> int:
+        return self.heads * self.dim
+
+    @property
+    def values(self) -> int:
+        return self.heads * self.vdim
+
+    @property
+    def state_elems(self) -> int:
+        return self.heads * self.dim * self.vdim
+
+
+@dataclass
+class LightningSpec:
+    """Linear attention with one constant decay per head."""
+    heads: int
+    dim: int
+    vdim: int
+    decay: List[float]
+
+    qk = GatedLinearSpec.qk
+    values = GatedLinearSpec.values
+    state_elems = GatedLinearSpec.state_elems
+
+
+@dataclass
+class BiasedAttentionSpec:
+    """Grouped-query attention without rotation: soft-capped scores plus a learned bias per distance bucket (`buckets`
+    rows, None: the checkpoint tells; logarithmic up to `bias_max`), over the query itself and the `window` - 1 tokens
+    before it."""
+    heads: int
+    kv_heads: int
+    dim: int
+    vdim: int
+    window: int
+    scale: float
+    softcap: float
+    bias_max: int
+    buckets: Optional[int] = None
+
+    @property
+    def group(self) -> int:
+        return self.heads // self.kv_heads
+
+    @property
+    def group_pad(self) -> int:
+        """Query heads per key / value head the kernels compute: the next power of two (the added ones are zeros)."""
+        return 1 << (self.group - 1).bit_length()
+
+    @property
+    def head_dim(self) -> int:
+        """Columns of a cached key or value and of a query row, zeros past dim / vdim."""
+        need = max(self.dim, self.vdim)
+        return 64 if need <= 64 else 128 if need <= 128 else -(-need // 128) * 128
+
+    def bucket(self, n: int) -> int:
+        """Bias row of the distance n: a row each for the first half, then logarithmic."""
+        half = self.buckets // 2
+        if n < half:
+            return n
+        far = math.log(n / half) / math.log(self.bias_max / half) * (self.buckets - half)
+        return min(self.buckets - 1, half + math.floor(far + 1e-9))     # a distance on a bucket's edge stays on it
+
+
+@dataclass
+class ParallelSpec:
+    """Windowed attention and lightning attention side by side on the same input."""
+    left: BiasedAttentionSpec
+    right: LightningSpec
+    left_scale: float
+    right_scale: float
+
+
+@dataclass
+class DenseSpec:
+    ff: int
+
+
+@dataclass
+class ExpertsSpec:
+    """`experts` clamped-GLU experts of width `ff` and `identity` more router outputs whose expert returns its input."""
+    experts: int
+    identity: int
+    top: int
+    ff: int
+    limit: float
+
+    @property
+    def outputs(self) -> int:
+        return self.experts + self.identity
+
+
+@dataclass
+class BlockSpec:
+    mixer: Union[GatedLinearSpec, ParallelSpec]
+    ff: Union[DenseSpec, ExpertsSpec, None]
+
+    @property
+    def attention(self) -> Optional[BiasedAttentionSpec]:
+        return self.mixer.left if isinstance(self.mixer, ParallelSpec) else None
+
+    @property
+    def recurrent(self) -> Union[GatedLinearSpec, LightningSpec]:
+        """The part of the mixer whose state is carried from token to token."""
+        return self.mixer.right if isinstance(self.mixer, ParallelSpec) else self.mixer
+
+
+# ------------------------------------------------------------------ Retodra
+def _retodra_mixer(i: int, kind: str, m: dict):
+    if kind == "gla":
+        return GatedLinearSpec(m["heads"], m["dim"], m["vdim"], float(m["tau"]), m.get("rank"))
+    if kind != "parallel":
+        raise ValueError(f"layer {i}: unknown mixer {kind!r}")
+    a, b = m["left"], m["right"]
+    left = BiasedAttentionSpec(a["heads"], a["kv_heads"], a["dim"], a["vdim"], a["mask"]["size"], float(a["scale"]),
+                               float(a["softcap"]), a["bias_max"], a.get("buckets"))
+    right = LightningSpec(b["heads"], b["dim"], b["vdim"], [float(x) for x in b["decay"]])
+    if left.heads % left.kv_heads or left.window < 1 or left.softcap <= 0:
+        raise ValueError(f"layer {i}: {left.heads} query heads on {left.kv_heads}, window {left.window}, soft cap {left.softcap}")
+    if len(right.decay) != right.heads or not all(0 < x <= 1 for x in right.decay):
+        raise ValueError(f"layer {i}: decays {right.decay} for {right.heads} heads")
+    return ParallelSpec(left, right, float(m["left_scale"]), float(m["right_scale"]))
+
+
+def _retodra_ff(i: int, mlp: Optional[dict]):
+    if mlp is None:
+        return None
+    if mlp["kind"] == "dense":
+        return DenseSpec(mlp["ff"])
+    if mlp["kind"] != "moe":
+        raise ValueError(f"layer {i}: unknown feed-forward {mlp['kind']!r}")
+    r, e = mlp["router"], mlp["expert"]
+    s = ExpertsSpec(r["experts"], r.get("identity", 0), r["top"], e["ff"], float(e["limit"]))
+    if not 1 <= s.top <= s.outputs:
+        raise ValueError(f"layer {i}: {s.top} of {s.outputs} router outputs")
+    return s
+
+
+def retodra_config(cfg: dict, name: str):
+    from .config import ModelConfig
+    blocks = [BlockSpec(_retodra_mixer(i, x["type"], x["mixer"]), _retodra_ff(i, x.get("mlp"))) for i, x in enumerate(cfg["layers"])]
+    att = [b.attention for b in blocks if b.attention is not None]
+    ffs = [b.ff.ff for b in blocks if b.ff is not None]
+    return ModelConfig(
+        model_type="retodra", hidden_size=cfg["width"], intermediate_size=max(ffs, default=0), num_hidden_layers=len(blocks),
+        num_attention_heads=max((a.kv_heads * a.group_pad for a in att), default=1),
+        num_key_value_heads=max((a.kv_heads for a in att), default=1), head_dim=max((a.head_dim for a in att), default=64),
+        vocab_size=cfg["vocab"], max_position_embeddings=cfg.get("max_position_embeddings", 131072),
+        rms_norm_eps=cfg["norm"]["eps"], tie_word_embeddings=False, embed_scale=float(cfg["embedding"]["scale"]),
+        norm_plus_one=True, sandwich_norm=True, blocks=blocks, dtype="bfloat16", name=name)
+
+
+def retodra_dict(cfg) -> dict:
+    """The `config.json` dictionary `retodra_config` reads `cfg` from."""
+    layers = []
+    for b in cfg.blocks:
+        m = b.mixer
+        if isinstance(m, GatedLinearSpec):
+            d = {"type": "gla", "mixer": {"heads": m.heads, "dim": m.dim, "vdim": m.vdim, "tau": m.tau}}
+        else:
+            a, r = m.left, m.right
+            d = {"type": "parallel", "mixer": {
+                "left": {"heads": a.heads, "kv_heads": a.kv_heads, "dim": a.dim, "vdim": a.vdim, "mask": {"size": a.window},
+                         "scale": a.scale, "softcap": a.softcap, "bias_max": a.bias_max},
+                "right": {"heads": r.heads, "dim": r.dim, "vdim": r.vdim, "decay": list(r.decay)},
+                "left_scale": m.left_scale, "right_scale": m.right_scale}}
+        f = b.ff
+        if f is None:
+            d["mlp"] = None
+        elif isinstance(f, DenseSpec):
+            d["mlp"] = {"kind": "dense", "ff": f.ff}
+        else:
+            d["mlp"] = {"kind": "moe", "expert": {"ff": f.ff, "limit": f.limit},
+                        "router": {"experts": f.experts, "identity": f.identity, "top": f.top}}
+        layers.append(d)
+    return {"architecture": "Retodra", "width": cfg.hidden_size, "vocab": cfg.vocab_size, "layers": layers,
+            "norm": {"eps": cfg.rms_norm_eps}, "embedding": {"scale": cfg.embed_scale}}
+
+
+def retodra_shape(layers: int = 32, width: int = 4096, gla_heads: int = 8, gla_dim: int = 256, gla_vdim: int = 512, rank: int = 16,
+                  tau: float = 16.0, heads: int = 32, kv_heads: int = 8, dim: int = 128, window: int = 1024, buckets: int = 32,
+                  right_heads: int = 16, right_dim: int = 128, right_vdim: int = 128, ff: int = 11008, experts: int = 32,
+                  identity: int = 4, top: int = 4, expert_ff: int = 2048, vocab: int = 128256) -> dict:
+    """config.json dictionary of a model that alternates gated linear attention with a dense feed-forward and parallel
+    mixers with experts."""
+    spec = []
+    decay = [math.exp(-2.0 ** (-8.0 * (h + 1) / right_heads)) for h in range(right_heads)]
+    for i in range(layers):
+        if i % 2 == 0:
+            spec.append({"type": "gla", "mixer": {"heads": gla_heads, "dim": gla_dim, "vdim": gla_vdim, "tau": tau, "rank": rank},
+                         "mlp": {"kind": "dense", "ff": ff}})
+        else:
+            left = {"heads": heads, "kv_heads": kv_heads, "dim": dim, "vdim": dim, "mask": {"size": window}, "scale": dim ** -0.5,
+                    "softcap": 30.0, "bias_max": 2 * window, "buckets": buckets}
+            right = {"heads": right_heads, "dim": right_dim, "vdim": right_vdim, "decay": decay}
+            spec.append({"type": "parallel", "mixer": {"left": left, "right": right, "left_scale": 0.75, "right_scale": 0.6},
+                         "mlp": {"kind": "moe", "expert": {"ff": expert_ff, "limit": 7.0},
+                                 "router": {"experts": experts, "identity": identity, "top": top}}})
+    return {"architecture": "Retodra", "width": width, "vocab": vocab, "layers": spec, "norm": {"eps": 1e-5},
+            "embedding": {"scale": float(width) ** 0.5}}

@@ -10,11 +10,13 @@ from dataclasses import dataclass, field, asdict
 from pathlib import Path
 from typing import Optional
 
+from .block_spec import BlockSpec, retodra_config, retodra_shape
+
 LLAMA_LIKE = {"llama", "qwen2", "qwen3", "mistral", "phi3"}   # pre-norm decoder blocks with SwiGLU and rotate-half RoPE
 # `model_type` strings of checkpoints this build loads (the architecture registry of the loader)
 SUPPORTED_MODEL_TYPES = ("llama", "mistral", "qwen2", "qwen3", "phi3", "qwen3_moe", "mixtral", "olmo2", "olmo3", "gpt_oss",
                          "qwen3_5", "qwen3_next", "mamba2_hybrid", "gemma2", "gemma3_text", "gemma3", "qwen2_moe", "qwen2_vl",
-                         "qwen2_audio", "puzutar")
+                         "qwen2_audio", "puzutar", "retodra")
 MAMBA_TYPES = {"mamba2_hybrid"}         # Mamba-2 (state-space) mixers in llama-like blocks, between full-attention layers
 GDN_TYPES = {"qwen3_5", "qwen3_next"}   # hybrids: Gated DeltaNet (linear attention) layers between full-attention layers
 POST_NORM = {"olmo2", "olmo3"}       # same block with the norms after attention / MLP and q, k norms over all heads
@@ -23,7 +25,7 @@ MOE_TYPES = {"qwen3_moe", "mixtral", "gpt_oss", "qwen2_moe"}
 # alternating local / global layers (Gemma-3: a RoPE base of their own for the local ones; Gemma-2: soft-capped logits)
 GEMMA_TYPES = {"gemma2", "gemma3_text", "gemma3"}
 # configs that name the design under "architecture" instead of "model_type"
-ARCHITECTURES = {"Puzutar": "puzutar"}
+ARCHITECTURES = {"Puzutar": "puzutar", "Retodra": "retodra"}
 
 
 def config_model_type(cfg: dict) -> str:
@@ -133,6 +135,8 @@ class ModelConfig:
     norm_groups: int = 1               # RMSNorm over this many equal parts of the width, each with its own mean square
     token_shift: bool = False          # the mixer reads h + (previous token's h - h) * shift: state of a sequence
     token_side_dim: int = 0            # width of the per-layer token input (0: none)
+    # layers described one by one: sandwich-normed blocks over a 32-bit residual stream
+    blocks: Optional[list] = None      # BlockSpec per layer
     # quantisation of the linear weights: None | "fp8_block" (128x128 weight scales)
     quantization: Optional[str] = None
     dtype: str = "bfloat16"
@@ -161,7 +165,7 @@ class ModelConfig:
     def recurrent_layers(self) -> list:
         """Layers whose state lives in the recurrent-state cache (Gated DeltaNet or Mamba-2)."""
         return [li for li in range(self.num_hidden_layers)
-                if self.token_shift or self.is_linear_layer(li) or self.is_mamba_layer(li)]
+                if self.token_shift or self.blocks is not None or self.is_linear_layer(li) or self.is_mamba_layer(li)]
 
     @property
     def latent_cache_layers(self) -> list:
@@ -175,10 +179,24 @@ class ModelConfig:
         return {li: own[li if s.kv_from is None else s.kv_from] for li, s in enumerate(self.latent)}
 
     @property
+    def stream32(self) -> bool:
+        """The residual stream is 32-bit, and the whole model also runs in true 32-bit on the device."""
+        return self.latent is not None or self.blocks is not None
+
+    @property
+    def kv_layers(self) -> list:
+        """(kv heads, head dim) of every layer that writes keys and values, in order."""
+        if self.blocks is not None:
+            return [(b.attention.kv_heads, b.attention.head_dim) for b in self.blocks if b.attention is not None]
+        return [(self.num_key_value_heads, self.head_dim)] * self.num_hidden_layers
+
+    @property
     def kv_elems_per_token(self) -> int:
         """Cache elements one token takes over all layers (unsharded)."""
         if self.latent is not None:
             return len(self.latent_cache_layers) * self.latent_row
+        if self.blocks is not None:
+            return sum(2 * h * d for h, d in self.kv_layers)
         return self.num_hidden_layers * 2 * self.num_key_value_heads * self.head_dim
 
     @property
@@ -213,6 +231,9 @@ class ModelConfig:
         """Keys left of the query that layer `li` sees (-1: all). HF `sliding_window` counts the query itself."""
         if self.latent is not None:
             return self.latent[li].window - 1
+        if self.blocks is not None:
+            a = self.blocks[li].attention
+            return a.window - 1 if a is not None else 0
         if not self.sliding_window or self.sliding_window <= 0:
             return -1
         if self.layer_types is not None and self.layer_types[li] != "sliding_attention":
@@ -241,6 +262,8 @@ class ModelConfig:
         mt = config_model_type(cfg) or "llama"
         if mt == "puzutar":
             return _puzutar_config(cfg, name)
+        if mt == "retodra":
+            return retodra_config(cfg, name)
         if mt == "gemma3" and "text_config" in cfg:       # multimodal wrapper: the language model's own section
             cfg = dict(cfg["text_config"], model_type="gemma3_text")
             mt = "gemma3_text"
@@ -511,20 +534,24 @@ PRESETS = {
                            dtype="float32"),
 }
 
-# presets of designs whose layers are described one by one: the arguments of `puzutar_shape`
+# presets of designs whose layers are described one by one: reader, shape and the shape's arguments
 LAYERED_PRESETS = {
-    "puzutar-8b": dict(),
-    "tiny-puzutar": dict(layers=3, width=256, heads=2, dim=48, rot_dim=16, vdim=40, kv_rank=64, window=40, ff=384, vocab=32000,
-                         groups=2, side=16),
+    "puzutar-8b": (_puzutar_config, puzutar_shape, dict()),
+    "retodra-8b": (retodra_config, retodra_shape, dict()),
+    "tiny-puzutar": (_puzutar_config, puzutar_shape, dict(layers=3, width=256, heads=2, dim=48, rot_dim=16, vdim=40, kv_rank=64, window=40, ff=384, vocab=32000,
+                         groups=2, side=16)),
+    "tiny-retodra": (retodra_config, retodra_shape, dict(
+        layers=4, width=256, gla_heads=2, gla_dim=48, gla_vdim=64, rank=8, heads=6, kv_heads=2, dim=40, window=50, buckets=12,
+        right_heads=3, right_dim=32, right_vdim=40, ff=384, experts=6, identity=2, top=3, expert_ff=96, vocab=32000)),
 }
 
 
 def preset(name: str, **overrides) -> ModelConfig:
     if name in LAYERED_PRESETS:
-        shape = dict(LAYERED_PRESETS[name])
+        read, build, args = LAYERED_PRESETS[name]
         if "num_hidden_layers" in overrides:
-            shape["layers"] = overrides.pop("num_hidden_layers")
-        cfg = _puzutar_config(puzutar_shape(**shape), name)
+            args = dict(args, layers=overrides.pop("num_hidden_layers"))
+        cfg = read(build(**args), name)
         for k, v in overrides.items():
             setattr(cfg, k, v)
         return cfg

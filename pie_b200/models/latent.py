@@ -2,7 +2,7 @@
 
 One layer: h = grouped RMSNorm(x), hs = h shifted towards the previous token's h; x += mixer(hs) + ff(h); then the
 per-layer token input, x += RMSNorm(W_proj (gelu(W_gate x) * e)). The norm of a layer also finishes the token input of
-the layer before (`LatentStream` carries what is pending), and the products that end both sublayers run as one GEMM over
+the layer before (`ResidualStream` carries what is pending), and the products that end both sublayers run as one GEMM over
 their inputs side by side.
 
 Latent attention decodes in its absorbed form: with W_uk folded into the query and W_uv applied to the result, keys and
@@ -14,21 +14,8 @@ from __future__ import annotations
 import torch
 
 from ..ops import latent as lops
-from .config import ModelConfig, _pad
-
-
-class LatentStream:
-    """The residual stream between layers: x [N, padded width] fp32, and a token input not yet added to it."""
-
-    def __init__(self, x):
-        self.x, self.y, self.y_norm = x, None, None
-
-    def finish(self, cfg: ModelConfig):
-        """The stream with everything pending added."""
-        if self.y is not None:
-            self.x, _, _ = lops.stream_norm(self.x, cfg.hidden_size, cfg.rms_norm_eps, self.y, self.y_norm)
-            self.y = self.y_norm = None
-        return self.x
+from .config import _pad
+from .stream import ResidualStream
 
 
 def rope_table(base: float, dims: int, device) -> torch.Tensor:
@@ -83,7 +70,7 @@ def latent_mixer(m, hs, lw: dict, li: int, fi, cache, out) -> None:
     lops.per_head(o, lw["w_uv_p"], out.as_strided((n, s.heads, s.vdim), (out.stride(0), s.vdim, 1)))
 
 
-def parallel_latent_block(m, st: LatentStream, lw: dict, li: int, fi, cache) -> None:
+def parallel_latent_block(m, st: ResidualStream, lw: dict, li: int, fi, cache) -> None:
     cfg = m.cfg
     s, ff, W, eps = cfg.latent[li], cfg.ff_sizes[li], cfg.hidden_size, cfg.rms_norm_eps
     x, h, hs = lops.stream_norm(st.x, W, eps, st.y, st.y_norm, lw["ln1"], cfg.norm_groups, lw.get("shift"), fi.rs, li)

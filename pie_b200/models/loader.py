@@ -13,7 +13,9 @@ against a safetensors reader, producing this rank's weight dict. Ops:
   Cast(dtype) / DequantFp8Block() dtype change / 128x128 block-scaled fp8 -> bf16
   Transpose(a, b)                 swap two dimensions (GPT-OSS stores experts as [E, in, out])
   Mxfp4(blocks, scales)           e2m1 nibbles with one e8m0 scale per 32 -> values [.., rows, cols]
-  Pad(multiple)                   zeros appended until every dimension is a multiple (tile and TMA alignment)
+  Pad(multiple)                   zeros appended until every dimension is a multiple (tile and TMA alignment); a list gives
+                                  one multiple per dimension
+  Keep32(x)                       the value stays 32-bit whatever the runtime type
   Attach(path)                    store under a runtime name
 
 The program is serialisable (`program_to_json`), so a per-rank plan can be compiled once and
@@ -31,6 +33,7 @@ from typing import Callable, Dict, List, Optional, Sequence, Tuple
 
 import torch
 
+from .block_spec import DenseSpec, ExpertsSpec, GatedLinearSpec, retodra_dict
 from .config import ModelConfig, _pad, _puzutar_dict
 from .weights import kv_head_range, torch_dtype
 
@@ -60,6 +63,7 @@ def Transpose(x, a, b): return Op("transpose", {"a": a, "b": b}, [x])
 def AddScalar(x, value): return Op("add_scalar", {"value": value}, [x])
 def RowScales(scale, like): return Op("row_scales", {"like": like}, [scale])
 def Pad(x, multiple=8): return Op("pad", {"multiple": multiple}, [x])
+def Keep32(x): return Op("keep32", {}, [x])
 def Mxfp4(blocks, scales): return Op("mxfp4", {}, [blocks, scales])
 
 _E2M1 = (0.0, 0.5, 1.0, 1.5, 2.0, 3.0, 4.0, 6.0, -0.0, -0.5, -1.0, -1.5, -2.0, -3.0, -4.0, -6.0)
@@ -140,6 +144,8 @@ def compile_program(cfg: ModelConfig, names: Sequence[str], tp_size: int = 1, tp
     names = set(names)
     if cfg.latent is not None:
         return _compile_latent(cfg, names, tp_size, dtype)
+    if cfg.blocks is not None:
+        return _compile_blocks(cfg, names, tp_size, dtype)
     T, r, d = tp_size, tp_rank, cfg.head_dim
     kv0, kvn = kv_head_range(cfg, r, T)
     # the language model's tensors may sit under a prefix ("model.", or a multimodal wrapper's "model.language_model.")
@@ -347,6 +353,78 @@ def _compile_latent(cfg: ModelConfig, names: set, tp_size: int, dtype: str) -> P
     return Program(att, dtype, {"tp_size": 1, "tp_rank": 0, "ep": False, "layers": cfg.num_hidden_layers, "vocab_start": 0})
 
 
+def complete_blocks(cfg: ModelConfig, reader) -> None:
+    """Sizes that only the checkpoint's tensors give: the rank of a decay projection, the rows of a bias table."""
+    have = set(reader.names())
+    for i, b in enumerate(cfg.blocks):
+        name = f"l{i}.mix.a1" if isinstance(b.mixer, GatedLinearSpec) else f"l{i}.mix.left.rel"
+        if name not in have:
+            raise KeyError(f"checkpoint has no tensor {name}")
+        rows = int(reader.get_slice(name).get_shape()[0])
+        if isinstance(b.mixer, GatedLinearSpec):
+            b.mixer.rank = rows
+        else:
+            b.attention.buckets = rows
+            if rows < 2 or b.attention.bias_max <= rows // 2:
+                raise LoaderTypeError(f"{name}: {rows} rows for distances up to {b.attention.bias_max}")
+
+
+def _compile_blocks(cfg: ModelConfig, names: set, tp_size: int, dtype: str) -> Program:
+    """Layout plan of sandwich-normed blocks (Retodra names). Fused per layer: every projection that reads the mixer's input
+    (`w_in`, each part on a multiple of 8 rows: `sandwich.projection_columns`), the output projections of two mixers side
+    by side along K (`w_out`), gate and up interleaved. Dimensions a GEMM sees are padded with zeros, those of a gated
+    feed-forward to 16."""
+    if tp_size > 1:
+        raise NotImplementedError("layers described one by one under tensor parallelism")
+    W = cfg.hidden_size
+    att: Dict[str, Op] = {}
+
+    def r(n, *shape):
+        if n not in names:
+            raise KeyError(f"checkpoint has no tensor {n}")
+        return Op("read", {"name": n, "shape": list(shape)})
+
+    def gate_up(n, ff):
+        return Interleave(Pad(r(n + "gate", ff, W), [16, 8]), Pad(r(n + "up", ff, W), [16, 8]))
+
+    att["embed"], att["lm_head"] = r("embed", cfg.vocab_size, W), Pad(r("head", cfg.vocab_size, W))
+    att["final_norm"] = r("final.norm", W)
+    for li, b in enumerate(cfg.blocks):
+        L, P, X = f"l{li}.", f"layers.{li}.", f"l{li}.mix."
+        halves = ("1", "2") if b.ff is not None else ("1",)
+        for h in halves:
+            att[P + "ln" + h], att[P + f"ln{h}b"], att[P + "ls" + h] = r(L + "norm" + h, W), r(L + f"norm{h}b", W), r(L + "ls" + h, W)
+        m = b.mixer
+        if isinstance(m, GatedLinearSpec):
+            if m.rank is None:
+                raise ValueError(f"layer {li}: the rank of the decay projection is not known (complete_blocks)")
+            rows = [("q", m.qk), ("k", m.qk), ("v", m.values), ("g", m.values), ("a1", m.rank)]
+            att[P + "a2"], att[P + "a2_b"], att[P + "o_norm"] = r(X + "a2", m.qk, m.rank), r(X + "a2.b", m.qk), r(X + "norm", m.vdim)
+            att[P + "w_out"] = Pad(r(X + "o", W, m.values))
+        else:
+            a, s = m.left, m.right
+            if a.buckets is None:
+                raise ValueError(f"layer {li}: the rows of the bias table are not known (complete_blocks)")
+            nq, nk = a.heads * a.dim, a.kv_heads * a.dim
+            rows = [("left.q", nq), ("left.k", nk), ("left.v", a.kv_heads * a.vdim), ("left.g", a.heads * a.vdim),
+                    ("right.q", s.qk), ("right.k", s.qk), ("right.v", s.values), ("right.g", s.values)]
+            att[P + "q_norm"], att[P + "k_norm"] = r(X + "left.q.norm", nq), r(X + "left.k.norm", nk)
+            att[P + "rel"] = Keep32(r(X + "left.rel", a.buckets, a.heads))
+            att[P + "o_norm"] = r(X + "right.norm", s.values)
+            att[P + "w_out"] = Concat([Pad(r(X + "left.o", W, a.heads * a.vdim)), Pad(r(X + "right.o", W, s.values))], 1)
+        att[P + "w_in"] = Concat([Pad(r(X + n, k, W)) for n, k in rows], 0)
+        F = L + "mlp."
+        if isinstance(b.ff, DenseSpec):
+            att[P + "w_gate_up"], att[P + "w_down"] = gate_up(F, b.ff.ff), Pad(r(F + "down", W, b.ff.ff), [8, 16])
+        elif isinstance(b.ff, ExpertsSpec):
+            each = [f"{F}e{e}." for e in range(b.ff.experts)]
+            att[P + "experts_gate_up"] = Stack([gate_up(e, b.ff.ff) for e in each])
+            att[P + "experts_down"] = Stack([Pad(r(e + "down", W, b.ff.ff), [8, 16]) for e in each])
+            att[P + "router"] = Pad(r(F + "router", b.ff.outputs, W), [1, 8])
+            att[P + "correction"] = Keep32(r(F + "correction", b.ff.outputs))
+    return Program(att, dtype, {"tp_size": 1, "tp_rank": 0, "ep": False, "layers": cfg.num_hidden_layers, "vocab_start": 0})
+
+
 class TensorDictReader:
     """The reader interface over a dictionary of checkpoint tensors (random initialisation, tests)."""
 
@@ -426,7 +504,7 @@ def _eval(op: Op, reader, dtype) -> torch.Tensor:
         return y.view(torch.float8_e4m3fn) if f8 else y
     if k == "pad":
         m, x = op.args["multiple"], xs[0]
-        extra = [(-n) % m for n in x.shape]
+        extra = [(-n) % k for n, k in zip(x.shape, m if isinstance(m, list) else [m] * x.dim())]
         return torch.nn.functional.pad(x, [v for e in reversed(extra) for v in (0, e)]) if any(extra) else x
     if k == "stack":
         return torch.stack(xs, dim=0)
@@ -434,7 +512,7 @@ def _eval(op: Op, reader, dtype) -> torch.Tensor:
         return torch.zeros_like(xs[0])
     if k == "squeeze":
         return xs[0].squeeze(op.args["dim"])
-    if k == "float":
+    if k in ("float", "keep32"):
         return xs[0].float()
     if k == "add_scalar":
         return xs[0] + op.args["value"]
@@ -493,10 +571,11 @@ def infer_shape(op: Op, reader) -> Tuple[int, ...]:
         if any(y != x for y in xs):
             raise LoaderTypeError(f"stack of unequal shapes {sorted(set(xs))}")
         return (len(xs),) + x
-    if k in ("zeros_like", "float", "add_scalar"):
+    if k in ("zeros_like", "float", "keep32", "add_scalar"):
         return x
     if k == "pad":
-        return tuple(_pad(n, op.args["multiple"]) for n in x)
+        m = op.args["multiple"]
+        return tuple(_pad(n, k2) for n, k2 in zip(x, m if isinstance(m, list) else [m] * len(x)))
     if k == "squeeze":
         d = op.args["dim"]
         if x[d] != 1:
@@ -556,7 +635,7 @@ def typecheck_program(prog: Program, cfg: ModelConfig, reader) -> Dict[str, Tupl
     architecture needs on this rank; all mismatches are reported together, before any tensor is read.
     Returns the inferred shapes. Counterpart of the weight loader's type checker in the reference
     (driver/weight_loader/src/typecheck.rs)."""
-    want = {} if cfg.latent is not None else expected_shapes(cfg, prog.meta.get("tp_size", 1), prog.meta.get("ep", False))
+    want = {} if cfg.stream32 else expected_shapes(cfg, prog.meta.get("tp_size", 1), prog.meta.get("ep", False))
     shapes, errors = {}, []
     for path, op in prog.attach.items():
         try:
@@ -588,7 +667,7 @@ def execute_program(prog: Program, reader, device="cpu") -> dict:
         if path.endswith("@scale"):
             scales[path[:-len("@scale")]] = t.float().contiguous().to(device)
             continue
-        if t.dtype != torch.float8_e4m3fn:
+        if t.dtype != torch.float8_e4m3fn and op.kind != "keep32":
             t = t.to(dtype)
         t = t.contiguous().to(device)
         if path.startswith("layers."):
@@ -724,6 +803,8 @@ def load_checkpoint(path, device="cpu", tp_size: int = 1, tp_rank: int = 0, ep: 
         return cfg, _cached_load(ggufs[0], prog, reader, device)
     cfg = ModelConfig.from_path(path)
     reader = SafetensorsReader(path)
+    if cfg.blocks is not None:
+        complete_blocks(cfg, reader)
     prog = compile_program(cfg, reader.names(), tp_size, tp_rank, ep, dtype or cfg.dtype)
     typecheck_program(prog, cfg, reader)
     return cfg, _cached_load(p, prog, reader, device)
@@ -752,6 +833,36 @@ def _latent_tensors(cfg: ModelConfig, weights: dict) -> Dict[str, torch.Tensor]:
     return t
 
 
+def _block_tensors(cfg: ModelConfig, weights: dict) -> Dict[str, torch.Tensor]:
+    """Checkpoint tensors of sandwich-normed blocks from their runtime layout (the inverse of `_compile_blocks`)."""
+    from .sandwich import projection_columns
+    W = cfg.hidden_size
+    t = {"embed": weights["embed"], "head": weights["lm_head"][:cfg.vocab_size, :W], "final.norm": weights["final_norm"]}
+    for li, (lw, b) in enumerate(zip(weights["layers"], cfg.blocks)):
+        L, X, F, m, f = f"l{li}.", f"l{li}.mix.", f"l{li}.mlp.", b.mixer, b.ff
+        for h in ("1", "2") if f is not None else ("1",):
+            t[L + "norm" + h], t[L + f"norm{h}b"], t[L + "ls" + h] = lw["ln" + h], lw[f"ln{h}b"], lw["ls" + h]
+        for n, (at, k) in projection_columns(m).items():
+            t[X + n] = lw["w_in"][at:at + k, :W]
+        if isinstance(m, GatedLinearSpec):
+            t[X + "a2"], t[X + "a2.b"], t[X + "norm"], t[X + "o"] = lw["a2"], lw["a2_b"], lw["o_norm"], lw["w_out"][:W, :m.values]
+        else:
+            hv = m.left.heads * m.left.vdim
+            t[X + "left.q.norm"], t[X + "left.k.norm"], t[X + "left.rel"] = lw["q_norm"], lw["k_norm"], lw["rel"].to(lw["w_in"].dtype)
+            t[X + "left.o"], t[X + "right.o"] = lw["w_out"][:W, :hv], lw["w_out"][:W, _pad(hv):_pad(hv) + m.right.values]
+            t[X + "right.norm"] = lw["o_norm"]
+        split = lambda gu: (gu[0::2][:f.ff, :W], gu[1::2][:f.ff, :W])
+        if isinstance(f, DenseSpec):
+            t[F + "gate"], t[F + "up"] = split(lw["w_gate_up"])
+            t[F + "down"] = lw["w_down"][:W, :f.ff]
+        elif isinstance(f, ExpertsSpec):
+            for e in range(f.experts):
+                t[F + f"e{e}.gate"], t[F + f"e{e}.up"] = split(lw["experts_gate_up"][e])
+                t[F + f"e{e}.down"] = lw["experts_down"][e][:W, :f.ff]
+            t[F + "router"], t[F + "correction"] = lw["router"][:, :W], lw["correction"].to(lw["router"].dtype)
+    return t
+
+
 def export_hf_checkpoint(cfg: ModelConfig, weights: dict, path) -> None:
     """Write unsharded runtime weights back out under Hugging Face names (tests, tooling)."""
     from safetensors.torch import save_file
@@ -760,6 +871,10 @@ def export_hf_checkpoint(cfg: ModelConfig, weights: dict, path) -> None:
     if cfg.latent is not None:
         save_file({k: v.contiguous().cpu() for k, v in _latent_tensors(cfg, weights).items()}, str(p / "model.safetensors"))
         (p / "config.json").write_text(json.dumps(_puzutar_dict(cfg)))
+        return
+    if cfg.blocks is not None:
+        save_file({k: v.contiguous().cpu() for k, v in _block_tensors(cfg, weights).items()}, str(p / "model.safetensors"))
+        (p / "config.json").write_text(json.dumps(retodra_dict(cfg)))
         return
     d, hq, hkv = cfg.head_dim, cfg.num_attention_heads, cfg.num_key_value_heads
     ungain = (lambda g: g.float() - 1.0) if cfg.norm_plus_one else (lambda g: g)      # Gemma stores (gain - 1)

@@ -64,15 +64,16 @@ def moe_reference(cfg: ModelConfig, x: torch.Tensor, lw: dict) -> torch.Tensor:
 
 
 def _buffers(model, n: int, lw: dict, device) -> "ops.MoeBuffers":
-    """Scratch for up to n tokens, grown in powers of two and kept on the model (fixed addresses
-    let the block be captured in CUDA graphs)."""
+    """Scratch for up to n tokens, in powers of two. Every size stays with the model at its address, so that CUDA graphs
+    captured on one go on working when a larger batch has come by."""
     cap = 1 << max(0, (max(n, 1) - 1).bit_length())
-    buf = getattr(model, "_moe_buf", None)
     e, n2, hdim = lw["experts_gate_up"].shape
-    if buf is None or buf.n < cap or buf.I != n2 // 2 or buf.E != e:
-        buf = ops.MoeBuffers(cap, hdim, n2 // 2, e, model.cfg.num_experts_per_tok, device)
-        model._moe_buf = buf
-    return buf
+    k = lw["top"] if "top" in lw else model.cfg.num_experts_per_tok
+    bufs = model.__dict__.setdefault("_moe_bufs", {})
+    key = (cap, e, n2, hdim, k)
+    if key not in bufs:
+        bufs[key] = ops.MoeBuffers(cap, hdim, n2 // 2, e, k, device)
+    return bufs[key]
 
 
 def moe_block(model, x: torch.Tensor, lw: dict, h: torch.Tensor) -> torch.Tensor:
@@ -145,10 +146,9 @@ def _moe_block_biased(model, x: torch.Tensor, lw: dict, h: torch.Tensor) -> torc
     ops.moe_align(buf, mt)
     ops.moe_permute(x, buf)
     rows = mt * 128
-    gu = getattr(model, "_moe_gu", None)
-    if gu is None or gu.shape[0] < rows or gu.shape[1] != 2 * buf.I:
-        gu = torch.empty(max(rows, buf.xs.shape[0]), 2 * buf.I, dtype=x.dtype, device=x.device)
-        model._moe_gu = gu
+    if getattr(buf, "gate_up", None) is None:
+        buf.gate_up = torch.empty(buf.xs.shape[0], 2 * buf.I, dtype=x.dtype, device=x.device)
+    gu = buf.gate_up
     ops.grouped_gemm(buf.xs, lw["experts_gate_up"], buf.tile_expert, gu, mt, ops.EPI_STORE)
     if x.dtype == torch.bfloat16 and gu.is_contiguous() and buf.act.is_contiguous():
         ops.moe_bias_glu(gu, lw["experts_gate_up_bias"], buf.tile_expert, buf.act, mt, cfg.swiglu_limit)

@@ -23,7 +23,8 @@ from .. import ops
 from ..ops import latent as lops, reference
 from ..driver.lora import apply_lora
 from .config import ModelConfig, _pad
-from .latent import LatentStream, final_rows, parallel_latent_block, prepare_latent
+from . import latent, sandwich
+from .stream import ResidualStream
 
 
 @dataclass
@@ -67,16 +68,19 @@ class Transformer:
         # fp8 KV pages: per-(token, head) scales [layers, pages, 2, hkv, page] set by the driver, else None
         self.kv_scale = None
         if cfg.latent is not None:
-            prepare_latent(self)
+            latent.prepare_latent(self)
+        elif cfg.blocks is not None:
+            sandwich.prepare_blocks(self)
 
     @property
     def prefill_group(self) -> int:
         """Query heads per key / value head of the prefill kernels' tiles."""
-        return 1 if self.cfg.latent is not None else self.hq // self.hkv
+        return 1 if self.cfg.stream32 else self.hq // self.hkv
 
     def prefill_tile_rows(self, page_size: int) -> int:
-        """Rows of a prefill tile (`ops.prefill_tile_rows`); latent attention runs prefill on expanded heads."""
-        if self.cfg.latent is not None:
+        """Rows of a prefill tile (`ops.prefill_tile_rows`); latent attention runs prefill on expanded heads, layers described
+        one by one plan tiles of their own."""
+        if self.cfg.stream32:
             return 256
         return ops.prefill_tile_rows(self.hq, self.hkv, self.cfg.head_dim, page_size, softcap=bool(self.cfg.attn_softcap))
 
@@ -197,28 +201,32 @@ class Transformer:
         if self._fused_tp():
             return self._forward_hidden_tp(fi, kv_cache)
         cfg, w = self.cfg, self.w
-        page_size = kv_cache.shape[-2]
-        if cfg.latent is not None:
-            h = lops.stream_embed(fi.tokens, w["embed"], _pad(cfg.hidden_size))
+        if cfg.stream32:
+            h = lops.stream_embed(fi.tokens, w["embed"], _pad(cfg.hidden_size), cfg.embed_scale)
         elif self.par.tp_size > 1 and w.get("embed_sharded", False):
             h = ops.embed(fi.tokens, w["embed"], vocab_start=w["embed_vocab_start"])
             h = self.par.comm.all_reduce(h)
         else:
             h = ops.embed(fi.tokens, w["embed"])
-        if cfg.embed_scale != 1.0:
+        if cfg.embed_scale != 1.0 and not cfg.stream32:
             # the factor is rounded to the activation dtype first, as the checkpoints' own code does
             h = h * torch.tensor(cfg.embed_scale, dtype=h.dtype).item()
         for feats, src, dst, cnt in fi.media or ():
             # rows of an encoded image / video take the place of their placeholder tokens' embeddings
             h[dst:dst + cnt, :cfg.hidden_size] = feats[src:src + cnt].to(h.dtype)
         n = h.shape[0]
-        stream = LatentStream(h) if cfg.latent is not None else None
+        stream = ResidualStream(h) if cfg.stream32 else None
+        page_size = kv_cache.shape[-2] if stream is None else None
         for li in range(cfg.num_hidden_layers):
             lw = w["layers"][li]
             post = cfg.post_norm
-            if stream is not None:
+            if cfg.latent is not None:
                 # parallel block: latent attention and feed-forward of one norm, added to the 32-bit stream together
-                parallel_latent_block(self, stream, lw, li, fi, kv_cache)
+                latent.parallel_latent_block(self, stream, lw, li, fi, kv_cache)
+                continue
+            if cfg.blocks is not None:
+                # sandwich-normed block with a mixer and a feed-forward of its own
+                sandwich.sandwich_block(self, stream, lw, li, fi, kv_cache)
                 continue
             if "w_mamba_in" in lw:
                 # Mamba-2 layer: state-space mixer, state in the recurrent-state cache
@@ -299,14 +307,14 @@ class Transformer:
 
     def logits(self, h: torch.Tensor, fi: ForwardInputs) -> torch.Tensor:
         """lm_head on the requested rows only ('compact logit rows')."""
-        rows = h if fi.logit_rows is None else ops.gather_rows(h, fi.logit_rows) if self.cfg.latent is None or not h.is_cuda else \
+        rows = h if fi.logit_rows is None else ops.gather_rows(h, fi.logit_rows) if not self.cfg.stream32 or not h.is_cuda else \
             ops.gather_rows(h.view(torch.bfloat16), fi.logit_rows).view(torch.float32)      # a 32-bit row moves as 16-bit halves
         if self._fused_tp():
             # h is already final-normalised and gathered; every rank computes its vocabulary slice and
             # keeps it: token samplers run sharded (TPComm.sample_sharded), only probes gather
             return self.par.comm.gemm_gated(self.w["lm_head"], rows.shape[0], x=rows)
-        if self.cfg.latent is not None:
-            x = final_rows(self, rows)
+        if self.cfg.stream32:
+            x = (latent if self.cfg.latent is not None else sandwich).final_rows(self, rows)
             return self._gemm(x, self.w["lm_head"])[:, :self.cfg.vocab_size]
         x = ops.rmsnorm(rows, self.w["final_norm"], self.cfg.rms_norm_eps)
         y = self._gemm(x, self.w["lm_head"])

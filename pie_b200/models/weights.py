@@ -12,6 +12,7 @@ Runtime layout per layer (this rank's shard under tensor parallelism):
   Gemma-2/3 (sandwich norms): ln1 / ln2 before attention / MLP, ln_pa / ln_pf on their outputs before the
   residual add; gains hold the full multiplier (the loader adds the checkpoint's implicit 1)
   Puzutar (latent attention in parallel blocks): see `loader._compile_latent`
+  Retodra (linear attention in sandwich-normed blocks): see `loader._compile_blocks`
 MoE layers replace w_gate_up / w_down by router [E, H], experts_gate_up [E_local, 2*Im, H]
 (interleaved) and experts_down [E_local, H, Im].
 
@@ -92,6 +93,8 @@ def random_weights(cfg: ModelConfig, device="cpu", dtype=None, seed: int = 0, tp
     gen = _Gen(seed, device, dtype, std)
     if cfg.latent is not None:
         return _random_latent(cfg, gen, tp_size)
+    if cfg.blocks is not None:
+        return _random_blocks(cfg, gen, tp_size)
     H, d = cfg.hidden_size, cfg.head_dim
     hq, hkv = cfg.num_attention_heads, cfg.num_key_value_heads
     T, r = tp_size, tp_rank
@@ -237,6 +240,42 @@ def _random_latent(cfg: ModelConfig, gen: _Gen, tp_size: int) -> dict:
         if S:
             t[L + "side.gate"], t[L + "side.proj"] = gen.normal(S, W, std=W ** -0.5), gen.normal(W, S)
             t[L + "side.norm"] = gen.normal(W, std=0.1)
+    prog = compile_program(cfg, list(t), tp_size, 0, False, str(gen.dtype).replace("torch.", ""))
+    return execute_program(prog, TensorDictReader(t), gen.device)
+
+
+def _random_blocks(cfg: ModelConfig, gen: _Gen, tp_size: int) -> dict:
+    """Random checkpoint tensors of sandwich-normed blocks, brought into the runtime layout by the loader."""
+    from .block_spec import DenseSpec, GatedLinearSpec
+    from .loader import TensorDictReader, compile_program, execute_program
+    W = cfg.hidden_size
+    near = lambda n: gen.normal(n, std=0.1)
+    t = {"embed": gen.normal(cfg.vocab_size, W), "head": gen.normal(cfg.vocab_size, W), "final.norm": near(W)}
+    for li, b in enumerate(cfg.blocks):
+        L, X, F, m, f = f"l{li}.", f"l{li}.mix.", f"l{li}.mlp.", b.mixer, b.ff
+        for h in ("1", "2") if f is not None else ("1",):
+            t[L + "norm" + h], t[L + f"norm{h}b"], t[L + "ls" + h] = near(W), near(W), 0.3 + near(W)
+        if isinstance(m, GatedLinearSpec):
+            m.rank = m.rank or 16
+            for n, k in (("q", m.qk), ("k", m.qk), ("v", m.values), ("g", m.values), ("a1", m.rank)):
+                t[X + n] = gen.normal(k, W)
+            t[X + "a2"], t[X + "a2.b"] = gen.normal(m.qk, m.rank, std=m.rank ** -0.5), gen.normal(m.qk, std=1.0)
+            t[X + "norm"], t[X + "o"] = 1 + near(m.vdim), gen.normal(W, m.values)
+        else:
+            a, s = m.left, m.right
+            a.buckets = a.buckets or 32
+            for n, k in (("left.q", a.heads * a.dim), ("left.k", a.kv_heads * a.dim), ("left.v", a.kv_heads * a.vdim),
+                         ("left.g", a.heads * a.vdim), ("right.q", s.qk), ("right.k", s.qk), ("right.v", s.values), ("right.g", s.values)):
+                t[X + n] = gen.normal(k, W)
+            t[X + "left.q.norm"], t[X + "left.k.norm"] = 1 + near(a.heads * a.dim), 1 + near(a.kv_heads * a.dim)
+            t[X + "left.rel"], t[X + "left.o"] = gen.normal(a.buckets, a.heads, std=0.5), gen.normal(W, a.heads * a.vdim)
+            t[X + "right.norm"], t[X + "right.o"] = 1 + near(s.values), gen.normal(W, s.values)
+        if isinstance(f, DenseSpec):
+            t[F + "gate"], t[F + "up"], t[F + "down"] = gen.normal(f.ff, W), gen.normal(f.ff, W), gen.normal(W, f.ff)
+        elif f is not None:
+            for e in range(f.experts):
+                t[F + f"e{e}.gate"], t[F + f"e{e}.up"], t[F + f"e{e}.down"] = gen.normal(f.ff, W), gen.normal(f.ff, W), gen.normal(W, f.ff)
+            t[F + "router"], t[F + "correction"] = gen.normal(f.outputs, W, std=W ** -0.5), gen.normal(f.outputs, std=0.02)
     prog = compile_program(cfg, list(t), tp_size, 0, False, str(gen.dtype).replace("torch.", ""))
     return execute_program(prog, TensorDictReader(t), gen.device)
 

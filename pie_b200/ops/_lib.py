@@ -61,8 +61,8 @@ _SIGNATURES = {
     "pie_gdn_mixer": [p, i32, p, p, p, p, p, p, p, p, p, p, p, p, i32, i32, i32, i32, i32, i32, i32, f32, p],
     "pie_gdn_copy_slot": [p, i64, i64, i32, i32, i32, p],
     "pie_mamba2_mixer": [p, i32, p, p, p, p, p, p, p, p, p, p, p, p, p, i32, i32, i32, i32, i32, i32, p],
-    "pie_stream_embed": [p, p, p, i32, i32, i32, i32, i32, p],
-    "pie_stream_norm": [p, i32, i32, p],
+    "pie_stream_embed": [p, p, p, i32, i32, i32, i32, f32, i32, p],
+    "pie_stream_norm": [p, i32, i32, i32, p],
     "pie_latent_rows": [p, i32, p],
     "pie_latent_attn_warp": [p, i32, p],
     "pie_gemm_bf16_xielu": [p, p, p, p, p, i32, i32, i32, i32, i32, i32, p, i32, p],
@@ -76,6 +76,20 @@ _SIGNATURES = {
     "pie_bias_xielu": [p, i32, p, p, i32, i32, i32, p],
     "pie_stream_add": [p, p, p, p, p, i32, i32, i32, p],
     "pie_side_gate": [p, i32, i64, i32, i32, p, i32, p, p, i32, i32, i32, i32, i32, i32, p],
+    "pie_linear_attn_serial": [p, i32, p],
+    "pie_linear_attn_chunk_supported": [i32],
+    "pie_linear_attn_chunk_tokens": [],
+    "pie_linear_attn_chunked": [p, p],
+    "pie_linear_decay": [p, i32, p, p, p, i32, i32, i32, f32, i32, p],
+    "pie_gated_norm": [p, i32, i32, p],
+    "pie_biased_rows": [p, i32, p],
+    "pie_biased_any": [p, i32, p],
+    "pie_biased_mma_supported": [i32, i32],
+    "pie_biased_decode": [p, p],
+    "pie_biased_prefill": [p, i32, p, p],
+    "pie_moe_route_scored": [p, i32, i64, i32, i32, i32, i32, i32, p, p, p, p, p, p],
+    "pie_moe_combine_identity": [p, p, p, p, i32, i32, i32, i32, p, i32, p],
+    "pie_grouped_gemm_clamp_glu": [p, p, p, p, i32, i32, i32, i32, i32, i32, f32, p, i32, p],
     "pie_gemm_set_workspace": [i32, p, i64, p, i32],
     "pie_gemm_set_pairs": [i32],
     "pie_gemm_set_swap": [i32],

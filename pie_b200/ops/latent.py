@@ -41,13 +41,14 @@ def _f32(t) -> int:
     return 1 if t.dtype == torch.float32 else 0
 
 
-def stream_embed(tokens, table, ld: int):
-    """Rows of `table` as a 32-bit stream [N, ld] (zeros beyond the table's width)."""
+def stream_embed(tokens, table, ld: int, scale: float = 1.0):
+    """Rows of `table` times `scale` as a 32-bit stream [N, ld] (zeros beyond the table's width)."""
     if not table.is_cuda:
-        return ref.stream_embed(tokens, table, ld)
+        return ref.stream_embed(tokens, table, ld, scale)
     n, w = tokens.numel(), table.shape[1]
     x = torch.empty(n, ld, dtype=torch.float32, device=table.device)
-    check(fn("pie_stream_embed")(ptr(tokens), ptr(table), ptr(x), n, w, ld, table.shape[0], _f32(table), stream_ptr()), "stream_embed")
+    check(fn("pie_stream_embed")(ptr(tokens), ptr(table), ptr(x), n, w, ld, table.shape[0], scale, _f32(table),
+                                 stream_ptr()), "stream_embed")
     return x
 
 
@@ -55,7 +56,8 @@ def stream_norm(x, width: int, eps: float, y=None, y_norm=None, norm_w=None, gro
                 dtype=None):
     """Per token: x += y / rms(y) * y_norm (if y); h = RMSNorm(x) in `groups` parts * norm_w; hs = h + (h of the token
     before - h) * shift. The token before the first one of a portion comes from the sequence's state in `rs`
-    (a `driver.recurrent.RecurrentInputs`), which advances. Returns (x, h, hs); what was not asked for is None."""
+    (a `driver.recurrent.RecurrentInputs`), which advances. The gains (norm_w, y_norm) are in the activation type or, both,
+    in 32-bit; `dtype` then names the activation type. Returns (x, h, hs); what was not asked for is None."""
     dtype = dtype or (norm_w if norm_w is not None else y).dtype
     if not x.is_cuda:
         return ref.stream_norm(x, width, eps, y, y_norm, norm_w, groups, shift, rs, layer, dtype)
@@ -67,7 +69,7 @@ def stream_norm(x, width: int, eps: float, y=None, y_norm=None, norm_w=None, gro
     a = StreamNormArgs(x=ptr(x), y=ptr(y), y_norm=ptr(y_norm), x_out=ptr(x_out), norm_w=ptr(norm_w), shift=ptr(shift), h=ptr(h),
                        hs=ptr(hs), n=n, width=width, ldx=ld, ldy=y.stride(0) if y is not None else 0, ldh=ld, groups=groups,
                        rows_per_block=max(1, min(8, n // 592)), eps=eps)
-    commit = 0
+    commit, gain_f32 = 0, _f32(norm_w if norm_w is not None else y_norm)
     if shift is not None:
         state = rs.shift_state[layer]
         a.tok_req, a.qo_indptr, a.slots, a.reset = ptr(rs.tok_req), ptr(rs.qo_indptr), ptr(rs.slots), ptr(rs.reset)
@@ -75,7 +77,7 @@ def stream_norm(x, width: int, eps: float, y=None, y_norm=None, norm_w=None, gro
         if rs.staged is None:               # portions of two tokens or more leave their last h in the stage
             rs.staged = len(rs.slots_host) if any(b - a > 1 for a, b in zip(rs.qo_host, rs.qo_host[1:])) else 0
         commit = rs.staged
-    check(fn("pie_stream_norm")(C.byref(a), 1 if dtype == torch.float32 else 0, commit, stream_ptr()), "stream_norm")
+    check(fn("pie_stream_norm")(C.byref(a), 1 if dtype == torch.float32 else 0, gain_f32, commit, stream_ptr()), "stream_norm")
     return (x if x_out is None else x_out), h, hs
 
 

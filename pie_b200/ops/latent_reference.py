@@ -4,9 +4,9 @@ from __future__ import annotations
 import torch
 
 
-def stream_embed(tokens, table, ld):
+def stream_embed(tokens, table, ld, scale=1.0):
     x = torch.zeros(tokens.numel(), ld, dtype=torch.float32)
-    x[:, :table.shape[1]] = table[tokens.long()].float()
+    x[:, :table.shape[1]] = table[tokens.long()].float() * scale
     return x
 
 

@@ -198,7 +198,8 @@ def cmd_model(args) -> int:
     for name in LAYERED_PRESETS:
         c = preset(name)
         print(f"  {name:18s} {c.model_type:10s} layers={c.num_hidden_layers:3d} hidden={c.hidden_size:5d} "
-              f"heads={c.num_attention_heads} latent={c.latent[0].kv_rank} vocab={c.vocab_size}")
+              + (f"heads={c.num_attention_heads} latent={c.latent[0].kv_rank} " if c.latent else
+                 f"mixers={'+'.join(sorted({type(b.mixer).__name__.replace('Spec', '') for b in c.blocks}))} ") + f"vocab={c.vocab_size}")
     return 0
 
 
