@@ -16,14 +16,14 @@ enum GemmEpilogue : int {
     EPI_RS = 3,        // reduce-scatter: rows go to their owner rank's receive buffer (peer stores)
     EPI_XIELU = 4,     // C = xIELU(acc + bias), see EpiArgs
     EPI_STREAM = 5,    // out32 = res32 + acc + bias: a 32-bit residual stream; C = the same in bf16
+    EPI_CLAMP_GLU = 6, // as EPI_SWIGLU with g = min(gate, limit), u = clamp(up, +-limit): g * sigmoid(1.702 g) * (u + 1)
     // Swapped operands (small batches): the kernel computes C^T = W * A^T, so its rows are output
-    // features and its columns tokens; these epilogues write the tile back transposed.
-    EPI_STORE_T = 6,
-    EPI_RESIDUAL_T = 7,
-    EPI_SWIGLU_T = 8,
-    EPI_XIELU_T = 9,
-    EPI_STREAM_T = 10,
-    EPI_CLAMP_GLU = 11,  // as EPI_SWIGLU with g = min(gate, limit), u = clamp(up, +-limit): g * sigmoid(1.702 g) * (u + 1)
+    // features and its columns tokens; these epilogues write the tile back transposed. EPI_STORE_T is the first of them.
+    EPI_STORE_T = 7,
+    EPI_RESIDUAL_T = 8,
+    EPI_SWIGLU_T = 9,
+    EPI_XIELU_T = 10,
+    EPI_STREAM_T = 11,
 };
 
 // Operands of the epilogues with a bias. xIELU(z) = a z^2 + z / 2 for z > 0, b (e^z - 1 - z) + z / 2 below, with
