@@ -364,9 +364,10 @@ def complete_blocks(cfg: ModelConfig, reader) -> None:
         if isinstance(b.mixer, GatedLinearSpec):
             b.mixer.rank = rows
         else:
-            b.attention.buckets = rows
-            if rows < 2 or b.attention.bias_max <= rows // 2:
-                raise LoaderTypeError(f"{name}: {rows} rows for distances up to {b.attention.bias_max}")
+            a = b.attention
+            a.buckets = rows
+            if a.window > rows // 2 and a.bias_max <= rows // 2:
+                raise LoaderTypeError(f"{name}: {rows} rows for distances up to {a.bias_max}")
 
 
 def _compile_blocks(cfg: ModelConfig, names: set, tp_size: int, dtype: str) -> Program:

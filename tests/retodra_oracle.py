@@ -126,6 +126,10 @@ def clamped_expert(h, w, limit):
     return (g * sigmoid(1.702 * g) * (u + 1)) @ w["down"].t()
 
 
+def identity_expert(h):
+    return h
+
+
 def route(h, router, correction, top):
     """(ids, weights) [T, top]: chosen by score + correction, weighted by the score itself."""
     s = torch.softmax(h @ router.t(), -1)
@@ -139,7 +143,7 @@ def moe(h, w, mlp):
     out = torch.zeros_like(h)
     for t in range(h.shape[0]):
         for e, c in zip(ids[t].tolist(), weights[t]):
-            y = h[t] if e >= r["experts"] else clamped_expert(h[t], sub(w, f"e{e}."), mlp["expert"]["limit"])
+            y = identity_expert(h[t]) if e >= r["experts"] else clamped_expert(h[t], sub(w, f"e{e}."), mlp["expert"]["limit"])
             out[t] += c * y
     return out
 
