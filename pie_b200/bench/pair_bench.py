@@ -1,10 +1,12 @@
-"""Prefill and decode throughput of the Puzutar design beside the closest model of equal size (the Llama-8B shape with a
-sliding window): same width, heads, window, vocabulary and parameters per layer, random weights, bf16.
+"""Prefill and decode throughput of a design beside the closest other model of equal size, random weights, bf16.
 
-    python bench.py --config 7 [--layers 32]
+    python bench.py --config 7 [--layers 32]    Puzutar beside the Llama-8B shape with a sliding window
+    python bench.py --config 8 [--layers 32]    Retodra beside Gated DeltaNet and windowed attention with experts
 
-Device-timed with CUDA events after warm-up. Decode replays the captured step over contexts of `--context` tokens; the
-weights read per step exceed the L2. Prefill runs whole prompts as one batch. One JSON line.
+Both models of a pair have the same width, heads, window, vocabulary and feed-forward sizes (config 8: also the same
+states of the linear mixers, experts and routes per token). Device-timed with CUDA events after warm-up. Decode replays
+the captured step over contexts of `--context` tokens; the weights read per step exceed the L2. Prefill runs whole prompts
+as one batch. One JSON line.
 """
 from __future__ import annotations
 
@@ -14,7 +16,7 @@ import json
 
 import numpy as np
 
-PAIR = ("puzutar-8b", "llama-8b-window")
+PAIRS = {7: ("puzutar-8b", "llama-8b-window"), 8: ("retodra-19b", "gdn-moe-window-19b")}
 DECODE_ROWS = (16, 64, 256)
 PREFILL = ((1, 2048), (4, 2048), (1, 8192))
 
@@ -27,7 +29,8 @@ def _driver(name: str, layers: int, max_tokens: int, rows: int, pages: int):
     drv = TorchDriver(cfg, "cuda", page_size=16, num_pages=pages, max_requests=rows, max_tokens=max_tokens,
                       rs_slots=rows if cfg.recurrent_layers else 0)
     torch.manual_seed(0)
-    drv.kv.data.normal_(0.0, 0.5)
+    for t in drv.kv.parts:
+        t.normal_(0.0, 0.5)
     return cfg, drv
 
 
@@ -86,13 +89,14 @@ def main(argv=None):
     ap.add_argument("--warmup", type=int, default=4)
     ap.add_argument("--layers", type=int, default=0)
     ap.add_argument("--context", type=int, default=2048)
+    ap.add_argument("--config", type=int, default=7, choices=sorted(PAIRS))
     ap.add_argument("--only", default="", help="one of the two models")
     a = ap.parse_args(argv)
     from . import harness
     clk = harness.ClockSampler(0).start()
-    runs = [measure(m, a.layers, a.context, a.steps, max(3, a.warmup)) for m in PAIR if not a.only or a.only == m]
+    runs = [measure(m, a.layers, a.context, a.steps, max(3, a.warmup)) for m in PAIRS[a.config] if not a.only or a.only == m]
     clocks = clk.stop()
-    line = {"config": 7, "metric": "decode and prefill tokens/s of two models of equal size", "unit": "tokens/s", "n_gpus": 1,
+    line = {"config": a.config, "metric": "decode and prefill tokens/s of two models of equal size", "unit": "tokens/s", "n_gpus": 1,
             "dtype": "bf16", "data": "synthetic random tokens and cache contents, random-init weights", "runs": runs,
             "l2": "weights and cache per step exceed the 126 MB L2; no flush needed", "clocks": clocks}
     print(json.dumps(line), flush=True)

@@ -149,9 +149,10 @@ __global__ void moe_permute_kernel(const bf16* __restrict__ x, int ldx, const in
     for (int c = threadIdx.x; c < H / 8; c += blockDim.x) dst[c] = src[c];
 }
 
-// One block per token. `self`: a route without a slot is an expert that returns its input, row t of `self`. RS: the (partial) row goes to the receive buffer of the rank that owns
-// token t (reduce-scatter by peer stores, same protocol as the GEMM's EPI_RS epilogue); the last
-// block to finish raises this rank's flag on every owner.
+// One block per token. `self`: a route without a slot is an expert that returns its input, row t of `self`.
+// RS: the (partial) row goes to the receive buffer of the rank that owns token t (reduce-scatter by peer
+// stores, same protocol as the GEMM's EPI_RS epilogue); the last block to finish raises this rank's flag on
+// every owner.
 template <bool RS>
 __global__ void moe_combine_kernel(const bf16* __restrict__ y, const int* __restrict__ slot_of,
                                    const float* __restrict__ w, const bf16* __restrict__ residual, int ldr, int H,

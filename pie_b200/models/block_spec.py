@@ -199,7 +199,7 @@ def retodra_dict(cfg) -> dict:
             "norm": {"eps": cfg.rms_norm_eps}, "embedding": {"scale": cfg.embed_scale}}
 
 
-def retodra_shape(layers: int = 32, width: int = 4096, gla_heads: int = 8, gla_dim: int = 256, gla_vdim: int = 512, rank: int = 16,
+def retodra_shape(layers: int = 32, width: int = 4096, gla_heads: int = 16, gla_dim: int = 128, gla_vdim: int = 256, rank: int = 16,
                   tau: float = 16.0, heads: int = 32, kv_heads: int = 8, dim: int = 128, window: int = 1024, buckets: int = 32,
                   right_heads: int = 16, right_dim: int = 128, right_vdim: int = 128, ff: int = 11008, experts: int = 32,
                   identity: int = 4, top: int = 4, expert_ff: int = 2048, vocab: int = 128256) -> dict:

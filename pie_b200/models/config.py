@@ -462,6 +462,13 @@ PRESETS = {
     "llama-8b-window": dict(model_type="mistral", hidden_size=4096, intermediate_size=14336, num_hidden_layers=32,
                             num_attention_heads=32, num_key_value_heads=8, head_dim=128, vocab_size=128256,
                             rope_theta=500000.0, rms_norm_eps=1e-5, sliding_window=1024),
+    # Gated DeltaNet and windowed attention with experts, layer about: what `retodra-19b` is measured beside
+    "gdn-moe-window-19b": dict(model_type="qwen3_next", hidden_size=4096, intermediate_size=11008, num_hidden_layers=32,
+                               num_attention_heads=32, num_key_value_heads=8, head_dim=128, vocab_size=128256, rope_theta=500000.0,
+                               rms_norm_eps=1e-5, qk_norm=True, sliding_window=1024,
+                               layer_types=["linear_attention", "sliding_attention"] * 16, linear_num_key_heads=16,
+                               linear_num_value_heads=32, linear_key_head_dim=128, linear_value_head_dim=128, num_experts=32,
+                               num_experts_per_tok=4, moe_intermediate_size=2048),
     "qwen3-32b": dict(model_type="qwen3", hidden_size=5120, intermediate_size=25600,
                       num_hidden_layers=64, num_attention_heads=64, num_key_value_heads=8, head_dim=128,
                       vocab_size=151936, rope_theta=1000000.0, rms_norm_eps=1e-6, qk_norm=True),
@@ -537,9 +544,9 @@ PRESETS = {
 # presets of designs whose layers are described one by one: reader, shape and the shape's arguments
 LAYERED_PRESETS = {
     "puzutar-8b": (_puzutar_config, puzutar_shape, dict()),
-    "retodra-8b": (retodra_config, retodra_shape, dict()),
-    "tiny-puzutar": (_puzutar_config, puzutar_shape, dict(layers=3, width=256, heads=2, dim=48, rot_dim=16, vdim=40, kv_rank=64, window=40, ff=384, vocab=32000,
-                         groups=2, side=16)),
+    "retodra-19b": (retodra_config, retodra_shape, dict()),
+    "tiny-puzutar": (_puzutar_config, puzutar_shape, dict(
+        layers=3, width=256, heads=2, dim=48, rot_dim=16, vdim=40, kv_rank=64, window=40, ff=384, vocab=32000, groups=2, side=16)),
     "tiny-retodra": (retodra_config, retodra_shape, dict(
         layers=4, width=256, gla_heads=2, gla_dim=48, gla_vdim=64, rank=8, heads=6, kv_heads=2, dim=40, window=50, buckets=12,
         right_heads=3, right_dim=32, right_vdim=40, ff=384, experts=6, identity=2, top=3, expert_ff=96, vocab=32000)),

@@ -175,13 +175,15 @@ def biased_attention(q, cache, bias, plan, rs, slots, spec):
         a.qo_indptr, a.tok_req, a.slots = ptr(rs.qo_indptr), ptr(rs.tok_req), ptr(slots)
         check(fn("pie_biased_any")(C.byref(a), _f32(q), stream_ptr()), "biased_any")
     elif decode:
-        a.item_req, a.item_start, a.item_end, a.req_item_indptr = ptr(plan.item_req), ptr(plan.item_start), ptr(plan.item_end), ptr(plan.req_item_indptr)
-        a.num_items, a.scratch, a.max_items, a.num_reqs, a.num_ctas = ptr(plan.num_items), ptr(plan.scratch), plan.max_items, plan.num_reqs, plan.num_ctas
+        a.item_req, a.item_start, a.item_end = ptr(plan.item_req), ptr(plan.item_start), ptr(plan.item_end)
+        a.req_item_indptr, a.num_items, a.scratch = ptr(plan.req_item_indptr), ptr(plan.num_items), ptr(plan.scratch)
+        a.max_items, a.num_reqs, a.num_ctas = plan.max_items, plan.num_reqs, plan.num_ctas
         check(fn("pie_biased_decode")(C.byref(a), stream_ptr()), "biased_decode")
     else:
         rows = 256 if page == 16 and D <= 128 else 64
         t = _prefill_tiles(plan, spec.group_pad, rows, q.device)
-        a.qo_indptr, a.tile_req, a.tile_qstart, a.num_tiles, a.total_pages = ptr(plan.qo_indptr), ptr(t[0]), ptr(t[1]), t.shape[1], cache.shape[0]
+        a.qo_indptr, a.tile_req, a.tile_qstart = ptr(plan.qo_indptr), ptr(t[0]), ptr(t[1])
+        a.num_tiles, a.total_pages = t.shape[1], cache.shape[0]
         check(fn("pie_biased_prefill")(C.byref(a), rows, ptr(ops.kernel_status(q.device)), stream_ptr()), "biased_prefill")
     return out
 

@@ -41,8 +41,8 @@ CONFIGS = {
                    gla(5, 7, 11, 30.0, moe(2, 5, 4, 10))], 100, 131),
     # a window of one token, one head, one expert, keys of one number; experts on linear layers and dense parallel ones.
     # (Values of one number are left to the tests of the ops: normed, they are nothing but a sign.)
-    "ones": config([par(1, 1, 4, 8, 1, 90, (1, 1, 8), dense(16)), gla(1, 1, 16, 1.0, moe(1, 1, 2, 8)), par(1, 1, 16, 8, 3, 90, (1, 8, 8), moe(1, 0, 1, 9))],
-                   48, 97, scale=1.0),
+    "ones": config([par(1, 1, 4, 8, 1, 90, (1, 1, 8), dense(16)), gla(1, 1, 16, 1.0, moe(1, 1, 2, 8)),
+                    par(1, 1, 16, 8, 3, 90, (1, 8, 8), moe(1, 0, 1, 9))], 48, 97, scale=1.0),
     # heads of 128, groups of four and eight, several pieces and key blocks; strong channel decays
     "wide": config([gla(2, 96, 128, 1.0, dense(200)), par(8, 2, 128, 128, 150, 400, (2, 64, 96), moe(6, 2, 2, 64)),
                     par(8, 1, 72, 100, 70, 150, (2, 128, 32), None)], 256, 300),

@@ -342,7 +342,8 @@ def test_experts_with_identity_outputs(path, experts, identity, top, ff, width, 
     corr = torch.randperm(e, generator=torch.Generator().manual_seed(2)).float() * 0.3
     w = {"router": router, "correction": corr}
     for i in range(experts):
-        w[f"e{i}.gate"], w[f"e{i}.up"] = rnd(ff, width, seed=10 + i, dtype=dt, std=1.5 * width ** -0.5), rnd(ff, width, seed=90 + i, dtype=dt, std=1.5 * width ** -0.5)
+        for j, name in ((10, "gate"), (90, "up")):
+            w[f"e{i}.{name}"] = rnd(ff, width, seed=j + i, dtype=dt, std=1.5 * width ** -0.5)
         w[f"e{i}.down"] = rnd(width, ff, seed=170 + i, dtype=dt, std=ff ** -0.5)
     ref = oracle.moe(h, w, {"router": {"experts": experts, "top": top}, "expert": {"limit": 1.2}})
     gu, down = torch.zeros(experts, 2 * fp, wp), torch.zeros(experts, wp, fp)

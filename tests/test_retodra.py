@@ -239,7 +239,7 @@ def test_configuration_and_registry():
         change(bad)
         with pytest.raises(ValueError):
             ModelConfig.from_hf(bad)
-    assert preset("retodra-8b", num_hidden_layers=2).num_hidden_layers == 2
+    assert preset("retodra-19b", num_hidden_layers=2).num_hidden_layers == 2
 
 
 @pytest.mark.parametrize("rows,far", [(12, 90), (8, 64), (32, 128), (2, 9), (16, 1000)])
