@@ -27,7 +27,7 @@ struct BiasedRowsArgs {
     float eps;
 };
 
-template <typename T>
+template <typename T, int VEC>
 __global__ void __launch_bounds__(256) biased_rows_kernel(const BiasedRowsArgs a) {
     __shared__ float red[32];
     pdl_trigger();
@@ -37,29 +37,51 @@ __global__ void __launch_bounds__(256) biased_rows_kernel(const BiasedRowsArgs a
     const T* k = static_cast<const T*>(a.k) + (size_t)t * a.ld;
     const T* v = static_cast<const T*>(a.v) + (size_t)t * a.ld;
     const int nq = a.heads * a.dim, nk = a.kv_heads * a.dim;
-    float sq = 0.f, sk = 0.f;
-    for (int i = threadIdx.x; i < nq; i += 256) { const float f = to_f(q[i]); sq += f * f; }
-    for (int i = threadIdx.x; i < nk; i += 256) { const float f = to_f(k[i]); sk += f * f; }
+    auto squares = [&](const T* x, int n) {
+        float s = 0.f;
+        for (int i = threadIdx.x * VEC; i < n; i += 256 * VEC) {
+            float f[VEC];
+            load_vec<VEC>(x + i, f);
+#pragma unroll
+            for (int e = 0; e < VEC; ++e) s += f[e] * f[e];
+        }
+        return s;
+    };
+    const float sq = squares(q, nq), sk = squares(k, nk);
     const float iq = 1.f / sqrtf(block_sum(sq, red) / (float)nq + a.eps);
     const float ik = 1.f / sqrtf(block_sum(sk, red) / (float)nk + a.eps);
     const T* wq = static_cast<const T*>(a.q_norm);
     const T* wk = static_cast<const T*>(a.k_norm);
+    // columns past a head's size and rows past a group's are zeros
+    auto emit = [&](T* dst, const T* src, const T* w, float inv, bool ok) {
+        float f[VEC], g[VEC];
+#pragma unroll
+        for (int e = 0; e < VEC; ++e) f[e] = 0.f;
+        if (ok) {
+            load_vec<VEC>(src, f);
+            if (w) {
+                load_vec<VEC>(w, g);
+#pragma unroll
+                for (int e = 0; e < VEC; ++e) f[e] *= inv * g[e];
+            }
+        }
+        store_vec<VEC>(dst, f);
+    };
     T* qo = static_cast<T*>(a.q_out) + (size_t)t * a.kv_heads * a.group_pad * a.D;
-    for (int i = threadIdx.x; i < a.kv_heads * a.group_pad * a.D; i += 256) {
+    for (int i = threadIdx.x * VEC; i < a.kv_heads * a.group_pad * a.D; i += 256 * VEC) {
         const int hp = i / a.D, d = i - hp * a.D, kv = hp / a.group_pad, g = hp - kv * a.group_pad;
         const int src = (kv * a.group + g) * a.dim + d;
-        qo[i] = from_f<T>(g < a.group && d < a.dim ? to_f(q[src]) * iq * to_f(wq[src]) : 0.f);
+        emit(qo + i, q + src, wq + src, iq, g < a.group && d < a.dim);
     }
     const int slot = a.slots[t];
     if (slot < 0) return;
     const int page = slot / a.page_size, off = slot % a.page_size;
     T* base = static_cast<T*>(a.cache) + (size_t)page * 2 * a.kv_heads * a.page_size * a.D;
-    for (int i = threadIdx.x; i < 2 * a.kv_heads * a.D; i += 256) {
+    for (int i = threadIdx.x * VEC; i < 2 * a.kv_heads * a.D; i += 256 * VEC) {
         const int hv = i / a.D, d = i - hv * a.D, h = hv % a.kv_heads;
-        float f = 0.f;
-        if (hv < a.kv_heads) { if (d < a.dim) f = to_f(k[h * a.dim + d]) * ik * to_f(wk[h * a.dim + d]); }
-        else if (d < a.vdim) f = to_f(v[h * a.vdim + d]);
-        base[((size_t)hv * a.page_size + off) * a.D + d] = from_f<T>(f);
+        T* dst = base + ((size_t)hv * a.page_size + off) * a.D + d;
+        if (hv < a.kv_heads) emit(dst, k + h * a.dim + d, wk + h * a.dim + d, ik, d < a.dim);
+        else emit(dst, v + h * a.vdim + d, nullptr, 1.f, d < a.vdim);
     }
 }
 
@@ -148,8 +170,12 @@ PIE_API int pie_biased_rows(const BiasedRowsArgs* args, int f32, cudaStream_t st
     const BiasedRowsArgs& a = *args;
     if (a.n <= 0) return 0;
     if (a.group > a.group_pad || a.heads != a.kv_heads * a.group || a.dim > a.D || a.vdim > a.D) return (int)cudaErrorInvalidValue;
-    return (int)(f32 ? launch_pdl(biased_rows_kernel<float>, dim3(a.n), dim3(256), 0, st, a)
-                     : launch_pdl(biased_rows_kernel<bf16>, dim3(a.n), dim3(256), 0, st, a));
+    auto aligned = [](const void* p) { return ((uintptr_t)p & 15) == 0; };
+    const bool vec = a.dim % 4 == 0 && a.vdim % 4 == 0 && a.ld % 4 == 0 && aligned(a.q) && aligned(a.k) && aligned(a.v) &&
+                     aligned(a.q_norm) && aligned(a.k_norm) && aligned(a.q_out) && aligned(a.cache);
+    auto kern = f32 ? (vec ? biased_rows_kernel<float, 4> : biased_rows_kernel<float, 1>)
+                    : (vec ? biased_rows_kernel<bf16, 4> : biased_rows_kernel<bf16, 1>);
+    return (int)launch_pdl(kern, dim3(a.n), dim3(256), 0, st, a);
 }
 
 PIE_API int pie_biased_any(const BiasedAttnArgs* args, int f32, cudaStream_t st) {

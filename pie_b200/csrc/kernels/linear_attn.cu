@@ -22,7 +22,7 @@ __device__ __forceinline__ float la_silu(float x) { return x / (1.f + expf(-x));
 
 struct LinAttnArgs {
     const void *q, *k, *v;       // row t, head h at t * ld + h * dim (h * vdim for v), type T
-    const float* log_decay;      // [n, heads * dim] base 2, or null
+    float* log_decay;            // [n, heads * dim] base 2, or null; the chunked form leaves running sums of the pieces
     const float* head_decay;     // [heads] the factor itself (null with log_decay)
     float* out;                  // [n, heads * vdim]
     float* state;                // this layer's part of slot 0: [heads][dim][vdim]
@@ -125,168 +125,274 @@ __global__ void __launch_bounds__(256) la_serial_kernel(const LinAttnArgs a) {
 
 // ----------------------------------------------------------------- chunked
 constexpr int LA_C = 64;                  // tokens per piece
-constexpr int LA_VT = 32;                 // value columns per pass of the output kernel
+constexpr int LA_VT = 64;                 // value columns per pass
+constexpr int LA_VP = LA_VT + 8;          // pitch of a tile read as (row by t, column by g): fragment reads hit 32 banks
+constexpr int LA_SP = LA_C + 4;           // pitch of the scores, and of values read at rows 2 t, 2 t + 1
+constexpr int LA_THREADS = 256;
 
 __device__ __forceinline__ uint32_t tf32(float x) {
     uint32_t r;
     asm("cvt.rna.tf32.f32 %0, %1;" : "=r"(r) : "f"(x));
     return r;
 }
+__device__ __forceinline__ float tf32_f(float x) { return __uint_as_float(tf32(x)); }
 // C (16 x 8) += A (16 x 8, row) B (8 x 8, col); lane (g = lane / 4, t = lane % 4) holds A (g | g + 8, t | t + 4),
-// B (t | t + 4, g) and C (g | g + 8, 2 t | 2 t + 1)
-__device__ __forceinline__ void mma_tf32(float (&c)[4], const uint32_t (&a)[4], uint32_t b0, uint32_t b1) {
+// B (t | t + 4, g) and C (g | g + 8, 2 t | 2 t + 1). Operands are already rounded to tf32.
+__device__ __forceinline__ void mma_tf32(float (&c)[4], const float (&a)[4], float b0, float b1) {
     asm volatile("mma.sync.aligned.m16n8k8.row.col.f32.tf32.tf32.f32 {%0,%1,%2,%3}, {%4,%5,%6,%7}, {%8,%9}, {%0,%1,%2,%3};\n"
                  : "+f"(c[0]), "+f"(c[1]), "+f"(c[2]), "+f"(c[3])
-                 : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b0), "r"(b1));
+                 : "r"(__float_as_uint(a[0])), "r"(__float_as_uint(a[1])), "r"(__float_as_uint(a[2])), "r"(__float_as_uint(a[3])),
+                   "r"(__float_as_uint(b0)), "r"(__float_as_uint(b1)));
 }
 
-// Rows of a chunk in shared memory: pitch of the [64][dim] arrays, in elements
-__host__ __device__ constexpr int la_pitch(int dim) { return (dim + 15) / 16 * 16 + 8; }
+__host__ __device__ constexpr int la_dimp(int dim) { return (dim + 15) / 16 * 16; }
+// Pitch of a [64][dim] array of bf16 (queries, keys) and of 32-bit decayed keys: 8 (mod 32) words or 4 (mod 16)
+__host__ __device__ constexpr int la_pitch(int dim) { return la_dimp(dim) + 8; }
 
-template <bool CHAN>
-__global__ void __launch_bounds__(128) la_chunk_state_kernel(const LinAttnArgs a) {
-    extern __shared__ float sm[];
+// Eight bf16 of a row of a projection as floats (with the activation, rounded to tf32), zeros outside; VEC: one 16-byte load.
+template <bool VEC>
+__device__ __forceinline__ void la_load8(const bf16* p, int valid, bool act, float (&f)[8]) {
+    if (VEC && valid >= 8) {
+        unpack8(*reinterpret_cast<const bf16x8*>(p), f);
+    } else {
+#pragma unroll
+        for (int e = 0; e < 8; ++e) f[e] = e < valid ? to_f(p[e]) : 0.f;
+    }
+    if (act) {
+#pragma unroll
+        for (int e = 0; e < 8; ++e) f[e] = tf32_f(f[e] / (1.f + __expf(-f[e])));
+    }
+}
+
+// A tile of values [64 tokens][64 columns] on its way from global to shared memory: two 8-column vectors per thread.
+template <bool VEC>
+struct ValueTile {
+    float f[2][8];
+    __device__ __forceinline__ void load(const bf16* v, int ld, int len, int cols, bool act) {
+#pragma unroll
+        for (int i = 0; i < 2; ++i) {
+            const int u = threadIdx.x + i * LA_THREADS, s = u >> 3, j = (u & 7) * 8;
+            la_load8<VEC>(v + (size_t)s * ld + j, s < len ? min(8, cols - j) : 0, act, f[i]);
+        }
+    }
+    template <int PITCH>
+    __device__ __forceinline__ void store(float* dst) const {
+#pragma unroll
+        for (int i = 0; i < 2; ++i) {
+            const int u = threadIdx.x + i * LA_THREADS, s = u >> 3, j = (u & 7) * 8;
+            float4* d = reinterpret_cast<float4*>(dst + s * PITCH + j);
+            d[0] = make_float4(f[i][0], f[i][1], f[i][2], f[i][3]);
+            d[1] = make_float4(f[i][4], f[i][5], f[i][6], f[i][7]);
+        }
+    }
+};
+
+// U and the piece's decay; turns log_decay into its running sum from the piece's start (in place), which la_chunk_out reads.
+template <bool CHAN, bool VEC>
+__global__ void __launch_bounds__(LA_THREADS) la_chunk_state_kernel(const LinAttnArgs a) {
+    extern __shared__ __align__(16) float sm[];
     const int c = blockIdx.x, h = blockIdx.y, r = a.chunk_req[c];
     const int row0 = a.chunk_start[c], len = min(LA_C, a.qo_indptr[r + 1] - row0);
-    const int dimp = (a.dim + 15) / 16 * 16, kp = la_pitch(a.dim), vp = 72;
+    const int dimp = la_dimp(a.dim), kp = la_pitch(a.dim);
     float* sk = sm;                        // [64][kp] decayed keys
-    float* sv = sk + LA_C * kp;            // [64][72] a tile of values
+    float* sv = sk + LA_C * kp;            // [64][LA_VP] a tile of values
+    float* tot = sv + LA_C * LA_VP;        // [128] decay of the first 32 tokens
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, g = lane >> 2, t = lane & 3;
-    const float lh = CHAN ? 0.f : log2f(a.head_decay[h]);
-    const bf16* kb = static_cast<const bf16*>(a.k) + h * a.dim;
-    for (int d = threadIdx.x; d < dimp; d += 128) {
-        float w = 0.f;                     // base-2 decay from this token to the end of the piece
-        for (int s = LA_C - 1; s >= 0; --s) {
-            float k = 0.f;
-            if (s < len && d < a.dim) {
-                const size_t row = (size_t)(row0 + s);
-                k = to_f(kb[row * a.ld + d]);
-                if (a.silu) k = la_silu(k);
-                k *= exp2f(w);
-                w += CHAN ? a.log_decay[row * a.heads * a.dim + h * a.dim + d] : lh;
+    const bf16* kb = static_cast<const bf16*>(a.k) + (size_t)row0 * a.ld + h * a.dim;
+    const bf16* vb = static_cast<const bf16*>(a.v) + (size_t)row0 * a.ld + h * a.vdim;
+    ValueTile<VEC> vt;
+    vt.load(vb, a.ld, len, a.vdim, a.silu);
+    if (CHAN) {
+        const int half = threadIdx.x >> 7;
+        float* dec = a.piece_decay + ((size_t)c * a.heads + h) * a.dim;
+        for (int d0 = 0; d0 < dimp; d0 += 128) {
+            const int d = d0 + (threadIdx.x & 127);
+            const bool ok = d < a.dim;
+            float* lg = a.log_decay + ((size_t)(row0 + half * 32) * a.heads + h) * a.dim + d;
+            const size_t step = (size_t)a.heads * a.dim;
+            float b[32], k[32], run = 0.f;
+#pragma unroll
+            for (int s = 0; s < 32; ++s) {
+                const bool in = ok && half * 32 + s < len;
+                b[s] = in ? lg[s * step] : 0.f;
+                k[s] = in ? to_f(kb[(size_t)(half * 32 + s) * a.ld + d]) : 0.f;
             }
-            sk[s * kp + d] = k;
+#pragma unroll
+            for (int s = 0; s < 32; ++s) b[s] = run += b[s];
+            if (half == 0) tot[threadIdx.x] = run;
+            __syncthreads();
+            const float base = half ? tot[threadIdx.x & 127] : 0.f;
+            __syncthreads();
+            if (half) tot[threadIdx.x & 127] = base + run;
+            __syncthreads();
+            const float all = tot[threadIdx.x & 127];
+            if (half && ok) dec[d] = all;
+            if (d < dimp) {
+#pragma unroll
+                for (int s = 0; s < 32; ++s) {
+                    const float x = base + b[s];
+                    if (ok && half * 32 + s < len) lg[s * step] = x;
+                    float kv = k[s];
+                    if (a.silu) kv = la_silu(kv);
+                    sk[(half * 32 + s) * kp + d] = tf32_f(kv * exp2f(all - x));
+                }
+            }
+            __syncthreads();               // `tot` is free for the next channels
         }
-        if (d < a.dim) a.piece_decay[((size_t)c * a.heads + h) * a.dim + d] = w;
+    } else {
+        const float lh = log2f(a.head_decay[h]);
+        for (int u = threadIdx.x; u < LA_C * (dimp / 8); u += LA_THREADS) {
+            const int s = u / (dimp / 8), d = (u - s * (dimp / 8)) * 8;
+            float f[8];
+            la_load8<VEC>(kb + (size_t)s * a.ld + d, s < len ? min(8, a.dim - d) : 0, a.silu, f);
+            const float w = s < len ? exp2f((float)(len - 1 - s) * lh) : 0.f;
+#pragma unroll
+            for (int e = 0; e < 8; ++e) sk[s * kp + d + e] = tf32_f(f[e] * w);
+        }
+        for (int d = threadIdx.x; d < a.dim; d += LA_THREADS)
+            a.piece_decay[((size_t)c * a.heads + h) * a.dim + d] = (float)len * lh;
     }
     float* U = a.u + ((size_t)c * a.heads + h) * a.dim * a.vdim;
-    const bf16* vb = static_cast<const bf16*>(a.v) + h * a.vdim;
-    for (int v0 = 0; v0 < a.vdim; v0 += 64) {
+    for (int v0 = 0; v0 < a.vdim; v0 += LA_VT) {
         __syncthreads();
-        for (int i = threadIdx.x; i < LA_C * 64; i += 128) {
-            const int s = i >> 6, j = i & 63;
-            float v = 0.f;
-            if (s < len && v0 + j < a.vdim) {
-                v = to_f(vb[(size_t)(row0 + s) * a.ld + v0 + j]);
-                if (a.silu) v = la_silu(v);
-            }
-            sv[s * vp + j] = v;
-        }
+        vt.template store<LA_VP>(sv);
         __syncthreads();
-        const int nt = min(8, (a.vdim - v0 + 7) / 8);
-        for (int m = warp; m < dimp / 16; m += 4) {
+        if (v0 + LA_VT < a.vdim) vt.load(vb + v0 + LA_VT, a.ld, len, a.vdim - v0 - LA_VT, a.silu);
+        for (int m = warp; m < dimp / 16; m += LA_THREADS / 32) {
             float acc[8][4];
 #pragma unroll
             for (int n = 0; n < 8; ++n) acc[n][0] = acc[n][1] = acc[n][2] = acc[n][3] = 0.f;
-#pragma unroll
+#pragma unroll 2
             for (int ks = 0; ks < LA_C / 8; ++ks) {
                 const float* kr = sk + (ks * 8 + t) * kp + m * 16 + g;
-                const uint32_t fa[4] = {tf32(kr[0]), tf32(kr[8]), tf32(kr[4 * kp]), tf32(kr[4 * kp + 8])};
+                const float fa[4] = {kr[0], kr[8], kr[4 * kp], kr[4 * kp + 8]};
+                const float* vr = sv + (ks * 8 + t) * LA_VP + g;
 #pragma unroll
-                for (int n = 0; n < 8; ++n) {
-                    if (n >= nt) break;
-                    const float* vr = sv + (ks * 8 + t) * vp + n * 8 + g;
-                    mma_tf32(acc[n], fa, tf32(vr[0]), tf32(vr[4 * vp]));
-                }
+                for (int n = 0; n < 8; ++n) mma_tf32(acc[n], fa, vr[n * 8], vr[4 * LA_VP + n * 8]);
             }
 #pragma unroll
             for (int n = 0; n < 8; ++n)
 #pragma unroll
-                for (int e = 0; e < 4; ++e) {
-                    const int d = m * 16 + g + (e >> 1) * 8, j = v0 + n * 8 + 2 * t + (e & 1);
-                    if (d < a.dim && j < a.vdim) U[(size_t)d * a.vdim + j] = acc[n][e];
+                for (int e = 0; e < 4; e += 2) {
+                    const int d = m * 16 + g + (e >> 1) * 8, j = v0 + n * 8 + 2 * t;
+                    if (d >= a.dim) continue;
+                    float* u = U + (size_t)d * a.vdim + j;
+                    if (VEC && j + 1 < a.vdim) {
+                        *reinterpret_cast<float2*>(u) = make_float2(acc[n][e], acc[n][e + 1]);
+                    } else {
+                        if (j < a.vdim) u[0] = acc[n][e];
+                        if (j + 1 < a.vdim) u[1] = acc[n][e + 1];
+                    }
                 }
         }
     }
 }
 
-// One thread per state element: U becomes the state before each piece; the state after the last goes back to its slot.
+// One thread per V state elements: U becomes the state before each piece; the state after the last goes back to its slot.
+template <int V>
 __global__ void __launch_bounds__(256) la_chunk_scan_kernel(const LinAttnArgs a) {
     const int r = blockIdx.y, slot = a.slots[r];
     const int c0 = a.req_chunks[r], c1 = a.req_chunks[r + 1];
-    const long elems = (long)a.heads * a.dim * a.vdim, i = blockIdx.x * 256L + threadIdx.x;
+    const long elems = (long)a.heads * a.dim * a.vdim, i = (blockIdx.x * 256L + threadIdx.x) * V;
     if (i >= elems || c1 <= c0 || slot < 0) return;
     float* sp = a.state + (size_t)slot * a.slot_stride + i;
-    float s = a.reset[r] ? 0.f : *sp;
+    float s[V];
+    load_vec<V>(sp, s);
+    if (a.reset[r])
+#pragma unroll
+        for (int e = 0; e < V; ++e) s[e] = 0.f;
     float* u = a.u + i;
     const float* dec = a.piece_decay + i / a.vdim;
     const long dstep = (long)a.heads * a.dim;
-    int c = c0;
-    for (; c + 4 <= c1; c += 4) {
-        float x[4], w[4];
+    constexpr int AHEAD = 8;
+    for (int c = c0; c < c1; c += AHEAD) {
+        float x[AHEAD][V], w[AHEAD];
 #pragma unroll
-        for (int j = 0; j < 4; ++j) { x[j] = u[(c + j) * elems]; w[j] = dec[(c + j) * dstep]; }
+        for (int j = 0; j < AHEAD; ++j)
+            if (c + j < c1) {
+                load_vec<V>(u + (c + j) * elems, x[j]);
+                w[j] = dec[(c + j) * dstep];
+            }
 #pragma unroll
-        for (int j = 0; j < 4; ++j) {
-            u[(c + j) * elems] = s;
-            s = exp2f(w[j]) * s + x[j];
-        }
+        for (int j = 0; j < AHEAD; ++j)
+            if (c + j < c1) {
+                store_vec<V>(u + (c + j) * elems, s);
+                const float f = exp2f(w[j]);
+#pragma unroll
+                for (int e = 0; e < V; ++e) s[e] = f * s[e] + x[j][e];
+            }
     }
-    for (; c < c1; ++c) {
-        const float x = u[c * elems], w = dec[c * dstep];
-        u[c * elems] = s;
-        s = exp2f(w) * s + x;
-    }
-    *sp = s;
+    store_vec<V>(sp, s);
 }
 
-template <bool CHAN>
-__global__ void __launch_bounds__(128) la_chunk_out_kernel(const LinAttnArgs a) {
-    extern __shared__ float sm[];
+// Shared memory of la_chunk_out, in bytes: decays, then decayed queries | keys, then scores | queries, then values | state tile
+struct LaOutSmem {
+    int xp, kp;
+    size_t k, q, s, total;
+    __host__ __device__ explicit LaOutSmem(int dim) {
+        const size_t tile = (size_t)LA_C * LA_SP * 4;
+        xp = la_dimp(dim) + 4;
+        kp = la_pitch(dim);
+        const size_t half = (size_t)LA_C * kp * 2;
+        k = (size_t)LA_C * xp * 4;
+        q = k + (half > tile ? half : tile);
+        s = q + (half > tile ? half : tile);
+        total = s + (size_t)la_dimp(dim) * LA_VP * 4;
+    }
+};
+
+template <bool CHAN, bool VEC>
+__global__ void __launch_bounds__(LA_THREADS) la_chunk_out_kernel(const LinAttnArgs a) {
+    extern __shared__ __align__(16) float sm[];
+    const LaOutSmem lay(a.dim);
     const int c = blockIdx.x, h = blockIdx.y, r = a.chunk_req[c];
     const int row0 = a.chunk_start[c], len = min(LA_C, a.qo_indptr[r + 1] - row0);
-    const int dimp = (a.dim + 15) / 16 * 16, kp = la_pitch(a.dim), xp = dimp + 4, sp = LA_VT + 8, vp = LA_VT + 4;
-    // xp (row index by g, column by t) and sp (row by t, column by g) keep fragment reads off each other's banks
-    float* sb = sm;                                        // [64][xp] decay from the piece's start (CHAN), then decayed queries
-    float* ss = sb + LA_C * xp;                            // [dimp][sp] a tile of the state
-    float* sv = ss + dimp * sp;                            // [64][vp] a tile of values
-    bf16* sq = reinterpret_cast<bf16*>(sv + LA_C * vp);    // [64][kp]
-    bf16* sk = sq + LA_C * kp;                             // [64][kp]
+    const int dimp = la_dimp(a.dim), xp = lay.xp, kp = lay.kp;
+    uint8_t* base = reinterpret_cast<uint8_t*>(sm);
+    float* sb = sm;                                            // [64][xp]
+    bf16* sk = reinterpret_cast<bf16*>(base + lay.k);          // [64][kp]
+    float* sc = reinterpret_cast<float*>(base + lay.k);        // [64][LA_SP] scores of query rows
+    bf16* sq = reinterpret_cast<bf16*>(base + lay.q);          // [64][kp]
+    float* sv = reinterpret_cast<float*>(base + lay.q);        // [64][LA_SP] a tile of values
+    float* ss = reinterpret_cast<float*>(base + lay.s);        // [dimp][LA_VP] a tile of the state
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, g = lane >> 2, t = lane & 3;
+    const int rb = warp & 3, half = warp >> 2, w0 = rb * 16;   // 16 query rows per warp; two warps share them
     const float lh = CHAN ? 0.f : log2f(a.head_decay[h]);
-    const bf16* qb = static_cast<const bf16*>(a.q) + h * a.dim;
-    const bf16* kb = static_cast<const bf16*>(a.k) + h * a.dim;
-    for (int i = threadIdx.x; i < LA_C * dimp; i += 128) {
-        const int s = i / dimp, d = i - s * dimp;
-        bf16 q = __float2bfloat16(0.f), k = q;
-        if (s < len && d < a.dim) {
-            const size_t o = (size_t)(row0 + s) * a.ld + d;
-            q = qb[o];
-            k = kb[o];
-            if (a.silu) {
-                q = __float2bfloat16(la_silu(to_f(q)));
-                k = __float2bfloat16(la_silu(to_f(k)));
-            }
-        }
-        sq[s * kp + d] = q;
-        sk[s * kp + d] = k;
-    }
-    if (CHAN) {
-        for (int d = threadIdx.x; d < dimp; d += 128) {
-            float w = 0.f;
-            for (int s = 0; s < LA_C; ++s) {
-                if (s < len && d < a.dim) w += a.log_decay[(size_t)(row0 + s) * a.heads * a.dim + h * a.dim + d];
-                sb[s * xp + d] = w;
+    const bf16* qb = static_cast<const bf16*>(a.q) + (size_t)row0 * a.ld + h * a.dim;
+    const bf16* kb = static_cast<const bf16*>(a.k) + (size_t)row0 * a.ld + h * a.dim;
+    const bf16* vb = static_cast<const bf16*>(a.v) + (size_t)row0 * a.ld + h * a.vdim;
+    const int vecs = dimp / 8;
+    for (int u = threadIdx.x; u < LA_C * vecs; u += LA_THREADS) {
+        const int s = u / vecs, d = (u - s * vecs) * 8, valid = s < len ? min(8, a.dim - d) : 0;
+        float f[8];
+        la_load8<VEC>(qb + (size_t)s * a.ld + d, valid, a.silu, f);
+        *reinterpret_cast<bf16x8*>(sq + s * kp + d) = pack8(f);
+        la_load8<VEC>(kb + (size_t)s * a.ld + d, valid, a.silu, f);
+        *reinterpret_cast<bf16x8*>(sk + s * kp + d) = pack8(f);
+        if (CHAN) {
+            // running sums; rows past the piece repeat its last one
+            const float* b = a.log_decay + ((size_t)(row0 + min(s, len - 1)) * a.heads + h) * a.dim + d;
+            float* dst = sb + s * xp + d;
+            if (VEC && a.dim - d >= 8) {
+                reinterpret_cast<float4*>(dst)[0] = reinterpret_cast<const float4*>(b)[0];
+                reinterpret_cast<float4*>(dst)[1] = reinterpret_cast<const float4*>(b)[1];
+            } else {
+#pragma unroll
+                for (int e = 0; e < 8; ++e) dst[e] = d + e < a.dim ? b[e] : 0.f;
             }
         }
     }
+    // the first tiles of values and state are on their way while the scores are formed
+    const float* S = a.u + ((size_t)c * a.heads + h) * a.dim * a.vdim;
+    ValueTile<VEC> vt;
+    vt.load(vb, a.ld, len, a.vdim, a.silu);
     __syncthreads();
 
-    // scores of this warp's 16 queries against the keys up to the end of their own 16-token block
-    const int w0 = warp * 16;
-    float sc[8][4];
+    // scores of the 16 queries against the keys up to the end of their own 16-token block; this warp takes the 8-key tiles
+    // 2 J + half of every block J
+    float acc[4][4];
 #pragma unroll
-    for (int n = 0; n < 8; ++n) sc[n][0] = sc[n][1] = sc[n][2] = sc[n][3] = 0.f;
+    for (int n = 0; n < 4; ++n) acc[n][0] = acc[n][1] = acc[n][2] = acc[n][3] = 0.f;
     bool exact = false;
     if (CHAN) {
         float range = 0.f;
@@ -295,121 +401,141 @@ __global__ void __launch_bounds__(128) la_chunk_out_kernel(const LinAttnArgs a) 
     }
     for (int ks = 0; ks < dimp / 8; ++ks) {
         const int d0 = ks * 8 + t, d1 = d0 + 4;
-        float q4[4] = {to_f(sq[(w0 + g) * kp + d0]), to_f(sq[(w0 + g + 8) * kp + d0]), to_f(sq[(w0 + g) * kp + d1]),
-                       to_f(sq[(w0 + g + 8) * kp + d1])};
-        uint32_t fa[4];
-        float b4[4], r0 = 0.f, r1 = 0.f;
+        const float q4[4] = {to_f(sq[(w0 + g) * kp + d0]), to_f(sq[(w0 + g + 8) * kp + d0]), to_f(sq[(w0 + g) * kp + d1]),
+                             to_f(sq[(w0 + g + 8) * kp + d1])};
+        float fa[4] = {q4[0], q4[1], q4[2], q4[3]}, b4[4], r0 = 0.f, r1 = 0.f;
+        auto key = [&](int s, float& k0, float& k1) {
+            k0 = to_f(sk[s * kp + d0]);
+            k1 = to_f(sk[s * kp + d1]);
+            if (CHAN) {
+                k0 = tf32_f(k0 * exp2f(r0 - sb[s * xp + d0]));
+                k1 = tf32_f(k1 * exp2f(r1 - sb[s * xp + d1]));
+            }
+        };
+        auto queries = [&]() {
+#pragma unroll
+            for (int e = 0; e < 4; ++e) fa[e] = tf32_f(q4[e] * exp2f(b4[e] - (e < 2 ? r0 : r1)));
+        };
         if (CHAN) {
             b4[0] = sb[(w0 + g) * xp + d0]; b4[1] = sb[(w0 + g + 8) * xp + d0];
             b4[2] = sb[(w0 + g) * xp + d1]; b4[3] = sb[(w0 + g + 8) * xp + d1];
-            if (w0) { r0 = sb[(w0 - 1) * xp + d0]; r1 = sb[(w0 - 1) * xp + d1]; }
-#pragma unroll
-            for (int e = 0; e < 4; ++e) fa[e] = tf32(q4[e] * exp2f(b4[e] - (e < 2 ? r0 : r1)));
-        } else {
-#pragma unroll
-            for (int e = 0; e < 4; ++e) fa[e] = __float_as_uint(q4[e]);
+            if (rb) {
+                r0 = sb[(w0 - 1) * xp + d0];
+                r1 = sb[(w0 - 1) * xp + d1];
+                queries();
+            }
         }
 #pragma unroll
-        for (int n = 0; n < 6; ++n) {
-            if (n >= 2 * warp) break;
-            const int s = n * 8 + g;
-            float k0 = to_f(sk[s * kp + d0]), k1 = to_f(sk[s * kp + d1]);
-            if (CHAN) {
-                k0 *= exp2f(r0 - sb[s * xp + d0]);
-                k1 *= exp2f(r1 - sb[s * xp + d1]);
-            }
-            mma_tf32(sc[n], fa, tf32(k0), tf32(k1));
+        for (int J = 0; J < 3; ++J) {
+            if (J >= rb) break;
+            float k0, k1;
+            key(J * 16 + half * 8 + g, k0, k1);
+            mma_tf32(acc[J], fa, k0, k1);
         }
         if (exact) continue;
         if (CHAN) {
             r0 = sb[(w0 + 7) * xp + d0];
             r1 = sb[(w0 + 7) * xp + d1];
-#pragma unroll
-            for (int e = 0; e < 4; ++e) fa[e] = tf32(q4[e] * exp2f(b4[e] - (e < 2 ? r0 : r1)));
+            queries();
         }
-#pragma unroll
-        for (int n2 = 0; n2 < 2; ++n2) {
-            const int s = w0 + n2 * 8 + g;
-            float k0 = to_f(sk[s * kp + d0]), k1 = to_f(sk[s * kp + d1]);
-            if (CHAN) {
-                k0 *= exp2f(r0 - sb[s * xp + d0]);
-                k1 *= exp2f(r1 - sb[s * xp + d1]);
-            }
-            const uint32_t b0 = tf32(k0), b1 = tf32(k1);
-#pragma unroll
-            for (int w = 0; w < 4; ++w)
-                if (w == warp) mma_tf32(sc[2 * w + n2], fa, b0, b1);
-        }
+        float k0, k1;
+        key(w0 + half * 8 + g, k0, k1);
+        mma_tf32(acc[3], fa, k0, k1);             // the diagonal block
     }
     // decay between the two tokens (constant per head), causal limit
 #pragma unroll
-    for (int n = 0; n < 8; ++n) {
-        if (n >= 2 * warp + 2) break;
+    for (int n = 0; n < 4; ++n) {
+        const int J = n < 3 ? n : rb;
+        if (n < 3 && n >= rb) continue;
 #pragma unroll
         for (int e = 0; e < 4; ++e) {
-            const int q = w0 + g + (e >> 1) * 8, s = n * 8 + 2 * t + (e & 1);
-            if (s > q) { sc[n][e] = 0.f; continue; }
-            if (!CHAN) sc[n][e] *= exp2f((float)(q - s) * lh);
-            if (CHAN && exact && n >= 2 * warp) {
+            const int q = w0 + g + (e >> 1) * 8, s = J * 16 + half * 8 + 2 * t + (e & 1);
+            if (s > q) { acc[n][e] = 0.f; continue; }
+            if (!CHAN) acc[n][e] *= exp2f((float)(q - s) * lh);
+            if (CHAN && exact && n == 3) {
                 float x = 0.f;
                 for (int d = 0; d < dimp; ++d)
                     x += to_f(sq[q * kp + d]) * to_f(sk[s * kp + d]) * exp2f(sb[q * xp + d] - sb[s * xp + d]);
-                sc[n][e] = x;
+                acc[n][e] = x;
             }
         }
+    }
+    __syncthreads();                              // keys are done with: the scores take their place
+#pragma unroll
+    for (int n = 0; n < 4; ++n) {
+        const int J = n < 3 ? n : rb;
+        if (n < 3 && n >= rb) continue;
+#pragma unroll
+        for (int e = 0; e < 4; e += 2)
+            *reinterpret_cast<float2*>(sc + (w0 + g + (e >> 1) * 8) * LA_SP + J * 16 + half * 8 + 2 * t) =
+                make_float2(tf32_f(acc[n][e]), tf32_f(acc[n][e + 1]));
     }
     // queries with the decay from the start of the piece, for the state before it
-    __syncthreads();
-    for (int i = threadIdx.x; i < LA_C * dimp; i += 128) {
-        const int s = i / dimp, d = i - s * dimp;
-        const float q = to_f(sq[s * kp + d]);
-        sb[s * xp + d] = CHAN ? q * exp2f(sb[s * xp + d]) : q * exp2f((float)(s + 1) * lh);
+    for (int u = threadIdx.x; u < LA_C * vecs; u += LA_THREADS) {
+        const int s = u / vecs, d = (u - s * vecs) * 8;
+        float f[8];
+        unpack8(*reinterpret_cast<const bf16x8*>(sq + s * kp + d), f);
+        const float w = CHAN ? 0.f : exp2f((float)(s + 1) * lh);
+#pragma unroll
+        for (int e = 0; e < 8; ++e) sb[s * xp + d + e] = tf32_f(CHAN ? f[e] * exp2f(sb[s * xp + d + e]) : f[e] * w);
     }
-
-    const float* S = a.u + ((size_t)c * a.heads + h) * a.dim * a.vdim;
-    const bf16* vb = static_cast<const bf16*>(a.v) + h * a.vdim;
+    constexpr int SV = LA_VT / 4;                 // 16-byte pieces of a state row
     for (int v0 = 0; v0 < a.vdim; v0 += LA_VT) {
         __syncthreads();
-        for (int i = threadIdx.x; i < dimp * LA_VT; i += 128) {
-            const int d = i / LA_VT, j = i % LA_VT;
-            ss[d * sp + j] = d < a.dim && v0 + j < a.vdim ? S[(size_t)d * a.vdim + v0 + j] : 0.f;
-        }
-        for (int i = threadIdx.x; i < LA_C * LA_VT; i += 128) {
-            const int s = i / LA_VT, j = i % LA_VT;
-            float v = 0.f;
-            if (s < len && v0 + j < a.vdim) {
-                v = to_f(vb[(size_t)(row0 + s) * a.ld + v0 + j]);
-                if (a.silu) v = la_silu(v);
+        vt.template store<LA_SP>(sv);
+        for (int u = threadIdx.x; u < dimp * SV; u += LA_THREADS) {
+            const int d = u / SV, j = (u % SV) * 4;
+            float f[4] = {0.f, 0.f, 0.f, 0.f};
+            if (d < a.dim) {
+                const float* src = S + (size_t)d * a.vdim + v0 + j;
+                if (VEC && v0 + j + 3 < a.vdim) {
+                    load_vec<4>(src, f);
+                } else {
+#pragma unroll
+                    for (int e = 0; e < 4; ++e)
+                        if (v0 + j + e < a.vdim) f[e] = src[e];
+                }
             }
-            sv[s * vp + j] = v;
+#pragma unroll
+            for (int e = 0; e < 4; ++e) f[e] = tf32_f(f[e]);
+            store_vec<4>(ss + d * LA_VP + j, f);
         }
         __syncthreads();
-        float acc[LA_VT / 8][4];
+        if (v0 + LA_VT < a.vdim) vt.load(vb + v0 + LA_VT, a.ld, len, a.vdim - v0 - LA_VT, a.silu);
+        float o[4][4];
 #pragma unroll
-        for (int n = 0; n < LA_VT / 8; ++n) acc[n][0] = acc[n][1] = acc[n][2] = acc[n][3] = 0.f;
+        for (int n = 0; n < 4; ++n) o[n][0] = o[n][1] = o[n][2] = o[n][3] = 0.f;
+        const int col = half * 32 + g;            // this warp's 32 of the tile's columns
+#pragma unroll 4
         for (int ks = 0; ks < dimp / 8; ++ks) {
             const float* q0 = sb + (w0 + g) * xp + ks * 8 + t;
-            const float* q1 = q0 + 8 * xp;
-            const uint32_t fa[4] = {tf32(q0[0]), tf32(q1[0]), tf32(q0[4]), tf32(q1[4])};
-            const float* sr = ss + (ks * 8 + t) * sp + g;
+            const float fa[4] = {q0[0], q0[8 * xp], q0[4], q0[8 * xp + 4]};
+            const float* sr = ss + (ks * 8 + t) * LA_VP + col;
 #pragma unroll
-            for (int n = 0; n < LA_VT / 8; ++n) mma_tf32(acc[n], fa, tf32(sr[n * 8]), tf32(sr[4 * sp + n * 8]));
+            for (int n = 0; n < 4; ++n) mma_tf32(o[n], fa, sr[n * 8], sr[4 * LA_VP + n * 8]);
         }
-        // scores as the A operand: its columns t and t + 4 stand for the keys 2 t and 2 t + 1 that this lane holds
+        // columns t and t + 4 of the A operand stand for the keys 2 t and 2 t + 1
+        for (int ks = 0; ks < 2 * rb + 2; ++ks) {
+            const float2 x = *reinterpret_cast<const float2*>(sc + (w0 + g) * LA_SP + ks * 8 + 2 * t);
+            const float2 y = *reinterpret_cast<const float2*>(sc + (w0 + g + 8) * LA_SP + ks * 8 + 2 * t);
+            const float fa[4] = {x.x, y.x, x.y, y.y};
+            const float* vr = sv + (ks * 8 + 2 * t) * LA_SP + col;
 #pragma unroll
-        for (int ks = 0; ks < 8; ++ks) {
-            if (ks >= 2 * warp + 2) break;
-            const uint32_t fa[4] = {tf32(sc[ks][0]), tf32(sc[ks][2]), tf32(sc[ks][1]), tf32(sc[ks][3])};
-            const float* vr = sv + (ks * 8 + 2 * t) * vp + g;
-#pragma unroll
-            for (int n = 0; n < LA_VT / 8; ++n) mma_tf32(acc[n], fa, tf32(vr[n * 8]), tf32(vr[vp + n * 8]));
+            for (int n = 0; n < 4; ++n) mma_tf32(o[n], fa, vr[n * 8], vr[LA_SP + n * 8]);
         }
 #pragma unroll
-        for (int n = 0; n < LA_VT / 8; ++n)
+        for (int n = 0; n < 4; ++n)
 #pragma unroll
-            for (int e = 0; e < 4; ++e) {
-                const int q = w0 + g + (e >> 1) * 8, j = v0 + n * 8 + 2 * t + (e & 1);
-                if (q < len && j < a.vdim) a.out[(size_t)(row0 + q) * a.heads * a.vdim + h * a.vdim + j] = acc[n][e] * a.q_scale;
+            for (int e = 0; e < 4; e += 2) {
+                const int q = w0 + g + (e >> 1) * 8, j = v0 + half * 32 + n * 8 + 2 * t;
+                if (q >= len) continue;
+                float* dst = a.out + (size_t)(row0 + q) * a.heads * a.vdim + h * a.vdim + j;
+                if (VEC && j + 1 < a.vdim) {
+                    *reinterpret_cast<float2*>(dst) = make_float2(o[n][e] * a.q_scale, o[n][e + 1] * a.q_scale);
+                } else {
+                    if (j < a.vdim) dst[0] = o[n][e] * a.q_scale;
+                    if (j + 1 < a.vdim) dst[1] = o[n][e + 1] * a.q_scale;
+                }
             }
     }
 }
@@ -420,13 +546,13 @@ constexpr int LD_TOK = 8;
 template <typename T>
 __global__ void __launch_bounds__(256) la_decay_kernel(const T* __restrict__ x, int ld, const T* __restrict__ a2, const T* __restrict__ bias,
                                                        float* __restrict__ out, int n, int channels, int rank, float inv_tau) {
-    extern __shared__ float sx[];          // [LD_TOK][rank]
+    extern __shared__ __align__(16) float sx[];          // [rank][LD_TOK]
     pdl_trigger();
     pdl_wait();
     const int t0 = blockIdx.x * LD_TOK, nt = min(LD_TOK, n - t0);
     for (int i = threadIdx.x; i < LD_TOK * rank; i += 256) {
         const int s = i / rank, j = i - s * rank;
-        sx[i] = s < nt ? to_f(x[(size_t)(t0 + s) * ld + j]) : 0.f;
+        sx[j * LD_TOK + s] = s < nt ? to_f(x[(size_t)(t0 + s) * ld + j]) : 0.f;
     }
     __syncthreads();
     const int c = blockIdx.y * 256 + threadIdx.x;
@@ -436,10 +562,12 @@ __global__ void __launch_bounds__(256) la_decay_kernel(const T* __restrict__ x, 
 #pragma unroll
     for (int s = 0; s < LD_TOK; ++s) z[s] = b;
     const T* w = a2 + (size_t)c * rank;
+#pragma unroll 4
     for (int j = 0; j < rank; ++j) {
         const float wj = to_f(w[j]);
-#pragma unroll
-        for (int s = 0; s < LD_TOK; ++s) z[s] += wj * sx[s * rank + j];
+        const float4 p = reinterpret_cast<const float4*>(sx)[2 * j], q = reinterpret_cast<const float4*>(sx)[2 * j + 1];
+        z[0] += wj * p.x; z[1] += wj * p.y; z[2] += wj * p.z; z[3] += wj * p.w;
+        z[4] += wj * q.x; z[5] += wj * q.y; z[6] += wj * q.z; z[7] += wj * q.w;
     }
 #pragma unroll
     for (int s = 0; s < LD_TOK; ++s)
@@ -462,50 +590,72 @@ struct GatedNormArgs {
     int n;
 };
 
-template <typename T>
+template <typename T, int VEC>
 __global__ void __launch_bounds__(256) la_gated_norm_kernel(const GatedNormArgs args) {
-    extern __shared__ float buf[];
+    extern __shared__ __align__(16) float buf[];
     pdl_trigger();
     pdl_wait();
     const GatedNormPart& p = args.part[blockIdx.y];
     const int t = blockIdx.x;
     const T* gate = static_cast<const T*>(p.gate) + (size_t)t * p.ldg;
+    const T* w = static_cast<const T*>(p.w);
     T* dst = static_cast<T*>(p.dst) + (size_t)t * p.ldd;
-    auto source = [&](int j) {
-        const int h = j / p.head_cols;
-        const size_t at = (size_t)t * p.ldx + (size_t)(h / p.group * p.group_pad + h % p.group) * p.head_ld + (j - h * p.head_cols);
-        return p.x_f32 ? static_cast<const float*>(p.x)[at] : to_f(static_cast<const T*>(p.x)[at]);
+    auto source = [&](int j, float (&v)[VEC]) {
+        size_t at = (size_t)t * p.ldx + j;
+        if (p.head_ld != p.head_cols || p.group != p.group_pad) {
+            const int h = j / p.head_cols;
+            at = (size_t)t * p.ldx + (size_t)(h / p.group * p.group_pad + h % p.group) * p.head_ld + (j - h * p.head_cols);
+        }
+        if (p.x_f32) load_vec<VEC>(static_cast<const float*>(p.x) + at, v);
+        else load_vec<VEC>(static_cast<const T*>(p.x) + at, v);
     };
-    auto finish = [&](int j, float v) {
-        const float z = to_f(gate[j]), s = 1.f / (1.f + expf(-z));
-        dst[j] = from_f<T>(v * (p.act ? z * s : s) * p.scale);
+    auto finish = [&](int j, float (&v)[VEC], float inv, int wcol) {
+        float z[VEC], gain[VEC];
+        load_vec<VEC>(gate + j, z);
+        if (w) load_vec<VEC>(w + wcol, gain);
+#pragma unroll
+        for (int e = 0; e < VEC; ++e) {
+            const float s = 1.f / (1.f + __expf(-z[e]));
+            v[e] = v[e] * (w ? inv * gain[e] : 1.f) * (p.act ? z[e] * s : s) * p.scale;
+        }
+        store_vec<VEC>(dst + j, v);
     };
+    const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
     if (p.norm_cols == 0) {
-        for (int j = threadIdx.x; j < p.cols; j += 256) finish(j, source(j));
+        for (int j = threadIdx.x * VEC; j < p.cols; j += 256 * VEC) {
+            float v[VEC];
+            source(j, v);
+            finish(j, v, 1.f, 0);
+        }
+    } else if (p.norm_cols == p.cols) {
+        float ss = 0.f;
+        for (int j = threadIdx.x * VEC; j < p.cols; j += 256 * VEC) {
+            float v[VEC];
+            source(j, v);
+            store_vec<VEC>(buf + 32 + j, v);
+#pragma unroll
+            for (int e = 0; e < VEC; ++e) ss += v[e] * v[e];
+        }
+        const float inv = 1.f / sqrtf(block_sum(ss, buf) / (float)p.cols + p.eps);
+        for (int j = threadIdx.x * VEC; j < p.cols; j += 256 * VEC) {
+            float v[VEC];
+            load_vec<VEC>(buf + 32 + j, v);
+            finish(j, v, inv, j);
+        }
     } else {
-        const T* w = static_cast<const T*>(p.w);
-        const int groups = p.cols / p.norm_cols, lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
-        if (groups == 1) {
+        for (int gr = warp; gr < p.cols / p.norm_cols; gr += 8) {
             float ss = 0.f;
-            for (int j = threadIdx.x; j < p.cols; j += 256) {
-                const float v = source(j);
-                buf[32 + j] = v;
-                ss += v * v;
+            for (int j = lane * VEC; j < p.norm_cols; j += 32 * VEC) {
+                float v[VEC];
+                source(gr * p.norm_cols + j, v);
+#pragma unroll
+                for (int e = 0; e < VEC; ++e) ss += v[e] * v[e];
             }
-            const float inv = 1.f / sqrtf(block_sum(ss, buf) / (float)p.cols + p.eps);
-            for (int j = threadIdx.x; j < p.cols; j += 256) finish(j, buf[32 + j] * inv * to_f(w[j]));
-        } else {
-            for (int gr = warp; gr < groups; gr += 8) {
-                float ss = 0.f;
-                for (int j = lane; j < p.norm_cols; j += 32) {
-                    const float v = source(gr * p.norm_cols + j);
-                    ss += v * v;
-                }
-                const float inv = 1.f / sqrtf(warp_sum(ss) / (float)p.norm_cols + p.eps);
-                for (int j = lane; j < p.norm_cols; j += 32) {
-                    const int c = gr * p.norm_cols + j;
-                    finish(c, source(c) * inv * to_f(w[c % p.w_cols]));
-                }
+            const float inv = 1.f / sqrtf(warp_sum(ss) / (float)p.norm_cols + p.eps);
+            for (int j = lane * VEC; j < p.norm_cols; j += 32 * VEC) {
+                float v[VEC];
+                source(gr * p.norm_cols + j, v);
+                finish(gr * p.norm_cols + j, v, inv, (gr * p.norm_cols + j) % p.w_cols);
             }
         }
     }
@@ -543,14 +693,10 @@ PIE_API int pie_linear_attn_serial(const LinAttnArgs* args, int f32, cudaStream_
 #undef GO
 }
 
-static size_t la_state_smem(int dim) { return (size_t)LA_C * (la_pitch(dim) + 72) * 4; }
-static size_t la_out_smem(int dim) {
-    const int dimp = (dim + 15) / 16 * 16;
-    return ((size_t)LA_C * (dimp + 4) + (size_t)dimp * (LA_VT + 8) + (size_t)LA_C * (LA_VT + 4)) * 4 + 2ul * LA_C * la_pitch(dim) * 2;
-}
+static size_t la_state_smem(int dim) { return ((size_t)LA_C * (la_pitch(dim) + LA_VP) + 128) * 4; }
 // 1 when the chunked form takes heads of this key size.
 PIE_API int pie_linear_attn_chunk_supported(int dim) {
-    return dim > 0 && la_out_smem(dim) <= 227 * 1024 && la_state_smem(dim) <= 227 * 1024 ? 1 : 0;
+    return dim > 0 && LaOutSmem(dim).total <= 227 * 1024 && la_state_smem(dim) <= 227 * 1024 ? 1 : 0;
 }
 PIE_API int pie_linear_attn_chunk_tokens() { return LA_C; }
 
@@ -559,17 +705,24 @@ PIE_API int pie_linear_attn_chunked(const LinAttnArgs* args, cudaStream_t st) {
     if (a.n <= 0 || a.reqs <= 0 || a.chunks <= 0) return 0;
     if (!pie_linear_attn_chunk_supported(a.dim) || a.vdim <= 0 || (!a.log_decay && !a.head_decay) || !a.u || !a.piece_decay)
         return (int)cudaErrorInvalidValue;
+    auto aligned = [](const void* p) { return ((uintptr_t)p & 15) == 0; };
+    const bool vec = a.dim % 8 == 0 && a.vdim % 8 == 0 && a.ld % 8 == 0 && aligned(a.q) && aligned(a.k) && aligned(a.v) && aligned(a.log_decay) &&
+                     aligned(a.u) && aligned(a.out) && aligned(a.state) && a.slot_stride % 4 == 0;
     const dim3 grid(a.chunks, a.heads);
-    const size_t s1 = la_state_smem(a.dim), s3 = la_out_smem(a.dim);
-    auto k1 = a.log_decay ? la_chunk_state_kernel<true> : la_chunk_state_kernel<false>;
-    auto k3 = a.log_decay ? la_chunk_out_kernel<true> : la_chunk_out_kernel<false>;
+    const size_t s1 = la_state_smem(a.dim), s3 = LaOutSmem(a.dim).total;
+    auto k1 = a.log_decay ? (vec ? la_chunk_state_kernel<true, true> : la_chunk_state_kernel<true, false>)
+                          : (vec ? la_chunk_state_kernel<false, true> : la_chunk_state_kernel<false, false>);
+    auto k3 = a.log_decay ? (vec ? la_chunk_out_kernel<true, true> : la_chunk_out_kernel<true, false>)
+                          : (vec ? la_chunk_out_kernel<false, true> : la_chunk_out_kernel<false, false>);
     cudaError_t e = cudaFuncSetAttribute(k1, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)s1);
     if (e == cudaSuccess) e = cudaFuncSetAttribute(k3, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)s3);
     if (e != cudaSuccess) return (int)e;
-    k1<<<grid, 128, s1, st>>>(a);
-    const long elems = (long)a.heads * a.dim * a.vdim;
-    la_chunk_scan_kernel<<<dim3((unsigned)((elems + 255) / 256), a.reqs), 256, 0, st>>>(a);
-    k3<<<grid, 128, s3, st>>>(a);
+    k1<<<grid, LA_THREADS, s1, st>>>(a);
+    const long elems = (long)a.heads * a.dim * a.vdim / (vec ? 4 : 1);
+    const dim3 sgrid((unsigned)((elems + 255) / 256), a.reqs);
+    if (vec) la_chunk_scan_kernel<4><<<sgrid, 256, 0, st>>>(a);
+    else la_chunk_scan_kernel<1><<<sgrid, 256, 0, st>>>(a);
+    k3<<<grid, LA_THREADS, s3, st>>>(a);
     return (int)cudaGetLastError();
 }
 
@@ -592,15 +745,20 @@ PIE_API int pie_gated_norm(const GatedNormArgs* args, int parts, int f32, cudaSt
     if (a.n <= 0) return 0;
     if (parts < 1 || parts > 2) return (int)cudaErrorInvalidValue;
     size_t sm = 0;
+    bool vec = true;
+    auto aligned = [](const void* p) { return ((uintptr_t)p & 15) == 0; };
     for (int i = 0; i < parts; ++i) {
         const GatedNormPart& p = a.part[i];
         if (p.head_cols <= 0 || p.group <= 0 || p.cols <= 0 || (p.norm_cols && (p.cols % p.norm_cols || !p.w || p.w_cols <= 0)))
             return (int)cudaErrorInvalidValue;
         if (p.norm_cols == p.cols) sm = (size_t)(32 + p.cols) * 4 > sm ? (size_t)(32 + p.cols) * 4 : sm;
+        vec = vec && p.head_cols % 4 == 0 && p.head_ld % 4 == 0 && p.norm_cols % 4 == 0 && (!p.w || p.w_cols % 4 == 0) &&
+              p.cols % 4 == 0 && p.ldx % 4 == 0 && p.ldg % 4 == 0 && p.ldd % 4 == 0 && aligned(p.x) && aligned(p.gate) && aligned(p.dst) && aligned(p.w);
     }
     if (sm > 227 * 1024) return (int)cudaErrorInvalidValue;
     const dim3 grid(a.n, parts);
-    auto kern = f32 ? la_gated_norm_kernel<float> : la_gated_norm_kernel<bf16>;
+    auto kern = f32 ? (vec ? la_gated_norm_kernel<float, 4> : la_gated_norm_kernel<float, 1>)
+                    : (vec ? la_gated_norm_kernel<bf16, 4> : la_gated_norm_kernel<bf16, 1>);
     if (sm > 48 * 1024) {
         const cudaError_t e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)sm);
         if (e != cudaSuccess) return (int)e;

@@ -74,7 +74,7 @@ def test_linear_attention_in_portions(path, h, d, e, kind):
     q, k, v, logs = channel_case(n, h, d, e, dt, strength)
     decay = torch.tensor([1.0, 0.97, 0.4][:h] + [0.9] * max(0, h - 3))
     silu = kind == "head"
-    act = (lambda x: (oracle.silu(x).to(dt).float() if dt == BF16 else oracle.silu(x))) if silu else (lambda x: x)
+    act = oracle.silu if silu else (lambda x: x)
     a = decay[None, :, None].expand(n, h, d) if silu else logs.view(n, h, d).exp()
     states = []
     ref = plain(act(q) * d ** -0.5, act(k), act(v), a, h, states)
@@ -90,8 +90,9 @@ def test_linear_attention_in_portions(path, h, d, e, kind):
         out.append(lin.linear_attention(qq, kk, vv, spec, rs, state, size == 1, None if silu else base[at:at + size].to(dev).contiguous(),
                                         decay.to(dev) if silu else None, silu, d ** -0.5).cpu())
         at += size
-    close(torch.cat(out), ref[:at], dt, bf16=4e-3)
-    close(state[1].cpu().view(h, d, e), states[at - 1], dt, bf16=4e-3)
+    limit = 8e-3 if silu else 4e-3                # the activations of a prompt's queries and keys may be rounded
+    close(torch.cat(out), ref[:at], dt, bf16=limit)
+    close(state[1].cpu().view(h, d, e), states[at - 1], dt, bf16=limit)
     assert not state[0].isfinite().any() and not state[2].isfinite().any()
 
 
