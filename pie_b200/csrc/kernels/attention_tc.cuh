@@ -85,6 +85,25 @@ __device__ __forceinline__ float fast_exp2(float x) {
     return y;
 }
 
+// Two 32-bit numbers in one register pair: the packed arithmetic of sm_100.
+typedef unsigned long long F2;
+__device__ __forceinline__ F2 f2(float lo, float hi) {
+    F2 d;
+    asm("mov.b64 %0, {%1, %2};" : "=l"(d) : "f"(lo), "f"(hi));
+    return d;
+}
+__device__ __forceinline__ F2 f2(float x) { return f2(x, x); }
+__device__ __forceinline__ void unpack2(F2 v, float& lo, float& hi) { asm("mov.b64 {%0, %1}, %2;" : "=f"(lo), "=f"(hi) : "l"(v)); }
+__device__ __forceinline__ F2 mul2(F2 a, F2 b) {
+    F2 d;
+    asm("mul.rn.f32x2 %0, %1, %2;" : "=l"(d) : "l"(a), "l"(b));
+    return d;
+}
+__device__ __forceinline__ F2 fma2(F2 a, F2 b, F2 c) {
+    F2 d;
+    asm("fma.rn.f32x2 %0, %1, %2, %3;" : "=l"(d) : "l"(a), "l"(b), "l"(c));
+    return d;
+}
 __device__ __forceinline__ float fast_tanh(float x) {
     float y;
     asm("tanh.approx.f32 %0, %1;" : "=f"(y) : "f"(x));
@@ -351,28 +370,27 @@ paged_prefill_attn_tc_kernel(const __grid_constant__ CUtensorMap tma_q, const __
             }
             const int kb0 = (jb + j) * AT_BK;
             if (BIAS) {
-                float big = 0.f;
-#pragma unroll
-                for (int i = 0; i < AT_BK; ++i) {
-                    sv[i] *= cap_pre;
-                    big = fmaxf(big, fabsf(sv[i]));
-                }
-                if (__all_sync(0xffffffffu, big <= 0.35f)) {       // odd Taylor polynomial of tanh: below 2^-23 up to 0.35
-#pragma unroll
-                    for (int i = 0; i < AT_BK; ++i) {
-                        const float x2 = sv[i] * sv[i];
-                        const float p = fmaf(x2, fmaf(x2, fmaf(x2, fmaf(x2, 62.f / 2835.f, -17.f / 315.f), 2.f / 15.f), -1.f / 3.f), 1.f);
-                        sv[i] *= p;
-                    }
-                } else {
-#pragma unroll
-                    for (int i = 0; i < AT_BK; ++i) sv[i] = 1.f - __fdividef(2.f, 1.f + fast_exp2(2.8853900817779268f * sv[i]));
-                }
                 // distance of key i of the block: n - i (keys after the query, which only a custom mask shows, read the guard)
                 const int n = kb0 < lim && kb0 + AT_BK > lo ? max(kv_len - qo_len + qtok - kb0, -1) : 0;
                 const float* tb = table + (row % G) * bias_pitch + AT_BIAS_GUARD + n;
+                float big = 0.f;
 #pragma unroll
-                for (int i = 0; i < AT_BK; ++i) sv[i] = fmaf(cap_post, sv[i], tb[-i]);
+                for (int i = 0; i < AT_BK; i += 2) big = fmaxf(big, fmaxf(fabsf(sv[i]), fabsf(sv[i + 1])));
+                if (__all_sync(0xffffffffu, big * cap_pre <= 0.35f)) {
+                    // odd Taylor polynomial of tanh, below 2^-23 up to 0.35, two scores at a time
+                    const F2 pre = f2(cap_pre), c0 = f2(cap_post), c1 = f2(cap_post * (-1.f / 3.f)), c2 = f2(cap_post * (2.f / 15.f)),
+                             c3 = f2(cap_post * (-17.f / 315.f)), c4 = f2(cap_post * (62.f / 2835.f));
+#pragma unroll
+                    for (int i = 0; i < AT_BK; i += 2) {
+                        const F2 x = mul2(f2(sv[i], sv[i + 1]), pre), y = mul2(x, x);
+                        const F2 p = fma2(y, fma2(y, fma2(y, fma2(y, c4, c3), c2), c1), c0);
+                        unpack2(fma2(x, p, f2(tb[-i], tb[-i - 1])), sv[i], sv[i + 1]);
+                    }
+                } else {
+#pragma unroll
+                    for (int i = 0; i < AT_BK; ++i)
+                        sv[i] = fmaf(cap_post, 1.f - __fdividef(2.f, 1.f + fast_exp2(2.8853900817779268f * cap_pre * sv[i])), tb[-i]);
+                }
             }
             const bool inner = !custom && kb0 + AT_BK <= lim && kb0 >= lo;
             if (!__all_sync(0xffffffffu, inner)) {
