@@ -753,7 +753,8 @@ PIE_API int pie_gated_norm(const GatedNormArgs* args, int parts, int f32, cudaSt
             return (int)cudaErrorInvalidValue;
         if (p.norm_cols == p.cols) sm = (size_t)(32 + p.cols) * 4 > sm ? (size_t)(32 + p.cols) * 4 : sm;
         vec = vec && p.head_cols % 4 == 0 && p.head_ld % 4 == 0 && p.norm_cols % 4 == 0 && (!p.w || p.w_cols % 4 == 0) &&
-              p.cols % 4 == 0 && p.ldx % 4 == 0 && p.ldg % 4 == 0 && p.ldd % 4 == 0 && aligned(p.x) && aligned(p.gate) && aligned(p.dst) && aligned(p.w);
+              p.cols % 4 == 0 && p.ldx % 4 == 0 && p.ldg % 4 == 0 && p.ldd % 4 == 0 && aligned(p.x) && aligned(p.gate) &&
+              aligned(p.dst) && aligned(p.w);
     }
     if (sm > 227 * 1024) return (int)cudaErrorInvalidValue;
     const dim3 grid(a.n, parts);

@@ -165,9 +165,6 @@ def test_gated_norms(path, heads, kv, vdim, cols):
 
 
 # ------------------------------------------------------------------ attention with a distance bias
-def pages_of(n, page, order):
-    return order[:-(-n // page)]
-
 
 def attention_case(spec, kv_lens, qlens, page, dev, dt, seed=0, stand_out=True):
     """Normed rows in pages, with one far and one near key per sequence that a query matches strongly."""
