@@ -214,12 +214,10 @@ paged_prefill_attn_tc_kernel(const __grid_constant__ CUtensorMap tma_q, const __
         tmem_alloc(smem_addr(const_cast<uint32_t*>(tmem_slot)), AtCfg<NT, D>::TMEM_COLS);
         tmem_relinquish();
     }
-    const float* table = BIAS ? bias + (size_t)h * G * bias_pitch : nullptr;
     if (BIAS && bias_smem) {
         float4* dst = reinterpret_cast<float4*>(base_ptr + Cfg::TABLE);
-        const float4* src = reinterpret_cast<const float4*>(table);
+        const float4* src = reinterpret_cast<const float4*>(bias + (size_t)h * G * bias_pitch);
         for (int i = threadIdx.x; i < G * bias_pitch / 4; i += Cfg::THREADS) dst[i] = src[i];
-        table = reinterpret_cast<const float*>(dst);
     }
     tc_fence_before();
     __syncthreads();
@@ -372,25 +370,31 @@ paged_prefill_attn_tc_kernel(const __grid_constant__ CUtensorMap tma_q, const __
             if (BIAS) {
                 // distance of key i of the block: n - i (keys after the query, which only a custom mask shows, read the guard)
                 const int n = kb0 < lim && kb0 + AT_BK > lo ? max(kv_len - qo_len + qtok - kb0, -1) : 0;
-                const float* tb = table + (row % G) * bias_pitch + AT_BIAS_GUARD + n;
+                const int at = (row % G) * bias_pitch + AT_BIAS_GUARD + n;
                 float big = 0.f;
 #pragma unroll
                 for (int i = 0; i < AT_BK; i += 2) big = fmaxf(big, fmaxf(fabsf(sv[i]), fabsf(sv[i + 1])));
-                if (__all_sync(0xffffffffu, big * cap_pre <= 0.35f)) {
-                    // odd Taylor polynomial of tanh, below 2^-23 up to 0.35, two scores at a time
-                    const F2 pre = f2(cap_pre), c0 = f2(cap_post), c1 = f2(cap_post * (-1.f / 3.f)), c2 = f2(cap_post * (2.f / 15.f)),
-                             c3 = f2(cap_post * (-17.f / 315.f)), c4 = f2(cap_post * (62.f / 2835.f));
+                const bool small = __all_sync(0xffffffffu, big * cap_pre <= 0.35f);
+                auto add_bias = [&](const float* tb) {
+                    if (small) {
+                        // odd Taylor polynomial of tanh, below 2^-23 up to 0.35, two scores at a time
+                        const F2 pre = f2(cap_pre), c0 = f2(cap_post), c1 = f2(cap_post * (-1.f / 3.f)), c2 = f2(cap_post * (2.f / 15.f)),
+                                 c3 = f2(cap_post * (-17.f / 315.f)), c4 = f2(cap_post * (62.f / 2835.f));
 #pragma unroll
-                    for (int i = 0; i < AT_BK; i += 2) {
-                        const F2 x = mul2(f2(sv[i], sv[i + 1]), pre), y = mul2(x, x);
-                        const F2 p = fma2(y, fma2(y, fma2(y, fma2(y, c4, c3), c2), c1), c0);
-                        unpack2(fma2(x, p, f2(tb[-i], tb[-i - 1])), sv[i], sv[i + 1]);
+                        for (int i = 0; i < AT_BK; i += 2) {
+                            const F2 x = mul2(f2(sv[i], sv[i + 1]), pre), y = mul2(x, x);
+                            const F2 p = fma2(y, fma2(y, fma2(y, fma2(y, c4, c3), c2), c1), c0);
+                            unpack2(fma2(x, p, f2(tb[-i], tb[-i - 1])), sv[i], sv[i + 1]);
+                        }
+                    } else {
+#pragma unroll
+                        for (int i = 0; i < AT_BK; ++i)
+                            sv[i] = fmaf(cap_post, 1.f - __fdividef(2.f, 1.f + fast_exp2(2.8853900817779268f * cap_pre * sv[i])), tb[-i]);
                     }
-                } else {
-#pragma unroll
-                    for (int i = 0; i < AT_BK; ++i)
-                        sv[i] = fmaf(cap_post, 1.f - __fdividef(2.f, 1.f + fast_exp2(2.8853900817779268f * cap_pre * sv[i])), tb[-i]);
-                }
+                };
+                // one copy per memory the table may lie in, so that each is read with that memory's loads
+                if (bias_smem) add_bias(reinterpret_cast<const float*>(base_ptr + Cfg::TABLE) + at);
+                else add_bias(bias + (size_t)h * G * bias_pitch + at);
             }
             const bool inner = !custom && kb0 + AT_BK <= lim && kb0 >= lo;
             if (!__all_sync(0xffffffffu, inner)) {

@@ -189,7 +189,7 @@ struct ValueTile {
 
 // U and the piece's decay; turns log_decay into its running sum from the piece's start (in place), which la_chunk_out reads.
 template <bool CHAN, bool VEC>
-__global__ void __launch_bounds__(LA_THREADS) la_chunk_state_kernel(const LinAttnArgs a) {
+__global__ void __launch_bounds__(LA_THREADS, 3) la_chunk_state_kernel(const LinAttnArgs a) {
     extern __shared__ __align__(16) float sm[];
     const int c = blockIdx.x, h = blockIdx.y, r = a.chunk_req[c];
     const int row0 = a.chunk_start[c], len = min(LA_C, a.qo_indptr[r + 1] - row0);
@@ -210,13 +210,10 @@ __global__ void __launch_bounds__(LA_THREADS) la_chunk_state_kernel(const LinAtt
             const bool ok = d < a.dim;
             float* lg = a.log_decay + ((size_t)(row0 + half * 32) * a.heads + h) * a.dim + d;
             const size_t step = (size_t)a.heads * a.dim;
-            float b[32], k[32], run = 0.f;
+            const bf16* kd = kb + (size_t)half * 32 * a.ld + d;
+            float b[32], run = 0.f;
 #pragma unroll
-            for (int s = 0; s < 32; ++s) {
-                const bool in = ok && half * 32 + s < len;
-                b[s] = in ? lg[s * step] : 0.f;
-                k[s] = in ? to_f(kb[(size_t)(half * 32 + s) * a.ld + d]) : 0.f;
-            }
+            for (int s = 0; s < 32; ++s) b[s] = ok && half * 32 + s < len ? lg[s * step] : 0.f;
 #pragma unroll
             for (int s = 0; s < 32; ++s) b[s] = run += b[s];
             if (half == 0) tot[threadIdx.x] = run;
@@ -229,12 +226,16 @@ __global__ void __launch_bounds__(LA_THREADS) la_chunk_state_kernel(const LinAtt
             if (half && ok) dec[d] = all;
             if (d < dimp) {
 #pragma unroll
-                for (int s = 0; s < 32; ++s) {
-                    const float x = base + b[s];
-                    if (ok && half * 32 + s < len) lg[s * step] = x;
-                    float kv = k[s];
-                    if (a.silu) kv = la_silu(kv);
-                    sk[(half * 32 + s) * kp + d] = tf32_f(kv * exp2f(all - x));
+                for (int s0 = 0; s0 < 32; s0 += 16) {
+                    float k[16];
+#pragma unroll
+                    for (int s = 0; s < 16; ++s) k[s] = ok && half * 32 + s0 + s < len ? to_f(kd[(size_t)(s0 + s) * a.ld]) : 0.f;
+#pragma unroll
+                    for (int s = 0; s < 16; ++s) {
+                        const float x = base + b[s0 + s];
+                        if (ok && half * 32 + s0 + s < len) lg[(s0 + s) * step] = x;
+                        sk[(half * 32 + s0 + s) * kp + d] = tf32_f((a.silu ? la_silu(k[s]) : k[s]) * exp2f(all - x));
+                    }
                 }
             }
             __syncthreads();               // `tot` is free for the next channels
