@@ -189,7 +189,7 @@ struct ValueTile {
 
 // U and the piece's decay; turns log_decay into its running sum from the piece's start (in place), which la_chunk_out reads.
 template <bool CHAN, bool VEC>
-__global__ void __launch_bounds__(LA_THREADS, 3) la_chunk_state_kernel(const LinAttnArgs a) {
+__global__ void __launch_bounds__(LA_THREADS, CHAN ? 2 : 3) la_chunk_state_kernel(const LinAttnArgs a) {
     extern __shared__ __align__(16) float sm[];
     const int c = blockIdx.x, h = blockIdx.y, r = a.chunk_req[c];
     const int row0 = a.chunk_start[c], len = min(LA_C, a.qo_indptr[r + 1] - row0);

@@ -315,6 +315,30 @@ def test_greedy_generation_through_the_engine(path):
         e.shutdown()
 
 
+@pytest.mark.gpu
+def test_memory_is_planned_beside_the_states():
+    """Pages, passes and state slots from what the device has left; the model then runs."""
+    cfg = preset("tiny-retodra")
+    drv = TorchDriver(cfg, "cuda", num_pages=0, max_requests=8, max_tokens=512, gpu_mem_utilization=0.3)
+    assert drv.rs.num_slots == 16 and drv.kv.num_pages >= 64 and drv.memory_plan.arena_bytes > 0
+    rp, toks = Replay(drv), list(range(1, 130))
+    a = run_cuts(rp, "a", toks, [])
+    assert error(run_cuts(rp, "b", toks, [60, 100, 128]), a).max() < 0.03
+
+
+def test_bytes_of_pages_and_slots():
+    from pie_b200.driver import memory_planner as mp
+    from pie_b200.driver.recurrent import RecurrentStateCache
+    cfg = ModelConfig.from_hf(rm.CONFIGS["mixed"])
+    assert mp.kv_bytes_per_page(cfg, 16) == 2 * 16 * 2 * (2 * 64 + 4 * 64)
+    rs = RecurrentStateCache(cfg, 3, "cpu")
+    assert rs.bytes_per_slot == 4 * (3 * 24 * 40 + 2 * 16 * 24 + 2 * 48 * 24 + 5 * 24 * 8)
+    rs.linear_state[1] = torch.arange(rs.linear_state.shape[1])
+    rs.copy_slot(1, 2)
+    assert torch.equal(rs.linear_state[1], rs.linear_state[2]) and not rs.linear_state[0].any()
+    assert mp.arena_bytes(cfg, 1024, 8) > 1024 * 96 * 16
+
+
 def test_swap_copies_pages_of_unequal_layers():
     from pie_b200.driver.kv_cache import KVCache
     from pie_b200.driver.schema import CopyDir, CopyRequest
