@@ -37,9 +37,11 @@ static int launch_decode(const void* q, const void* kv_layer, const int* page_in
                          void* out, float* scratch, int max_items, int num_reqs, int hq, int hkv,
                          int head_dim, int page_size, float sm_scale, int num_ctas, int run_merge,
                          int window_left, const float* sinks_log2, const int* item_slot,
-                         const int* item_tile, const int* tile_members, cudaStream_t st, float softcap = 0.f) {
+                         const int* item_tile, const int* tile_members, cudaStream_t st, float softcap = 0.f,
+                         int keep_first = 0) {
     if (num_reqs <= 0) return 0;
     if (hkv <= 0 || hq % hkv || page_size % 16) return (int)cudaErrorInvalidValue;
+    if (keep_first < 0) return (int)cudaErrorInvalidValue;
     const bool cascade = item_tile != nullptr;
     if (cascade && (!item_slot || !tile_members || window_left >= 0 || softcap > 0.f)) return (int)cudaErrorInvalidValue;
     const int group = hq / hkv;
@@ -56,7 +58,7 @@ static int launch_decode(const void* q, const void* kv_layer, const int* page_in
                 (const bf16*)q, (const bf16*)kv_layer, page_indices, kv_page_indptr, item_req,
                 item_start, item_end, req_item_indptr, num_items_ptr, (bf16*)out, o_part, lse_part, hq,
                 hkv, page_size, scale_log2, window_left, sinks_log2, max_items, num_reqs, pie_status_word_current(),
-                (const int*)nullptr, (const int*)nullptr, (const int*)nullptr, cap_log2, (const float*)nullptr, 0);
+                (const int*)nullptr, (const int*)nullptr, (const int*)nullptr, cap_log2, (const float*)nullptr, 0, keep_first);
         } else if (cascade) {
             auto kern = paged_decode_attn_kernel<D, G, true>;
             cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, SM);
@@ -64,7 +66,7 @@ static int launch_decode(const void* q, const void* kv_layer, const int* page_in
                 (const bf16*)q, (const bf16*)kv_layer, page_indices, kv_page_indptr, item_req,
                 item_start, item_end, req_item_indptr, num_items_ptr, (bf16*)out, o_part, lse_part, hq,
                 hkv, page_size, scale_log2, window_left, sinks_log2, max_items, num_reqs, pie_status_word_current(),
-                item_slot, item_tile, tile_members, 0.f, (const float*)nullptr, 0);
+                item_slot, item_tile, tile_members, 0.f, (const float*)nullptr, 0, 0);
         } else {
             auto kern = paged_decode_attn_kernel<D, G, false>;
             cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, SM);
@@ -72,7 +74,7 @@ static int launch_decode(const void* q, const void* kv_layer, const int* page_in
                 (const bf16*)q, (const bf16*)kv_layer, page_indices, kv_page_indptr, item_req,
                 item_start, item_end, req_item_indptr, num_items_ptr, (bf16*)out, o_part, lse_part, hq,
                 hkv, page_size, scale_log2, window_left, sinks_log2, max_items, num_reqs, pie_status_word_current(),
-                (const int*)nullptr, (const int*)nullptr, (const int*)nullptr, 0.f, (const float*)nullptr, 0);
+                (const int*)nullptr, (const int*)nullptr, (const int*)nullptr, 0.f, (const float*)nullptr, 0, keep_first);
         }
     });
     int err = (int)cudaGetLastError();
@@ -120,6 +122,20 @@ PIE_API int pie_paged_decode_attn_softcap(const void* q, const void* kv_layer, c
                          num_ctas, run_merge, window_left, sinks_log2, nullptr, nullptr, nullptr, st, softcap);
 }
 
+// The window form with the first `keep_first` keys visible beside the window; the items must cover them.
+PIE_API int pie_paged_decode_attn_kept(const void* q, const void* kv_layer, const int* page_indices,
+                                       const int* kv_page_indptr, const int* item_req,
+                                       const int* item_start, const int* item_end,
+                                       const int* req_item_indptr, const int* num_items_ptr,
+                                       void* out, float* scratch, int max_items, int num_reqs, int hq,
+                                       int hkv, int head_dim, int page_size, float sm_scale,
+                                       int num_ctas, int window_left, int keep_first,
+                                       const float* sinks_log2, cudaStream_t st) {
+    return launch_decode(q, kv_layer, page_indices, kv_page_indptr, item_req, item_start, item_end, req_item_indptr,
+                         num_items_ptr, out, scratch, max_items, num_reqs, hq, hkv, head_dim, page_size, sm_scale,
+                         num_ctas, 1, window_left, sinks_log2, nullptr, nullptr, nullptr, st, 0.f, keep_first);
+}
+
 // Decode attention over a plan with shared-prefix items (see the kernel): requests that were forked
 // from one context read their common pages once. item_req of a shared item names the member whose
 // page table addresses the range. req_item_indptr counts partial-result slots, all below max_items.
@@ -149,6 +165,10 @@ PIE_API int pie_paged_decode_attn(const void* q, const void* kv_layer, const int
                                         head_dim, page_size, sm_scale, num_ctas, run_merge, -1, nullptr, st);
 }
 
+PIE_API int pie_paged_prefill_attn_kept(const void*, const void*, const int*, const int*, const int*, const int*, const int*, const int*, int,
+                                        const uint32_t*, const long*, void*, float*, int, int, int, int, float, int, const float*, float,
+                                        int, cudaStream_t);
+
 // softcap > 0: softmax over softcap * tanh(q.k * sm_scale / softcap) (Gemma-2).
 PIE_API int pie_paged_prefill_attn_softcap(const void* q, const void* kv_layer, const int* page_indices,
                                            const int* kv_page_indptr, const int* qo_indptr,
@@ -158,7 +178,22 @@ PIE_API int pie_paged_prefill_attn_softcap(const void* q, const void* kv_layer, 
                                            int hkv, int head_dim, int page_size, float sm_scale,
                                            int window_left, const float* sinks_log2, float softcap,
                                            cudaStream_t st) {
+    return pie_paged_prefill_attn_kept(q, kv_layer, page_indices, kv_page_indptr, qo_indptr, kv_lens, tile_req, tile_qstart,
+                                       num_tiles, mask_bits, mask_word_indptr, out, lse_out, hq, hkv, head_dim, page_size,
+                                       sm_scale, window_left, sinks_log2, softcap, 0, st);
+}
+
+// The same with the first `keep_first` keys visible beside the window.
+PIE_API int pie_paged_prefill_attn_kept(const void* q, const void* kv_layer, const int* page_indices,
+                                        const int* kv_page_indptr, const int* qo_indptr,
+                                        const int* kv_lens, const int* tile_req, const int* tile_qstart,
+                                        int num_tiles, const uint32_t* mask_bits,
+                                        const long* mask_word_indptr, void* out, float* lse_out, int hq,
+                                        int hkv, int head_dim, int page_size, float sm_scale,
+                                        int window_left, const float* sinks_log2, float softcap, int keep_first,
+                                        cudaStream_t st) {
     if (num_tiles <= 0) return 0;
+    if (keep_first < 0) return (int)cudaErrorInvalidValue;
     if (hkv <= 0 || hq % hkv || page_size % 16) return (int)cudaErrorInvalidValue;
     const int group = hq / hkv;
     const float scale_log2 = softcap > 0.f ? sm_scale / softcap : sm_scale * 1.4426950408889634f;
@@ -172,14 +207,14 @@ PIE_API int pie_paged_prefill_attn_softcap(const void* q, const void* kv_layer, 
             kern<<<grid, PF_WARPS * 32, SM, st>>>(
                 (const bf16*)q, (const bf16*)kv_layer, page_indices, kv_page_indptr, qo_indptr, kv_lens,
                 tile_req, tile_qstart, mask_bits, mask_word_indptr, (bf16*)out, lse_out, sinks_log2, hq, hkv,
-                page_size, scale_log2, window_left, cap_log2, nullptr, 0);
+                page_size, scale_log2, window_left, cap_log2, nullptr, 0, keep_first);
         } else {
             auto kern = paged_prefill_attn_kernel<D, G>;
             cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, SM);
             kern<<<grid, PF_WARPS * 32, SM, st>>>(
                 (const bf16*)q, (const bf16*)kv_layer, page_indices, kv_page_indptr, qo_indptr, kv_lens,
                 tile_req, tile_qstart, mask_bits, mask_word_indptr, (bf16*)out, lse_out, sinks_log2, hq, hkv,
-                page_size, scale_log2, window_left, 0.f, nullptr, 0);
+                page_size, scale_log2, window_left, 0.f, nullptr, 0, keep_first);
         }
     });
     return (int)cudaGetLastError();

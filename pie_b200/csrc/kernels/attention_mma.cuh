@@ -7,6 +7,8 @@
 //    by a second kernel when a request has more than one item.
 //  * paged_prefill_attn: ragged query lengths, causal or custom bit-mask,
 //    optional sliding window, 64-row tiles of (query token, head-in-group).
+//  Beside a sliding window the first `keep_first` keys stay visible; 16-key (prefill: 64-key) blocks without a visible key
+//  are skipped.
 //
 // KV layer layout: [pages][2][Hkv][page_size][D] bf16 (K then V per page), so a
 // (page, head) K or V block is one contiguous page_size*D*2-byte run.
@@ -228,7 +230,7 @@ paged_decode_attn_kernel(const bf16* __restrict__ q, const bf16* __restrict__ kv
                          const float* __restrict__ sinks_log2, int max_items, int num_reqs,
                          int* __restrict__ status, const int* __restrict__ item_slot,
                          const int* __restrict__ item_tile, const int* __restrict__ tile_members,
-                         float cap_log2, const float* __restrict__ bias = nullptr, int bias_pitch = 0) {
+                         float cap_log2, const float* __restrict__ bias, int bias_pitch, int keep_first) {
     static_assert(G <= 16, "at most 16 query heads per KV head");
     constexpr int ROWS = CASCADE ? (16 / G) * G : G;      // rows of the Q tile in use
     extern __shared__ __align__(1024) uint8_t smem[];
@@ -286,12 +288,16 @@ paged_decode_attn_kernel(const bf16* __restrict__ q, const bf16* __restrict__ kv
 
         AttnState<D> st;
         st.init();
-        const int nb_total = (kv_end - kv_start + 15) >> 4;
+        // blocks [hidden, hidden + gap) of the item lie between the kept first keys and the window
+        const int nb_item = (kv_end - kv_start + 15) >> 4;
+        const int hidden = min(nb_item, max(0, (keep_first - kv_start + 15) >> 4));
+        const int gap = max(0, min(nb_item, (kv_lo - kv_start) >> 4) - hidden), nb_total = nb_item - gap;
+        auto block_start = [&](int b) { return kv_start + (b < hidden ? b : b + gap) * 16; };
         const int my_count = nb_total > warp ? (nb_total - warp + DEC_WARPS - 1) / DEC_WARPS : 0;
         const int* pages = page_indices + kv_page_indptr[req];
 
         auto issue = [&](int j) {
-            const int tok0 = kv_start + (warp + DEC_WARPS * j) * 16;
+            const int tok0 = block_start(warp + DEC_WARPS * j);
             const int page = pages[tok0 / page_size];
             const int off = tok0 % page_size;
             const bf16* ksrc = kv_layer + ((((size_t)page * 2) * hkv + h) * page_size + off) * D;
@@ -316,10 +322,14 @@ paged_decode_attn_kernel(const bf16* __restrict__ q, const bf16* __restrict__ kv
             cp_async_commit();
             cp_async_wait<DEC_STAGES - 1>();
             __syncwarp();
-            const int tok0 = kv_start + (warp + DEC_WARPS * i) * 16;
+            const int tok0 = block_start(warp + DEC_WARPS * i);
             const int nvalid = kv_end - tok0;
             uint32_t allow = nvalid >= 16 ? 0xffffu : ((1u << nvalid) - 1u);
-            if (kv_lo > tok0) allow &= kv_lo - tok0 >= 16 ? 0u : ~((1u << (kv_lo - tok0)) - 1u);
+            if (kv_lo > tok0) {
+                uint32_t see = kv_lo - tok0 >= 16 ? 0u : ~((1u << (kv_lo - tok0)) - 1u);
+                if (keep_first > tok0) see |= keep_first - tok0 >= 16 ? 0xffffu : (1u << (keep_first - tok0)) - 1u;
+                allow &= see;
+            }
             const uint32_t kt = warp_smem + (i % DEC_STAGES) * 2 * TILE_BYTES;
             DistanceBias db{};
             if (MODE == MODE_BIAS) {
@@ -459,8 +469,8 @@ paged_prefill_attn_kernel(const bf16* __restrict__ q, const bf16* __restrict__ k
                           const uint32_t* __restrict__ mask_bits,
                           const long* __restrict__ mask_word_indptr, bf16* __restrict__ out,
                           float* __restrict__ lse_out, const float* __restrict__ sinks_log2, int hq, int hkv, int page_size,
-                          float scale_log2, int window_left, float cap_log2, const float* __restrict__ bias = nullptr,
-                          int bias_pitch = 0) {
+                          float scale_log2, int window_left, float cap_log2, const float* __restrict__ bias,
+                          int bias_pitch, int keep_first) {
     extern __shared__ __align__(1024) uint8_t smem[];
     constexpr int CH = D / 8;
     constexpr int TQ = PF_ROWS / G;  // query tokens per tile
@@ -509,10 +519,16 @@ paged_prefill_attn_kernel(const bf16* __restrict__ q, const bf16* __restrict__ k
     // the warp's last row has the largest causal limit of the warp
     const int warp_last_q = min(qstart + (warp * 16 + 15) / G, qo_len - 1);
     const int warp_hi = custom ? kv_len : kv_len - qo_len + warp_last_q + 1;
-    const int nkb = (kv_hi + PF_KV - 1) / PF_KV;
+    // key blocks [hidden, hidden + gap) lie between the kept first keys and the window of the tile's first query
+    const int nkb_all = (kv_hi + PF_KV - 1) / PF_KV;
+    const int hidden = min(nkb_all, (keep_first + PF_KV - 1) / PF_KV);
+    const int gap = window_left >= 0 ? max(0, min(nkb_all, max(0, kv_len - qo_len + qstart - window_left) / PF_KV) - hidden) : 0;
+    const int nkb = nkb_all - gap;
+    auto key_block = [&](int i) { return i < hidden ? i : i + gap; };
 
-    auto load_stage = [&](int kb) {
-        const uint32_t kdst = kv_smem + (kb & 1) * 2 * KV_TILE;
+    auto load_stage = [&](int i_kb) {
+        const int kb = key_block(i_kb);
+        const uint32_t kdst = kv_smem + (i_kb & 1) * 2 * KV_TILE;
         const uint32_t vdst = kdst + KV_TILE;
 #pragma unroll
         for (int i = 0; i < (PF_KV * CH) / (PF_WARPS * 32); ++i) {
@@ -542,12 +558,13 @@ paged_prefill_attn_kernel(const bf16* __restrict__ q, const bf16* __restrict__ k
     st.init();
     if (nkb > 0) load_stage(0);
     cp_async_commit();
-    for (int kb = 0; kb < nkb; ++kb) {
-        if (kb + 1 < nkb) load_stage(kb + 1);
+    for (int i_kb = 0; i_kb < nkb; ++i_kb) {
+        if (i_kb + 1 < nkb) load_stage(i_kb + 1);
         cp_async_commit();
         cp_async_wait<1>();
         __syncthreads();
-        const uint32_t kt = kv_smem + (kb & 1) * 2 * KV_TILE;
+        const int kb = key_block(i_kb);
+        const uint32_t kt = kv_smem + (i_kb & 1) * 2 * KV_TILE;
 #pragma unroll
         for (int sb = 0; sb < PF_KV / 16; ++sb) {
             const int tb = kb * PF_KV + sb * 16;
@@ -558,7 +575,11 @@ paged_prefill_attn_kernel(const bf16* __restrict__ q, const bf16* __restrict__ k
                 const int n = lim[hh] - tb;
                 uint32_t a = n >= 16 ? 0xffffu : (n <= 0 ? 0u : ((1u << n) - 1u));
                 const int nl = lo[hh] - tb;
-                if (nl > 0) a &= nl >= 16 ? 0u : ~((1u << nl) - 1u);
+                if (nl > 0) {
+                    uint32_t see = nl >= 16 ? 0u : ~((1u << nl) - 1u);
+                    if (keep_first > tb) see |= keep_first - tb >= 16 ? 0xffffu : (1u << (keep_first - tb)) - 1u;
+                    a &= see;
+                }
                 if (custom && a) {
                     const uint32_t wv = req_mask[(size_t)qtok[hh] * mask_words + (tb >> 5)];
                     a &= (wv >> (tb & 31)) & 0xffffu;

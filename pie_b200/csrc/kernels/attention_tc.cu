@@ -10,6 +10,10 @@ PIE_API int pie_prefill_attn_tc_supported(int hq, int hkv, int head_dim, int pag
     return (head_dim == 128 || head_dim == 64) && page_size == 16 && (g == 1 || g == 2 || g == 4 || g == 8 || g == 16) ? 1 : 0;
 }
 
+PIE_API int pie_paged_prefill_attn_tc_kept(const void*, const void*, const int*, const int*, const int*, const int*, const int*, const int*,
+                                           int, const uint32_t*, const long*, void*, float*, int, int, int, int, int, float, int, int,
+                                           const float*, int*, float, int, cudaStream_t);
+
 // Same contract as pie_paged_prefill_attn, with tiles of tile_rows / group query tokens (tile_rows = 128 or
 // 256: one or two MMA tiles per CTA) and `total_pages` = pages of kv_layer including the pad page (last).
 // softcap > 0 (tile_rows 256 only): softmax over softcap * tanh(q.k * sm_scale / softcap).
@@ -20,7 +24,21 @@ PIE_API int pie_paged_prefill_attn_tc_softcap(const void* q, const void* kv_laye
                                               float* lse_out, int n_tokens, int hq, int hkv, int head_dim, int total_pages,
                                               float sm_scale, int window_left, int tile_rows, const float* sinks_log2,
                                               int* status, float softcap, cudaStream_t st) {
+    return pie_paged_prefill_attn_tc_kept(q, kv_layer, page_indices, kv_page_indptr, qo_indptr, kv_lens, tile_req, tile_qstart,
+                                          num_tiles, mask_bits, mask_word_indptr, out, lse_out, n_tokens, hq, hkv, head_dim,
+                                          total_pages, sm_scale, window_left, tile_rows, sinks_log2, status, softcap, 0, st);
+}
+
+// The same with the first `keep_first` keys visible beside the window.
+PIE_API int pie_paged_prefill_attn_tc_kept(const void* q, const void* kv_layer, const int* page_indices,
+                                           const int* kv_page_indptr, const int* qo_indptr, const int* kv_lens,
+                                           const int* tile_req, const int* tile_qstart, int num_tiles,
+                                           const uint32_t* mask_bits, const long* mask_word_indptr, void* out,
+                                           float* lse_out, int n_tokens, int hq, int hkv, int head_dim, int total_pages,
+                                           float sm_scale, int window_left, int tile_rows, const float* sinks_log2,
+                                           int* status, float softcap, int keep_first, cudaStream_t st) {
     if (num_tiles <= 0) return 0;
+    if (keep_first < 0) return (int)cudaErrorInvalidValue;
     const int D_ = head_dim;
     if (!pie_prefill_attn_tc_supported(hq, hkv, head_dim, 16) || (tile_rows != 128 && tile_rows != 256) || !status)
         return (int)cudaErrorInvalidValue;
@@ -61,7 +79,7 @@ PIE_API int pie_paged_prefill_attn_tc_softcap(const void* q, const void* kv_laye
         kern<<<grid, Cfg::THREADS, Cfg::SMEM, st>>>(                                                                  \
             tq, tkv, page_indices, kv_page_indptr, qo_indptr, kv_lens, tile_req, tile_qstart, mask_bits,              \
             mask_word_indptr, (bf16*)out, lse_out, sinks_log2, hq, hkv, total_pages - 1, scale_log2, window_left,     \
-            status, cap_pre, cap_post, hq * D_, D_, nullptr, 0, 0);                                                                  \
+            status, cap_pre, cap_post, hq * D_, D_, nullptr, 0, 0, keep_first);                                                                 \
         return (int)cudaGetLastError();                                                                               \
     }
 #define GO2(G_, NT_)           \
@@ -134,7 +152,7 @@ PIE_API int pie_projected_prefill_attn_tc(const void* q, const void* kv, const i
         kern<<<grid, Cfg::THREADS, Cfg::SMEM, st>>>(tq, tkv, page_indices, kv_page_indptr, qo_indptr, kv_lens, tile_req,  \
                                                     tile_qstart, mask_bits, mask_word_indptr, (bf16*)out, nullptr,    \
                                                     nullptr, heads, heads, total_tokens / 16, scale_log2, window_left, status,  \
-                                                    0.f, 0.f, out_ld, vdim, nullptr, 0, 0);                                          \
+                                                    0.f, 0.f, out_ld, vdim, nullptr, 0, 0, 0);                                         \
         return (int)cudaGetLastError();                                                                               \
     }
     if (D_ == 128) GO(128) else GO(64)

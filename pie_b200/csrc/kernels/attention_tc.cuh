@@ -110,6 +110,7 @@ __device__ __forceinline__ float fast_tanh(float x) {
     return y;
 }
 
+// Beside a sliding window the first `keep_first` keys stay visible.
 // CAP: soft-capped scores (Gemma-2). A raw score s becomes cap_post * tanh(s * cap_pre) with cap_pre = sm_scale / cap
 // and cap_post = cap / sm_scale, so that the unchanged scale by sm_scale * log2(e) gives cap * tanh(s * sm_scale / cap).
 // G = query heads per KV head; NT = MMA tiles of 128 rows per CTA (they share the K/V stages);
@@ -130,8 +131,8 @@ paged_prefill_attn_tc_kernel(const __grid_constant__ CUtensorMap tma_q, const __
                              const uint32_t* __restrict__ mask_bits, const long* __restrict__ mask_word_indptr,
                              bf16* __restrict__ out, float* __restrict__ lse_out, const float* __restrict__ sinks_log2,
                              int hq, int hkv, int pad_page, float scale_log2, int window_left, int* status,
-                             float cap_pre, float cap_post, int out_ld, int out_cols, const float* __restrict__ bias = nullptr,
-                             int bias_pitch = 0, int bias_smem = 0) {
+                             float cap_pre, float cap_post, int out_ld, int out_cols, const float* __restrict__ bias,
+                             int bias_pitch, int bias_smem, int keep_first) {
     constexpr int TQ = AT_ROWS / G;          // query tokens per MMA tile
     constexpr int HALVES = D / 64;
     using Cfg = AtCfg<NT, D, (BIAS && D == 128) ? 2 : AT_STAGES>;
@@ -184,11 +185,14 @@ paged_prefill_attn_tc_kernel(const __grid_constant__ CUtensorMap tma_q, const __
         kv_hi = max(kv_hi, hi);
     }
     const int npages = (kv_hi + 15) >> 4;
-    // a sliding window hides every block before the one its first query's first key lies in: blocks are counted from there
-    const int jb = window_left >= 0 ? max(0, kv_len - qo_len + qstart - window_left) / AT_BK : 0;
+    // a sliding window hides every block before the one its first query's first key lies in, except those with the first
+    // `keep_first` keys: blocks are counted without the hidden ones
+    const int kept = (keep_first + AT_BK - 1) / AT_BK;
+    const int gap = window_left >= 0 ? max(0, max(0, kv_len - qo_len + qstart - window_left) / AT_BK - kept) : 0;
+    auto key_block = [&](int j) { return j < kept ? j : j + gap; };
 #pragma unroll
-    for (int t = 0; t < NT; ++t) nkb_t[t] = max(0, nkb_t[t] - jb);
-    nkb = max(0, nkb - jb);
+    for (int t = 0; t < NT; ++t) nkb_t[t] = max(0, nkb_t[t] - gap);
+    nkb = max(0, nkb - gap);
 
     if (threadIdx.x == 0) {
         mbar_init(q_full(), 1);
@@ -243,7 +247,7 @@ paged_prefill_attn_tc_kernel(const __grid_constant__ CUtensorMap tma_q, const __
                 int pg_id[4];
 #pragma unroll
                 for (int pg = 0; pg < 4; ++pg) {
-                    const int pi = (jb + j) * 4 + pg;
+                    const int pi = key_block(j) * 4 + pg;
                     pg_id[pg] = pi < npages ? pages[pi] : pad_page;
                 }
                 if (!mbar_wait(k_empty(s), par, status, PIE_ERR_WAIT_TMA)) { ok = false; break; }
@@ -366,7 +370,7 @@ paged_prefill_attn_tc_kernel(const __grid_constant__ CUtensorMap tma_q, const __
                 for (int i = 0; i < 32; ++i)
                     sv[c * 32 + i] = CAP ? cap_post * fast_tanh(__uint_as_float(v[i]) * cap_pre) : __uint_as_float(v[i]);
             }
-            const int kb0 = (jb + j) * AT_BK;
+            const int kb0 = key_block(j) * AT_BK;
             if (BIAS) {
                 // distance of key i of the block: n - i (keys after the query, which only a custom mask shows, read the guard)
                 const int n = kb0 < lim && kb0 + AT_BK > lo ? max(kv_len - qo_len + qtok - kb0, -1) : 0;
@@ -401,7 +405,12 @@ paged_prefill_attn_tc_kernel(const __grid_constant__ CUtensorMap tma_q, const __
                 // 64-bit allow mask of this row for the block
                 const int n = lim - kb0, nl = lo - kb0;
                 unsigned long long allow = n >= 64 ? ~0ull : (n <= 0 ? 0ull : ((1ull << n) - 1ull));
-                if (nl > 0) allow &= nl >= 64 ? 0ull : ~((1ull << nl) - 1ull);
+                if (nl > 0) {
+                    unsigned long long see = nl >= 64 ? 0ull : ~((1ull << nl) - 1ull);
+                    const int first = keep_first - kb0;
+                    if (first > 0) see |= first >= 64 ? ~0ull : (1ull << first) - 1ull;
+                    allow &= see;
+                }
                 if (row_mask && allow) {
                     const unsigned long long w0 = row_mask[kb0 >> 5];
                     const unsigned long long w1 = (kb0 + 32 < kv_len) ? row_mask[(kb0 >> 5) + 1] : 0u;

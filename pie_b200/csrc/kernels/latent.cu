@@ -27,9 +27,9 @@ struct StreamNormArgs {
     const void* y;              // [n, ldy] pending token input, or null: x += y / rms(y) * y_norm
     const void* y_norm;
     float* x_out;               // [n, ldx] updated stream (null when y is null); never aliases x
-    const void* norm_w;         // null: only the pending update
+    const void* norm_w;         // null: only the pending update, and with h a copy of the stream in the activation type
     const void* shift;          // null: no token shift
-    void* h;                    // [n, ldh] norm(x)
+    void* h;                    // [n, ldh] norm(x); null without norm_w: none
     void* hs;                   // [n, ldh] h + (previous token's h - h) * shift
     const int* tok_req;         // request of a token
     const int* qo_indptr;
@@ -162,8 +162,8 @@ __global__ void __launch_bounds__(256) stream_norm_kernel(const StreamNormArgs a
             }
             for (int i = a.width + threadIdx.x; i < a.ldx; i += 256) xo[i] = 0.f;
         }
-        if (!norm_w) continue;
-        normalise(v);
+        if (!a.h) continue;
+        if (norm_w) normalise(v);
         T* hr = static_cast<T*>(a.h) + (size_t)t * a.ldh;
         T* hsr = shift ? static_cast<T*>(a.hs) + (size_t)t * a.ldh : nullptr;
         float* keep = nullptr;
@@ -202,17 +202,19 @@ __global__ void shift_commit_kernel(const float* __restrict__ stage, float* __re
 
 // ------------------------------------- query rotation + latent cache rows
 struct LatentRowsArgs {
-    const void* qkv;            // [n, ld]: heads x (dim | rot_dim) queries, then (latent | shared key part) if `cache`
+    const void* q;              // [n, ld]: heads x (dim | rot_dim) queries
+    const void* kv;             // [n, ld_kv]: latent | shared key part (read if `cache`)
     const int* positions;
     const int* slots;           // cache slot (page * page_size + offset), < 0: no write
     const float* inv_freq;      // [rot_dims / 2]
     const void* norm_w;         // [rank]
     void* q_out;                // rows of q_width per (token, head)
     void* cache;                // [slots, cache_row], null for a layer that borrows another's rows
-    int n, ld, heads, dim, rot_dim, rot_dims, rank, rank_pad, cache_row;
+    int n, ld, ld_kv, heads, dim, rot_dim, rot_dims, rank, rank_pad, cache_row;
     int copy_nope;              // 1: q_out = (dim | rotated part | zeros); 0: (.. | rotated part | zeros), see q_zero
     int q_width, q_rot, q_zero; // row width, column of the rotated part, first column zeroed before it
-    float eps;
+    int adjacent;               // 1: the halves of a rotated pair are neighbours, 0: rot_dims / 2 apart
+    float eps, rot_factor;      // factor on cos and sin
 };
 
 // One warp per (token, head) and one more per token for the latent.
@@ -225,12 +227,11 @@ __global__ void __launch_bounds__(256) latent_rows_kernel(const LatentRowsArgs a
     const int lane = threadIdx.x & 31;
     if (w >= (long)a.n * units) return;
     const int t = (int)(w / units), u = (int)(w - (long)t * units);
-    const T* row = static_cast<const T*>(a.qkv) + (size_t)t * a.ld;
     const bool is_q = u < a.heads;
     const T* rot_src;
     T *rot_dst, *end;
     if (is_q) {
-        const T* src = row + (size_t)u * (a.dim + a.rot_dim);
+        const T* src = static_cast<const T*>(a.q) + (size_t)t * a.ld + (size_t)u * (a.dim + a.rot_dim);
         T* dst = static_cast<T*>(a.q_out) + ((size_t)t * a.heads + u) * a.q_width;
         if (a.copy_nope) {
             constexpr int E = 16 / sizeof(T);
@@ -247,7 +248,7 @@ __global__ void __launch_bounds__(256) latent_rows_kernel(const LatentRowsArgs a
     } else {
         const int slot = a.slots[t];
         if (slot < 0) return;
-        const T* src = row + (size_t)a.heads * (a.dim + a.rot_dim);
+        const T* src = static_cast<const T*>(a.kv) + (size_t)t * a.ld_kv;
         T* dst = static_cast<T*>(a.cache) + (size_t)slot * a.cache_row;
         const T* nw = static_cast<const T*>(a.norm_w);
         float ss = 0.f;
@@ -263,9 +264,12 @@ __global__ void __launch_bounds__(256) latent_rows_kernel(const LatentRowsArgs a
     for (int i = lane; i < half; i += 32) {
         float s, c;
         sincosf(pos * a.inv_freq[i], &s, &c);
-        const float p = to_f(rot_src[i]), q = to_f(rot_src[i + half]);
-        rot_dst[i] = from_f<T>(p * c - q * s);
-        rot_dst[i + half] = from_f<T>(q * c + p * s);
+        s *= a.rot_factor;
+        c *= a.rot_factor;
+        const int e0 = a.adjacent ? 2 * i : i, e1 = a.adjacent ? e0 + 1 : i + half;
+        const float p = to_f(rot_src[e0]), q = to_f(rot_src[e1]);
+        rot_dst[e0] = from_f<T>(p * c - q * s);
+        rot_dst[e1] = from_f<T>(q * c + p * s);
     }
     for (int i = a.rot_dims + lane; i < a.rot_dim; i += 32) rot_dst[i] = rot_src[i];
     for (T* p = rot_dst + a.rot_dim + lane; p < end; p += 32) *p = from_f<T>(0.f);
@@ -414,7 +418,7 @@ PIE_API int pie_stream_norm(const StreamNormArgs* args, int f32, int gain_f32, i
     const StreamNormArgs& a = *args;
     if (a.n <= 0) return 0;
     if (a.groups <= 0 || a.width % a.groups || a.rows_per_block <= 0 || a.x_out == a.x || (a.y && !a.x_out) ||
-        (a.shift && (!a.norm_w || !a.hs || !a.state || (commit_requests > 0 && !a.stage))))
+        (a.norm_w && !a.h) || (a.shift && (!a.norm_w || !a.hs || !a.state || (commit_requests > 0 && !a.stage))))
         return (int)cudaErrorInvalidValue;
     const int part = a.width / a.groups;
     const bool vec = part % 4 == 0 && a.ldx % 4 == 0 && a.ldy % 4 == 0 && a.ldh % 4 == 0;

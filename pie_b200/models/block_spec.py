@@ -1,12 +1,90 @@
-"""Descriptions of layers that a configuration lists one by one (sandwich-normed blocks over a 32-bit residual stream):
-each block names its mixer and its feed-forward, with sizes and constants of its own. The Retodra reader and writer of
-`config.json` are at the end.
+"""Descriptions of layers that a configuration lists one by one (blocks over a 32-bit residual stream): each block names
+its mixer and its feed-forward, with sizes and constants of its own. The Retodra reader and writer of `config.json` are at
+the end, those of Nukelix in `nukelix.py`.
 """
 from __future__ import annotations
 
 import math
 from dataclasses import dataclass
-from typing import List, Optional, Union
+from typing import Dict, List, Optional, Tuple, Union
+
+
+EVERYTHING = 1 << 30            # a window no context fills: every earlier token is visible
+
+
+def _pad(n: int, m: int = 8) -> int:
+    return -(-n // m) * m
+
+
+@dataclass
+class RotarySpec:
+    """Rotary positions on the first `dims` dimensions: pairs are neighbours (`adjacent`) or half of `dims` apart. `scaling`:
+    a `rope_scaling` dictionary (`ops.reference.rope_inv_freq`); "yarn" also multiplies cos and sin."""
+    dims: int
+    base: float
+    adjacent: bool = False
+    scaling: Optional[dict] = None
+
+    @property
+    def factor(self) -> float:
+        s = self.scaling
+        return 0.1 * math.log(s["factor"]) + 1.0 if s and s["rope_type"] == "yarn" else 1.0
+
+    def frequencies(self, device="cpu"):
+        """Angle per position of every pair, 32-bit [dims / 2]."""
+        from ..ops import reference
+        return reference.rope_inv_freq(self.dims, self.base, self.scaling, device)
+
+
+@dataclass
+class LatentSpec:
+    """Sizes of one latent-attention mixer: per head `dim` unrotated and `rot_dim` rotated query / key dimensions
+    (the first `rot_dims` of the latter rotate) and `vdim` value dimensions; keys and values are projections of a
+    latent of `kv_rank` numbers per token, which is cached together with one rotated key part shared by all heads.
+    A query sees itself and the `window` - 1 tokens before it. `kv_from`: the layer whose cache this one reads.
+    `q_rank`: queries are projections of a normed latent of their own. `head_gate`: each head's output is scaled by a
+    sigmoid of the mixer's input. The rotation is `RotarySpec`'s."""
+    heads: int
+    dim: int
+    rot_dim: int
+    vdim: int
+    kv_rank: int
+    window: int
+    scale: float
+    rope_base: float
+    rot_dims: int
+    kv_from: Optional[int] = None
+    q_rank: Optional[int] = None
+    head_gate: bool = False
+    rot_adjacent: bool = False
+    rot_scaling: Optional[dict] = None
+
+    @property
+    def rotary(self) -> RotarySpec:
+        return RotarySpec(self.rot_dims, self.rope_base, self.rot_adjacent, self.rot_scaling)
+
+    @property
+    def qk_dim(self) -> int:
+        return self.dim + self.rot_dim
+
+    @property
+    def rank_pad(self) -> int:
+        """Columns of the latent inside a cache row: a multiple of 16 (one tensor-core k step)."""
+        return _pad(self.kv_rank, 16)
+
+    @property
+    def row(self) -> int:
+        """Columns of a cache row: latent, then the rotated key part, each padded with zeros."""
+        return self.rank_pad + _pad(self.rot_dim, 16)
+
+    @property
+    def q_rows(self) -> int:
+        return self.heads * self.qk_dim
+
+    @property
+    def proj_rows(self) -> int:
+        """Rows of the fused query (+ latent and shared key, unless the layer borrows another's cache) projection."""
+        return self.q_rows + (self.kv_rank + self.rot_dim if self.kv_from is None else 0)
 
 
 @dataclass
@@ -85,10 +163,50 @@ class BiasedAttentionSpec:
 
 
 @dataclass
+class GroupedAttentionSpec:
+    """Grouped-query attention with biased projections, q and k normed over all heads together, rotary positions and one
+    sigmoid gate per head. A query sees itself, the `window` - 1 tokens before it and the first `keep_first` tokens. `sink`:
+    a score of 0 without a value takes its share of the softmax. `v_mix`: the values are mixed with those of the first layer
+    that has the flag."""
+    heads: int
+    kv_heads: int
+    dim: int
+    vdim: int
+    scale: float
+    rot: RotarySpec
+    window: int = EVERYTHING
+    keep_first: int = 0
+    sink: bool = False
+    v_mix: bool = False
+
+    group = BiasedAttentionSpec.group
+    group_pad = BiasedAttentionSpec.group_pad
+    head_dim = BiasedAttentionSpec.head_dim
+
+
+@dataclass
+class MatrixMemorySpec:
+    """Matrix memory with exponential input and forget gates (the mLSTM of xLSTM): per head a state [dim, vdim], a
+    normaliser [dim] and a running maximum of the gates' logarithms; `gate_cap` limits the gates softly."""
+    heads: int
+    dim: int
+    vdim: int
+    gate_cap: float
+
+    qk = GatedLinearSpec.qk
+    values = GatedLinearSpec.values
+
+    @property
+    def state_elems(self) -> int:
+        """The states of all heads, then the normalisers, then the maxima."""
+        return self.heads * (self.dim * self.vdim + self.dim + 1)
+
+
+@dataclass
 class ParallelSpec:
-    """Windowed attention and lightning attention side by side on the same input."""
-    left: BiasedAttentionSpec
-    right: LightningSpec
+    """Attention and a recurrent mixer side by side on the same input."""
+    left: Union[BiasedAttentionSpec, GroupedAttentionSpec]
+    right: Union[LightningSpec, MatrixMemorySpec]
     left_scale: float
     right_scale: float
 
@@ -100,12 +218,18 @@ class DenseSpec:
 
 @dataclass
 class ExpertsSpec:
-    """`experts` clamped-GLU experts of width `ff` and `identity` more router outputs whose expert returns its input."""
+    """`experts` GLU experts of width `ff` and `identity` more router outputs whose expert returns its input. Scores are a
+    softmax plus a correction for the choice, or ("sigmoid") the sigmoid of each output. `weight_input`: an expert's weight
+    scales what it reads instead of what it returns. `limit`: clamped GLU, None: SwiGLU. `shared`: width of a SwiGLU expert
+    that every token uses (0: none)."""
     experts: int
     identity: int
     top: int
     ff: int
-    limit: float
+    limit: Optional[float] = None
+    score: str = "softmax"
+    weight_input: bool = False
+    shared: int = 0
 
     @property
     def outputs(self) -> int:
@@ -114,17 +238,47 @@ class ExpertsSpec:
 
 @dataclass
 class BlockSpec:
-    mixer: Union[GatedLinearSpec, ParallelSpec]
+    mixer: Union[GatedLinearSpec, ParallelSpec, GroupedAttentionSpec, LatentSpec]
     ff: Union[DenseSpec, ExpertsSpec, None]
 
     @property
-    def attention(self) -> Optional[BiasedAttentionSpec]:
-        return self.mixer.left if isinstance(self.mixer, ParallelSpec) else None
+    def attention(self) -> Union[BiasedAttentionSpec, GroupedAttentionSpec, None]:
+        """The part of the mixer that keeps keys and values in pages."""
+        a = self.mixer.left if isinstance(self.mixer, ParallelSpec) else self.mixer
+        return a if isinstance(a, (BiasedAttentionSpec, GroupedAttentionSpec)) else None
 
     @property
-    def recurrent(self) -> Union[GatedLinearSpec, LightningSpec]:
+    def latent(self) -> Optional[LatentSpec]:
+        return self.mixer if isinstance(self.mixer, LatentSpec) else None
+
+    @property
+    def recurrent(self) -> Union[GatedLinearSpec, LightningSpec, MatrixMemorySpec, None]:
         """The part of the mixer whose state is carried from token to token."""
-        return self.mixer.right if isinstance(self.mixer, ParallelSpec) else self.mixer
+        r = self.mixer.right if isinstance(self.mixer, ParallelSpec) else self.mixer
+        return r if isinstance(r, (GatedLinearSpec, LightningSpec, MatrixMemorySpec)) else None
+
+
+def projection_sizes(mixer) -> Dict[str, int]:
+    """Checkpoint name (within the mixer) -> rows of the projections of its input that run as one product, in order."""
+    if isinstance(mixer, GatedLinearSpec):
+        return {"q": mixer.qk, "k": mixer.qk, "v": mixer.values, "g": mixer.values, "a1": mixer.rank}
+    if isinstance(mixer, LatentSpec):
+        return {"dq": mixer.q_rank, "dkv": mixer.kv_rank + mixer.rot_dim, "g": mixer.heads}
+    if isinstance(mixer, ParallelSpec):
+        return {f"{side}.{n}": k for side, part in (("left", mixer.left), ("right", mixer.right)) for n, k in projection_sizes(part).items()}
+    if isinstance(mixer, (LightningSpec, MatrixMemorySpec)):
+        return {"q": mixer.qk, "k": mixer.qk, "v": mixer.values, "g": mixer.values}
+    gates = mixer.heads if isinstance(mixer, GroupedAttentionSpec) else mixer.heads * mixer.vdim
+    return {"q": mixer.heads * mixer.dim, "k": mixer.kv_heads * mixer.dim, "v": mixer.kv_heads * mixer.vdim, "g": gates}
+
+
+def projection_columns(mixer) -> Dict[str, Tuple[int, int]]:
+    """Name -> (first column, columns) of the mixer's fused input projection; every part starts on a multiple of 8."""
+    out, at = {}, 0
+    for name, n in projection_sizes(mixer).items():
+        out[name] = (at, n)
+        at += _pad(n)
+    return out
 
 
 # ------------------------------------------------------------------ Retodra

@@ -10,13 +10,14 @@ from dataclasses import dataclass, field, asdict
 from pathlib import Path
 from typing import Optional
 
-from .block_spec import BlockSpec, retodra_config, retodra_shape
+from .block_spec import EVERYTHING, LatentSpec, _pad, retodra_config, retodra_shape
+from .nukelix import nukelix_config, nukelix_shape
 
 LLAMA_LIKE = {"llama", "qwen2", "qwen3", "mistral", "phi3"}   # pre-norm decoder blocks with SwiGLU and rotate-half RoPE
 # `model_type` strings of checkpoints this build loads (the architecture registry of the loader)
 SUPPORTED_MODEL_TYPES = ("llama", "mistral", "qwen2", "qwen3", "phi3", "qwen3_moe", "mixtral", "olmo2", "olmo3", "gpt_oss",
                          "qwen3_5", "qwen3_next", "mamba2_hybrid", "gemma2", "gemma3_text", "gemma3", "qwen2_moe", "qwen2_vl",
-                         "qwen2_audio", "puzutar", "retodra")
+                         "qwen2_audio", "puzutar", "retodra", "nukelix")
 MAMBA_TYPES = {"mamba2_hybrid"}         # Mamba-2 (state-space) mixers in llama-like blocks, between full-attention layers
 GDN_TYPES = {"qwen3_5", "qwen3_next"}   # hybrids: Gated DeltaNet (linear attention) layers between full-attention layers
 POST_NORM = {"olmo2", "olmo3"}       # same block with the norms after attention / MLP and q, k norms over all heads
@@ -25,57 +26,12 @@ MOE_TYPES = {"qwen3_moe", "mixtral", "gpt_oss", "qwen2_moe"}
 # alternating local / global layers (Gemma-3: a RoPE base of their own for the local ones; Gemma-2: soft-capped logits)
 GEMMA_TYPES = {"gemma2", "gemma3_text", "gemma3"}
 # configs that name the design under "architecture" instead of "model_type"
-ARCHITECTURES = {"Puzutar": "puzutar", "Retodra": "retodra"}
+ARCHITECTURES = {"Puzutar": "puzutar", "Retodra": "retodra", "Nukelix": "nukelix"}
 
 
 def config_model_type(cfg: dict) -> str:
     """The registry name a `config.json` dictionary asks for ("" when it names none)."""
     return cfg.get("model_type") or ARCHITECTURES.get(cfg.get("architecture", ""), "")
-
-
-@dataclass
-class LatentSpec:
-    """Sizes of one latent-attention mixer: per head `dim` unrotated and `rot_dim` rotated query / key dimensions
-    (the first `rot_dims` of the latter rotate) and `vdim` value dimensions; keys and values are projections of a
-    latent of `kv_rank` numbers per token, which is cached together with one rotated key part shared by all heads.
-    A query sees itself and the `window` - 1 tokens before it. `kv_from`: the layer whose cache this one reads."""
-    heads: int
-    dim: int
-    rot_dim: int
-    vdim: int
-    kv_rank: int
-    window: int
-    scale: float
-    rope_base: float
-    rot_dims: int
-    kv_from: Optional[int] = None
-
-    @property
-    def qk_dim(self) -> int:
-        return self.dim + self.rot_dim
-
-    @property
-    def rank_pad(self) -> int:
-        """Columns of the latent inside a cache row: a multiple of 16 (one tensor-core k step)."""
-        return _pad(self.kv_rank, 16)
-
-    @property
-    def row(self) -> int:
-        """Columns of a cache row: latent, then the rotated key part, each padded with zeros."""
-        return self.rank_pad + _pad(self.rot_dim, 16)
-
-    @property
-    def q_rows(self) -> int:
-        return self.heads * self.qk_dim
-
-    @property
-    def proj_rows(self) -> int:
-        """Rows of the fused query (+ latent and shared key, unless the layer borrows another's cache) projection."""
-        return self.q_rows + (self.kv_rank + self.rot_dim if self.kv_from is None else 0)
-
-
-def _pad(n: int, m: int = 8) -> int:
-    return -(-n // m) * m
 
 
 @dataclass
@@ -135,7 +91,8 @@ class ModelConfig:
     norm_groups: int = 1               # RMSNorm over this many equal parts of the width, each with its own mean square
     token_shift: bool = False          # the mixer reads h + (previous token's h - h) * shift: state of a sequence
     token_side_dim: int = 0            # width of the per-layer token input (0: none)
-    # layers described one by one: sandwich-normed blocks over a 32-bit residual stream
+    # layers described one by one over a 32-bit residual stream: sandwich-normed blocks, or (post_norm) blocks that norm
+    # their sublayers' outputs only
     blocks: Optional[list] = None      # BlockSpec per layer
     # quantisation of the linear weights: None | "fp8_block" (128x128 weight scales)
     quantization: Optional[str] = None
@@ -184,10 +141,16 @@ class ModelConfig:
         return self.latent is not None or self.blocks is not None
 
     @property
+    def latent_specs(self) -> list:
+        """The latent-attention mixers of all layers."""
+        return self.latent if self.latent is not None else [b.latent for b in self.blocks or () if b.latent is not None]
+
+    @property
     def kv_layers(self) -> list:
-        """(kv heads, head dim) of every layer that writes keys and values, in order."""
+        """(kv heads, head dim) of every layer that has a cache, in order; latent rows count as no head of the row's width."""
         if self.blocks is not None:
-            return [(b.attention.kv_heads, b.attention.head_dim) for b in self.blocks if b.attention is not None]
+            return [(0, b.latent.row) if b.latent is not None else (b.attention.kv_heads, b.attention.head_dim)
+                    for b in self.blocks if b.latent is not None or b.attention is not None]
         return [(self.num_key_value_heads, self.head_dim)] * self.num_hidden_layers
 
     @property
@@ -196,7 +159,7 @@ class ModelConfig:
         if self.latent is not None:
             return len(self.latent_cache_layers) * self.latent_row
         if self.blocks is not None:
-            return sum(2 * h * d for h, d in self.kv_layers)
+            return sum(2 * h * d if h else d for h, d in self.kv_layers)
         return self.num_hidden_layers * 2 * self.num_key_value_heads * self.head_dim
 
     @property
@@ -228,12 +191,14 @@ class ModelConfig:
         return self.gdn_conv_channels + self.linear_num_value_heads * self.linear_value_head_dim + 2 * self.linear_num_value_heads
 
     def layer_window_left(self, li: int) -> int:
-        """Keys left of the query that layer `li` sees (-1: all). HF `sliding_window` counts the query itself."""
+        """Keys left of the query that layer `li` sees (-1: all, or far ones beside a window). HF `sliding_window` counts the
+        query itself."""
         if self.latent is not None:
             return self.latent[li].window - 1
         if self.blocks is not None:
-            a = self.blocks[li].attention
-            return a.window - 1 if a is not None else 0
+            b = self.blocks[li]
+            a = b.latent or b.attention
+            return 0 if a is None else -1 if a.window == EVERYTHING or getattr(a, "keep_first", 0) else a.window - 1
         if not self.sliding_window or self.sliding_window <= 0:
             return -1
         if self.layer_types is not None and self.layer_types[li] != "sliding_attention":
@@ -264,6 +229,8 @@ class ModelConfig:
             return _puzutar_config(cfg, name)
         if mt == "retodra":
             return retodra_config(cfg, name)
+        if mt == "nukelix":
+            return nukelix_config(cfg, name)
         if mt == "gemma3" and "text_config" in cfg:       # multimodal wrapper: the language model's own section
             cfg = dict(cfg["text_config"], model_type="gemma3_text")
             mt = "gemma3_text"
@@ -545,11 +512,15 @@ PRESETS = {
 LAYERED_PRESETS = {
     "puzutar-8b": (_puzutar_config, puzutar_shape, dict()),
     "retodra-19b": (retodra_config, retodra_shape, dict()),
+    "nukelix-20b": (nukelix_config, nukelix_shape, dict()),
     "tiny-puzutar": (_puzutar_config, puzutar_shape, dict(
         layers=3, width=256, heads=2, dim=48, rot_dim=16, vdim=40, kv_rank=64, window=40, ff=384, vocab=32000, groups=2, side=16)),
     "tiny-retodra": (retodra_config, retodra_shape, dict(
         layers=4, width=256, gla_heads=2, gla_dim=48, gla_vdim=64, rank=8, heads=6, kv_heads=2, dim=40, window=50, buckets=12,
         right_heads=3, right_dim=32, right_vdim=40, ff=384, experts=6, identity=2, top=3, expert_ff=96, vocab=32000)),
+    "tiny-nukelix": (nukelix_config, nukelix_shape, dict(
+        layers=4, width=256, heads=6, kv_heads=2, dim=40, window=50, keep_first=3, right_heads=3, right_dim=32, right_vdim=40, lat_heads=4,
+        lat_dim=24, rot_dim=8, q_rank=72, kv_rank=48, ff=96, experts=6, top=2, shared=112, vocab=32000)),
 }
 
 

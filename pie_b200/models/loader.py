@@ -33,8 +33,10 @@ from typing import Callable, Dict, List, Optional, Sequence, Tuple
 
 import torch
 
-from .block_spec import DenseSpec, ExpertsSpec, GatedLinearSpec, retodra_dict
+from .block_spec import (BiasedAttentionSpec, DenseSpec, ExpertsSpec, GatedLinearSpec, GroupedAttentionSpec, LatentSpec, MatrixMemorySpec,
+                         ParallelSpec, projection_columns, projection_sizes, retodra_dict)
 from .config import ModelConfig, _pad, _puzutar_dict
+from .nukelix import nukelix_dict
 from .weights import kv_head_range, torch_dtype
 
 
@@ -357,6 +359,8 @@ def complete_blocks(cfg: ModelConfig, reader) -> None:
     """Sizes that only the checkpoint's tensors give: the rank of a decay projection, the rows of a bias table."""
     have = set(reader.names())
     for i, b in enumerate(cfg.blocks):
+        if not isinstance(b.mixer, GatedLinearSpec) and not isinstance(b.attention, BiasedAttentionSpec):
+            continue
         name = f"l{i}.mix.a1" if isinstance(b.mixer, GatedLinearSpec) else f"l{i}.mix.left.rel"
         if name not in have:
             raise KeyError(f"checkpoint has no tensor {name}")
@@ -371,10 +375,10 @@ def complete_blocks(cfg: ModelConfig, reader) -> None:
 
 
 def _compile_blocks(cfg: ModelConfig, names: set, tp_size: int, dtype: str) -> Program:
-    """Layout plan of sandwich-normed blocks (Retodra names). Fused per layer: every projection that reads the mixer's input
-    (`w_in`, each part on a multiple of 8 rows: `sandwich.projection_columns`), the output projections of two mixers side
-    by side along K (`w_out`), gate and up interleaved. Dimensions a GEMM sees are padded with zeros, those of a gated
-    feed-forward to 16."""
+    """Layout plan of layers described one by one (Retodra and Nukelix names). Fused per layer: every projection that reads
+    the mixer's input (`w_in`, each part on a multiple of 8 rows: `block_spec.projection_columns`), the output projections of
+    two mixers side by side along K (`w_out`), gate and up interleaved. Gates of a matrix memory stay apart (`w_gates`): they
+    are wanted in 32-bit. Dimensions a GEMM sees are padded with zeros, those of a gated feed-forward to 16."""
     if tp_size > 1:
         raise NotImplementedError("layers described one by one under tensor parallelism")
     W = cfg.hidden_size
@@ -388,32 +392,52 @@ def _compile_blocks(cfg: ModelConfig, names: set, tp_size: int, dtype: str) -> P
     def gate_up(n, ff):
         return Interleave(Pad(r(n + "gate", ff, W), [16, 8]), Pad(r(n + "up", ff, W), [16, 8]))
 
-    att["embed"], att["lm_head"] = r("embed", cfg.vocab_size, W), Pad(r("head", cfg.vocab_size, W))
+    def attention(P, X, a):
+        """Norms and biases of grouped attention (`X`: the checkpoint's prefix); returns its output projection."""
+        nq, nk, nv = a.heads * a.dim, a.kv_heads * a.dim, a.kv_heads * a.vdim
+        att[P + "q_norm"], att[P + "k_norm"] = r(X + "q.norm", nq), r(X + "k.norm", nk)
+        if isinstance(a, BiasedAttentionSpec):
+            if a.buckets is None:
+                raise ValueError(f"{X}rel: the rows of the bias table are not known (complete_blocks)")
+            att[P + "rel"] = Keep32(r(X + "rel", a.buckets, a.heads))
+        else:
+            att[P + "q_b"], att[P + "k_b"], att[P + "v_b"] = r(X + "q.b", nq), r(X + "k.b", nk), r(X + "v.b", nv)
+            if a.v_mix:
+                att[P + "vmix"] = Keep32(r(X + "vmix"))
+        return Pad(r(X + "o", W, a.heads * a.vdim))
+
+    att["embed"] = r("embed", cfg.vocab_size, W)
+    att["lm_head"] = Pad(r("embed" if cfg.tie_word_embeddings else "head", cfg.vocab_size, W))
     att["final_norm"] = r("final.norm", W)
     for li, b in enumerate(cfg.blocks):
         L, P, X = f"l{li}.", f"layers.{li}.", f"l{li}.mix."
-        halves = ("1", "2") if b.ff is not None else ("1",)
-        for h in halves:
-            att[P + "ln" + h], att[P + f"ln{h}b"], att[P + "ls" + h] = r(L + "norm" + h, W), r(L + f"norm{h}b", W), r(L + "ls" + h, W)
+        for h in ("1", "2") if b.ff is not None else ("1",):
+            if cfg.post_norm:
+                att[P + f"ln{h}b"] = r(L + "norm" + h, W)
+            else:
+                att[P + "ln" + h], att[P + f"ln{h}b"], att[P + "ls" + h] = r(L + "norm" + h, W), r(L + f"norm{h}b", W), r(L + "ls" + h, W)
         m = b.mixer
         if isinstance(m, GatedLinearSpec):
             if m.rank is None:
                 raise ValueError(f"layer {li}: the rank of the decay projection is not known (complete_blocks)")
-            rows = [("q", m.qk), ("k", m.qk), ("v", m.values), ("g", m.values), ("a1", m.rank)]
             att[P + "a2"], att[P + "a2_b"], att[P + "o_norm"] = r(X + "a2", m.qk, m.rank), r(X + "a2.b", m.qk), r(X + "norm", m.vdim)
             att[P + "w_out"] = Pad(r(X + "o", W, m.values))
+        elif isinstance(m, LatentSpec):
+            att[P + "q_latent_norm"], att[P + "latent_norm"] = r(X + "dq.norm", m.q_rank), r(X + "dkv.norm", m.kv_rank)
+            att[P + "w_uq"] = Pad(r(X + "uq", m.q_rows, m.q_rank))
+            att[P + "w_uk"], att[P + "w_uv"] = r(X + "uk", m.heads * m.dim, m.kv_rank), r(X + "uv", m.heads * m.vdim, m.kv_rank)
+            att[P + "w_out"] = Pad(r(X + "o", W, m.heads * m.vdim))
+        elif isinstance(m, GroupedAttentionSpec):
+            att[P + "w_out"] = attention(P, X, m)
         else:
-            a, s = m.left, m.right
-            if a.buckets is None:
-                raise ValueError(f"layer {li}: the rows of the bias table are not known (complete_blocks)")
-            nq, nk = a.heads * a.dim, a.kv_heads * a.dim
-            rows = [("left.q", nq), ("left.k", nk), ("left.v", a.kv_heads * a.vdim), ("left.g", a.heads * a.vdim),
-                    ("right.q", s.qk), ("right.k", s.qk), ("right.v", s.values), ("right.g", s.values)]
-            att[P + "q_norm"], att[P + "k_norm"] = r(X + "left.q.norm", nq), r(X + "left.k.norm", nk)
-            att[P + "rel"] = Keep32(r(X + "left.rel", a.buckets, a.heads))
+            s = m.right
+            left = attention(P, X + "left.", m.left)
             att[P + "o_norm"] = r(X + "right.norm", s.values)
-            att[P + "w_out"] = Concat([Pad(r(X + "left.o", W, a.heads * a.vdim)), Pad(r(X + "right.o", W, s.values))], 1)
-        att[P + "w_in"] = Concat([Pad(r(X + n, k, W)) for n, k in rows], 0)
+            att[P + "w_out"] = Concat([left, Pad(r(X + "right.o", W, s.values))], 1)
+            if isinstance(s, MatrixMemorySpec):
+                att[P + "w_gates"] = Pad(Concat([r(X + "right.i", s.heads, W), r(X + "right.f", s.heads, W)], 0), [1, 8])
+                att[P + "b_gates"] = Keep32(Concat([r(X + "right.i.b", s.heads), r(X + "right.f.b", s.heads)], 0))
+        att[P + "w_in"] = Concat([Pad(r(X + n, k, W)) for n, k in projection_sizes(m).items()], 0)
         F = L + "mlp."
         if isinstance(b.ff, DenseSpec):
             att[P + "w_gate_up"], att[P + "w_down"] = gate_up(F, b.ff.ff), Pad(r(F + "down", W, b.ff.ff), [8, 16])
@@ -422,7 +446,11 @@ def _compile_blocks(cfg: ModelConfig, names: set, tp_size: int, dtype: str) -> P
             att[P + "experts_gate_up"] = Stack([gate_up(e, b.ff.ff) for e in each])
             att[P + "experts_down"] = Stack([Pad(r(e + "down", W, b.ff.ff), [8, 16]) for e in each])
             att[P + "router"] = Pad(r(F + "router", b.ff.outputs, W), [1, 8])
-            att[P + "correction"] = Keep32(r(F + "correction", b.ff.outputs))
+            if b.ff.score == "softmax":
+                att[P + "correction"] = Keep32(r(F + "correction", b.ff.outputs))
+            if b.ff.shared:
+                att[P + "shared_gate_up"] = gate_up(F + "shared.", b.ff.shared)
+                att[P + "shared_down"] = Pad(r(F + "shared.down", W, b.ff.shared), [8, 16])
     return Program(att, dtype, {"tp_size": 1, "tp_rank": 0, "ep": False, "layers": cfg.num_hidden_layers, "vocab_start": 0})
 
 
@@ -835,32 +863,56 @@ def _latent_tensors(cfg: ModelConfig, weights: dict) -> Dict[str, torch.Tensor]:
 
 
 def _block_tensors(cfg: ModelConfig, weights: dict) -> Dict[str, torch.Tensor]:
-    """Checkpoint tensors of sandwich-normed blocks from their runtime layout (the inverse of `_compile_blocks`)."""
-    from .sandwich import projection_columns
+    """Checkpoint tensors of layers described one by one from their runtime layout (the inverse of `_compile_blocks`)."""
     W = cfg.hidden_size
-    t = {"embed": weights["embed"], "head": weights["lm_head"][:cfg.vocab_size, :W], "final.norm": weights["final_norm"]}
+    t = {"embed": weights["embed"], "final.norm": weights["final_norm"]}
+    if not cfg.tie_word_embeddings:
+        t["head"] = weights["lm_head"][:cfg.vocab_size, :W]
     for li, (lw, b) in enumerate(zip(weights["layers"], cfg.blocks)):
         L, X, F, m, f = f"l{li}.", f"l{li}.mix.", f"l{li}.mlp.", b.mixer, b.ff
+        dt = lw["w_in"].dtype
         for h in ("1", "2") if f is not None else ("1",):
-            t[L + "norm" + h], t[L + f"norm{h}b"], t[L + "ls" + h] = lw["ln" + h], lw[f"ln{h}b"], lw["ls" + h]
+            if cfg.post_norm:
+                t[L + "norm" + h] = lw[f"ln{h}b"]
+            else:
+                t[L + "norm" + h], t[L + f"norm{h}b"], t[L + "ls" + h] = lw["ln" + h], lw[f"ln{h}b"], lw["ls" + h]
         for n, (at, k) in projection_columns(m).items():
             t[X + n] = lw["w_in"][at:at + k, :W]
+        a, side = b.attention, "left." if isinstance(m, ParallelSpec) else ""
+        hv = a.heads * a.vdim if a is not None else 0
+        if a is not None:
+            t[X + side + "q.norm"], t[X + side + "k.norm"], t[X + side + "o"] = lw["q_norm"], lw["k_norm"], lw["w_out"][:W, :hv]
+            if isinstance(a, BiasedAttentionSpec):
+                t[X + side + "rel"] = lw["rel"].to(dt)
+            else:
+                t[X + side + "q.b"], t[X + side + "k.b"], t[X + side + "v.b"] = lw["q_b"], lw["k_b"], lw["v_b"]
+                if a.v_mix:
+                    t[X + side + "vmix"] = lw["vmix"].to(dt)
         if isinstance(m, GatedLinearSpec):
             t[X + "a2"], t[X + "a2.b"], t[X + "norm"], t[X + "o"] = lw["a2"], lw["a2_b"], lw["o_norm"], lw["w_out"][:W, :m.values]
-        else:
-            hv = m.left.heads * m.left.vdim
-            t[X + "left.q.norm"], t[X + "left.k.norm"], t[X + "left.rel"] = lw["q_norm"], lw["k_norm"], lw["rel"].to(lw["w_in"].dtype)
-            t[X + "left.o"], t[X + "right.o"] = lw["w_out"][:W, :hv], lw["w_out"][:W, _pad(hv):_pad(hv) + m.right.values]
-            t[X + "right.norm"] = lw["o_norm"]
-        split = lambda gu: (gu[0::2][:f.ff, :W], gu[1::2][:f.ff, :W])
+        elif isinstance(m, LatentSpec):
+            t[X + "dq.norm"], t[X + "dkv.norm"], t[X + "uq"] = lw["q_latent_norm"], lw["latent_norm"], lw["w_uq"][:m.q_rows, :m.q_rank]
+            t[X + "uk"], t[X + "uv"], t[X + "o"] = lw["w_uk"], lw["w_uv"], lw["w_out"][:W, :m.heads * m.vdim]
+        elif isinstance(m, ParallelSpec):
+            t[X + "right.norm"], t[X + "right.o"] = lw["o_norm"], lw["w_out"][:W, _pad(hv):_pad(hv) + m.right.values]
+            if isinstance(m.right, MatrixMemorySpec):
+                for j, n in enumerate(("i", "f")):
+                    rows = slice(j * m.right.heads, (j + 1) * m.right.heads)
+                    t[X + "right." + n], t[X + f"right.{n}.b"] = lw["w_gates"][rows, :W], lw["b_gates"][rows].to(dt)
+        split = lambda gu, ff: (gu[0::2][:ff, :W], gu[1::2][:ff, :W])
         if isinstance(f, DenseSpec):
-            t[F + "gate"], t[F + "up"] = split(lw["w_gate_up"])
+            t[F + "gate"], t[F + "up"] = split(lw["w_gate_up"], f.ff)
             t[F + "down"] = lw["w_down"][:W, :f.ff]
         elif isinstance(f, ExpertsSpec):
             for e in range(f.experts):
-                t[F + f"e{e}.gate"], t[F + f"e{e}.up"] = split(lw["experts_gate_up"][e])
+                t[F + f"e{e}.gate"], t[F + f"e{e}.up"] = split(lw["experts_gate_up"][e], f.ff)
                 t[F + f"e{e}.down"] = lw["experts_down"][e][:W, :f.ff]
-            t[F + "router"], t[F + "correction"] = lw["router"][:, :W], lw["correction"].to(lw["router"].dtype)
+            t[F + "router"] = lw["router"][:, :W]
+            if f.score == "softmax":
+                t[F + "correction"] = lw["correction"].to(lw["router"].dtype)
+            if f.shared:
+                t[F + "shared.gate"], t[F + "shared.up"] = split(lw["shared_gate_up"], f.shared)
+                t[F + "shared.down"] = lw["shared_down"][:W, :f.shared]
     return t
 
 
@@ -875,7 +927,7 @@ def export_hf_checkpoint(cfg: ModelConfig, weights: dict, path) -> None:
         return
     if cfg.blocks is not None:
         save_file({k: v.contiguous().cpu() for k, v in _block_tensors(cfg, weights).items()}, str(p / "model.safetensors"))
-        (p / "config.json").write_text(json.dumps(retodra_dict(cfg)))
+        (p / "config.json").write_text(json.dumps((nukelix_dict if cfg.model_type == "nukelix" else retodra_dict)(cfg)))
         return
     d, hq, hkv = cfg.head_dim, cfg.num_attention_heads, cfg.num_key_value_heads
     ungain = (lambda g: g.float() - 1.0) if cfg.norm_plus_one else (lambda g: g)      # Gemma stores (gain - 1)

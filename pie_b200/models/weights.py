@@ -12,7 +12,7 @@ Runtime layout per layer (this rank's shard under tensor parallelism):
   Gemma-2/3 (sandwich norms): ln1 / ln2 before attention / MLP, ln_pa / ln_pf on their outputs before the
   residual add; gains hold the full multiplier (the loader adds the checkpoint's implicit 1)
   Puzutar (latent attention in parallel blocks): see `loader._compile_latent`
-  Retodra (linear attention in sandwich-normed blocks): see `loader._compile_blocks`
+  Retodra, Nukelix (layers described one by one): see `loader._compile_blocks`
 MoE layers replace w_gate_up / w_down by router [E, H], experts_gate_up [E_local, 2*Im, H]
 (interleaved) and experts_down [E_local, H, Im].
 
@@ -245,37 +245,60 @@ def _random_latent(cfg: ModelConfig, gen: _Gen, tp_size: int) -> dict:
 
 
 def _random_blocks(cfg: ModelConfig, gen: _Gen, tp_size: int) -> dict:
-    """Random checkpoint tensors of sandwich-normed blocks, brought into the runtime layout by the loader."""
-    from .block_spec import DenseSpec, GatedLinearSpec
+    """Random checkpoint tensors of layers described one by one, brought into the runtime layout by the loader. Gains are
+    drawn as their distance from one where the checkpoint stores that (`norm_plus_one`)."""
+    from .block_spec import (BiasedAttentionSpec, DenseSpec, GatedLinearSpec, LatentSpec, MatrixMemorySpec, ParallelSpec, projection_sizes)
     from .loader import TensorDictReader, compile_program, execute_program
     W = cfg.hidden_size
     near = lambda n: gen.normal(n, std=0.1)
-    t = {"embed": gen.normal(cfg.vocab_size, W), "head": gen.normal(cfg.vocab_size, W), "final.norm": near(W)}
+    gain = near if cfg.norm_plus_one else lambda n: 1 + near(n)
+    t = {"embed": gen.normal(cfg.vocab_size, W, **({"std": 1.0} if cfg.post_norm else {})), "final.norm": gain(W)}
+    if not cfg.tie_word_embeddings:
+        t["head"] = gen.normal(cfg.vocab_size, W)
     for li, b in enumerate(cfg.blocks):
         L, X, F, m, f = f"l{li}.", f"l{li}.mix.", f"l{li}.mlp.", b.mixer, b.ff
         for h in ("1", "2") if f is not None else ("1",):
-            t[L + "norm" + h], t[L + f"norm{h}b"], t[L + "ls" + h] = near(W), near(W), 0.3 + near(W)
+            t[L + "norm" + h] = gain(W)
+            if not cfg.post_norm:
+                t[L + f"norm{h}b"], t[L + "ls" + h] = gain(W), 0.3 + near(W)
         if isinstance(m, GatedLinearSpec):
             m.rank = m.rank or 16
-            for n, k in (("q", m.qk), ("k", m.qk), ("v", m.values), ("g", m.values), ("a1", m.rank)):
-                t[X + n] = gen.normal(k, W)
+        for n, k in projection_sizes(m).items():
+            t[X + n] = gen.normal(k, W)
+        a, A = b.attention, X + ("left." if isinstance(m, ParallelSpec) else "")
+        if a is not None:
+            nq, nk, nv = a.heads * a.dim, a.kv_heads * a.dim, a.kv_heads * a.vdim
+            t[A + "q.norm"], t[A + "k.norm"], t[A + "o"] = 1 + near(nq), 1 + near(nk), gen.normal(W, a.heads * a.vdim)
+            if isinstance(a, BiasedAttentionSpec):
+                a.buckets = a.buckets or 32
+                t[A + "rel"] = gen.normal(a.buckets, a.heads, std=0.5)
+            else:
+                t[A + "q.b"], t[A + "k.b"], t[A + "v.b"] = near(nq), near(nk), near(nv)
+                if a.v_mix:
+                    t[A + "vmix"] = (0.4 + near(1))[0]
+        if isinstance(m, GatedLinearSpec):
             t[X + "a2"], t[X + "a2.b"] = gen.normal(m.qk, m.rank, std=m.rank ** -0.5), gen.normal(m.qk, std=1.0)
             t[X + "norm"], t[X + "o"] = 1 + near(m.vdim), gen.normal(W, m.values)
-        else:
-            a, s = m.left, m.right
-            a.buckets = a.buckets or 32
-            for n, k in (("left.q", a.heads * a.dim), ("left.k", a.kv_heads * a.dim), ("left.v", a.kv_heads * a.vdim),
-                         ("left.g", a.heads * a.vdim), ("right.q", s.qk), ("right.k", s.qk), ("right.v", s.values), ("right.g", s.values)):
-                t[X + n] = gen.normal(k, W)
-            t[X + "left.q.norm"], t[X + "left.k.norm"] = 1 + near(a.heads * a.dim), 1 + near(a.kv_heads * a.dim)
-            t[X + "left.rel"], t[X + "left.o"] = gen.normal(a.buckets, a.heads, std=0.5), gen.normal(W, a.heads * a.vdim)
+        elif isinstance(m, LatentSpec):
+            t[X + "dq.norm"], t[X + "dkv.norm"] = 1 + near(m.q_rank), 1 + near(m.kv_rank)
+            t[X + "uq"] = gen.normal(m.q_rows, m.q_rank, std=m.q_rank ** -0.5)
+            t[X + "uk"] = gen.normal(m.heads * m.dim, m.kv_rank, std=m.kv_rank ** -0.5)
+            t[X + "uv"] = gen.normal(m.heads * m.vdim, m.kv_rank, std=m.kv_rank ** -0.5)
+            t[X + "o"] = gen.normal(W, m.heads * m.vdim)
+        elif isinstance(m, ParallelSpec):
+            s = m.right
             t[X + "right.norm"], t[X + "right.o"] = 1 + near(s.values), gen.normal(W, s.values)
+            if isinstance(s, MatrixMemorySpec):
+                t[X + "right.i"], t[X + "right.f"] = gen.normal(s.heads, W, std=W ** -0.5), gen.normal(s.heads, W, std=W ** -0.5)
+                t[X + "right.i.b"], t[X + "right.f.b"] = near(s.heads), 3 + gen.normal(s.heads, std=1.0)
         if isinstance(f, DenseSpec):
             t[F + "gate"], t[F + "up"], t[F + "down"] = gen.normal(f.ff, W), gen.normal(f.ff, W), gen.normal(W, f.ff)
         elif f is not None:
-            for e in range(f.experts):
-                t[F + f"e{e}.gate"], t[F + f"e{e}.up"], t[F + f"e{e}.down"] = gen.normal(f.ff, W), gen.normal(f.ff, W), gen.normal(W, f.ff)
-            t[F + "router"], t[F + "correction"] = gen.normal(f.outputs, W, std=W ** -0.5), gen.normal(f.outputs, std=0.02)
+            for e, n in [(f"e{e}.", f.ff) for e in range(f.experts)] + ([("shared.", f.shared)] if f.shared else []):
+                t[F + e + "gate"], t[F + e + "up"], t[F + e + "down"] = gen.normal(n, W), gen.normal(n, W), gen.normal(W, n)
+            t[F + "router"] = gen.normal(f.outputs, W, std=W ** -0.5)
+            if f.score == "softmax":
+                t[F + "correction"] = gen.normal(f.outputs, std=0.02)
     prog = compile_program(cfg, list(t), tp_size, 0, False, str(gen.dtype).replace("torch.", ""))
     return execute_program(prog, TensorDictReader(t), gen.device)
 

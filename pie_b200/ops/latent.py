@@ -23,8 +23,9 @@ def _struct(name: str, *fields):
 # mirrors of the argument structs in csrc/kernels/latent.cu and latent_attn.cu
 StreamNormArgs = _struct("StreamNormArgs", ("x y y_norm x_out norm_w shift h hs tok_req qo_indptr slots reset state stage", p),
                          ("n width ldx ldy ldh groups rows_per_block", i32), ("eps", f32))
-LatentRowsArgs = _struct("LatentRowsArgs", ("qkv positions slots inv_freq norm_w q_out cache", p),
-                         ("n ld heads dim rot_dim rot_dims rank rank_pad cache_row copy_nope q_width q_rot q_zero", i32), ("eps", f32))
+LatentRowsArgs = _struct("LatentRowsArgs", ("q kv positions slots inv_freq norm_w q_out cache", p),
+                         ("n ld ld_kv heads dim rot_dim rot_dims rank rank_pad cache_row copy_nope q_width q_rot q_zero adjacent", i32),
+                         ("eps rot_factor", f32))
 LatentAttnArgs = _struct("LatentAttnArgs", ("q cache page_indices kv_page_indptr qo_indptr kv_lens tok_req slots mask_bits "
                                             "mask_word_indptr out", p),
                          ("n heads row rank_pad cache_row page_size window_left", i32), ("scale", f32))
@@ -53,23 +54,30 @@ def stream_embed(tokens, table, ld: int, scale: float = 1.0):
 
 
 def stream_norm(x, width: int, eps: float, y=None, y_norm=None, norm_w=None, groups: int = 1, shift=None, rs=None, layer: int = 0,
-                dtype=None):
+                dtype=None, copy: bool = False):
     """Per token: x += y / rms(y) * y_norm (if y); h = RMSNorm(x) in `groups` parts * norm_w; hs = h + (h of the token
     before - h) * shift. The token before the first one of a portion comes from the sequence's state in `rs`
     (a `driver.recurrent.RecurrentInputs`), which advances. The gains (norm_w, y_norm) are in the activation type or, both,
-    in 32-bit; `dtype` then names the activation type. Returns (x, h, hs); what was not asked for is None."""
+    in 32-bit; `dtype` then names the activation type. `copy`: h = x in the activation type, without a norm (x itself where
+    that is 32-bit). Returns (x, h, hs); what was not asked for is None."""
     dtype = dtype or (norm_w if norm_w is not None else y).dtype
     if not x.is_cuda:
-        return ref.stream_norm(x, width, eps, y, y_norm, norm_w, groups, shift, rs, layer, dtype)
+        x, h, hs = ref.stream_norm(x, width, eps, y, y_norm, norm_w, groups, shift, rs, layer, dtype)
+        return x, x.to(dtype) if copy else h, hs
+    if copy and dtype == torch.float32:
+        if y is not None:
+            x = stream_norm(x, width, eps, y, y_norm, dtype=dtype)[0]
+        return x, x, None
     n, ld = x.shape
     new = lambda dt: torch.empty(n, ld, dtype=dt, device=x.device)
     x_out = new(torch.float32) if y is not None else None
-    h = new(dtype) if norm_w is not None else None
+    h = new(dtype) if norm_w is not None or copy else None
     hs = new(dtype) if shift is not None else None
     a = StreamNormArgs(x=ptr(x), y=ptr(y), y_norm=ptr(y_norm), x_out=ptr(x_out), norm_w=ptr(norm_w), shift=ptr(shift), h=ptr(h),
                        hs=ptr(hs), n=n, width=width, ldx=ld, ldy=y.stride(0) if y is not None else 0, ldh=ld, groups=groups,
                        rows_per_block=max(1, min(8, n // 592)), eps=eps)
-    commit, gain_f32 = 0, _f32(norm_w if norm_w is not None else y_norm)
+    gain = norm_w if norm_w is not None else y_norm
+    commit, gain_f32 = 0, _f32(gain) if gain is not None else 0
     if shift is not None:
         state = rs.shift_state[layer]
         a.tok_req, a.qo_indptr, a.slots, a.reset = ptr(rs.tok_req), ptr(rs.qo_indptr), ptr(rs.slots), ptr(rs.reset)
@@ -81,17 +89,20 @@ def stream_norm(x, width: int, eps: float, y=None, y_norm=None, norm_w=None, gro
     return (x if x_out is None else x_out), h, hs
 
 
-def latent_rows(qkv, positions, slots, inv_freq, norm_w, cache, spec, eps: float, q_width: int, q_rot: int, copy_nope: bool):
-    """Rotate the queries of the fused projection into rows [N, heads, q_width] (rotated part at column q_rot; with
-    `copy_nope` the unrotated part in front of it, else the columns before rank_pad are left for `per_head`), and write
-    the new tokens' cache rows: normalised latent, rotated shared key part. `cache` None: a layer that borrows rows."""
+def latent_rows(qkv, positions, slots, inv_freq, norm_w, cache, spec, eps: float, q_width: int, q_rot: int, copy_nope: bool, kv=None):
+    """Rotate the queries of a projection into rows [N, heads, q_width] (rotated part at column q_rot; with `copy_nope` the
+    unrotated part in front of it, else the columns before rank_pad are left for `per_head`), and write the new tokens'
+    cache rows: normalised latent, rotated shared key part. They are read from `kv` (latent | key part, may be a column
+    range), or from behind the queries. `cache` None: a layer that borrows rows."""
     n = qkv.shape[0]
     q = torch.empty(n, spec.heads, q_width, dtype=qkv.dtype, device=qkv.device)
+    if kv is None:
+        kv = qkv[:, spec.q_rows:]
     if not qkv.is_cuda:
-        return ref.latent_rows(qkv, positions, slots, inv_freq, norm_w, cache, spec, eps, q, q_rot, copy_nope)
-    a = LatentRowsArgs(qkv=ptr(qkv), positions=ptr(positions), slots=ptr(slots), inv_freq=ptr(inv_freq), norm_w=ptr(norm_w),
-                       q_out=ptr(q), cache=ptr(cache), n=n, ld=qkv.stride(0), heads=spec.heads, dim=spec.dim, rot_dim=spec.rot_dim,
-                       rot_dims=spec.rot_dims, rank=spec.kv_rank, rank_pad=spec.rank_pad,
+        return ref.latent_rows(qkv, kv, positions, slots, inv_freq, norm_w, cache, spec, eps, q, q_rot, copy_nope)
+    a = LatentRowsArgs(q=ptr(qkv), kv=ptr(kv), positions=ptr(positions), slots=ptr(slots), inv_freq=ptr(inv_freq), norm_w=ptr(norm_w),
+                       q_out=ptr(q), cache=ptr(cache), n=n, ld=qkv.stride(0), ld_kv=kv.stride(0), heads=spec.heads, dim=spec.dim,
+                       rot_dim=spec.rot_dim, rot_dims=spec.rot_dims, adjacent=1 if spec.rot_adjacent else 0, rot_factor=spec.rotary.factor, rank=spec.kv_rank, rank_pad=spec.rank_pad,
                        cache_row=cache.shape[-1] if cache is not None else 0, copy_nope=1 if copy_nope else 0, q_width=q_width,
                        q_rot=q_rot, q_zero=q_rot if copy_nope else spec.kv_rank, eps=eps)
     check(fn("pie_latent_rows")(C.byref(a), _f32(qkv), stream_ptr()), "latent_rows")

@@ -37,25 +37,29 @@ def stream_norm(x, width, eps, y, y_norm, norm_w, groups, shift, rs, layer, dtyp
     return x, h, hs
 
 
-def _rotate(x, positions, inv_freq):
+def rotate(x, positions, inv_freq, adjacent=False, factor=1.0):
+    """The first 2 * len(inv_freq) columns of x [N, ..., D] turned; halves of a pair adjacent or half the width apart."""
     half = inv_freq.numel()
     ang = positions.float()[:, None] * inv_freq.float()[None, :]
     ang = ang.reshape(ang.shape[0], *([1] * (x.dim() - 2)), half)
-    u, v = x[..., :half].float(), x[..., half:2 * half].float()
-    return torch.cat([u * ang.cos() - v * ang.sin(), v * ang.cos() + u * ang.sin(), x[..., 2 * half:].float()], -1)
+    c, s = ang.cos() * factor, ang.sin() * factor
+    r, rest = x[..., :2 * half].float(), x[..., 2 * half:].float()
+    u, v = (r[..., 0::2], r[..., 1::2]) if adjacent else (r[..., :half], r[..., half:])
+    a, b = u * c - v * s, v * c + u * s
+    return torch.cat([torch.stack([a, b], -1).flatten(-2) if adjacent else torch.cat([a, b], -1), rest], -1)
 
 
-def latent_rows(qkv, positions, slots, inv_freq, norm_w, cache, spec, eps, q, q_rot, copy_nope):
+def latent_rows(qkv, kv, positions, slots, inv_freq, norm_w, cache, spec, eps, q, q_rot, copy_nope):
     n, qk = qkv.shape[0], spec.qk_dim
     src = qkv[:, :spec.q_rows].reshape(n, spec.heads, qk)
     q.zero_()
     if copy_nope:
         q[..., :spec.dim] = src[..., :spec.dim]
-    q[..., q_rot:q_rot + spec.rot_dim] = _rotate(src[..., spec.dim:], positions, inv_freq).to(q.dtype)
+    q[..., q_rot:q_rot + spec.rot_dim] = rotate(src[..., spec.dim:], positions, inv_freq, spec.rot_adjacent, spec.rotary.factor).to(q.dtype)
     if cache is not None:
-        c = qkv[:, spec.q_rows:spec.q_rows + spec.kv_rank].float()
+        c = kv[:, :spec.kv_rank].float()
         c = c * torch.rsqrt(c.pow(2).mean(-1, keepdim=True) + eps) * norm_w.float()
-        kr = _rotate(qkv[:, spec.q_rows + spec.kv_rank:spec.proj_rows], positions, inv_freq)
+        kr = rotate(kv[:, spec.kv_rank:spec.kv_rank + spec.rot_dim], positions, inv_freq, spec.rot_adjacent, spec.rotary.factor)
         keep = slots >= 0
         rows = cache.view(-1, cache.shape[-1])
         sl = slots[keep].long()
