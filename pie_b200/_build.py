@@ -34,6 +34,10 @@ LATENT_SOURCES = ("attention_tc", "elementwise", "gemm2_tcgen05", "gemm_tcgen05"
 SANDWICH_SOURCES = ("attention_bias", "elementwise", "gdn", "gemm2_tcgen05", "gemm_tcgen05", "latent", "latent_attn", "linear_attn", "moe",
                     "sampling")
 
+# sources whose kernels blocks normed on the way out (grouped and latent attention, matrix memory) launch
+POST_NORM_SOURCES = ("attention", "attention_gqa", "attention_tc", "elementwise", "gdn", "gemm2_tcgen05", "gemm_tcgen05", "latent",
+                     "latent_attn", "latent_attn_tc", "linear_attn", "moe", "sampling")
+
 NVCC_FLAGS = [
     "-gencode", "arch=compute_100a,code=sm_100a", "-lineinfo", "-O3", "-std=c++17",
     "--expt-relaxed-constexpr", "-Xcompiler", "-fPIC", "-Xcompiler", "-fvisibility=hidden",
@@ -100,6 +104,8 @@ def kernels_for(cfg) -> Path:
         return KERNEL_LIB
     if cfg.latent is not None:
         return build_kernels(only=LATENT_SOURCES, target=OUT / "libpie_kernels_latent.so")
+    if cfg.blocks is not None and cfg.post_norm:
+        return build_kernels(only=POST_NORM_SOURCES, target=OUT / "libpie_kernels_post_norm.so")
     if cfg.blocks is not None:
         return build_kernels(only=SANDWICH_SOURCES, target=OUT / "libpie_kernels_sandwich.so")
     return build_kernels()

@@ -542,6 +542,27 @@ PIE_API int pie_brle_expand_ragged(const uint32_t* run_ends, const int* indptr, 
     return (int)cudaGetLastError();
 }
 
+// ------------------------------------------------------------ soft cap
+// y = cap * tanh(y / cap) in place, in 32-bit arithmetic; rows of `cols` at ld.
+namespace pie {
+template <typename T>
+__global__ void softcap_kernel(T* __restrict__ y, int cols, long ld, float cap) {
+    pdl_trigger();
+    pdl_wait();
+    T* row = y + blockIdx.y * ld;
+    for (int c = blockIdx.x * blockDim.x + threadIdx.x; c < cols; c += gridDim.x * blockDim.x)
+        row[c] = (T)(cap * tanhf((float)row[c] / cap));
+}
+}  // namespace pie
+
+PIE_API int pie_softcap(void* y, int rows, int cols, long ld, float cap, int f32, cudaStream_t st) {
+    if (rows <= 0 || cols <= 0) return 0;
+    if (cap <= 0.f || rows > 65535) return (int)cudaErrorInvalidValue;
+    const dim3 grid(min((cols + 255) / 256, 512), rows);
+    if (f32) return (int)pie::launch_pdl(pie::softcap_kernel<float>, grid, dim3(256), 0, st, (float*)y, cols, ld, cap);
+    return (int)pie::launch_pdl(pie::softcap_kernel<bf16>, grid, dim3(256), 0, st, (bf16*)y, cols, ld, cap);
+}
+
 // ------------------------------------------------------------- token feed
 // Decode pipelining: the input token of row i is the token sampled for row
 // src_row[i] by the previous step (still on the device), unless src_row[i] < 0,

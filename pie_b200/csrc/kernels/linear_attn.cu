@@ -1,6 +1,8 @@
 // Linear attention with a decaying state: per head S_t = diag(a_t) S_(t-1) + k_t v_t^T, o_t = S_t^T q_t, S in 32-bit
-// [dim][vdim], one state per (slot, head), carried from fire to fire. Two decays: one per key channel and token
-// (`log_decay`, base-2 logarithms, at most 0), or one constant per head.
+// [dim][vdim], one state per (slot, head), carried from fire to fire. Three decays: one per key channel and token
+// (`log_decay`, base-2 logarithms, at most 0), one constant per head, or one per head and token (`tok_decay`) beside a
+// factor on the token's key (`tok_input`). The last also carries a normaliser n, n_t = a_t n_(t-1) + k_t, after the states
+// of all heads, and returns n_t . q_t per token and head.
 //
 //   serial   token by token, S in registers: decode steps, and every shape in true 32-bit. A thread holds VEC columns of
 //            dim / 8 rows; the eight row groups meet in shared memory once per token.
@@ -24,16 +26,24 @@ struct LinAttnArgs {
     const void *q, *k, *v;       // row t, head h at t * ld + h * dim (h * vdim for v), type T
     float* log_decay;            // [n, heads * dim] base 2, or null; the chunked form leaves running sums of the pieces
     const float* head_decay;     // [heads] the factor itself (null with log_decay)
+    const float *tok_decay, *tok_input;   // [n, heads] base-2 logarithms of decay and key factor, at most 0 (null with the others)
+    float* den;                  // [n, heads] n_t . q_t (with tok_decay)
     float* out;                  // [n, heads * vdim]
     float* state;                // this layer's part of slot 0: [heads][dim][vdim]
     const int *qo_indptr, *slots, *reset;
     // chunked form
     const int *chunk_req, *chunk_start, *req_chunks;   // request and first row of a piece; pieces of a request (indptr)
-    float *u, *piece_decay;      // [chunks][heads][dim][vdim], [chunks][heads][dim] (base-2 logarithm)
+    float *u, *piece_decay;      // [chunks][heads][dim][vdim] (with tok_decay then [heads][dim]), [chunks][heads][dim] (base-2 logarithm)
     long slot_stride;
     int n, ld, reqs, heads, dim, vdim, silu, chunks;
     float q_scale;
 };
+
+enum LaDecay : int { LA_HEAD = 0, LA_CHANNEL = 1, LA_TOKEN = 2 };
+// 32-bit numbers of the state of one slot, or of one piece's update, that decay together
+__host__ __device__ __forceinline__ long la_elems(const LinAttnArgs& a) {
+    return (long)a.heads * a.dim * a.vdim + (a.tok_decay ? (long)a.heads * a.dim : 0);
+}
 
 // ------------------------------------------------------------------ serial
 template <typename T, int RPT, int VEC>
@@ -46,9 +56,11 @@ __global__ void __launch_bounds__(256) la_serial_kernel(const LinAttnArgs a) {
     const int r = blockIdx.x, h = blockIdx.y, lane = threadIdx.x & 31, rg = threadIdx.x >> 5;
     const int first = a.qo_indptr[r], len = a.qo_indptr[r + 1] - first, slot = a.slots[r];
     if (len <= 0 || slot < 0) return;          // a padding request of a decode graph: no state, no output
-    const int c0 = blockIdx.z * COLS + lane * VEC;
-    const bool col = c0 < a.vdim;              // VEC > 1 only where vdim is a multiple of it
-    float* sp = a.state + (size_t)slot * a.slot_stride + (size_t)h * a.dim * a.vdim;
+    // with a normaliser the last block of a head keeps it: one column whose values are ones
+    const bool ones = a.tok_decay && blockIdx.z == gridDim.z - 1;
+    const int width = ones ? 1 : a.vdim, cb = ones ? 0 : blockIdx.z * COLS, c0 = cb + lane * VEC;
+    const bool col = c0 < width;               // VEC > 1 only where vdim is a multiple of it
+    float* sp = a.state + (size_t)slot * a.slot_stride + (ones ? (size_t)a.heads * a.dim * a.vdim : 0) + (size_t)h * a.dim * width;
     float S[RPT][VEC];
     const bool fresh = a.reset[r] != 0;
 #pragma unroll
@@ -57,10 +69,11 @@ __global__ void __launch_bounds__(256) la_serial_kernel(const LinAttnArgs a) {
         const bool ok = col && !fresh && d < a.dim;
         if constexpr (VEC == 4) {
             float4 x = make_float4(0.f, 0.f, 0.f, 0.f);
-            if (ok) x = *reinterpret_cast<const float4*>(sp + (size_t)d * a.vdim + c0);
+            if (ok && ones) x.x = sp[d];
+            else if (ok) x = *reinterpret_cast<const float4*>(sp + (size_t)d * a.vdim + c0);
             S[i][0] = x.x; S[i][1] = x.y; S[i][2] = x.z; S[i][3] = x.w;
         } else {
-            S[i][0] = ok ? sp[(size_t)d * a.vdim + c0] : 0.f;
+            S[i][0] = ok ? sp[(size_t)d * width + c0] : 0.f;
         }
     }
     const float hd = a.head_decay ? a.head_decay[h] : 1.f;
@@ -68,21 +81,24 @@ __global__ void __launch_bounds__(256) la_serial_kernel(const LinAttnArgs a) {
         const size_t row = (size_t)(first + t);
         const T* qr = static_cast<const T*>(a.q) + row * a.ld + h * a.dim;
         const T* kr = static_cast<const T*>(a.k) + row * a.ld + h * a.dim;
+        const float td = a.tok_decay ? exp2f(a.tok_decay[row * a.heads + h]) : hd;
+        const float ti = a.tok_decay ? exp2f(a.tok_input[row * a.heads + h]) : 1.f;
         for (int d = threadIdx.x; d < ROWS; d += 256) {
             float q = 0.f, k = 0.f, g = 1.f;
             if (d < a.dim) {
                 q = to_f(qr[d]);
                 k = to_f(kr[d]);
                 if (a.silu) { q = la_silu(q); k = la_silu(k); }
-                g = a.log_decay ? exp2f(a.log_decay[row * a.heads * a.dim + h * a.dim + d]) : hd;
+                g = a.log_decay ? exp2f(a.log_decay[row * a.heads * a.dim + h * a.dim + d]) : td;
             }
             sq[d] = q * a.q_scale;
-            sk[d] = k;
+            sk[d] = k * ti;
             sa[d] = g;
         }
         float v[VEC];
 #pragma unroll
         for (int j = 0; j < VEC; ++j) {
+            if (ones) { v[j] = lane == 0 && j == 0 ? 1.f : 0.f; continue; }
             v[j] = col ? to_f(static_cast<const T*>(a.v)[row * a.ld + h * a.vdim + c0 + j]) : 0.f;
             if (a.silu) v[j] = la_silu(v[j]);
         }
@@ -104,19 +120,22 @@ __global__ void __launch_bounds__(256) la_serial_kernel(const LinAttnArgs a) {
         for (int j = 0; j < VEC; ++j) red[rg][lane * VEC + j] = o[j];
         __syncthreads();
         for (int c = threadIdx.x; c < COLS; c += 256) {
-            const int cc = blockIdx.z * COLS + c;
-            if (cc >= a.vdim) continue;
+            const int cc = cb + c;
+            if (cc >= width) continue;
             float s = 0.f;
 #pragma unroll
             for (int g = 0; g < 8; ++g) s += red[g][c];
-            a.out[row * a.heads * a.vdim + h * a.vdim + cc] = s;
+            if (ones) a.den[row * a.heads + h] = s;
+            else a.out[row * a.heads * a.vdim + h * a.vdim + cc] = s;
         }
     }
 #pragma unroll
     for (int i = 0; i < RPT; ++i) {
         const int d = rg + 8 * i;
         if (!col || d >= a.dim) continue;
-        if constexpr (VEC == 4)
+        if (ones)
+            sp[d] = S[i][0];
+        else if constexpr (VEC == 4)
             *reinterpret_cast<float4*>(sp + (size_t)d * a.vdim + c0) = make_float4(S[i][0], S[i][1], S[i][2], S[i][3]);
         else
             sp[(size_t)d * a.vdim + c0] = S[i][0];
@@ -187,10 +206,33 @@ struct ValueTile {
     }
 };
 
+// Running sum of the piece's token decays (sb[t]: decay from before the piece's first token to t) and its key factors, by
+// the first two warps; rows past the piece repeat its last sum and have no key.
+__device__ __forceinline__ void la_token_sums(const LinAttnArgs& a, int row0, int len, int h, float* sb, float* si, float* half) {
+    if (threadIdx.x < LA_C) {
+        const int s = threadIdx.x, lane = s & 31;
+        const size_t at = (size_t)(row0 + s) * a.heads + h;
+        float x = s < len ? a.tok_decay[at] : 0.f;
+        si[s] = s < len ? a.tok_input[at] : -INFINITY;
+#pragma unroll
+        for (int o = 1; o < 32; o <<= 1) {
+            const float y = __shfl_up_sync(0xffffffffu, x, o);
+            if (lane >= o) x += y;
+        }
+        if (s == 31) *half = x;
+        sb[s] = x;
+    }
+    __syncthreads();
+    if (threadIdx.x >= 32 && threadIdx.x < LA_C) sb[threadIdx.x] += *half;
+    __syncthreads();
+}
+
 // U and the piece's decay; turns log_decay into its running sum from the piece's start (in place), which la_chunk_out reads.
-template <bool CHAN, bool VEC>
-__global__ void __launch_bounds__(LA_THREADS, CHAN ? 2 : 3) la_chunk_state_kernel(const LinAttnArgs a) {
+template <int DEC, bool VEC>
+__global__ void __launch_bounds__(LA_THREADS, DEC == LA_CHANNEL ? 2 : 3) la_chunk_state_kernel(const LinAttnArgs a) {
+    constexpr bool CHAN = DEC == LA_CHANNEL;
     extern __shared__ __align__(16) float sm[];
+    __shared__ float tb[LA_C], ti[LA_C], th;
     const int c = blockIdx.x, h = blockIdx.y, r = a.chunk_req[c];
     const int row0 = a.chunk_start[c], len = min(LA_C, a.qo_indptr[r + 1] - row0);
     const int dimp = la_dimp(a.dim), kp = la_pitch(a.dim);
@@ -241,19 +283,31 @@ __global__ void __launch_bounds__(LA_THREADS, CHAN ? 2 : 3) la_chunk_state_kerne
             __syncthreads();               // `tot` is free for the next channels
         }
     } else {
-        const float lh = log2f(a.head_decay[h]);
+        if (DEC == LA_TOKEN) la_token_sums(a, row0, len, h, tb, ti, &th);
+        const float lh = DEC == LA_TOKEN ? 0.f : log2f(a.head_decay[h]);
+        const float whole = DEC == LA_TOKEN ? tb[LA_C - 1] : (float)len * lh;
         for (int u = threadIdx.x; u < LA_C * (dimp / 8); u += LA_THREADS) {
             const int s = u / (dimp / 8), d = (u - s * (dimp / 8)) * 8;
             float f[8];
             la_load8<VEC>(kb + (size_t)s * a.ld + d, s < len ? min(8, a.dim - d) : 0, a.silu, f);
-            const float w = s < len ? exp2f((float)(len - 1 - s) * lh) : 0.f;
+            const float w = s >= len ? 0.f : exp2f(DEC == LA_TOKEN ? whole - tb[s] + ti[s] : (float)(len - 1 - s) * lh);
 #pragma unroll
             for (int e = 0; e < 8; ++e) sk[s * kp + d + e] = tf32_f(f[e] * w);
         }
         for (int d = threadIdx.x; d < a.dim; d += LA_THREADS)
-            a.piece_decay[((size_t)c * a.heads + h) * a.dim + d] = (float)len * lh;
+            a.piece_decay[((size_t)c * a.heads + h) * a.dim + d] = whole;
     }
-    float* U = a.u + ((size_t)c * a.heads + h) * a.dim * a.vdim;
+    const long elems = la_elems(a);
+    float* U = a.u + c * elems + (size_t)h * a.dim * a.vdim;
+    if (DEC == LA_TOKEN) {
+        __syncthreads();
+        for (int d = threadIdx.x; d < a.dim; d += LA_THREADS) {
+            float x = 0.f;
+#pragma unroll 8
+            for (int s = 0; s < LA_C; ++s) x += sk[s * kp + d];
+            a.u[c * elems + (long)a.heads * a.dim * a.vdim + h * a.dim + d] = x;
+        }
+    }
     for (int v0 = 0; v0 < a.vdim; v0 += LA_VT) {
         __syncthreads();
         vt.template store<LA_VP>(sv);
@@ -294,7 +348,7 @@ template <int V>
 __global__ void __launch_bounds__(256) la_chunk_scan_kernel(const LinAttnArgs a) {
     const int r = blockIdx.y, slot = a.slots[r];
     const int c0 = a.req_chunks[r], c1 = a.req_chunks[r + 1];
-    const long elems = (long)a.heads * a.dim * a.vdim, i = (blockIdx.x * 256L + threadIdx.x) * V;
+    const long elems = la_elems(a), states = (long)a.heads * a.dim * a.vdim, i = (blockIdx.x * 256L + threadIdx.x) * V;
     if (i >= elems || c1 <= c0 || slot < 0) return;
     float* sp = a.state + (size_t)slot * a.slot_stride + i;
     float s[V];
@@ -303,7 +357,8 @@ __global__ void __launch_bounds__(256) la_chunk_scan_kernel(const LinAttnArgs a)
 #pragma unroll
         for (int e = 0; e < V; ++e) s[e] = 0.f;
     float* u = a.u + i;
-    const float* dec = a.piece_decay + i / a.vdim;
+    // the V elements share a factor, also in the normaliser, whose neighbours are channels of one head (V divides dim)
+    const float* dec = a.piece_decay + (i < states ? i / a.vdim : i - states);
     const long dstep = (long)a.heads * a.dim;
     constexpr int AHEAD = 8;
     for (int c = c0; c < c1; c += AHEAD) {
@@ -342,9 +397,11 @@ struct LaOutSmem {
     }
 };
 
-template <bool CHAN, bool VEC>
+template <int DEC, bool VEC>
 __global__ void __launch_bounds__(LA_THREADS) la_chunk_out_kernel(const LinAttnArgs a) {
+    constexpr bool CHAN = DEC == LA_CHANNEL;
     extern __shared__ __align__(16) float sm[];
+    __shared__ float tb[LA_C], ti[LA_C], th;
     const LaOutSmem lay(a.dim);
     const int c = blockIdx.x, h = blockIdx.y, r = a.chunk_req[c];
     const int row0 = a.chunk_start[c], len = min(LA_C, a.qo_indptr[r + 1] - row0);
@@ -358,7 +415,8 @@ __global__ void __launch_bounds__(LA_THREADS) la_chunk_out_kernel(const LinAttnA
     float* ss = reinterpret_cast<float*>(base + lay.s);        // [dimp][LA_VP] a tile of the state
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, g = lane >> 2, t = lane & 3;
     const int rb = warp & 3, half = warp >> 2, w0 = rb * 16;   // 16 query rows per warp; two warps share them
-    const float lh = CHAN ? 0.f : log2f(a.head_decay[h]);
+    const float lh = DEC == LA_HEAD ? log2f(a.head_decay[h]) : 0.f;
+    if (DEC == LA_TOKEN) la_token_sums(a, row0, len, h, tb, ti, &th);
     const bf16* qb = static_cast<const bf16*>(a.q) + (size_t)row0 * a.ld + h * a.dim;
     const bf16* kb = static_cast<const bf16*>(a.k) + (size_t)row0 * a.ld + h * a.dim;
     const bf16* vb = static_cast<const bf16*>(a.v) + (size_t)row0 * a.ld + h * a.vdim;
@@ -384,7 +442,7 @@ __global__ void __launch_bounds__(LA_THREADS) la_chunk_out_kernel(const LinAttnA
         }
     }
     // the first tiles of values and state are on their way while the scores are formed
-    const float* S = a.u + ((size_t)c * a.heads + h) * a.dim * a.vdim;
+    const float* S = a.u + c * la_elems(a) + (size_t)h * a.dim * a.vdim;
     ValueTile<VEC> vt;
     vt.load(vb, a.ld, len, a.vdim, a.silu);
     __syncthreads();
@@ -452,7 +510,7 @@ __global__ void __launch_bounds__(LA_THREADS) la_chunk_out_kernel(const LinAttnA
         for (int e = 0; e < 4; ++e) {
             const int q = w0 + g + (e >> 1) * 8, s = J * 16 + half * 8 + 2 * t + (e & 1);
             if (s > q) { acc[n][e] = 0.f; continue; }
-            if (!CHAN) acc[n][e] *= exp2f((float)(q - s) * lh);
+            if (!CHAN) acc[n][e] *= exp2f(DEC == LA_TOKEN ? tb[q] - tb[s] + ti[s] : (float)(q - s) * lh);
             if (CHAN && exact && n == 3) {
                 float x = 0.f;
                 for (int d = 0; d < dimp; ++d)
@@ -476,9 +534,21 @@ __global__ void __launch_bounds__(LA_THREADS) la_chunk_out_kernel(const LinAttnA
         const int s = u / vecs, d = (u - s * vecs) * 8;
         float f[8];
         unpack8(*reinterpret_cast<const bf16x8*>(sq + s * kp + d), f);
-        const float w = CHAN ? 0.f : exp2f((float)(s + 1) * lh);
+        const float w = CHAN ? 0.f : exp2f(DEC == LA_TOKEN ? tb[s] : (float)(s + 1) * lh);
 #pragma unroll
         for (int e = 0; e < 8; ++e) sb[s * xp + d + e] = tf32_f(CHAN ? f[e] * exp2f(sb[s * xp + d + e]) : f[e] * w);
+    }
+    if (DEC == LA_TOKEN) {
+        // n_t . q_t: the row's scores, and its decayed query against the normaliser before the piece; four threads per row
+        __syncthreads();
+        const int q = threadIdx.x >> 2, part = threadIdx.x & 3;
+        const float* N = a.u + c * la_elems(a) + (size_t)a.heads * a.dim * a.vdim + (size_t)h * a.dim;
+        float x = 0.f;
+        for (int s = part; s <= q; s += 4) x += sc[q * LA_SP + s];
+        for (int d = part; d < a.dim; d += 4) x += sb[q * xp + d] * N[d];
+        x += __shfl_xor_sync(0xffffffffu, x, 1);
+        x += __shfl_xor_sync(0xffffffffu, x, 2);
+        if (part == 0 && q < len) a.den[(size_t)(row0 + q) * a.heads + h] = x * a.q_scale;
     }
     constexpr int SV = LA_VT / 4;                 // 16-byte pieces of a state row
     for (int v0 = 0; v0 < a.vdim; v0 += LA_VT) {
@@ -575,15 +645,107 @@ __global__ void __launch_bounds__(256) la_decay_kernel(const T* __restrict__ x, 
         if (s < nt) out[(size_t)(t0 + s) * channels + c] = (fminf(z[s], 0.f) - log1pf(expf(-fabsf(z[s])))) * (1.4426950408889634f * inv_tau);
 }
 
+// ------------------------------------------- exponential gates of a matrix memory
+// Per head logarithms i = cap tanh(z_i / cap) and f = logsigmoid(cap tanh(z_f / cap)) of the input and forget gates, and a
+// running maximum m_t = max(f_t + m_(t-1), i_t), m from 0, that takes the size out of the state: decay exp(f_t + m_(t-1) -
+// m_t), key factor exp(i_t - m_t), both at most 1.
+struct MemoryGatesArgs {
+    const float *z, *bias;          // `splits` arrays [n, ldz] that add up to (z_i | z_f), heads columns each; [2 * heads]
+    const int *qo_indptr, *slots, *reset, *tok_req;
+    float* m;                       // this layer's maxima of slot 0, [heads]
+    float *decay, *input, *floor;   // [n, heads] base-2 logarithms; exp(-m_t)
+    long slot_stride, split_stride;
+    int n, reqs, heads, ldz, splits;
+    float cap;
+};
+
+struct MemoryGate { float i, f; };
+__device__ __forceinline__ MemoryGate memory_gate(const MemoryGatesArgs& a, size_t t, int h) {
+    float zi = a.bias[h], zf = a.bias[a.heads + h];
+    for (int s = 0; s < a.splits; ++s) {
+        zi += a.z[s * a.split_stride + t * a.ldz + h];
+        zf += a.z[s * a.split_stride + t * a.ldz + a.heads + h];
+    }
+    const float x = a.cap * tanhf(zf / a.cap);
+    return {a.cap * tanhf(zi / a.cap), fminf(x, 0.f) - log1pf(expf(-fabsf(x)))};
+}
+// Writes a token's factors and returns the new maximum.
+__device__ __forceinline__ float memory_step(const MemoryGatesArgs& a, size_t at, MemoryGate g, float m) {
+    const float kept = g.f + m, next = fmaxf(kept, g.i);
+    a.decay[at] = (kept - next) * 1.4426950408889634f;
+    a.input[at] = (g.i - next) * 1.4426950408889634f;
+    a.floor[at] = expf(-next);
+    return next;
+}
+
+// One token per request: a thread per (request, head). Rows without a slot (padding of a decode graph) get zeros.
+__global__ void __launch_bounds__(128) memory_gates_step_kernel(const MemoryGatesArgs a) {
+    pdl_trigger();
+    pdl_wait();
+    const int i = blockIdx.x * 128 + threadIdx.x;
+    if (i >= a.reqs * a.heads) return;
+    const int r = i / a.heads, h = i - r * a.heads, t = a.qo_indptr[r], slot = a.slots[r];
+    if (a.qo_indptr[r + 1] <= t) return;
+    const size_t at = (size_t)t * a.heads + h;
+    if (slot < 0) { a.decay[at] = a.input[at] = a.floor[at] = 0.f; return; }
+    float* m = a.m + (size_t)slot * a.slot_stride + h;
+    *m = memory_step(a, at, memory_gate(a, t, h), a.reset[r] ? 0.f : *m);
+}
+
+// Portions: a block per (request, head). m_t is a composition of maps m -> max(m + F, B): threads compose theirs over equal
+// runs of tokens, a scan over the threads gives each the maximum before its run, which it then walks.
+__global__ void __launch_bounds__(256) memory_gates_kernel(const MemoryGatesArgs a) {
+    __shared__ float sF[8], sB[8];
+    pdl_trigger();
+    pdl_wait();
+    const int r = blockIdx.x, h = blockIdx.y, first = a.qo_indptr[r], len = a.qo_indptr[r + 1] - first, slot = a.slots[r];
+    if (len <= 0 || slot < 0) return;
+    for (int s = threadIdx.x; s < len; s += 256) {
+        const MemoryGate g = memory_gate(a, first + s, h);
+        const size_t at = (size_t)(first + s) * a.heads + h;
+        a.decay[at] = g.f;
+        a.input[at] = g.i;
+    }
+    __syncthreads();
+    const int run = (len + 255) / 256, s0 = min(len, (int)threadIdx.x * run), s1 = min(len, s0 + run);
+    float F = 0.f, B = -INFINITY;
+    for (int s = s0; s < s1; ++s) {
+        const size_t at = (size_t)(first + s) * a.heads + h;
+        F += a.decay[at];
+        B = fmaxf(B + a.decay[at], a.input[at]);
+    }
+    const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
+#pragma unroll
+    for (int o = 1; o < 32; o <<= 1) {               // after the maps of earlier lanes
+        const float pF = __shfl_up_sync(0xffffffffu, F, o), pB = __shfl_up_sync(0xffffffffu, B, o);
+        if (lane >= o) { B = fmaxf(pB + F, B); F += pF; }
+    }
+    if (lane == 31) { sF[warp] = F; sB[warp] = B; }
+    float* mp = a.m + (size_t)slot * a.slot_stride + h;
+    float m = a.reset[r] ? 0.f : *mp;
+    const float eF = __shfl_up_sync(0xffffffffu, F, 1), eB = __shfl_up_sync(0xffffffffu, B, 1);
+    __syncthreads();
+    for (int w = 0; w < warp; ++w) m = fmaxf(m + sF[w], sB[w]);
+    if (lane) m = fmaxf(m + eF, eB);
+    for (int s = s0; s < s1; ++s) {
+        const size_t at = (size_t)(first + s) * a.heads + h;
+        m = memory_step(a, at, {a.input[at], a.decay[at]}, m);
+    }
+    if (s1 == len && s0 < len) *mp = m;
+}
+
 // -------------------------------------------------------- norm and gate of a mixer's output
 // dst[t, :] = scale * act(gate) * (rms-normed x) [* w]; the mean square runs over `norm_cols` consecutive columns (0: no
-// norm). Column j of the output is column (head / group * group_pad + head % group) * head_ld + j % head_cols of x, so that
-// x may hold padded heads. Columns from cols to dst_cols are written as zeros.
+// norm). gate: one number per `gate_cols` columns, or null. den / floor [n, groups of norm_cols]: what is normed is
+// x / (max(|den|, floor) + 1e-6), whose division the norm takes up. Column j of the output is column
+// (head / group * group_pad + head % group) * head_ld + j % head_cols of x, so that x may hold padded heads. Columns from cols
+// to dst_cols are written as zeros.
 struct GatedNormPart {
     const void* x;
     const void *w, *gate;
     void* dst;
-    int x_f32, ldx, head_cols, head_ld, group, group_pad, norm_cols, w_cols, ldg, ldd, cols, dst_cols, act;   // act 0: sigmoid, 1: SiLU
+    const float *den, *floor;
+    int x_f32, ldx, head_cols, head_ld, group, group_pad, norm_cols, w_cols, ldg, gate_cols, ldd, cols, dst_cols, act;   // act 0: sigmoid, 1: SiLU
     float eps, scale;
 };
 struct GatedNormArgs {
@@ -612,14 +774,29 @@ __global__ void __launch_bounds__(256) la_gated_norm_kernel(const GatedNormArgs 
     };
     auto finish = [&](int j, float (&v)[VEC], float inv, int wcol) {
         float z[VEC], gain[VEC];
-        load_vec<VEC>(gate + j, z);
+        if (!p.gate) {
+#pragma unroll
+            for (int e = 0; e < VEC; ++e) z[e] = 0.f;
+        } else if (p.gate_cols == 1) {
+            load_vec<VEC>(gate + j, z);
+        } else {                                // VEC divides gate_cols
+            const float g = to_f(gate[j / p.gate_cols]);
+#pragma unroll
+            for (int e = 0; e < VEC; ++e) z[e] = g;
+        }
         if (w) load_vec<VEC>(w + wcol, gain);
 #pragma unroll
         for (int e = 0; e < VEC; ++e) {
             const float s = 1.f / (1.f + __expf(-z[e]));
-            v[e] = v[e] * (w ? inv * gain[e] : 1.f) * (p.act ? z[e] * s : s) * p.scale;
+            v[e] = v[e] * (w ? inv * gain[e] : 1.f) * (p.gate ? (p.act ? z[e] * s : s) : 1.f) * p.scale;
         }
         store_vec<VEC>(dst + j, v);
+    };
+    auto squared_size = [&](int group) {
+        if (!p.den) return 1.f;
+        const size_t at = (size_t)t * (p.cols / p.norm_cols) + group;
+        const float d = fmaxf(fabsf(p.den[at]), p.floor[at]) + 1e-6f;
+        return d * d;
     };
     const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
     if (p.norm_cols == 0) {
@@ -637,7 +814,7 @@ __global__ void __launch_bounds__(256) la_gated_norm_kernel(const GatedNormArgs 
 #pragma unroll
             for (int e = 0; e < VEC; ++e) ss += v[e] * v[e];
         }
-        const float inv = 1.f / sqrtf(block_sum(ss, buf) / (float)p.cols + p.eps);
+        const float inv = 1.f / sqrtf(block_sum(ss, buf) / (float)p.cols + p.eps * squared_size(0));
         for (int j = threadIdx.x * VEC; j < p.cols; j += 256 * VEC) {
             float v[VEC];
             load_vec<VEC>(buf + 32 + j, v);
@@ -652,7 +829,7 @@ __global__ void __launch_bounds__(256) la_gated_norm_kernel(const GatedNormArgs 
 #pragma unroll
                 for (int e = 0; e < VEC; ++e) ss += v[e] * v[e];
             }
-            const float inv = 1.f / sqrtf(warp_sum(ss) / (float)p.norm_cols + p.eps);
+            const float inv = 1.f / sqrtf(warp_sum(ss) / (float)p.norm_cols + p.eps * squared_size(gr));
             for (int j = lane * VEC; j < p.norm_cols; j += 32 * VEC) {
                 float v[VEC];
                 source(gr * p.norm_cols + j, v);
@@ -667,13 +844,17 @@ __global__ void __launch_bounds__(256) la_gated_norm_kernel(const GatedNormArgs 
 
 using namespace pie;
 
+static bool la_decay_ok(const LinAttnArgs& a) {
+    return (a.log_decay != nullptr) + (a.head_decay != nullptr) + (a.tok_decay != nullptr) == 1 && (!a.tok_decay || (a.tok_input && a.den));
+}
+
 PIE_API int pie_linear_attn_serial(const LinAttnArgs* args, int f32, cudaStream_t st) {
     const LinAttnArgs& a = *args;
     if (a.n <= 0 || a.reqs <= 0) return 0;
-    if (a.dim <= 0 || a.dim > 512 || a.vdim <= 0 || (!a.log_decay && !a.head_decay)) return (int)cudaErrorInvalidValue;
+    if (a.dim <= 0 || a.dim > 512 || a.vdim <= 0 || !la_decay_ok(a)) return (int)cudaErrorInvalidValue;
     const bool vec = a.vdim % 4 == 0 && a.vdim >= 64 && a.dim <= 256 && a.slot_stride % 4 == 0 && ((uintptr_t)a.state & 15) == 0;
     const int cols = vec ? 128 : 32, rpt = (a.dim + 7) / 8;
-    const dim3 grid(a.reqs, a.heads, (a.vdim + cols - 1) / cols);
+    const dim3 grid(a.reqs, a.heads, (a.vdim + cols - 1) / cols + (a.tok_decay ? 1 : 0));
 #define GO(T_, R_, V_)                                                                                  \
     return (int)launch_pdl(la_serial_kernel<T_, R_, V_>, grid, dim3(256), 0, st, a)
 #define GO_R(T_)                                                                                        \
@@ -697,29 +878,31 @@ PIE_API int pie_linear_attn_serial(const LinAttnArgs* args, int f32, cudaStream_
 static size_t la_state_smem(int dim) { return ((size_t)LA_C * (la_pitch(dim) + LA_VP) + 128) * 4; }
 // 1 when the chunked form takes heads of this key size.
 PIE_API int pie_linear_attn_chunk_supported(int dim) {
-    return dim > 0 && LaOutSmem(dim).total <= 227 * 1024 && la_state_smem(dim) <= 227 * 1024 ? 1 : 0;
+    return dim > 0 && LaOutSmem(dim).total <= 226 * 1024 && la_state_smem(dim) <= 226 * 1024 ? 1 : 0;
 }
 PIE_API int pie_linear_attn_chunk_tokens() { return LA_C; }
 
 PIE_API int pie_linear_attn_chunked(const LinAttnArgs* args, cudaStream_t st) {
     const LinAttnArgs& a = *args;
     if (a.n <= 0 || a.reqs <= 0 || a.chunks <= 0) return 0;
-    if (!pie_linear_attn_chunk_supported(a.dim) || a.vdim <= 0 || (!a.log_decay && !a.head_decay) || !a.u || !a.piece_decay)
+    if (!pie_linear_attn_chunk_supported(a.dim) || a.vdim <= 0 || !la_decay_ok(a) || !a.u || !a.piece_decay)
         return (int)cudaErrorInvalidValue;
     auto aligned = [](const void* p) { return ((uintptr_t)p & 15) == 0; };
     const bool vec = a.dim % 8 == 0 && a.vdim % 8 == 0 && a.ld % 8 == 0 && aligned(a.q) && aligned(a.k) && aligned(a.v) && aligned(a.log_decay) &&
                      aligned(a.u) && aligned(a.out) && aligned(a.state) && a.slot_stride % 4 == 0;
     const dim3 grid(a.chunks, a.heads);
     const size_t s1 = la_state_smem(a.dim), s3 = LaOutSmem(a.dim).total;
-    auto k1 = a.log_decay ? (vec ? la_chunk_state_kernel<true, true> : la_chunk_state_kernel<true, false>)
-                          : (vec ? la_chunk_state_kernel<false, true> : la_chunk_state_kernel<false, false>);
-    auto k3 = a.log_decay ? (vec ? la_chunk_out_kernel<true, true> : la_chunk_out_kernel<true, false>)
-                          : (vec ? la_chunk_out_kernel<false, true> : la_chunk_out_kernel<false, false>);
+    auto k1 = a.tok_decay ? (vec ? la_chunk_state_kernel<LA_TOKEN, true> : la_chunk_state_kernel<LA_TOKEN, false>)
+            : a.log_decay ? (vec ? la_chunk_state_kernel<LA_CHANNEL, true> : la_chunk_state_kernel<LA_CHANNEL, false>)
+                          : (vec ? la_chunk_state_kernel<LA_HEAD, true> : la_chunk_state_kernel<LA_HEAD, false>);
+    auto k3 = a.tok_decay ? (vec ? la_chunk_out_kernel<LA_TOKEN, true> : la_chunk_out_kernel<LA_TOKEN, false>)
+            : a.log_decay ? (vec ? la_chunk_out_kernel<LA_CHANNEL, true> : la_chunk_out_kernel<LA_CHANNEL, false>)
+                          : (vec ? la_chunk_out_kernel<LA_HEAD, true> : la_chunk_out_kernel<LA_HEAD, false>);
     cudaError_t e = cudaFuncSetAttribute(k1, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)s1);
     if (e == cudaSuccess) e = cudaFuncSetAttribute(k3, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)s3);
     if (e != cudaSuccess) return (int)e;
     k1<<<grid, LA_THREADS, s1, st>>>(a);
-    const long elems = (long)a.heads * a.dim * a.vdim / (vec ? 4 : 1);
+    const long elems = la_elems(a) / (vec ? 4 : 1);
     const dim3 sgrid((unsigned)((elems + 255) / 256), a.reqs);
     if (vec) la_chunk_scan_kernel<4><<<sgrid, 256, 0, st>>>(a);
     else la_chunk_scan_kernel<1><<<sgrid, 256, 0, st>>>(a);
@@ -740,6 +923,15 @@ PIE_API int pie_linear_decay(const void* x, int ld, const void* a2, const void* 
                            channels, rank, inv_tau);
 }
 
+// single: every request brings one token.
+PIE_API int pie_memory_gates(const MemoryGatesArgs* args, int single, cudaStream_t st) {
+    const MemoryGatesArgs& a = *args;
+    if (a.n <= 0 || a.reqs <= 0) return 0;
+    if (a.heads <= 0 || a.cap <= 0.f || a.splits < 1) return (int)cudaErrorInvalidValue;
+    if (single) return (int)launch_pdl(memory_gates_step_kernel, dim3((a.reqs * a.heads + 127) / 128), dim3(128), 0, st, a);
+    return (int)launch_pdl(memory_gates_kernel, dim3(a.reqs, a.heads), dim3(256), 0, st, a);
+}
+
 // One or two parts (parts: 1 or 2) over the same tokens.
 PIE_API int pie_gated_norm(const GatedNormArgs* args, int parts, int f32, cudaStream_t st) {
     const GatedNormArgs& a = *args;
@@ -750,11 +942,13 @@ PIE_API int pie_gated_norm(const GatedNormArgs* args, int parts, int f32, cudaSt
     auto aligned = [](const void* p) { return ((uintptr_t)p & 15) == 0; };
     for (int i = 0; i < parts; ++i) {
         const GatedNormPart& p = a.part[i];
-        if (p.head_cols <= 0 || p.group <= 0 || p.cols <= 0 || (p.norm_cols && (p.cols % p.norm_cols || !p.w || p.w_cols <= 0)))
+        if (p.head_cols <= 0 || p.group <= 0 || p.cols <= 0 || p.gate_cols <= 0 || (p.den && (!p.floor || !p.norm_cols)) ||
+            (p.norm_cols && (p.cols % p.norm_cols || !p.w || p.w_cols <= 0)))
             return (int)cudaErrorInvalidValue;
         if (p.norm_cols == p.cols) sm = (size_t)(32 + p.cols) * 4 > sm ? (size_t)(32 + p.cols) * 4 : sm;
         vec = vec && p.head_cols % 4 == 0 && p.head_ld % 4 == 0 && p.norm_cols % 4 == 0 && (!p.w || p.w_cols % 4 == 0) &&
-              p.cols % 4 == 0 && p.ldx % 4 == 0 && p.ldg % 4 == 0 && p.ldd % 4 == 0 && aligned(p.x) && aligned(p.gate) &&
+              (p.gate_cols == 1 || p.gate_cols % 4 == 0) && p.cols % 4 == 0 && p.ldx % 4 == 0 &&
+              (p.gate_cols > 1 || (p.ldg % 4 == 0 && aligned(p.gate))) && p.ldd % 4 == 0 && aligned(p.x) &&
               aligned(p.dst) && aligned(p.w);
     }
     if (sm > 227 * 1024) return (int)cudaErrorInvalidValue;

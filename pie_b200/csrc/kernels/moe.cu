@@ -26,12 +26,15 @@ constexpr int MOE_TILE = 128;
 // ids receives the expert index relative to e_lo, or -1 for an expert outside [e_lo, e_lo+e_cnt)
 // (expert parallelism: those routes belong to another rank and take no slot here).
 // SCORED: experts are chosen by probability + `correction` and weighted by the probability alone (never renormalised); the
-// logits are `splits` fp32 arrays, split_stride apart, that add up to them.
-template <typename T, bool SCORED = false>
+// logits are `splits` fp32 arrays, split_stride apart, that add up to them. SIGMOID: the same with the sigmoid of each logit
+// for a score and no correction (the choice looks at the logits themselves, which saturated scores no longer tell apart).
+enum MoeScore : int { MOE_SOFTMAX = 0, MOE_SCORED = 1, MOE_SIGMOID = 2 };
+template <typename T, int SCORE = MOE_SOFTMAX>
 __global__ void moe_route_kernel(const T* __restrict__ logits, int ld, int n, int E, int k, int renorm,
                                  int e_lo, int e_cnt, int* __restrict__ ids, float* __restrict__ w,
                                  int* __restrict__ pos, int* __restrict__ counts, const float* __restrict__ correction = nullptr,
                                  int splits = 1, long split_stride = 0) {
+    constexpr bool SCORED = SCORE != MOE_SOFTMAX, SIGMOID = SCORE == MOE_SIGMOID;
     const int warp = (blockIdx.x * blockDim.x + threadIdx.x) >> 5, lane = threadIdx.x & 31;
     if (warp >= n) return;
     const T* row = logits + (size_t)warp * ld;
@@ -49,17 +52,18 @@ __global__ void moe_route_kernel(const T* __restrict__ logits, int ld, int n, in
     float sum = 0.f;
 #pragma unroll
     for (int i = 0; i < MOE_MAX_E / 32; ++i) {
+        if (SIGMOID) break;
         v[i] = (i * 32 + lane) < E ? (SCORED ? expf(v[i] - mx) : __expf(v[i] - mx)) : -1.f;   // -1 = excluded
         if (v[i] > 0.f) sum += v[i];
     }
-    sum = warp_sum(sum);
+    sum = SIGMOID ? 1.f : warp_sum(sum);
     float prob[SCORED ? MOE_MAX_E / 32 : 1];
     if (SCORED) {
 #pragma unroll
         for (int i = 0; i < MOE_MAX_E / 32; ++i) {
             const int e = i * 32 + lane;
-            prob[i] = v[i];
-            v[i] = e < E ? v[i] / sum + correction[e] : -INFINITY;
+            prob[i] = SIGMOID ? 1.f / (1.f + expf(-v[i])) : v[i];
+            if (!SIGMOID) v[i] = e < E ? v[i] / sum + correction[e] : -INFINITY;
         }
     }
     float picked_sum = 0.f;
@@ -131,11 +135,11 @@ __global__ void moe_align_kernel(int* __restrict__ counts, int E, int max_mtiles
     for (int t = start_of[E] + tid; t < max_mtiles; t += blockDim.x) tile_expert[t] = -1;
 }
 
-// One block per route: xs[slot] = x[token]; routes of experts that are not local (ids < 0) take
+// One block per route: xs[slot] = x[token], times the route's weight with `scale`; routes of experts that are not local (ids < 0) take
 // no slot.
 __global__ void moe_permute_kernel(const bf16* __restrict__ x, int ldx, const int* __restrict__ ids,
                                    const int* __restrict__ pos, const int* __restrict__ seg_start, int H, int k,
-                                   bf16* __restrict__ xs, int* __restrict__ slot_of) {
+                                   bf16* __restrict__ xs, int* __restrict__ slot_of, const float* __restrict__ scale) {
     const int route = blockIdx.x;
     const int e = ids[route];
     if (e < 0) {
@@ -146,7 +150,18 @@ __global__ void moe_permute_kernel(const bf16* __restrict__ x, int ldx, const in
     if (threadIdx.x == 0) slot_of[route] = slot;
     const bf16x8* src = reinterpret_cast<const bf16x8*>(x + (size_t)(route / k) * ldx);
     bf16x8* dst = reinterpret_cast<bf16x8*>(xs + (size_t)slot * H);
-    for (int c = threadIdx.x; c < H / 8; c += blockDim.x) dst[c] = src[c];
+    if (!scale) {
+        for (int c = threadIdx.x; c < H / 8; c += blockDim.x) dst[c] = src[c];
+        return;
+    }
+    const float w = scale[route];
+    for (int c = threadIdx.x; c < H / 8; c += blockDim.x) {
+        float f[8];
+        unpack8(src[c], f);
+#pragma unroll
+        for (int i = 0; i < 8; ++i) f[i] *= w;
+        dst[c] = pack8(f);
+    }
 }
 
 // One block per token. `self`: a route without a slot is an expert that returns its input, row t of `self`.
@@ -175,7 +190,7 @@ __global__ void moe_combine_kernel(const bf16* __restrict__ y, const int* __rest
         for (int j = 0; j < k; ++j) {
             const int slot = slot_of[(size_t)t * k + j];
             if (slot < 0 && !self) continue;
-            const float wj = w[(size_t)t * k + j];
+            const float wj = w ? w[(size_t)t * k + j] : 1.f;
             float v[8];
             unpack8(*reinterpret_cast<const bf16x8*>(slot < 0 ? self + (size_t)t * lds + c * 8 : y + (size_t)slot * H + c * 8), v);
 #pragma unroll
@@ -213,8 +228,19 @@ PIE_API int pie_moe_route_scored(const float* logits, int splits, long split_str
     if (n <= 0) return 0;
     if (E > MOE_MAX_E || k > 32 || k > E || k <= 0 || splits < 1 || !correction || e_cnt > E) return (int)cudaErrorInvalidValue;
     const int threads = 128, blocks = (n * 32 + threads - 1) / threads;
-    moe_route_kernel<float, true><<<blocks, threads, 0, st>>>(logits, ld, n, E, k, 0, 0, e_cnt, ids, w, pos, counts, correction, splits,
+    moe_route_kernel<float, MOE_SCORED><<<blocks, threads, 0, st>>>(logits, ld, n, E, k, 0, 0, e_cnt, ids, w, pos, counts, correction, splits,
                                                               split_stride);
+    return (int)cudaGetLastError();
+}
+
+// Routing by the sigmoid of each of E outputs, weights not renormalised.
+PIE_API int pie_moe_route_sigmoid(const float* logits, int splits, long split_stride, int ld, int n, int E, int k, int* ids, float* w,
+                                  int* pos, int* counts, cudaStream_t st) {
+    if (n <= 0) return 0;
+    if (E > MOE_MAX_E || k > 32 || k > E || k <= 0 || splits < 1) return (int)cudaErrorInvalidValue;
+    const int threads = 128, blocks = (n * 32 + threads - 1) / threads;
+    moe_route_kernel<float, MOE_SIGMOID><<<blocks, threads, 0, st>>>(logits, ld, n, E, k, 0, 0, E, ids, w, pos, counts, nullptr, splits,
+                                                                     split_stride);
     return (int)cudaGetLastError();
 }
 
@@ -229,10 +255,20 @@ PIE_API int pie_moe_permute(const void* x, int ldx, const int* ids, const int* p
                             int H, int k, void* xs, int* slot_of, cudaStream_t st) {
     if (n <= 0) return 0;
     if (H % 8 || ldx % 8) return (int)cudaErrorInvalidValue;
-    moe_permute_kernel<<<n * k, 128, 0, st>>>((const bf16*)x, ldx, ids, pos, seg_start, H, k, (bf16*)xs, slot_of);
+    moe_permute_kernel<<<n * k, 128, 0, st>>>((const bf16*)x, ldx, ids, pos, seg_start, H, k, (bf16*)xs, slot_of, nullptr);
     return (int)cudaGetLastError();
 }
 
+// The same with every row times its route's weight `w` (an expert's weight scales what it reads); combine then takes w = null.
+PIE_API int pie_moe_permute_weighted(const void* x, int ldx, const int* ids, const int* pos, const int* seg_start, const float* w, int n,
+                                     int H, int k, void* xs, int* slot_of, cudaStream_t st) {
+    if (n <= 0) return 0;
+    if (H % 8 || ldx % 8 || !w) return (int)cudaErrorInvalidValue;
+    moe_permute_kernel<<<n * k, 128, 0, st>>>((const bf16*)x, ldx, ids, pos, seg_start, H, k, (bf16*)xs, slot_of, w);
+    return (int)cudaGetLastError();
+}
+
+// w null: the weights are ones.
 PIE_API int pie_moe_combine(const void* y, const int* slot_of, const float* w, const void* residual, int ldr, int n,
                             int H, int k, void* out, int ldo, cudaStream_t st) {
     if (n <= 0) return 0;

@@ -210,9 +210,9 @@ class TorchDriver:
         self.max_items = max_requests + self.num_ctas * 8
         # CTAs a latent decode plan is cut for: one per SM where every layer runs on the tcgen05 kernel, else two
         self.latent_ctas = 0
-        if cfg.latent is not None and self.cuda:
+        if cfg.latent_specs and self.cuda:
             from ..ops import latent as lops
-            tc = self.dtype == torch.bfloat16 and all(lops.decode_on_tcgen05(s, page_size) for s in cfg.latent)
+            tc = self.dtype == torch.bfloat16 and all(lops.decode_on_tcgen05(s, page_size) for s in cfg.latent_specs)
             self.latent_ctas = ops.num_sms(self.device) * (1 if tc else 2)
         # shared-prefix decode plans: forks of one context read their common pages once per step
         import os as _os
@@ -273,7 +273,8 @@ class TorchDriver:
         tp = self.par.tp_size
         if self.cfg.blocks is not None:
             # linear-attention states are large (a slot holds every layer's [heads, dim, vdim] in 32-bit)
-            usable -= 4 * sum(b.recurrent.state_elems for b in self.cfg.blocks) * (rs_slots or self._default_rs_slots(max_requests))
+            elems = sum(b.recurrent.state_elems for b in self.cfg.blocks if b.recurrent is not None)
+            usable -= 4 * elems * (rs_slots or self._default_rs_slots(max_requests))
         if profile:
             plan = mp.plan(self.cfg, usable, 1.0, profile, self.page_size, tp)
             max_requests, max_tokens = plan.max_requests, plan.max_tokens
@@ -439,8 +440,8 @@ class TorchDriver:
             item_start=s.d("item_start"), item_end=s.d("item_end"), req_item_indptr=s.d("req_item_indptr"),
             num_items=s.d("num_items"), scratch=self.scratch, max_items=self.max_items, num_reqs=rb,
             num_ctas=self.num_ctas, page_size=self.page_size, window_left=self.window_left, kv_lens=s.d("kv_lens"))
-        if self.cfg.latent is not None:
-            plan.num_ctas, plan.cta_items = self.latent_ctas, s.d("item_slot", self.latent_ctas + 1)
+        if self.latent_ctas:
+            plan.cta_items = s.d("item_slot", self.latent_ctas + 1)
         if cascade:
             plan.item_slot, plan.item_tile, plan.tile_members = s.d("item_slot"), s.d("item_tile"), s.d("tile_members")
         return ForwardInputs(tokens=s.d("tokens", rb), positions=s.d("positions", rb), slots=s.d("slots", rb),
@@ -498,7 +499,7 @@ class TorchDriver:
             self.stats["cascade_tokens_saved"] = self.stats.get("cascade_tokens_saved", 0) + plan.shared_tokens
         else:
             plan = None
-            if self.cfg.latent is not None:
+            if self.latent_ctas:
                 item_req, st, en, indptr, cta_items = ops.plan_even_items(kv_lens, self.latent_ctas, self.max_items, self.window_left)
                 s.h("item_slot")[:len(cta_items)] = cta_items
             else:

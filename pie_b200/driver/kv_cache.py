@@ -18,7 +18,8 @@ from .schema import CopyDir, CopyRequest
 
 
 class LayerPages:
-    """Pages of layers with unequal shapes: one tensor [pages + 1, 2, kv heads, page, D] per layer that has a cache."""
+    """Pages of layers with unequal shapes: one tensor [pages + 1, 2, kv heads, page, D] (latent rows: [pages + 1, page, row])
+    per layer that has a cache."""
 
     def __init__(self, layers):
         self.layers = layers
@@ -41,7 +42,7 @@ class KVCache:
         that all heads share) in ``[layers, pages + 1, page_size, row]``; `layers` counts the layers that write rows.
 
         `layer_shapes`: (kv heads, head_dim) of every layer that has a cache, where a model's layers differ (`data` is then a
-        `LayerPages`; it may be empty)."""
+        `LayerPages`; it may be empty); no heads: latent rows of that width."""
         if page_size % 16:
             raise ValueError("kv page size must be a multiple of 16")
         if kv_dtype not in ("auto", "bf16", "fp8_e4m3"):
@@ -57,7 +58,7 @@ class KVCache:
         self.page_size, self.head_dim, self.dtype = page_size, head_dim, dtype
         self.device = torch.device(device)
         if layer_shapes is not None:
-            shapes = [(1, (2, h, page_size, d)) for h, d in layer_shapes]
+            shapes = [(1, (2, h, page_size, d) if h else (page_size, d)) for h, d in layer_shapes]
         else:
             shapes = [(layers, (page_size, head_dim) if latent else (2, kv_heads, page_size, head_dim))]
         # zero-filled: unwritten slots are multiplied by p == 0 in attention and must be finite

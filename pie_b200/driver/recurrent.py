@@ -1,7 +1,8 @@
 """Recurrent-state cache of the Gated DeltaNet and Mamba-2 layers and of token-shifted blocks: per (recurrent layer,
 slot) the tail of the short convolution's inputs and the fp32 state (delta-rule state [heads, dk, dv], or state-space
 state [heads, head_dim, state]), or the previous token's normalised input (token shift, [width] fp32). Linear-attention
-mixers of layers described one by one (any head sizes) keep [heads, dim, vdim] fp32 each, all layers of a slot in one row.
+mixers of layers described one by one (any head sizes) keep [heads, dim, vdim] fp32 each (a matrix memory also [heads, dim]
+and [heads]), all layers of a slot in one row.
 A slot belongs to one resident context; the runtime's
 slot pool (`runtime/rs_cache.py`) hands slots out, tells the driver when a slot must start from zero
 (`rs_reset`) and asks for a slot copy when a context forks.
@@ -40,6 +41,11 @@ class RecurrentInputs:
     pieces: Optional[tuple] = None # the portions cut for the chunked form (`ops.linear.chunk_pieces`)
     staged: Optional[int] = None   # requests the stage is committed for (0: none of this fire's portions uses it)
 
+    def state_of(self, li: int, elems: int) -> torch.Tensor:
+        """Layer `li`'s columns of the linear-attention state cache [slots, all layers]."""
+        at = self.linear_at[li]
+        return self.linear_state[:, at:at + elems]
+
 
 class RecurrentStateCache:
     def __init__(self, cfg: ModelConfig, num_slots: int, device):
@@ -54,9 +60,10 @@ class RecurrentStateCache:
         if cfg.blocks is not None:
             self.linear_at, at = {}, 0
             for li, b in enumerate(cfg.blocks):
-                self.linear_at[li] = at
-                at += -(-b.recurrent.state_elems // 4) * 4
-            self.linear_state = torch.zeros(num_slots, at, dtype=torch.float32, device=self.device)
+                if b.recurrent is not None:
+                    self.linear_at[li] = at
+                    at += -(-b.recurrent.state_elems // 4) * 4
+            self.linear_state = torch.zeros(num_slots, max(at, 4), dtype=torch.float32, device=self.device)
             return
         if cfg.token_shift:
             if cfg.mamba_layers or cfg.linear_layers:

@@ -18,54 +18,50 @@ from .config import _pad
 from .stream import ResidualStream
 
 
-def rope_table(base: float, dims: int, device) -> torch.Tensor:
-    inv = float(base) ** (-2.0 * torch.arange(dims // 2, dtype=torch.float64) / dims)
-    return inv.float().to(device)
+def prepare_latent_layer(m, s, lw: dict, tables: dict) -> None:
+    """The per-head factors of one mixer in the layout the absorbed products read, its rotation table (shared by `tables`)."""
+    key = (s.rope_base, s.rot_dims, str(s.rot_scaling))
+    if key not in tables:
+        tables[key] = s.rotary.frequencies(m.device)
+    lw["rope"] = tables[key]
+    # query into the latent: [H, rank, dim]; latent into the value: [H, vdim, rank_pad] (a cached row is padded)
+    lw["w_uk_t"] = lw["w_uk"].view(s.heads, s.dim, s.kv_rank).transpose(1, 2).contiguous()
+    uv = lw["w_uv"].view(s.heads, s.vdim, s.kv_rank)
+    lw["w_uv_p"] = torch.nn.functional.pad(uv, (0, s.rank_pad - s.kv_rank)).contiguous()
+    d = lops.projected_width(s)
+    if m.device.type == "cuda" and m.dtype == torch.bfloat16 and d:
+        # cache row -> (key | value) of every head, D columns each; the rotated key part is copied by a unit block
+        w = torch.zeros(s.heads, 2, d, s.row, dtype=m.dtype, device=m.device)
+        w[:, 0, :s.dim, :s.kv_rank] = lw["w_uk"].view(s.heads, s.dim, s.kv_rank)
+        w[:, 0, s.dim:s.qk_dim, s.rank_pad:s.rank_pad + s.rot_dim] = torch.eye(s.rot_dim, dtype=m.dtype, device=m.device)
+        w[:, 1, :s.vdim, :s.kv_rank] = uv
+        lw["w_kv_row"] = w.view(-1, s.row)
 
 
 def prepare_latent(m) -> None:
-    """Derived tensors of every layer: the per-head factors in the layout the absorbed products read, rotation tables."""
+    """Derived tensors of every layer."""
     cfg, tables = m.cfg, {}
     m.vocab_local = cfg.vocab_size
     m.cache_index = cfg.latent_cache_index
     if m.w["lm_head"].shape == m.w["embed"].shape:
         m.w["lm_head"] = m.w["embed"]                   # tied and unpadded: one copy
     for s, lw in zip(cfg.latent, m.w["layers"]):
-        key = (s.rope_base, s.rot_dims)
-        if key not in tables:
-            tables[key] = rope_table(*key, m.device)
-        lw["rope"] = tables[key]
-        # query into the latent: [H, rank, dim]; latent into the value: [H, vdim, rank_pad] (a cached row is padded)
-        lw["w_uk_t"] = lw["w_uk"].view(s.heads, s.dim, s.kv_rank).transpose(1, 2).contiguous()
-        uv = lw["w_uv"].view(s.heads, s.vdim, s.kv_rank)
-        lw["w_uv_p"] = torch.nn.functional.pad(uv, (0, s.rank_pad - s.kv_rank)).contiguous()
-        d = lops.projected_width(s)
-        if m.device.type == "cuda" and m.dtype == torch.bfloat16 and d:
-            # cache row -> (key | value) of every head, D columns each; the rotated key part is copied by a unit block
-            w = torch.zeros(s.heads, 2, d, s.row, dtype=m.dtype, device=m.device)
-            w[:, 0, :s.dim, :s.kv_rank] = lw["w_uk"].view(s.heads, s.dim, s.kv_rank)
-            w[:, 0, s.dim:s.qk_dim, s.rank_pad:s.rank_pad + s.rot_dim] = torch.eye(s.rot_dim, dtype=m.dtype, device=m.device)
-            w[:, 1, :s.vdim, :s.kv_rank] = uv
-            lw["w_kv_row"] = w.view(-1, s.row)
+        prepare_latent_layer(m, s, lw, tables)
 
 
-def latent_mixer(m, hs, lw: dict, li: int, fi, cache, out) -> None:
-    """Latent attention of layer `li` on hs [N, width]; the heads' values go to out [N, heads * vdim] (W_o follows)."""
-    s, n = m.cfg.latent[li], hs.shape[0]
-    page = cache.shape[2]
-    layer_cache = cache[m.cache_index[li]]
-    qkv = m._gemm(hs, lw["w_latent_in"])
+def latent_attend(m, q_in, kv, lw: dict, s, fi, layer_cache, out) -> None:
+    """Latent attention with queries q_in [N, >= heads * qk_dim] and the new tokens' rows kv [N, kv_rank + rot_dim] (None: a
+    layer that reads another's); the heads' values go to out [N, heads * vdim], which may be a column range."""
+    n, page, eps = q_in.shape[0], layer_cache.shape[1], m.cfg.rms_norm_eps
+    cache = layer_cache if kv is not None else None
+    rows = lambda width, rot, copy: lops.latent_rows(q_in, fi.positions, fi.slots, lw["rope"], lw.get("latent_norm"), cache, s, eps, width,
+                                                     rot, copy, kv)
     if "w_kv_row" in lw and not fi.is_decode and fi.attn.mask_bits is None and page % 16 == 0:
-        q = lops.latent_rows(qkv, fi.positions, fi.slots, lw["rope"], lw.get("latent_norm"),
-                             layer_cache if s.kv_from is None else None, s, m.cfg.rms_norm_eps, lops.projected_width(s), s.dim,
-                             copy_nope=True)
-        lops.projected_prefill_attention(q, layer_cache, fi.attn, lw["w_kv_row"], s, page, s.window - 1, out)
+        lops.projected_prefill_attention(rows(lops.projected_width(s), s.dim, True), layer_cache, fi.attn, lw["w_kv_row"], s, page,
+                                         s.window - 1, out)
         return
-    q = lops.latent_rows(qkv, fi.positions, fi.slots, lw["rope"], lw.get("latent_norm"), layer_cache if s.kv_from is None else None,
-                         s, m.cfg.rms_norm_eps, s.row, s.rank_pad, copy_nope=False)
-    nope = qkv[:, :s.q_rows].view(n, s.heads, s.qk_dim)[..., :s.dim] if qkv.shape[1] == s.q_rows else \
-        qkv.as_strided((n, s.heads, s.dim), (qkv.stride(0), s.qk_dim, 1))
-    lops.per_head(nope, lw["w_uk_t"], q[..., :s.kv_rank])
+    q = rows(s.row, s.rank_pad, False)
+    lops.per_head(q_in.as_strided((n, s.heads, s.dim), (q_in.stride(0), s.qk_dim, 1)), lw["w_uk_t"], q[..., :s.kv_rank])
     o = lops.latent_attention(q, layer_cache, fi.attn, fi.rs, fi.slots, s, page, s.window - 1)
     lops.per_head(o, lw["w_uv_p"], out.as_strided((n, s.heads, s.vdim), (out.stride(0), s.vdim, 1)))
 
@@ -79,7 +75,8 @@ def parallel_latent_block(m, st: ResidualStream, lw: dict, li: int, fi, cache) -
     both = torch.empty(n, cols, dtype=h.dtype, device=h.device)       # attention heads | feed-forward activations
     if _pad(hv) > hv:
         both[:, hv:_pad(hv)] = 0
-    latent_mixer(m, hs if hs is not None else h, lw, li, fi, cache, both[:, :hv])
+    qkv = m._gemm(hs if hs is not None else h, lw["w_latent_in"])
+    latent_attend(m, qkv, qkv[:, s.q_rows:s.proj_rows] if s.kv_from is None else None, lw, s, fi, cache[m.cache_index[li]], both[:, :hv])
     side = cfg.token_side_dim
     fused = m.gemm_backend == "tcgen05" and h.dtype == torch.bfloat16
     if ff and fused:

@@ -11,6 +11,7 @@ class ResidualStream:
 
     def __init__(self, x):
         self.x, self.y, self.y_norm = x, None, None
+        self.values = None          # values of the first layer that mixes them (32-bit, one row per token)
 
     def finish(self, cfg: ModelConfig):
         """The stream with everything pending added."""
@@ -22,5 +23,11 @@ class ResidualStream:
     def normed(self, cfg: ModelConfig, gain, dtype):
         """Add what is pending, then RMSNorm(x) * gain in `dtype`."""
         self.x, h, _ = lops.stream_norm(self.x, cfg.hidden_size, cfg.rms_norm_eps, self.y, self.y_norm, gain, dtype=dtype)
+        self.y = self.y_norm = None
+        return h
+
+    def plain(self, cfg: ModelConfig, dtype):
+        """Add what is pending; the stream itself in `dtype`."""
+        self.x, h, _ = lops.stream_norm(self.x, cfg.hidden_size, cfg.rms_norm_eps, self.y, self.y_norm, dtype=dtype, copy=True)
         self.y = self.y_norm = None
         return h

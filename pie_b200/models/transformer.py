@@ -225,8 +225,8 @@ class Transformer:
                 latent.parallel_latent_block(self, stream, lw, li, fi, kv_cache)
                 continue
             if cfg.blocks is not None:
-                # sandwich-normed block with a mixer and a feed-forward of its own
-                sandwich.sandwich_block(self, stream, lw, li, fi, kv_cache)
+                # a mixer and a feed-forward of its own
+                sandwich.block(self, stream, lw, li, fi, kv_cache)
                 continue
             if "w_mamba_in" in lw:
                 # Mamba-2 layer: state-space mixer, state in the recurrent-state cache
@@ -315,7 +315,8 @@ class Transformer:
             return self.par.comm.gemm_gated(self.w["lm_head"], rows.shape[0], x=rows)
         if self.cfg.stream32:
             x = (latent if self.cfg.latent is not None else sandwich).final_rows(self, rows)
-            return self._gemm(x, self.w["lm_head"])[:, :self.cfg.vocab_size]
+            y = self._gemm(x, self.w["lm_head"])[:, :self.cfg.vocab_size]
+            return ops.softcap_(y, self.cfg.final_softcap) if self.cfg.final_softcap else y
         x = ops.rmsnorm(rows, self.w["final_norm"], self.cfg.rms_norm_eps)
         y = self._gemm(x, self.w["lm_head"])
         if self.par.tp_size > 1 and self.par.comm is not None:

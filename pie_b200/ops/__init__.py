@@ -180,6 +180,17 @@ def gather_rows(x, idx, out=None):
     return out
 
 
+def softcap_(y, cap: float):
+    """y = cap * tanh(y / cap) in place (32-bit arithmetic); y [rows, cols] may be a column range."""
+    if not y.is_cuda:
+        return y.copy_(torch.tanh(y.float() / cap) * cap)
+    for a in range(0, y.shape[0], 32768):
+        part = y[a:a + 32768]
+        check(fn("pie_softcap")(ptr(part), part.shape[0], part.shape[1], part.stride(0), cap, 1 if y.dtype == torch.float32 else 0,
+                                stream_ptr()), "softcap")
+    return y
+
+
 def feed_tokens(tokens, src_row, prev_sampled, n: int):
     """tokens[i] = prev_sampled[src_row[i]] where src_row[i] >= 0 (device-side token feed)."""
     if not tokens.is_cuda:
@@ -486,8 +497,13 @@ def moe_align(buf: "MoeBuffers", max_mtiles: int = 0):
                               ptr(buf.tile_expert), ptr(buf.counts_out), stream_ptr()), "moe_align")
 
 
-def moe_permute(x, buf: "MoeBuffers"):
+def moe_permute(x, buf: "MoeBuffers", weighted: bool = False):
+    """Rows to their experts' segments, `weighted`: times the route's weight."""
     n, h = x.shape
+    if weighted:
+        check(fn("pie_moe_permute_weighted")(ptr(x), x.stride(0), ptr(buf.ids), ptr(buf.pos), ptr(buf.seg_start), ptr(buf.w), n, h, buf.k,
+                                             ptr(buf.xs), ptr(buf.slot_of), stream_ptr()), "moe_permute")
+        return
     check(fn("pie_moe_permute")(ptr(x), x.stride(0), ptr(buf.ids), ptr(buf.pos), ptr(buf.seg_start), n, h, buf.k,
                                 ptr(buf.xs), ptr(buf.slot_of), stream_ptr()), "moe_permute")
 
@@ -515,10 +531,10 @@ def moe_row_bias(y, bias, tile_expert, mtiles: int):
     return y
 
 
-def moe_combine(buf: "MoeBuffers", n: int, residual=None, out=None):
+def moe_combine(buf: "MoeBuffers", n: int, residual=None, out=None, weighted: bool = True):
     if out is None:
         out = torch.empty(n, buf.H, dtype=buf.ys.dtype, device=buf.ys.device)
-    check(fn("pie_moe_combine")(ptr(buf.ys), ptr(buf.slot_of), ptr(buf.w), ptr(residual),
+    check(fn("pie_moe_combine")(ptr(buf.ys), ptr(buf.slot_of), ptr(buf.w) if weighted else None, ptr(residual),
                                 residual.stride(0) if residual is not None else 0, n, buf.H, buf.k, ptr(out),
                                 out.stride(0), stream_ptr()), "moe_combine")
     return out
@@ -811,7 +827,7 @@ class DecodePlan:
     item_tile: Optional[torch.Tensor] = None
     tile_members: Optional[torch.Tensor] = None
     kv_lens: Optional[torch.Tensor] = None
-    cta_items: Optional[torch.Tensor] = None    # plans of `plan_even_items`: the items of every CTA (num_ctas + 1 offsets)
+    cta_items: Optional[torch.Tensor] = None    # plans of `plan_even_items`: the items of every CTA (CTAs + 1 offsets)
 
 
 def decode_scratch_floats(max_items: int, hq: int, head_dim: int) -> int:
@@ -832,15 +848,25 @@ def dequant_kv_pages(kv8_layer, scale_layer, pages: torch.Tensor, pad_zero_page:
 
 
 def paged_decode_attention(q, kv_layer, plan: DecodePlan, sm_scale: float, out=None, window_left=None,
-                           sinks_log2=None, kv_scale=None, softcap: float = 0.0):
+                           sinks_log2=None, kv_scale=None, softcap: float = 0.0, keep_first: int = 0):
     """q [R, hq, D] (one token per request) against paged KV; split-KV + merge. `window_left`
     overrides the plan's window for this call (a layer with its own window; the plan's items
-    must then cover at least that window), `sinks_log2` [hq] fp32 = sink logits * log2(e)."""
+    must then cover at least that window), `sinks_log2` [hq] fp32 = sink logits * log2(e). `keep_first`: keys that stay
+    visible beside the window (covered by the plan's items)."""
     if out is None:
         out = torch.empty_like(q)
     wl = plan.window_left if window_left is None else window_left
     r, hq, d = q.shape
     hkv = kv_layer.shape[2]
+    if keep_first:
+        if kv_scale is not None or plan.item_tile is not None or softcap:
+            raise NotImplementedError("kept first keys over fp8 KV pages, shared-prefix plans or soft-capped scores")
+        check(fn("pie_paged_decode_attn_kept")(
+            ptr(q), ptr(kv_layer), ptr(plan.page_indices), ptr(plan.kv_page_indptr), ptr(plan.item_req),
+            ptr(plan.item_start), ptr(plan.item_end), ptr(plan.req_item_indptr), ptr(plan.num_items),
+            ptr(out), ptr(plan.scratch), plan.max_items, plan.num_reqs, hq, hkv, d, plan.page_size,
+            sm_scale, plan.num_ctas, wl, keep_first, ptr(sinks_log2), stream_ptr()), "paged_decode_attn_kept")
+        return out
     if softcap:                     # softmax over softcap * tanh(score / softcap) (Gemma-2)
         if kv_scale is not None or plan.item_tile is not None:
             raise NotImplementedError("soft-capped scores over fp8 KV pages or shared-prefix plans")
@@ -894,12 +920,27 @@ class PrefillPlan:
 
 
 def paged_prefill_attention(q, kv_layer, plan: PrefillPlan, sm_scale: float, out=None, lse_out=None,
-                            window_left=None, sinks_log2=None, softcap: float = 0.0):
+                            window_left=None, sinks_log2=None, softcap: float = 0.0, keep_first: int = 0):
     if out is None:
         out = torch.empty_like(q)
     wl = plan.window_left if window_left is None else window_left
     n, hq, d = q.shape
     hkv = kv_layer.shape[2]
+    if keep_first:                  # keys that stay visible beside the window
+        if plan.tile_rows > 64:
+            check(fn("pie_paged_prefill_attn_tc_kept")(
+                ptr(q), ptr(kv_layer), ptr(plan.page_indices), ptr(plan.kv_page_indptr), ptr(plan.qo_indptr),
+                ptr(plan.kv_lens), ptr(plan.tile_req), ptr(plan.tile_qstart), plan.num_tiles,
+                ptr(plan.mask_bits), ptr(plan.mask_word_indptr), ptr(out), ptr(lse_out), n, hq, hkv, d,
+                kv_layer.shape[0], sm_scale, wl, plan.tile_rows, ptr(sinks_log2), ptr(kernel_status(q.device)),
+                float(softcap), keep_first, stream_ptr()), "paged_prefill_attn_tc_kept")
+        else:
+            check(fn("pie_paged_prefill_attn_kept")(
+                ptr(q), ptr(kv_layer), ptr(plan.page_indices), ptr(plan.kv_page_indptr), ptr(plan.qo_indptr),
+                ptr(plan.kv_lens), ptr(plan.tile_req), ptr(plan.tile_qstart), plan.num_tiles,
+                ptr(plan.mask_bits), ptr(plan.mask_word_indptr), ptr(out), ptr(lse_out), hq, hkv, d,
+                plan.page_size, sm_scale, wl, ptr(sinks_log2), float(softcap), keep_first, stream_ptr()), "paged_prefill_attn_kept")
+        return out
     if softcap and plan.tile_rows > 64:
         if plan.tile_rows != 256:
             raise ValueError("soft-capped scores on the tcgen05 kernel need 256-row tiles: plan with prefill_tile_rows(..., softcap=True)")

@@ -76,6 +76,16 @@ _SIGNATURES = {
     "pie_bias_xielu": [p, i32, p, p, i32, i32, i32, p],
     "pie_stream_add": [p, p, p, p, p, i32, i32, i32, p],
     "pie_side_gate": [p, i32, i64, i32, i32, p, i32, p, p, i32, i32, i32, i32, i32, i32, p],
+    "pie_paged_decode_attn_kept": [p, p, p, p, p, p, p, p, p, p, p, i32, i32, i32, i32, i32, i32, f32, i32, i32, i32, p, p],
+    "pie_paged_prefill_attn_kept": [p, p, p, p, p, p, p, p, i32, p, p, p, p, i32, i32, i32, i32, f32, i32, p, f32, i32, p],
+    "pie_paged_prefill_attn_tc_kept": [p, p, p, p, p, p, p, p, i32, p, p, p, p, i32, i32, i32, i32, i32, f32, i32, i32, p, p, f32, i32, p],
+    "pie_gqa_rows": [p, i32, p],
+    "pie_gqa_any": [p, i32, p],
+    "pie_gqa_mma_supported": [i32, i32, i32],
+    "pie_memory_gates": [p, i32, p],
+    "pie_softcap": [p, i32, i32, i64, f32, i32, p],
+    "pie_moe_route_sigmoid": [p, i32, i64, i32, i32, i32, i32, p, p, p, p, p],
+    "pie_moe_permute_weighted": [p, i32, p, p, p, p, i32, i32, i32, p, p, p],
     "pie_linear_attn_serial": [p, i32, p],
     "pie_linear_attn_chunk_supported": [i32],
     "pie_linear_attn_chunk_tokens": [],

@@ -102,9 +102,10 @@ def latent_rows(qkv, positions, slots, inv_freq, norm_w, cache, spec, eps: float
         return ref.latent_rows(qkv, kv, positions, slots, inv_freq, norm_w, cache, spec, eps, q, q_rot, copy_nope)
     a = LatentRowsArgs(q=ptr(qkv), kv=ptr(kv), positions=ptr(positions), slots=ptr(slots), inv_freq=ptr(inv_freq), norm_w=ptr(norm_w),
                        q_out=ptr(q), cache=ptr(cache), n=n, ld=qkv.stride(0), ld_kv=kv.stride(0), heads=spec.heads, dim=spec.dim,
-                       rot_dim=spec.rot_dim, rot_dims=spec.rot_dims, adjacent=1 if spec.rot_adjacent else 0, rot_factor=spec.rotary.factor, rank=spec.kv_rank, rank_pad=spec.rank_pad,
+                       rot_dim=spec.rot_dim, rot_dims=spec.rot_dims, rank=spec.kv_rank, rank_pad=spec.rank_pad,
                        cache_row=cache.shape[-1] if cache is not None else 0, copy_nope=1 if copy_nope else 0, q_width=q_width,
-                       q_rot=q_rot, q_zero=q_rot if copy_nope else spec.kv_rank, eps=eps)
+                       q_rot=q_rot, q_zero=q_rot if copy_nope else spec.kv_rank, adjacent=1 if spec.rot_adjacent else 0, eps=eps,
+                       rot_factor=spec.rotary.factor)
     check(fn("pie_latent_rows")(C.byref(a), _f32(qkv), stream_ptr()), "latent_rows")
     return q
 
@@ -155,7 +156,7 @@ def latent_attention(q, cache, plan, rs, slots, spec, page_size: int, window_lef
     if decode:
         a.item_req, a.item_start, a.item_end = ptr(plan.item_req), ptr(plan.item_start), ptr(plan.item_end)
         a.req_item_indptr, a.cta_items, a.scratch = ptr(plan.req_item_indptr), ptr(plan.cta_items), ptr(plan.scratch)
-        a.max_items, ctas = plan.max_items, plan.num_ctas
+        a.max_items, ctas = plan.max_items, plan.cta_items.numel() - 1
         if decode_on_tcgen05(spec, page_size):
             check(fn("pie_latent_attn_tc")(C.byref(a), ctas, ptr(ops.kernel_status(q.device)), stream_ptr()), "latent_attn_tc")
             return out

@@ -19,11 +19,14 @@ LOG2E = 1.4426950408889634
 GUARD = 64              # entries before and after a bias row that the kernels may touch for hidden keys
 
 # mirrors of the argument structs in csrc/kernels/linear_attn.cu and attention_bias.cu
-LinAttnArgs = _struct("LinAttnArgs", ("q k v log_decay head_decay out state qo_indptr slots reset chunk_req chunk_start req_chunks "
-                                      "u piece_decay", p), ("slot_stride", i64),
+LinAttnArgs = _struct("LinAttnArgs", ("q k v log_decay head_decay tok_decay tok_input den out state qo_indptr slots reset chunk_req "
+                                      "chunk_start req_chunks u piece_decay", p), ("slot_stride", i64),
                       ("n ld reqs heads dim vdim silu chunks", i32), ("q_scale", f32))
-GatedNormPart = _struct("GatedNormPart", ("x w gate dst", p),
-                        ("x_f32 ldx head_cols head_ld group group_pad norm_cols w_cols ldg ldd cols dst_cols act", i32), ("eps scale", f32))
+MemoryGatesArgs = _struct("MemoryGatesArgs", ("z bias qo_indptr slots reset tok_req m decay input floor", p), ("slot_stride split_stride", i64),
+                          ("n reqs heads ldz splits", i32), ("cap", f32))
+GatedNormPart = _struct("GatedNormPart", ("x w gate dst den floor", p),
+                        ("x_f32 ldx head_cols head_ld group group_pad norm_cols w_cols ldg gate_cols ldd cols dst_cols act", i32),
+                        ("eps scale", f32))
 BiasedRowsArgs = _struct("BiasedRowsArgs", ("q k v q_norm k_norm slots q_out cache", p),
                          ("n ld heads kv_heads group group_pad dim vdim D page_size", i32), ("eps", f32))
 BiasedAttnArgs = _struct("BiasedAttnArgs", ("q kv out bias page_indices kv_page_indptr kv_lens qo_indptr tok_req slots tile_req tile_qstart "
@@ -64,55 +67,86 @@ def chunk_pieces(rs, device):
     return rs.pieces
 
 
-def linear_attention(q, k, v, spec, rs, state, decode: bool, log_decay=None, head_decay=None, silu: bool = False, q_scale: float = 1.0):
+def memory_gates(h, w, bias, spec, rs, state, decode: bool):
+    """Exponential gates of a matrix memory (`MatrixMemorySpec`) on the mixer's input h: (decay, key factor) [N, heads] as
+    base-2 logarithms for `linear_attention`, and exp(-m_t). The running maxima m are the last numbers of `state`, this layer's
+    columns of the state cache, and advance. w: rows of the input gates, then of the forget gates; bias 32-bit."""
+    from .latent import split_product
+    n, heads = h.shape[0], spec.heads
+    m = state[:, spec.state_elems - heads:]
+    if not h.is_cuda:
+        return ref.memory_gates(torch.matmul(h.float(), w.float().t()) + bias, spec, rs, m)
+    z = split_product(h, w) if h.dtype == torch.bfloat16 else torch.matmul(h, w.t())[None]
+    out = torch.empty(3, n, heads, dtype=torch.float32, device=h.device)
+    a = MemoryGatesArgs(z=ptr(z), bias=ptr(bias), qo_indptr=ptr(rs.qo_indptr), slots=ptr(rs.slots), reset=ptr(rs.reset), tok_req=ptr(rs.tok_req),
+                        m=ptr(m), decay=ptr(out[0]), input=ptr(out[1]), floor=ptr(out[2]), slot_stride=state.stride(0),
+                        split_stride=z.stride(0), n=n, reqs=len(rs.slots_host), heads=heads, ldz=z.stride(1), splits=z.shape[0], cap=spec.gate_cap)
+    check(fn("pie_memory_gates")(C.byref(a), 1 if decode else 0, stream_ptr()), "memory_gates")
+    return out[0], out[1], out[2]
+
+
+def linear_attention(q, k, v, spec, rs, state, decode: bool, log_decay=None, head_decay=None, silu: bool = False, q_scale: float = 1.0,
+                     gates=None):
     """o [N, heads * vdim] in 32-bit of S_t = diag(a_t) S_(t-1) + k_t v_t^T, o_t = S_t^T q_t over the ragged batch `rs`.
-    q, k, v: column ranges [N, heads * dim (vdim)] of one projection. The decay is per key channel (`log_decay`) or per head
-    (`head_decay` [heads] 32-bit). `state`: this layer's columns of the state cache [slots, all layers]."""
+    q, k, v: column ranges [N, heads * dim (vdim)] of one projection. The decay is per key channel (`log_decay`), per head
+    (`head_decay` [heads] 32-bit), or per head and token with a factor on the key (`gates`: both as base-2 logarithms
+    [N, heads]; the state then ends in a normaliser, n_t = a_t n_(t-1) + k_t, and (o, n_t . q_t [N, heads]) is returned).
+    `state`: this layer's columns of the state cache [slots, all layers]."""
     n, h, d, e = q.shape[0], spec.heads, spec.dim, spec.vdim
+    if not q.is_cuda and gates is not None:
+        o, den = ref.normalised_linear_attention(q.reshape(n, h, d), k.reshape(n, h, d), v.reshape(n, h, e), *gates, state, rs, q_scale)
+        return o.view(n, h * e), den
     if not q.is_cuda:
         ld = log_decay.view(n, h, d) if log_decay is not None else None
         return ref.linear_attention(q.reshape(n, h, d), k.reshape(n, h, d), v.reshape(n, h, e), ld, head_decay,
                                     state.view(state.shape[0], h, d, e), rs, silu, q_scale).view(n, h * e)
     out = torch.empty(n, h * e, dtype=torch.float32, device=q.device)
-    a = LinAttnArgs(q=ptr(q), k=ptr(k), v=ptr(v), log_decay=ptr(log_decay), head_decay=ptr(head_decay), out=ptr(out), state=ptr(state),
+    den = torch.empty(n, h, dtype=torch.float32, device=q.device) if gates is not None else None
+    tok_decay, tok_input = gates if gates is not None else (None, None)
+    a = LinAttnArgs(q=ptr(q), k=ptr(k), v=ptr(v), log_decay=ptr(log_decay), head_decay=ptr(head_decay), tok_decay=ptr(tok_decay),
+                    tok_input=ptr(tok_input), den=ptr(den), out=ptr(out), state=ptr(state),
                     qo_indptr=ptr(rs.qo_indptr), slots=ptr(rs.slots), reset=ptr(rs.reset), slot_stride=state.stride(0), n=n, ld=q.stride(0),
                     reqs=len(rs.slots_host), heads=h, dim=d, vdim=e, silu=1 if silu else 0, q_scale=q_scale)
     if decode or q.dtype == torch.float32 or not fn("pie_linear_attn_chunk_supported")(d):
         check(fn("pie_linear_attn_serial")(C.byref(a), _f32(q), stream_ptr()), "linear_attn_serial")
-        return out
+        return out if den is None else (out, den)
     req, start, indptr = chunk_pieces(rs, q.device)
     c = req.numel()
-    u = torch.empty(c, h, d, e, dtype=torch.float32, device=q.device)
+    u = torch.empty(c, h * d * (e + (den is not None)), dtype=torch.float32, device=q.device)
     dec = torch.empty(c, h, d, dtype=torch.float32, device=q.device)
     a.chunk_req, a.chunk_start, a.req_chunks, a.u, a.piece_decay, a.chunks = ptr(req), ptr(start), ptr(indptr), ptr(u), ptr(dec), c
     check(fn("pie_linear_attn_chunked")(C.byref(a), stream_ptr()), "linear_attn_chunked")
-    return out
+    return out if den is None else (out, den)
 
 
 def gated_norm(parts):
     """Outputs of one mixer or of two side by side: for each part (x, w, gate, dst, kw) dst = RMSNorm(x) * w * act(gate) *
-    scale. kw: act "silu" | "sigmoid", norm_cols (columns per mean square, 0: no norm), eps, scale, and for attention outputs
-    in padded rows `spec` (a BiasedAttentionSpec). dst may be a column range; `pad` columns after it are set to zero."""
+    scale. kw: act "silu" | "sigmoid", norm_cols (columns per mean square, 0: no norm), eps, scale; for attention outputs in
+    padded rows `spec` (an attention spec); `cols` of the output where the gate (None: none) has one number per `gate_cols`
+    of them; den and floor [N, groups of norm_cols]: the norm is that of x / (max(|den|, floor) + 1e-6). dst may be a column
+    range; the columns after the output's are set to zero."""
     if not parts[0][0].is_cuda:
         for x, w, gate, dst, kw in parts:
             s = kw.get("spec")
             if s is not None:
                 x = x.view(x.shape[0], s.kv_heads, s.group_pad, s.head_dim)[:, :, :s.group, :s.vdim].reshape(x.shape[0], -1)
-            y = ref.gated_norm(x.float(), w, gate, kw["act"], kw["scale"], kw["norm_cols"], kw.get("eps", 0.0))
+            y = ref.gated_norm(x.float(), w, gate, kw.get("act"), kw["scale"], kw["norm_cols"], kw.get("eps", 0.0), kw.get("gate_cols", 1),
+                               kw.get("den"), kw.get("floor"))
             dst[:, :y.shape[1]] = y.to(dst.dtype)
             dst[:, y.shape[1]:] = 0
         return
     a = GatedNormArgs()
     a.n = parts[0][0].shape[0]
     for i, (x, w, gate, dst, kw) in enumerate(parts):
-        s = kw.get("spec")
-        cols = gate.shape[1]
+        s, gc = kw.get("spec"), kw.get("gate_cols", 1)
+        cols = gate.shape[1] * gc if gate is not None else kw["cols"]
         a.part[i] = GatedNormPart(
-            x=ptr(x), w=ptr(w), gate=ptr(gate), dst=ptr(dst), x_f32=_f32(x), ldx=x.stride(0), head_cols=s.vdim if s else cols,
-            head_ld=s.head_dim if s else cols, group=s.group if s else 1, group_pad=s.group_pad if s else 1, norm_cols=kw["norm_cols"],
-            w_cols=w.numel() if w is not None else 1, ldg=gate.stride(0), ldd=dst.stride(0), cols=cols, dst_cols=dst.shape[1],
-            act=1 if kw["act"] == "silu" else 0, eps=kw.get("eps", 0.0), scale=kw["scale"])
-    check(fn("pie_gated_norm")(C.byref(a), len(parts), _f32(parts[0][2]), stream_ptr()), "gated_norm")
+            x=ptr(x), w=ptr(w), gate=ptr(gate), dst=ptr(dst), den=ptr(kw.get("den")), floor=ptr(kw.get("floor")), x_f32=_f32(x),
+            ldx=x.stride(0), head_cols=s.vdim if s else cols, head_ld=s.head_dim if s else cols, group=s.group if s else 1,
+            group_pad=s.group_pad if s else 1, norm_cols=kw["norm_cols"], w_cols=w.numel() if w is not None else 1,
+            ldg=gate.stride(0) if gate is not None else 0, gate_cols=gc, ldd=dst.stride(0), cols=cols, dst_cols=dst.shape[1],
+            act=1 if kw.get("act") == "silu" else 0, eps=kw.get("eps", 0.0), scale=kw["scale"])
+    check(fn("pie_gated_norm")(C.byref(a), len(parts), _f32(parts[0][3]), stream_ptr()), "gated_norm")
 
 
 # ------------------------------------------------------------------ attention with a distance bias
@@ -189,6 +223,22 @@ def biased_attention(q, cache, bias, plan, rs, slots, spec):
 
 
 # ------------------------------------------------------------------ experts
+def sigmoid_experts(x, router, gate_up, down, spec, buf, shared=None):
+    """SwiGLU experts chosen by the sigmoid of the router's outputs (32-bit), whose weight scales what they read; `shared`
+    [N, W] is added. bf16 on the grouped tcgen05 GEMMs (static shapes, no host synchronisation); `buf`: ops.MoeBuffers."""
+    from .latent import split_product
+    n = x.shape[0]
+    z = split_product(x, router)
+    check(fn("pie_moe_route_sigmoid")(ptr(z), z.shape[0], z.stride(0), spec.experts, n, spec.experts, spec.top, ptr(buf.ids), ptr(buf.w),
+                                      ptr(buf.pos), ptr(buf.counts), stream_ptr()), "moe_route_sigmoid")
+    mt = ops.moe_max_mtiles(n, spec.top, spec.experts)
+    ops.moe_align(buf, mt)
+    ops.moe_permute(x, buf, weighted=True)
+    ops.grouped_gemm(buf.xs, gate_up, buf.tile_expert, buf.act, mt, ops.EPI_SWIGLU)
+    ops.grouped_gemm(buf.act, down, buf.tile_expert, buf.ys, mt, ops.EPI_STORE)
+    return ops.moe_combine(buf, n, shared, weighted=False)
+
+
 def scored_experts(x, router, correction, gate_up, down, spec, buf):
     """Experts chosen by softmax score + correction and weighted by the score, identity experts included. bf16 on the
     grouped tcgen05 GEMMs (static shapes, no host synchronisation); `buf`: ops.MoeBuffers."""

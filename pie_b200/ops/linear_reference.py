@@ -1,6 +1,8 @@
 """PyTorch statements of the ops in :mod:`.linear`: what they compute on CPU tensors."""
 from __future__ import annotations
 
+import math
+
 import torch
 
 
@@ -32,15 +34,62 @@ def linear_attention(q, k, v, log_decay, head_decay, state, rs, silu: bool, q_sc
     return out
 
 
-def gated_norm(x, w, gate, act: str, scale: float, norm_cols: int, eps: float):
-    """x [N, C] fp32: RMSNorm over runs of norm_cols columns (0: none) * w, times act(gate) * scale."""
+def memory_gates(z, spec, rs, m):
+    """z [N, 2 * heads] biased gate inputs; m [slots, heads] the running maxima, which advance."""
+    n, h = z.shape[0], spec.heads
+    z = spec.gate_cap * torch.tanh(z / spec.gate_cap)
+    i, f = z[:, :h], torch.nn.functional.logsigmoid(z[:, h:])
+    decay, key, floor = torch.zeros(n, h), torch.zeros(n, h), torch.zeros(n, h)
+    for r, (a, b) in enumerate(zip(rs.qo_host, rs.qo_host[1:])):
+        slot = rs.slots_host[r]
+        if slot < 0 or a == b:
+            continue
+        x = torch.zeros(h) if rs.reset_host[r] else m[slot].clone()
+        for t in range(a, b):
+            new = torch.maximum(f[t] + x, i[t])
+            decay[t], key[t], floor[t] = f[t] + x - new, i[t] - new, torch.exp(-new)
+            x = new
+        m[slot] = x
+    return decay / math.log(2), key / math.log(2), floor
+
+
+def normalised_linear_attention(q, k, v, decay, key, state, rs, q_scale: float):
+    """q, k [N, H, K], v [N, H, V]; base-2 logarithms [N, H]; state [slots, H * K * V + H * K + ..] advances. Returns
+    (S_t^T q_t, n_t . q_t)."""
+    q, k, v = q.float() * q_scale, k.float(), v.float()
+    n, h, d, e = q.shape[0], q.shape[1], q.shape[2], v.shape[2]
+    out, den = torch.zeros(n, h, e), torch.zeros(n, h)
+    for r, (a, b) in enumerate(zip(rs.qo_host, rs.qo_host[1:])):
+        slot = rs.slots_host[r]
+        if slot < 0 or a == b:
+            continue
+        s, c = state[slot, :h * d * e].view(h, d, e).clone(), state[slot, h * d * e:h * d * (e + 1)].view(h, d).clone()
+        if rs.reset_host[r]:
+            s, c = torch.zeros_like(s), torch.zeros_like(c)
+        for t in range(a, b):
+            g, kt = torch.exp2(decay[t])[:, None], k[t] * torch.exp2(key[t])[:, None]
+            s = g[..., None] * s + kt[..., None] * v[t][:, None]
+            c = g * c + kt
+            out[t], den[t] = torch.einsum("hkv,hk->hv", s, q[t]), (c * q[t]).sum(-1)
+        state[slot, :h * d * e], state[slot, h * d * e:h * d * (e + 1)] = s.flatten(), c.flatten()
+    return out, den
+
+
+def gated_norm(x, w, gate, act, scale: float, norm_cols: int, eps: float, gate_cols: int = 1, den=None, floor=None):
+    """x [N, C] fp32: RMSNorm over runs of norm_cols columns (0: none) * w, times act(gate) * scale; a gate number serves
+    gate_cols columns. den, floor: x / (max(|den|, floor) + 1e-6) is normed, one of each per run."""
     n, c = x.shape
     if norm_cols:
         x = x.view(n, -1, norm_cols)
+        if den is not None:
+            x = x / (torch.maximum(den.abs(), floor) + 1e-6)[..., None]
         x = x / torch.sqrt((x * x).mean(-1, keepdim=True) + eps)
         x = (x * w.float().view(-1, norm_cols)).reshape(n, c)
-    g = torch.sigmoid(gate.float())
-    return x * (g * gate.float() if act == "silu" else g) * scale
+    if gate is None:
+        return x * scale
+    gate = gate.float().repeat_interleave(gate_cols, -1)
+    g = torch.sigmoid(gate)
+    return x * (g * gate if act == "silu" else g) * scale
 
 
 def biased_rows(q, k, v, q_norm, k_norm, slots, cache, spec, eps: float):
@@ -93,3 +142,14 @@ def experts(x, logits, correction, gate_up, down, spec):
     y = torch.bmm((g * torch.sigmoid(1.702 * g) * (u + 1)).to(x.dtype), down.transpose(1, 2))
     out = torch.einsum("enw,ne->nw", y.float(), weight[:, :spec.experts])
     return (out + weight[:, spec.experts:].sum(-1, keepdim=True) * x.float()).to(x.dtype)
+
+
+def sigmoid_experts(x, logits, gate_up, down, spec):
+    """Sum of the chosen experts' outputs on x times the expert's score; gate_up [E, 2 F, W] holds interleaved gate and up
+    rows. An expert that was not chosen reads zeros and returns zeros."""
+    ids = torch.topk(logits.float(), spec.top, -1).indices
+    weight = torch.zeros_like(logits, dtype=torch.float32).scatter(1, ids, torch.sigmoid(torch.gather(logits.float(), 1, ids)))
+    xs = (x.float()[None] * weight.t()[..., None]).to(x.dtype)
+    gu = torch.bmm(xs, gate_up.transpose(1, 2))
+    y = torch.bmm((_silu(gu[..., 0::2].float()) * gu[..., 1::2].float()).to(x.dtype), down.transpose(1, 2))
+    return y.float().sum(0).to(x.dtype)

@@ -99,8 +99,7 @@ def test_latent_rows(path, kw):
     pos = torch.tensor([0, 1, 2, 5, 63, 64, 1000, 4095, 7])
     slots = torch.tensor([4, 9, 0, 31, 17, 2, -1, 30, 16], dtype=torch.int32)
     nw = rnd(s.kv_rank, seed=1, dtype=dt)
-    from pie_b200.models.latent import rope_table
-    table = rope_table(s.rope_base, s.rot_dims, dev)
+    table = s.rotary.frequencies(dev)
     cache = torch.full((2, 16, s.row + 16), 7.0, dtype=dt, device=dev)
     q = lops.latent_rows(qkv.to(dev, dt), pos.to(dev, torch.int32), slots.to(dev), table, nw.to(dev, dt), cache, s, 1e-5, s.row,
                          s.rank_pad, copy_nope=False)
