@@ -356,13 +356,13 @@ def retodra_dict(cfg) -> dict:
 def retodra_shape(layers: int = 32, width: int = 4096, gla_heads: int = 16, gla_dim: int = 128, gla_vdim: int = 256, rank: int = 16,
                   tau: float = 16.0, heads: int = 32, kv_heads: int = 8, dim: int = 128, window: int = 1024, buckets: int = 32,
                   right_heads: int = 16, right_dim: int = 128, right_vdim: int = 128, ff: int = 11008, experts: int = 32,
-                  identity: int = 4, top: int = 4, expert_ff: int = 2048, vocab: int = 128256) -> dict:
-    """config.json dictionary of a model that alternates gated linear attention with a dense feed-forward and parallel
-    mixers with experts."""
+                  identity: int = 4, top: int = 4, expert_ff: int = 2048, vocab: int = 128256, linear_every: int = 2) -> dict:
+    """config.json dictionary of a model of parallel mixers with experts, every `linear_every`-th layer (0: none) gated linear
+    attention with a dense feed-forward instead."""
     spec = []
     decay = [math.exp(-2.0 ** (-8.0 * (h + 1) / right_heads)) for h in range(right_heads)]
     for i in range(layers):
-        if i % 2 == 0:
+        if linear_every and i % linear_every == 0:
             spec.append({"type": "gla", "mixer": {"heads": gla_heads, "dim": gla_dim, "vdim": gla_vdim, "tau": tau, "rank": rank},
                          "mlp": {"kind": "dense", "ff": ff}})
         else:

@@ -513,6 +513,8 @@ LAYERED_PRESETS = {
     "puzutar-8b": (_puzutar_config, puzutar_shape, dict()),
     "retodra-19b": (retodra_config, retodra_shape, dict()),
     "nukelix-20b": (nukelix_config, nukelix_shape, dict()),
+    # parallel mixers and experts only: what `nukelix-20b` is measured beside (a fifth route for the shared expert)
+    "retodra-parallel-20b": (retodra_config, retodra_shape, dict(layers=24, linear_every=0, right_vdim=256, identity=0, top=5)),
     "tiny-puzutar": (_puzutar_config, puzutar_shape, dict(
         layers=3, width=256, heads=2, dim=48, rot_dim=16, vdim=40, kv_rank=64, window=40, ff=384, vocab=32000, groups=2, side=16)),
     "tiny-retodra": (retodra_config, retodra_shape, dict(

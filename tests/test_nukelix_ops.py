@@ -263,7 +263,7 @@ def test_grouped_attention_under_a_custom_mask(path, name):
 
 
 # ------------------------------------------------------------------ matrix memory
-SHAPES = [(1, 1, 1), (3, 7, 11), (2, 32, 64), (2, 40, 24), (1, 128, 128), (3, 96, 36), (1, 200, 64), (1, 272, 24), (2, 64, 260)]
+SHAPES = [(1, 1, 1), (3, 7, 11), (2, 32, 64), (2, 40, 24), (1, 128, 128), (3, 96, 36), (1, 200, 64), (1, 272, 24), (1, 64, 260)]
 
 
 def memory_case(n, h, d, e, dt, kind, width=24):
