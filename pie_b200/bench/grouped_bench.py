@@ -102,7 +102,7 @@ def rows(b: Bench, cfg) -> None:
               lambda: lin.biased_rows(q, k, v, lw["q_norm"], lw["k_norm"], at, cache, biased, 1e-5), 4.0 * y.numel())
         o1, g1, z1 = torch.randn(n, nq, **BF16), torch.randn(n, a.heads, **BF16), torch.empty(n, nq + s.values, **BF16)
         e1, o2, g2 = torch.randn(n, nq, **BF16), torch.randn(n, s.values, device="cuda"), torch.randn(n, s.values, **BF16)
-        w2, den = torch.ones(s.values, **BF16), torch.ones(n, s.heads, device="cuda")
+        w2, den = torch.ones(s.values, **BF16), torch.ones(s.heads, n, device="cuda")
         right = lambda **kw: (o2, w2, g2, z1[:, nq:], dict(act="sigmoid", eps=1e-5, scale=1.0, **kw))
         b.run(f"gates of both mixers, {n} rows", lambda: lin.gated_norm([
             (o1, None, g1, z1[:, :nq], dict(act="sigmoid", norm_cols=0, scale=1.0, spec=a, gate_cols=a.vdim)),

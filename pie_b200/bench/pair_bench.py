@@ -5,9 +5,9 @@
     python bench.py --config 9 [--layers 24]    Nukelix beside Retodra's parallel mixers with experts
 
 Both models of a pair have the same width, heads, window, vocabulary and feed-forward sizes (configs 8 and 9: also the same
-states of the linear mixers, experts and routes per token; a shared expert counts as a route). Device-timed with CUDA events after warm-up. Decode replays
-the captured step over contexts of `--context` tokens; the weights read per step exceed the L2. Prefill runs whole prompts
-as one batch. One JSON line.
+states of the linear mixers, experts and routes per token; a shared expert counts as a route). Device-timed with CUDA
+events after warm-up. Decode replays the captured step over contexts of `--context` tokens; the weights read per step
+exceed the L2. Prefill runs whole prompts as one batch. One JSON line.
 """
 from __future__ import annotations
 
@@ -17,7 +17,8 @@ import json
 
 import numpy as np
 
-PAIRS = {7: ("puzutar-8b", "llama-8b-window"), 8: ("retodra-19b", "gdn-moe-window-19b"), 9: ("nukelix-20b", "retodra-parallel-20b")}
+PAIRS = {7: ("puzutar-8b", "llama-8b-window"), 8: ("retodra-19b", "gdn-moe-window-19b"),
+         9: ("nukelix-20b", "retodra-parallel-20b")}
 DECODE_ROWS = (16, 64, 256)
 PREFILL = ((1, 2048), (4, 2048), (1, 8192))
 

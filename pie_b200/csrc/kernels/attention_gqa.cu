@@ -72,24 +72,57 @@ __global__ void __launch_bounds__(256) gqa_rows_kernel(const GqaRowsArgs a) {
     scale(a.q_norm, iq, nq, sq);
     scale(a.k_norm, ik, nk, sk);
     __syncthreads();
-    // element d of a head at x: rotated, or as it is
-    auto turned = [&](const float* x, int d) {
-        if (d >= a.rot_dims) return x[d];
-        const int p = a.adjacent ? d >> 1 : (d < half ? d : d - half);
-        const bool lower = a.adjacent ? (d & 1) == 0 : d < half;
-        const int other = a.adjacent ? d ^ 1 : (lower ? d + half : d - half);
-        return lower ? x[d] * cs[p] - x[other] * cs[half + p] : x[d] * cs[p] + x[other] * cs[half + p];
-    };
-    auto emit = [&](T* dst, const float* head, int d, bool ok) {
-        float f[VEC];
+    // VEC elements of a head from d on: rotated, or as they are. A vector's partners are neighbours or another vector where
+    // pairs and halves fall on vectors.
+    const bool whole = VEC == 4 && a.rot_dims % 4 == 0 && (a.adjacent || half % 4 == 0);
+    auto head_vec = [&](const float* x, int d, float (&f)[VEC]) {
+        if (VEC == 4 && (whole || d >= a.rot_dims)) {
+            load_vec<VEC>(x + d, f);
+            if (d >= a.rot_dims) return;
+            if (a.adjacent) {
 #pragma unroll
-        for (int e = 0; e < VEC; ++e) f[e] = ok && d + e < a.dim ? turned(head, d + e) : 0.f;
-        store_vec<VEC>(dst, f);
+                for (int e = 0; e + 1 < VEC; e += 2) {
+                    const float c = cs[(d + e) >> 1], sn = cs[half + ((d + e) >> 1)], u = f[e], v = f[e + 1];
+                    f[e] = u * c - v * sn;
+                    f[e + 1] = v * c + u * sn;
+                }
+            } else {
+                const bool lower = d < half;
+                const int p = lower ? d : d - half;
+                float o[VEC], c[VEC], sn[VEC];
+                load_vec<VEC>(x + (lower ? d + half : p), o);
+                load_vec<VEC>(cs + p, c);
+                load_vec<VEC>(cs + half + p, sn);
+#pragma unroll
+                for (int e = 0; e < VEC; ++e) f[e] = f[e] * c[e] + (lower ? -o[e] : o[e]) * sn[e];
+            }
+            return;
+        }
+#pragma unroll
+        for (int e = 0; e < VEC; ++e) {
+            const int i = d + e;
+            f[e] = x[i];
+            if (i >= a.rot_dims) continue;
+            const int p = a.adjacent ? i >> 1 : (i < half ? i : i - half);
+            const bool lower = a.adjacent ? (i & 1) == 0 : i < half;
+            const float o = x[a.adjacent ? i ^ 1 : (lower ? i + half : i - half)];
+            f[e] = f[e] * cs[p] + (lower ? -o : o) * cs[half + p];
+        }
+    };
+    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+    auto emit = [&](T* dst, const float* head) {         // one warp per row of D; null: zeros
+        for (int d = lane * VEC; d < a.D; d += 32 * VEC) {
+            float f[VEC];
+#pragma unroll
+            for (int e = 0; e < VEC; ++e) f[e] = 0.f;
+            if (head && d < a.dim) head_vec(head, d, f);
+            store_vec<VEC>(dst + d, f);
+        }
     };
     T* qo = static_cast<T*>(a.q_out) + (size_t)t * a.kv_heads * a.group_pad * a.D;
-    for (int i = threadIdx.x * VEC; i < a.kv_heads * a.group_pad * a.D; i += 256 * VEC) {
-        const int hp = i / a.D, d = i - hp * a.D, kv = hp / a.group_pad, g = hp - kv * a.group_pad;
-        emit(qo + i, sq + (kv * a.group + g) * a.dim, d, g < a.group);
+    for (int hp = warp; hp < a.kv_heads * a.group_pad; hp += 8) {
+        const int kv = hp / a.group_pad, g = hp - kv * a.group_pad;
+        emit(qo + (size_t)hp * a.D, g < a.group ? sq + (kv * a.group + g) * a.dim : nullptr);
     }
     const int slot = a.slots[t];
     T* base = nullptr;
@@ -97,37 +130,34 @@ __global__ void __launch_bounds__(256) gqa_rows_kernel(const GqaRowsArgs a) {
     if (slot >= 0) {
         off = slot % a.page_size;
         base = static_cast<T*>(a.cache) + (size_t)(slot / a.page_size) * 2 * a.kv_heads * a.page_size * a.D;
-        for (int i = threadIdx.x * VEC; i < a.kv_heads * a.D; i += 256 * VEC) {
-            const int h = i / a.D, d = i - h * a.D;
-            emit(base + ((size_t)h * a.page_size + off) * a.D + d, sk + h * a.dim, d, true);
-        }
+        for (int h = warp; h < a.kv_heads; h += 8) emit(base + ((size_t)h * a.page_size + off) * a.D, sk + h * a.dim);
     }
     if (!base && !a.v_keep) return;
     const T* vr = static_cast<const T*>(a.v) + (size_t)t * a.ld;
     const T* vb = static_cast<const T*>(a.v_b);
-    for (int i = threadIdx.x * VEC; i < a.kv_heads * a.D; i += 256 * VEC) {
-        const int h = i / a.D, d = i - h * a.D;
-        float f[VEC];
+    for (int h = warp; h < a.kv_heads; h += 8)
+        for (int d = lane * VEC; d < a.D; d += 32 * VEC) {
+            float f[VEC];
 #pragma unroll
-        for (int e = 0; e < VEC; ++e) f[e] = 0.f;
-        if (d < a.vdim) {
-            const int at = h * a.vdim + d;
-            float g[VEC];
-            load_vec<VEC>(vr + at, f);
-            if (vb) {
-                load_vec<VEC>(vb + at, g);
+            for (int e = 0; e < VEC; ++e) f[e] = 0.f;
+            if (d < a.vdim) {
+                const int at = h * a.vdim + d;
+                float g[VEC];
+                load_vec<VEC>(vr + at, f);
+                if (vb) {
+                    load_vec<VEC>(vb + at, g);
 #pragma unroll
-                for (int e = 0; e < VEC; ++e) f[e] += g[e];
+                    for (int e = 0; e < VEC; ++e) f[e] += g[e];
+                }
+                if (a.v_keep) store_vec<VEC>(a.v_keep + (size_t)t * nv + at, f);
+                if (a.v_first) {
+                    load_vec<VEC>(a.v_first + (size_t)t * nv + at, g);
+#pragma unroll
+                    for (int e = 0; e < VEC; ++e) f[e] = (1.f - a.mix) * f[e] + a.mix * g[e];
+                }
             }
-            if (a.v_keep) store_vec<VEC>(a.v_keep + (size_t)t * nv + at, f);
-            if (a.v_first) {
-                load_vec<VEC>(a.v_first + (size_t)t * nv + at, g);
-#pragma unroll
-                for (int e = 0; e < VEC; ++e) f[e] = (1.f - a.mix) * f[e] + a.mix * g[e];
-            }
+            if (base) store_vec<VEC>(base + ((size_t)(a.kv_heads + h) * a.page_size + off) * a.D + d, f);
         }
-        if (base) store_vec<VEC>(base + ((size_t)(a.kv_heads + h) * a.page_size + off) * a.D + d, f);
-    }
 }
 
 struct GqaAnyArgs {

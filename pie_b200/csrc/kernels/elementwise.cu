@@ -553,12 +553,29 @@ __global__ void softcap_kernel(T* __restrict__ y, int cols, long ld, float cap) 
     for (int c = blockIdx.x * blockDim.x + threadIdx.x; c < cols; c += gridDim.x * blockDim.x)
         row[c] = (T)(cap * tanhf((float)row[c] / cap));
 }
+// Eight columns at a time; tanh by its exponential, with an absolute error of a few 2^-24.
+__global__ void __launch_bounds__(256) softcap8_kernel(bf16* __restrict__ y, int vecs, long ld, float cap) {
+    pdl_trigger();
+    pdl_wait();
+    bf16x8* row = reinterpret_cast<bf16x8*>(y + blockIdx.y * ld);
+    const float pre = 2.8853900817779268f / cap;
+    for (int c = blockIdx.x * 256 + threadIdx.x; c < vecs; c += gridDim.x * 256) {
+        float f[8];
+        unpack8(row[c], f);
+#pragma unroll
+        for (int e = 0; e < 8; ++e) f[e] = cap * (1.f - __fdividef(2.f, 1.f + exp2f(f[e] * pre)));
+        row[c] = pack8(f);
+    }
+}
 }  // namespace pie
 
 PIE_API int pie_softcap(void* y, int rows, int cols, long ld, float cap, int f32, cudaStream_t st) {
     if (rows <= 0 || cols <= 0) return 0;
     if (cap <= 0.f || rows > 65535) return (int)cudaErrorInvalidValue;
     const dim3 grid(min((cols + 255) / 256, 512), rows);
+    if (!f32 && cols % 8 == 0 && ld % 8 == 0 && ((uintptr_t)y & 15) == 0)
+        return (int)pie::launch_pdl(pie::softcap8_kernel, dim3(min((cols / 8 + 255) / 256, 64), rows), dim3(256), 0, st, (bf16*)y, cols / 8, ld,
+                                    cap);
     if (f32) return (int)pie::launch_pdl(pie::softcap_kernel<float>, grid, dim3(256), 0, st, (float*)y, cols, ld, cap);
     return (int)pie::launch_pdl(pie::softcap_kernel<bf16>, grid, dim3(256), 0, st, (bf16*)y, cols, ld, cap);
 }

@@ -26,8 +26,8 @@ struct LinAttnArgs {
     const void *q, *k, *v;       // row t, head h at t * ld + h * dim (h * vdim for v), type T
     float* log_decay;            // [n, heads * dim] base 2, or null; the chunked form leaves running sums of the pieces
     const float* head_decay;     // [heads] the factor itself (null with log_decay)
-    const float *tok_decay, *tok_input;   // [n, heads] base-2 logarithms of decay and key factor, at most 0 (null with the others)
-    float* den;                  // [n, heads] n_t . q_t (with tok_decay)
+    const float *tok_decay, *tok_input;   // [heads, n] base-2 logarithms of decay and key factor, at most 0 (null with the others)
+    float* den;                  // [heads, n] n_t . q_t (with tok_decay)
     float* out;                  // [n, heads * vdim]
     float* state;                // this layer's part of slot 0: [heads][dim][vdim]
     const int *qo_indptr, *slots, *reset;
@@ -46,22 +46,23 @@ __host__ __device__ __forceinline__ long la_elems(const LinAttnArgs& a) {
 }
 
 // ------------------------------------------------------------------ serial
-template <typename T, int RPT, int VEC>
+template <typename T, int RPT, int VEC, bool TOK>
 __global__ void __launch_bounds__(256) la_serial_kernel(const LinAttnArgs a) {
     constexpr int ROWS = RPT * 8, COLS = 32 * VEC;
     __shared__ float sq[ROWS], sk[ROWS], sa[ROWS];
-    __shared__ float red[8][COLS];
+    __shared__ float red[8][COLS], red_n[8];
     pdl_trigger();
     pdl_wait();
     const int r = blockIdx.x, h = blockIdx.y, lane = threadIdx.x & 31, rg = threadIdx.x >> 5;
     const int first = a.qo_indptr[r], len = a.qo_indptr[r + 1] - first, slot = a.slots[r];
     if (len <= 0 || slot < 0) return;          // a padding request of a decode graph: no state, no output
-    // with a normaliser the last block of a head keeps it: one column whose values are ones
-    const bool ones = a.tok_decay && blockIdx.z == gridDim.z - 1;
-    const int width = ones ? 1 : a.vdim, cb = ones ? 0 : blockIdx.z * COLS, c0 = cb + lane * VEC;
-    const bool col = c0 < width;               // VEC > 1 only where vdim is a multiple of it
-    float* sp = a.state + (size_t)slot * a.slot_stride + (ones ? (size_t)a.heads * a.dim * a.vdim : 0) + (size_t)h * a.dim * width;
-    float S[RPT][VEC];
+    const int c0 = blockIdx.z * COLS + lane * VEC;
+    const bool col = c0 < a.vdim;              // VEC > 1 only where vdim is a multiple of it
+    float* sp = a.state + (size_t)slot * a.slot_stride + (size_t)h * a.dim * a.vdim;
+    // the first block of a head also keeps the normaliser; the lanes of a warp hold the same rows of it
+    const bool norm = TOK && blockIdx.z == 0;
+    float* np = a.state + (size_t)slot * a.slot_stride + (size_t)a.heads * a.dim * a.vdim + (size_t)h * a.dim;
+    float S[RPT][VEC], N[TOK ? RPT : 1];
     const bool fresh = a.reset[r] != 0;
 #pragma unroll
     for (int i = 0; i < RPT; ++i) {
@@ -69,20 +70,20 @@ __global__ void __launch_bounds__(256) la_serial_kernel(const LinAttnArgs a) {
         const bool ok = col && !fresh && d < a.dim;
         if constexpr (VEC == 4) {
             float4 x = make_float4(0.f, 0.f, 0.f, 0.f);
-            if (ok && ones) x.x = sp[d];
-            else if (ok) x = *reinterpret_cast<const float4*>(sp + (size_t)d * a.vdim + c0);
+            if (ok) x = *reinterpret_cast<const float4*>(sp + (size_t)d * a.vdim + c0);
             S[i][0] = x.x; S[i][1] = x.y; S[i][2] = x.z; S[i][3] = x.w;
         } else {
-            S[i][0] = ok ? sp[(size_t)d * width + c0] : 0.f;
+            S[i][0] = ok ? sp[(size_t)d * a.vdim + c0] : 0.f;
         }
+        if constexpr (TOK) N[i] = norm && !fresh && d < a.dim ? np[d] : 0.f;
     }
     const float hd = a.head_decay ? a.head_decay[h] : 1.f;
     for (int t = 0; t < len; ++t) {
         const size_t row = (size_t)(first + t);
         const T* qr = static_cast<const T*>(a.q) + row * a.ld + h * a.dim;
         const T* kr = static_cast<const T*>(a.k) + row * a.ld + h * a.dim;
-        const float td = a.tok_decay ? exp2f(a.tok_decay[row * a.heads + h]) : hd;
-        const float ti = a.tok_decay ? exp2f(a.tok_input[row * a.heads + h]) : 1.f;
+        const float td = TOK ? exp2f(a.tok_decay[(size_t)h * a.n + row]) : hd;
+        const float ti = TOK ? exp2f(a.tok_input[(size_t)h * a.n + row]) : 1.f;
         for (int d = threadIdx.x; d < ROWS; d += 256) {
             float q = 0.f, k = 0.f, g = 1.f;
             if (d < a.dim) {
@@ -98,7 +99,6 @@ __global__ void __launch_bounds__(256) la_serial_kernel(const LinAttnArgs a) {
         float v[VEC];
 #pragma unroll
         for (int j = 0; j < VEC; ++j) {
-            if (ones) { v[j] = lane == 0 && j == 0 ? 1.f : 0.f; continue; }
             v[j] = col ? to_f(static_cast<const T*>(a.v)[row * a.ld + h * a.vdim + c0 + j]) : 0.f;
             if (a.silu) v[j] = la_silu(v[j]);
         }
@@ -106,6 +106,7 @@ __global__ void __launch_bounds__(256) la_serial_kernel(const LinAttnArgs a) {
         float o[VEC];
 #pragma unroll
         for (int j = 0; j < VEC; ++j) o[j] = 0.f;
+        float on = 0.f;
 #pragma unroll
         for (int i = 0; i < RPT; ++i) {
             const int d = rg + 8 * i;
@@ -115,27 +116,37 @@ __global__ void __launch_bounds__(256) la_serial_kernel(const LinAttnArgs a) {
                 S[i][j] = g * S[i][j] + k * v[j];
                 o[j] += q * S[i][j];
             }
+            if constexpr (TOK) {
+                N[i] = g * N[i] + k;
+                on += q * N[i];
+            }
         }
 #pragma unroll
         for (int j = 0; j < VEC; ++j) red[rg][lane * VEC + j] = o[j];
+        if (TOK && lane == 0) red_n[rg] = on;
         __syncthreads();
+        if (norm && threadIdx.x == 0) {
+            float s = 0.f;
+#pragma unroll
+            for (int g = 0; g < 8; ++g) s += red_n[g];
+            a.den[(size_t)h * a.n + row] = s;
+        }
         for (int c = threadIdx.x; c < COLS; c += 256) {
-            const int cc = cb + c;
-            if (cc >= width) continue;
+            const int cc = blockIdx.z * COLS + c;
+            if (cc >= a.vdim) continue;
             float s = 0.f;
 #pragma unroll
             for (int g = 0; g < 8; ++g) s += red[g][c];
-            if (ones) a.den[row * a.heads + h] = s;
-            else a.out[row * a.heads * a.vdim + h * a.vdim + cc] = s;
+            a.out[row * a.heads * a.vdim + h * a.vdim + cc] = s;
         }
     }
 #pragma unroll
     for (int i = 0; i < RPT; ++i) {
         const int d = rg + 8 * i;
+        if constexpr (TOK)
+            if (norm && lane == 0 && d < a.dim) np[d] = N[i];
         if (!col || d >= a.dim) continue;
-        if (ones)
-            sp[d] = S[i][0];
-        else if constexpr (VEC == 4)
+        if constexpr (VEC == 4)
             *reinterpret_cast<float4*>(sp + (size_t)d * a.vdim + c0) = make_float4(S[i][0], S[i][1], S[i][2], S[i][3]);
         else
             sp[(size_t)d * a.vdim + c0] = S[i][0];
@@ -211,7 +222,7 @@ struct ValueTile {
 __device__ __forceinline__ void la_token_sums(const LinAttnArgs& a, int row0, int len, int h, float* sb, float* si, float* half) {
     if (threadIdx.x < LA_C) {
         const int s = threadIdx.x, lane = s & 31;
-        const size_t at = (size_t)(row0 + s) * a.heads + h;
+        const size_t at = (size_t)h * a.n + row0 + s;
         float x = s < len ? a.tok_decay[at] : 0.f;
         si[s] = s < len ? a.tok_input[at] : -INFINITY;
 #pragma unroll
@@ -548,7 +559,7 @@ __global__ void __launch_bounds__(LA_THREADS) la_chunk_out_kernel(const LinAttnA
         for (int d = part; d < a.dim; d += 4) x += sb[q * xp + d] * N[d];
         x += __shfl_xor_sync(0xffffffffu, x, 1);
         x += __shfl_xor_sync(0xffffffffu, x, 2);
-        if (part == 0 && q < len) a.den[(size_t)(row0 + q) * a.heads + h] = x * a.q_scale;
+        if (part == 0 && q < len) a.den[(size_t)h * a.n + row0 + q] = x * a.q_scale;
     }
     constexpr int SV = LA_VT / 4;                 // 16-byte pieces of a state row
     for (int v0 = 0; v0 < a.vdim; v0 += LA_VT) {
@@ -651,9 +662,9 @@ __global__ void __launch_bounds__(256) la_decay_kernel(const T* __restrict__ x, 
 // m_t), key factor exp(i_t - m_t), both at most 1.
 struct MemoryGatesArgs {
     const float *z, *bias;          // `splits` arrays [n, ldz] that add up to (z_i | z_f), heads columns each; [2 * heads]
-    const int *qo_indptr, *slots, *reset, *tok_req;
+    const int *qo_indptr, *slots, *reset;
     float* m;                       // this layer's maxima of slot 0, [heads]
-    float *decay, *input, *floor;   // [n, heads] base-2 logarithms; exp(-m_t)
+    float *decay, *input, *floor;   // [heads, n] base-2 logarithms; exp(-m_t)
     long slot_stride, split_stride;
     int n, reqs, heads, ldz, splits;
     float cap;
@@ -662,6 +673,7 @@ struct MemoryGatesArgs {
 struct MemoryGate { float i, f; };
 __device__ __forceinline__ MemoryGate memory_gate(const MemoryGatesArgs& a, size_t t, int h) {
     float zi = a.bias[h], zf = a.bias[a.heads + h];
+#pragma unroll 4
     for (int s = 0; s < a.splits; ++s) {
         zi += a.z[s * a.split_stride + t * a.ldz + h];
         zf += a.z[s * a.split_stride + t * a.ldz + a.heads + h];
@@ -669,12 +681,12 @@ __device__ __forceinline__ MemoryGate memory_gate(const MemoryGatesArgs& a, size
     const float x = a.cap * tanhf(zf / a.cap);
     return {a.cap * tanhf(zi / a.cap), fminf(x, 0.f) - log1pf(expf(-fabsf(x)))};
 }
-// Writes a token's factors and returns the new maximum.
-__device__ __forceinline__ float memory_step(const MemoryGatesArgs& a, size_t at, MemoryGate g, float m) {
+// A token's factors and the new maximum.
+__device__ __forceinline__ float memory_step(MemoryGate g, float m, float& decay, float& input, float& floor) {
     const float kept = g.f + m, next = fmaxf(kept, g.i);
-    a.decay[at] = (kept - next) * 1.4426950408889634f;
-    a.input[at] = (g.i - next) * 1.4426950408889634f;
-    a.floor[at] = expf(-next);
+    decay = (kept - next) * 1.4426950408889634f;
+    input = (g.i - next) * 1.4426950408889634f;
+    floor = expf(-next);
     return next;
 }
 
@@ -686,57 +698,86 @@ __global__ void __launch_bounds__(128) memory_gates_step_kernel(const MemoryGate
     if (i >= a.reqs * a.heads) return;
     const int r = i / a.heads, h = i - r * a.heads, t = a.qo_indptr[r], slot = a.slots[r];
     if (a.qo_indptr[r + 1] <= t) return;
-    const size_t at = (size_t)t * a.heads + h;
+    const size_t at = (size_t)h * a.n + t;
     if (slot < 0) { a.decay[at] = a.input[at] = a.floor[at] = 0.f; return; }
     float* m = a.m + (size_t)slot * a.slot_stride + h;
-    *m = memory_step(a, at, memory_gate(a, t, h), a.reset[r] ? 0.f : *m);
+    *m = memory_step(memory_gate(a, t, h), a.reset[r] ? 0.f : *m, a.decay[at], a.input[at], a.floor[at]);
 }
 
-// Portions: a block per (request, head). m_t is a composition of maps m -> max(m + F, B): threads compose theirs over equal
-// runs of tokens, a scan over the threads gives each the maximum before its run, which it then walks.
-__global__ void __launch_bounds__(256) memory_gates_kernel(const MemoryGatesArgs a) {
-    __shared__ float sF[8], sB[8];
+// Portions, first pass: the gates' logarithms of every token, f into `decay` and i into `input`.
+__global__ void __launch_bounds__(256) memory_gates_log_kernel(const MemoryGatesArgs a) {
+    pdl_trigger();
+    pdl_wait();
+    const long i = blockIdx.x * 256L + threadIdx.x;
+    if (i >= (long)a.n * a.heads) return;
+    const long t = i / a.heads;
+    const int h = (int)(i - t * a.heads);
+    const MemoryGate g = memory_gate(a, t, h);
+    a.decay[(size_t)h * a.n + t] = g.f;
+    a.input[(size_t)h * a.n + t] = g.i;
+}
+
+// Second pass: a block per (request, head). m_t is a composition of maps m -> max(m + F, B): over tiles of 1024 tokens the
+// threads compose those of four tokens each, a scan gives each the maximum before its tokens, which it then walks.
+constexpr int MG_RUN = 4;
+__global__ void __launch_bounds__(256) memory_gates_scan_kernel(const MemoryGatesArgs a) {
+    __shared__ float sF[2][8], sB[2][8];
     pdl_trigger();
     pdl_wait();
     const int r = blockIdx.x, h = blockIdx.y, first = a.qo_indptr[r], len = a.qo_indptr[r + 1] - first, slot = a.slots[r];
     if (len <= 0 || slot < 0) return;
-    for (int s = threadIdx.x; s < len; s += 256) {
-        const MemoryGate g = memory_gate(a, first + s, h);
-        const size_t at = (size_t)(first + s) * a.heads + h;
-        a.decay[at] = g.f;
-        a.input[at] = g.i;
-    }
-    __syncthreads();
-    const int run = (len + 255) / 256, s0 = min(len, (int)threadIdx.x * run), s1 = min(len, s0 + run);
-    float F = 0.f, B = -INFINITY;
-    for (int s = s0; s < s1; ++s) {
-        const size_t at = (size_t)(first + s) * a.heads + h;
-        F += a.decay[at];
-        B = fmaxf(B + a.decay[at], a.input[at]);
-    }
+    const size_t at = (size_t)h * a.n + first;
     const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
-#pragma unroll
-    for (int o = 1; o < 32; o <<= 1) {               // after the maps of earlier lanes
-        const float pF = __shfl_up_sync(0xffffffffu, F, o), pB = __shfl_up_sync(0xffffffffu, B, o);
-        if (lane >= o) { B = fmaxf(pB + F, B); F += pF; }
-    }
-    if (lane == 31) { sF[warp] = F; sB[warp] = B; }
     float* mp = a.m + (size_t)slot * a.slot_stride + h;
     float m = a.reset[r] ? 0.f : *mp;
-    const float eF = __shfl_up_sync(0xffffffffu, F, 1), eB = __shfl_up_sync(0xffffffffu, B, 1);
-    __syncthreads();
-    for (int w = 0; w < warp; ++w) m = fmaxf(m + sF[w], sB[w]);
-    if (lane) m = fmaxf(m + eF, eB);
-    for (int s = s0; s < s1; ++s) {
-        const size_t at = (size_t)(first + s) * a.heads + h;
-        m = memory_step(a, at, {a.input[at], a.decay[at]}, m);
+    float f[MG_RUN], g[MG_RUN];
+    auto load = [&](int s0) {
+#pragma unroll
+        for (int j = 0; j < MG_RUN; ++j) {
+            f[j] = s0 + j < len ? a.decay[at + s0 + j] : 0.f;
+            g[j] = s0 + j < len ? a.input[at + s0 + j] : -INFINITY;
+        }
+    };
+    load(threadIdx.x * MG_RUN);
+    for (int tile = 0, b = 0; tile < len; tile += 256 * MG_RUN, b ^= 1) {
+        const int s0 = tile + threadIdx.x * MG_RUN;
+        MemoryGate own[MG_RUN];
+        float F = 0.f, B = -INFINITY;
+#pragma unroll
+        for (int j = 0; j < MG_RUN; ++j) {
+            own[j] = {g[j], f[j]};
+            B = fmaxf(B + f[j], g[j]);
+            F += f[j];
+        }
+        if (tile + 256 * MG_RUN < len) load(s0 + 256 * MG_RUN);
+#pragma unroll
+        for (int o = 1; o < 32; o <<= 1) {           // after the maps of earlier lanes
+            const float pF = __shfl_up_sync(0xffffffffu, F, o), pB = __shfl_up_sync(0xffffffffu, B, o);
+            if (lane >= o) { B = fmaxf(pB + F, B); F += pF; }
+        }
+        if (lane == 31) { sF[b][warp] = F; sB[b][warp] = B; }
+        const float eF = __shfl_up_sync(0xffffffffu, F, 1), eB = __shfl_up_sync(0xffffffffu, B, 1);
+        __syncthreads();
+        float x = m;
+#pragma unroll
+        for (int w = 0; w < 8; ++w) {
+            if (w == warp) x = m;
+            m = fmaxf(m + sF[b][w], sB[b][w]);
+        }
+        if (lane) x = fmaxf(x + eF, eB);
+#pragma unroll
+        for (int j = 0; j < MG_RUN; ++j)
+            if (s0 + j < len) {
+                const size_t o = at + s0 + j;
+                x = memory_step(own[j], x, a.decay[o], a.input[o], a.floor[o]);
+            }
+        if (s0 < len && s0 + MG_RUN >= len) *mp = x;
     }
-    if (s1 == len && s0 < len) *mp = m;
 }
 
 // -------------------------------------------------------- norm and gate of a mixer's output
 // dst[t, :] = scale * act(gate) * (rms-normed x) [* w]; the mean square runs over `norm_cols` consecutive columns (0: no
-// norm). gate: one number per `gate_cols` columns, or null. den / floor [n, groups of norm_cols]: what is normed is
+// norm). gate: one number per `gate_cols` columns, or null. den / floor [groups of norm_cols, n]: what is normed is
 // x / (max(|den|, floor) + 1e-6), whose division the norm takes up. Column j of the output is column
 // (head / group * group_pad + head % group) * head_ld + j % head_cols of x, so that x may hold padded heads. Columns from cols
 // to dst_cols are written as zeros.
@@ -794,20 +835,20 @@ __global__ void __launch_bounds__(256) la_gated_norm_kernel(const GatedNormArgs 
     };
     auto squared_size = [&](int group) {
         if (!p.den) return 1.f;
-        const size_t at = (size_t)t * (p.cols / p.norm_cols) + group;
+        const size_t at = (size_t)group * args.n + t;
         const float d = fmaxf(fabsf(p.den[at]), p.floor[at]) + 1e-6f;
         return d * d;
     };
     const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
     if (p.norm_cols == 0) {
-        for (int j = threadIdx.x * VEC; j < p.cols; j += 256 * VEC) {
+        for (int j = threadIdx.x * VEC; j < p.cols; j += blockDim.x * VEC) {
             float v[VEC];
             source(j, v);
             finish(j, v, 1.f, 0);
         }
     } else if (p.norm_cols == p.cols) {
         float ss = 0.f;
-        for (int j = threadIdx.x * VEC; j < p.cols; j += 256 * VEC) {
+        for (int j = threadIdx.x * VEC; j < p.cols; j += blockDim.x * VEC) {
             float v[VEC];
             source(j, v);
             store_vec<VEC>(buf + 32 + j, v);
@@ -815,13 +856,13 @@ __global__ void __launch_bounds__(256) la_gated_norm_kernel(const GatedNormArgs 
             for (int e = 0; e < VEC; ++e) ss += v[e] * v[e];
         }
         const float inv = 1.f / sqrtf(block_sum(ss, buf) / (float)p.cols + p.eps * squared_size(0));
-        for (int j = threadIdx.x * VEC; j < p.cols; j += 256 * VEC) {
+        for (int j = threadIdx.x * VEC; j < p.cols; j += blockDim.x * VEC) {
             float v[VEC];
             load_vec<VEC>(buf + 32 + j, v);
             finish(j, v, inv, j);
         }
     } else {
-        for (int gr = warp; gr < p.cols / p.norm_cols; gr += 8) {
+        for (int gr = warp; gr < p.cols / p.norm_cols; gr += blockDim.x / 32) {
             float ss = 0.f;
             for (int j = lane * VEC; j < p.norm_cols; j += 32 * VEC) {
                 float v[VEC];
@@ -837,7 +878,7 @@ __global__ void __launch_bounds__(256) la_gated_norm_kernel(const GatedNormArgs 
             }
         }
     }
-    for (int j = p.cols + threadIdx.x; j < p.dst_cols; j += 256) dst[j] = from_f<T>(0.f);
+    for (int j = p.cols + threadIdx.x; j < p.dst_cols; j += blockDim.x) dst[j] = from_f<T>(0.f);
 }
 
 }  // namespace pie
@@ -854,9 +895,9 @@ PIE_API int pie_linear_attn_serial(const LinAttnArgs* args, int f32, cudaStream_
     if (a.dim <= 0 || a.dim > 512 || a.vdim <= 0 || !la_decay_ok(a)) return (int)cudaErrorInvalidValue;
     const bool vec = a.vdim % 4 == 0 && a.vdim >= 64 && a.dim <= 256 && a.slot_stride % 4 == 0 && ((uintptr_t)a.state & 15) == 0;
     const int cols = vec ? 128 : 32, rpt = (a.dim + 7) / 8;
-    const dim3 grid(a.reqs, a.heads, (a.vdim + cols - 1) / cols + (a.tok_decay ? 1 : 0));
+    const dim3 grid(a.reqs, a.heads, (a.vdim + cols - 1) / cols);
 #define GO(T_, R_, V_)                                                                                  \
-    return (int)launch_pdl(la_serial_kernel<T_, R_, V_>, grid, dim3(256), 0, st, a)
+    return (int)launch_pdl(a.tok_decay ? la_serial_kernel<T_, R_, V_, true> : la_serial_kernel<T_, R_, V_, false>, grid, dim3(256), 0, st, a)
 #define GO_R(T_)                                                                                        \
     if (vec) {                                                                                          \
         if (rpt <= 4) GO(T_, 4, 4);                                                                     \
@@ -929,7 +970,9 @@ PIE_API int pie_memory_gates(const MemoryGatesArgs* args, int single, cudaStream
     if (a.n <= 0 || a.reqs <= 0) return 0;
     if (a.heads <= 0 || a.cap <= 0.f || a.splits < 1) return (int)cudaErrorInvalidValue;
     if (single) return (int)launch_pdl(memory_gates_step_kernel, dim3((a.reqs * a.heads + 127) / 128), dim3(128), 0, st, a);
-    return (int)launch_pdl(memory_gates_kernel, dim3(a.reqs, a.heads), dim3(256), 0, st, a);
+    const cudaError_t e = launch_pdl(memory_gates_log_kernel, dim3((unsigned)(((long)a.n * a.heads + 255) / 256)), dim3(256), 0, st, a);
+    if (e != cudaSuccess) return (int)e;
+    return (int)launch_pdl(memory_gates_scan_kernel, dim3(a.reqs, a.heads), dim3(256), 0, st, a);
 }
 
 // One or two parts (parts: 1 or 2) over the same tokens.
@@ -938,6 +981,7 @@ PIE_API int pie_gated_norm(const GatedNormArgs* args, int parts, int f32, cudaSt
     if (a.n <= 0) return 0;
     if (parts < 1 || parts > 2) return (int)cudaErrorInvalidValue;
     size_t sm = 0;
+    int widest = 0;
     bool vec = true;
     auto aligned = [](const void* p) { return ((uintptr_t)p & 15) == 0; };
     for (int i = 0; i < parts; ++i) {
@@ -945,6 +989,7 @@ PIE_API int pie_gated_norm(const GatedNormArgs* args, int parts, int f32, cudaSt
         if (p.head_cols <= 0 || p.group <= 0 || p.cols <= 0 || p.gate_cols <= 0 || (p.den && (!p.floor || !p.norm_cols)) ||
             (p.norm_cols && (p.cols % p.norm_cols || !p.w || p.w_cols <= 0)))
             return (int)cudaErrorInvalidValue;
+        widest = p.cols > widest ? p.cols : widest;
         if (p.norm_cols == p.cols) sm = (size_t)(32 + p.cols) * 4 > sm ? (size_t)(32 + p.cols) * 4 : sm;
         vec = vec && p.head_cols % 4 == 0 && p.head_ld % 4 == 0 && p.norm_cols % 4 == 0 && (!p.w || p.w_cols % 4 == 0) &&
               (p.gate_cols == 1 || p.gate_cols % 4 == 0) && p.cols % 4 == 0 && p.ldx % 4 == 0 &&
@@ -959,5 +1004,5 @@ PIE_API int pie_gated_norm(const GatedNormArgs* args, int parts, int f32, cudaSt
         const cudaError_t e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)sm);
         if (e != cudaSuccess) return (int)e;
     }
-    return (int)launch_pdl(kern, grid, dim3(256), sm, st, a);
+    return (int)launch_pdl(kern, grid, dim3(widest <= 2048 ? 128 : 256), sm, st, a);
 }

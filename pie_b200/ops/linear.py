@@ -22,7 +22,7 @@ GUARD = 64              # entries before and after a bias row that the kernels m
 LinAttnArgs = _struct("LinAttnArgs", ("q k v log_decay head_decay tok_decay tok_input den out state qo_indptr slots reset chunk_req "
                                       "chunk_start req_chunks u piece_decay", p), ("slot_stride", i64),
                       ("n ld reqs heads dim vdim silu chunks", i32), ("q_scale", f32))
-MemoryGatesArgs = _struct("MemoryGatesArgs", ("z bias qo_indptr slots reset tok_req m decay input floor", p), ("slot_stride split_stride", i64),
+MemoryGatesArgs = _struct("MemoryGatesArgs", ("z bias qo_indptr slots reset m decay input floor", p), ("slot_stride split_stride", i64),
                           ("n reqs heads ldz splits", i32), ("cap", f32))
 GatedNormPart = _struct("GatedNormPart", ("x w gate dst den floor", p),
                         ("x_f32 ldx head_cols head_ld group group_pad norm_cols w_cols ldg gate_cols ldd cols dst_cols act", i32),
@@ -68,7 +68,7 @@ def chunk_pieces(rs, device):
 
 
 def memory_gates(h, w, bias, spec, rs, state, decode: bool):
-    """Exponential gates of a matrix memory (`MatrixMemorySpec`) on the mixer's input h: (decay, key factor) [N, heads] as
+    """Exponential gates of a matrix memory (`MatrixMemorySpec`) on the mixer's input h: (decay, key factor) [heads, N] as
     base-2 logarithms for `linear_attention`, and exp(-m_t). The running maxima m are the last numbers of `state`, this layer's
     columns of the state cache, and advance. w: rows of the input gates, then of the forget gates; bias 32-bit."""
     from .latent import split_product
@@ -77,8 +77,8 @@ def memory_gates(h, w, bias, spec, rs, state, decode: bool):
     if not h.is_cuda:
         return ref.memory_gates(torch.matmul(h.float(), w.float().t()) + bias, spec, rs, m)
     z = split_product(h, w) if h.dtype == torch.bfloat16 else torch.matmul(h, w.t())[None]
-    out = torch.empty(3, n, heads, dtype=torch.float32, device=h.device)
-    a = MemoryGatesArgs(z=ptr(z), bias=ptr(bias), qo_indptr=ptr(rs.qo_indptr), slots=ptr(rs.slots), reset=ptr(rs.reset), tok_req=ptr(rs.tok_req),
+    out = torch.empty(3, heads, n, dtype=torch.float32, device=h.device)
+    a = MemoryGatesArgs(z=ptr(z), bias=ptr(bias), qo_indptr=ptr(rs.qo_indptr), slots=ptr(rs.slots), reset=ptr(rs.reset),
                         m=ptr(m), decay=ptr(out[0]), input=ptr(out[1]), floor=ptr(out[2]), slot_stride=state.stride(0),
                         split_stride=z.stride(0), n=n, reqs=len(rs.slots_host), heads=heads, ldz=z.stride(1), splits=z.shape[0], cap=spec.gate_cap)
     check(fn("pie_memory_gates")(C.byref(a), 1 if decode else 0, stream_ptr()), "memory_gates")
@@ -90,7 +90,7 @@ def linear_attention(q, k, v, spec, rs, state, decode: bool, log_decay=None, hea
     """o [N, heads * vdim] in 32-bit of S_t = diag(a_t) S_(t-1) + k_t v_t^T, o_t = S_t^T q_t over the ragged batch `rs`.
     q, k, v: column ranges [N, heads * dim (vdim)] of one projection. The decay is per key channel (`log_decay`), per head
     (`head_decay` [heads] 32-bit), or per head and token with a factor on the key (`gates`: both as base-2 logarithms
-    [N, heads]; the state then ends in a normaliser, n_t = a_t n_(t-1) + k_t, and (o, n_t . q_t [N, heads]) is returned).
+    [heads, N]; the state then ends in a normaliser, n_t = a_t n_(t-1) + k_t, and (o, n_t . q_t [heads, N]) is returned).
     `state`: this layer's columns of the state cache [slots, all layers]."""
     n, h, d, e = q.shape[0], spec.heads, spec.dim, spec.vdim
     if not q.is_cuda and gates is not None:
@@ -101,7 +101,7 @@ def linear_attention(q, k, v, spec, rs, state, decode: bool, log_decay=None, hea
         return ref.linear_attention(q.reshape(n, h, d), k.reshape(n, h, d), v.reshape(n, h, e), ld, head_decay,
                                     state.view(state.shape[0], h, d, e), rs, silu, q_scale).view(n, h * e)
     out = torch.empty(n, h * e, dtype=torch.float32, device=q.device)
-    den = torch.empty(n, h, dtype=torch.float32, device=q.device) if gates is not None else None
+    den = torch.empty(h, n, dtype=torch.float32, device=q.device) if gates is not None else None
     tok_decay, tok_input = gates if gates is not None else (None, None)
     a = LinAttnArgs(q=ptr(q), k=ptr(k), v=ptr(v), log_decay=ptr(log_decay), head_decay=ptr(head_decay), tok_decay=ptr(tok_decay),
                     tok_input=ptr(tok_input), den=ptr(den), out=ptr(out), state=ptr(state),
@@ -123,7 +123,7 @@ def gated_norm(parts):
     """Outputs of one mixer or of two side by side: for each part (x, w, gate, dst, kw) dst = RMSNorm(x) * w * act(gate) *
     scale. kw: act "silu" | "sigmoid", norm_cols (columns per mean square, 0: no norm), eps, scale; for attention outputs in
     padded rows `spec` (an attention spec); `cols` of the output where the gate (None: none) has one number per `gate_cols`
-    of them; den and floor [N, groups of norm_cols]: the norm is that of x / (max(|den|, floor) + 1e-6). dst may be a column
+    of them; den and floor [groups of norm_cols, N]: the norm is that of x / (max(|den|, floor) + 1e-6). dst may be a column
     range; the columns after the output's are set to zero."""
     if not parts[0][0].is_cuda:
         for x, w, gate, dst, kw in parts:

@@ -50,12 +50,12 @@ def memory_gates(z, spec, rs, m):
             decay[t], key[t], floor[t] = f[t] + x - new, i[t] - new, torch.exp(-new)
             x = new
         m[slot] = x
-    return decay / math.log(2), key / math.log(2), floor
+    return decay.t() / math.log(2), key.t() / math.log(2), floor.t()
 
 
 def normalised_linear_attention(q, k, v, decay, key, state, rs, q_scale: float):
-    """q, k [N, H, K], v [N, H, V]; base-2 logarithms [N, H]; state [slots, H * K * V + H * K + ..] advances. Returns
-    (S_t^T q_t, n_t . q_t)."""
+    """q, k [N, H, K], v [N, H, V]; base-2 logarithms [H, N]; state [slots, H * K * V + H * K + ..] advances. Returns
+    (S_t^T q_t, n_t . q_t [H, N])."""
     q, k, v = q.float() * q_scale, k.float(), v.float()
     n, h, d, e = q.shape[0], q.shape[1], q.shape[2], v.shape[2]
     out, den = torch.zeros(n, h, e), torch.zeros(n, h)
@@ -67,12 +67,12 @@ def normalised_linear_attention(q, k, v, decay, key, state, rs, q_scale: float):
         if rs.reset_host[r]:
             s, c = torch.zeros_like(s), torch.zeros_like(c)
         for t in range(a, b):
-            g, kt = torch.exp2(decay[t])[:, None], k[t] * torch.exp2(key[t])[:, None]
+            g, kt = torch.exp2(decay[:, t])[:, None], k[t] * torch.exp2(key[:, t])[:, None]
             s = g[..., None] * s + kt[..., None] * v[t][:, None]
             c = g * c + kt
             out[t], den[t] = torch.einsum("hkv,hk->hv", s, q[t]), (c * q[t]).sum(-1)
         state[slot, :h * d * e], state[slot, h * d * e:h * d * (e + 1)] = s.flatten(), c.flatten()
-    return out, den
+    return out, den.t()
 
 
 def gated_norm(x, w, gate, act, scale: float, norm_cols: int, eps: float, gate_cols: int = 1, den=None, floor=None):
@@ -82,7 +82,7 @@ def gated_norm(x, w, gate, act, scale: float, norm_cols: int, eps: float, gate_c
     if norm_cols:
         x = x.view(n, -1, norm_cols)
         if den is not None:
-            x = x / (torch.maximum(den.abs(), floor) + 1e-6)[..., None]
+            x = x / (torch.maximum(den.abs(), floor) + 1e-6).t()[..., None]
         x = x / torch.sqrt((x * x).mean(-1, keepdim=True) + eps)
         x = (x * w.float().view(-1, norm_cols)).reshape(n, c)
     if gate is None:

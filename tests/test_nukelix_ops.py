@@ -288,7 +288,7 @@ def run_memory(x, w, b, q, k, v, spec, rs, state, dev, dt, single):
     decay, key, floor = lin.memory_gates(x.to(dev, dt), w.to(dev, dt), b.to(dev), spec, rs, state, single)
     qq, kk, vv = padded([q, k, v], dev, dt)
     o, den = lin.linear_attention(qq, kk, vv, spec, rs, state, single, q_scale=spec.dim ** -0.5, gates=(decay, key))
-    return (o.view(len(x), spec.heads, spec.vdim) / (torch.maximum(den.abs(), floor) + 1e-6)[..., None]).cpu()
+    return (o.view(len(x), spec.heads, spec.vdim) / (torch.maximum(den.abs(), floor) + 1e-6).t()[..., None]).cpu()
 
 
 def same_heads(got, want, dt, bf16=1e-2):
@@ -359,7 +359,7 @@ def test_matrix_memory_over_a_ragged_batch(path):
 def test_gates_of_single_tokens_and_portions(path):
     """The factors and the floor themselves, over a long portion and token by token; a padding row stays out."""
     dev, dt = path
-    h, n, cap = 3, 70 if dev == "cpu" else 1000, 4.0
+    h, n, cap = 3, 70 if dev == "cpu" else 2500, 4.0
     spec = MatrixMemorySpec(h, 2, 2, cap)
     x, w, b, *_ = memory_case(n, h, 2, 2, dt, "spikes")
     i, f = oracle.log_gates(x.double(), {"i": w[:h].double(), "f": w[h:].double(), "i.b": b[:h].double(), "f.b": b[h:].double()}, cap)
@@ -375,8 +375,9 @@ def test_gates_of_single_tokens_and_portions(path):
     steps, short = [], 40
     for t in range(short):
         rs = recurrent([0, 1, 2], [1, -1], [1 if t == 0 else 0, 0], dev)
-        steps.append(torch.stack(lin.memory_gates(xs[[t, t]], ws, bs, spec, rs, state, True))[:, 0].cpu())
-    for got, ref in ((whole, want), (torch.stack(steps, 1), want[:, :short])):
+        steps.append(torch.stack(lin.memory_gates(xs[[t, t]], ws, bs, spec, rs, state, True))[..., 0].cpu())
+    want = want.transpose(1, 2)
+    for got, ref in ((whole, want), (torch.stack(steps, -1), want[..., :short])):
         close(got[0] * np.log(2), ref[0], F32, f32=2e-5)
         close(got[1] * np.log(2), ref[1], F32, f32=2e-5)
         close(got[2], ref[2], F32, f32=2e-5)
@@ -403,7 +404,7 @@ def test_gates_per_head_and_norm_of_a_quotient(path, heads, kv, vdim, rh, rv):
     z = torch.full((n, cut + rh * rv + 8), 5.0, dtype=dt, device=dev)
     lin.gated_norm([(x.view(n, -1).to(dev, dt), None, ga, z[:, :cut], dict(act="sigmoid", norm_cols=0, scale=0.7, spec=spec, gate_cols=vdim)),
                     (right.reshape(n, -1).to(dev), w.to(dev, dt), gb, z[:, cut:],
-                     dict(act="sigmoid", norm_cols=rv, eps=eps, scale=1.3, den=den.to(dev), floor=floor.to(dev)))])
+                     dict(act="sigmoid", norm_cols=rv, eps=eps, scale=1.3, den=den.t().contiguous().to(dev), floor=floor.t().contiguous().to(dev)))])
     close(z[:, :heads * vdim], 0.7 * oracle.head_gate(left, g1, torch.eye(heads)).reshape(n, -1), dt)
     o = right / (torch.maximum(den.abs(), floor) + 1e-6)[..., None]
     close(z[:, cut:cut + rh * rv], 1.3 * oracle.rms(o, eps).reshape(n, -1) * w * oracle.sigmoid(g2), dt)
