@@ -50,7 +50,7 @@ template <typename T, int RPT, int VEC, bool TOK>
 __global__ void __launch_bounds__(256) la_serial_kernel(const LinAttnArgs a) {
     constexpr int ROWS = RPT * 8, COLS = 32 * VEC;
     __shared__ float sq[ROWS], sk[ROWS], sa[ROWS];
-    __shared__ float red[8][COLS], red_n[8];
+    __shared__ float red[8][COLS], sn[2][TOK ? ROWS : 1];
     pdl_trigger();
     pdl_wait();
     const int r = blockIdx.x, h = blockIdx.y, lane = threadIdx.x & 31, rg = threadIdx.x >> 5;
@@ -59,11 +59,17 @@ __global__ void __launch_bounds__(256) la_serial_kernel(const LinAttnArgs a) {
     const int c0 = blockIdx.z * COLS + lane * VEC;
     const bool col = c0 < a.vdim;              // VEC > 1 only where vdim is a multiple of it
     float* sp = a.state + (size_t)slot * a.slot_stride + (size_t)h * a.dim * a.vdim;
-    // the first block of a head also keeps the normaliser; the lanes of a warp hold the same rows of it
+    // the first block of a head also keeps the normaliser, the rows each thread stages
+    constexpr int NR = (ROWS + 255) / 256;
     const bool norm = TOK && blockIdx.z == 0;
     float* np = a.state + (size_t)slot * a.slot_stride + (size_t)a.heads * a.dim * a.vdim + (size_t)h * a.dim;
-    float S[RPT][VEC], N[TOK ? RPT : 1];
+    float S[RPT][VEC], N[NR];
     const bool fresh = a.reset[r] != 0;
+#pragma unroll
+    for (int i = 0; i < NR; ++i) {
+        const int d = threadIdx.x + i * 256;
+        N[i] = norm && !fresh && d < a.dim ? np[d] : 0.f;
+    }
 #pragma unroll
     for (int i = 0; i < RPT; ++i) {
         const int d = rg + 8 * i;
@@ -75,7 +81,6 @@ __global__ void __launch_bounds__(256) la_serial_kernel(const LinAttnArgs a) {
         } else {
             S[i][0] = ok ? sp[(size_t)d * a.vdim + c0] : 0.f;
         }
-        if constexpr (TOK) N[i] = norm && !fresh && d < a.dim ? np[d] : 0.f;
     }
     const float hd = a.head_decay ? a.head_decay[h] : 1.f;
     for (int t = 0; t < len; ++t) {
@@ -84,7 +89,10 @@ __global__ void __launch_bounds__(256) la_serial_kernel(const LinAttnArgs a) {
         const T* kr = static_cast<const T*>(a.k) + row * a.ld + h * a.dim;
         const float td = TOK ? exp2f(a.tok_decay[(size_t)h * a.n + row]) : hd;
         const float ti = TOK ? exp2f(a.tok_input[(size_t)h * a.n + row]) : 1.f;
-        for (int d = threadIdx.x; d < ROWS; d += 256) {
+#pragma unroll
+        for (int i = 0; i < NR; ++i) {
+            const int d = threadIdx.x + i * 256;
+            if (d >= ROWS) break;
             float q = 0.f, k = 0.f, g = 1.f;
             if (d < a.dim) {
                 q = to_f(qr[d]);
@@ -95,6 +103,10 @@ __global__ void __launch_bounds__(256) la_serial_kernel(const LinAttnArgs a) {
             sq[d] = q * a.q_scale;
             sk[d] = k * ti;
             sa[d] = g;
+            if (norm) {
+                N[i] = g * N[i] + k * ti;
+                sn[t & 1][d] = q * a.q_scale * N[i];
+            }
         }
         float v[VEC];
 #pragma unroll
@@ -106,7 +118,6 @@ __global__ void __launch_bounds__(256) la_serial_kernel(const LinAttnArgs a) {
         float o[VEC];
 #pragma unroll
         for (int j = 0; j < VEC; ++j) o[j] = 0.f;
-        float on = 0.f;
 #pragma unroll
         for (int i = 0; i < RPT; ++i) {
             const int d = rg + 8 * i;
@@ -116,20 +127,16 @@ __global__ void __launch_bounds__(256) la_serial_kernel(const LinAttnArgs a) {
                 S[i][j] = g * S[i][j] + k * v[j];
                 o[j] += q * S[i][j];
             }
-            if constexpr (TOK) {
-                N[i] = g * N[i] + k;
-                on += q * N[i];
-            }
         }
 #pragma unroll
         for (int j = 0; j < VEC; ++j) red[rg][lane * VEC + j] = o[j];
-        if (TOK && lane == 0) red_n[rg] = on;
         __syncthreads();
-        if (norm && threadIdx.x == 0) {
+        if (norm && rg == 7) {                 // the other buffer is written before every warp has read this one
             float s = 0.f;
 #pragma unroll
-            for (int g = 0; g < 8; ++g) s += red_n[g];
-            a.den[(size_t)h * a.n + row] = s;
+            for (int d = lane; d < ROWS; d += 32) s += sn[t & 1][d];
+            s = warp_sum(s);
+            if (lane == 0) a.den[(size_t)h * a.n + row] = s;
         }
         for (int c = threadIdx.x; c < COLS; c += 256) {
             const int cc = blockIdx.z * COLS + c;
@@ -143,14 +150,15 @@ __global__ void __launch_bounds__(256) la_serial_kernel(const LinAttnArgs a) {
 #pragma unroll
     for (int i = 0; i < RPT; ++i) {
         const int d = rg + 8 * i;
-        if constexpr (TOK)
-            if (norm && lane == 0 && d < a.dim) np[d] = N[i];
         if (!col || d >= a.dim) continue;
         if constexpr (VEC == 4)
             *reinterpret_cast<float4*>(sp + (size_t)d * a.vdim + c0) = make_float4(S[i][0], S[i][1], S[i][2], S[i][3]);
         else
             sp[(size_t)d * a.vdim + c0] = S[i][0];
     }
+#pragma unroll
+    for (int i = 0; i < NR; ++i)
+        if (norm && threadIdx.x + i * 256 < a.dim) np[threadIdx.x + i * 256] = N[i];
 }
 
 // ----------------------------------------------------------------- chunked
@@ -673,7 +681,7 @@ struct MemoryGatesArgs {
 struct MemoryGate { float i, f; };
 __device__ __forceinline__ MemoryGate memory_gate(const MemoryGatesArgs& a, size_t t, int h) {
     float zi = a.bias[h], zf = a.bias[a.heads + h];
-#pragma unroll 4
+#pragma unroll 8
     for (int s = 0; s < a.splits; ++s) {
         zi += a.z[s * a.split_stride + t * a.ldz + h];
         zf += a.z[s * a.split_stride + t * a.ldz + a.heads + h];
