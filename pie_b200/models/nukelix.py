@@ -76,7 +76,7 @@ def nukelix_config(cfg: dict, name: str):
         num_key_value_heads=max((a.kv_heads for a in att), default=1),
         head_dim=max([a.head_dim for a in att] + [s.row for s in lat]), vocab_size=cfg["vocab"],
         max_position_embeddings=cfg.get("max_position_embeddings", 131072), rms_norm_eps=cfg["norm"]["eps"], tie_word_embeddings=True,
-        post_norm=True, final_softcap=float(cfg["logit_softcap"]), blocks=blocks, dtype="bfloat16", name=name)
+        post_norm=True, final_softcap=float(cfg.get("logit_softcap") or 0.0), blocks=blocks, dtype="bfloat16", name=name)
 
 
 def _grouped_dict(a: GroupedAttentionSpec) -> dict:
