@@ -38,6 +38,10 @@ SANDWICH_SOURCES = ("attention_bias", "elementwise", "gdn", "gemm2_tcgen05", "ge
 POST_NORM_SOURCES = ("attention", "attention_gqa", "attention_tc", "elementwise", "gdn", "gemm2_tcgen05", "gemm_tcgen05", "latent",
                      "latent_attn", "latent_attn_tc", "linear_attn", "moe", "sampling")
 
+# sources whose kernels blocks that read the stream through a layer norm and a convolution launch
+LAYER_NORM_SOURCES = ("attention_gqa", "attention_pool", "attention_tc", "delta_rule", "elementwise", "gdn", "gemm2_tcgen05", "gemm_tcgen05",
+                      "latent", "latent_attn", "linear_attn", "sampling", "stream_conv")
+
 NVCC_FLAGS = [
     "-gencode", "arch=compute_100a,code=sm_100a", "-lineinfo", "-O3", "-std=c++17",
     "--expt-relaxed-constexpr", "-Xcompiler", "-fPIC", "-Xcompiler", "-fvisibility=hidden",
@@ -104,6 +108,8 @@ def kernels_for(cfg) -> Path:
         return KERNEL_LIB
     if cfg.latent is not None:
         return build_kernels(only=LATENT_SOURCES, target=OUT / "libpie_kernels_latent.so")
+    if cfg.blocks is not None and cfg.layer_norm:
+        return build_kernels(only=LAYER_NORM_SOURCES, target=OUT / "libpie_kernels_layer_norm.so")
     if cfg.blocks is not None and cfg.post_norm:
         return build_kernels(only=POST_NORM_SOURCES, target=OUT / "libpie_kernels_post_norm.so")
     if cfg.blocks is not None:

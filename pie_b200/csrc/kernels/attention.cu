@@ -58,7 +58,7 @@ static int launch_decode(const void* q, const void* kv_layer, const int* page_in
                 (const bf16*)q, (const bf16*)kv_layer, page_indices, kv_page_indptr, item_req,
                 item_start, item_end, req_item_indptr, num_items_ptr, (bf16*)out, o_part, lse_part, hq,
                 hkv, page_size, scale_log2, window_left, sinks_log2, max_items, num_reqs, pie_status_word_current(),
-                (const int*)nullptr, (const int*)nullptr, (const int*)nullptr, cap_log2, (const float*)nullptr, 0, keep_first);
+                (const int*)nullptr, (const int*)nullptr, (const int*)nullptr, cap_log2, (const float*)nullptr, 0, keep_first, KeyLayout());
         } else if (cascade) {
             auto kern = paged_decode_attn_kernel<D, G, true>;
             cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, SM);
@@ -66,7 +66,7 @@ static int launch_decode(const void* q, const void* kv_layer, const int* page_in
                 (const bf16*)q, (const bf16*)kv_layer, page_indices, kv_page_indptr, item_req,
                 item_start, item_end, req_item_indptr, num_items_ptr, (bf16*)out, o_part, lse_part, hq,
                 hkv, page_size, scale_log2, window_left, sinks_log2, max_items, num_reqs, pie_status_word_current(),
-                item_slot, item_tile, tile_members, 0.f, (const float*)nullptr, 0, 0);
+                item_slot, item_tile, tile_members, 0.f, (const float*)nullptr, 0, 0, KeyLayout());
         } else {
             auto kern = paged_decode_attn_kernel<D, G, false>;
             cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, SM);
@@ -74,7 +74,7 @@ static int launch_decode(const void* q, const void* kv_layer, const int* page_in
                 (const bf16*)q, (const bf16*)kv_layer, page_indices, kv_page_indptr, item_req,
                 item_start, item_end, req_item_indptr, num_items_ptr, (bf16*)out, o_part, lse_part, hq,
                 hkv, page_size, scale_log2, window_left, sinks_log2, max_items, num_reqs, pie_status_word_current(),
-                (const int*)nullptr, (const int*)nullptr, (const int*)nullptr, 0.f, (const float*)nullptr, 0, keep_first);
+                (const int*)nullptr, (const int*)nullptr, (const int*)nullptr, 0.f, (const float*)nullptr, 0, keep_first, KeyLayout());
         }
     });
     int err = (int)cudaGetLastError();
@@ -207,14 +207,14 @@ PIE_API int pie_paged_prefill_attn_kept(const void* q, const void* kv_layer, con
             kern<<<grid, PF_WARPS * 32, SM, st>>>(
                 (const bf16*)q, (const bf16*)kv_layer, page_indices, kv_page_indptr, qo_indptr, kv_lens,
                 tile_req, tile_qstart, mask_bits, mask_word_indptr, (bf16*)out, lse_out, sinks_log2, hq, hkv,
-                page_size, scale_log2, window_left, cap_log2, nullptr, 0, keep_first);
+                page_size, scale_log2, window_left, cap_log2, nullptr, 0, keep_first, KeyLayout());
         } else {
             auto kern = paged_prefill_attn_kernel<D, G>;
             cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, SM);
             kern<<<grid, PF_WARPS * 32, SM, st>>>(
                 (const bf16*)q, (const bf16*)kv_layer, page_indices, kv_page_indptr, qo_indptr, kv_lens,
                 tile_req, tile_qstart, mask_bits, mask_word_indptr, (bf16*)out, lse_out, sinks_log2, hq, hkv,
-                page_size, scale_log2, window_left, 0.f, nullptr, 0, keep_first);
+                page_size, scale_log2, window_left, 0.f, nullptr, 0, keep_first, KeyLayout());
         }
     });
     return (int)cudaGetLastError();

@@ -213,7 +213,7 @@ PIE_API int pie_biased_decode(const BiasedAttnArgs* args, cudaStream_t st) {
                            a.kv_page_indptr, a.item_req, a.item_start, a.item_end, a.req_item_indptr, a.num_items, (bf16*)a.out, a.scratch,
                            lse, a.hq, a.hkv, a.page_size, a.scale / a.softcap, a.window_left, (const float*)nullptr, a.max_items,
                            a.num_reqs, pie_status_word_current(), (const int*)nullptr, (const int*)nullptr, (const int*)nullptr,
-                           a.softcap * 1.4426950408889634f, a.bias, a.bias_pitch, 0);
+                           a.softcap * 1.4426950408889634f, a.bias, a.bias_pitch, 0, KeyLayout());
         if (e == cudaSuccess)
             e = launch_pdl(paged_decode_merge_kernel<D>, dim3(a.num_reqs, a.hq), dim3(D), 0, st, (const float*)a.scratch, (const float*)lse,
                            a.req_item_indptr, (bf16*)a.out, a.hq, a.hkv, group, (const float*)nullptr, a.max_items);
@@ -238,7 +238,8 @@ PIE_API int pie_biased_prefill(const BiasedAttnArgs* args, int tile_rows, int* s
             if (e != cudaSuccess) return (int)e;
             kern<<<grid, PF_WARPS * 32, SM, st>>>((const bf16*)a.q, (const bf16*)a.kv, a.page_indices, a.kv_page_indptr, a.qo_indptr,
                                                   a.kv_lens, a.tile_req, a.tile_qstart, a.mask_bits, a.mask_word_indptr, (bf16*)a.out,
-                                                  nullptr, nullptr, a.hq, a.hkv, a.page_size, pre, a.window_left, post, a.bias, a.bias_pitch, 0);
+                                                  nullptr, nullptr, a.hq, a.hkv, a.page_size, pre, a.window_left, post, a.bias, a.bias_pitch, 0,
+                                                  KeyLayout());
             return (int)cudaGetLastError();
         });
         return (int)cudaErrorInvalidValue;
@@ -268,7 +269,7 @@ PIE_API int pie_biased_prefill(const BiasedAttnArgs* args, int tile_rows, int* s
         const size_t smem = Cfg::SMEM + (in_smem ? table : 0);                                                                   \
         const cudaError_t e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);                \
         if (e != cudaSuccess) return (int)e;                                                                                     \
-        kern<<<grid, Cfg::THREADS, smem, st>>>(tq, tkv, a.page_indices, a.kv_page_indptr, a.qo_indptr, a.kv_lens, a.tile_req,    \
+        kern<<<grid, Cfg::THREADS, smem, st>>>(tq, tkv, tkv, TcMeans(), 2, a.page_indices, a.kv_page_indptr, a.qo_indptr, a.kv_lens, a.tile_req,    \
                                                a.tile_qstart, a.mask_bits, a.mask_word_indptr, (bf16*)a.out, nullptr, nullptr,   \
                                                a.hq, a.hkv, a.total_pages - 1, 1.f, a.window_left, status, pre, post,            \
                                                a.hq * D_, D_, a.bias, a.bias_pitch, in_smem, 0);                                  \

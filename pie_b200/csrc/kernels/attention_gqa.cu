@@ -2,6 +2,7 @@
 // and rotated in part:
 //
 //   pie_gqa_rows   bias, RMS norm over the whole projection, rotation, value mixing, padded query rows, page writes
+//   pie_head_rows  the same without biases, with a norm per head or none, half-apart pairs, a factor on the query by position
 //   pie_gqa_any    attention, one warp per (token, head): any sizes, bf16 or true 32-bit
 //
 // Keys and values live in the ordinary KV pages ([pages][2][hkv][page][D], zeros past a head's own sizes); attention on
@@ -160,13 +161,114 @@ __global__ void __launch_bounds__(256) gqa_rows_kernel(const GqaRowsArgs a) {
         }
 }
 
+struct HeadRowsArgs {
+    const void *q, *k, *v;          // row t at t * ld: heads x dim, kv_heads x dim, kv_heads x vdim; v null: the values are the keys
+    const float *q_norm, *k_norm;   // [dim], or null
+    const int *positions, *slots;   // KV slot of every token (< 0: no write)
+    const float* inv_freq;          // [rot_dims / 2]
+    void* q_out;                    // [n][kv_heads * group_pad][D]
+    void* cache;                    // this layer's pages, two planes or (v null) one
+    int n, ld, heads, kv_heads, group, group_pad, dim, vdim, D, page_size, rot_dims, temp_every;   // temp_every 0: no factor
+    float eps, rot_factor, temp_coef;
+};
+
+// One block per token; a warp takes a head at a time through its row in shared memory, where a rotated element finds its
+// partner. The factor on the query at position p is 1 + temp_coef * ln(floor((p + 1) / temp_every) + 1).
+template <typename T, int VEC>
+__global__ void __launch_bounds__(256) head_rows_kernel(const HeadRowsArgs a) {
+    extern __shared__ __align__(16) float sm[];
+    pdl_trigger();
+    const int t = blockIdx.x, half = a.rot_dims / 2, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+    float* cs = sm;                     // [half] cos, [half] sin
+    float* row = cs + (a.rot_dims + 3) / 4 * 4 + warp * ((a.dim + 3) / 4 * 4);
+    pdl_wait();
+    const int pos = a.positions[t];
+    for (int i = threadIdx.x; i < half; i += 256) {
+        float s, c;
+        sincosf((float)pos * a.inv_freq[i], &s, &c);
+        cs[i] = c * a.rot_factor;
+        cs[half + i] = s * a.rot_factor;
+    }
+    __syncthreads();
+    const float temp = a.temp_every ? 1.f + a.temp_coef * logf((float)((pos + 1) / a.temp_every) + 1.f) : 1.f;
+    auto emit = [&](T* dst, const T* src, int n, const float* norm, bool turn, float scale) {       // src null: zeros
+        float inv = 1.f;
+        if (src && norm) {
+            float ss = 0.f;
+            for (int d = lane * VEC; d < n; d += 32 * VEC) {
+                float f[VEC];
+                load_vec<VEC>(src + d, f);
+#pragma unroll
+                for (int e = 0; e < VEC; ++e) ss += f[e] * f[e];
+            }
+            inv = 1.f / sqrtf(warp_sum(ss) / (float)n + a.eps);
+        }
+        turn = turn && src && half > 0;
+        auto value = [&](int d, float (&f)[VEC]) {
+            load_vec<VEC>(src + d, f);
+            if (norm) {
+                float g[VEC];
+                load_vec<VEC>(norm + d, g);
+#pragma unroll
+                for (int e = 0; e < VEC; ++e) f[e] *= inv * g[e];
+            }
+        };
+        if (turn) {
+            __syncwarp();
+            for (int d = lane * VEC; d < n; d += 32 * VEC) {
+                float f[VEC];
+                value(d, f);
+                store_vec<VEC>(row + d, f);
+            }
+            __syncwarp();
+        }
+        for (int d = lane * VEC; d < a.D; d += 32 * VEC) {
+            float f[VEC];
+#pragma unroll
+            for (int e = 0; e < VEC; ++e) f[e] = 0.f;
+            if (src && d < n) {
+                if (turn) {
+#pragma unroll
+                    for (int e = 0; e < VEC; ++e) {
+                        const int i = d + e, p = i < half ? i : i - half;
+                        f[e] = row[i];
+                        if (i < a.rot_dims) f[e] = f[e] * cs[p] + (i < half ? -row[i + half] : row[p]) * cs[half + p];
+                    }
+                } else {
+                    value(d, f);
+                }
+#pragma unroll
+                for (int e = 0; e < VEC; ++e) f[e] *= scale;
+            }
+            store_vec<VEC>(dst + d, f);
+        }
+    };
+    const T* q = static_cast<const T*>(a.q) + (size_t)t * a.ld;
+    T* qo = static_cast<T*>(a.q_out) + (size_t)t * a.kv_heads * a.group_pad * a.D;
+    const int nq = a.kv_heads * a.group_pad, slot = a.slots[t], planes = a.v ? 2 : 1;
+    T* base = slot < 0 ? nullptr : static_cast<T*>(a.cache) + (size_t)(slot / a.page_size) * planes * a.kv_heads * a.page_size * a.D;
+    for (int u = warp; u < nq + (base ? planes * a.kv_heads : 0); u += 8) {
+        if (u < nq) {
+            const int kv = u / a.group_pad, g = u - kv * a.group_pad;
+            emit(qo + (size_t)u * a.D, g < a.group ? q + (kv * a.group + g) * a.dim : nullptr, a.dim, a.q_norm, true, temp);
+            continue;
+        }
+        T* dst = base + ((size_t)(u - nq) * a.page_size + slot % a.page_size) * a.D;
+        const int h = (u - nq) % a.kv_heads;
+        if (u - nq < a.kv_heads) emit(dst, static_cast<const T*>(a.k) + (size_t)t * a.ld + h * a.dim, a.dim, a.k_norm, true, 1.f);
+        else emit(dst, static_cast<const T*>(a.v) + (size_t)t * a.ld + h * a.vdim, a.vdim, nullptr, false, 1.f);
+    }
+}
+
 struct GqaAnyArgs {
     const void *q, *kv;             // [n][hq][D], this layer's pages
     void* out;                      // [n][hq][D]
+    const float* sink_scores;       // [hq] natural logarithms, or null
+    const void* means;              // with pool: means of key and value blocks, see KeyLayout in attention_mma.cuh
     const int *page_indices, *kv_page_indptr, *kv_lens, *qo_indptr, *tok_req, *slots;
     const uint32_t* mask_bits;      // custom mask words, or null (causal)
     const long* mask_word_indptr;
-    int n, hq, hkv, D, page_size, window_left, keep_first, sink;   // window_left < 0: no window
+    int n, hq, hkv, D, page_size, window_left, keep_first, sink, planes, pool, per_page;   // window_left < 0: no window; sink: a score of 0
     float scale;
 };
 
@@ -194,12 +296,8 @@ __global__ void __launch_bounds__(128) gqa_any_kernel(const GqaAnyArgs a) {
         const int* pages = a.page_indices + a.kv_page_indptr[r];
         const int hi = bits ? kv_len : pos + 1, lo = a.window_left >= 0 ? max(0, pos - a.window_left) : 0;
         if (a.sink) { m = 0.f; l = 1.f; }
-        for (int j = 0; j < hi; ++j) {
-            if (j >= a.keep_first && j < lo) { j = lo - 1; continue; }
-            if (bits && !(bits[j >> 5] >> (j & 31) & 1u)) continue;
-            const T* kr = static_cast<const T*>(a.kv) +
-                          (((size_t)pages[j / a.page_size] * 2 * a.hkv + kvh) * a.page_size + j % a.page_size) * a.D;
-            const T* vr = kr + (size_t)a.hkv * a.page_size * a.D;
+        if (a.sink_scores) { m = a.sink_scores[h]; l = 1.f; }
+        auto attend = [&](const T* kr, const T* vr) {
             float s = 0.f, v[ME];
 #pragma unroll
             for (int i = 0; i < ME; ++i) {
@@ -213,6 +311,23 @@ __global__ void __launch_bounds__(128) gqa_any_kernel(const GqaAnyArgs a) {
             l = l * c + p;
 #pragma unroll
             for (int i = 0; i < ME; ++i) acc[i] = acc[i] * c + p * v[i];
+        };
+        auto hidden = [&](int j) { return bits && !(bits[j >> 5] >> (j & 31) & 1u); };
+        // the mean of a block counts once the block lies before the window, and under a mask if that shows all its tokens
+        for (int b = 0; a.pool && b < lo / a.pool; ++b) {
+            bool whole = true;
+            for (int j = b * a.pool; bits && j < (b + 1) * a.pool; ++j) whole = whole && !hidden(j);
+            if (!whole) continue;
+            const int page_at = ((b + 1) * a.pool - 1) / a.page_size, row = b - page_at * a.page_size / a.pool;
+            const T* kr = static_cast<const T*>(a.means) + (((size_t)pages[page_at] * 2 * a.hkv + kvh) * a.per_page + row) * a.D;
+            attend(kr, kr + (size_t)a.hkv * a.per_page * a.D);
+        }
+        for (int j = 0; j < hi; ++j) {
+            if (j >= a.keep_first && j < lo) { j = lo - 1; continue; }
+            if (hidden(j)) continue;
+            const T* kr = static_cast<const T*>(a.kv) +
+                          (((size_t)pages[j / a.page_size] * a.planes * a.hkv + kvh) * a.page_size + j % a.page_size) * a.D;
+            attend(kr, kr + (size_t)(a.planes - 1) * a.hkv * a.page_size * a.D);
         }
     }
     const float inv = l > 0.f ? 1.f / l : 0.f;
@@ -249,10 +364,28 @@ PIE_API int pie_gqa_rows(const GqaRowsArgs* args, int f32, cudaStream_t st) {
     return (int)launch_pdl(kern, dim3(a.n), dim3(256), sm, st, a);
 }
 
+PIE_API int pie_head_rows(const HeadRowsArgs* args, int f32, cudaStream_t st) {
+    const HeadRowsArgs& a = *args;
+    if (a.n <= 0) return 0;
+    if (a.group > a.group_pad || a.heads != a.kv_heads * a.group || a.dim > a.D || a.vdim > a.D || a.rot_dims % 2 || a.rot_dims > a.dim ||
+        a.page_size <= 0 || a.temp_every < 0 || (!a.q_norm) != (!a.k_norm))
+        return (int)cudaErrorInvalidValue;
+    auto aligned = [](const void* p) { return ((uintptr_t)p & 15) == 0; };
+    const bool vec = a.dim % 4 == 0 && a.vdim % 4 == 0 && a.D % 4 == 0 && a.ld % 4 == 0 && aligned(a.q) && aligned(a.k) && aligned(a.v) &&
+                     aligned(a.q_norm) && aligned(a.k_norm) && aligned(a.q_out) && aligned(a.cache);
+    const int sm = ((a.rot_dims + 3) / 4 * 4 + 8 * ((a.dim + 3) / 4 * 4)) * 4;
+    if (sm > 48 * 1024) return (int)cudaErrorInvalidValue;
+    auto kern = f32 ? (vec ? head_rows_kernel<float, 4> : head_rows_kernel<float, 1>)
+                    : (vec ? head_rows_kernel<bf16, 4> : head_rows_kernel<bf16, 1>);
+    return (int)launch_pdl(kern, dim3(a.n), dim3(256), sm, st, a);
+}
+
 PIE_API int pie_gqa_any(const GqaAnyArgs* args, int f32, cudaStream_t st) {
     const GqaAnyArgs& a = *args;
     if (a.n <= 0) return 0;
-    if (a.hkv <= 0 || a.hq % a.hkv || a.D > 1024 || a.page_size <= 0 || a.keep_first < 0) return (int)cudaErrorInvalidValue;
+    if (a.hkv <= 0 || a.hq % a.hkv || a.D > 1024 || a.page_size <= 0 || a.keep_first < 0 || (a.planes != 1 && a.planes != 2) ||
+        (a.pool && (a.pool < 0 || !a.means || a.window_left < 0)))
+        return (int)cudaErrorInvalidValue;
     const dim3 grid((unsigned)(((long)a.n * a.hq + 3) / 4));
 #define GO(T_, M_) return (int)launch_pdl(gqa_any_kernel<T_, M_>, grid, dim3(128), 0, st, a)
 #define GO_M(T_) \

@@ -217,7 +217,27 @@ constexpr int decode_smem_bytes() {
 // MODE_BIAS: `bias` [hq][bias_pitch] holds BIAS_GUARD guard entries, the bias of every distance the window shows, and a
 // guard again.
 constexpr int BIAS_GUARD = 64;
-template <int D, int G, bool CASCADE, int MODE = MODE_PLAIN>
+
+// Where a layer's keys and values lie. planes 1: the values are the keys, pages hold them once ([pages][hkv][page][D]).
+// POOL kernels: beside the window a query sees the mean key and value of every block of `pool` tokens wholly before it. A mean
+// lies with the page of its block's last token, [pages][2][hkv][per_page][D], `per_page` = ceil(page / pool); prefill reads
+// them gathered into 16-row pages, [pages][2][hkv][16][D], `first`[r] the first of request r.
+struct KeyLayout {
+    int planes = 2, pool = 0, per_page = 0;
+    const bf16* means = nullptr;
+    const int* first = nullptr;
+};
+// Means that a query at `pos` sees beside the window_left tokens before it.
+__device__ __forceinline__ int means_seen(int pos, int window_left, int pool) { return max(0, pos - window_left) / pool; }
+// Row of block b among the means of its page, and that page's place in the request's table.
+__device__ __forceinline__ int mean_row(int b, int pool, int page_size, int& page_at) {
+    page_at = ((b + 1) * pool - 1) / page_size;
+    return b - page_at * page_size / pool;
+}
+
+// POOL: an item of a request takes its share of the 16-key tiles (means, then the window's tokens) whatever range the plan
+// gave it, so that any plan spreads the work evenly.
+template <int D, int G, bool CASCADE, int MODE = MODE_PLAIN, bool POOL = false>
 __global__ void __launch_bounds__(DEC_WARPS * 32)
 paged_decode_attn_kernel(const bf16* __restrict__ q, const bf16* __restrict__ kv_layer,
                          const int* __restrict__ page_indices,
@@ -230,7 +250,7 @@ paged_decode_attn_kernel(const bf16* __restrict__ q, const bf16* __restrict__ kv
                          const float* __restrict__ sinks_log2, int max_items, int num_reqs,
                          int* __restrict__ status, const int* __restrict__ item_slot,
                          const int* __restrict__ item_tile, const int* __restrict__ tile_members,
-                         float cap_log2, const float* __restrict__ bias, int bias_pitch, int keep_first) {
+                         float cap_log2, const float* __restrict__ bias, int bias_pitch, int keep_first, const KeyLayout kl) {
     static_assert(G <= 16, "at most 16 query heads per KV head");
     constexpr int ROWS = CASCADE ? (16 / G) * G : G;      // rows of the Q tile in use
     extern __shared__ __align__(1024) uint8_t smem[];
@@ -257,7 +277,7 @@ paged_decode_attn_kernel(const bf16* __restrict__ q, const bf16* __restrict__ kv
             if (threadIdx.x == 0 && status) atomicCAS(status, 0, PIE_ERR_BOUNDS);
             continue;
         }
-        const int kv_start = item_start[it], kv_end = item_end[it];
+        const int kv_start = POOL ? 0 : item_start[it], kv_end = item_end[POOL ? req_item_indptr[req + 1] - 1 : it];
         const int tile = CASCADE ? item_tile[it] : -1;
         const int* members = (CASCADE && tile >= 0) ? tile_members + (size_t)tile * 16 : nullptr;
         // sliding window: the query sits at position kv_len - 1 (kv_len = end of the request's last
@@ -291,17 +311,53 @@ paged_decode_attn_kernel(const bf16* __restrict__ q, const bf16* __restrict__ kv
         // blocks [hidden, hidden + gap) of the item lie between the kept first keys and the window
         const int nb_item = (kv_end - kv_start + 15) >> 4;
         const int hidden = min(nb_item, max(0, (keep_first - kv_start + 15) >> 4));
-        const int gap = max(0, min(nb_item, (kv_lo - kv_start) >> 4) - hidden), nb_total = nb_item - gap;
-        auto block_start = [&](int b) { return kv_start + (b < hidden ? b : b + gap) * 16; };
+        const int gap = max(0, min(nb_item, (kv_lo - kv_start) >> 4) - hidden);
+        // POOL: this item's tiles are first_tile .. first_tile + nb_total - 1, tile t < mean_tiles being sixteen means
+        const int n_means = POOL ? means_seen(kv_end - 1, window_left, kl.pool) : 0, mean_tiles = (n_means + 15) >> 4;
+        int first_tile = 0, nb_total = nb_item - gap;
+        if (POOL) {
+            const long all = mean_tiles + nb_total;
+            const int i0 = req_item_indptr[req], parts = req_item_indptr[req + 1] - i0;
+            first_tile = (int)(all * (it - i0) / parts);
+            nb_total = (int)(all * (it - i0 + 1) / parts) - first_tile;
+        }
+        auto block_start = [&](int b) {
+            if (POOL) return (first_tile + b - mean_tiles + gap) * 16;
+            return kv_start + (b < hidden ? b : b + gap) * 16;
+        };
         const int my_count = nb_total > warp ? (nb_total - warp + DEC_WARPS - 1) / DEC_WARPS : 0;
         const int* pages = page_indices + kv_page_indptr[req];
 
         auto issue = [&](int j) {
+            if (POOL && first_tile + warp + DEC_WARPS * j < mean_tiles) {
+                // lane r knows where mean r of the tile lies
+                const int b = (first_tile + warp + DEC_WARPS * j) * 16 + (lane & 15);
+                long at = -1;
+                if (b < n_means) {
+                    int pg;
+                    const int row = mean_row(b, kl.pool, page_size, pg);
+                    at = ((((long)pages[pg] * 2) * hkv + h) * kl.per_page + row) * D;
+                }
+                const uint32_t kdst = warp_smem + (j % DEC_STAGES) * 2 * TILE_BYTES;
+#pragma unroll
+                for (int i = 0; i < (16 * CH) / 32; ++i) {
+                    const int c = lane + 32 * i, row = c / CH, col = c - row * CH;
+                    const long src = __shfl_sync(0xffffffffu, at, row);
+                    if (src >= 0) {
+                        cp_async16(kdst + swz<D>(row, col), kl.means + src + col * 8);
+                        cp_async16(kdst + TILE_BYTES + swz<D>(row, col), kl.means + src + (long)hkv * kl.per_page * D + col * 8);
+                    } else {           // multiplied by p == 0: must be finite
+                        uint8_t* z = smem + (kdst - q_smem) + swz<D>(row, col);
+                        *reinterpret_cast<uint4*>(z) = *reinterpret_cast<uint4*>(z + TILE_BYTES) = make_uint4(0, 0, 0, 0);
+                    }
+                }
+                return;
+            }
             const int tok0 = block_start(warp + DEC_WARPS * j);
             const int page = pages[tok0 / page_size];
             const int off = tok0 % page_size;
-            const bf16* ksrc = kv_layer + ((((size_t)page * 2) * hkv + h) * page_size + off) * D;
-            const bf16* vsrc = kv_layer + ((((size_t)page * 2 + 1) * hkv + h) * page_size + off) * D;
+            const bf16* ksrc = kv_layer + ((((size_t)page * kl.planes) * hkv + h) * page_size + off) * D;
+            const bf16* vsrc = kl.planes == 2 ? ksrc + (size_t)hkv * page_size * D : nullptr;
             const uint32_t kdst = warp_smem + (j % DEC_STAGES) * 2 * TILE_BYTES;
             const uint32_t vdst = kdst + TILE_BYTES;
 #pragma unroll
@@ -309,7 +365,7 @@ paged_decode_attn_kernel(const bf16* __restrict__ q, const bf16* __restrict__ kv
                 const int c = lane + 32 * i;
                 const int row = c / CH, col = c - row * CH;
                 cp_async16(kdst + swz<D>(row, col), ksrc + (size_t)c * 8);
-                cp_async16(vdst + swz<D>(row, col), vsrc + (size_t)c * 8);
+                if (vsrc) cp_async16(vdst + swz<D>(row, col), vsrc + (size_t)c * 8);
             }
         };
 #pragma unroll
@@ -322,10 +378,11 @@ paged_decode_attn_kernel(const bf16* __restrict__ q, const bf16* __restrict__ kv
             cp_async_commit();
             cp_async_wait<DEC_STAGES - 1>();
             __syncwarp();
-            const int tok0 = block_start(warp + DEC_WARPS * i);
-            const int nvalid = kv_end - tok0;
+            const bool means = POOL && first_tile + warp + DEC_WARPS * i < mean_tiles;
+            const int tok0 = means ? (first_tile + warp + DEC_WARPS * i) * 16 : block_start(warp + DEC_WARPS * i);
+            const int nvalid = (means ? n_means : kv_end) - tok0;
             uint32_t allow = nvalid >= 16 ? 0xffffu : ((1u << nvalid) - 1u);
-            if (kv_lo > tok0) {
+            if (!means && kv_lo > tok0) {
                 uint32_t see = kv_lo - tok0 >= 16 ? 0u : ~((1u << (kv_lo - tok0)) - 1u);
                 if (keep_first > tok0) see |= keep_first - tok0 >= 16 ? 0xffffu : (1u << (keep_first - tok0)) - 1u;
                 allow &= see;
@@ -338,7 +395,7 @@ paged_decode_attn_kernel(const bf16* __restrict__ q, const bf16* __restrict__ kv
                 db = DistanceBias{tab + (g < G ? g : 0) * bias_pitch, tab + (g + 8 < G ? g + 8 : 0) * bias_pitch, n, n,
                                   bias_pitch - 2 * BIAS_GUARD - 1};
             }
-            attn_block16<D, MODE>(qf, kt, kt + TILE_BYTES, scale_log2, allow, allow, st, cap_log2, db);
+            attn_block16<D, MODE>(qf, kt, kl.planes == 1 ? kt : kt + TILE_BYTES, scale_log2, allow, allow, st, cap_log2, db);
             __syncwarp();
         }
         cp_async_wait<0>();
@@ -459,7 +516,7 @@ constexpr int prefill_smem_bytes() {
     return PF_ROWS * D * 2 + 2 * 2 * PF_KV * D * 2;
 }
 
-template <int D, int G, int MODE = MODE_PLAIN>
+template <int D, int G, int MODE = MODE_PLAIN, bool POOL = false>
 __global__ void __launch_bounds__(PF_WARPS * 32)
 paged_prefill_attn_kernel(const bf16* __restrict__ q, const bf16* __restrict__ kv_layer,
                           const int* __restrict__ page_indices,
@@ -470,7 +527,7 @@ paged_prefill_attn_kernel(const bf16* __restrict__ q, const bf16* __restrict__ k
                           const long* __restrict__ mask_word_indptr, bf16* __restrict__ out,
                           float* __restrict__ lse_out, const float* __restrict__ sinks_log2, int hq, int hkv, int page_size,
                           float scale_log2, int window_left, float cap_log2, const float* __restrict__ bias,
-                          int bias_pitch, int keep_first) {
+                          int bias_pitch, int keep_first, const KeyLayout kl) {
     extern __shared__ __align__(1024) uint8_t smem[];
     constexpr int CH = D / 8;
     constexpr int TQ = PF_ROWS / G;  // query tokens per tile
@@ -523,11 +580,14 @@ paged_prefill_attn_kernel(const bf16* __restrict__ q, const bf16* __restrict__ k
     const int nkb_all = (kv_hi + PF_KV - 1) / PF_KV;
     const int hidden = min(nkb_all, (keep_first + PF_KV - 1) / PF_KV);
     const int gap = window_left >= 0 ? max(0, min(nkb_all, max(0, kv_len - qo_len + qstart - window_left) / PF_KV) - hidden) : 0;
-    const int nkb = nkb_all - gap;
-    auto key_block = [&](int i) { return i < hidden ? i : i + gap; };
+    // POOL: blocks of means come first, as many as the tile's last query sees
+    const int n_means = POOL ? means_seen(kv_len - qo_len + last_q, window_left, kl.pool) : 0, mean_blocks = (n_means + PF_KV - 1) / PF_KV;
+    const int nkb = nkb_all - gap + mean_blocks;
+    auto key_block = [&](int i) { return POOL ? i - mean_blocks + gap : (i < hidden ? i : i + gap); };
 
     auto load_stage = [&](int i_kb) {
-        const int kb = key_block(i_kb);
+        const bool means = POOL && i_kb < mean_blocks;
+        const int kb = means ? i_kb : key_block(i_kb);
         const uint32_t kdst = kv_smem + (i_kb & 1) * 2 * KV_TILE;
         const uint32_t vdst = kdst + KV_TILE;
 #pragma unroll
@@ -535,13 +595,16 @@ paged_prefill_attn_kernel(const bf16* __restrict__ q, const bf16* __restrict__ k
             const int c = threadIdx.x + PF_WARPS * 32 * i;
             const int row = c / CH, col = c - row * CH;
             const int tok = kb * PF_KV + row;
-            if (tok < kv_hi) {
+            if (means && tok < n_means) {
+                const bf16* ksrc = kl.means + ((((size_t)kl.first[req] + tok / 16) * 2 * hkv + h) * 16 + tok % 16) * D + col * 8;
+                cp_async16(kdst + swz<D>(row, col), ksrc);
+                cp_async16(vdst + swz<D>(row, col), ksrc + (size_t)hkv * 16 * D);
+            } else if (!means && tok < kv_hi) {
                 const int page = pages[tok / page_size];
                 const int off = tok % page_size;
                 const bf16* ksrc =
-                    kv_layer + ((((size_t)page * 2) * hkv + h) * page_size + off) * D + col * 8;
-                const bf16* vsrc =
-                    kv_layer + ((((size_t)page * 2 + 1) * hkv + h) * page_size + off) * D + col * 8;
+                    kv_layer + ((((size_t)page * kl.planes) * hkv + h) * page_size + off) * D + col * 8;
+                const bf16* vsrc = ksrc + (size_t)(kl.planes - 1) * hkv * page_size * D;
                 cp_async16(kdst + swz<D>(row, col), ksrc);
                 cp_async16(vdst + swz<D>(row, col), vsrc);
             } else {
@@ -563,18 +626,19 @@ paged_prefill_attn_kernel(const bf16* __restrict__ q, const bf16* __restrict__ k
         cp_async_commit();
         cp_async_wait<1>();
         __syncthreads();
-        const int kb = key_block(i_kb);
+        const bool means = POOL && i_kb < mean_blocks;
+        const int kb = means ? i_kb : key_block(i_kb);
         const uint32_t kt = kv_smem + (i_kb & 1) * 2 * KV_TILE;
 #pragma unroll
         for (int sb = 0; sb < PF_KV / 16; ++sb) {
             const int tb = kb * PF_KV + sb * 16;
-            if (tb >= warp_hi || tb >= kv_hi) break;
+            if (means ? tb >= n_means : (tb >= warp_hi || tb >= kv_hi)) break;
             uint32_t allow[2];
 #pragma unroll
             for (int hh = 0; hh < 2; ++hh) {
-                const int n = lim[hh] - tb;
+                const int n = (means ? lo[hh] / kl.pool : lim[hh]) - tb;
                 uint32_t a = n >= 16 ? 0xffffu : (n <= 0 ? 0u : ((1u << n) - 1u));
-                const int nl = lo[hh] - tb;
+                const int nl = means ? 0 : lo[hh] - tb;
                 if (nl > 0) {
                     uint32_t see = nl >= 16 ? 0u : ~((1u << nl) - 1u);
                     if (keep_first > tb) see |= keep_first - tb >= 16 ? 0xffffu : (1u << (keep_first - tb)) - 1u;

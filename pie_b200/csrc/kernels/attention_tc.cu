@@ -77,7 +77,7 @@ PIE_API int pie_paged_prefill_attn_tc_kept(const void* q, const void* kv_layer, 
         cudaError_t e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)Cfg::SMEM);      \
         if (e != cudaSuccess) return (int)e;                                                                          \
         kern<<<grid, Cfg::THREADS, Cfg::SMEM, st>>>(                                                                  \
-            tq, tkv, page_indices, kv_page_indptr, qo_indptr, kv_lens, tile_req, tile_qstart, mask_bits,              \
+            tq, tkv, tkv, TcMeans(), 2, page_indices, kv_page_indptr, qo_indptr, kv_lens, tile_req, tile_qstart, mask_bits,              \
             mask_word_indptr, (bf16*)out, lse_out, sinks_log2, hq, hkv, total_pages - 1, scale_log2, window_left,     \
             status, cap_pre, cap_post, hq * D_, D_, nullptr, 0, 0, keep_first);                                                                 \
         return (int)cudaGetLastError();                                                                               \
@@ -149,7 +149,7 @@ PIE_API int pie_projected_prefill_attn_tc(const void* q, const void* kv, const i
         using Cfg = AtCfg<2, D__>;                                                                                    \
         cudaError_t e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)Cfg::SMEM);      \
         if (e != cudaSuccess) return (int)e;                                                                          \
-        kern<<<grid, Cfg::THREADS, Cfg::SMEM, st>>>(tq, tkv, page_indices, kv_page_indptr, qo_indptr, kv_lens, tile_req,  \
+        kern<<<grid, Cfg::THREADS, Cfg::SMEM, st>>>(tq, tkv, tkv, TcMeans(), 2, page_indices, kv_page_indptr, qo_indptr, kv_lens, tile_req,  \
                                                     tile_qstart, mask_bits, mask_word_indptr, (bf16*)out, nullptr,    \
                                                     nullptr, heads, heads, total_tokens / 16, scale_log2, window_left, status,  \
                                                     0.f, 0.f, out_ld, vdim, nullptr, 0, 0, 0);                                         \

@@ -85,25 +85,6 @@ __device__ __forceinline__ float fast_exp2(float x) {
     return y;
 }
 
-// Two 32-bit numbers in one register pair: the packed arithmetic of sm_100.
-typedef unsigned long long F2;
-__device__ __forceinline__ F2 f2(float lo, float hi) {
-    F2 d;
-    asm("mov.b64 %0, {%1, %2};" : "=l"(d) : "f"(lo), "f"(hi));
-    return d;
-}
-__device__ __forceinline__ F2 f2(float x) { return f2(x, x); }
-__device__ __forceinline__ void unpack2(F2 v, float& lo, float& hi) { asm("mov.b64 {%0, %1}, %2;" : "=f"(lo), "=f"(hi) : "l"(v)); }
-__device__ __forceinline__ F2 mul2(F2 a, F2 b) {
-    F2 d;
-    asm("mul.rn.f32x2 %0, %1, %2;" : "=l"(d) : "l"(a), "l"(b));
-    return d;
-}
-__device__ __forceinline__ F2 fma2(F2 a, F2 b, F2 c) {
-    F2 d;
-    asm("fma.rn.f32x2 %0, %1, %2, %3;" : "=l"(d) : "l"(a), "l"(b), "l"(c));
-    return d;
-}
 __device__ __forceinline__ float fast_tanh(float x) {
     float y;
     asm("tanh.approx.f32 %0, %1;" : "=f"(y) : "f"(x));
@@ -118,13 +99,22 @@ __device__ __forceinline__ float fast_tanh(float x) {
 // TOK: keys and values lie token by token, [tokens][hkv][2][D] (tma_kv then has the dimensions D, hkv * 2, tokens), and a
 // "page" is 16 consecutive tokens: the layout a projection of latents writes. Its value heads may be narrower than D.
 // out_ld / out_cols: elements per token of `out` and per head (columns past out_cols are not stored; a multiple of 8).
+// planes 1: the values are the keys, pages hold [hkv][16][D] once.
+// POOL: beside the window a query sees the mean key and value of every block of ml.pool tokens that lies wholly before it. The
+// means come in 16-row pages of their own ([pages][2][hkv][16][D], the last one zeros), ml.first[r] the first of request r; key
+// blocks count them first, then the window's tokens. No custom masks.
 // BIAS: soft-capped scores plus a learned bias per distance, in units of log2 (scale_log2 is 1, cap_post the cap times
 // log2(e)). bias [hkv * G][bias_pitch]: AT_BIAS_GUARD entries like the first distance, the bias of the distances 0 .. window_left, as many
 // unused ones, so that a block that a window or the diagonal cuts reads inside the row. With bias_smem the CTA's G rows are
 // copied to shared memory first.
-template <int G, int NT, int D, bool CAP = false, bool TOK = false, bool BIAS = false>
+struct TcMeans {
+    const int* first = nullptr;     // [requests]
+    int pool = 0, pad_page = 0;
+};
+template <int G, int NT, int D, bool CAP = false, bool TOK = false, bool BIAS = false, bool POOL = false>
 __global__ void __launch_bounds__(AtCfg<NT, D>::THREADS, 1)
 paged_prefill_attn_tc_kernel(const __grid_constant__ CUtensorMap tma_q, const __grid_constant__ CUtensorMap tma_kv,
+                             const __grid_constant__ CUtensorMap tma_means, const TcMeans ml, int planes,
                              const int* __restrict__ page_indices, const int* __restrict__ kv_page_indptr,
                              const int* __restrict__ qo_indptr, const int* __restrict__ kv_lens,
                              const int* __restrict__ tile_req, const int* __restrict__ tile_qstart,
@@ -189,10 +179,13 @@ paged_prefill_attn_tc_kernel(const __grid_constant__ CUtensorMap tma_q, const __
     // `keep_first` keys: blocks are counted without the hidden ones
     const int kept = (keep_first + AT_BK - 1) / AT_BK;
     const int gap = window_left >= 0 ? max(0, max(0, kv_len - qo_len + qstart - window_left) / AT_BK - kept) : 0;
-    auto key_block = [&](int j) { return j < kept ? j : j + gap; };
+    // blocks of means, as many as the CTA's last query sees
+    const int means_hi = POOL ? max(0, kv_len - qo_len + min(qstart + NT * TQ, qo_len) - 1 - window_left) / ml.pool : 0;
+    const int nmb = (means_hi + AT_BK - 1) / AT_BK, means_page0 = POOL ? ml.first[req] : 0;
+    auto key_block = [&](int j) { return POOL ? j - nmb + gap : (j < kept ? j : j + gap); };
 #pragma unroll
-    for (int t = 0; t < NT; ++t) nkb_t[t] = max(0, nkb_t[t] - gap);
-    nkb = max(0, nkb - gap);
+    for (int t = 0; t < NT; ++t) nkb_t[t] = POOL && nkb_t[t] == 0 ? 0 : max(0, nkb_t[t] - gap + nmb);
+    nkb = POOL && nkb == 0 ? 0 : max(0, nkb - gap + nmb);
 
     if (threadIdx.x == 0) {
         mbar_init(q_full(), 1);
@@ -247,35 +240,40 @@ paged_prefill_attn_tc_kernel(const __grid_constant__ CUtensorMap tma_q, const __
                 int pg_id[4];
 #pragma unroll
                 for (int pg = 0; pg < 4; ++pg) {
+                    if (POOL && j < nmb) {
+                        pg_id[pg] = (j * 4 + pg) * 16 < means_hi ? means_page0 + j * 4 + pg : ml.pad_page;
+                        continue;
+                    }
                     const int pi = key_block(j) * 4 + pg;
                     pg_id[pg] = pi < npages ? pages[pi] : pad_page;
                 }
+                const CUtensorMap* map = POOL && j < nmb ? &tma_means : &tma_kv;
                 if (!mbar_wait(k_empty(s), par, status, PIE_ERR_WAIT_TMA)) { ok = false; break; }
                 mbar_arrive_expect_tx(k_full(s), AT_KV_TILE);
 #pragma unroll
                 for (int pg = 0; pg < 4; ++pg) {
-                    const int krow = ((pg_id[pg] * 2) * hkv + h) * 16;
+                    const int krow = ((pg_id[pg] * planes) * hkv + h) * 16;
 #pragma unroll
                     for (int half = 0; half < HALVES; ++half) {
                         const uint32_t dst = k_s + s * AT_KV_TILE + half * AT_KV_HALF + pg * 2048;
                         if constexpr (TOK)
                             tma_load_3d(dst, &tma_kv, k_full(s), half * 64, 2 * h, pg_id[pg] * 16);
                         else
-                            tma_load_2d(dst, &tma_kv, k_full(s), half * 64, krow);
+                            tma_load_2d(dst, map, k_full(s), half * 64, krow);
                     }
                 }
                 if (!mbar_wait(v_empty(s), par, status, PIE_ERR_WAIT_TMA)) { ok = false; break; }
                 mbar_arrive_expect_tx(v_full(s), AT_KV_TILE);
 #pragma unroll
                 for (int pg = 0; pg < 4; ++pg) {
-                    const int vrow = ((pg_id[pg] * 2 + 1) * hkv + h) * 16;
+                    const int vrow = ((pg_id[pg] * planes + planes - 1) * hkv + h) * 16;
 #pragma unroll
                     for (int half = 0; half < HALVES; ++half) {
                         const uint32_t dst = v_s + s * AT_KV_TILE + half * AT_KV_HALF + pg * 2048;
                         if constexpr (TOK)
                             tma_load_3d(dst, &tma_kv, v_full(s), half * 64, 2 * h + 1, pg_id[pg] * 16);
                         else
-                            tma_load_2d(dst, &tma_kv, v_full(s), half * 64, vrow);
+                            tma_load_2d(dst, map, v_full(s), half * 64, vrow);
                     }
                 }
             }
@@ -347,6 +345,7 @@ paged_prefill_attn_tc_kernel(const __grid_constant__ CUtensorMap tma_q, const __
         const bool valid = qtok < qo_len;
         const int lim = valid ? (custom ? kv_len : kv_len - qo_len + qtok + 1) : 0;
         const int lo = (window_left >= 0 && valid) ? max(0, kv_len - qo_len + qtok - window_left) : 0;
+        const int means_row = POOL ? lo / ml.pool : 0;
         const int mask_words = (kv_len + 31) >> 5;
         const uint32_t* row_mask = (custom && valid) ? mask_bits + mask_word_indptr[req] + (size_t)qtok * mask_words : nullptr;
         const uint32_t tm_t = tmem_base + t * 256 + ((uint32_t)(q4 * 32) << 16);
@@ -370,7 +369,8 @@ paged_prefill_attn_tc_kernel(const __grid_constant__ CUtensorMap tma_q, const __
                 for (int i = 0; i < 32; ++i)
                     sv[c * 32 + i] = CAP ? cap_post * fast_tanh(__uint_as_float(v[i]) * cap_pre) : __uint_as_float(v[i]);
             }
-            const int kb0 = key_block(j) * AT_BK;
+            const bool means = POOL && j < nmb;
+            const int kb0 = (means ? j : key_block(j)) * AT_BK;
             if (BIAS) {
                 // distance of key i of the block: n - i (keys after the query, which only a custom mask shows, read the guard)
                 const int n = kb0 < lim && kb0 + AT_BK > lo ? max(kv_len - qo_len + qtok - kb0, -1) : 0;
@@ -400,10 +400,11 @@ paged_prefill_attn_tc_kernel(const __grid_constant__ CUtensorMap tma_q, const __
                 if (bias_smem) add_bias(reinterpret_cast<const float*>(base_ptr + Cfg::TABLE) + at);
                 else add_bias(bias + (size_t)h * G * bias_pitch + at);
             }
-            const bool inner = !custom && kb0 + AT_BK <= lim && kb0 >= lo;
+            const int hi = means ? means_row : lim, low = means ? 0 : lo;
+            const bool inner = !custom && kb0 + AT_BK <= hi && kb0 >= low;
             if (!__all_sync(0xffffffffu, inner)) {
                 // 64-bit allow mask of this row for the block
-                const int n = lim - kb0, nl = lo - kb0;
+                const int n = hi - kb0, nl = low - kb0;
                 unsigned long long allow = n >= 64 ? ~0ull : (n <= 0 ? 0ull : ((1ull << n) - 1ull));
                 if (nl > 0) {
                     unsigned long long see = nl >= 64 ? 0ull : ~((1ull << nl) - 1ull);

@@ -128,6 +128,26 @@ __device__ __forceinline__ bf16x8 pack8(const float* f) {
     return p;
 }
 
+// Two 32-bit numbers in one register pair: the packed arithmetic of sm_100.
+typedef unsigned long long F2;
+__device__ __forceinline__ F2 f2(float lo, float hi) {
+    F2 d;
+    asm("mov.b64 %0, {%1, %2};" : "=l"(d) : "f"(lo), "f"(hi));
+    return d;
+}
+__device__ __forceinline__ F2 f2(float x) { return f2(x, x); }
+__device__ __forceinline__ void unpack2(F2 v, float& lo, float& hi) { asm("mov.b64 {%0, %1}, %2;" : "=f"(lo), "=f"(hi) : "l"(v)); }
+__device__ __forceinline__ F2 mul2(F2 a, F2 b) {
+    F2 d;
+    asm("mul.rn.f32x2 %0, %1, %2;" : "=l"(d) : "l"(a), "l"(b));
+    return d;
+}
+__device__ __forceinline__ F2 fma2(F2 a, F2 b, F2 c) {
+    F2 d;
+    asm("fma.rn.f32x2 %0, %1, %2, %3;" : "=l"(d) : "l"(a), "l"(b), "l"(c));
+    return d;
+}
+
 // 64-bit mix used for counter-based random numbers (SplitMix64 finaliser).
 __device__ __host__ __forceinline__ uint64_t splitmix64(uint64_t x) {
     x += 0x9E3779B97F4A7C15ull;

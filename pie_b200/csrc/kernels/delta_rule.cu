@@ -1,0 +1,351 @@
+// Delta rule with a decay and a removal rate per key channel: per head, with the unit key u = k / sqrt(sum k^2 + 1e-6),
+//   S_t = diag(w_t) S_(t-1) - (a_t * u_t) (u_t^T S_(t-1)) + k_t v_t^T,   o_t = S_t^T r_t,
+// S in 32-bit [dim][dim], one state per (slot, head), carried from fire to fire. Everything but the projections (r, k, v and the
+// product behind a) is 32-bit. Both sums of a token run over the old state:
+//   y = S^T u,  z = S^T (r * w),   o = z - (r . (a * u)) y + (r . k) v,
+// so that columns of the state never meet, and a column's rows once per token.
+//
+//   step       one token per request: a block holds 128 columns (VEC per lane) of a head, an eighth of the rows per warp
+//   portions   any lengths: a thread holds one column's rows, LPC lanes share a column; the tokens' vectors are prepared CT at
+//              a time in shared memory while the tokens before them run
+#include "typed.cuh"
+
+namespace pie {
+
+struct DeltaArgs {
+    const void *r, *k, *v, *a;      // row t, head h at t * ld + h * dim, type T; a: the removal rate's product
+    const float* a_bias;            // [heads * dim]
+    const float* log_decay;         // [n, heads * dim] base 2
+    float* out;                     // [n, heads * dim]
+    float* state;                   // this layer's part of slot 0: [heads][dim][dim]
+    const int *qo_indptr, *slots, *reset;
+    long slot_stride;
+    int n, ld, reqs, heads, dim;
+};
+
+__device__ __forceinline__ float delta_rate(float z) { return 1.f / (1.f + expf(-z)); }
+
+template <typename T, int RPT, int VEC>
+__global__ void __launch_bounds__(256) delta_step_kernel(const DeltaArgs a) {
+    constexpr int ROWS = RPT * 8, COLS = 32 * VEC;
+    __shared__ float su[ROWS], sau[ROWS], sw[ROWS], srw[ROWS], sk[ROWS], red[32];
+    __shared__ __align__(16) float ry[8][COLS], rz[8][COLS];
+    pdl_trigger();
+    pdl_wait();
+    const int q = blockIdx.x, h = blockIdx.y, lane = threadIdx.x & 31, rg = threadIdx.x >> 5;
+    const int t = a.qo_indptr[q], slot = a.slots[q];
+    if (a.qo_indptr[q + 1] <= t || slot < 0) return;       // a padding request of a decode graph: no state, no output
+    const int c0 = blockIdx.z * COLS + lane * VEC;
+    const bool col = c0 < a.dim;                           // VEC > 1 only where dim is a multiple of it
+    float* sp = a.state + (size_t)slot * a.slot_stride + (size_t)h * a.dim * a.dim;
+    const bool fresh = a.reset[q] != 0;
+    float S[RPT][VEC];
+#pragma unroll
+    for (int i = 0; i < RPT; ++i) {
+        const int d = rg + 8 * i;
+#pragma unroll
+        for (int j = 0; j < VEC; ++j) S[i][j] = 0.f;
+        if (col && !fresh && d < a.dim) load_vec<VEC>(sp + (size_t)d * a.dim + c0, S[i]);
+    }
+    const size_t row = (size_t)t * a.ld + h * a.dim;
+    float v[VEC];
+#pragma unroll
+    for (int j = 0; j < VEC; ++j) v[j] = 0.f;
+    if (col) load_vec<VEC>(static_cast<const T*>(a.v) + row + c0, v);
+    constexpr int PER = (ROWS + 255) / 256;
+    float k[PER], ss = 0.f;
+#pragma unroll
+    for (int i = 0; i < PER; ++i) {
+        const int d = threadIdx.x + i * 256;
+        k[i] = d < a.dim ? to_f(static_cast<const T*>(a.k)[row + d]) : 0.f;
+        ss += k[i] * k[i];
+    }
+    const float inv = 1.f / sqrtf(block_sum(ss, red) + 1e-6f);
+    float rau = 0.f, rk = 0.f;
+#pragma unroll
+    for (int i = 0; i < PER; ++i) {
+        const int d = threadIdx.x + i * 256;
+        if (d >= ROWS) break;
+        float r = 0.f, w = 1.f, rate = 0.f;
+        if (d < a.dim) {
+            r = to_f(static_cast<const T*>(a.r)[row + d]);
+            w = exp2f(a.log_decay[((size_t)t * a.heads + h) * a.dim + d]);
+            rate = delta_rate(to_f(static_cast<const T*>(a.a)[row + d]) + a.a_bias[h * a.dim + d]);
+        }
+        const float u = k[i] * inv, au = rate * u;
+        su[d] = u; sau[d] = au; sw[d] = w; srw[d] = r * w; sk[d] = k[i];
+        rau += r * au;
+        rk += r * k[i];
+    }
+    rau = block_sum(rau, red);
+    rk = block_sum(rk, red);
+    float y[VEC], z[VEC];
+#pragma unroll
+    for (int j = 0; j < VEC; ++j) y[j] = z[j] = 0.f;
+#pragma unroll
+    for (int i = 0; i < RPT; ++i) {
+        const float u = su[rg + 8 * i], rw = srw[rg + 8 * i];
+#pragma unroll
+        for (int j = 0; j < VEC; ++j) {
+            y[j] += u * S[i][j];
+            z[j] += rw * S[i][j];
+        }
+    }
+#pragma unroll
+    for (int j = 0; j < VEC; ++j) {
+        ry[rg][lane * VEC + j] = y[j];
+        rz[rg][lane * VEC + j] = z[j];
+    }
+    __syncthreads();
+#pragma unroll
+    for (int j = 0; j < VEC; ++j) {
+        y[j] = z[j] = 0.f;
+#pragma unroll
+        for (int g = 0; g < 8; ++g) {
+            y[j] += ry[g][lane * VEC + j];
+            if (rg == 0) z[j] += rz[g][lane * VEC + j];
+        }
+    }
+    if (!col) return;
+    if (rg == 0) {
+        float* dst = a.out + ((size_t)t * a.heads + h) * a.dim + c0;
+#pragma unroll
+        for (int j = 0; j < VEC; ++j) dst[j] = z[j] - rau * y[j] + rk * v[j];
+    }
+#pragma unroll
+    for (int i = 0; i < RPT; ++i) {
+        const int d = rg + 8 * i;
+        if (d >= a.dim) continue;
+        const float w = sw[d], au = sau[d], kk = sk[d];
+#pragma unroll
+        for (int j = 0; j < VEC; ++j) S[i][j] = w * S[i][j] - au * y[j] + kk * v[j];
+        store_vec<VEC>(sp + (size_t)d * a.dim + c0, S[i]);
+    }
+}
+
+template <int RPL, int LPC, int CT>
+struct DeltaSmem {
+    static constexpr int DP = RPL * LPC, COLS = 256 / LPC;
+    static constexpr int VECS = 5 * DP;                    // u, r * w, w, a * u, k of a token
+    float vec[2][CT][VECS];
+    float v[2][CT][COLS], o[2][CT][COLS];
+    float2 dots[2][CT];                                    // r . (a * u), r . k
+};
+
+// Lane g of a column holds the rows 4 (g + LPC i) + e: a warp's 16-byte reads of a vector fall on consecutive addresses.
+template <typename T, int RPL, int LPC, int CT>
+__global__ void __launch_bounds__(256) delta_portion_kernel(const DeltaArgs a) {
+    using Smem = DeltaSmem<RPL, LPC, CT>;
+    constexpr int DP = Smem::DP, COLS = Smem::COLS, TPW = CT / 8, EPL = DP / 32, VPT = (CT * COLS + 255) / 256;
+    extern __shared__ __align__(16) uint8_t raw[];
+    Smem& sm = *reinterpret_cast<Smem*>(raw);
+    const int q = blockIdx.x, h = blockIdx.y, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+    const int first = a.qo_indptr[q], len = a.qo_indptr[q + 1] - first, slot = a.slots[q];
+    if (len <= 0 || slot < 0) return;
+    const int g = lane % LPC, cl = warp * (32 / LPC) + lane / LPC, c = blockIdx.z * COLS + cl;
+    float* sp = a.state + (size_t)slot * a.slot_stride + (size_t)h * a.dim * a.dim;
+    const bool fresh = a.reset[q] != 0;
+    F2 S[RPL / 2];
+#pragma unroll
+    for (int i = 0; i < RPL / 4; ++i) {
+        float f[4];
+#pragma unroll
+        for (int e = 0; e < 4; ++e) {
+            const int d = 4 * (g + LPC * i) + e;
+            f[e] = !fresh && c < a.dim && d < a.dim ? sp[(size_t)d * a.dim + c] : 0.f;
+        }
+        S[2 * i] = f2(f[0], f[1]);
+        S[2 * i + 1] = f2(f[2], f[3]);
+    }
+    const T* R = static_cast<const T*>(a.r) + (size_t)first * a.ld + h * a.dim;
+    const T* K = static_cast<const T*>(a.k) + (size_t)first * a.ld + h * a.dim;
+    const T* V = static_cast<const T*>(a.v) + (size_t)first * a.ld + h * a.dim;
+    const T* A = static_cast<const T*>(a.a) + (size_t)first * a.ld + h * a.dim;
+    const float* W = a.log_decay + ((size_t)first * a.heads + h) * a.dim;
+    float* O = a.out + ((size_t)first * a.heads + h) * a.dim;
+    const size_t step = (size_t)a.heads * a.dim;
+    float bias[EPL];
+#pragma unroll
+    for (int i = 0; i < EPL; ++i) bias[i] = lane + 32 * i < a.dim ? a.a_bias[h * a.dim + lane + 32 * i] : 0.f;
+
+    T pr[TPW][EPL], pk[TPW][EPL], pa[TPW][EPL], pv[VPT];
+    float pw[TPW][EPL];
+    auto load = [&](int t0) {
+#pragma unroll
+        for (int s = 0; s < TPW; ++s) {
+            const int t = t0 + warp * TPW + s;
+#pragma unroll
+            for (int i = 0; i < EPL; ++i) {
+                const int d = lane + 32 * i;
+                const bool ok = t < len && d < a.dim;
+                const size_t at = (size_t)t * a.ld + d;
+                pr[s][i] = ok ? R[at] : from_f<T>(0.f);
+                pk[s][i] = ok ? K[at] : from_f<T>(0.f);
+                pa[s][i] = ok ? A[at] : from_f<T>(0.f);
+                pw[s][i] = ok ? W[(size_t)t * step + d] : 0.f;
+            }
+        }
+#pragma unroll
+        for (int i = 0; i < VPT; ++i) {
+            const int x = threadIdx.x + i * 256, t = t0 + x / COLS, cc = blockIdx.z * COLS + x % COLS;
+            pv[i] = x < CT * COLS && t < len && cc < a.dim ? V[(size_t)t * a.ld + cc] : from_f<T>(0.f);
+        }
+    };
+    auto prepare = [&](int b) {
+#pragma unroll
+        for (int s = 0; s < TPW; ++s) {
+            float ss = 0.f, rau = 0.f, rk = 0.f;
+#pragma unroll
+            for (int i = 0; i < EPL; ++i) ss += to_f(pk[s][i]) * to_f(pk[s][i]);
+            const float inv = 1.f / sqrtf(warp_sum(ss) + 1e-6f);
+            float* dst = sm.vec[b][warp * TPW + s] + lane;
+#pragma unroll
+            for (int i = 0; i < EPL; ++i) {
+                const float k = to_f(pk[s][i]), r = to_f(pr[s][i]), w = exp2f(pw[s][i]), u = k * inv;
+                const float au = delta_rate(to_f(pa[s][i]) + bias[i]) * u;
+                dst[32 * i] = u;
+                dst[DP + 32 * i] = r * w;
+                dst[2 * DP + 32 * i] = w;
+                dst[3 * DP + 32 * i] = au;
+                dst[4 * DP + 32 * i] = k;
+                rau += r * au;
+                rk += r * k;
+            }
+            rau = warp_sum(rau);
+            rk = warp_sum(rk);
+            if (lane == 0) sm.dots[b][warp * TPW + s] = make_float2(rau, rk);
+        }
+#pragma unroll
+        for (int i = 0; i < VPT; ++i) {
+            const int x = threadIdx.x + i * 256;
+            if (x < CT * COLS) sm.v[b][x / COLS][x % COLS] = to_f(pv[i]);
+        }
+    };
+    auto run = [&](int b, int count) {
+        for (int t = 0; t < count; ++t) {
+            const float4* p = reinterpret_cast<const float4*>(sm.vec[b][t]) + g;
+            F2 y0 = f2(0.f), y1 = y0, z0 = y0, z1 = y0;
+#pragma unroll
+            for (int i = 0; i < RPL / 4; ++i) {
+                const float4 u = p[LPC * i], rw = p[DP / 4 + LPC * i];
+                y0 = fma2(f2(u.x, u.y), S[2 * i], y0);
+                y1 = fma2(f2(u.z, u.w), S[2 * i + 1], y1);
+                z0 = fma2(f2(rw.x, rw.y), S[2 * i], z0);
+                z1 = fma2(f2(rw.z, rw.w), S[2 * i + 1], z1);
+            }
+            float a0, a1, a2, a3;
+            unpack2(y0, a0, a1);
+            unpack2(y1, a2, a3);
+            float y = (a0 + a1) + (a2 + a3);
+            unpack2(z0, a0, a1);
+            unpack2(z1, a2, a3);
+            float z = (a0 + a1) + (a2 + a3);
+#pragma unroll
+            for (int o = 1; o < LPC; o <<= 1) {
+                y += __shfl_xor_sync(0xffffffffu, y, o);
+                z += __shfl_xor_sync(0xffffffffu, z, o);
+            }
+            const float v = sm.v[b][t][cl];
+            const float2 dots = sm.dots[b][t];
+            if (g == 0) sm.o[b][t][cl] = z - dots.x * y + dots.y * v;
+            const F2 ny = f2(-y), vv = f2(v);
+#pragma unroll
+            for (int i = 0; i < RPL / 4; ++i) {
+                const float4 w = p[2 * DP / 4 + LPC * i], au = p[3 * DP / 4 + LPC * i], k = p[4 * DP / 4 + LPC * i];
+                S[2 * i] = fma2(f2(au.x, au.y), ny, fma2(f2(w.x, w.y), S[2 * i], mul2(f2(k.x, k.y), vv)));
+                S[2 * i + 1] = fma2(f2(au.z, au.w), ny, fma2(f2(w.z, w.w), S[2 * i + 1], mul2(f2(k.z, k.w), vv)));
+            }
+        }
+    };
+    auto flush = [&](int b, int t0, int count) {
+        for (int x = threadIdx.x; x < count * COLS; x += 256) {
+            const int cc = blockIdx.z * COLS + x % COLS;
+            if (cc < a.dim) O[(size_t)(t0 + x / COLS) * step + cc] = sm.o[b][x / COLS][x % COLS];
+        }
+    };
+    load(0);
+    prepare(0);
+    __syncthreads();
+    int b = 0;
+    for (int t0 = 0; t0 < len; t0 += CT, b ^= 1) {
+        const bool more = t0 + CT < len;
+        if (more) load(t0 + CT);
+        run(b, min(CT, len - t0));
+        if (more) prepare(b ^ 1);
+        __syncthreads();
+        flush(b, t0, min(CT, len - t0));       // written again two rounds on, past the next barrier
+    }
+    if (c < a.dim) {
+#pragma unroll
+        for (int i = 0; i < RPL / 4; ++i) {
+            float f[4];
+            unpack2(S[2 * i], f[0], f[1]);
+            unpack2(S[2 * i + 1], f[2], f[3]);
+#pragma unroll
+            for (int e = 0; e < 4; ++e) {
+                const int d = 4 * (g + LPC * i) + e;
+                if (d < a.dim) sp[(size_t)d * a.dim + c] = f[e];
+            }
+        }
+    }
+}
+
+}  // namespace pie
+
+using namespace pie;
+
+static bool delta_ok(const DeltaArgs& a) {
+    return a.dim > 0 && a.dim <= 512 && a.heads > 0 && a.a_bias && a.log_decay && a.state;
+}
+
+// One token per request.
+PIE_API int pie_delta_step(const DeltaArgs* args, int f32, cudaStream_t st) {
+    const DeltaArgs& a = *args;
+    if (a.n <= 0 || a.reqs <= 0) return 0;
+    if (!delta_ok(a)) return (int)cudaErrorInvalidValue;
+    const bool vec = a.dim % 4 == 0 && a.dim >= 64 && a.dim <= 256 && a.slot_stride % 4 == 0 && ((uintptr_t)a.state & 15) == 0 &&
+                     ((uintptr_t)a.v & 15) == 0 && a.ld % 4 == 0;
+    const int cols = vec ? 128 : 32, rpt = (a.dim + 7) / 8;
+    const dim3 grid(a.reqs, a.heads, (a.dim + cols - 1) / cols);
+#define GO(T_, R_, V_) return (int)launch_pdl(delta_step_kernel<T_, R_, V_>, grid, dim3(256), 0, st, a)
+#define GO_R(T_)                            \
+    if (vec) {                              \
+        if (rpt <= 8) GO(T_, 8, 4);         \
+        if (rpt <= 16) GO(T_, 16, 4);       \
+        GO(T_, 32, 4);                      \
+    }                                       \
+    if (rpt <= 4) GO(T_, 4, 1);             \
+    if (rpt <= 8) GO(T_, 8, 1);             \
+    if (rpt <= 16) GO(T_, 16, 1);           \
+    if (rpt <= 32) GO(T_, 32, 1);           \
+    GO(T_, 64, 1)
+    if (f32) { GO_R(float); }
+    GO_R(bf16);
+#undef GO_R
+#undef GO
+}
+
+PIE_API int pie_delta_portions(const DeltaArgs* args, int f32, cudaStream_t st) {
+    const DeltaArgs& a = *args;
+    if (a.n <= 0 || a.reqs <= 0) return 0;
+    if (!delta_ok(a)) return (int)cudaErrorInvalidValue;
+#define GO(T_, R_, L_, C_)                                                                                        \
+    {                                                                                                             \
+        using Smem = DeltaSmem<R_, L_, C_>;                                                                       \
+        auto kern = delta_portion_kernel<T_, R_, L_, C_>;                                                         \
+        const cudaError_t e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)sizeof(Smem)); \
+        if (e != cudaSuccess) return (int)e;                                                                      \
+        kern<<<dim3(a.reqs, a.heads, (a.dim + Smem::COLS - 1) / Smem::COLS), 256, sizeof(Smem), st>>>(a);         \
+        return (int)cudaGetLastError();                                                                           \
+    }
+#define GO_R(T_)                            \
+    if (a.dim <= 32) GO(T_, 4, 8, 16)       \
+    if (a.dim <= 64) GO(T_, 8, 8, 16)       \
+    if (a.dim <= 128) GO(T_, 16, 8, 16)     \
+    if (a.dim <= 256) GO(T_, 32, 8, 16)     \
+    GO(T_, 32, 16, 8)
+    if (f32) { GO_R(float) }
+    GO_R(bf16)
+#undef GO_R
+#undef GO
+}

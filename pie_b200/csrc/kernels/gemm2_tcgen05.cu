@@ -362,6 +362,7 @@ int pie_gemm2_dispatch(const void* A, const void* W, void* C, const void* R, int
         case EPI_STORE: return launch_gemm2<BN_, EPI_STORE>(ta, tb, C, R, M, N, K, ldc, ldr, status, pairs, streamk, ws, cnt, st, tp, ex);       \
         case EPI_RESIDUAL: return launch_gemm2<BN_, EPI_RESIDUAL>(ta, tb, C, R, M, N, K, ldc, ldr, status, pairs, streamk, ws, cnt, st, tp, ex); \
         case EPI_SWIGLU: return launch_gemm2<BN_, EPI_SWIGLU>(ta, tb, C, R, M, N, K, ldc, ldr, status, pairs, streamk, ws, cnt, st, tp, ex);     \
+        case EPI_GEGLU: return launch_gemm2<BN_, EPI_GEGLU>(ta, tb, C, R, M, N, K, ldc, ldr, status, pairs, streamk, ws, cnt, st, tp, ex);       \
         case EPI_XIELU: return launch_gemm2<BN_, EPI_XIELU>(ta, tb, C, R, M, N, K, ldc, ldr, status, pairs, streamk, ws, cnt, st, tp, ex); \
         case EPI_STREAM: return launch_gemm2<BN_, EPI_STREAM>(ta, tb, C, R, M, N, K, ldc, ldr, status, pairs, streamk, ws, cnt, st, tp, ex); \
         case EPI_RS: return launch_gemm2<BN_, EPI_RS>(ta, tb, C, R, M, N, K, ldc, ldr, status, pairs, streamk, ws, cnt, st, tp, ex);             \

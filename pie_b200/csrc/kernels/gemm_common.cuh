@@ -17,13 +17,15 @@ enum GemmEpilogue : int {
     EPI_XIELU = 4,     // C = xIELU(acc + bias), see EpiArgs
     EPI_STREAM = 5,    // out32 = res32 + acc + bias: a 32-bit residual stream; C = the same in bf16
     EPI_CLAMP_GLU = 6, // as EPI_SWIGLU with g = min(gate, limit), u = clamp(up, +-limit): g * sigmoid(1.702 g) * (u + 1)
+    EPI_GEGLU = 7,     // as EPI_SWIGLU with the tanh form of GELU on the gate
     // Swapped operands (small batches): the kernel computes C^T = W * A^T, so its rows are output
     // features and its columns tokens; these epilogues write the tile back transposed. EPI_STORE_T is the first of them.
-    EPI_STORE_T = 7,
-    EPI_RESIDUAL_T = 8,
-    EPI_SWIGLU_T = 9,
-    EPI_XIELU_T = 10,
-    EPI_STREAM_T = 11,
+    EPI_STORE_T = 8,
+    EPI_RESIDUAL_T = 9,
+    EPI_SWIGLU_T = 10,
+    EPI_XIELU_T = 11,
+    EPI_STREAM_T = 12,
+    EPI_GEGLU_T = 13,
 };
 
 // Operands of the epilogues with a bias. xIELU(z) = a z^2 + z / 2 for z > 0, b (e^z - 1 - z) + z / 2 below, with
@@ -44,6 +46,8 @@ __device__ __forceinline__ float glu_value(float g, float u, float limit) {
         u = fminf(fmaxf(u, -limit), limit);
         return g / (1.f + __expf(-1.702f * g)) * (u + 1.f);
     }
+    // (1 + tanh(y)) / 2 = sigmoid(2 y)
+    if (EPI == EPI_GEGLU || EPI == EPI_GEGLU_T) return g / (1.f + __expf(-1.5957691216057308f * (g + 0.044715f * g * g * g))) * u;
     return g / (1.f + __expf(-g)) * u;
 }
 
@@ -177,7 +181,7 @@ __device__ __forceinline__ void epilogue_store_chunk(const uint32_t (&v)[32], in
             for (int e = 0; e < 8; ++e) o[e] = __uint_as_float(v[8 * j + e]);
             *reinterpret_cast<bf16x8*>(dst + 8 * j) = pack8(o);
         }
-    } else if (EPI == EPI_SWIGLU || EPI == EPI_CLAMP_GLU) {
+    } else if (EPI == EPI_SWIGLU || EPI == EPI_CLAMP_GLU || EPI == EPI_GEGLU) {
         bf16* dst = C + (size_t)row * ldc + (col0 >> 1);
         float o[16];
 #pragma unroll
@@ -225,7 +229,7 @@ __device__ __forceinline__ void epilogue_store_64(const uint32_t (&v0)[32], cons
                                                   const XieluCoef* act = nullptr) {
     const int lane = threadIdx.x & 31;
     auto slot = [&](int r, int c) { return reinterpret_cast<bf16x8*>(stage + r * 128 + ((c ^ (r & 7)) << 4)); };
-    if (EPI == EPI_SWIGLU || EPI == EPI_CLAMP_GLU) {
+    if (EPI == EPI_SWIGLU || EPI == EPI_CLAMP_GLU || EPI == EPI_GEGLU) {
         // 64 accumulator columns -> 32 outputs (64 B) per row
         float o[32];
 #pragma unroll
@@ -350,13 +354,13 @@ __device__ __forceinline__ void epilogue_store_64_t(const uint32_t (&v0)[32], co
     const int lane = threadIdx.x & 31;
     bf16* st = reinterpret_cast<bf16*>(stage);
     const int feat = feat0 + lane;
-    if (EPI == EPI_SWIGLU_T) {
+    if (EPI == EPI_SWIGLU_T || EPI == EPI_GEGLU_T) {
         // even lanes hold gate_j, odd lanes up_j of output j = feat / 2
 #pragma unroll
         for (int t = 0; t < 64; ++t) {
             const float mine = __uint_as_float(t < 32 ? v0[t] : v1[t - 32]);
             const float other = __shfl_xor_sync(0xffffffffu, mine, 1);
-            if (!(lane & 1)) st[t * 16 + (lane >> 1)] = __float2bfloat16(mine / (1.f + __expf(-mine)) * other);
+            if (!(lane & 1)) st[t * 16 + (lane >> 1)] = __float2bfloat16(glu_value<EPI>(mine, other, 0.f));
         }
         __syncwarp();
         const int oc0 = feat0 >> 1;

@@ -573,7 +573,7 @@ static int gemm_bf16(const void* A, const void* W, void* C, const void* R, int M
     if (M <= 0 || N <= 0) return 0;
     if (K <= 0 || K % 8 || N % 8 || ldc % 8 || (epilogue == EPI_RESIDUAL && ldr % 8))
         return (int)cudaErrorInvalidValue;
-    if (epilogue == EPI_SWIGLU && N % 32) return (int)cudaErrorInvalidValue;
+    if ((epilogue == EPI_SWIGLU || epilogue == EPI_GEGLU) && N % 32) return (int)cudaErrorInvalidValue;
     GemmWorkspace w;
     if (int rc = current_workspace(&w)) return rc;
     if (g_gemm_pairs && force_bn == 0) {
@@ -603,6 +603,7 @@ static int gemm_bf16(const void* A, const void* W, void* C, const void* R, int M
         case EPI_STORE: return launch_gemm<BN_, EPI_STORE_T>(ta, tb, C, R, N, M, K, ldc, ldr, status, plan, w, st); \
         case EPI_RESIDUAL: return launch_gemm<BN_, EPI_RESIDUAL_T>(ta, tb, C, R, N, M, K, ldc, ldr, status, plan, w, st); \
         case EPI_SWIGLU: return launch_gemm<BN_, EPI_SWIGLU_T>(ta, tb, C, R, N, M, K, ldc, ldr, status, plan, w, st); \
+        case EPI_GEGLU: return launch_gemm<BN_, EPI_GEGLU_T>(ta, tb, C, R, N, M, K, ldc, ldr, status, plan, w, st); \
         case EPI_XIELU: return launch_gemm<BN_, EPI_XIELU_T>(ta, tb, C, R, N, M, K, ldc, ldr, status, plan, w, st, TpArgs{}, ex); \
         case EPI_STREAM: return launch_gemm<BN_, EPI_STREAM_T>(ta, tb, C, R, N, M, K, ldc, ldr, status, plan, w, st, TpArgs{}, ex); \
         default: return (int)cudaErrorInvalidValue;                                               \
@@ -624,6 +625,7 @@ direct:
         case EPI_STORE: return launch_gemm<BN_, EPI_STORE>(ta, tb, C, R, M, N, K, ldc, ldr, status, plan, w, st); \
         case EPI_RESIDUAL: return launch_gemm<BN_, EPI_RESIDUAL>(ta, tb, C, R, M, N, K, ldc, ldr, status, plan, w, st); \
         case EPI_SWIGLU: return launch_gemm<BN_, EPI_SWIGLU>(ta, tb, C, R, M, N, K, ldc, ldr, status, plan, w, st); \
+        case EPI_GEGLU: return launch_gemm<BN_, EPI_GEGLU>(ta, tb, C, R, M, N, K, ldc, ldr, status, plan, w, st); \
         case EPI_XIELU: return launch_gemm<BN_, EPI_XIELU>(ta, tb, C, R, M, N, K, ldc, ldr, status, plan, w, st, TpArgs{}, ex); \
         case EPI_STREAM: return launch_gemm<BN_, EPI_STREAM>(ta, tb, C, R, M, N, K, ldc, ldr, status, plan, w, st, TpArgs{}, ex); \
         default: return (int)cudaErrorInvalidValue;                                               \
@@ -638,7 +640,7 @@ direct:
 PIE_API int pie_gemm_bf16(const void* A, const void* W, void* C, const void* R, int M, int N, int K,
                           int lda, int ldw, int ldc, int ldr, int epilogue, int force_bn,
                           int* status, int num_sms, cudaStream_t st) {
-    if (epilogue < EPI_STORE || epilogue > EPI_SWIGLU) return (int)cudaErrorInvalidValue;
+    if ((epilogue < EPI_STORE || epilogue > EPI_SWIGLU) && epilogue != EPI_GEGLU) return (int)cudaErrorInvalidValue;
     return gemm_bf16(A, W, C, R, M, N, K, lda, ldw, ldc, ldr, epilogue, force_bn, status, num_sms, st, EpiArgs());
 }
 

@@ -631,18 +631,20 @@ __global__ void __launch_bounds__(LA_THREADS) la_chunk_out_kernel(const LinAttnA
 }
 
 // ---------------------------------------------------------- channel decays
-// log_decay[t, c] = log2(sigmoid(z)) / tau, z = a2[c, :] . a1[t, :] + bias[c]; x holds a1 at column 0 of rows of ld.
+// log_decay[t, c] = log2(sigmoid(z)) * factor, z = a2[c, :] . a1[t, :] + bias[c]; x holds a1 at column 0 of rows of ld.
+// BOUNDED: -sigmoid(z) * factor * log2(e) with a1 passed through tanh first: a decay between exp(-factor) and 1.
 constexpr int LD_TOK = 8;
-template <typename T>
+template <typename T, bool BOUNDED>
 __global__ void __launch_bounds__(256) la_decay_kernel(const T* __restrict__ x, int ld, const T* __restrict__ a2, const T* __restrict__ bias,
-                                                       float* __restrict__ out, int n, int channels, int rank, float inv_tau) {
+                                                       float* __restrict__ out, int n, int channels, int rank, float factor) {
     extern __shared__ __align__(16) float sx[];          // [rank][LD_TOK]
     pdl_trigger();
     pdl_wait();
     const int t0 = blockIdx.x * LD_TOK, nt = min(LD_TOK, n - t0);
     for (int i = threadIdx.x; i < LD_TOK * rank; i += 256) {
         const int s = i / rank, j = i - s * rank;
-        sx[j * LD_TOK + s] = s < nt ? to_f(x[(size_t)(t0 + s) * ld + j]) : 0.f;
+        const float f = s < nt ? to_f(x[(size_t)(t0 + s) * ld + j]) : 0.f;
+        sx[j * LD_TOK + s] = BOUNDED ? tanhf(f) : f;
     }
     __syncthreads();
     const int c = blockIdx.y * 256 + threadIdx.x;
@@ -661,7 +663,9 @@ __global__ void __launch_bounds__(256) la_decay_kernel(const T* __restrict__ x, 
     }
 #pragma unroll
     for (int s = 0; s < LD_TOK; ++s)
-        if (s < nt) out[(size_t)(t0 + s) * channels + c] = (fminf(z[s], 0.f) - log1pf(expf(-fabsf(z[s])))) * (1.4426950408889634f * inv_tau);
+        if (s < nt)
+            out[(size_t)(t0 + s) * channels + c] = (BOUNDED ? -1.f / (1.f + expf(-z[s])) : fminf(z[s], 0.f) - log1pf(expf(-fabsf(z[s])))) *
+                                                   (1.4426950408889634f * factor);
 }
 
 // ------------------------------------------- exponential gates of a matrix memory
@@ -959,17 +963,20 @@ PIE_API int pie_linear_attn_chunked(const LinAttnArgs* args, cudaStream_t st) {
     return (int)cudaGetLastError();
 }
 
-PIE_API int pie_linear_decay(const void* x, int ld, const void* a2, const void* bias, float* out, int n, int channels, int rank, float inv_tau,
-                             int f32, cudaStream_t st) {
+PIE_API int pie_linear_decay(const void* x, int ld, const void* a2, const void* bias, float* out, int n, int channels, int rank, float factor,
+                             int bounded, int f32, cudaStream_t st) {
     if (n <= 0) return 0;
     if (rank <= 0 || rank > 1024 || channels <= 0) return (int)cudaErrorInvalidValue;
     const dim3 grid((n + LD_TOK - 1) / LD_TOK, (channels + 255) / 256);
     const size_t sm = (size_t)LD_TOK * rank * 4;
-    if (f32)
-        return (int)launch_pdl(la_decay_kernel<float>, grid, dim3(256), sm, st, (const float*)x, ld, (const float*)a2, (const float*)bias, out, n,
-                               channels, rank, inv_tau);
-    return (int)launch_pdl(la_decay_kernel<bf16>, grid, dim3(256), sm, st, (const bf16*)x, ld, (const bf16*)a2, (const bf16*)bias, out, n,
-                           channels, rank, inv_tau);
+#define GO(T_, B_) \
+    return (int)launch_pdl(la_decay_kernel<T_, B_>, grid, dim3(256), sm, st, (const T_*)x, ld, (const T_*)a2, (const T_*)bias, out, n, channels, \
+                           rank, factor)
+    if (f32 && bounded) GO(float, true);
+    if (f32) GO(float, false);
+    if (bounded) GO(bf16, true);
+    GO(bf16, false);
+#undef GO
 }
 
 // single: every request brings one token.

@@ -183,7 +183,7 @@ class TorchDriver:
                     num_pages = int(t.item())
         self.kv = KVCache(len(cfg.latent_cache_layers) if cfg.latent is not None else cfg.num_hidden_layers, num_pages, hkv,
                           page_size, cfg.head_dim, self.dtype, self.device, swap_pages, kv_dtype=kv_dtype,
-                          latent=cfg.latent is not None, layer_shapes=cfg.kv_layers if cfg.blocks is not None else None)
+                          latent=cfg.latent is not None, layer_shapes=cfg.kv_page_shapes(page_size) if cfg.blocks is not None else None)
         self.model.kv_scale = self.kv.scale
         # Gated DeltaNet, Mamba-2 and token-shifted layers keep their state in slots of a recurrent-state cache, one per resident context
         self.rs = None
@@ -273,8 +273,7 @@ class TorchDriver:
         tp = self.par.tp_size
         if self.cfg.blocks is not None:
             # linear-attention states are large (a slot holds every layer's [heads, dim, vdim] in 32-bit)
-            elems = sum(b.recurrent.state_elems for b in self.cfg.blocks if b.recurrent is not None)
-            usable -= 4 * elems * (rs_slots or self._default_rs_slots(max_requests))
+            usable -= 4 * self.cfg.slot_layout()[-1] * (rs_slots or self._default_rs_slots(max_requests))
         if profile:
             plan = mp.plan(self.cfg, usable, 1.0, profile, self.page_size, tp)
             max_requests, max_tokens = plan.max_requests, plan.max_tokens
@@ -459,7 +458,7 @@ class TorchDriver:
                 torch.arange(rb + 1, dtype=torch.int32, device=dev), torch.arange(rb, dtype=torch.int32, device=dev),
                 s.d("rs_slots", rb), s.d("rs_reset", rb), list(range(rb + 1)), [-1] * rb, [0] * rb,
                 self.rs.conv_state, self.rs.rec_state, self.rs.layer_index, shift_state=self.rs.shift_state,
-                linear_state=self.rs.linear_state, linear_at=self.rs.linear_at, **self.rs.device_scratch(rb, rb))
+                linear_state=self.rs.linear_state, linear_at=self.rs.linear_at, **self.rs.carried, **self.rs.device_scratch(rb, rb))
         return cache[rb]
 
     def _fill_rs_decode(self, req: ForwardRequest, r: int, rb: int) -> None:

@@ -18,11 +18,12 @@ from .schema import CopyDir, CopyRequest
 
 
 class LayerPages:
-    """Pages of layers with unequal shapes: one tensor [pages + 1, 2, kv heads, page, D] (latent rows: [pages + 1, page, row])
-    per layer that has a cache."""
+    """Pages of layers with unequal shapes: one tensor [pages + 1, 2, kv heads, page, D] (keys that are the values: 1 in place of
+    2; latent rows: [pages + 1, page, row]) per layer that has a cache. `means` [pages + 1, 2, kv heads, blocks, D]: of those
+    that keep the mean key and value of every block of tokens, with the page of the block's last one (else None)."""
 
-    def __init__(self, layers):
-        self.layers = layers
+    def __init__(self, layers, means):
+        self.layers, self.means = layers, means
 
     def __getitem__(self, i: int):
         return self.layers[i]
@@ -41,8 +42,8 @@ class KVCache:
         `latent`: pages of latent attention, one row of `head_dim` elements per token (latent, then the rotated key part
         that all heads share) in ``[layers, pages + 1, page_size, row]``; `layers` counts the layers that write rows.
 
-        `layer_shapes`: (kv heads, head_dim) of every layer that has a cache, where a model's layers differ (`data` is then a
-        `LayerPages`; it may be empty); no heads: latent rows of that width."""
+        `layer_shapes`: shapes of a page in every layer that has a cache (`ModelConfig.kv_page_shapes`), where a model's layers
+        differ (`data` is then a `LayerPages`; it may be empty)."""
         if page_size % 16:
             raise ValueError("kv page size must be a multiple of 16")
         if kv_dtype not in ("auto", "bf16", "fp8_e4m3"):
@@ -58,12 +59,17 @@ class KVCache:
         self.page_size, self.head_dim, self.dtype = page_size, head_dim, dtype
         self.device = torch.device(device)
         if layer_shapes is not None:
-            shapes = [(1, (2, h, page_size, d) if h else (page_size, d)) for h, d in layer_shapes]
+            shapes = [(1, rows) for rows, _ in layer_shapes] + [(1, means) for _, means in layer_shapes if means is not None]
         else:
             shapes = [(layers, (page_size, head_dim) if latent else (2, kv_heads, page_size, head_dim))]
         # zero-filled: unwritten slots are multiplied by p == 0 in attention and must be finite
         self.parts = [torch.zeros(n, num_pages + 1, *shape, dtype=dtype, device=self.device) for n, shape in shapes]
-        self.data = self.parts[0] if layer_shapes is None else LayerPages([t[0] for t in self.parts])
+        if layer_shapes is None:
+            self.data = self.parts[0]
+        else:
+            means = iter(self.parts[len(layer_shapes):])
+            self.data = LayerPages([t[0] for t in self.parts[:len(layer_shapes)]],
+                                   [next(means)[0] if m is not None else None for _, m in layer_shapes])
         self.pad_page = num_pages
         self.swap_pages = swap_pages
         self.host = None

@@ -2,7 +2,8 @@
 slot) the tail of the short convolution's inputs and the fp32 state (delta-rule state [heads, dk, dv], or state-space
 state [heads, head_dim, state]), or the previous token's normalised input (token shift, [width] fp32). Linear-attention
 mixers of layers described one by one (any head sizes) keep [heads, dim, vdim] fp32 each (a matrix memory also [heads, dim]
-and [heads]), all layers of a slot in one row.
+and [heads]), all layers of a slot in one row, with the last inputs of their input convolutions ([taps - 1, width] fp32 for
+each sublayer) and the token before where the embedding wants it (`ModelConfig.slot_layout`).
 A slot belongs to one resident context; the runtime's
 slot pool (`runtime/rs_cache.py`) hands slots out, tells the driver when a slot must start from zero
 (`rs_reset`) and asks for a slot copy when a context forks.
@@ -12,6 +13,7 @@ Counterpart of driver/cuda/src/recurrent_state_cache.hpp:1-40 (slabs per layer a
 from __future__ import annotations
 
 from dataclasses import dataclass
+from functools import cached_property
 from typing import Dict, List, Optional
 
 import numpy as np
@@ -38,6 +40,10 @@ class RecurrentInputs:
     shift_stage: Optional[torch.Tensor] = None   # [R, W] fp32: a portion's last input until its readers are done
     linear_state: Optional[torch.Tensor] = None  # [S, elements] fp32: the states of all linear-attention layers of a slot
     linear_at: Optional[Dict[int, int]] = None   # model layer -> its first element in a row of `linear_state`
+    history_at: Optional[dict] = None            # (model layer, half) -> first element of its convolution's history
+    history_elems: int = 0                       # numbers of one history
+    token_at: Optional[int] = None               # element that holds the token before, as an integer
+    conv_stage: Optional[torch.Tensor] = None    # [R, taps - 1, W] fp32: the new history of portions until its readers are done
     pieces: Optional[tuple] = None # the portions cut for the chunked form (`ops.linear.chunk_pieces`)
     staged: Optional[int] = None   # requests the stage is committed for (0: none of this fire's portions uses it)
 
@@ -45,6 +51,23 @@ class RecurrentInputs:
         """Layer `li`'s columns of the linear-attention state cache [slots, all layers]."""
         at = self.linear_at[li]
         return self.linear_state[:, at:at + elems]
+
+    def history_of(self, li: int, half: str) -> Optional[torch.Tensor]:
+        """Columns of the state cache with the history of an input convolution (None: it reaches no further back)."""
+        if not self.history_at:
+            return None
+        at = self.history_at[li, half]
+        return self.linear_state[:, at:at + self.history_elems]
+
+    @property
+    def token_before(self) -> torch.Tensor:
+        """int32 [slots] (strided): the token each sequence ended with."""
+        return self.linear_state[:, self.token_at].view(torch.int32)
+
+    @cached_property
+    def has_portions(self) -> bool:
+        """Whether some request of the fire brings more than one token."""
+        return any(b - a > 1 for a, b in zip(self.qo_host, self.qo_host[1:]))
 
 
 class RecurrentStateCache:
@@ -57,12 +80,10 @@ class RecurrentStateCache:
         self.conv_state = self.rec_state = self.shift_state = self.linear_state = None
         self.linear_at: Optional[Dict[int, int]] = None
         self.conv_channels = 0
+        self.carried: dict = {}
         if cfg.blocks is not None:
-            self.linear_at, at = {}, 0
-            for li, b in enumerate(cfg.blocks):
-                if b.recurrent is not None:
-                    self.linear_at[li] = at
-                    at += -(-b.recurrent.state_elems // 4) * 4
+            self.linear_at, histories, before, at = cfg.slot_layout()
+            self.carried = dict(history_at=histories, history_elems=max(0, cfg.conv_taps - 1) * cfg.hidden_size, token_at=before)
             self.linear_state = torch.zeros(num_slots, max(at, 4), dtype=torch.float32, device=self.device)
             return
         if cfg.token_shift:
@@ -91,6 +112,8 @@ class RecurrentStateCache:
 
     def device_scratch(self, n: int, r: int) -> dict:
         """Device scratch of a fire of n tokens in r requests."""
+        if self.device.type == "cuda" and self.carried.get("history_at") and n > r:
+            return {"conv_stage": torch.empty(max(r, 1), self.carried["history_elems"], dtype=torch.float32, device=self.device)}
         if self.device.type != "cuda" or self.linear_state is not None:
             return {}
         if self.shift_state is not None:
@@ -113,7 +136,7 @@ class RecurrentStateCache:
         t = lambda a: torch.from_numpy(a).to(dev)
         return RecurrentInputs(t(qo), t(tok_req), t(slots), t(reset), qo.tolist(), slots.tolist(), reset.tolist(),
                                self.conv_state, self.rec_state, self.layer_index, shift_state=self.shift_state,
-                               linear_state=self.linear_state, linear_at=self.linear_at, **self.device_scratch(int(qo[-1]), r))
+                               linear_state=self.linear_state, linear_at=self.linear_at, **self.carried, **self.device_scratch(int(qo[-1]), r))
 
     def copy_slot(self, src: int, dst: int) -> None:
         """dst <- src in every layer (a forked context continues from its parent's state)."""

@@ -1,6 +1,6 @@
 """Descriptions of layers that a configuration lists one by one (blocks over a 32-bit residual stream): each block names
 its mixer and its feed-forward, with sizes and constants of its own. The Retodra reader and writer of `config.json` are at
-the end, those of Nukelix in `nukelix.py`.
+the end, those of Nukelix in `nukelix.py`, those of Vulanex in `vulanex.py`.
 """
 from __future__ import annotations
 
@@ -203,17 +203,84 @@ class MatrixMemorySpec:
 
 
 @dataclass
+class PlainAttentionSpec:
+    """Grouped-query attention without biases or gates; the rest is optional. `head_norm`: q and k are normed head by head.
+    `rot`: rotary positions. `q_temp` (coef, every): the query at position p is multiplied by 1 + coef * ln(floor((p + 1) /
+    every) + 1). `shared_kv`: the values are the keys, cached once. A query sees itself, the `window` - 1 tokens before it and,
+    with `pool`, the mean key and value of every block of that many tokens wholly before the window. `sink`: a learned score
+    per head without a value takes its share of the softmax."""
+    heads: int
+    kv_heads: int
+    dim: int
+    vdim: int
+    scale: float
+    rot: Optional[RotarySpec] = None
+    head_norm: bool = False
+    q_temp: Optional[Tuple[float, int]] = None
+    shared_kv: bool = False
+    window: int = EVERYTHING
+    pool: int = 0
+    sink: bool = False
+
+    group = BiasedAttentionSpec.group
+    group_pad = BiasedAttentionSpec.group_pad
+    head_dim = BiasedAttentionSpec.head_dim
+
+    @property
+    def planes(self) -> int:
+        """Rows a page holds per token and head: a key and a value, or one for both."""
+        return 1 if self.shared_kv else 2
+
+
+@dataclass
+class DeltaRuleSpec:
+    """Delta rule with a decay and a removal rate per key channel: a state [dim, dim] per head. The decay lies between
+    exp(-`bound`) and 1; it is a projection of rank `rank` (None: the checkpoint tells)."""
+    heads: int
+    dim: int
+    rank: Optional[int] = None
+    bound: float = math.exp(-0.5)
+
+    qk = GatedLinearSpec.qk
+
+    @property
+    def vdim(self) -> int:
+        return self.dim
+
+    @property
+    def values(self) -> int:
+        return self.heads * self.dim
+
+    @property
+    def state_elems(self) -> int:
+        return self.heads * self.dim * self.dim
+
+
+@dataclass
 class ParallelSpec:
-    """Attention and a recurrent mixer side by side on the same input."""
-    left: Union[BiasedAttentionSpec, GroupedAttentionSpec]
-    right: Union[LightningSpec, MatrixMemorySpec]
+    """Attention and a recurrent mixer side by side on the same input. `out_norms`: each side's output projection is normed
+    before the sum."""
+    left: Union[BiasedAttentionSpec, GroupedAttentionSpec, PlainAttentionSpec]
+    right: Union[LightningSpec, MatrixMemorySpec, DeltaRuleSpec]
     left_scale: float
     right_scale: float
+    out_norms: bool = False
+
+
+@dataclass
+class PairSpec:
+    """An embedding row for the pair (token before, token): number (before * mul_prev + token * mul_cur) mod buckets, and one
+    more row for a sequence's first token."""
+    buckets: int
+    mul_prev: int
+    mul_cur: int
 
 
 @dataclass
 class DenseSpec:
+    """GLU feed-forward of width `ff`; `act`: activation of the gate ("silu" | "gelu_tanh")."""
     ff: int
+    act: str = "silu"
 
 
 @dataclass
@@ -238,24 +305,24 @@ class ExpertsSpec:
 
 @dataclass
 class BlockSpec:
-    mixer: Union[GatedLinearSpec, ParallelSpec, GroupedAttentionSpec, LatentSpec]
+    mixer: Union[GatedLinearSpec, ParallelSpec, GroupedAttentionSpec, PlainAttentionSpec, LatentSpec]
     ff: Union[DenseSpec, ExpertsSpec, None]
 
     @property
-    def attention(self) -> Union[BiasedAttentionSpec, GroupedAttentionSpec, None]:
+    def attention(self) -> Union[BiasedAttentionSpec, GroupedAttentionSpec, PlainAttentionSpec, None]:
         """The part of the mixer that keeps keys and values in pages."""
         a = self.mixer.left if isinstance(self.mixer, ParallelSpec) else self.mixer
-        return a if isinstance(a, (BiasedAttentionSpec, GroupedAttentionSpec)) else None
+        return a if isinstance(a, (BiasedAttentionSpec, GroupedAttentionSpec, PlainAttentionSpec)) else None
 
     @property
     def latent(self) -> Optional[LatentSpec]:
         return self.mixer if isinstance(self.mixer, LatentSpec) else None
 
     @property
-    def recurrent(self) -> Union[GatedLinearSpec, LightningSpec, MatrixMemorySpec, None]:
+    def recurrent(self) -> Union[GatedLinearSpec, LightningSpec, MatrixMemorySpec, DeltaRuleSpec, None]:
         """The part of the mixer whose state is carried from token to token."""
         r = self.mixer.right if isinstance(self.mixer, ParallelSpec) else self.mixer
-        return r if isinstance(r, (GatedLinearSpec, LightningSpec, MatrixMemorySpec)) else None
+        return r if isinstance(r, (GatedLinearSpec, LightningSpec, MatrixMemorySpec, DeltaRuleSpec)) else None
 
 
 def projection_sizes(mixer) -> Dict[str, int]:
@@ -268,6 +335,11 @@ def projection_sizes(mixer) -> Dict[str, int]:
         return {f"{side}.{n}": k for side, part in (("left", mixer.left), ("right", mixer.right)) for n, k in projection_sizes(part).items()}
     if isinstance(mixer, (LightningSpec, MatrixMemorySpec)):
         return {"q": mixer.qk, "k": mixer.qk, "v": mixer.values, "g": mixer.values}
+    if isinstance(mixer, DeltaRuleSpec):
+        return {"r": mixer.qk, "k": mixer.qk, "v": mixer.values, "g": mixer.values, "a": mixer.qk, "w1": mixer.rank}
+    if isinstance(mixer, PlainAttentionSpec):
+        rows = {"q": mixer.heads * mixer.dim, "k": mixer.kv_heads * mixer.dim}
+        return rows if mixer.shared_kv else {**rows, "v": mixer.kv_heads * mixer.vdim}
     gates = mixer.heads if isinstance(mixer, GroupedAttentionSpec) else mixer.heads * mixer.vdim
     return {"q": mixer.heads * mixer.dim, "k": mixer.kv_heads * mixer.dim, "v": mixer.kv_heads * mixer.vdim, "g": gates}
 

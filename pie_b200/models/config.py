@@ -6,18 +6,20 @@ Keys consumed mirror the reference's HF config reader
 from __future__ import annotations
 
 import json
+import math
 from dataclasses import dataclass, field, asdict
 from pathlib import Path
 from typing import Optional
 
-from .block_spec import EVERYTHING, LatentSpec, _pad, retodra_config, retodra_shape
+from .block_spec import EVERYTHING, LatentSpec, PairSpec, _pad, retodra_config, retodra_shape
 from .nukelix import nukelix_config, nukelix_shape
+from .vulanex import vulanex_config, vulanex_shape
 
 LLAMA_LIKE = {"llama", "qwen2", "qwen3", "mistral", "phi3"}   # pre-norm decoder blocks with SwiGLU and rotate-half RoPE
 # `model_type` strings of checkpoints this build loads (the architecture registry of the loader)
 SUPPORTED_MODEL_TYPES = ("llama", "mistral", "qwen2", "qwen3", "phi3", "qwen3_moe", "mixtral", "olmo2", "olmo3", "gpt_oss",
                          "qwen3_5", "qwen3_next", "mamba2_hybrid", "gemma2", "gemma3_text", "gemma3", "qwen2_moe", "qwen2_vl",
-                         "qwen2_audio", "puzutar", "retodra", "nukelix")
+                         "qwen2_audio", "puzutar", "retodra", "nukelix", "vulanex")
 MAMBA_TYPES = {"mamba2_hybrid"}         # Mamba-2 (state-space) mixers in llama-like blocks, between full-attention layers
 GDN_TYPES = {"qwen3_5", "qwen3_next"}   # hybrids: Gated DeltaNet (linear attention) layers between full-attention layers
 POST_NORM = {"olmo2", "olmo3"}       # same block with the norms after attention / MLP and q, k norms over all heads
@@ -26,7 +28,7 @@ MOE_TYPES = {"qwen3_moe", "mixtral", "gpt_oss", "qwen2_moe"}
 # alternating local / global layers (Gemma-3: a RoPE base of their own for the local ones; Gemma-2: soft-capped logits)
 GEMMA_TYPES = {"gemma2", "gemma3_text", "gemma3"}
 # configs that name the design under "architecture" instead of "model_type"
-ARCHITECTURES = {"Puzutar": "puzutar", "Retodra": "retodra", "Nukelix": "nukelix"}
+ARCHITECTURES = {"Puzutar": "puzutar", "Retodra": "retodra", "Nukelix": "nukelix", "Vulanex": "vulanex"}
 
 
 def config_model_type(cfg: dict) -> str:
@@ -91,9 +93,13 @@ class ModelConfig:
     norm_groups: int = 1               # RMSNorm over this many equal parts of the width, each with its own mean square
     token_shift: bool = False          # the mixer reads h + (previous token's h - h) * shift: state of a sequence
     token_side_dim: int = 0            # width of the per-layer token input (0: none)
-    # layers described one by one over a 32-bit residual stream: sandwich-normed blocks, or (post_norm) blocks that norm
-    # their sublayers' outputs only
+    # layers described one by one over a 32-bit residual stream: sandwich-normed blocks, (post_norm) blocks that norm their
+    # sublayers' outputs only, or (layer_norm) blocks that read the stream through a layer norm and a convolution
     blocks: Optional[list] = None      # BlockSpec per layer
+    layer_norm: bool = False
+    conv_taps: int = 0                 # taps of the causal convolution added to every sublayer's input (0: none): state of a sequence
+    token_pairs: Optional[PairSpec] = None   # embedding rows for (token before, token): state of a sequence
+    logit_scale: float = 1.0
     # quantisation of the linear weights: None | "fp8_block" (128x128 weight scales)
     quantization: Optional[str] = None
     dtype: str = "bfloat16"
@@ -147,20 +153,49 @@ class ModelConfig:
 
     @property
     def kv_layers(self) -> list:
-        """(kv heads, head dim) of every layer that has a cache, in order; latent rows count as no head of the row's width."""
+        """(kv heads, head dim) of every layer that has a cache, in order; latent rows count as no head of the row's width. Two
+        more numbers where a layer's pages are laid out otherwise: rows per token and head, tokens per mean (0: no means)."""
+        def shape(b):
+            if b.latent is not None:
+                return 0, b.latent.row
+            a = b.attention
+            planes, pool = getattr(a, "planes", 2), getattr(a, "pool", 0)
+            return (a.kv_heads, a.head_dim) if (planes, pool) == (2, 0) else (a.kv_heads, a.head_dim, planes, pool)
         if self.blocks is not None:
-            return [(0, b.latent.row) if b.latent is not None else (b.attention.kv_heads, b.attention.head_dim)
-                    for b in self.blocks if b.latent is not None or b.attention is not None]
+            return [shape(b) for b in self.blocks if b.latent is not None or b.attention is not None]
         return [(self.num_key_value_heads, self.head_dim)] * self.num_hidden_layers
 
-    @property
-    def kv_elems_per_token(self) -> int:
-        """Cache elements one token takes over all layers (unsharded)."""
+    def kv_page_shapes(self, page_size: int) -> list:
+        """Shapes of one page in every layer that has a cache: of its rows, and of the means beside them (None: none)."""
+        out = []
+        for h, d, *laid in self.kv_layers:
+            planes, pool = laid or (2, 0)
+            out.append(((planes, h, page_size, d) if h else (page_size, d), (2, h, -(-page_size // pool), d) if pool else None))
+        return out
+
+    def kv_elems_per_page(self, page_size: int) -> int:
+        """Cache elements one page takes over all layers (unsharded)."""
         if self.latent is not None:
-            return len(self.latent_cache_layers) * self.latent_row
+            return len(self.latent_cache_layers) * self.latent_row * page_size
         if self.blocks is not None:
-            return sum(2 * h * d if h else d for h, d in self.kv_layers)
-        return self.num_hidden_layers * 2 * self.num_key_value_heads * self.head_dim
+            return sum(math.prod(s) for pair in self.kv_page_shapes(page_size) for s in pair if s is not None)
+        return self.num_hidden_layers * 2 * self.num_key_value_heads * self.head_dim * page_size
+
+    def slot_layout(self) -> tuple:
+        """What a sequence carries in a row of the state cache of layers described one by one, by first element: recurrent
+        states by layer, histories of the input convolutions by (layer, half), the token before (None: not kept); the row's
+        elements."""
+        states, histories, before, at = {}, {}, None, 0
+        for li, b in enumerate(self.blocks):
+            if b.recurrent is not None:
+                states[li], at = at, at + _pad(b.recurrent.state_elems, 4)
+        if self.conv_taps > 1:
+            for li, b in enumerate(self.blocks):
+                for half in ("1", "2") if b.ff is not None else ("1",):
+                    histories[li, half], at = at, at + _pad((self.conv_taps - 1) * self.hidden_size, 4)
+        if self.token_pairs is not None:
+            before, at = at, at + 4
+        return states, histories, before, at
 
     @property
     def latent_row(self) -> int:
@@ -198,7 +233,7 @@ class ModelConfig:
         if self.blocks is not None:
             b = self.blocks[li]
             a = b.latent or b.attention
-            return 0 if a is None else -1 if a.window == EVERYTHING or getattr(a, "keep_first", 0) else a.window - 1
+            return 0 if a is None else -1 if a.window == EVERYTHING or getattr(a, "keep_first", 0) or getattr(a, "pool", 0) else a.window - 1
         if not self.sliding_window or self.sliding_window <= 0:
             return -1
         if self.layer_types is not None and self.layer_types[li] != "sliding_attention":
@@ -231,6 +266,8 @@ class ModelConfig:
             return retodra_config(cfg, name)
         if mt == "nukelix":
             return nukelix_config(cfg, name)
+        if mt == "vulanex":
+            return vulanex_config(cfg, name)
         if mt == "gemma3" and "text_config" in cfg:       # multimodal wrapper: the language model's own section
             cfg = dict(cfg["text_config"], model_type="gemma3_text")
             mt = "gemma3_text"
@@ -520,6 +557,10 @@ LAYERED_PRESETS = {
     "tiny-retodra": (retodra_config, retodra_shape, dict(
         layers=4, width=256, gla_heads=2, gla_dim=48, gla_vdim=64, rank=8, heads=6, kv_heads=2, dim=40, window=50, buckets=12,
         right_heads=3, right_dim=32, right_vdim=40, ff=384, experts=6, identity=2, top=3, expert_ff=96, vocab=32000)),
+    "vulanex-8b": (vulanex_config, vulanex_shape, dict()),
+    "tiny-vulanex": (vulanex_config, vulanex_shape, dict(
+        layers=4, width=256, heads=6, kv_heads=2, dim=40, vdim=56, window=50, pool=12, every=20, right_heads=3, right_dim=32, rank=8, ff=384,
+        vocab=32000, buckets=509, taps=3)),
     "tiny-nukelix": (nukelix_config, nukelix_shape, dict(
         layers=4, width=256, heads=6, kv_heads=2, dim=40, window=50, keep_first=3, right_heads=3, right_dim=32, right_vdim=40, lat_heads=4,
         lat_dim=24, rot_dim=8, q_rank=72, kv_rank=48, ff=96, experts=6, top=2, shared=112, vocab=32000)),

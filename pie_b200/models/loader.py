@@ -33,10 +33,11 @@ from typing import Callable, Dict, List, Optional, Sequence, Tuple
 
 import torch
 
-from .block_spec import (BiasedAttentionSpec, DenseSpec, ExpertsSpec, GatedLinearSpec, GroupedAttentionSpec, LatentSpec, MatrixMemorySpec,
-                         ParallelSpec, projection_columns, projection_sizes, retodra_dict)
+from .block_spec import (BiasedAttentionSpec, DeltaRuleSpec, DenseSpec, ExpertsSpec, GatedLinearSpec, GroupedAttentionSpec, LatentSpec,
+                         MatrixMemorySpec, ParallelSpec, PlainAttentionSpec, projection_columns, projection_sizes, retodra_dict)
 from .config import ModelConfig, _pad, _puzutar_dict
 from .nukelix import nukelix_dict
+from .vulanex import vulanex_dict
 from .weights import kv_head_range, torch_dtype
 
 
@@ -359,14 +360,15 @@ def complete_blocks(cfg: ModelConfig, reader) -> None:
     """Sizes that only the checkpoint's tensors give: the rank of a decay projection, the rows of a bias table."""
     have = set(reader.names())
     for i, b in enumerate(cfg.blocks):
-        if not isinstance(b.mixer, GatedLinearSpec) and not isinstance(b.attention, BiasedAttentionSpec):
+        ranked = b.recurrent if isinstance(b.recurrent, (GatedLinearSpec, DeltaRuleSpec)) else None
+        if ranked is None and not isinstance(b.attention, BiasedAttentionSpec):
             continue
-        name = f"l{i}.mix.a1" if isinstance(b.mixer, GatedLinearSpec) else f"l{i}.mix.left.rel"
+        name = f"l{i}.mix." + ("left.rel" if ranked is None else "a1" if isinstance(ranked, GatedLinearSpec) else "right.w1")
         if name not in have:
             raise KeyError(f"checkpoint has no tensor {name}")
         rows = int(reader.get_slice(name).get_shape()[0])
-        if isinstance(b.mixer, GatedLinearSpec):
-            b.mixer.rank = rows
+        if ranked is not None:
+            ranked.rank = rows
         else:
             a = b.attention
             a.buckets = rows
@@ -375,9 +377,9 @@ def complete_blocks(cfg: ModelConfig, reader) -> None:
 
 
 def _compile_blocks(cfg: ModelConfig, names: set, tp_size: int, dtype: str) -> Program:
-    """Layout plan of layers described one by one (Retodra and Nukelix names). Fused per layer: every projection that reads
+    """Layout plan of layers described one by one (Retodra, Nukelix and Vulanex names). Fused per layer: every projection that reads
     the mixer's input (`w_in`, each part on a multiple of 8 rows: `block_spec.projection_columns`), the output projections of
-    two mixers side by side along K (`w_out`), gate and up interleaved. Gates of a matrix memory stay apart (`w_gates`): they
+    two mixers side by side along K (`w_out`; apart where each is normed on its own: `w_left`, `w_right`), gate and up interleaved. Gates of a matrix memory stay apart (`w_gates`): they
     are wanted in 32-bit. Dimensions a GEMM sees are padded with zeros, those of a gated feed-forward to 16."""
     if tp_size > 1:
         raise NotImplementedError("layers described one by one under tensor parallelism")
@@ -395,6 +397,12 @@ def _compile_blocks(cfg: ModelConfig, names: set, tp_size: int, dtype: str) -> P
     def attention(P, X, a):
         """Norms and biases of grouped attention (`X`: the checkpoint's prefix); returns its output projection."""
         nq, nk, nv = a.heads * a.dim, a.kv_heads * a.dim, a.kv_heads * a.vdim
+        if isinstance(a, PlainAttentionSpec):
+            if a.head_norm:
+                att[P + "q_norm"], att[P + "k_norm"] = r(X + "q.norm", a.dim), r(X + "k.norm", a.dim)
+            if a.sink:
+                att[P + "sink"] = Keep32(r(X + "sink", a.heads))
+            return Pad(r(X + "o", W, a.heads * a.vdim))
         att[P + "q_norm"], att[P + "k_norm"] = r(X + "q.norm", nq), r(X + "k.norm", nk)
         if isinstance(a, BiasedAttentionSpec):
             if a.buckets is None:
@@ -409,10 +417,18 @@ def _compile_blocks(cfg: ModelConfig, names: set, tp_size: int, dtype: str) -> P
     att["embed"] = r("embed", cfg.vocab_size, W)
     att["lm_head"] = Pad(r("embed" if cfg.tie_word_embeddings else "head", cfg.vocab_size, W))
     att["final_norm"] = r("final.norm", W)
+    if cfg.layer_norm:
+        att["final_norm_b"] = r("final.norm.b", W)
+    if cfg.token_pairs is not None:
+        att["pairs"] = r("bigram", cfg.token_pairs.buckets + 1, W)
     for li, b in enumerate(cfg.blocks):
         L, P, X = f"l{li}.", f"layers.{li}.", f"l{li}.mix."
         for h in ("1", "2") if b.ff is not None else ("1",):
-            if cfg.post_norm:
+            if cfg.conv_taps:
+                att[P + "conv" + h] = r(L + "canon" + h, W, cfg.conv_taps)
+            if cfg.layer_norm:
+                att[P + "ln" + h], att[P + f"ln{h}_b"] = r(L + "norm" + h, W), r(L + f"norm{h}.b", W)
+            elif cfg.post_norm:
                 att[P + f"ln{h}b"] = r(L + "norm" + h, W)
             else:
                 att[P + "ln" + h], att[P + f"ln{h}b"], att[P + "ls" + h] = r(L + "norm" + h, W), r(L + f"norm{h}b", W), r(L + "ls" + h, W)
@@ -427,8 +443,16 @@ def _compile_blocks(cfg: ModelConfig, names: set, tp_size: int, dtype: str) -> P
             att[P + "w_uq"] = Pad(r(X + "uq", m.q_rows, m.q_rank))
             att[P + "w_uk"], att[P + "w_uv"] = r(X + "uk", m.heads * m.dim, m.kv_rank), r(X + "uv", m.heads * m.vdim, m.kv_rank)
             att[P + "w_out"] = Pad(r(X + "o", W, m.heads * m.vdim))
-        elif isinstance(m, GroupedAttentionSpec):
+        elif isinstance(m, (GroupedAttentionSpec, PlainAttentionSpec)):
             att[P + "w_out"] = attention(P, X, m)
+        elif isinstance(m.right, DeltaRuleSpec):
+            s, Y = m.right, X + "right."
+            if s.rank is None:
+                raise ValueError(f"layer {li}: the rank of the decay projection is not known (complete_blocks)")
+            att[P + "w_left"], att[P + "w_right"] = attention(P, X + "left.", m.left), Pad(r(Y + "o", W, s.values))
+            att[P + "left_norm"], att[P + "right_norm"] = r(X + "left.out", W), r(X + "right.out", W)
+            att[P + "w2"], att[P + "w0"], att[P + "o_norm"] = r(Y + "w2", s.qk, s.rank), r(Y + "w0", s.qk), r(Y + "norm", s.values)
+            att[P + "a_bias"] = Keep32(r(Y + "a.b", s.qk))
         else:
             s = m.right
             left = attention(P, X + "left.", m.left)
@@ -868,11 +892,19 @@ def _block_tensors(cfg: ModelConfig, weights: dict) -> Dict[str, torch.Tensor]:
     t = {"embed": weights["embed"], "final.norm": weights["final_norm"]}
     if not cfg.tie_word_embeddings:
         t["head"] = weights["lm_head"][:cfg.vocab_size, :W]
+    if cfg.layer_norm:
+        t["final.norm.b"] = weights["final_norm_b"]
+    if cfg.token_pairs is not None:
+        t["bigram"] = weights["pairs"]
     for li, (lw, b) in enumerate(zip(weights["layers"], cfg.blocks)):
         L, X, F, m, f = f"l{li}.", f"l{li}.mix.", f"l{li}.mlp.", b.mixer, b.ff
         dt = lw["w_in"].dtype
         for h in ("1", "2") if f is not None else ("1",):
-            if cfg.post_norm:
+            if cfg.conv_taps:
+                t[L + "canon" + h] = lw["conv" + h]
+            if cfg.layer_norm:
+                t[L + "norm" + h], t[L + f"norm{h}.b"] = lw["ln" + h], lw[f"ln{h}_b"]
+            elif cfg.post_norm:
                 t[L + "norm" + h] = lw[f"ln{h}b"]
             else:
                 t[L + "norm" + h], t[L + f"norm{h}b"], t[L + "ls" + h] = lw["ln" + h], lw[f"ln{h}b"], lw["ls" + h]
@@ -880,7 +912,13 @@ def _block_tensors(cfg: ModelConfig, weights: dict) -> Dict[str, torch.Tensor]:
             t[X + n] = lw["w_in"][at:at + k, :W]
         a, side = b.attention, "left." if isinstance(m, ParallelSpec) else ""
         hv = a.heads * a.vdim if a is not None else 0
-        if a is not None:
+        if isinstance(a, PlainAttentionSpec):
+            t[X + side + "o"] = lw["w_left" if side else "w_out"][:W, :hv]
+            if a.head_norm:
+                t[X + side + "q.norm"], t[X + side + "k.norm"] = lw["q_norm"], lw["k_norm"]
+            if a.sink:
+                t[X + side + "sink"] = lw["sink"].to(dt)
+        elif a is not None:
             t[X + side + "q.norm"], t[X + side + "k.norm"], t[X + side + "o"] = lw["q_norm"], lw["k_norm"], lw["w_out"][:W, :hv]
             if isinstance(a, BiasedAttentionSpec):
                 t[X + side + "rel"] = lw["rel"].to(dt)
@@ -893,6 +931,10 @@ def _block_tensors(cfg: ModelConfig, weights: dict) -> Dict[str, torch.Tensor]:
         elif isinstance(m, LatentSpec):
             t[X + "dq.norm"], t[X + "dkv.norm"], t[X + "uq"] = lw["q_latent_norm"], lw["latent_norm"], lw["w_uq"][:m.q_rows, :m.q_rank]
             t[X + "uk"], t[X + "uv"], t[X + "o"] = lw["w_uk"], lw["w_uv"], lw["w_out"][:W, :m.heads * m.vdim]
+        elif isinstance(m, ParallelSpec) and isinstance(m.right, DeltaRuleSpec):
+            t[X + "left.out"], t[X + "right.out"], t[X + "right.norm"] = lw["left_norm"], lw["right_norm"], lw["o_norm"]
+            t[X + "right.w2"], t[X + "right.w0"], t[X + "right.a.b"] = lw["w2"], lw["w0"], lw["a_bias"].to(dt)
+            t[X + "right.o"] = lw["w_right"][:W, :m.right.values]
         elif isinstance(m, ParallelSpec):
             t[X + "right.norm"], t[X + "right.o"] = lw["o_norm"], lw["w_out"][:W, _pad(hv):_pad(hv) + m.right.values]
             if isinstance(m.right, MatrixMemorySpec):
@@ -927,7 +969,7 @@ def export_hf_checkpoint(cfg: ModelConfig, weights: dict, path) -> None:
         return
     if cfg.blocks is not None:
         save_file({k: v.contiguous().cpu() for k, v in _block_tensors(cfg, weights).items()}, str(p / "model.safetensors"))
-        (p / "config.json").write_text(json.dumps((nukelix_dict if cfg.model_type == "nukelix" else retodra_dict)(cfg)))
+        (p / "config.json").write_text(json.dumps({"nukelix": nukelix_dict, "vulanex": vulanex_dict}.get(cfg.model_type, retodra_dict)(cfg)))
         return
     d, hq, hkv = cfg.head_dim, cfg.num_attention_heads, cfg.num_key_value_heads
     ungain = (lambda g: g.float() - 1.0) if cfg.norm_plus_one else (lambda g: g)      # Gemma stores (gain - 1)

@@ -1,7 +1,8 @@
 """Blocks over a 32-bit residual stream whose layers are described one by one, each with a mixer and a dense or expert
 feed-forward of its own. Sandwich-normed (Retodra): x += ls1 * norm1b(mixer(norm1(x))), then the same with the feed-forward,
 mixers gated linear attention, or windowed attention with a distance bias beside lightning attention. Normed on the way out
-only (Nukelix): x += norm1(mixer(x)), mixers in `mixers.py`.
+only (Nukelix): x += norm1(mixer(x)), mixers in `mixers.py`. Read through a layer norm and a convolution (Vulanex): x +=
+mixer(conv(norm1(x))), whose sublayers end in a product that accumulates into the stream.
 
 Output norm, layer scale, residual sum and the next input norm are one pass over the stream (`ResidualStream`); the
 projections of a mixer are one GEMM, also those of two mixers side by side, whose output projections are one GEMM over
@@ -11,7 +12,7 @@ from __future__ import annotations
 
 import torch
 
-from ..ops import latent as lops, linear as lin, linear_reference as lref
+from ..ops import latent as lops, linear as lin, linear_reference as lref, stream_conv as conv
 from .block_spec import BiasedAttentionSpec, ExpertsSpec, GatedLinearSpec, projection_columns
 from .config import _pad
 from .mixers import mixer_of, prepare_mixer
@@ -29,8 +30,17 @@ def prepare_blocks(m) -> None:
         m.w["lm_head"] = m.w["embed"]                   # tied and unpadded: one copy
     gain = lambda w: (1.0 + w.float() if cfg.norm_plus_one else w.float()).contiguous()
     m.final_gain = gain(m.w["final_norm"])
+    if cfg.layer_norm:              # the factor on the logits goes into the norm ahead of their product
+        m.final_gain, m.final_offset = m.final_gain * cfg.logit_scale, m.w["final_norm_b"].float() * cfg.logit_scale
     for b, lw in zip(cfg.blocks, m.w["layers"]):
         for h in ("1", "2") if b.ff is not None else ("1",):
+            if cfg.layer_norm:
+                lw["gain" + h], lw["offset" + h] = lw["ln" + h].float().contiguous(), lw[f"ln{h}_b"].float().contiguous()
+                if cfg.conv_taps:   # [taps, width], the input itself counted in
+                    taps = lw["conv" + h].float().t().contiguous()
+                    taps[-1] += 1.0
+                    lw["taps" + h] = taps
+                continue
             lw[f"gain{h}b"] = gain(lw[f"ln{h}b"])
             if not cfg.post_norm:
                 lw["gain" + h] = gain(lw["ln" + h])
@@ -92,6 +102,12 @@ def expert_ff(m, h, lw: dict, spec: ExpertsSpec) -> torch.Tensor:
 def block(m, st, lw: dict, li: int, fi, cache) -> None:
     cfg = m.cfg
     b = cfg.blocks[li]
+    if cfg.layer_norm:
+        mixer_of(b)(m, st.convolved(cfg, lw, "1", li, fi.rs, m.dtype), lw, li, fi, cache, st)
+        if b.ff is not None:
+            h = st.convolved(cfg, lw, "2", li, fi.rs, m.dtype)
+            st.add_product(m._gemm(h, lw["w_gate_up"], glu=b.ff.act), lw["w_down"])
+        return
     read = lambda half: st.plain(cfg, m.dtype) if cfg.post_norm else st.normed(cfg, lw["gain" + half], m.dtype)
     mixer = mixer_of(b) or (gla_mixer if isinstance(b.mixer, GatedLinearSpec) else parallel_mixer)
     st.y = mixer(m, read("1"), lw, li, fi, cache, st)
@@ -108,4 +124,6 @@ def block(m, st, lw: dict, li: int, fi, cache) -> None:
 
 def final_rows(m, rows) -> torch.Tensor:
     """The model's norm on the rows that need logits."""
+    if m.cfg.layer_norm:
+        return conv.conv_norm(rows, m.cfg.hidden_size, m.cfg.rms_norm_eps, w=m.final_gain, b=m.final_offset, dtype=m.dtype)[1]
     return lops.stream_norm(rows, m.cfg.hidden_size, m.cfg.rms_norm_eps, norm_w=m.final_gain, dtype=m.dtype)[1]

@@ -2,7 +2,9 @@
 norm reads the stream, and both run in one pass."""
 from __future__ import annotations
 
-from ..ops import latent as lops
+import torch
+
+from ..ops import latent as lops, stream_conv as conv
 from .config import ModelConfig
 
 
@@ -11,10 +13,14 @@ class ResidualStream:
 
     def __init__(self, x):
         self.x, self.y, self.y_norm = x, None, None
+        self.pair = ()              # (sublayer output, gain) pairs, each to be normed and added
         self.values = None          # values of the first layer that mixes them (32-bit, one row per token)
 
     def finish(self, cfg: ModelConfig):
         """The stream with everything pending added."""
+        if self.pair:
+            self.x, _ = conv.conv_norm(self.x, cfg.hidden_size, cfg.rms_norm_eps, self.pair)
+            self.pair = ()
         if self.y is not None:
             self.x, _, _ = lops.stream_norm(self.x, cfg.hidden_size, cfg.rms_norm_eps, self.y, self.y_norm, dtype=self.y.dtype)
             self.y = self.y_norm = None
@@ -31,3 +37,18 @@ class ResidualStream:
         self.x, h, _ = lops.stream_norm(self.x, cfg.hidden_size, cfg.rms_norm_eps, self.y, self.y_norm, dtype=dtype, copy=True)
         self.y = self.y_norm = None
         return h
+
+    def convolved(self, cfg: ModelConfig, lw: dict, half: str, li: int, rs, dtype):
+        """Add what is pending, then the layer norm and the convolution ahead of a sublayer, in `dtype`."""
+        history = rs.history_of(li, half) if cfg.conv_taps > 1 else None
+        self.x, h = conv.conv_norm(self.x, cfg.hidden_size, cfg.rms_norm_eps, self.pair, lw["gain" + half], lw["offset" + half],
+                                   lw.get("taps" + half), history, rs, dtype)
+        self.pair = ()
+        return h
+
+    def add_product(self, a, w):
+        """x += a @ w.T, accumulated in 32-bit (bf16 on the device: in the product's epilogue)."""
+        if a.is_cuda and a.dtype == torch.bfloat16:
+            lops.gemm_stream(a, w, None, self.x)
+        else:
+            self.x = self.x + torch.matmul(a, w.t()).float()

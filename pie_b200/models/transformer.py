@@ -20,7 +20,7 @@ from typing import Optional
 import torch
 
 from .. import ops
-from ..ops import latent as lops, reference
+from ..ops import latent as lops, reference, stream_conv as conv
 from ..driver.lora import apply_lora
 from .config import ModelConfig, _pad
 from . import latent, sandwich
@@ -85,7 +85,9 @@ class Transformer:
         return ops.prefill_tile_rows(self.hq, self.hkv, self.cfg.head_dim, page_size, softcap=bool(self.cfg.attn_softcap))
 
     # ------------------------------------------------------------------ linear algebra
-    def _gemm(self, x, w, residual=None, swiglu=False):
+    def _gemm(self, x, w, residual=None, swiglu=False, glu: str = ""):
+        """x @ w.T, + residual, or a GLU over interleaved gate / up columns (`swiglu`, or `glu` naming the gate's activation)."""
+        swiglu = swiglu or glu == "silu"
         if isinstance(w, ops.Fp8Linear):
             epi = ops.EPI_SWIGLU if swiglu else (ops.EPI_RESIDUAL if residual is not None else ops.EPI_STORE)
             if self.gemm_backend == "tcgen05" or not x.is_cuda:
@@ -93,11 +95,14 @@ class Transformer:
             w = w.dequant(x.dtype)      # library path: expand, then cuBLAS (the reference's scheme)
         if self.gemm_backend == "tcgen05" and x.dtype == torch.bfloat16:
             epi = ops.EPI_SWIGLU if swiglu else (ops.EPI_RESIDUAL if residual is not None else ops.EPI_STORE)
+            epi = ops.EPI_GEGLU if glu == "gelu_tanh" else epi
             return ops.gemm(x, w, residual=residual, epilogue=epi)
         # library path (cuBLAS through torch): the baseline the tcgen05 kernel is measured against
         y = torch.matmul(x, w.t())
         if swiglu:
             return reference.swiglu_interleaved(y) if not y.is_cuda else _swiglu_interleaved_cuda(y)
+        if glu:
+            return ops.glu_interleaved(y, glu)
         if residual is not None:
             y = y + residual
         return y
@@ -201,7 +206,9 @@ class Transformer:
         if self._fused_tp():
             return self._forward_hidden_tp(fi, kv_cache)
         cfg, w = self.cfg, self.w
-        if cfg.stream32:
+        if cfg.token_pairs is not None:
+            h = conv.pair_embed(fi.tokens, w["embed"], w["pairs"], cfg.token_pairs, _pad(cfg.hidden_size), fi.rs)
+        elif cfg.stream32:
             h = lops.stream_embed(fi.tokens, w["embed"], _pad(cfg.hidden_size), cfg.embed_scale)
         elif self.par.tp_size > 1 and w.get("embed_sharded", False):
             h = ops.embed(fi.tokens, w["embed"], vocab_start=w["embed_vocab_start"])

@@ -12,7 +12,7 @@ Runtime layout per layer (this rank's shard under tensor parallelism):
   Gemma-2/3 (sandwich norms): ln1 / ln2 before attention / MLP, ln_pa / ln_pf on their outputs before the
   residual add; gains hold the full multiplier (the loader adds the checkpoint's implicit 1)
   Puzutar (latent attention in parallel blocks): see `loader._compile_latent`
-  Retodra, Nukelix (layers described one by one): see `loader._compile_blocks`
+  Retodra, Nukelix, Vulanex (layers described one by one): see `loader._compile_blocks`
 MoE layers replace w_gate_up / w_down by router [E, H], experts_gate_up [E_local, 2*Im, H]
 (interleaved) and experts_down [E_local, H, Im].
 
@@ -247,7 +247,8 @@ def _random_latent(cfg: ModelConfig, gen: _Gen, tp_size: int) -> dict:
 def _random_blocks(cfg: ModelConfig, gen: _Gen, tp_size: int) -> dict:
     """Random checkpoint tensors of layers described one by one, brought into the runtime layout by the loader. Gains are
     drawn as their distance from one where the checkpoint stores that (`norm_plus_one`)."""
-    from .block_spec import (BiasedAttentionSpec, DenseSpec, GatedLinearSpec, LatentSpec, MatrixMemorySpec, ParallelSpec, projection_sizes)
+    from .block_spec import (BiasedAttentionSpec, DeltaRuleSpec, DenseSpec, GatedLinearSpec, LatentSpec, MatrixMemorySpec, ParallelSpec,
+                             PlainAttentionSpec, projection_sizes)
     from .loader import TensorDictReader, compile_program, execute_program
     W = cfg.hidden_size
     near = lambda n: gen.normal(n, std=0.1)
@@ -255,18 +256,32 @@ def _random_blocks(cfg: ModelConfig, gen: _Gen, tp_size: int) -> dict:
     t = {"embed": gen.normal(cfg.vocab_size, W, **({"std": 1.0} if cfg.post_norm else {})), "final.norm": gain(W)}
     if not cfg.tie_word_embeddings:
         t["head"] = gen.normal(cfg.vocab_size, W)
+    if cfg.layer_norm:
+        t["final.norm.b"] = near(W)
+    if cfg.token_pairs is not None:
+        t["bigram"] = gen.normal(cfg.token_pairs.buckets + 1, W)
     for li, b in enumerate(cfg.blocks):
         L, X, F, m, f = f"l{li}.", f"l{li}.mix.", f"l{li}.mlp.", b.mixer, b.ff
         for h in ("1", "2") if f is not None else ("1",):
             t[L + "norm" + h] = gain(W)
-            if not cfg.post_norm:
+            if cfg.conv_taps:
+                t[L + "canon" + h] = gen.normal(W, cfg.conv_taps, std=0.2)
+            if cfg.layer_norm:
+                t[L + f"norm{h}.b"] = near(W)
+            elif not cfg.post_norm:
                 t[L + f"norm{h}b"], t[L + "ls" + h] = gain(W), 0.3 + near(W)
-        if isinstance(m, GatedLinearSpec):
-            m.rank = m.rank or 16
+        if isinstance(b.recurrent, (GatedLinearSpec, DeltaRuleSpec)):
+            b.recurrent.rank = b.recurrent.rank or 16
         for n, k in projection_sizes(m).items():
             t[X + n] = gen.normal(k, W)
         a, A = b.attention, X + ("left." if isinstance(m, ParallelSpec) else "")
-        if a is not None:
+        if isinstance(a, PlainAttentionSpec):
+            t[A + "o"] = gen.normal(W, a.heads * a.vdim)
+            if a.head_norm:
+                t[A + "q.norm"], t[A + "k.norm"] = 1 + near(a.dim), 1 + near(a.dim)
+            if a.sink:
+                t[A + "sink"] = gen.normal(a.heads, std=1.0)
+        elif a is not None:
             nq, nk, nv = a.heads * a.dim, a.kv_heads * a.dim, a.kv_heads * a.vdim
             t[A + "q.norm"], t[A + "k.norm"], t[A + "o"] = 1 + near(nq), 1 + near(nk), gen.normal(W, a.heads * a.vdim)
             if isinstance(a, BiasedAttentionSpec):
@@ -288,6 +303,10 @@ def _random_blocks(cfg: ModelConfig, gen: _Gen, tp_size: int) -> dict:
         elif isinstance(m, ParallelSpec):
             s = m.right
             t[X + "right.norm"], t[X + "right.o"] = 1 + near(s.values), gen.normal(W, s.values)
+            if isinstance(s, DeltaRuleSpec):
+                t[X + "left.out"], t[X + "right.out"] = 1 + near(W), 1 + near(W)
+                t[X + "right.w2"], t[X + "right.w0"] = gen.normal(s.qk, s.rank, std=s.rank ** -0.5), gen.normal(s.qk, std=1.0)
+                t[X + "right.a.b"] = gen.normal(s.qk, std=1.0)
             if isinstance(s, MatrixMemorySpec):
                 t[X + "right.i"], t[X + "right.f"] = gen.normal(s.heads, W, std=W ** -0.5), gen.normal(s.heads, W, std=W ** -0.5)
                 t[X + "right.i.b"], t[X + "right.f.b"] = near(s.heads), 3 + gen.normal(s.heads, std=1.0)

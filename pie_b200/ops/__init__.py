@@ -17,7 +17,7 @@ import torch
 from . import _lib, reference
 from ._lib import check, fn, ptr, stream_ptr
 
-EPI_STORE, EPI_RESIDUAL, EPI_SWIGLU = 0, 1, 2
+EPI_STORE, EPI_RESIDUAL, EPI_SWIGLU, EPI_GEGLU = 0, 1, 2, 7
 
 _NUM_SMS = {}
 
@@ -310,13 +310,15 @@ def set_gemm_pairs(enabled: bool) -> None:
 
 
 def gemm(x, w, residual=None, epilogue: int = EPI_STORE, out=None, force_bn: int = 0):
-    """y = x @ w.T (+ residual | SwiGLU over interleaved gate/up columns). x [M,K], w [N,K]."""
+    """y = x @ w.T (+ residual | SwiGLU or GeGLU over interleaved gate/up columns). x [M,K], w [N,K]."""
     if not x.is_cuda:
         y = reference.gemm(x, w, residual if epilogue == EPI_RESIDUAL else None)
+        if epilogue == EPI_GEGLU:
+            return reference.glu_interleaved(y, "gelu_tanh")
         return reference.swiglu_interleaved(y) if epilogue == EPI_SWIGLU else y
     m, k = x.shape
     n = w.shape[0]
-    n_out = n // 2 if epilogue == EPI_SWIGLU else n
+    n_out = n // 2 if epilogue in (EPI_SWIGLU, EPI_GEGLU) else n
     if out is None:
         out = torch.empty(m, n_out, dtype=x.dtype, device=x.device)
     if m == 0:

@@ -90,7 +90,16 @@ _SIGNATURES = {
     "pie_linear_attn_chunk_supported": [i32],
     "pie_linear_attn_chunk_tokens": [],
     "pie_linear_attn_chunked": [p, p],
-    "pie_linear_decay": [p, i32, p, p, p, i32, i32, i32, f32, i32, p],
+    "pie_linear_decay": [p, i32, p, p, p, i32, i32, i32, f32, i32, i32, p],
+    "pie_pair_embed": [p, i32, i32, p],
+    "pie_conv_norm": [p, i32, i32, p],
+    "pie_delta_step": [p, i32, p],
+    "pie_delta_portions": [p, i32, p],
+    "pie_head_rows": [p, i32, p],
+    "pie_pool_rows": [p, i32, p],
+    "pie_pool_gather": [p, p],
+    "pie_laid_decode": [p, p],
+    "pie_laid_prefill": [p, i32, p, p],
     "pie_gated_norm": [p, i32, i32, p],
     "pie_biased_rows": [p, i32, p],
     "pie_biased_any": [p, i32, p],

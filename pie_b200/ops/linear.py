@@ -47,7 +47,7 @@ def decay_logs(x, a2, bias, tau: float):
         return ref.decay_logs(x, a2, bias, tau)
     n, rank = x.shape
     out = torch.empty(n, a2.shape[0], dtype=torch.float32, device=x.device)
-    check(fn("pie_linear_decay")(ptr(x), x.stride(0), ptr(a2), ptr(bias), ptr(out), n, a2.shape[0], rank, 1.0 / tau, _f32(x), stream_ptr()),
+    check(fn("pie_linear_decay")(ptr(x), x.stride(0), ptr(a2), ptr(bias), ptr(out), n, a2.shape[0], rank, 1.0 / tau, 0, _f32(x), stream_ptr()),
           "linear_decay")
     return out
 

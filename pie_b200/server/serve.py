@@ -186,7 +186,7 @@ def _build_drivers_direct(m: ModelSection):
         dev = torch.device("cuda", g[0])
         if m.path:
             _, weights = loader.load_checkpoint(m.path, dev)
-        per_page = cfg.kv_elems_per_token * d.kv_page_size * 2
+        per_page = cfg.kv_elems_per_page(d.kv_page_size) * 2
         swap = int(d.swap_pool_gb * (1 << 30) // per_page)
         drivers.append(TorchDriver(cfg, dev, weights=weights, page_size=d.kv_page_size, gemm_backend=d.gemm,
                                    use_graphs=d.cuda_graphs, gpu_mem_utilization=d.gpu_mem_utilization,

@@ -325,7 +325,7 @@ def test_bytes_of_pages_and_slots():
     from pie_b200.driver.recurrent import RecurrentStateCache
     cfg = ModelConfig.from_hf(nm.CONFIGS["mixed"])
     assert mp.kv_bytes_per_page(cfg, 16) == 2 * 16 * (2 * 64 * (2 + 2 + 2 + 4 + 4) + 64)
-    kv = KVCache(0, 4, 1, 16, 64, torch.float32, "cpu", layer_shapes=cfg.kv_layers)
+    kv = KVCache(0, 4, 1, 16, 64, torch.float32, "cpu", layer_shapes=cfg.kv_page_shapes(16))
     assert kv.data[2].shape == (5, 16, 64) and kv.data[4].shape == (5, 2, 4, 16, 64)
     assert kv.page_bytes_all_layers == 2 * mp.kv_bytes_per_page(cfg, 16)
     rs = RecurrentStateCache(cfg, 3, "cpu")

@@ -194,7 +194,7 @@ def test_configuration_and_registry(tmp_path):
     cfg = ModelConfig.from_hf(pm.CONFIGS["odd"])
     assert cfg.model_type == "puzutar" and cfg.ff_sizes == [70, 0, 21] and cfg.latent_cache_layers == [0, 1]
     assert cfg.latent_cache_index == {0: 0, 1: 1, 2: 0} and cfg.plan_window_left == 199 and cfg.recurrent_layers == [0, 1, 2]
-    assert cfg.kv_elems_per_token == 2 * cfg.latent_row
+    assert cfg.kv_elems_per_page(1) == 2 * cfg.latent_row
     bad = json.loads(json.dumps(pm.CONFIGS["shared"]))
     bad["layers"][1]["mixer"]["kv_rank"] = 24
     with pytest.raises(ValueError, match="kv_from"):

@@ -231,7 +231,7 @@ def test_configuration_and_registry():
     assert cfg.kv_layers == [(2, 64), (4, 64)] and cfg.plan_window_left == 69 and cfg.layer_window_left(1) == 36
     assert cfg.blocks[1].attention.group_pad == 4 and isinstance(cfg.blocks[1].ff, ExpertsSpec) and cfg.blocks[1].ff.outputs == 8
     assert ModelConfig.from_hf(rm.CONFIGS["odd"]).blocks[2].ff is None
-    assert ModelConfig.from_hf(rm.CONFIGS["linear"]).kv_elems_per_token == 0
+    assert ModelConfig.from_hf(rm.CONFIGS["linear"]).kv_elems_per_page(16) == 0
     for change in (lambda c: c["layers"][0].update(type="other"), lambda c: c["layers"][0]["mlp"].update(kind="other"),
                    lambda c: c["layers"][1]["mixer"]["left"].update(kv_heads=4), lambda c: c["layers"][1]["mixer"]["right"].update(decay=[0.5]),
                    lambda c: c["layers"][1]["mlp"]["router"].update(top=9), lambda c: c["layers"][1]["mixer"]["left"]["mask"].update(size=0)):
@@ -342,7 +342,7 @@ def test_bytes_of_pages_and_slots():
 def test_swap_copies_pages_of_unequal_layers():
     from pie_b200.driver.kv_cache import KVCache
     from pie_b200.driver.schema import CopyDir, CopyRequest
-    kv = KVCache(0, 4, 1, 16, 64, torch.float32, "cpu", swap_pages=2, layer_shapes=[(2, 64), (4, 128)])
+    kv = KVCache(0, 4, 1, 16, 64, torch.float32, "cpu", swap_pages=2, layer_shapes=[((2, 2, 16, 64), None), ((2, 4, 16, 128), None)])
     for i, t in enumerate(kv.parts):
         t[:, 1] = 7.0 + i
     assert kv.page_bytes_all_layers == 2 * 16 * (2 * 64 + 4 * 128) * 4
