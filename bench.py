@@ -38,12 +38,13 @@ def parse_args():
     ap.add_argument("--gpus", type=int, default=1)
     ap.add_argument("--steps", type=int, default=64)
     ap.add_argument("--warmup", type=int, default=8)
-    ap.add_argument("--config", type=int, default=2, choices=[2, 3, 4, 5, 6, 7, 8, 9],
+    ap.add_argument("--config", type=int, default=2, choices=[2, 3, 4, 5, 6, 7, 8, 9, 10],
                     help="2: the headline configuration (this file); 3 Qwen3-32B block-fp8, 4 Qwen3-30B-A3B MoE with "
                          "expert parallelism, 5 agentic fork, 6 GPT-OSS shapes: see pie_b200/bench/configs.py; 7 the Puzutar "
                          "design beside the Llama-8B shape with a sliding window; 8 the Retodra design beside "
                          "Gated DeltaNet with windowed attention and experts; 9 the Nukelix design beside Retodra's parallel "
-                         "mixers with experts: see pie_b200/bench/pair_bench.py")
+                         "mixers with experts; 10 the Vulanex design beside Gated DeltaNet and attention: see "
+                         "pie_b200/bench/pair_bench.py")
     ap.add_argument("--impl", default="ours", choices=["ours", "reference", "library", "vllm"])
     ap.add_argument("--no-baseline", action="store_true", help="skip the library comparator (vs_baseline stays null)")
     ap.add_argument("--model", default="llama-3.1-8b")
@@ -89,7 +90,7 @@ def main():
         return 0
     from pie_b200.bench import configs as _configs
     _configs._hang_dump()
-    if args.config in (7, 8, 9):
+    if args.config in (7, 8, 9, 10):
         from pie_b200.bench import pair_bench
         return pair_bench.main(["--config", str(args.config), "--steps", str(args.steps), "--warmup", str(args.warmup), "--layers", str(args.layers)])
     if args.config != 2:

@@ -3,9 +3,11 @@
     python bench.py --config 7 [--layers 32]    Puzutar beside the Llama-8B shape with a sliding window
     python bench.py --config 8 [--layers 32]    Retodra beside Gated DeltaNet and windowed attention with experts
     python bench.py --config 9 [--layers 24]    Nukelix beside Retodra's parallel mixers with experts
+    python bench.py --config 10 [--layers 32]   Vulanex beside Gated DeltaNet and attention
 
 Both models of a pair have the same width, heads, window, vocabulary and feed-forward sizes (configs 8 and 9: also the same
-states of the linear mixers, experts and routes per token; a shared expert counts as a route). Device-timed with CUDA
+states of the linear mixers, experts and routes per token; a shared expert counts as a route; config 10: the same states, and
+feed-forwards that make up for the parameters of a second mixer). Device-timed with CUDA
 events after warm-up. Decode replays the captured step over contexts of `--context` tokens; the weights read per step
 exceed the L2. Prefill runs whole prompts as one batch. One JSON line.
 """
@@ -18,7 +20,7 @@ import json
 import numpy as np
 
 PAIRS = {7: ("puzutar-8b", "llama-8b-window"), 8: ("retodra-19b", "gdn-moe-window-19b"),
-         9: ("nukelix-20b", "retodra-parallel-20b")}
+         9: ("nukelix-20b", "retodra-parallel-20b"), 10: ("vulanex-8b", "gdn-8b")}
 DECODE_ROWS = (16, 64, 256)
 PREFILL = ((1, 2048), (4, 2048), (1, 8192))
 

@@ -191,35 +191,24 @@ __global__ void __launch_bounds__(256) head_rows_kernel(const HeadRowsArgs a) {
     }
     __syncthreads();
     const float temp = a.temp_every ? 1.f + a.temp_coef * logf((float)((pos + 1) / a.temp_every) + 1.f) : 1.f;
+    const bool pairs_of_vecs = VEC == 4 && half % 4 == 0;
     auto emit = [&](T* dst, const T* src, int n, const float* norm, bool turn, float scale) {       // src null: zeros
-        float inv = 1.f;
-        if (src && norm) {
-            float ss = 0.f;
-            for (int d = lane * VEC; d < n; d += 32 * VEC) {
-                float f[VEC];
-                load_vec<VEC>(src + d, f);
-#pragma unroll
-                for (int e = 0; e < VEC; ++e) ss += f[e] * f[e];
-            }
-            inv = 1.f / sqrtf(warp_sum(ss) / (float)n + a.eps);
-        }
-        turn = turn && src && half > 0;
-        auto value = [&](int d, float (&f)[VEC]) {
-            load_vec<VEC>(src + d, f);
-            if (norm) {
-                float g[VEC];
-                load_vec<VEC>(norm + d, g);
-#pragma unroll
-                for (int e = 0; e < VEC; ++e) f[e] *= inv * g[e];
-            }
-        };
-        if (turn) {
+        float ss = 0.f;
+        turn = turn && half > 0;
+        if (src && (norm || turn)) {
             __syncwarp();
             for (int d = lane * VEC; d < n; d += 32 * VEC) {
-                float f[VEC];
-                value(d, f);
+                float f[VEC], g[VEC];
+                load_vec<VEC>(src + d, f);
+                if (norm) load_vec<VEC>(norm + d, g);
+#pragma unroll
+                for (int e = 0; e < VEC; ++e) {
+                    ss += f[e] * f[e];
+                    if (norm) f[e] *= g[e];
+                }
                 store_vec<VEC>(row + d, f);
             }
+            if (norm) scale *= 1.f / sqrtf(warp_sum(ss) / (float)n + a.eps);
             __syncwarp();
         }
         for (int d = lane * VEC; d < a.D; d += 32 * VEC) {
@@ -227,15 +216,23 @@ __global__ void __launch_bounds__(256) head_rows_kernel(const HeadRowsArgs a) {
 #pragma unroll
             for (int e = 0; e < VEC; ++e) f[e] = 0.f;
             if (src && d < n) {
-                if (turn) {
+                if (!norm && !turn) load_vec<VEC>(src + d, f);
+                else load_vec<VEC>(row + d, f);
+                if (turn && d < a.rot_dims && pairs_of_vecs) {
+                    const bool lower = d < half;
+                    const int p = lower ? d : d - half;
+                    float o[VEC], c[VEC], sn[VEC];
+                    load_vec<VEC>(row + (lower ? d + half : p), o);
+                    load_vec<VEC>(cs + p, c);
+                    load_vec<VEC>(cs + half + p, sn);
+#pragma unroll
+                    for (int e = 0; e < VEC; ++e) f[e] = f[e] * c[e] + (lower ? -o[e] : o[e]) * sn[e];
+                } else if (turn) {
 #pragma unroll
                     for (int e = 0; e < VEC; ++e) {
                         const int i = d + e, p = i < half ? i : i - half;
-                        f[e] = row[i];
                         if (i < a.rot_dims) f[e] = f[e] * cs[p] + (i < half ? -row[i + half] : row[p]) * cs[half + p];
                     }
-                } else {
-                    value(d, f);
                 }
 #pragma unroll
                 for (int e = 0; e < VEC; ++e) f[e] *= scale;

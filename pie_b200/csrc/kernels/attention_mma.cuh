@@ -237,7 +237,8 @@ __device__ __forceinline__ int mean_row(int b, int pool, int page_size, int& pag
 
 // POOL: an item of a request takes its share of the 16-key tiles (means, then the window's tokens) whatever range the plan
 // gave it, so that any plan spreads the work evenly.
-template <int D, int G, bool CASCADE, int MODE = MODE_PLAIN, bool POOL = false>
+// OWN: the values are the keys (planes 1); a stage then holds one tile, and there are twice as many.
+template <int D, int G, bool CASCADE, int MODE = MODE_PLAIN, bool POOL = false, bool OWN = false>
 __global__ void __launch_bounds__(DEC_WARPS * 32)
 paged_decode_attn_kernel(const bf16* __restrict__ q, const bf16* __restrict__ kv_layer,
                          const int* __restrict__ page_indices,
@@ -256,6 +257,7 @@ paged_decode_attn_kernel(const bf16* __restrict__ q, const bf16* __restrict__ kv
     extern __shared__ __align__(1024) uint8_t smem[];
     constexpr int CH = D / 8;              // 16-byte chunks per row
     constexpr int TILE_BYTES = 16 * D * 2; // one 16-token K or V tile
+    constexpr int STAGES = OWN ? 2 * DEC_STAGES : DEC_STAGES, STAGE_BYTES = (OWN ? 1 : 2) * TILE_BYTES;
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     const uint32_t q_smem = smem_u32(smem);
     const uint32_t warp_smem = q_smem + TILE_BYTES + warp * DEC_STAGES * 2 * TILE_BYTES;
@@ -338,7 +340,7 @@ paged_decode_attn_kernel(const bf16* __restrict__ q, const bf16* __restrict__ kv
                     const int row = mean_row(b, kl.pool, page_size, pg);
                     at = ((((long)pages[pg] * 2) * hkv + h) * kl.per_page + row) * D;
                 }
-                const uint32_t kdst = warp_smem + (j % DEC_STAGES) * 2 * TILE_BYTES;
+                const uint32_t kdst = warp_smem + (j % STAGES) * STAGE_BYTES;
 #pragma unroll
                 for (int i = 0; i < (16 * CH) / 32; ++i) {
                     const int c = lane + 32 * i, row = c / CH, col = c - row * CH;
@@ -356,27 +358,27 @@ paged_decode_attn_kernel(const bf16* __restrict__ q, const bf16* __restrict__ kv
             const int tok0 = block_start(warp + DEC_WARPS * j);
             const int page = pages[tok0 / page_size];
             const int off = tok0 % page_size;
-            const bf16* ksrc = kv_layer + ((((size_t)page * kl.planes) * hkv + h) * page_size + off) * D;
-            const bf16* vsrc = kl.planes == 2 ? ksrc + (size_t)hkv * page_size * D : nullptr;
-            const uint32_t kdst = warp_smem + (j % DEC_STAGES) * 2 * TILE_BYTES;
+            const bf16* ksrc = kv_layer + ((((size_t)page * (OWN ? 1 : 2)) * hkv + h) * page_size + off) * D;
+            const bf16* vsrc = ksrc + (size_t)hkv * page_size * D;
+            const uint32_t kdst = warp_smem + (j % STAGES) * STAGE_BYTES;
             const uint32_t vdst = kdst + TILE_BYTES;
 #pragma unroll
             for (int i = 0; i < (16 * CH) / 32; ++i) {
                 const int c = lane + 32 * i;
                 const int row = c / CH, col = c - row * CH;
                 cp_async16(kdst + swz<D>(row, col), ksrc + (size_t)c * 8);
-                if (vsrc) cp_async16(vdst + swz<D>(row, col), vsrc + (size_t)c * 8);
+                if (!OWN) cp_async16(vdst + swz<D>(row, col), vsrc + (size_t)c * 8);
             }
         };
 #pragma unroll
-        for (int s = 0; s < DEC_STAGES - 1; ++s) {
+        for (int s = 0; s < STAGES - 1; ++s) {
             if (s < my_count) issue(s);
             cp_async_commit();
         }
         for (int i = 0; i < my_count; ++i) {
-            if (i + DEC_STAGES - 1 < my_count) issue(i + DEC_STAGES - 1);
+            if (i + STAGES - 1 < my_count) issue(i + STAGES - 1);
             cp_async_commit();
-            cp_async_wait<DEC_STAGES - 1>();
+            cp_async_wait<STAGES - 1>();
             __syncwarp();
             const bool means = POOL && first_tile + warp + DEC_WARPS * i < mean_tiles;
             const int tok0 = means ? (first_tile + warp + DEC_WARPS * i) * 16 : block_start(warp + DEC_WARPS * i);
@@ -387,7 +389,7 @@ paged_decode_attn_kernel(const bf16* __restrict__ q, const bf16* __restrict__ kv
                 if (keep_first > tok0) see |= keep_first - tok0 >= 16 ? 0xffffu : (1u << (keep_first - tok0)) - 1u;
                 allow &= see;
             }
-            const uint32_t kt = warp_smem + (i % DEC_STAGES) * 2 * TILE_BYTES;
+            const uint32_t kt = warp_smem + (i % STAGES) * STAGE_BYTES;
             DistanceBias db{};
             if (MODE == MODE_BIAS) {
                 const int g = lane >> 2, n = item_end[req_item_indptr[req + 1] - 1] - 1 - tok0;
@@ -395,7 +397,7 @@ paged_decode_attn_kernel(const bf16* __restrict__ q, const bf16* __restrict__ kv
                 db = DistanceBias{tab + (g < G ? g : 0) * bias_pitch, tab + (g + 8 < G ? g + 8 : 0) * bias_pitch, n, n,
                                   bias_pitch - 2 * BIAS_GUARD - 1};
             }
-            attn_block16<D, MODE>(qf, kt, kl.planes == 1 ? kt : kt + TILE_BYTES, scale_log2, allow, allow, st, cap_log2, db);
+            attn_block16<D, MODE>(qf, kt, OWN ? kt : kt + TILE_BYTES, scale_log2, allow, allow, st, cap_log2, db);
             __syncwarp();
         }
         cp_async_wait<0>();

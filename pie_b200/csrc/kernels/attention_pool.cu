@@ -22,10 +22,9 @@ struct PoolArgs {
     int n, hkv, D, page_size, pool, per_page, total;
 };
 
-// One block per token; it works where the token ends a block of `pool` tokens. A warp takes 32 * VEC columns of one head's
-// keys or values.
+// One block per token; it works where the token ends a block of `pool` tokens.
 template <typename T, int VEC>
-__global__ void __launch_bounds__(128) pool_rows_kernel(const PoolArgs a) {
+__global__ void __launch_bounds__(256) pool_rows_kernel(const PoolArgs a) {
     pdl_trigger();
     pdl_wait();
     const int t = blockIdx.x;
@@ -38,16 +37,22 @@ __global__ void __launch_bounds__(128) pool_rows_kernel(const PoolArgs a) {
     const T* cache = static_cast<const T*>(a.cache);
     T* dst = static_cast<T*>(a.means) + (size_t)pages[page_at] * 2 * a.hkv * a.per_page * a.D;
     const int vecs = 2 * a.hkv * (a.D / VEC);
-    for (int i = threadIdx.x; i < vecs; i += 128) {
+    for (int i = threadIdx.x; i < vecs; i += 256) {
         const int head = i / (a.D / VEC), d = (i - head * (a.D / VEC)) * VEC;       // head: keys, then values
         float s[VEC];
 #pragma unroll
         for (int e = 0; e < VEC; ++e) s[e] = 0.f;
-        for (int j = pos + 1 - a.pool; j <= pos; ++j) {
-            float f[VEC];
-            load_vec<VEC>(cache + (((size_t)pages[j / a.page_size] * 2 * a.hkv + head) * a.page_size + j % a.page_size) * a.D + d, f);
+        for (int j0 = pos + 1 - a.pool; j0 <= pos; j0 += 8) {
+            float f[8][VEC];
 #pragma unroll
-            for (int e = 0; e < VEC; ++e) s[e] += f[e];
+            for (int u = 0; u < 8; ++u) {
+                const int j = min(j0 + u, pos);
+                load_vec<VEC>(cache + (((size_t)pages[j / a.page_size] * 2 * a.hkv + head) * a.page_size + j % a.page_size) * a.D + d, f[u]);
+            }
+#pragma unroll
+            for (int u = 0; u < 8; ++u)
+#pragma unroll
+                for (int e = 0; e < VEC; ++e) s[e] += j0 + u <= pos ? f[u][e] : 0.f;
         }
 #pragma unroll
         for (int e = 0; e < VEC; ++e) s[e] /= (float)a.pool;
@@ -106,7 +111,7 @@ PIE_API int pie_pool_rows(const PoolArgs* args, int f32, cudaStream_t st) {
     const bool vec = a.D % 4 == 0;
     auto kern = f32 ? (vec ? pool_rows_kernel<float, 4> : pool_rows_kernel<float, 1>)
                     : (vec ? pool_rows_kernel<bf16, 4> : pool_rows_kernel<bf16, 1>);
-    return (int)launch_pdl(kern, dim3(a.n), dim3(128), 0, st, a);
+    return (int)launch_pdl(kern, dim3(a.n), dim3(256), 0, st, a);
 }
 
 PIE_API int pie_pool_gather(const PoolArgs* args, cudaStream_t st) {
@@ -125,7 +130,8 @@ PIE_API int pie_laid_decode(const LaidAttnArgs* args, cudaStream_t st) {
     const KeyLayout kl{a.planes, a.pool, a.per_page, (const bf16*)a.means, nullptr};
     DISPATCH_DG(a.D, group, {
         constexpr int SM = decode_smem_bytes<D>();
-        auto kern = a.pool ? paged_decode_attn_kernel<D, G, false, MODE_PLAIN, true> : paged_decode_attn_kernel<D, G, false>;
+        auto kern = a.pool ? paged_decode_attn_kernel<D, G, false, MODE_PLAIN, true>
+                  : a.planes == 1 ? paged_decode_attn_kernel<D, G, false, MODE_PLAIN, false, true> : paged_decode_attn_kernel<D, G, false>;
         cudaError_t e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, SM);
         if (e == cudaSuccess)
             e = launch_pdl(kern, dim3(a.num_ctas), dim3(DEC_WARPS * 32), SM, st, (const bf16*)a.q, (const bf16*)a.kv, a.page_indices,

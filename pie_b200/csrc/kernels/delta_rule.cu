@@ -6,8 +6,8 @@
 // so that columns of the state never meet, and a column's rows once per token.
 //
 //   step       one token per request: a block holds 128 columns (VEC per lane) of a head, an eighth of the rows per warp
-//   portions   any lengths: a thread holds one column's rows, LPC lanes share a column; the tokens' vectors are prepared CT at
-//              a time in shared memory while the tokens before them run
+//   portions   any lengths: LPC lanes share CPT columns, each with R rows of them; a token's sums meet by halving (a lane ends up
+//              with one of them); the tokens' vectors are prepared CT at a time in shared memory while the tokens before run
 #include "typed.cuh"
 
 namespace pie {
@@ -123,45 +123,67 @@ __global__ void __launch_bounds__(256) delta_step_kernel(const DeltaArgs a) {
     }
 }
 
-template <int RPL, int LPC, int CT>
+constexpr int DELTA_WARPS = 4;
+constexpr int DELTA_CT = 8;                // tokens prepared at a time
+
+template <int R, int LPC, int CPT>
 struct DeltaSmem {
-    static constexpr int DP = RPL * LPC, COLS = 256 / LPC;
-    static constexpr int VECS = 5 * DP;                    // u, r * w, w, a * u, k of a token
-    float vec[2][CT][VECS];
-    float v[2][CT][COLS], o[2][CT][COLS];
-    float2 dots[2][CT];                                    // r . (a * u), r . k
+    static constexpr int DP = R * LPC, COLS = DELTA_WARPS * (32 / LPC) * CPT;
+    float vec[2][DELTA_CT][5 * DP];        // u, r * w, w, a * u, k of a token
+    float v[2][DELTA_CT][COLS], o[2][DELTA_CT][COLS];
+    float2 dots[2][DELTA_CT];              // r . (a * u), r . k
 };
 
-// Lane g of a column holds the rows 4 (g + LPC i) + e: a warp's 16-byte reads of a vector fall on consecutive addresses.
-template <typename T, int RPL, int LPC, int CT>
-__global__ void __launch_bounds__(256) delta_portion_kernel(const DeltaArgs a) {
-    using Smem = DeltaSmem<RPL, LPC, CT>;
-    constexpr int DP = Smem::DP, COLS = Smem::COLS, TPW = CT / 8, EPL = DP / 32, VPT = (CT * COLS + 255) / 256;
+// Sums of NV values over LPC lanes: halves change hands until a lane is left with one value (of index `which`, the lane's own
+// number in bits from the top); further lanes then add up copies of it.
+template <int NV, int LPC>
+__device__ __forceinline__ float halving_sum(float (&x)[NV], int g) {
+    if constexpr (NV == 1) {
+        float y = x[0];
+#pragma unroll
+        for (int o = LPC / 2; o; o >>= 1) y += __shfl_xor_sync(0xffffffffu, y, o);
+        return y;
+    } else {
+        const bool up = g & (LPC / 2);
+        float y[NV / 2];
+#pragma unroll
+        for (int i = 0; i < NV / 2; ++i) {
+            const float keep = up ? x[i + NV / 2] : x[i], give = up ? x[i] : x[i + NV / 2];
+            y[i] = keep + __shfl_xor_sync(0xffffffffu, give, LPC / 2);
+        }
+        return halving_sum<NV / 2, LPC / 2>(y, g);
+    }
+}
+
+// Lane g of a column group holds the rows 4 (g + LPC i) + e.
+template <typename T, int R, int LPC, int CPT>
+__global__ void __launch_bounds__(DELTA_WARPS * 32) delta_portion_kernel(const DeltaArgs a) {
+    using Smem = DeltaSmem<R, LPC, CPT>;
+    constexpr int THREADS = DELTA_WARPS * 32, CT = DELTA_CT, DP = Smem::DP, COLS = Smem::COLS, TPW = CT / DELTA_WARPS, EPL = DP / 32;
+    constexpr int VPT = (CT * COLS + THREADS - 1) / THREADS, NV = 2 * CPT;
+    static_assert(NV <= LPC && R % 4 == 0 && CPT % 2 == 0, "");
     extern __shared__ __align__(16) uint8_t raw[];
     Smem& sm = *reinterpret_cast<Smem*>(raw);
     const int q = blockIdx.x, h = blockIdx.y, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     const int first = a.qo_indptr[q], len = a.qo_indptr[q + 1] - first, slot = a.slots[q];
     if (len <= 0 || slot < 0) return;
-    const int g = lane % LPC, cl = warp * (32 / LPC) + lane / LPC, c = blockIdx.z * COLS + cl;
+    const int g = lane % LPC, cl = (warp * (32 / LPC) + lane / LPC) * CPT, c0 = blockIdx.z * COLS + cl;
     float* sp = a.state + (size_t)slot * a.slot_stride + (size_t)h * a.dim * a.dim;
     const bool fresh = a.reset[q] != 0;
-    F2 S[RPL / 2];
+    F2 S[CPT][R / 2];
 #pragma unroll
-    for (int i = 0; i < RPL / 4; ++i) {
-        float f[4];
+    for (int c = 0; c < CPT; ++c)
 #pragma unroll
-        for (int e = 0; e < 4; ++e) {
-            const int d = 4 * (g + LPC * i) + e;
-            f[e] = !fresh && c < a.dim && d < a.dim ? sp[(size_t)d * a.dim + c] : 0.f;
+        for (int i = 0; i < R / 2; ++i) {
+            const int d = 4 * (g + LPC * (i / 2)) + 2 * (i & 1);
+            const bool ok = !fresh && c0 + c < a.dim;
+            S[c][i] = f2(ok && d < a.dim ? sp[(size_t)d * a.dim + c0 + c] : 0.f, ok && d + 1 < a.dim ? sp[(size_t)(d + 1) * a.dim + c0 + c] : 0.f);
         }
-        S[2 * i] = f2(f[0], f[1]);
-        S[2 * i + 1] = f2(f[2], f[3]);
-    }
-    const T* R = static_cast<const T*>(a.r) + (size_t)first * a.ld + h * a.dim;
-    const T* K = static_cast<const T*>(a.k) + (size_t)first * a.ld + h * a.dim;
-    const T* V = static_cast<const T*>(a.v) + (size_t)first * a.ld + h * a.dim;
-    const T* A = static_cast<const T*>(a.a) + (size_t)first * a.ld + h * a.dim;
-    const float* W = a.log_decay + ((size_t)first * a.heads + h) * a.dim;
+    const T* Rp = static_cast<const T*>(a.r) + (size_t)first * a.ld + h * a.dim;
+    const T* Kp = static_cast<const T*>(a.k) + (size_t)first * a.ld + h * a.dim;
+    const T* Vp = static_cast<const T*>(a.v) + (size_t)first * a.ld + h * a.dim;
+    const T* Ap = static_cast<const T*>(a.a) + (size_t)first * a.ld + h * a.dim;
+    const float* Wp = a.log_decay + ((size_t)first * a.heads + h) * a.dim;
     float* O = a.out + ((size_t)first * a.heads + h) * a.dim;
     const size_t step = (size_t)a.heads * a.dim;
     float bias[EPL];
@@ -179,16 +201,16 @@ __global__ void __launch_bounds__(256) delta_portion_kernel(const DeltaArgs a) {
                 const int d = lane + 32 * i;
                 const bool ok = t < len && d < a.dim;
                 const size_t at = (size_t)t * a.ld + d;
-                pr[s][i] = ok ? R[at] : from_f<T>(0.f);
-                pk[s][i] = ok ? K[at] : from_f<T>(0.f);
-                pa[s][i] = ok ? A[at] : from_f<T>(0.f);
-                pw[s][i] = ok ? W[(size_t)t * step + d] : 0.f;
+                pr[s][i] = ok ? Rp[at] : from_f<T>(0.f);
+                pk[s][i] = ok ? Kp[at] : from_f<T>(0.f);
+                pa[s][i] = ok ? Ap[at] : from_f<T>(0.f);
+                pw[s][i] = ok ? Wp[(size_t)t * step + d] : 0.f;
             }
         }
 #pragma unroll
         for (int i = 0; i < VPT; ++i) {
-            const int x = threadIdx.x + i * 256, t = t0 + x / COLS, cc = blockIdx.z * COLS + x % COLS;
-            pv[i] = x < CT * COLS && t < len && cc < a.dim ? V[(size_t)t * a.ld + cc] : from_f<T>(0.f);
+            const int x = threadIdx.x + i * THREADS, t = t0 + x / COLS, cc = blockIdx.z * COLS + x % COLS;
+            pv[i] = x < CT * COLS && t < len && cc < a.dim ? Vp[(size_t)t * a.ld + cc] : from_f<T>(0.f);
         }
     };
     auto prepare = [&](int b) {
@@ -217,48 +239,65 @@ __global__ void __launch_bounds__(256) delta_portion_kernel(const DeltaArgs a) {
         }
 #pragma unroll
         for (int i = 0; i < VPT; ++i) {
-            const int x = threadIdx.x + i * 256;
+            const int x = threadIdx.x + i * THREADS;
             if (x < CT * COLS) sm.v[b][x / COLS][x % COLS] = to_f(pv[i]);
         }
     };
+    // the sum a lane ends up with: y of column `which`, or z of column `which - CPT`
+    constexpr int SPAN = LPC / NV;
+    const int which = g / SPAN, mine = which % CPT, base = lane - g;
     auto run = [&](int b, int count) {
         for (int t = 0; t < count; ++t) {
             const float4* p = reinterpret_cast<const float4*>(sm.vec[b][t]) + g;
-            F2 y0 = f2(0.f), y1 = y0, z0 = y0, z1 = y0;
+            F2 y[CPT], z[CPT];
 #pragma unroll
-            for (int i = 0; i < RPL / 4; ++i) {
+            for (int c = 0; c < CPT; ++c) y[c] = z[c] = f2(0.f);
+#pragma unroll
+            for (int i = 0; i < R / 4; ++i) {
                 const float4 u = p[LPC * i], rw = p[DP / 4 + LPC * i];
-                y0 = fma2(f2(u.x, u.y), S[2 * i], y0);
-                y1 = fma2(f2(u.z, u.w), S[2 * i + 1], y1);
-                z0 = fma2(f2(rw.x, rw.y), S[2 * i], z0);
-                z1 = fma2(f2(rw.z, rw.w), S[2 * i + 1], z1);
-            }
-            float a0, a1, a2, a3;
-            unpack2(y0, a0, a1);
-            unpack2(y1, a2, a3);
-            float y = (a0 + a1) + (a2 + a3);
-            unpack2(z0, a0, a1);
-            unpack2(z1, a2, a3);
-            float z = (a0 + a1) + (a2 + a3);
+                const F2 u0 = f2(u.x, u.y), u1 = f2(u.z, u.w), w0 = f2(rw.x, rw.y), w1 = f2(rw.z, rw.w);
 #pragma unroll
-            for (int o = 1; o < LPC; o <<= 1) {
-                y += __shfl_xor_sync(0xffffffffu, y, o);
-                z += __shfl_xor_sync(0xffffffffu, z, o);
+                for (int c = 0; c < CPT; ++c) {
+                    y[c] = fma2(u1, S[c][2 * i + 1], fma2(u0, S[c][2 * i], y[c]));
+                    z[c] = fma2(w1, S[c][2 * i + 1], fma2(w0, S[c][2 * i], z[c]));
+                }
             }
-            const float v = sm.v[b][t][cl];
-            const float2 dots = sm.dots[b][t];
-            if (g == 0) sm.o[b][t][cl] = z - dots.x * y + dots.y * v;
-            const F2 ny = f2(-y), vv = f2(v);
+            float x[NV];
 #pragma unroll
-            for (int i = 0; i < RPL / 4; ++i) {
+            for (int c = 0; c < CPT; ++c) {
+                float lo, hi;
+                unpack2(y[c], lo, hi);
+                x[c] = lo + hi;
+                unpack2(z[c], lo, hi);
+                x[CPT + c] = lo + hi;
+            }
+            const float sum = halving_sum<NV, LPC>(x, g);
+            float v[CPT], gone[CPT], my_v = 0.f, my_y = 0.f;
+#pragma unroll
+            for (int c = 0; c < CPT; ++c) {
+                v[c] = sm.v[b][t][cl + c];
+                gone[c] = __shfl_sync(0xffffffffu, sum, base + c * SPAN);
+                if (c == mine) { my_v = v[c]; my_y = gone[c]; }
+            }
+            if (which >= CPT && g % SPAN == 0) {
+                const float2 dots = sm.dots[b][t];
+                sm.o[b][t][cl + mine] = sum - dots.x * my_y + dots.y * my_v;
+            }
+#pragma unroll
+            for (int i = 0; i < R / 4; ++i) {
                 const float4 w = p[2 * DP / 4 + LPC * i], au = p[3 * DP / 4 + LPC * i], k = p[4 * DP / 4 + LPC * i];
-                S[2 * i] = fma2(f2(au.x, au.y), ny, fma2(f2(w.x, w.y), S[2 * i], mul2(f2(k.x, k.y), vv)));
-                S[2 * i + 1] = fma2(f2(au.z, au.w), ny, fma2(f2(w.z, w.w), S[2 * i + 1], mul2(f2(k.z, k.w), vv)));
+                const F2 w0 = f2(w.x, w.y), w1 = f2(w.z, w.w), a0 = f2(au.x, au.y), a1 = f2(au.z, au.w), k0 = f2(k.x, k.y), k1 = f2(k.z, k.w);
+#pragma unroll
+                for (int c = 0; c < CPT; ++c) {
+                    const F2 ny = f2(-gone[c]), vv = f2(v[c]);
+                    S[c][2 * i] = fma2(a0, ny, fma2(w0, S[c][2 * i], mul2(k0, vv)));
+                    S[c][2 * i + 1] = fma2(a1, ny, fma2(w1, S[c][2 * i + 1], mul2(k1, vv)));
+                }
             }
         }
     };
     auto flush = [&](int b, int t0, int count) {
-        for (int x = threadIdx.x; x < count * COLS; x += 256) {
+        for (int x = threadIdx.x; x < count * COLS; x += THREADS) {
             const int cc = blockIdx.z * COLS + x % COLS;
             if (cc < a.dim) O[(size_t)(t0 + x / COLS) * step + cc] = sm.o[b][x / COLS][x % COLS];
         }
@@ -275,19 +314,17 @@ __global__ void __launch_bounds__(256) delta_portion_kernel(const DeltaArgs a) {
         __syncthreads();
         flush(b, t0, min(CT, len - t0));       // written again two rounds on, past the next barrier
     }
-    if (c < a.dim) {
 #pragma unroll
-        for (int i = 0; i < RPL / 4; ++i) {
-            float f[4];
-            unpack2(S[2 * i], f[0], f[1]);
-            unpack2(S[2 * i + 1], f[2], f[3]);
+    for (int c = 0; c < CPT; ++c)
 #pragma unroll
-            for (int e = 0; e < 4; ++e) {
-                const int d = 4 * (g + LPC * i) + e;
-                if (d < a.dim) sp[(size_t)d * a.dim + c] = f[e];
-            }
+        for (int i = 0; i < R / 2; ++i) {
+            const int d = 4 * (g + LPC * (i / 2)) + 2 * (i & 1);
+            float lo, hi;
+            unpack2(S[c][i], lo, hi);
+            if (c0 + c >= a.dim) continue;
+            if (d < a.dim) sp[(size_t)d * a.dim + c0 + c] = lo;
+            if (d + 1 < a.dim) sp[(size_t)(d + 1) * a.dim + c0 + c] = hi;
         }
-    }
 }
 
 }  // namespace pie
@@ -335,15 +372,15 @@ PIE_API int pie_delta_portions(const DeltaArgs* args, int f32, cudaStream_t st) 
         auto kern = delta_portion_kernel<T_, R_, L_, C_>;                                                         \
         const cudaError_t e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)sizeof(Smem)); \
         if (e != cudaSuccess) return (int)e;                                                                      \
-        kern<<<dim3(a.reqs, a.heads, (a.dim + Smem::COLS - 1) / Smem::COLS), 256, sizeof(Smem), st>>>(a);         \
+        kern<<<dim3(a.reqs, a.heads, (a.dim + Smem::COLS - 1) / Smem::COLS), DELTA_WARPS * 32, sizeof(Smem), st>>>(a); \
         return (int)cudaGetLastError();                                                                           \
     }
 #define GO_R(T_)                            \
-    if (a.dim <= 32) GO(T_, 4, 8, 16)       \
-    if (a.dim <= 64) GO(T_, 8, 8, 16)       \
-    if (a.dim <= 128) GO(T_, 16, 8, 16)     \
-    if (a.dim <= 256) GO(T_, 32, 8, 16)     \
-    GO(T_, 32, 16, 8)
+    if (a.dim <= 32) GO(T_, 4, 8, 4)        \
+    if (a.dim <= 64) GO(T_, 4, 16, 4)       \
+    if (a.dim <= 128) GO(T_, 8, 16, 4)      \
+    if (a.dim <= 256) GO(T_, 8, 32, 4)      \
+    GO(T_, 16, 32, 2)
     if (f32) { GO_R(float) }
     GO_R(bf16)
 #undef GO_R

@@ -668,6 +668,59 @@ __global__ void __launch_bounds__(256) la_decay_kernel(const T* __restrict__ x, 
                                                    (1.4426950408889634f * factor);
 }
 
+// The bounded decay in bf16: products on mma.sync tiles, tanh(a1) as the sum of two bf16 numbers (16 digits), z in 32-bit. A block
+// takes 64 tokens and 64 channels, a warp 16 tokens and 32 channels.
+constexpr int BD_K = 32, BD_PITCH = BD_K + 8;            // rank per step; rows 80 bytes apart: fragment reads hit 32 banks
+__device__ __forceinline__ void bd_mma(float (&c)[4], const uint32_t (&a)[4], uint32_t b0, uint32_t b1) {
+    asm volatile("mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0,%1,%2,%3}, {%4,%5,%6,%7}, {%8,%9}, {%0,%1,%2,%3};\n"
+                 : "+f"(c[0]), "+f"(c[1]), "+f"(c[2]), "+f"(c[3]) : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b0), "r"(b1));
+}
+__global__ void __launch_bounds__(256) la_bounded_decay_kernel(const bf16* __restrict__ x, int ld, const bf16* __restrict__ a2,
+                                                               const bf16* __restrict__ bias, float* __restrict__ out, int n, int channels,
+                                                               int rank, float factor) {
+    __shared__ __align__(16) bf16 hi[64 * BD_PITCH], lo[64 * BD_PITCH], sw[64 * BD_PITCH];
+    pdl_trigger();
+    pdl_wait();
+    const int t0 = blockIdx.y * 64, c0 = blockIdx.x * 64;
+    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, g = lane >> 2, q = lane & 3, wt = (warp & 3) * 16, wc = (warp >> 2) * 32;
+    float acc[4][4];
+#pragma unroll
+    for (int i = 0; i < 4; ++i) acc[i][0] = acc[i][1] = acc[i][2] = acc[i][3] = 0.f;
+    for (int k0 = 0; k0 < rank; k0 += BD_K) {
+        __syncthreads();
+#pragma unroll
+        for (int i = 0; i < 64 * BD_K / 256; ++i) {
+            const int u = threadIdx.x + i * 256, row = u / BD_K, k = k0 + u % BD_K, at = row * BD_PITCH + u % BD_K;
+            const float f = t0 + row < n && k < rank ? tanhf(to_f(x[(size_t)(t0 + row) * ld + k])) : 0.f;
+            const bf16 h = __float2bfloat16(f);
+            hi[at] = h;
+            lo[at] = __float2bfloat16(f - __bfloat162float(h));
+            sw[at] = c0 + row < channels && k < rank ? a2[(size_t)(c0 + row) * rank + k] : __float2bfloat16(0.f);
+        }
+        __syncthreads();
+#pragma unroll
+        for (int ks = 0; ks < BD_K; ks += 16) {
+            auto word = [&](const bf16* m, int row, int col) { return *reinterpret_cast<const uint32_t*>(m + row * BD_PITCH + ks + col); };
+            const uint32_t ah[4] = {word(hi, wt + g, 2 * q), word(hi, wt + g + 8, 2 * q), word(hi, wt + g, 2 * q + 8), word(hi, wt + g + 8, 2 * q + 8)};
+            const uint32_t al[4] = {word(lo, wt + g, 2 * q), word(lo, wt + g + 8, 2 * q), word(lo, wt + g, 2 * q + 8), word(lo, wt + g + 8, 2 * q + 8)};
+#pragma unroll
+            for (int i = 0; i < 4; ++i) {
+                const uint32_t b0 = word(sw, wc + i * 8 + g, 2 * q), b1 = word(sw, wc + i * 8 + g, 2 * q + 8);
+                bd_mma(acc[i], ah, b0, b1);
+                bd_mma(acc[i], al, b0, b1);
+            }
+        }
+    }
+#pragma unroll
+    for (int i = 0; i < 4; ++i)
+#pragma unroll
+        for (int e = 0; e < 4; ++e) {
+            const int t = t0 + wt + g + (e >> 1) * 8, c = c0 + wc + i * 8 + 2 * q + (e & 1);
+            if (t < n && c < channels)
+                out[(size_t)t * channels + c] = -(1.4426950408889634f * factor) / (1.f + expf(-(acc[i][e] + to_f(bias[c]))));
+        }
+}
+
 // ------------------------------------------- exponential gates of a matrix memory
 // Per head logarithms i = cap tanh(z_i / cap) and f = logsigmoid(cap tanh(z_f / cap)) of the input and forget gates, and a
 // running maximum m_t = max(f_t + m_(t-1), i_t), m from 0, that takes the size out of the state: decay exp(f_t + m_(t-1) -
@@ -974,7 +1027,9 @@ PIE_API int pie_linear_decay(const void* x, int ld, const void* a2, const void* 
                            rank, factor)
     if (f32 && bounded) GO(float, true);
     if (f32) GO(float, false);
-    if (bounded) GO(bf16, true);
+    if (bounded)
+        return (int)launch_pdl(la_bounded_decay_kernel, dim3((channels + 63) / 64, (n + 63) / 64), dim3(256), 0, st, (const bf16*)x, ld,
+                               (const bf16*)a2, (const bf16*)bias, out, n, channels, rank, factor);
     GO(bf16, false);
 #undef GO
 }

@@ -473,6 +473,12 @@ PRESETS = {
                                layer_types=["linear_attention", "sliding_attention"] * 16, linear_num_key_heads=16,
                                linear_num_value_heads=32, linear_key_head_dim=128, linear_value_head_dim=128, num_experts=32,
                                num_experts_per_tok=4, moe_intermediate_size=2048),
+    # attention over everything and Gated DeltaNet with states of the same size, layer about, feed-forwards widened to the same
+    # parameters: what `vulanex-8b` is measured beside
+    "gdn-8b": dict(model_type="qwen3_next", hidden_size=4096, intermediate_size=13952, num_hidden_layers=32, num_attention_heads=32,
+                   num_key_value_heads=8, head_dim=128, vocab_size=128256, rope_theta=500000.0, rms_norm_eps=1e-5, qk_norm=True,
+                   layer_types=["full_attention", "linear_attention"] * 16, linear_num_key_heads=16, linear_num_value_heads=32,
+                   linear_key_head_dim=128, linear_value_head_dim=128),
     "qwen3-32b": dict(model_type="qwen3", hidden_size=5120, intermediate_size=25600,
                       num_hidden_layers=64, num_attention_heads=64, num_key_value_heads=8, head_dim=128,
                       vocab_size=151936, rope_theta=1000000.0, rms_norm_eps=1e-6, qk_norm=True),

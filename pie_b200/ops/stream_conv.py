@@ -14,8 +14,10 @@ from .latent import _struct, f32, i32, i64, p
 # mirrors of the argument structs in csrc/kernels/stream_conv.cu
 PairEmbedArgs = _struct("PairEmbedArgs", ("tokens table pairs x tok_req qo_indptr slots reset state", p),
                         ("slot_stride buckets mul_prev mul_cur", i64), ("n reqs width ldx vocab", i32))
-ConvNormArgs = _struct("ConvNormArgs", ("x x_out y0 y1 y0_norm y1_norm w b conv h tok_req qo_indptr slots reset state stage", p),
+ConvNormArgs = _struct("ConvNormArgs", ("x x_out y0 y1 y0_norm y1_norm w b conv h tok_req qo_indptr slots reset state stage stats", p),
                        ("slot_stride", i64), ("n width ldx ldy ldh taps rows_per_block", i32), ("eps", f32))
+
+MANY_ROWS = 512         # from here on statistics and convolution are two launches
 
 
 def pair_embed(tokens, table, pairs, spec, ld: int, rs):
@@ -45,7 +47,10 @@ def conv_norm(x, width: int, eps: float, pending=(), w=None, b=None, conv=None, 
     h = torch.empty(n, ld, dtype=dtype, device=x.device) if w is not None else None
     taps = conv.shape[0] if conv is not None else 0
     a = ConvNormArgs(x=ptr(x), x_out=ptr(x_out), w=ptr(w), b=ptr(b), conv=ptr(conv), h=ptr(h), n=n, width=width, ldx=ld, ldh=ld,
-                     taps=taps, rows_per_block=max(1, min(8, n // 592)), eps=eps)
+                     taps=taps, rows_per_block=16 if n >= MANY_ROWS else 1, eps=eps)
+    if n >= MANY_ROWS:
+        stats = torch.empty(n, 2, dtype=torch.float32, device=x.device)
+        a.stats = ptr(stats)
     if pending:
         if any(y.stride(0) != pending[0][0].stride(0) for y, _ in pending):
             raise ValueError("pending outputs of unequal pitch")
