@@ -8,6 +8,8 @@
 //   step       one token per request: a block holds 128 columns (VEC per lane) of a head, an eighth of the rows per warp
 //   portions   any lengths: LPC lanes share CPT columns, each with R rows of them; a token's sums meet by halving (a lane ends up
 //              with one of them); the tokens' vectors are prepared CT at a time in shared memory while the tokens before run
+//   chunked    prompts in bf16, heads of up to 128: 16 tokens at a time on tf32 tensor-core tiles, see below
+#include "tf32.cuh"
 #include "typed.cuh"
 
 namespace pie {
@@ -19,8 +21,11 @@ struct DeltaArgs {
     float* out;                     // [n, heads * dim]
     float* state;                   // this layer's part of slot 0: [heads][dim][dim]
     const int *qo_indptr, *slots, *reset;
+    // chunked form: request and first row of a piece of 16 tokens; pieces of a request (indptr)
+    const int *chunk_req, *chunk_start, *req_chunks;
+    void* pieces;                   // [chunks][heads] DeltaPiece
     long slot_stride;
-    int n, ld, reqs, heads, dim;
+    int n, ld, reqs, heads, dim, chunks;
 };
 
 __device__ __forceinline__ float delta_rate(float z) { return 1.f / (1.f + expf(-z)); }
@@ -327,6 +332,254 @@ __global__ void __launch_bounds__(DELTA_WARPS * 32) delta_portion_kernel(const D
         }
 }
 
+// ----------------------------------------------------------------- chunked
+// Sixteen tokens from a state S0. With G_t the product of the decays up to t and
+//   c_t = G_(t-1) u_t,  R_t = G_t r_t,  K_t = k_t / G_t,  B_t = (a_t u_t) / G_t      (1 / G_t <= e^9.8: decays are at least 0.54)
+// the rows p_t = u_t^T S_(t-1) that the tokens remove solve p_t + sum_(s < t) (c_t.B_s) p_s = c_t S0 + sum_(s < t) (c_t.K_s) v_s, and
+//   o_t = R_t S0 + sum_(s <= t) (R_t.K_s) v_s - (R_t.B_s) p_s,    S_16 = G_16 (S0 + sum_s K_s v_s^T - B_s p_s^T).
+//   delta_piece   all pieces at once: those vectors, the four 16 x 16 score matrices, the inverse of the triangular one
+//   delta_walk    piece by piece: a warp holds 16 value columns of S0 transposed, [columns][keys], as the accumulators of the
+//                 update, which are at the same time the A operand of c S0 and R S0 (a key step's columns t and t + 4 stand for the
+//                 keys 2 t and 2 t + 1); the next piece is on its way meanwhile
+// The state stays 32-bit; product operands are rounded to tf32.
+constexpr int DC_T = 16, DC_WARPS = 4, DC_COLS = DC_WARPS * 16, DC_SMALL = 24;
+
+template <int DP>
+struct DeltaPiece {
+    static constexpr int XP = DP + 8, KP = DP + 4;          // pitches: fragment reads hit 32 banks
+    float x[2 * DC_T][XP];                                  // c, then R
+    float k[DC_T][KP], b[DC_T][KP];
+    float m[DC_T][DC_SMALL], q[DC_T][DC_SMALL], nb[DC_T][DC_SMALL], t[DC_T][DC_SMALL];   // c.K, R.K, -R.B, inverse less 1
+    float g[DP];
+};
+
+template <int DP>
+__global__ void __launch_bounds__(128) delta_piece_kernel(const DeltaArgs a) {
+    using Piece = DeltaPiece<DP>;
+    extern __shared__ __align__(16) uint8_t raw[];
+    Piece& B = *reinterpret_cast<Piece*>(raw);
+    __shared__ __align__(16) float l[DC_T][DC_T + 4];       // c.B
+    __shared__ float squares[4][DC_T];
+    const int pc = blockIdx.x, h = blockIdx.y, hw = threadIdx.x >> 5, lane = threadIdx.x & 31, g = lane >> 2, t = lane & 3, d = threadIdx.x;
+    const int row0 = a.chunk_start[pc], len = min(DC_T, a.qo_indptr[a.chunk_req[pc] + 1] - row0);
+    const bool own = d < a.dim;
+    const size_t step = (size_t)a.heads * a.dim, at0 = (size_t)row0 * a.ld + h * a.dim + d;
+    const float* W = a.log_decay + (size_t)row0 * step + h * a.dim + d;
+    const bf16 none = __float2bfloat16(0.f);
+    bf16 pk[DC_T], pr[DC_T], pa[DC_T];
+    float pw[DC_T], sq[DC_T];
+#pragma unroll
+    for (int s = 0; s < DC_T; ++s) {
+        const bool ok = own && s < len;
+        const size_t at = at0 + (size_t)s * a.ld;
+        pk[s] = ok ? static_cast<const bf16*>(a.k)[at] : none;
+        pr[s] = ok ? static_cast<const bf16*>(a.r)[at] : none;
+        pa[s] = ok ? static_cast<const bf16*>(a.a)[at] : none;
+        pw[s] = ok ? W[s * step] : 0.f;
+    }
+#pragma unroll
+    for (int s = 0; s < DC_T; ++s) sq[s] = to_f(pk[s]) * to_f(pk[s]);
+    const float part = halving_sum<DC_T, 32>(sq, lane);     // of token lane / 2
+    if ((lane & 1) == 0) squares[hw][lane >> 1] = part;
+    __syncthreads();
+    const float inv = 1.f / sqrtf(squares[0][lane & 15] + squares[1][lane & 15] + squares[2][lane & 15] + squares[3][lane & 15] + 1e-6f);
+    const float bias = own ? a.a_bias[h * a.dim + d] : 0.f;
+    float sum = 0.f, before = 1.f;
+#pragma unroll
+    for (int s = 0; s < DC_T; ++s) {
+        const float unit = __shfl_sync(0xffffffffu, inv, s);
+        if (d >= DP) continue;
+        sum += pw[s];
+        const float now = exp2f(sum), back = exp2f(-sum), k = to_f(pk[s]), u = k * unit;
+        B.x[s][d] = tf32_f(before * u);
+        B.x[DC_T + s][d] = tf32_f(now * to_f(pr[s]));
+        B.k[s][d] = tf32_f(back * k);
+        B.b[s][d] = tf32_f(back * u * __fdividef(1.f, 1.f + __expf(-(to_f(pa[s]) + bias))));
+        before = now;
+    }
+    if (d < DP) B.g[d] = before;
+    __syncthreads();
+    // scores: this warp's eight keys (K of tokens 0-7, 8-15, then B) against c and R
+    float acc[2][4];
+#pragma unroll
+    for (int i = 0; i < 2; ++i) acc[i][0] = acc[i][1] = acc[i][2] = acc[i][3] = 0.f;
+    const float* row = (hw < 2 ? B.k : B.b)[(hw & 1) * 8 + g];
+#pragma unroll
+    for (int j = 0; j < DP / 8; ++j) {
+        const float2 f = *reinterpret_cast<const float2*>(row + j * 8 + 2 * t);
+#pragma unroll
+        for (int i = 0; i < 2; ++i) {
+            const float2 x0 = *reinterpret_cast<const float2*>(&B.x[i * DC_T + g][j * 8 + 2 * t]);
+            const float2 x1 = *reinterpret_cast<const float2*>(&B.x[i * DC_T + g + 8][j * 8 + 2 * t]);
+            const float fa[4] = {x0.x, x1.x, x0.y, x1.y};
+            mma_tf32(acc[i], fa, f.x, f.y);
+        }
+    }
+#pragma unroll
+    for (int e = 0; e < 4; ++e) {
+        const int i = g + (e >> 1) * 8, s = (hw & 1) * 8 + 2 * t + (e & 1);
+        const float c = s < i ? acc[0][e] : 0.f, r = s <= i ? acc[1][e] : 0.f;
+        if (hw < 2) {
+            B.m[i][s] = tf32_f(c);
+            B.q[i][s] = tf32_f(r);
+        } else {
+            l[i][s] = c;
+            B.nb[i][s] = tf32_f(-r);
+        }
+    }
+    __syncthreads();
+    if (hw == 0) {
+        // column `lane` of the inverse of 1 + l
+        float y[DC_T];
+#pragma unroll
+        for (int i = 0; i < DC_T; ++i) {
+            float z0 = i == lane ? 1.f : 0.f, z1 = 0.f;
+#pragma unroll
+            for (int s = 0; s < i; ++s) {
+                if (s & 1) z1 -= l[i][s] * y[s];
+                else z0 -= l[i][s] * y[s];
+            }
+            y[i] = z0 + z1;
+            if (lane < DC_T) B.t[i][lane] = i > lane ? tf32_f(y[i]) : 0.f;
+        }
+    }
+    __syncthreads();
+    float4* dst = reinterpret_cast<float4*>(static_cast<Piece*>(a.pieces) + (size_t)pc * a.heads + h);
+    const float4* src = reinterpret_cast<const float4*>(raw);
+    for (int i = threadIdx.x; i < (int)(sizeof(Piece) / 16); i += 128) dst[i] = src[i];
+}
+
+__device__ __forceinline__ void copy16(void* dst, const void* src) {
+    asm volatile("cp.async.cg.shared.global [%0], [%1], 16;\n" ::"r"((uint32_t)__cvta_generic_to_shared(dst)), "l"(src));
+}
+
+template <int DP>
+__global__ void __launch_bounds__(DC_WARPS * 32) delta_walk_kernel(const DeltaArgs a) {
+    using Piece = DeltaPiece<DP>;
+    constexpr int NT = DP / 8;
+    extern __shared__ __align__(16) uint8_t raw[];
+    Piece* buf = reinterpret_cast<Piece*>(raw);
+    const int q = blockIdx.x, h = blockIdx.y, warp = threadIdx.x >> 5, lane = threadIdx.x & 31, g = lane >> 2, t = lane & 3;
+    const int first = a.qo_indptr[q], len = a.qo_indptr[q + 1] - first, slot = a.slots[q];
+    if (len <= 0 || slot < 0) return;
+    const int pieces = (len + DC_T - 1) / DC_T, c0 = blockIdx.z * DC_COLS + warp * 16;
+    const Piece* src = static_cast<const Piece*>(a.pieces) + (size_t)a.req_chunks[q] * a.heads + h;
+    auto fetch = [&](int pc) {
+        const uint8_t* from = reinterpret_cast<const uint8_t*>(src + (size_t)pc * a.heads);
+        uint8_t* to = reinterpret_cast<uint8_t*>(buf + (pc & 1));
+        for (int i = threadIdx.x * 16; i < (int)sizeof(Piece); i += DC_WARPS * 32 * 16) copy16(to + i, from + i);
+    };
+    // values of a piece as A operands: [key step][token 2 t | 2 t + 1, column g | g + 8]
+    const bf16* V = static_cast<const bf16*>(a.v) + (size_t)first * a.ld + h * a.dim;
+    bf16 pv[2][4];
+    auto values = [&](int pc) {
+#pragma unroll
+        for (int j = 0; j < 2; ++j)
+#pragma unroll
+            for (int e = 0; e < 4; ++e) {
+                const int tok = pc * DC_T + j * 8 + 2 * t + (e >> 1), c = c0 + g + (e & 1) * 8;
+                pv[j][e] = tok < len && c < a.dim ? V[(size_t)tok * a.ld + c] : __float2bfloat16(0.f);
+            }
+    };
+    fetch(0);
+    asm volatile("cp.async.commit_group;\n");
+    values(0);
+    float* sp = a.state + (size_t)slot * a.slot_stride + (size_t)h * a.dim * a.dim;
+    const size_t step = (size_t)a.heads * a.dim;
+    float* O = a.out + ((size_t)first * a.heads + h) * a.dim;
+    const bool fresh = a.reset[q] != 0;
+    float S[NT][4];
+#pragma unroll
+    for (int j = 0; j < NT; ++j)
+#pragma unroll
+        for (int e = 0; e < 4; ++e) {
+            const int d = j * 8 + 2 * t + (e & 1), c = c0 + g + (e >> 1) * 8;
+            S[j][e] = !fresh && d < a.dim && c < a.dim ? sp[(size_t)d * a.dim + c] : 0.f;
+        }
+    for (int pc = 0; pc < pieces; ++pc) {
+        if (pc + 1 < pieces) fetch(pc + 1);
+        asm volatile("cp.async.commit_group;\n");
+        float va[2][4];
+#pragma unroll
+        for (int j = 0; j < 2; ++j)
+#pragma unroll
+            for (int e = 0; e < 4; ++e) va[j][e] = to_f(pv[j][e]);
+        if (pc + 1 < pieces) values(pc + 1);
+        asm volatile("cp.async.wait_group 1;\n" ::: "memory");
+        __syncthreads();
+        const Piece& B = buf[pc & 1];
+        float x[4][4];
+#pragma unroll
+        for (int i = 0; i < 4; ++i) x[i][0] = x[i][1] = x[i][2] = x[i][3] = 0.f;
+#pragma unroll
+        for (int j = 0; j < NT; ++j) {
+            const float fa[4] = {tf32_f(S[j][0]), tf32_f(S[j][2]), tf32_f(S[j][1]), tf32_f(S[j][3])};
+#pragma unroll
+            for (int i = 0; i < 4; ++i) {
+                const float2 f = *reinterpret_cast<const float2*>(&B.x[i * 8 + g][j * 8 + 2 * t]);
+                mma_tf32(x[i], fa, f.x, f.y);
+            }
+        }
+        float ya[2][4], p[2][4];
+        auto lower = [&](float (&acc)[4], const float (&m)[DC_T][DC_SMALL], int i, int j, const float (&fa)[4]) {
+            const float2 f = *reinterpret_cast<const float2*>(&m[i * 8 + g][j * 8 + 2 * t]);
+            mma_tf32(acc, fa, f.x, f.y);
+        };
+        auto operand = [&](float (&fa)[4], const float (&acc)[4]) {
+            fa[0] = tf32_f(acc[0]); fa[1] = tf32_f(acc[2]); fa[2] = tf32_f(acc[1]); fa[3] = tf32_f(acc[3]);
+        };
+#pragma unroll
+        for (int i = 0; i < 2; ++i)
+#pragma unroll
+            for (int j = 0; j <= i; ++j) {
+                lower(x[i], B.m, i, j, va[j]);
+                lower(x[2 + i], B.q, i, j, va[j]);
+            }
+#pragma unroll
+        for (int j = 0; j < 2; ++j) {
+#pragma unroll
+            for (int e = 0; e < 4; ++e) p[j][e] = x[j][e];
+            operand(ya[j], x[j]);
+        }
+#pragma unroll
+        for (int i = 0; i < 2; ++i)
+#pragma unroll
+            for (int j = 0; j <= i; ++j) lower(p[i], B.t, i, j, ya[j]);
+        operand(ya[0], p[0]);
+        operand(ya[1], p[1]);
+#pragma unroll
+        for (int i = 0; i < 2; ++i)
+#pragma unroll
+            for (int j = 0; j <= i; ++j) lower(x[2 + i], B.nb, i, j, ya[j]);
+#pragma unroll
+        for (int i = 0; i < 2; ++i)
+#pragma unroll
+            for (int e = 0; e < 4; ++e) {
+                const int tok = pc * DC_T + i * 8 + 2 * t + (e & 1), c = c0 + g + (e >> 1) * 8;
+                if (tok < len && c < a.dim) O[(size_t)tok * step + c] = x[2 + i][e];
+                ya[i][e] = -ya[i][e];
+            }
+#pragma unroll
+        for (int n = 0; n < NT; ++n) {
+#pragma unroll
+            for (int j = 0; j < 2; ++j) {
+                mma_tf32(S[n], va[j], B.k[j * 8 + 2 * t][n * 8 + g], B.k[j * 8 + 2 * t + 1][n * 8 + g]);
+                mma_tf32(S[n], ya[j], B.b[j * 8 + 2 * t][n * 8 + g], B.b[j * 8 + 2 * t + 1][n * 8 + g]);
+            }
+            const float2 f = *reinterpret_cast<const float2*>(&B.g[n * 8 + 2 * t]);
+            S[n][0] *= f.x; S[n][1] *= f.y; S[n][2] *= f.x; S[n][3] *= f.y;
+        }
+        __syncthreads();
+    }
+#pragma unroll
+    for (int j = 0; j < NT; ++j)
+#pragma unroll
+        for (int e = 0; e < 4; ++e) {
+            const int d = j * 8 + 2 * t + (e & 1), c = c0 + g + (e >> 1) * 8;
+            if (d < a.dim && c < a.dim) sp[(size_t)d * a.dim + c] = S[j][e];
+        }
+}
+
 }  // namespace pie
 
 using namespace pie;
@@ -359,6 +612,35 @@ PIE_API int pie_delta_step(const DeltaArgs* args, int f32, cudaStream_t st) {
     if (f32) { GO_R(float); }
     GO_R(bf16);
 #undef GO_R
+#undef GO
+}
+
+// Bytes of one piece of one head in the chunked form; 0: no such form for this head size.
+PIE_API int pie_delta_piece_bytes(int dim) {
+    return dim <= 0 || dim > 128 ? 0 : dim <= 32 ? (int)sizeof(DeltaPiece<32>) : dim <= 64 ? (int)sizeof(DeltaPiece<64>) : (int)sizeof(DeltaPiece<128>);
+}
+PIE_API int pie_delta_piece_tokens() { return DC_T; }
+
+// Prompts in bf16, head sizes with a piece.
+PIE_API int pie_delta_chunked(const DeltaArgs* args, cudaStream_t st) {
+    const DeltaArgs& a = *args;
+    if (a.n <= 0 || a.reqs <= 0 || a.chunks <= 0) return 0;
+    if (!delta_ok(a) || a.dim > 128 || !a.pieces || !a.chunk_req || !a.chunk_start || !a.req_chunks) return (int)cudaErrorInvalidValue;
+    const dim3 grid(a.reqs, a.heads, (a.dim + DC_COLS - 1) / DC_COLS);
+#define GO(D_)                                                                                                              \
+    {                                                                                                                       \
+        constexpr int bytes = (int)sizeof(DeltaPiece<D_>);                                                                  \
+        static_assert(bytes % 16 == 0, "");                                                                                 \
+        cudaError_t e = cudaFuncSetAttribute(delta_piece_kernel<D_>, cudaFuncAttributeMaxDynamicSharedMemorySize, bytes);   \
+        if (e == cudaSuccess) e = cudaFuncSetAttribute(delta_walk_kernel<D_>, cudaFuncAttributeMaxDynamicSharedMemorySize, 2 * bytes); \
+        if (e != cudaSuccess) return (int)e;                                                                                \
+        delta_piece_kernel<D_><<<dim3(a.chunks, a.heads), 128, bytes, st>>>(a);                                             \
+        delta_walk_kernel<D_><<<grid, DC_WARPS * 32, 2 * bytes, st>>>(a);                                                   \
+        return (int)cudaGetLastError();                                                                                     \
+    }
+    if (a.dim <= 32) GO(32)
+    if (a.dim <= 64) GO(64)
+    GO(128)
 #undef GO
 }
 

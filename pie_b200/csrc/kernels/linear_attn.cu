@@ -16,6 +16,7 @@
 //            by pair. Every other factor is at most 1, so nothing overflows whatever the decays.
 //
 // The form with sub-blocks follows S. Yang et al., "Gated Linear Attention Transformers with Hardware-Efficient Training".
+#include "tf32.cuh"
 #include "typed.cuh"
 
 namespace pie {
@@ -167,21 +168,6 @@ constexpr int LA_VT = 64;                 // value columns per pass
 constexpr int LA_VP = LA_VT + 8;          // pitch of a tile read as (row by t, column by g): fragment reads hit 32 banks
 constexpr int LA_SP = LA_C + 4;           // pitch of the scores, and of values read at rows 2 t, 2 t + 1
 constexpr int LA_THREADS = 256;
-
-__device__ __forceinline__ uint32_t tf32(float x) {
-    uint32_t r;
-    asm("cvt.rna.tf32.f32 %0, %1;" : "=r"(r) : "f"(x));
-    return r;
-}
-__device__ __forceinline__ float tf32_f(float x) { return __uint_as_float(tf32(x)); }
-// C (16 x 8) += A (16 x 8, row) B (8 x 8, col); lane (g = lane / 4, t = lane % 4) holds A (g | g + 8, t | t + 4),
-// B (t | t + 4, g) and C (g | g + 8, 2 t | 2 t + 1). Operands are already rounded to tf32.
-__device__ __forceinline__ void mma_tf32(float (&c)[4], const float (&a)[4], float b0, float b1) {
-    asm volatile("mma.sync.aligned.m16n8k8.row.col.f32.tf32.tf32.f32 {%0,%1,%2,%3}, {%4,%5,%6,%7}, {%8,%9}, {%0,%1,%2,%3};\n"
-                 : "+f"(c[0]), "+f"(c[1]), "+f"(c[2]), "+f"(c[3])
-                 : "r"(__float_as_uint(a[0])), "r"(__float_as_uint(a[1])), "r"(__float_as_uint(a[2])), "r"(__float_as_uint(a[3])),
-                   "r"(__float_as_uint(b0)), "r"(__float_as_uint(b1)));
-}
 
 __host__ __device__ constexpr int la_dimp(int dim) { return (dim + 15) / 16 * 16; }
 // Pitch of a [64][dim] array of bf16 (queries, keys) and of 32-bit decayed keys: 8 (mod 32) words or 4 (mod 16)
@@ -669,38 +655,45 @@ __global__ void __launch_bounds__(256) la_decay_kernel(const T* __restrict__ x, 
 }
 
 // The bounded decay in bf16: products on mma.sync tiles, tanh(a1) as the sum of two bf16 numbers (16 digits), z in 32-bit. A block
-// takes 64 tokens and 64 channels, a warp 16 tokens and 32 channels.
-constexpr int BD_K = 32, BD_PITCH = BD_K + 8;            // rank per step; rows 80 bytes apart: fragment reads hit 32 banks
+// takes 64 tokens and `tiles` times 64 channels, a warp 16 tokens and 32 channels of a tile. Rows of rank + 8 (rank rounded up to
+// a multiple of 32, which makes fragment reads hit 32 banks at an odd multiple of 8 words).
+constexpr int BD_MAX_RANK = 256;
+__host__ __device__ constexpr int bd_rank(int rank) { return (rank + 31) / 32 * 32; }
 __device__ __forceinline__ void bd_mma(float (&c)[4], const uint32_t (&a)[4], uint32_t b0, uint32_t b1) {
     asm volatile("mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0,%1,%2,%3}, {%4,%5,%6,%7}, {%8,%9}, {%0,%1,%2,%3};\n"
                  : "+f"(c[0]), "+f"(c[1]), "+f"(c[2]), "+f"(c[3]) : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b0), "r"(b1));
 }
 __global__ void __launch_bounds__(256) la_bounded_decay_kernel(const bf16* __restrict__ x, int ld, const bf16* __restrict__ a2,
                                                                const bf16* __restrict__ bias, float* __restrict__ out, int n, int channels,
-                                                               int rank, float factor) {
-    __shared__ __align__(16) bf16 hi[64 * BD_PITCH], lo[64 * BD_PITCH], sw[64 * BD_PITCH];
+                                                               int rank, float factor, int tiles) {
+    extern __shared__ __align__(16) bf16 bd_smem[];
+    const int rp = bd_rank(rank), pitch = rp + 8;
+    bf16 *hi = bd_smem, *lo = hi + 64 * pitch, *sw = lo + 64 * pitch;
     pdl_trigger();
     pdl_wait();
-    const int t0 = blockIdx.y * 64, c0 = blockIdx.x * 64;
+    const int t0 = blockIdx.y * 64;
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, g = lane >> 2, q = lane & 3, wt = (warp & 3) * 16, wc = (warp >> 2) * 32;
-    float acc[4][4];
-#pragma unroll
-    for (int i = 0; i < 4; ++i) acc[i][0] = acc[i][1] = acc[i][2] = acc[i][3] = 0.f;
-    for (int k0 = 0; k0 < rank; k0 += BD_K) {
+    for (int u = threadIdx.x; u < 64 * rp; u += 256) {
+        const int row = u / rp, k = u - row * rp;
+        const float f = t0 + row < n && k < rank ? tanhf(to_f(x[(size_t)(t0 + row) * ld + k])) : 0.f;
+        const bf16 h = __float2bfloat16(f);
+        hi[row * pitch + k] = h;
+        lo[row * pitch + k] = __float2bfloat16(f - __bfloat162float(h));
+    }
+    for (int tile = 0; tile < tiles; ++tile) {
+        const int c0 = (blockIdx.x * tiles + tile) * 64;
+        if (c0 >= channels) break;
         __syncthreads();
-#pragma unroll
-        for (int i = 0; i < 64 * BD_K / 256; ++i) {
-            const int u = threadIdx.x + i * 256, row = u / BD_K, k = k0 + u % BD_K, at = row * BD_PITCH + u % BD_K;
-            const float f = t0 + row < n && k < rank ? tanhf(to_f(x[(size_t)(t0 + row) * ld + k])) : 0.f;
-            const bf16 h = __float2bfloat16(f);
-            hi[at] = h;
-            lo[at] = __float2bfloat16(f - __bfloat162float(h));
-            sw[at] = c0 + row < channels && k < rank ? a2[(size_t)(c0 + row) * rank + k] : __float2bfloat16(0.f);
+        for (int u = threadIdx.x; u < 64 * rp; u += 256) {
+            const int row = u / rp, k = u - row * rp;
+            sw[row * pitch + k] = c0 + row < channels && k < rank ? a2[(size_t)(c0 + row) * rank + k] : __float2bfloat16(0.f);
         }
         __syncthreads();
+        float acc[4][4];
 #pragma unroll
-        for (int ks = 0; ks < BD_K; ks += 16) {
-            auto word = [&](const bf16* m, int row, int col) { return *reinterpret_cast<const uint32_t*>(m + row * BD_PITCH + ks + col); };
+        for (int i = 0; i < 4; ++i) acc[i][0] = acc[i][1] = acc[i][2] = acc[i][3] = 0.f;
+        for (int ks = 0; ks < rp; ks += 16) {
+            auto word = [&](const bf16* m, int row, int col) { return *reinterpret_cast<const uint32_t*>(m + row * pitch + ks + col); };
             const uint32_t ah[4] = {word(hi, wt + g, 2 * q), word(hi, wt + g + 8, 2 * q), word(hi, wt + g, 2 * q + 8), word(hi, wt + g + 8, 2 * q + 8)};
             const uint32_t al[4] = {word(lo, wt + g, 2 * q), word(lo, wt + g + 8, 2 * q), word(lo, wt + g, 2 * q + 8), word(lo, wt + g + 8, 2 * q + 8)};
 #pragma unroll
@@ -710,15 +703,26 @@ __global__ void __launch_bounds__(256) la_bounded_decay_kernel(const bf16* __res
                 bd_mma(acc[i], al, b0, b1);
             }
         }
-    }
 #pragma unroll
-    for (int i = 0; i < 4; ++i)
+        for (int i = 0; i < 4; ++i) {
+            const int c = c0 + wc + i * 8 + 2 * q;
+            const float b0 = c < channels ? to_f(bias[c]) : 0.f, b1 = c + 1 < channels ? to_f(bias[c + 1]) : 0.f;
 #pragma unroll
-        for (int e = 0; e < 4; ++e) {
-            const int t = t0 + wt + g + (e >> 1) * 8, c = c0 + wc + i * 8 + 2 * q + (e & 1);
-            if (t < n && c < channels)
-                out[(size_t)t * channels + c] = -(1.4426950408889634f * factor) / (1.f + expf(-(acc[i][e] + to_f(bias[c]))));
+            for (int e = 0; e < 4; e += 2) {
+                const int t = t0 + wt + g + (e >> 1) * 8;
+                if (t >= n) continue;
+                const float f = -1.4426950408889634f * factor;
+                const float y0 = __fdividef(f, 1.f + expf(-(acc[i][e] + b0))), y1 = __fdividef(f, 1.f + expf(-(acc[i][e + 1] + b1)));
+                float* dst = out + (size_t)t * channels + c;
+                if (c + 1 < channels && channels % 2 == 0) {
+                    *reinterpret_cast<float2*>(dst) = make_float2(y0, y1);
+                } else {
+                    if (c < channels) dst[0] = y0;
+                    if (c + 1 < channels) dst[1] = y1;
+                }
+            }
         }
+    }
 }
 
 // ------------------------------------------- exponential gates of a matrix memory
@@ -1027,9 +1031,14 @@ PIE_API int pie_linear_decay(const void* x, int ld, const void* a2, const void* 
                            rank, factor)
     if (f32 && bounded) GO(float, true);
     if (f32) GO(float, false);
-    if (bounded)
-        return (int)launch_pdl(la_bounded_decay_kernel, dim3((channels + 63) / 64, (n + 63) / 64), dim3(256), 0, st, (const bf16*)x, ld,
-                               (const bf16*)a2, (const bf16*)bias, out, n, channels, rank, factor);
+    if (bounded && rank > BD_MAX_RANK) GO(bf16, true);
+    if (bounded) {
+        const int bytes = 3 * 64 * (bd_rank(rank) + 8) * 2, tiles = n >= 1024 ? 4 : 1;
+        const cudaError_t e = cudaFuncSetAttribute(la_bounded_decay_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, bytes);
+        if (e != cudaSuccess) return (int)e;
+        return (int)launch_pdl(la_bounded_decay_kernel, dim3((channels + 64 * tiles - 1) / (64 * tiles), (n + 63) / 64), dim3(256), bytes, st,
+                               (const bf16*)x, ld, (const bf16*)a2, (const bf16*)bias, out, n, channels, rank, factor, tiles);
+    }
     GO(bf16, false);
 #undef GO
 }

@@ -12,7 +12,7 @@ Counterpart of driver/cuda/src/recurrent_state_cache.hpp:1-40 (slabs per layer a
 """
 from __future__ import annotations
 
-from dataclasses import dataclass
+from dataclasses import dataclass, field
 from functools import cached_property
 from typing import Dict, List, Optional
 
@@ -44,7 +44,7 @@ class RecurrentInputs:
     history_elems: int = 0                       # numbers of one history
     token_at: Optional[int] = None               # element that holds the token before, as an integer
     conv_stage: Optional[torch.Tensor] = None    # [R, taps - 1, W] fp32: the new history of portions until its readers are done
-    pieces: Optional[tuple] = None # the portions cut for the chunked form (`ops.linear.chunk_pieces`)
+    pieces: dict = field(default_factory=dict)   # piece size -> the portions cut for a chunked form (`ops.linear.chunk_pieces`)
     staged: Optional[int] = None   # requests the stage is committed for (0: none of this fire's portions uses it)
 
     def state_of(self, li: int, elems: int) -> torch.Tensor:

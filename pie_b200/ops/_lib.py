@@ -95,6 +95,9 @@ _SIGNATURES = {
     "pie_conv_norm": [p, i32, i32, p],
     "pie_delta_step": [p, i32, p],
     "pie_delta_portions": [p, i32, p],
+    "pie_delta_chunked": [p, p],
+    "pie_delta_piece_bytes": [i32],
+    "pie_delta_piece_tokens": [],
     "pie_head_rows": [p, i32, p],
     "pie_pool_rows": [p, i32, p],
     "pie_pool_gather": [p, p],

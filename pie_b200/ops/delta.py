@@ -11,10 +11,11 @@ import torch
 
 from ._lib import check, fn, ptr, stream_ptr
 from .latent import _f32, _struct, i32, i64, p
+from .linear import chunk_pieces
 
 # mirror of the argument struct in csrc/kernels/delta_rule.cu
-DeltaArgs = _struct("DeltaArgs", ("r k v a a_bias log_decay out state qo_indptr slots reset", p), ("slot_stride", i64),
-                    ("n ld reqs heads dim", i32))
+DeltaArgs = _struct("DeltaArgs", ("r k v a a_bias log_decay out state qo_indptr slots reset chunk_req chunk_start req_chunks pieces", p),
+                    ("slot_stride", i64), ("n ld reqs heads dim chunks", i32))
 LOG2E = 1.4426950408889634
 
 
@@ -41,6 +42,13 @@ def delta_rule(r, k, v, a, a_bias, log_decay, spec, rs, state, decode: bool):
     args = DeltaArgs(r=ptr(r), k=ptr(k), v=ptr(v), a=ptr(a), a_bias=ptr(a_bias), log_decay=ptr(log_decay), out=ptr(out), state=ptr(state),
                      qo_indptr=ptr(rs.qo_indptr), slots=ptr(rs.slots), reset=ptr(rs.reset), slot_stride=state.stride(0), n=n, ld=r.stride(0),
                      reqs=len(rs.slots_host), heads=spec.heads, dim=spec.dim)
+    size = fn("pie_delta_piece_bytes")(spec.dim) if not decode and r.dtype == torch.bfloat16 else 0
+    if size:
+        req, start, indptr = chunk_pieces(rs, r.device, fn("pie_delta_piece_tokens")())
+        pieces = torch.empty(req.numel() * spec.heads * size, dtype=torch.uint8, device=r.device)
+        args.chunk_req, args.chunk_start, args.req_chunks, args.pieces, args.chunks = ptr(req), ptr(start), ptr(indptr), ptr(pieces), req.numel()
+        check(fn("pie_delta_chunked")(C.byref(args), stream_ptr()), "delta_chunked")
+        return out
     name = "delta_step" if decode else "delta_portions"
     check(fn("pie_" + name)(C.byref(args), _f32(r), stream_ptr()), name)
     return out

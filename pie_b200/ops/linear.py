@@ -52,19 +52,18 @@ def decay_logs(x, a2, bias, tau: float):
     return out
 
 
-def chunk_pieces(rs, device):
-    """Pieces of a fire's portions for the chunked form: (request, first row) of every piece and the pieces of every
-    request, as device tensors; kept with the fire's recurrent inputs."""
-    if rs.pieces is None:
-        size = fn("pie_linear_attn_chunk_tokens")()
+def chunk_pieces(rs, device, size: int):
+    """Pieces of `size` tokens of a fire's portions for a chunked form: (request, first row) of every piece and the pieces of
+    every request, as device tensors; kept with the fire's recurrent inputs."""
+    if size not in rs.pieces:
         qo = np.asarray(rs.qo_host, dtype=np.int64)
         per = -(-np.diff(qo) // size)
         req = np.repeat(np.arange(len(per)), per)
         indptr = np.concatenate([[0], np.cumsum(per)])
         start = qo[req] + (np.arange(len(req)) - indptr[req]) * size
         buf = torch.from_numpy(np.concatenate([req, start, indptr]).astype(np.int32)).to(device)
-        rs.pieces = buf.split([len(req), len(req), len(indptr)])
-    return rs.pieces
+        rs.pieces[size] = buf.split([len(req), len(req), len(indptr)])
+    return rs.pieces[size]
 
 
 def memory_gates(h, w, bias, spec, rs, state, decode: bool):
@@ -110,7 +109,7 @@ def linear_attention(q, k, v, spec, rs, state, decode: bool, log_decay=None, hea
     if decode or q.dtype == torch.float32 or not fn("pie_linear_attn_chunk_supported")(d):
         check(fn("pie_linear_attn_serial")(C.byref(a), _f32(q), stream_ptr()), "linear_attn_serial")
         return out if den is None else (out, den)
-    req, start, indptr = chunk_pieces(rs, q.device)
+    req, start, indptr = chunk_pieces(rs, q.device, fn("pie_linear_attn_chunk_tokens")())
     c = req.numel()
     u = torch.empty(c, h * d * (e + (den is not None)), dtype=torch.float32, device=q.device)
     dec = torch.empty(c, h, d, dtype=torch.float32, device=q.device)
