@@ -60,15 +60,15 @@ __global__ void __launch_bounds__(256) pool_rows_kernel(const PoolArgs a) {
     }
 }
 
-// One block per page of sixteen means; rows past a request's last are zeros, and so is the last page.
+// One block per page of sixteen means and head (keys, then values); rows past a request's last are zeros, and so is the last page.
 __global__ void __launch_bounds__(128) pool_gather_kernel(const PoolArgs a) {
-    const int p = blockIdx.x, r = p < a.total - 1 ? a.page_req[p] : -1, ch = a.D / 8;
+    const int p = blockIdx.x, head = blockIdx.y, r = p < a.total - 1 ? a.page_req[p] : -1, ch = a.D / 8;
     const int b0 = r >= 0 ? (p - a.first[r]) * 16 : 0, seen = r >= 0 ? a.seen[r] : 0;
     const int* pages = r >= 0 ? a.page_indices + a.kv_page_indptr[r] : nullptr;
     const bf16* means = static_cast<const bf16*>(a.means);
-    uint4* dst = static_cast<uint4*>(a.gathered) + (size_t)p * 2 * a.hkv * 16 * ch;
-    for (int i = threadIdx.x; i < 2 * a.hkv * 16 * ch; i += 128) {
-        const int head = i / (16 * ch), row = i / ch % 16, c = i % ch, b = b0 + row;
+    uint4* dst = static_cast<uint4*>(a.gathered) + ((size_t)p * 2 * a.hkv + head) * 16 * ch;
+    for (int i = threadIdx.x; i < 16 * ch; i += 128) {
+        const int row = i / ch, c = i % ch, b = b0 + row;
         uint4 v = make_uint4(0, 0, 0, 0);
         if (b < seen) {
             int page_at;
@@ -117,7 +117,7 @@ PIE_API int pie_pool_rows(const PoolArgs* args, int f32, cudaStream_t st) {
 PIE_API int pie_pool_gather(const PoolArgs* args, cudaStream_t st) {
     const PoolArgs& a = *args;
     if (a.total <= 0 || a.D % 8 || a.pool <= 0) return (int)cudaErrorInvalidValue;
-    pool_gather_kernel<<<a.total, 128, 0, st>>>(a);
+    pool_gather_kernel<<<dim3(a.total, 2 * a.hkv), 128, 0, st>>>(a);
     return (int)cudaGetLastError();
 }
 

@@ -684,9 +684,18 @@ __global__ void __launch_bounds__(256) la_bounded_decay_kernel(const bf16* __res
         const int c0 = (blockIdx.x * tiles + tile) * 64;
         if (c0 >= channels) break;
         __syncthreads();
-        for (int u = threadIdx.x; u < 64 * rp; u += 256) {
-            const int row = u / rp, k = u - row * rp;
-            sw[row * pitch + k] = c0 + row < channels && k < rank ? a2[(size_t)(c0 + row) * rank + k] : __float2bfloat16(0.f);
+        if (rank % 8 == 0) {                   // eight numbers at a time
+            for (int u = threadIdx.x; u < 8 * rp; u += 256) {
+                const int row = u / (rp / 8), k = (u - row * (rp / 8)) * 8;
+                uint4 w = make_uint4(0, 0, 0, 0);
+                if (c0 + row < channels && k < rank) w = *reinterpret_cast<const uint4*>(a2 + (size_t)(c0 + row) * rank + k);
+                *reinterpret_cast<uint4*>(sw + row * pitch + k) = w;
+            }
+        } else {
+            for (int u = threadIdx.x; u < 64 * rp; u += 256) {
+                const int row = u / rp, k = u - row * rp;
+                sw[row * pitch + k] = c0 + row < channels && k < rank ? a2[(size_t)(c0 + row) * rank + k] : __float2bfloat16(0.f);
+            }
         }
         __syncthreads();
         float acc[4][4];
@@ -712,7 +721,7 @@ __global__ void __launch_bounds__(256) la_bounded_decay_kernel(const bf16* __res
                 const int t = t0 + wt + g + (e >> 1) * 8;
                 if (t >= n) continue;
                 const float f = -1.4426950408889634f * factor;
-                const float y0 = __fdividef(f, 1.f + expf(-(acc[i][e] + b0))), y1 = __fdividef(f, 1.f + expf(-(acc[i][e + 1] + b1)));
+                const float y0 = __fdividef(f, 1.f + __expf(-(acc[i][e] + b0))), y1 = __fdividef(f, 1.f + __expf(-(acc[i][e + 1] + b1)));
                 float* dst = out + (size_t)t * channels + c;
                 if (c + 1 < channels && channels % 2 == 0) {
                     *reinterpret_cast<float2*>(dst) = make_float2(y0, y1);
