@@ -670,20 +670,9 @@ __global__ void __launch_bounds__(256) la_bounded_decay_kernel(const bf16* __res
     const int rp = bd_rank(rank), pitch = rp + 8;
     bf16 *hi = bd_smem, *lo = hi + 64 * pitch, *sw = lo + 64 * pitch;
     pdl_trigger();
-    pdl_wait();
     const int t0 = blockIdx.y * 64;
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, g = lane >> 2, q = lane & 3, wt = (warp & 3) * 16, wc = (warp >> 2) * 32;
-    for (int u = threadIdx.x; u < 64 * rp; u += 256) {
-        const int row = u / rp, k = u - row * rp;
-        const float f = t0 + row < n && k < rank ? tanhf(to_f(x[(size_t)(t0 + row) * ld + k])) : 0.f;
-        const bf16 h = __float2bfloat16(f);
-        hi[row * pitch + k] = h;
-        lo[row * pitch + k] = __float2bfloat16(f - __bfloat162float(h));
-    }
-    for (int tile = 0; tile < tiles; ++tile) {
-        const int c0 = (blockIdx.x * tiles + tile) * 64;
-        if (c0 >= channels) break;
-        __syncthreads();
+    auto weights = [&](int c0) {
         if (rank % 8 == 0) {                   // eight numbers at a time
             for (int u = threadIdx.x; u < 8 * rp; u += 256) {
                 const int row = u / (rp / 8), k = (u - row * (rp / 8)) * 8;
@@ -696,6 +685,23 @@ __global__ void __launch_bounds__(256) la_bounded_decay_kernel(const bf16* __res
                 const int row = u / rp, k = u - row * rp;
                 sw[row * pitch + k] = c0 + row < channels && k < rank ? a2[(size_t)(c0 + row) * rank + k] : __float2bfloat16(0.f);
             }
+        }
+    };
+    weights(blockIdx.x * tiles * 64);          // constants: before the kernel ahead is done
+    pdl_wait();
+    for (int u = threadIdx.x; u < 64 * rp; u += 256) {
+        const int row = u / rp, k = u - row * rp;
+        const float f = t0 + row < n && k < rank ? tanhf(to_f(x[(size_t)(t0 + row) * ld + k])) : 0.f;
+        const bf16 h = __float2bfloat16(f);
+        hi[row * pitch + k] = h;
+        lo[row * pitch + k] = __float2bfloat16(f - __bfloat162float(h));
+    }
+    for (int tile = 0; tile < tiles; ++tile) {
+        const int c0 = (blockIdx.x * tiles + tile) * 64;
+        if (c0 >= channels) break;
+        if (tile) {
+            __syncthreads();
+            weights(c0);
         }
         __syncthreads();
         float acc[4][4];

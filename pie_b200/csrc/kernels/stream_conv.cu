@@ -265,9 +265,24 @@ __global__ void __launch_bounds__(256) conv_norm_kernel(const ConvNormArgs a) {
     extern __shared__ float2 stats[];                   // [taps - 1 + rows_per_block]
     __shared__ float red[64];
     pdl_trigger();
+    // on their way to the L2 while the kernel ahead drains: what the norm and the convolution multiply with, then the history
+    auto ahead = [](const float* p, long n) {
+        for (long i = threadIdx.x * 32L; p && i < n; i += 256 * 32) asm volatile("prefetch.global.L2 [%0];" ::"l"(p + i));
+    };
+    ahead(a.y0_norm, a.width);
+    ahead(a.y1_norm, a.width);
+    ahead(a.w, a.width);
+    ahead(a.b, a.width);
+    ahead(a.conv, (long)a.taps * a.width);
     pdl_wait();
     const int back = a.conv ? a.taps - 1 : 0, t0 = blockIdx.x * a.rows_per_block, t1 = min(a.n, t0 + a.rows_per_block);
-    for (int t = back ? max(a.qo_indptr[a.tok_req[t0]], t0 - back) : t0; t < t1; ++t) {
+    int start = t0;
+    if (back) {
+        const int r = a.tok_req[t0], slot = a.slots[r];
+        start = max(a.qo_indptr[r], t0 - back);
+        if (slot >= 0) ahead(a.state + (size_t)slot * a.slot_stride, (long)back * a.width);
+    }
+    for (int t = start; t < t1; ++t) {
         const float2 s = row_stats<T, VEC, true>(a, t, red);
         if (threadIdx.x == 0) stats[t - t0 + back] = s;
     }

@@ -121,29 +121,33 @@ def plain_attention_mixer(m, h, lw: dict, li: int, fi, cache, st) -> None:
     a, n = m.cfg.blocks[li].mixer, h.shape[0]
     y = m._gemm(h, lw["w_in"])
     col = {k: y[:, c:c + w] for k, (c, w) in lw["columns"].items()}
-    z = attend_plain(m, col, "", a, lw, li, fi, cache).view(n, -1)
-    if z.shape[1] != lw["w_out"].shape[1] or (a.group, a.vdim) != (a.group_pad, a.head_dim):       # padded heads: side by side
-        o, z = z, torch.empty(n, lw["w_out"].shape[1], dtype=h.dtype, device=h.device)
-        lin.gated_norm([(o, None, None, z, dict(norm_cols=0, scale=1.0, spec=a, cols=a.heads * a.vdim))])
-    st.add_product(z, lw["w_out"])
+    st.add_product(side_by_side(attend_plain(m, col, "", a, lw, li, fi, cache).view(n, -1), a, lw["w_out"]), lw["w_out"])
+
+
+def side_by_side(o, a: PlainAttentionSpec, w):
+    """The heads of padded rows next to each other, as the product with `w` reads them."""
+    if o.shape[1] == w.shape[1] and (a.group, a.vdim) == (a.group_pad, a.head_dim):
+        return o
+    z = torch.empty(o.shape[0], w.shape[1], dtype=o.dtype, device=o.device)
+    lin.gated_norm([(o, None, None, z, dict(norm_cols=0, scale=1.0, spec=a, cols=a.heads * a.vdim))])
+    return z
 
 
 def delta_mixer(m, h, lw: dict, li: int, fi, cache, st) -> None:
-    """Attention and a delta rule side by side, each output normed on its own."""
+    """Attention and a delta rule side by side, each output normed on its own. On the device the delta rule runs on a stream of
+    its own beside the attention."""
     s, n, eps = m.cfg.blocks[li].mixer, h.shape[0], m.cfg.rms_norm_eps
     a, r = s.left, s.right
     y = m._gemm(h, lw["w_in"])
     col = {k: y[:, c:c + w] for k, (c, w) in lw["columns"].items()}
-    logs = delta.bounded_decay_logs(col["right.w1"], lw["w2"], lw["w0"], r.bound)
-    o = delta.delta_rule(col["right.r"], col["right.k"], col["right.v"], col["right.a"], lw["a_bias"], logs, r, fi.rs,
-                         fi.rs.state_of(li, r.state_elems), fi.is_decode)
-    zr = torch.empty(n, lw["w_right"].shape[1], dtype=h.dtype, device=h.device)
-    parts = [(o, lw["o_norm"], col["right.g"], zr, dict(act="sigmoid", norm_cols=r.dim, eps=eps, scale=1.0))]
-    zl = attend_plain(m, col, "left.", a, lw, li, fi, cache).view(n, -1)
-    if zl.shape[1] != lw["w_left"].shape[1] or (a.group, a.vdim) != (a.group_pad, a.head_dim):
-        left, zl = zl, torch.empty(n, lw["w_left"].shape[1], dtype=h.dtype, device=h.device)
-        parts.append((left, None, None, zl, dict(norm_cols=0, scale=1.0, spec=a, cols=a.heads * a.vdim)))
-    lin.gated_norm(parts)
+    with m.beside() as joined:
+        logs = delta.bounded_decay_logs(col["right.w1"], lw["w2"], lw["w0"], r.bound)
+        o = delta.delta_rule(col["right.r"], col["right.k"], col["right.v"], col["right.a"], lw["a_bias"], logs, r, fi.rs,
+                             fi.rs.state_of(li, r.state_elems), fi.is_decode)
+        zr = torch.empty(n, lw["w_right"].shape[1], dtype=h.dtype, device=h.device)
+        lin.gated_norm([(o, lw["o_norm"], col["right.g"], zr, dict(act="sigmoid", norm_cols=r.dim, eps=eps, scale=1.0))])
+    zl = side_by_side(attend_plain(m, col, "left.", a, lw, li, fi, cache).view(n, -1), a, lw["w_left"])
+    joined()
     st.pair = ((m._gemm(zl, lw["w_left"]), lw["left_gain"]), (m._gemm(zr, lw["w_right"]), lw["right_gain"]))
 
 

@@ -14,6 +14,7 @@ of the context (positions only feed RoPE), as in driver/cuda/src/kernels/kv_page
 from __future__ import annotations
 
 import math
+from contextlib import contextmanager
 from dataclasses import dataclass
 from typing import Optional
 
@@ -67,6 +68,7 @@ class Transformer:
         self.vocab_local = weights["lm_head"].shape[0] * (self.par.tp_size if self.par.comm is not None else 1)
         # fp8 KV pages: per-(token, head) scales [layers, pages, 2, hkv, page] set by the driver, else None
         self.kv_scale = None
+        self._second = None             # stream of `beside`
         if cfg.latent is not None:
             latent.prepare_latent(self)
         elif cfg.blocks is not None:
@@ -83,6 +85,22 @@ class Transformer:
         if self.cfg.stream32:
             return 256
         return ops.prefill_tile_rows(self.hq, self.hkv, self.cfg.head_dim, page_size, softcap=bool(self.cfg.attn_softcap))
+
+    @contextmanager
+    def beside(self):
+        """Run the body on a second stream, after everything launched so far; yields a function that makes the current stream
+        wait for it. What the body allocates may be used until the next such body. No matrix products: they share a
+        workspace. On the CPU the body simply runs."""
+        if self.device.type != "cuda":
+            yield lambda: None
+            return
+        if self._second is None:
+            self._second = torch.cuda.Stream(self.device)
+        here, done = torch.cuda.current_stream(self.device), torch.cuda.Event()
+        self._second.wait_stream(here)
+        with torch.cuda.stream(self._second):
+            yield lambda: here.wait_event(done)
+            done.record(self._second)
 
     # ------------------------------------------------------------------ linear algebra
     def _gemm(self, x, w, residual=None, swiglu=False, glu: str = ""):
