@@ -198,9 +198,11 @@ __device__ __forceinline__ void load_q_frags(uint32_t q_smem, int row0, uint32_t
 constexpr int DEC_WARPS = 4;
 constexpr int DEC_STAGES = 3;
 
-template <int D>
+constexpr int DEC_OWN_STAGES = 4;      // of one tile each, see OWN below
+
+template <int D, bool OWN = false>
 constexpr int decode_smem_bytes() {
-    return 16 * D * 2 + DEC_WARPS * DEC_STAGES * 2 * 16 * D * 2;
+    return 16 * D * 2 + DEC_WARPS * (OWN ? DEC_OWN_STAGES : 2 * DEC_STAGES) * 16 * D * 2;
 }
 
 // CASCADE: shared-prefix items. A work item may then cover a KV range that up to 16 / G requests
@@ -237,9 +239,9 @@ __device__ __forceinline__ int mean_row(int b, int pool, int page_size, int& pag
 
 // POOL: an item of a request takes its share of the 16-key tiles (means, then the window's tokens) whatever range the plan
 // gave it, so that any plan spreads the work evenly.
-// OWN: the values are the keys (planes 1); a stage then holds one tile, and there are twice as many.
+// OWN: the values are the keys (planes 1); a stage then holds one tile, which leaves room for a third block per SM.
 template <int D, int G, bool CASCADE, int MODE = MODE_PLAIN, bool POOL = false, bool OWN = false>
-__global__ void __launch_bounds__(DEC_WARPS * 32)
+__global__ void __launch_bounds__(DEC_WARPS * 32, OWN && D <= 128 ? 3 : 1)
 paged_decode_attn_kernel(const bf16* __restrict__ q, const bf16* __restrict__ kv_layer,
                          const int* __restrict__ page_indices,
                          const int* __restrict__ kv_page_indptr, const int* __restrict__ item_req,
@@ -257,10 +259,10 @@ paged_decode_attn_kernel(const bf16* __restrict__ q, const bf16* __restrict__ kv
     extern __shared__ __align__(1024) uint8_t smem[];
     constexpr int CH = D / 8;              // 16-byte chunks per row
     constexpr int TILE_BYTES = 16 * D * 2; // one 16-token K or V tile
-    constexpr int STAGES = OWN ? 2 * DEC_STAGES : DEC_STAGES, STAGE_BYTES = (OWN ? 1 : 2) * TILE_BYTES;
+    constexpr int STAGES = OWN ? DEC_OWN_STAGES : DEC_STAGES, STAGE_BYTES = (OWN ? 1 : 2) * TILE_BYTES;
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     const uint32_t q_smem = smem_u32(smem);
-    const uint32_t warp_smem = q_smem + TILE_BYTES + warp * DEC_STAGES * 2 * TILE_BYTES;
+    const uint32_t warp_smem = q_smem + TILE_BYTES + warp * STAGES * STAGE_BYTES;
     pdl_trigger();
     pdl_wait();
     // The work count lives in device memory (graph replays refresh it): never trust it past the

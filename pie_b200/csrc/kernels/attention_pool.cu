@@ -129,12 +129,13 @@ PIE_API int pie_laid_decode(const LaidAttnArgs* args, cudaStream_t st) {
     float* lse = a.scratch + (size_t)a.max_items * a.hq * a.D;
     const KeyLayout kl{a.planes, a.pool, a.per_page, (const bf16*)a.means, nullptr};
     DISPATCH_DG(a.D, group, {
-        constexpr int SM = decode_smem_bytes<D>();
+        const int SM = a.planes == 1 ? decode_smem_bytes<D, true>() : decode_smem_bytes<D>();
+        const int ctas = a.planes == 1 && D <= 128 ? a.num_ctas * 3 / 2 : a.num_ctas;
         auto kern = a.pool ? paged_decode_attn_kernel<D, G, false, MODE_PLAIN, true>
                   : a.planes == 1 ? paged_decode_attn_kernel<D, G, false, MODE_PLAIN, false, true> : paged_decode_attn_kernel<D, G, false>;
         cudaError_t e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, SM);
         if (e == cudaSuccess)
-            e = launch_pdl(kern, dim3(a.num_ctas), dim3(DEC_WARPS * 32), SM, st, (const bf16*)a.q, (const bf16*)a.kv, a.page_indices,
+            e = launch_pdl(kern, dim3(ctas), dim3(DEC_WARPS * 32), SM, st, (const bf16*)a.q, (const bf16*)a.kv, a.page_indices,
                            a.kv_page_indptr, a.item_req, a.item_start, a.item_end, a.req_item_indptr, a.num_items, (bf16*)a.out, a.scratch,
                            lse, a.hq, a.hkv, a.page_size, a.scale * 1.4426950408889634f, a.window_left, a.sinks_log2, a.max_items,
                            a.num_reqs, pie_status_word_current(), (const int*)nullptr, (const int*)nullptr, (const int*)nullptr, 0.f,

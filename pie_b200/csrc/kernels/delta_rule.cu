@@ -617,7 +617,8 @@ PIE_API int pie_delta_step(const DeltaArgs* args, int f32, cudaStream_t st) {
 
 // Bytes of one piece of one head in the chunked form; 0: no such form for this head size.
 PIE_API int pie_delta_piece_bytes(int dim) {
-    return dim <= 0 || dim > 128 ? 0 : dim <= 32 ? (int)sizeof(DeltaPiece<32>) : dim <= 64 ? (int)sizeof(DeltaPiece<64>) : (int)sizeof(DeltaPiece<128>);
+    if (dim <= 0 || dim > 128) return 0;
+    return dim <= 32 ? (int)sizeof(DeltaPiece<32>) : dim <= 64 ? (int)sizeof(DeltaPiece<64>) : (int)sizeof(DeltaPiece<128>);
 }
 PIE_API int pie_delta_piece_tokens() { return DC_T; }
 

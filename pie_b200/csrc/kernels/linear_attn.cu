@@ -709,8 +709,9 @@ __global__ void __launch_bounds__(256) la_bounded_decay_kernel(const bf16* __res
         for (int i = 0; i < 4; ++i) acc[i][0] = acc[i][1] = acc[i][2] = acc[i][3] = 0.f;
         for (int ks = 0; ks < rp; ks += 16) {
             auto word = [&](const bf16* m, int row, int col) { return *reinterpret_cast<const uint32_t*>(m + row * pitch + ks + col); };
-            const uint32_t ah[4] = {word(hi, wt + g, 2 * q), word(hi, wt + g + 8, 2 * q), word(hi, wt + g, 2 * q + 8), word(hi, wt + g + 8, 2 * q + 8)};
-            const uint32_t al[4] = {word(lo, wt + g, 2 * q), word(lo, wt + g + 8, 2 * q), word(lo, wt + g, 2 * q + 8), word(lo, wt + g + 8, 2 * q + 8)};
+            const int r0 = wt + g, r1 = r0 + 8, k0 = 2 * q, k1 = k0 + 8;
+            const uint32_t ah[4] = {word(hi, r0, k0), word(hi, r1, k0), word(hi, r0, k1), word(hi, r1, k1)};
+            const uint32_t al[4] = {word(lo, r0, k0), word(lo, r1, k0), word(lo, r0, k1), word(lo, r1, k1)};
 #pragma unroll
             for (int i = 0; i < 4; ++i) {
                 const uint32_t b0 = word(sw, wc + i * 8 + g, 2 * q), b1 = word(sw, wc + i * 8 + g, 2 * q + 8);

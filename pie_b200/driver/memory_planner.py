@@ -70,12 +70,14 @@ def arena_bytes(cfg: ModelConfig, max_tokens: int, max_requests: int, tp: int = 
 
 def _block_bytes(b) -> int:
     """Activation bytes per token of one layer described on its own: projections, 32-bit mixer outputs, the states between the
-    64-token pieces of a prompt (a delta rule: four vectors per token of its 16-token pieces), latent queries with the keys and values of every head, feed-forward (an expert's segment may
-    be padded by 128 rows: the experts' weights dwarf it)."""
+    64-token pieces of a prompt (a delta rule: decays, and five vectors' worth per token of its 16-token pieces), latent queries
+    with the keys and values of every head, feed-forward (an expert's segment may be padded by 128 rows: the experts' weights
+    dwarf it)."""
     r, a, s, f = b.recurrent, b.attention, b.latent, b.ff
     bytes_ = 0
     if r is not None:
-        bytes_ += 2 * (2 * r.qk + 2 * r.values) + 4 * (r.qk + 2 * r.values) + (5 * 4 * r.qk + 4 * r.qk if isinstance(r, DeltaRuleSpec) else 4 * r.state_elems // 64)
+        bytes_ += 2 * (2 * r.qk + 2 * r.values) + 4 * (r.qk + 2 * r.values)
+        bytes_ += 4 * 6 * r.qk if isinstance(r, DeltaRuleSpec) else 4 * r.state_elems // 64
     if a is not None:
         bytes_ += 2 * (a.heads * (a.dim + 2 * a.vdim) + a.kv_heads * (a.dim + a.vdim) + 2 * a.kv_heads * a.group_pad * a.head_dim)
     if s is not None:

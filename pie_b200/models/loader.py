@@ -379,8 +379,9 @@ def complete_blocks(cfg: ModelConfig, reader) -> None:
 def _compile_blocks(cfg: ModelConfig, names: set, tp_size: int, dtype: str) -> Program:
     """Layout plan of layers described one by one (Retodra, Nukelix and Vulanex names). Fused per layer: every projection that reads
     the mixer's input (`w_in`, each part on a multiple of 8 rows: `block_spec.projection_columns`), the output projections of
-    two mixers side by side along K (`w_out`; apart where each is normed on its own: `w_left`, `w_right`), gate and up interleaved. Gates of a matrix memory stay apart (`w_gates`): they
-    are wanted in 32-bit. Dimensions a GEMM sees are padded with zeros, those of a gated feed-forward to 16."""
+    two mixers side by side along K (`w_out`; apart where each is normed on its own: `w_left`, `w_right`), gate and up
+    interleaved. Gates of a matrix memory stay apart (`w_gates`): they are wanted in 32-bit. Dimensions a GEMM sees are padded
+    with zeros, those of a gated feed-forward to 16."""
     if tp_size > 1:
         raise NotImplementedError("layers described one by one under tensor parallelism")
     W = cfg.hidden_size

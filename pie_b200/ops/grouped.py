@@ -1,7 +1,8 @@
 """Ops of grouped-query attention with biased projections, norms over all heads together, rotation in part, mixed values, a
 window beside kept first tokens, and a softmax sink; of attention whose heads are normed one by one, whose values may be the
 keys, and whose window may stand beside means of the blocks ahead of it. CUDA tensors go to
-`csrc/kernels/attention_{gqa,pool}.cu` and the paged attention kernels (bf16 when serving, float32 on the 32-bit path), CPU tensors to the plain statements at the end.
+`csrc/kernels/attention_{gqa,pool}.cu` and the paged attention kernels (bf16 when serving, float32 on the 32-bit path), CPU
+tensors to the plain statements at the end.
 """
 from __future__ import annotations
 
@@ -23,7 +24,8 @@ GqaRowsArgs = _struct("GqaRowsArgs", ("q k v q_b k_b v_b q_norm k_norm positions
 HeadRowsArgs = _struct("HeadRowsArgs", ("q k v q_norm k_norm positions slots inv_freq q_out cache", p),
                        ("n ld heads kv_heads group group_pad dim vdim D page_size rot_dims temp_every", i32),
                        ("eps rot_factor temp_coef", f32))
-GqaAnyArgs = _struct("GqaAnyArgs", ("q kv out sink_scores means page_indices kv_page_indptr kv_lens qo_indptr tok_req slots mask_bits mask_word_indptr", p),
+GqaAnyArgs = _struct("GqaAnyArgs", ("q kv out sink_scores means page_indices kv_page_indptr kv_lens qo_indptr tok_req slots mask_bits "
+                                    "mask_word_indptr", p),
                      ("n hq hkv D page_size window_left keep_first sink planes pool per_page", i32), ("scale", f32))
 # mirrors of the argument structs in csrc/kernels/attention_pool.cu
 PoolArgs = _struct("PoolArgs", ("cache means page_indices kv_page_indptr kv_lens qo_indptr tok_req slots gathered first seen page_req", p),
@@ -152,8 +154,8 @@ def laid_attention(q, cache, means, plan, rs, slots, spec, sinks=None):
     per_page = means.shape[3] if means is not None else 0
     masked = getattr(plan, "mask_bits", None) is not None
     if q.dtype == torch.float32 or not fn("pie_gqa_mma_supported")(spec.group_pad, D, page) or (masked and spec.pool):
-        _attend_any(q, cache, plan, rs, slots, spec, page, out, window_left=window, planes=planes, sink_scores=ptr(sinks[0] if sinks is not None else None), means=ptr(means),
-                    pool=spec.pool, per_page=per_page)
+        _attend_any(q, cache, plan, rs, slots, spec, page, out, window_left=window, planes=planes, means=ptr(means), pool=spec.pool,
+                    per_page=per_page, sink_scores=ptr(sinks[0] if sinks is not None else None))
         return out
     a = LaidAttnArgs(q=ptr(q), kv=ptr(cache), out=ptr(out), page_indices=ptr(plan.page_indices), kv_page_indptr=ptr(plan.kv_page_indptr),
                      kv_lens=ptr(plan.kv_lens), n=n, hq=hq, hkv=spec.kv_heads, D=D, page_size=page, window_left=window, planes=planes,

@@ -446,7 +446,8 @@ def test_delta_rule_over_a_ragged_batch(path, h, d):
     spec, slots = DeltaRuleSpec(h, d, 4), [3, 0, 5, 1, 2, -1]
     start = rnd(6, spec.state_elems, seed=9)
     state = start.clone().to(dev)
-    got = delta.delta_rule(*padded([r, k, v, a], dev, dt), b.to(dev), (decay / math.log(2)).to(dev), spec, recurrent(qo, slots, reset, dev), state, False)
+    got = delta.delta_rule(*padded([r, k, v, a], dev, dt), b.to(dev), (decay / math.log(2)).to(dev), spec, recurrent(qo, slots, reset, dev),
+                           state, False)
     for i, (p, e) in enumerate(zip(qo[:-2], qo[1:-1])):
         heads = lambda y: y[p:e].double().view(e - p, h, d)
         old = None if reset[i] else start[slots[i]].double().view(h, d, d)
