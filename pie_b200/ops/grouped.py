@@ -141,8 +141,8 @@ def _gathered_means(cache, means, plan, spec):
 def laid_attention(q, cache, means, plan, rs, slots, spec, sinks=None):
     """Softmax over the visible keys of q [N, kv * group_pad, D] in pages as `PlainAttentionSpec` lays them out: keys that are
     their own values, a window beside the `means` of the blocks ahead of it (None: none), a learned sink score per padded
-    head (`sinks`: 32-bit, as natural and as base-2 logarithms). Under a custom mask a mean counts if the mask shows all its tokens. Same
-    shape out."""
+    head (`sinks`: 32-bit, as natural and as base-2 logarithms). Under a custom mask a mean counts if the mask shows all its
+    tokens. Same shape out."""
     if not q.is_cuda:
         return _laid_attention(q, cache, means, plan, spec, sinks[0] if sinks is not None else None)
     from ..models.block_spec import EVERYTHING
